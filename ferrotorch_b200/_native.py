@@ -31,6 +31,9 @@ _PKG = Path(__file__).resolve().parent
 CSRC = _PKG / "csrc"
 OUT = _PKG / "_C"
 KERNELS_SO = OUT / "libft_kernels.so"
+# Programs that only serve decoders (bin/trace_run) need a part of the sources: with FT_KERNEL_SET=decoder a checkout
+# without a built library compiles these alone.  A library that is already complete is used as it is.
+KERNEL_SETS = {"decoder": ("ft_host", "gemm_tcgen05", "norm_act", "paged_attn", "paged_prefill")}
 HOST_SO = OUT / "libft_host.so"
 
 NVCC_FLAGS = [
@@ -61,19 +64,26 @@ def _run(cmd: list[str]) -> None:
         raise RuntimeError("build failed: %s\n%s\n%s" % (" ".join(cmd), proc.stdout, proc.stderr))
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> Path:
-    """Compile ``csrc/*.cu`` into ``_C/libft_kernels.so`` (no-op when up to date)."""
+def build_kernels(force: bool = False, verbose: bool = False, kernel_set: str | None = None) -> Path:
+    """Compile ``csrc/*.cu`` into ``_C/libft_kernels.so`` (no-op when up to date), or the sources of a
+    ``kernel_set`` into ``_C/libft_<set>.so`` when the complete library is not up to date."""
     srcs = sorted(CSRC.glob("*.cu"))
-    deps = srcs + sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    if not force and KERNELS_SO.exists() and KERNELS_SO.stat().st_mtime >= _newest(deps):
+    headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+    if not force and KERNELS_SO.exists() and KERNELS_SO.stat().st_mtime >= _newest(srcs + headers):
         return KERNELS_SO
+    target = KERNELS_SO
+    if kernel_set is not None:
+        srcs = [s for s in srcs if s.stem in KERNEL_SETS[kernel_set]]
+        target = OUT / ("libft_%s.so" % kernel_set)
+        if not force and target.exists() and target.stat().st_mtime >= _newest(srcs + headers):
+            return target
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found; cannot build libft_kernels.so")
     OUT.mkdir(exist_ok=True)
     objdir = OUT / "obj"
     objdir.mkdir(exist_ok=True)
-    hdr_m = _newest(sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h")))
+    hdr_m = _newest(headers)
 
     def compile_one(src: Path) -> Path:
         obj = objdir / (src.stem + ".o")
@@ -86,10 +96,10 @@ def build_kernels(force: bool = False, verbose: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:
         objs = list(ex.map(compile_one, srcs))
-    tmp = KERNELS_SO.with_suffix(".so.tmp%d" % os.getpid())
+    tmp = target.with_suffix(".so.tmp%d" % os.getpid())
     _run([nvcc, "-shared", "-o", str(tmp), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a"])
-    os.replace(tmp, KERNELS_SO)
-    return KERNELS_SO
+    os.replace(tmp, target)
+    return target
 
 
 def build_host(force: bool = False) -> Path:
@@ -167,11 +177,12 @@ def kernels(required: bool = True) -> ctypes.CDLL | None:
         if _kernels is not None:
             return _kernels
         try:
+            so = KERNELS_SO
             if os.environ.get("FT_NO_AUTOBUILD") != "1" and _nvcc() is not None:
-                build_kernels()
-            if not KERNELS_SO.exists():
-                raise RuntimeError("%s does not exist (run `python -c 'import __graft_entry__ as g; g.build()'`)" % KERNELS_SO)
-            lib = ctypes.CDLL(str(KERNELS_SO), mode=ctypes.RTLD_GLOBAL)
+                so = build_kernels(kernel_set=os.environ.get("FT_KERNEL_SET") or None)
+            if not so.exists():
+                raise RuntimeError("%s does not exist (run `python -c 'import __graft_entry__ as g; g.build()'`)" % so)
+            lib = ctypes.CDLL(str(so), mode=ctypes.RTLD_GLOBAL)
             _bind(lib, _KERNEL_PROTOS)
             _kernels = lib
         except Exception:

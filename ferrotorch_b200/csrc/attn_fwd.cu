@@ -19,13 +19,11 @@
 //              max/sum need no shuffles; P goes back through shared memory (128B swizzle)
 //              as the A operand of the second MMA; O is rescaled in TMEM when a row max moves
 // All waits are bounded and report through the device status word.
+#include "attn_row.cuh"
 #include "ft_host.h"
-#include "ft_ptx.cuh"
 
 namespace ft {
 
-constexpr int ATT_BM = 128;
-constexpr int ATT_BN = 128;
 constexpr int ATT_THREADS = 256;
 constexpr int ATT_KV_STAGES = 2;
 
@@ -339,7 +337,6 @@ static int launch_fwd(const CUtensorMap& tq, const CUtensorMap& tk, const CUtens
 // than 8 (a factor 256, harmless in fp32 / bf16), so after the first blocks the softmax groups
 // do not touch O at all.
 constexpr int ATT2_THREADS = 384;
-constexpr float ATT2_RESCALE_THRESHOLD = 8.f;
 
 template <int HD>
 struct Att2Cfg {
@@ -353,31 +350,6 @@ struct Att2Cfg {
   static constexpr int S_COL = 0;       // S_i at S_COL + i * 128; P_i aliases its first 64 columns
   static constexpr int O_COL = 256;     // O_i at O_COL + i * 128
 };
-
-// p = 2^(s * scale + neg_m) for one row of 128 scores held as packed pairs; writes the bf16 pairs
-// and returns the row sum (four independent partial sums of pairs).  Moving a share of the
-// exponentials from the special-function unit to a polynomial on the FMA pipe was measured at
-// 0 / 25 / 37 / 50 / 62 %: 908 / 904 / 902 / 880 / 811 TFLOP/s at B4 S4096 H32/8 D128, so all of
-// them stay on ex2.approx.
-__device__ __forceinline__ float att2_exp_row(const f32x2 (&sp)[ATT_BN / 2], float scale, float neg_m,
-                                              uint32_t (&pk)[ATT_BN / 2]) {
-  const f32x2 sc2 = f2_pack(scale, scale), nm2 = f2_pack(neg_m, neg_m);
-  f32x2 acc[4];
-#pragma unroll
-  for (int k = 0; k < 4; ++k) acc[k] = f2_pack(0.f, 0.f);
-#pragma unroll
-  for (int i = 0; i < ATT_BN / 2; ++i) {
-    float x0, x1;
-    f2_unpack(f2_fma(sp[i], sc2, nm2), x0, x1);
-    const float e0 = fast_exp2(x0), e1 = fast_exp2(x1);
-    acc[i & 3] = f2_add(acc[i & 3], f2_pack(e0, e1));
-    pk[i] = pack_bf16x2(e0, e1);
-  }
-  float a, b, c, d;
-  f2_unpack(f2_add(acc[0], acc[1]), a, b);
-  f2_unpack(f2_add(acc[2], acc[3]), c, d);
-  return (a + b) + (c + d);
-}
 
 template <int HD>
 __global__ void __launch_bounds__(ATT2_THREADS, 1)
@@ -562,50 +534,10 @@ flash_fwd2_tcgen05_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       tc_fence_after();
       // the row as 64 packed pairs: every later step works on two keys per instruction
       f32x2 sp[ATT_BN / 2];
-      {
-        uint32_t t0[32], t1[32], t2[32], t3[32];
-        tmem_ld_32x32(s_addr, t0);
-        tmem_ld_32x32(s_addr + 32, t1);
-        tmem_ld_32x32(s_addr + 64, t2);
-        tmem_ld_32x32(s_addr + 96, t3);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          sp[i] = f2_pack(__uint_as_float(t0[2 * i]), __uint_as_float(t0[2 * i + 1]));
-          sp[16 + i] = f2_pack(__uint_as_float(t1[2 * i]), __uint_as_float(t1[2 * i + 1]));
-          sp[32 + i] = f2_pack(__uint_as_float(t2[2 * i]), __uint_as_float(t2[2 * i + 1]));
-          sp[48 + i] = f2_pack(__uint_as_float(t3[2 * i]), __uint_as_float(t3[2 * i + 1]));
-        }
-      }
+      att2_load_row(s_addr, sp);
       const int kv0 = j * ATT_BN;
-      const bool masked = kv0 + ATT_BN - 1 > warp_limit;   // warp-uniform
-      if (masked) {
-#pragma unroll
-        for (int i = 0; i < ATT_BN / 2; ++i) {
-          float a, b;
-          f2_unpack(sp[i], a, b);
-          if (kv0 + 2 * i > limit) a = -INFINITY;
-          if (kv0 + 2 * i + 1 > limit) b = -INFINITY;
-          sp[i] = f2_pack(a, b);
-        }
-      }
-      float mx;
-      {
-        float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;   // four independent chains
-#pragma unroll
-        for (int i = 0; i < ATT_BN / 2; i += 4) {
-          float a, b;
-          f2_unpack(sp[i], a, b);
-          m0 = max3(m0, a, b);
-          f2_unpack(sp[i + 1], a, b);
-          m1 = max3(m1, a, b);
-          f2_unpack(sp[i + 2], a, b);
-          m2 = max3(m2, a, b);
-          f2_unpack(sp[i + 3], a, b);
-          m3 = max3(m3, a, b);
-        }
-        mx = fmaxf(max3(m0, m1, m2), m3);
-      }
+      if (kv0 + ATT_BN - 1 > warp_limit) att2_mask_row(sp, kv0, limit);   // warp-uniform branch
+      float mx = att2_row_max(sp);
       mx *= p.scale_log2;  // scale > 0, so the maximum commutes with it
       // lazy reference maximum
       float alpha = 1.f;

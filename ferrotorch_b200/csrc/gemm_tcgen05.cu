@@ -1137,6 +1137,39 @@ __global__ void small_m_finalize_kernel(const float* __restrict__ ws, __nv_bfloa
   }
 }
 
+// The same sum for an fp32 result: C[m, n] (+)= sum_ks ws[ks][n, m], with the next layer's dynamic tanh
+// applied to the new value on its way out: dyt_out = (tanh(alpha C) w + b) as bf16.  Being element by
+// element, that norm needs no pass of its own over the residual stream.
+__global__ void small_m_finalize_f32_kernel(const float* __restrict__ ws, float* __restrict__ C, int accumulate,
+                                            const float* __restrict__ alpha_p, const float* __restrict__ w,
+                                            const float* __restrict__ b, __nv_bfloat16* __restrict__ dyt_out, float dyt_scale,
+                                            int M, int N, int ld_ws, int ksplit, int slice_rows, long long ldc, long long ldd) {
+  __shared__ float tile[32][33];
+  const int n0 = blockIdx.x * 32, m0 = blockIdx.y * 32;
+  const long long slice = static_cast<long long>(slice_rows) * ld_ws;
+  for (int i = threadIdx.y; i < 32; i += 8) {
+    const int n = n0 + i, m = m0 + threadIdx.x;
+    float v = 0.f;
+    if (n < N && m < M) {
+      const float* src = ws + static_cast<long long>(n) * ld_ws + m;
+      for (int ks = 0; ks < ksplit; ++ks) v += src[ks * slice];
+    }
+    tile[i][threadIdx.x] = v;
+  }
+  __syncthreads();
+  const float alpha = dyt_out ? *alpha_p : 0.f;
+  for (int i = threadIdx.y; i < 32; i += 8) {
+    const int m = m0 + i, n = n0 + threadIdx.x;
+    if (m < M && n < N) {
+      float v = tile[threadIdx.x][i];
+      float* c = C + static_cast<long long>(m) * ldc + n;
+      if (accumulate) v += *c;
+      *c = v;
+      if (dyt_out) dyt_out[static_cast<long long>(m) * ldd + n] = __float2bfloat16((tanhf(alpha * v) * w[n] + b[n]) * dyt_scale);
+    }
+  }
+}
+
 }  // namespace ft
 
 constexpr int SMALL_M_MAX_SPLIT = 16;
@@ -1146,6 +1179,63 @@ FT_API long long ft_gemm_small_m_workspace(int M, int N) {
   const int mpad = M <= 64 ? 64 : 128;
   return static_cast<long long>((N + 255) / 256 * 256) * mpad * SMALL_M_MAX_SPLIT;
 }
+
+namespace ft {
+
+// How many pieces the contraction of a small-batch GEMM is cut into (>= min_split).
+static int small_m_pick_split(int N, int K, int ksplit, int min_split, int device) {
+  const int pairs = sm_count(device) / 2;
+  const int tiles = (N + 255) / 256;
+  const int k_blocks = (K + GEMM_BK - 1) / GEMM_BK;
+  if (ksplit <= 0) {
+    ksplit = 1;
+    if (tiles < pairs) {
+      // one wave: as many pieces per tile as there are CTA pairs to take them, each piece long
+      // enough (>= 4 k-blocks) to be worth a pipeline fill
+      ksplit = pairs / tiles;
+      const int max_split = k_blocks / 4 > 0 ? k_blocks / 4 : 1;
+      if (ksplit > max_split) ksplit = max_split;
+      if (ksplit < 1) ksplit = 1;
+    }
+  }
+  if (ksplit < min_split) ksplit = min_split;
+  if (ksplit > k_blocks) ksplit = k_blocks;
+  return ksplit > SMALL_M_MAX_SPLIT ? SMALL_M_MAX_SPLIT : ksplit;
+}
+
+// Launch the split contraction of a small-batch GEMM into `workspace` (slices of ceil(N / 256) * 256 rows
+// x 64 or 128 columns); *ksplit returns the number of slices.
+static int small_m_split(const void* X, const void* W, float* workspace, int M, int N, int K, long long ldx, long long ldw,
+                         int* ksplit, int min_split, int device, cudaStream_t stream) {
+  const int bn = M <= 64 ? 64 : 128;
+  const int k_blocks = (K + GEMM_BK - 1) / GEMM_BK;
+  const int pieces = small_m_pick_split(N, K, *ksplit, min_split, device);
+  GemmParams p;
+  p.bias = nullptr; p.M = N; p.N = M; p.K = K;   // tile space: rows of W x batch
+  p.status = device_status_word(device);
+  p.taps = 1; p.cblocks = 0;
+  for (int t = 0; t < GEMM_MAX_TAPS; ++t) p.shift[t] = 0;
+  p.gHp = p.gWp = p.cHo = p.cWo = p.c_oh = p.c_ow = 0;
+  const int per = (k_blocks + pieces - 1) / pieces;
+  p.ksplit = *ksplit = (k_blocks + per - 1) / per;
+  p.C = workspace; p.ldc = bn;
+  p.flags = GEMM_OUT_F32;
+  // a slice is a whole number of 256-row tiles, so a tile that hangs over the end of W stays
+  // inside its own slice
+  p.split_rows = (N + 255) / 256 * 256;
+  CUtensorMap tmA, tmB, tmC;
+  int rc = make_tmap_2d(&tmA, W, 2, K, N, ldw * 2, GEMM_BK, GEMM_BM, 3);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tmB, X, 2, K, M, ldx * 2, GEMM_BK, bn / 2, 3);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tmC, workspace, 4, bn, static_cast<uint64_t>(p.ksplit) * p.split_rows,
+                    static_cast<uint64_t>(bn) * 4, 32, 32, 3);
+  if (rc) return rc;
+  return bn == 64 ? launch_pair<64, false, false, 2>(tmA, tmB, tmC, p, device, 0, stream)
+                  : launch_pair<128, false, false, 2>(tmA, tmB, tmC, p, device, 0, stream);
+}
+
+}  // namespace ft
 
 // C[M, N] = X[M, K] W[N, K]^T (+ bias[N]) (+ residual[M, N]) for a small batch M <= 128 (decode):
 // the weight is the 128-row MMA operand, so every byte of W crosses the tensor core once with all
@@ -1167,64 +1257,64 @@ FT_API int ft_gemm_small_m(const void* X, const void* W, void* C, const void* bi
   FT_REQUIRE(!(flags & (GEMM_OUT_F32 | GEMM_ACCUMULATE)), "ft_gemm_small_m: bf16 output, no accumulation");
   FT_REQUIRE(!(flags & (GEMM_BIAS | GEMM_BIAS_F32)) || bias, "ft_gemm_small_m: bias flag without bias");
   const int bn = M <= 64 ? 64 : 128;
-  const int sms = sm_count(device);
-  const int pairs = sms / 2;
-  const int tiles = (N + 255) / 256;
   const int k_blocks = (K + GEMM_BK - 1) / GEMM_BK;
-  if (ksplit <= 0) {
-    ksplit = 1;
-    if (tiles < pairs && workspace) {
-      // one wave: as many pieces per tile as there are CTA pairs to take them, each piece long
-      // enough (>= 4 k-blocks) to be worth a pipeline fill
-      ksplit = pairs / tiles;
-      const int max_split = k_blocks / 4 > 0 ? k_blocks / 4 : 1;
-      if (ksplit > max_split) ksplit = max_split;
-      if (ksplit < 1) ksplit = 1;
-    }
-  }
-  if (ksplit > SMALL_M_MAX_SPLIT) ksplit = SMALL_M_MAX_SPLIT;
+  if (ksplit <= 0) ksplit = workspace ? small_m_pick_split(N, K, 0, 1, device) : 1;
   // the residual is added by the finalize pass, which only the split path has
   if (residual && ksplit == 1 && workspace && k_blocks >= 2) ksplit = 2;
   FT_REQUIRE(ksplit == 1 || workspace, "ft_gemm_small_m: a split contraction needs the workspace");
   FT_REQUIRE(ksplit > 1 || !residual, "ft_gemm_small_m: the residual is added by the split path only");
-  GemmParams p;
-  p.bias = bias; p.M = N; p.N = M; p.K = K;   // tile space: rows of W x batch
-  p.status = device_status_word(device);
-  p.taps = ksplit > 1 ? 1 : 0; p.cblocks = 0; p.ksplit = 1;
-  for (int t = 0; t < GEMM_MAX_TAPS; ++t) p.shift[t] = 0;
-  p.gHp = p.gWp = p.cHo = p.cWo = p.c_oh = p.c_ow = 0; p.split_rows = 0;
-  CUtensorMap tmA, tmB, tmC;
-  int rc = make_tmap_2d(&tmA, W, 2, K, N, ldw * 2, GEMM_BK, GEMM_BM, 3);
-  if (rc) return rc;
-  rc = make_tmap_2d(&tmB, X, 2, K, M, ldx * 2, GEMM_BK, bn / 2, 3);
-  if (rc) return rc;
+  int rc;
   if (ksplit == 1) {
+    GemmParams p;
+    p.bias = bias; p.M = N; p.N = M; p.K = K;   // tile space: rows of W x batch
+    p.status = device_status_word(device);
+    p.taps = 0; p.cblocks = 0; p.ksplit = 1;
+    for (int t = 0; t < GEMM_MAX_TAPS; ++t) p.shift[t] = 0;
+    p.gHp = p.gWp = p.cHo = p.cWo = p.c_oh = p.c_ow = 0; p.split_rows = 0;
     p.C = C; p.ldc = ldc;
     p.flags = (flags & 0xFFFF) | GEMM_EPI_TRANSPOSED;
+    CUtensorMap tmA, tmB, tmC;
+    rc = make_tmap_2d(&tmA, W, 2, K, N, ldw * 2, GEMM_BK, GEMM_BM, 3);
+    if (rc) return rc;
+    rc = make_tmap_2d(&tmB, X, 2, K, M, ldx * 2, GEMM_BK, bn / 2, 3);
+    if (rc) return rc;
     // the store map is not used by the transposed epilogue; point it at W so that it is valid
     rc = make_tmap_2d(&tmC, W, 2, K, N, ldw * 2, 64, 32, 3);
     if (rc) return rc;
     return bn == 64 ? launch_pair<64, false, false, 0>(tmA, tmB, tmC, p, device, 0, stream)
                     : launch_pair<128, false, false, 0>(tmA, tmB, tmC, p, device, 0, stream);
   }
-  const int per = (k_blocks + ksplit - 1) / ksplit;
-  p.ksplit = (k_blocks + per - 1) / per;
-  p.C = workspace; p.ldc = bn;
-  p.flags = GEMM_OUT_F32;
-  // a slice is a whole number of 256-row tiles, so a tile that hangs over the end of W stays
-  // inside its own slice
-  p.split_rows = tiles * 256;
-  rc = make_tmap_2d(&tmC, workspace, 4, bn, static_cast<uint64_t>(p.ksplit) * p.split_rows,
-                    static_cast<uint64_t>(bn) * 4, 32, 32, 3);
-  if (rc) return rc;
-  rc = bn == 64 ? launch_pair<64, false, false, 2>(tmA, tmB, tmC, p, device, 0, stream)
-                : launch_pair<128, false, false, 2>(tmA, tmB, tmC, p, device, 0, stream);
+  rc = small_m_split(X, W, workspace, M, N, K, ldx, ldw, &ksplit, 2, device, stream);
   if (rc) return rc;
   dim3 grid((N + 31) / 32, (M + 31) / 32), block(32, 8);
   small_m_finalize_kernel<<<grid, block, 0, stream>>>(workspace, static_cast<__nv_bfloat16*>(C),
                                                       static_cast<const __nv_bfloat16*>(residual), bias,
-                                                      (flags & GEMM_BIAS_F32) ? 1 : 0, M, N, bn, p.ksplit,
-                                                      p.split_rows, ldc, ldr);
+                                                      (flags & GEMM_BIAS_F32) ? 1 : 0, M, N, bn, ksplit,
+                                                      (N + 255) / 256 * 256, ldc, ldr);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// C[M, N] (fp32) (+)= X[M, K] W[N, K]^T for a small batch M <= 128, always through the split contraction
+// and its finalize pass (see ft_gemm_small_m), which also writes dyt_out[M, N] = (tanh(alpha C) w + b) * dyt_scale
+// as bf16 when dyt_out is given.  workspace: ft_gemm_small_m_workspace(M, N) floats.
+FT_API int ft_gemm_small_m_f32(const void* X, const void* W, float* C, int accumulate, const float* alpha, const float* dyt_w,
+                               const float* dyt_b, void* dyt_out, float dyt_scale, float* workspace, int M, int N, int K,
+                               long long ldx, long long ldw, long long ldc, long long ldd, int ksplit, int device,
+                               cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  using namespace ft;
+  FT_REQUIRE(X && W && C && workspace, "ft_gemm_small_m_f32: null operand");
+  FT_REQUIRE(M > 0 && M <= 128 && N > 0 && K > GEMM_BK, "ft_gemm_small_m_f32: M=%d must be in 1..128, K=%d above %d (N=%d)", M, K, GEMM_BK, N);
+  FT_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0, "ft_gemm_small_m_f32: strides must be multiples of 8");
+  FT_REQUIRE(!dyt_out || (alpha && dyt_w && dyt_b), "ft_gemm_small_m_f32: the fused norm needs its parameters");
+  int rc = small_m_split(X, W, workspace, M, N, K, ldx, ldw, &ksplit, 2, device, stream);
+  if (rc) return rc;
+  dim3 grid((N + 31) / 32, (M + 31) / 32), block(32, 8);
+  small_m_finalize_f32_kernel<<<grid, block, 0, stream>>>(workspace, C, accumulate, alpha, dyt_w, dyt_b,
+                                                          static_cast<__nv_bfloat16*>(dyt_out), dyt_scale, M, N, M <= 64 ? 64 : 128,
+                                                          ksplit, (N + 255) / 256 * 256, ldc, ldd);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

@@ -1,6 +1,9 @@
 // Memory-bound transformer kernels for sm_100a: RMSNorm (+ fused residual add)
 // forward/backward, rotary embedding (both pair conventions) forward/backward,
-// SwiGLU forward/backward, embedding gather / scatter-add.
+// SwiGLU forward/backward, embedding gather / scatter-add, dynamic tanh on an fp32
+// residual stream (optionally fused with the embedding gather), and the step between a
+// decoder layer's packed input projection and its attention (projection norms, query
+// temperature, KV append, MLP activation).
 //
 // Semantics follow the reference: RMSNorm = x * rsqrt(mean(x^2) + eps) * w with fp32
 // statistics (ferrotorch-gpu/src/bf16.rs:1340-1346, kernels.rs:10578, 10725); RoPE
@@ -419,6 +422,157 @@ __global__ void embedding_bwd_kernel(const long long* __restrict__ ids, const __
   }
 }
 
+// ---------------------------------------------------------------- 8-element rows of either dtype
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float* f) {
+  unpack8(*reinterpret_cast<const uint4*>(p), f);
+}
+__device__ __forceinline__ void load8(const float* p, float* f) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float* f) { *reinterpret_cast<uint4*>(p) = pack8(f); }
+__device__ __forceinline__ void store8(float* p, const float* f) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+}
+
+// ---------------------------------------------------------------- dynamic tanh
+// y = (tanh(alpha * x) * w + b) * scale, element by element (no row statistic), fp32 input and
+// parameters.  With `ids` the input row is table[ids[row]] (a row of the embedding, TI) and is also
+// written to x_out, the fp32 residual stream.  A thread owns eight columns and walks rows, so w and b
+// stay in registers.
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(NORM_THREADS)
+dyt_kernel(const TI* __restrict__ x, const long long* __restrict__ ids, int vocab, float* __restrict__ x_out,
+           const float* __restrict__ alpha_p, const float* __restrict__ w, const float* __restrict__ b,
+           TO* __restrict__ y, int rows, int H, long long ldx, long long ldy, float scale) {
+  const int v = blockIdx.x * blockDim.x + threadIdx.x;
+  if (v >= (H >> 3)) return;
+  const float alpha = *alpha_p;
+  float wv[8], bv[8];
+  load8(w + v * 8, wv);
+  load8(b + v * 8, bv);
+  for (int row = blockIdx.y; row < rows; row += gridDim.y) {
+    long long src = row;
+    if (ids) {
+      src = ids[row];
+      if (src < 0 || src >= vocab) src = 0;  // host validates; never read out of range
+    }
+    float f[8], o[8];
+    load8(x + src * ldx + v * 8, f);
+    if (x_out) store8(x_out + static_cast<long long>(row) * H + v * 8, f);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = (tanhf(alpha * f[j]) * wv[j] + bv[j]) * scale;
+    store8(y + static_cast<long long>(row) * ldy + v * 8, o);
+  }
+}
+
+// ---------------------------------------------------------------- packed projection -> attention
+// One pass over a row of the packed input projection [ .. q .. k .. v .. up .. ] of a decoder layer
+// whose attention and feed-forward read the same input:
+//   q   RMS-normalised over the whole projection (all heads at once), times the query temperature
+//       1 + coef * ln(floor((pos + 1) / every) + 1), written back in place
+//   k   RMS-normalised over the whole projection, written to its cache page
+//   v   copied to its cache page
+//   up  act(up), written to the input of the output projection
+// Each part is optional (null weight: no norm; coef 0: no temperature; no act output: no MLP).  The
+// means divide by q_count / k_count, the true sizes of the projections: padded elements are zero.
+struct QkvFinishParams {
+  void* packed;                 // [rows, ld]
+  long long ld;
+  const int* pos;
+  const int* slots;
+  const int* block_table;
+  void* k_cache;
+  void* v_cache;
+  const float* q_weight;
+  const float* k_weight;
+  void* act_out;                // [rows, ld_act]
+  long long ld_act;
+  int rows, q_off, q_n, k_off, k_n, v_off, v_n, up_off, up_n, q_count, k_count;
+  float eps, temp_coef;
+  double temp_every;
+  int act, block_size, max_blocks, num_blocks;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(NORM_THREADS)
+qkv_finish_kernel(const QkvFinishParams p) {
+  __shared__ float red[2][NORM_THREADS / 32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float* nul = nullptr;
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    T* y = static_cast<T*>(p.packed) + static_cast<long long>(row) * p.ld;
+    const int position = p.pos[row];
+    float sq = 0.f, sk = 0.f;
+    if (p.q_weight != nul)
+      for (int i = threadIdx.x * 8; i < p.q_n; i += NORM_THREADS * 8) {
+        float f[8];
+        load8(y + p.q_off + i, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sq += f[j] * f[j];
+      }
+    if (p.k_weight != nul)
+      for (int i = threadIdx.x * 8; i < p.k_n; i += NORM_THREADS * 8) {
+        float f[8];
+        load8(y + p.k_off + i, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sk += f[j] * f[j];
+      }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    __syncthreads();                       // the previous row's sums have been read
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+    // the MLP activation does not wait for the sums
+    for (int i = threadIdx.x * 8; i < p.up_n; i += NORM_THREADS * 8) {
+      float f[8];
+      load8(y + p.up_off + i, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] = act_fwd(f[j], p.act);
+      store8(static_cast<T*>(p.act_out) + static_cast<long long>(row) * p.ld_act + i, f);
+    }
+    const int blk = p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + position / p.block_size];
+    const bool cached = blk >= 0 && blk < p.num_blocks;    // host validates; never write out of range
+    const long long token = static_cast<long long>(blk) * p.block_size + position % p.block_size;
+    if (cached)
+      for (int i = threadIdx.x * 8; i < p.v_n; i += NORM_THREADS * 8) {
+        float f[8];
+        load8(y + p.v_off + i, f);
+        store8(static_cast<T*>(p.v_cache) + token * p.v_n + i, f);
+      }
+    __syncthreads();
+    sq = 0.f; sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < NORM_THREADS / 32; ++w) { sq += red[0][w]; sk += red[1][w]; }
+    float rq = 1.f;
+    if (p.q_weight != nul) rq = 1.f / sqrtf(sq / static_cast<float>(p.q_count) + p.eps);
+    if (p.temp_coef != 0.f)
+      rq *= 1.f + p.temp_coef * logf(static_cast<float>(floor((position + 1) / p.temp_every)) + 1.f);
+    if (p.q_weight != nul || p.temp_coef != 0.f)
+      for (int i = threadIdx.x * 8; i < p.q_n; i += NORM_THREADS * 8) {
+        float f[8], w[8];
+        load8(y + p.q_off + i, f);
+        if (p.q_weight != nul) load8(p.q_weight + i, w);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] *= p.q_weight != nul ? rq * w[j] : rq;
+        store8(y + p.q_off + i, f);
+      }
+    if (cached) {
+      const float rk = p.k_weight != nul ? 1.f / sqrtf(sk / static_cast<float>(p.k_count) + p.eps) : 1.f;
+      for (int i = threadIdx.x * 8; i < p.k_n; i += NORM_THREADS * 8) {
+        float f[8], w[8];
+        load8(y + p.k_off + i, f);
+        if (p.k_weight != nul) {
+          load8(p.k_weight + i, w);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) f[j] *= rk * w[j];
+        }
+        store8(static_cast<T*>(p.k_cache) + token * p.k_n + i, f);
+      }
+    }
+  }
+}
+
 static inline int blocks_for(long long work, int threads, int device, int per_sm = 8) {
   long long b = (work + threads - 1) / threads;
   const long long cap = static_cast<long long>(sm_count(device)) * per_sm;
@@ -549,6 +703,74 @@ FT_API int ft_embedding_bwd(const long long* ids, const void* dy, void* dw, int 
   const int grid = T < sm_count(device) * 16 ? T : sm_count(device) * 16;
   embedding_bwd_kernel<<<grid, 128, 0, stream>>>(ids, static_cast<const __nv_bfloat16*>(dy),
                                                  static_cast<__nv_bfloat16*>(dw), T, H, vocab);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// Dynamic tanh: y[rows, H] = (tanh(alpha x) w + b) * scale.  x: fp32 [rows, ldx], or with ids (int64
+// [rows]) the rows table[ids] of a bf16 (in_bf16) or fp32 table [vocab, ldx], which are then also
+// written to x_out (fp32 [rows, H]).  y: bf16, or fp32 with out_f32.  alpha: one fp32 on the device.
+FT_API int ft_dyt_fwd(const void* x, const long long* ids, int vocab, int in_bf16, float* x_out, const float* alpha,
+                      const float* w, const float* b, void* y, int out_f32, int rows, int H, long long ldx, long long ldy,
+                      float scale, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(x && alpha && w && b && y, "ft_dyt_fwd: null pointer");
+  FT_REQUIRE(H > 0 && H % 8 == 0 && ldx % 8 == 0 && ldy % 8 == 0 && ldx >= H && ldy >= H, "ft_dyt_fwd: H=%d and strides must be multiples of 8", H);
+  FT_REQUIRE(((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w) |
+               reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(x_out)) & 15) == 0, "ft_dyt_fwd: pointers must be 16-byte aligned");
+  FT_REQUIRE(!ids || vocab > 0, "ft_dyt_fwd: a gather needs the table size");
+  if (rows <= 0) return FT_E_OK;
+  const int gx = (H / 8 + NORM_THREADS - 1) / NORM_THREADS;
+  int gy = sm_count(device) * 8 / gx;
+  if (gy < 1) gy = 1;
+  if (gy > rows) gy = rows;
+  const dim3 grid(gx, gy);
+#define FT_DYT(TI, TO)                                                                                             \
+  dyt_kernel<TI, TO><<<grid, NORM_THREADS, 0, stream>>>(static_cast<const TI*>(x), ids, vocab, x_out, alpha, w, b, \
+                                                        static_cast<TO*>(y), rows, H, ldx, ldy, scale)
+  if (in_bf16) {
+    if (out_f32) FT_DYT(__nv_bfloat16, float); else FT_DYT(__nv_bfloat16, __nv_bfloat16);
+  } else {
+    if (out_f32) FT_DYT(float, float); else FT_DYT(float, __nv_bfloat16);
+  }
+#undef FT_DYT
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// The pass between a packed input projection and its attention (see qkv_finish_kernel).  packed, caches
+// and act_out are bf16, or fp32 with f32.  Offsets and sizes in elements, multiples of 8.
+FT_API int ft_qkv_finish(void* packed, long long ld, const int* pos, const int* slots, const int* block_table, void* k_cache,
+                         void* v_cache, const float* q_weight, const float* k_weight, void* act_out, long long ld_act,
+                         int rows, int q_off, int q_n, int k_off, int k_n, int v_off, int v_n, int up_off, int up_n,
+                         int q_count, int k_count, float eps, float temp_coef, float temp_every, int act, int f32,
+                         int block_size, int max_blocks, int num_blocks, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(packed && pos && slots && block_table && k_cache && v_cache, "ft_qkv_finish: null pointer");
+  FT_REQUIRE(((q_off | q_n | k_off | k_n | v_off | v_n | up_off | up_n) & 7) == 0 && ld % 8 == 0 && ld_act % 8 == 0,
+             "ft_qkv_finish: offsets, sizes and strides must be multiples of 8");
+  FT_REQUIRE(q_n > 0 && k_n > 0 && v_n > 0 && up_n >= 0 && q_off >= 0 && k_off >= 0 && v_off >= 0 && up_off >= 0 &&
+                 q_off + q_n <= ld && k_off + k_n <= ld && v_off + v_n <= ld && up_off + up_n <= ld && (up_n == 0 || (act_out && up_n <= ld_act)),
+             "ft_qkv_finish: a segment lies outside the row");
+  FT_REQUIRE(((reinterpret_cast<uintptr_t>(packed) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) |
+               reinterpret_cast<uintptr_t>(q_weight) | reinterpret_cast<uintptr_t>(k_weight) | reinterpret_cast<uintptr_t>(act_out)) & 15) == 0,
+             "ft_qkv_finish: pointers must be 16-byte aligned");
+  FT_REQUIRE(block_size > 0 && max_blocks > 0 && num_blocks > 0 && q_count > 0 && k_count > 0 && temp_every > 0.f && act >= 0 && act <= 2,
+             "ft_qkv_finish: bad argument");
+  if (rows <= 0) return FT_E_OK;
+  QkvFinishParams p;
+  p.packed = packed; p.ld = ld; p.pos = pos; p.slots = slots; p.block_table = block_table;
+  p.k_cache = k_cache; p.v_cache = v_cache; p.q_weight = q_weight; p.k_weight = k_weight;
+  p.act_out = act_out; p.ld_act = ld_act; p.rows = rows;
+  p.q_off = q_off; p.q_n = q_n; p.k_off = k_off; p.k_n = k_n; p.v_off = v_off; p.v_n = v_n;
+  p.up_off = up_off; p.up_n = up_n; p.q_count = q_count; p.k_count = k_count;
+  p.eps = eps; p.temp_coef = temp_coef; p.temp_every = temp_every;
+  p.act = act; p.block_size = block_size; p.max_blocks = max_blocks; p.num_blocks = num_blocks;
+  const int grid = rows < sm_count(device) * 8 ? rows : sm_count(device) * 8;
+  if (f32) qkv_finish_kernel<float><<<grid, NORM_THREADS, 0, stream>>>(p);
+  else qkv_finish_kernel<__nv_bfloat16><<<grid, NORM_THREADS, 0, stream>>>(p);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

@@ -9,13 +9,17 @@
 //
 //   ft_kv_append        scatter new K/V rows (a prefill chunk or one decode token per sequence)
 //                       into the cache through the block table.
-//   ft_paged_decode     one query token per sequence: softmax(q K^T / sqrt(d)) V over the cached
+//   ft_paged_decode     one query token per row: softmax(scale * q K^T) V over the cached
 //                       context, GQA (all query heads of a KV group share one pass over K/V),
-//                       flash-decoding split over the context with a second combine pass.
-// Decode attention is bandwidth bound (every cached byte is read once per step).  head_dim 128
-// runs on the tensor-core kernel (paged_decode_tc_kernel: cp.async rows -> shared memory ->
-// tcgen05.mma); head_dim 64 on the CUDA-core kernel, which reads K with
-// one key per lane (full rows, no shuffles in the dot products) and V with one row per warp step.
+//                       flash-decoding split over the context with a second combine pass, and an
+//                       optional output gate per head.
+//   ft_paged_rows       the same for any mixture of rows (each with its own sequence and number of
+//                       visible keys), any head sizes, bf16 or fp32: the exact, simple kernel.
+// Decode attention is bandwidth bound (every cached byte is read once per step).  Key / value head
+// sizes up to 128 (multiples of 16; they may differ) run on the tensor-core kernel
+// (paged_decode_tc_kernel: cp.async rows -> shared memory -> tcgen05.mma).  The CUDA-core kernel for
+// equal sizes of 64 or 128 reads K with one key per lane (full rows, no shuffles in the dot products)
+// and V with one row per warp step; it serves rows whose pointers or strides are not 16-byte aligned.
 #include "ft_host.h"
 #include "ft_ptx.cuh"
 
@@ -23,7 +27,17 @@ namespace ft {
 
 constexpr int PD_THREADS = 128;
 constexpr int PD_WARPS = PD_THREADS / 32;
-constexpr int PD_MAX_G = 8;
+
+// Output gate: head h of a row is multiplied by sigmoid(gate[row, h]) when a gate is given.
+struct HeadGate {
+  const void* g;       // null: no gate
+  long long ld;        // row stride in elements
+};
+__device__ __forceinline__ float gate_value(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float head_gate_bf16(const HeadGate& gt, int row, int head) {
+  if (!gt.g) return 1.f;
+  return gate_value(__bfloat162float(static_cast<const __nv_bfloat16*>(gt.g)[static_cast<long long>(row) * gt.ld + head]));
+}
 
 // k_new / v_new: [T, Hkv, D] rows with token stride ld (elements).  Token i goes to sequence
 // seq_ids[i] (or i / tokens_per_seq when null) at position pos[i].
@@ -59,9 +73,9 @@ template <int D, int G>
 __global__ void __launch_bounds__(PD_THREADS)
 paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_table,
-                    const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
-                    float* __restrict__ part_ml, int Hq, int Hkv, long long ldq, long long ldo, int block_size,
-                    int max_blocks, int num_blocks, float scale_log2, int n_splits) {
+                    const int* __restrict__ row_slot, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
+                    float* __restrict__ part_o, float* __restrict__ part_ml, int Hq, int Hkv, long long ldq, long long ldo,
+                    int block_size, int max_blocks, int num_blocks, float scale_log2, int n_splits, HeadGate gate) {
   constexpr int DV = D / 16;  // dims per lane in the PV phase (half-warp covers D)
   const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -89,7 +103,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 #pragma unroll
     for (int j = 0; j < DV; ++j) o[g][j] = 0.f;
   }
-  const int* bt = block_table + static_cast<long long>(b) * max_blocks;
+  const int* bt = block_table + static_cast<long long>(row_slot ? row_slot[b] : b) * max_blocks;
   const long long row_stride = static_cast<long long>(Hkv) * D;
   const long long head_off = static_cast<long long>(kvh) * D;
 
@@ -207,7 +221,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     }
     const int hq = kvh * G + g;
     if (n_splits == 1) {
-      out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+      out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] =
+          __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq) : 0.f);
     } else {
       const long long pidx = (static_cast<long long>(b) * Hq + hq) * n_splits + split;
       part_o[pidx * D + d] = acc;
@@ -216,9 +231,9 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   }
 }
 
-template <int D>
 __global__ void paged_decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                            __nv_bfloat16* __restrict__ out, int Hq, long long ldo, int n_splits) {
+                                            __nv_bfloat16* __restrict__ out, int Hq, int D, long long ldo, int n_splits,
+                                            HeadGate gate) {
   const int hq = blockIdx.x, b = blockIdx.y;
   const long long base = (static_cast<long long>(b) * Hq + hq) * n_splits;
   float mm = -INFINITY;
@@ -231,13 +246,16 @@ __global__ void paged_decode_combine_kernel(const float* __restrict__ part_o, co
       ll += part_ml[(base + s) * 2 + 1] * sc;
       acc += part_o[(base + s) * D + d] * sc;
     }
-    out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+    out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] =
+        __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq) : 0.f);
   }
 }
 
 
 // ----------------------------------------------------------------------------- tensor-core decode
-// The decode kernel for head_dim 128 (any page size).  A CTA owns one (sequence, KV head, context
+// The decode kernel for key and value head sizes up to 128 (any page size).  Head sizes below the tile's
+// (64 or 128 for keys, 128 for values: an MMA with 64 rows lays its accumulator out differently) leave
+// zeroed columns in the operand tiles.  A CTA owns one (sequence, KV head, context
 // split) and walks its keys in tiles of 128; all query heads of the KV group ride along as the
 // (padded) 16-wide N dimension of two small MMAs per tile:
 //     S^T[key, head] = K_tile[key, :] . Q[head, :]          (M = 128 keys, N = 16, K = head_dim)
@@ -260,12 +278,15 @@ constexpr int PT_STAGES = 3;
 constexpr int PT_N = 16;       // MMA N: query heads of the group, zero-padded
 constexpr float PT_RESCALE = 8.f;
 
-template <int D>
-struct PtCfg {  // D = 128 (an MMA with 64 rows lays its accumulator out differently)
-  static constexpr int KV_BYTES = PT_TILE * D * 2;        // one K or V tile
-  static constexpr int STAGE_BYTES = 2 * KV_BYTES;
+constexpr int PT_VD = 128;     // rows of O^T
+
+template <int HD>
+struct PtCfg {  // HD: width of the K tile (64 or 128)
+  static constexpr int K_BYTES = PT_TILE * HD * 2;
+  static constexpr int V_BYTES = PT_TILE * PT_VD * 2;
+  static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;
   static constexpr int CHUNK = PT_TILE * 128;             // one 64-wide column chunk of a tile
-  static constexpr int Q_BYTES = PT_N * D * 2;            // Q^T operand: 16 rows x head_dim
+  static constexpr int Q_BYTES = PT_N * HD * 2;           // Q^T operand: 16 rows x key head size
   static constexpr int P_BYTES = PT_N * PT_TILE * 2;      // P^T operand: 16 rows x 128 keys
   static constexpr int OFF_Q = PT_STAGES * STAGE_BYTES;
   static constexpr int OFF_P = OFF_Q + Q_BYTES;           // two buffers
@@ -274,14 +295,17 @@ struct PtCfg {  // D = 128 (an MMA with 64 rows lays its accumulator out differe
   static constexpr int SMEM_BYTES = OFF_BAR + 256 + 1024;
 };
 
-template <int D, int G>
+// G: query heads of a group, rounded up to 1 / 2 / 4 / 8 / 16 (g_real of them exist).  D, Dv: key and value
+// head sizes, multiples of 16.
+template <int HD, int G>
 __global__ void __launch_bounds__(PT_THREADS, 1)
 paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
                        const __nv_bfloat16* __restrict__ q, const int* __restrict__ block_table,
-                       const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
-                       float* __restrict__ part_ml, int Hq, int Hkv, long long ldq, long long ldo, int block_size,
-                       int max_blocks, int num_blocks, float scale_log2, int n_splits, int* status) {
-  using Cfg = PtCfg<D>;
+                       const int* __restrict__ row_slot, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
+                       float* __restrict__ part_o, float* __restrict__ part_ml, int Hq, int Hkv, int D, int Dv, int g_real,
+                       long long ldq, long long ldo, int block_size, int max_blocks, int num_blocks, float scale_log2,
+                       int n_splits, HeadGate gate, int* status) {
+  using Cfg = PtCfg<HD>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
@@ -320,23 +344,21 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
     tmem_alloc(smem_u32(tmem_slot), 64);
     tmem_relinquish();
   }
-  // Q^T operand (scaled, bf16, rows >= G zero) and zeroed P^T buffers, written by all threads
+  // Q^T operand (bf16, rows past the group zero; the scale is applied to the fp32 scores) and zeroed
+  // P^T buffers, written by all threads.  Head sizes below the tile's: the columns that the loaders
+  // never write are zeroed in every stage.
   for (int i = threadIdx.x; i < (Cfg::Q_BYTES + 2 * Cfg::P_BYTES) / 16; i += blockDim.x)
     reinterpret_cast<uint4*>(smem + Cfg::OFF_Q)[i] = make_uint4(0u, 0u, 0u, 0u);
+  if (D < HD || Dv < PT_VD)
+    for (int i = threadIdx.x; i < PT_STAGES * Cfg::STAGE_BYTES / 16; i += blockDim.x)
+      reinterpret_cast<uint4*>(smem)[i] = make_uint4(0u, 0u, 0u, 0u);
   __syncthreads();
-  for (int i = threadIdx.x; i < G * (D / 8); i += blockDim.x) {
+  for (int i = threadIdx.x; i < g_real * (D / 8); i += blockDim.x) {
     const int g = i / (D / 8), j = i - g * (D / 8);  // 16-byte chunk j of head g
     const uint4 raw = *reinterpret_cast<const uint4*>(q + static_cast<long long>(b) * ldq +
-                                                      static_cast<long long>(kvh * G + g) * D + j * 8);
-    const float2 a0 = unpack_bf16x2(raw.x), a1 = unpack_bf16x2(raw.y), a2 = unpack_bf16x2(raw.z),
-                 a3 = unpack_bf16x2(raw.w);
-    uint4 o;
-    o.x = pack_bf16x2(a0.x * scale_log2, a0.y * scale_log2);
-    o.y = pack_bf16x2(a1.x * scale_log2, a1.y * scale_log2);
-    o.z = pack_bf16x2(a2.x * scale_log2, a2.y * scale_log2);
-    o.w = pack_bf16x2(a3.x * scale_log2, a3.y * scale_log2);
+                                                      static_cast<long long>(kvh * g_real + g) * D + j * 8);
     const int c = j >> 3, jj = j & 7;                // 64-wide chunk, 16-byte unit inside it
-    *reinterpret_cast<uint4*>(smem + Cfg::OFF_Q + c * (PT_N * 128) + g * 128 + ((jj ^ (g & 7)) << 4)) = o;
+    *reinterpret_cast<uint4*>(smem + Cfg::OFF_Q + c * (PT_N * 128) + g * 128 + ((jj ^ (g & 7)) << 4)) = raw;
   }
   fence_proxy_async_smem();
   tc_fence_before();
@@ -351,9 +373,8 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
     // and of the V tile: 16 consecutive threads read one 256-byte cache row.
     const int lt = threadIdx.x - 256;
     const int unit = lt & 15, row0 = lt >> 4;
-    const int* bt = block_table + static_cast<long long>(b) * max_blocks;
-    const long long row_stride = static_cast<long long>(Hkv) * D;
-    const long long col_off = static_cast<long long>(kvh) * D + unit * 8;
+    const int* bt = block_table + static_cast<long long>(row_slot ? row_slot[b] : b) * max_blocks;
+    const bool has_k = unit * 8 < D, has_v = unit * 8 < Dv;   // this thread's 16-byte column exists
     const uint32_t chunk_off = static_cast<uint32_t>(unit >> 3) * Cfg::CHUNK;
     constexpr int AHEAD = PT_STAGES - 1;
     bool ok = true;
@@ -372,7 +393,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
         ok = mbar_wait(bar(ST_EMPTY + st), ((t / PT_STAGES) & 1) ^ 1u, abort_word, FT_ERR_TIMEOUT_PRODUCER);
         if (ok) {
           const int key0 = (tile_lo + t) * PT_TILE;
-          const uint32_t sK = sbase + st * Cfg::STAGE_BYTES + chunk_off, sV = sK + Cfg::KV_BYTES;
+          const uint32_t sK = sbase + st * Cfg::STAGE_BYTES + chunk_off, sV = sK + Cfg::K_BYTES;
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
             const int row = row0 + 8 * i;
@@ -380,13 +401,15 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
             const int page = key / block_size;
             int blk = (key < len && page < max_blocks) ? __ldg(bt + page) : 0;
             blk = min(max(blk, 0), num_blocks - 1);
-            const long long src = (static_cast<long long>(blk) * block_size + key % block_size) * row_stride + col_off;
+            const long long src = ((static_cast<long long>(blk) * block_size + key % block_size) * Hkv + kvh);
             const uint32_t dst = static_cast<uint32_t>(row) * 128u + (static_cast<uint32_t>((unit & 7) ^ (row & 7)) << 4);
             const uint32_t nbytes = key < len ? 16u : 0u;   // rows past the context are zero-filled
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sK + dst), "l"(k_cache + src), "r"(nbytes)
-                         : "memory");
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sV + dst), "l"(v_cache + src), "r"(nbytes)
-                         : "memory");
+            if (has_k)
+              asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sK + dst),
+                           "l"(k_cache + src * D + unit * 8), "r"(nbytes) : "memory");
+            if (has_v)
+              asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sV + dst),
+                           "l"(v_cache + src * Dv + unit * 8), "r"(nbytes) : "memory");
           }
         }
       }
@@ -397,12 +420,12 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0 && n_tiles > 0) {
       constexpr uint32_t idesc_qk = make_idesc_f16(PT_TILE, PT_N, 1, 0, 0);   // keys x heads, both K-major
-      constexpr uint32_t idesc_pv = make_idesc_f16(D, PT_N, 1, 1, 0);         // dims x heads, A (V^T) MN-major
+      constexpr uint32_t idesc_pv = make_idesc_f16(PT_VD, PT_N, 1, 1, 0);     // dims x heads, A (V^T) MN-major
       auto issue_qk = [&](int t) {
         const uint32_t sK = sbase + (t % PT_STAGES) * Cfg::STAGE_BYTES;
         const uint32_t d = tmem_base + COL_S + (t & 1) * PT_N;
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < HD / 16; ++kk) {
           const uint32_t ko = (kk >> 2) * Cfg::CHUNK + (kk & 3) * 32;
           const uint32_t qo = (kk >> 2) * (PT_N * 128) + (kk & 3) * 32;
           umma_f16_ss(d, make_smem_desc_sw128(sK + ko, 16, 1024), make_smem_desc_sw128(sQ + qo, 16, 1024),
@@ -427,7 +450,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
         ok = mbar_wait(bar(P_FULL + (t & 1)), (t >> 1) & 1, abort_word, FT_ERR_TIMEOUT_MMA);
         if (!ok) break;
         tc_fence_after();
-        const uint32_t sV = sbase + st * Cfg::STAGE_BYTES + Cfg::KV_BYTES;
+        const uint32_t sV = sbase + st * Cfg::STAGE_BYTES + Cfg::K_BYTES;
         const uint32_t pb = sP + (t & 1) * Cfg::P_BYTES;
 #pragma unroll
         for (int kk = 0; kk < PT_TILE / 16; ++kk) {
@@ -467,7 +490,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
       float s[G], mx[G];
 #pragma unroll
       for (int g = 0; g < G; ++g) {
-        s[g] = valid ? __uint_as_float(sv[g]) : -INFINITY;
+        s[g] = valid ? __uint_as_float(sv[g]) * scale_log2 : -INFINITY;
         mx[g] = warp_max(s[g]);
       }
       if (lane == 0) {
@@ -533,7 +556,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
     asm volatile("bar.sync 1, 128;" ::: "memory");
 #pragma unroll
     for (int g = 0; g < G; ++g) l_tot[g] = s_red[g] + s_red[PT_N + g] + s_red[2 * PT_N + g] + s_red[3 * PT_N + g];
-    if (ok && r < D) {
+    if (ok) {                                     // whole warps: the TMEM load is a warp-wide instruction
       uint32_t ov[16];
 #pragma unroll
       for (int i = 0; i < 16; ++i) ov[i] = 0u;
@@ -543,14 +566,15 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
       }
 #pragma unroll
       for (int g = 0; g < G; ++g) {
-        const int hq = kvh * G + g;
+        if (g >= g_real || r >= Dv) continue;
+        const int hq = kvh * g_real + g;
         const float acc = __uint_as_float(ov[g]);
         if (n_splits == 1) {
-          out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + r] =
-              __float2bfloat16(l_tot[g] > 0.f ? acc / l_tot[g] : 0.f);
+          out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * Dv + r] =
+              __float2bfloat16(l_tot[g] > 0.f ? acc / l_tot[g] * head_gate_bf16(gate, b, hq) : 0.f);
         } else {
           const long long pidx = (static_cast<long long>(b) * Hq + hq) * n_splits + split;
-          part_o[pidx * D + r] = acc;
+          part_o[pidx * Dv + r] = acc;
           if (r == 0) { part_ml[pidx * 2] = m_ref[g]; part_ml[pidx * 2 + 1] = l_tot[g]; }
         }
       }
@@ -564,6 +588,124 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
     tmem_dealloc(tmem_base, 64);
   }
   if (threadIdx.x == 0 && *abort_word != 0 && status) atomicCAS(status, 0, *abort_word);
+}
+
+// ----------------------------------------------------------------------------- any rows, any sizes
+// Row i attends to keys 0 .. visible[i] - 1 of sequence row_slot[i].  A CTA owns one row and up to
+// PR_HEADS query heads of one KV head; its four warps walk tiles of 32 keys (lane = key while scoring,
+// lane = value dim while accumulating) with an fp32 online softmax each, merged at the end.
+constexpr int PR_HEADS = 8;
+
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void from_f32(float v, float* p) { *p = v; }
+__device__ __forceinline__ void from_f32(float v, __nv_bfloat16* p) { *p = __float2bfloat16(v); }
+
+template <typename T>
+__global__ void __launch_bounds__(PD_THREADS)
+paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
+                  const int* __restrict__ block_table, const int* __restrict__ row_slot, const int* __restrict__ visible,
+                  HeadGate gate, T* __restrict__ out, int rows, int Hq, int Hkv, int D, int Dv, long long ldq, long long ldo,
+                  int block_size, int max_blocks, int num_blocks, float scale, int head_groups) {
+  extern __shared__ float sm[];
+  const int g_all = Hq / Hkv;
+  const int kvh = blockIdx.y / head_groups, h0 = (blockIdx.y % head_groups) * PR_HEADS;
+  const int g = min(PR_HEADS, g_all - h0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* s_q = sm;                                   // [g][D], scaled by scale * log2(e)
+  float* s_o = s_q + PR_HEADS * D;                   // [warps][g][Dv]
+  float* s_p = s_o + PD_WARPS * PR_HEADS * Dv;       // [warps][g][32]
+  float* s_m = s_p + PD_WARPS * PR_HEADS * 32;       // [warps][g]
+  float* s_l = s_m + PD_WARPS * PR_HEADS;
+  for (int row = blockIdx.x; row < rows; row += gridDim.x) {
+    __syncthreads();
+    const int len = min(visible[row], max_blocks * block_size);
+    const int* bt = block_table + static_cast<long long>(row_slot[row]) * max_blocks;
+    for (int i = threadIdx.x; i < g * D; i += PD_THREADS) {
+      const int h = i / D, d = i - h * D;
+      s_q[h * D + d] = to_f32(q[static_cast<long long>(row) * ldq + static_cast<long long>(kvh * g_all + h0 + h) * D + d]) *
+                       (scale * 1.4426950408889634f);
+    }
+    for (int i = threadIdx.x; i < PD_WARPS * PR_HEADS * Dv; i += PD_THREADS) s_o[i] = 0.f;
+    float m[PR_HEADS], l[PR_HEADS];
+#pragma unroll
+    for (int h = 0; h < PR_HEADS; ++h) { m[h] = -INFINITY; l[h] = 0.f; }
+    __syncthreads();
+    for (int key0 = warp * 32; key0 < len; key0 += PD_WARPS * 32) {
+      const int key = key0 + lane;
+      const bool valid = key < len;
+      const int kk = valid ? key : key0;
+      const int blk = min(max(bt[kk / block_size], 0), num_blocks - 1);
+      const T* kr = k_cache + ((static_cast<long long>(blk) * block_size + kk % block_size) * Hkv + kvh) * D;
+      float s[PR_HEADS];
+#pragma unroll
+      for (int h = 0; h < PR_HEADS; ++h) s[h] = 0.f;
+      for (int d = 0; d < D; ++d) {
+        const float kd = to_f32(kr[d]);
+#pragma unroll
+        for (int h = 0; h < PR_HEADS; ++h)
+          if (h < g) s[h] += kd * s_q[h * D + d];
+      }
+      float* o = s_o + warp * PR_HEADS * Dv;
+      float* pr = s_p + warp * PR_HEADS * 32;
+      float alpha[PR_HEADS];
+#pragma unroll
+      for (int h = 0; h < PR_HEADS; ++h) {
+        alpha[h] = 1.f;
+        if (h >= g) continue;
+        const float sv = valid ? s[h] : -INFINITY;
+        const float m_new = fmaxf(m[h], warp_max(sv));
+        const float pv = valid ? exp2f(sv - m_new) : 0.f;
+        alpha[h] = exp2f(m[h] - m_new);              // first tile: exp2(-inf) = 0
+        l[h] = l[h] * alpha[h] + warp_sum(pv);
+        m[h] = m_new;
+        pr[h * 32 + lane] = pv;
+      }
+      __syncwarp();
+      const int n_keys = min(32, len - key0);
+      for (int d = lane; d < Dv; d += 32) {
+        float acc[PR_HEADS];
+#pragma unroll
+        for (int h = 0; h < PR_HEADS; ++h) acc[h] = h < g ? o[h * Dv + d] * alpha[h] : 0.f;
+        for (int j = 0; j < n_keys; ++j) {
+          const int kj = key0 + j;
+          const int bj = min(max(bt[kj / block_size], 0), num_blocks - 1);
+          const float vd = to_f32(v_cache[((static_cast<long long>(bj) * block_size + kj % block_size) * Hkv + kvh) * Dv + d]);
+#pragma unroll
+          for (int h = 0; h < PR_HEADS; ++h)
+            if (h < g) acc[h] += pr[h * 32 + j] * vd;
+        }
+#pragma unroll
+        for (int h = 0; h < PR_HEADS; ++h)
+          if (h < g) o[h * Dv + d] = acc[h];
+      }
+      __syncwarp();
+    }
+    if (lane == 0) {
+#pragma unroll
+      for (int h = 0; h < PR_HEADS; ++h)
+        if (h < g) { s_m[warp * PR_HEADS + h] = m[h]; s_l[warp * PR_HEADS + h] = l[h]; }
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < g * Dv; i += PD_THREADS) {
+      const int h = i / Dv, d = i - h * Dv;
+      float mm = -INFINITY;
+#pragma unroll
+      for (int w = 0; w < PD_WARPS; ++w) mm = fmaxf(mm, s_m[w * PR_HEADS + h]);
+      float ll = 0.f, acc = 0.f;
+#pragma unroll
+      for (int w = 0; w < PD_WARPS; ++w) {
+        const float mw = s_m[w * PR_HEADS + h];
+        const float sc = mw == -INFINITY ? 0.f : exp2f(mw - mm);
+        ll += s_l[w * PR_HEADS + h] * sc;
+        acc += s_o[(w * PR_HEADS + h) * Dv + d] * sc;
+      }
+      const int hq = kvh * g_all + h0 + h;
+      float v = ll > 0.f ? acc / ll : 0.f;
+      if (gate.g) v *= gate_value(to_f32(static_cast<const T*>(gate.g)[static_cast<long long>(row) * gate.ld + hq]));
+      from_f32(v, out + static_cast<long long>(row) * ldo + static_cast<long long>(hq) * Dv + d);
+    }
+  }
 }
 
 }  // namespace ft
@@ -589,69 +731,64 @@ FT_API int ft_kv_append(const void* k_new, const void* v_new, void* k_cache, voi
   return FT_E_OK;
 }
 
-// Scratch floats needed for n_splits > 1: B * Hq * n_splits * (D + 2).
-FT_API long long ft_paged_decode_scratch(int B, int Hq, int D, int n_splits) {
-  return n_splits > 1 ? static_cast<long long>(B) * Hq * n_splits * (D + 2) : 0;
+// Scratch floats needed for n_splits > 1: B * Hq * n_splits * (Dv + 2).
+FT_API long long ft_paged_decode_scratch(int B, int Hq, int Dv, int n_splits) {
+  return n_splits > 1 ? static_cast<long long>(B) * Hq * n_splits * (Dv + 2) : 0;
 }
 
-// q: [B, Hq, D] (row stride ldq), out: [B, Hq, D] (row stride ldo), ctx_len: int32 [B] = number of
-// cached tokens to attend to (including the current one, which must already be appended).
+// q: [B, Hq, D] (row stride ldq), out: [B, Hq, Dv] (row stride ldo), ctx_len: int32 [B] = number of
+// cached tokens to attend to (including the current one, which must already be appended).  Row b reads
+// sequence row_slot[b] of the block table (null: sequence b).  gate (bf16 [B, Hq], row stride ldg, or
+// null): output heads are multiplied by sigmoid(gate).
 FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
-                           const int* ctx_len, void* out, float* scratch, int B, int Hq, int Hkv, int D,
-                           long long ldq, long long ldo, int block_size, int max_blocks, int num_blocks,
-                           float scale, int n_splits, int device, cudaStream_t stream) {
+                           const int* row_slot, const int* ctx_len, const void* gate, void* out, float* scratch, int B,
+                           int Hq, int Hkv, int D, int Dv, long long ldq, long long ldg, long long ldo, int block_size,
+                           int max_blocks, int num_blocks, float scale, int n_splits, int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(q && k_cache && v_cache && block_table && ctx_len && out, "ft_paged_decode: null pointer");
-  FT_REQUIRE(D == 64 || D == 128, "ft_paged_decode: head_dim %d not supported (64, 128)", D);
-  FT_REQUIRE(Hq % Hkv == 0 && Hq / Hkv <= PD_MAX_G, "ft_paged_decode: group size %d not supported (max %d)", Hq / Hkv, PD_MAX_G);
+  FT_REQUIRE(B >= 0 && Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0, "ft_paged_decode: bad shape");
   FT_REQUIRE(n_splits >= 1 && (n_splits == 1 || scratch), "ft_paged_decode: splits need scratch");
-  if (B <= 0) return FT_E_OK;
+  if (B == 0) return FT_E_OK;
   const float sl2 = scale * 1.4426950408889634f;
   float* part_o = scratch;
-  float* part_ml = scratch ? scratch + static_cast<long long>(B) * Hq * n_splits * D : nullptr;
+  float* part_ml = scratch ? scratch + static_cast<long long>(B) * Hq * n_splits * Dv : nullptr;
   dim3 grid(n_splits, Hkv, B);
   const int G = Hq / Hkv;
-  const bool tensor_core = D == 128 && (G == 1 || G == 2 || G == 4 || G == 8) && block_size >= 1 &&
+  const HeadGate hg = {gate, ldg};
+  const bool tensor_core = D >= 16 && D <= 128 && D % 16 == 0 && Dv >= 16 && Dv <= 128 && Dv % 16 == 0 && G <= PT_N &&
                            (reinterpret_cast<uintptr_t>(q) & 15) == 0 && ldq % 8 == 0 &&
                            ((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) == 0;
   if (tensor_core) {
-    using Cfg = PtCfg<128>;
     int* status = device_status_word(device);
-#define FT_PT_LAUNCH(GG)                                                                                        \
+#define FT_PT_LAUNCH(HH, GG)                                                                                    \
   {                                                                                                             \
-    auto kern = paged_decode_tc_kernel<128, GG>;                                                                \
+    auto kern = paged_decode_tc_kernel<HH, GG>;                                                                 \
     static bool attr_set[64] = {false};                                                                         \
     if (!attr_set[device]) {                                                                                    \
-      FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));  \
+      FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, PtCfg<HH>::SMEM_BYTES)); \
       attr_set[device] = true;                                                                                  \
     }                                                                                                           \
-    kern<<<grid, PT_THREADS, Cfg::SMEM_BYTES, stream>>>(                                                        \
+    kern<<<grid, PT_THREADS, PtCfg<HH>::SMEM_BYTES, stream>>>(                                                  \
         static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache),                \
-        static_cast<const __nv_bfloat16*>(q), block_table, ctx_len, static_cast<__nv_bfloat16*>(out),           \
-        part_o, part_ml, Hq, Hkv, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, status);         \
+        static_cast<const __nv_bfloat16*>(q), block_table, row_slot, ctx_len, static_cast<__nv_bfloat16*>(out), \
+        part_o, part_ml, Hq, Hkv, D, Dv, G, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, hg, status); \
   }
-    switch (G) {
-      case 1: FT_PT_LAUNCH(1) break;
-      case 2: FT_PT_LAUNCH(2) break;
-      case 4: FT_PT_LAUNCH(4) break;
-      default: FT_PT_LAUNCH(8) break;
-    }
+#define FT_PT_BY_G(HH)                     \
+  if (G == 1) FT_PT_LAUNCH(HH, 1)          \
+  else if (G == 2) FT_PT_LAUNCH(HH, 2)     \
+  else if (G <= 4) FT_PT_LAUNCH(HH, 4)     \
+  else if (G <= 8) FT_PT_LAUNCH(HH, 8)     \
+  else FT_PT_LAUNCH(HH, 16)
+    if (D > 64) { FT_PT_BY_G(128) } else { FT_PT_BY_G(64) }
+#undef FT_PT_BY_G
 #undef FT_PT_LAUNCH
-    FT_CUDA_CHECK(cudaGetLastError());
-    count_launch();
-    if (n_splits > 1) {
-      dim3 g2(Hq, B);
-      paged_decode_combine_kernel<128><<<g2, 128, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, ldo, n_splits);
-      FT_CUDA_CHECK(cudaGetLastError());
-      count_launch();
-    }
-    return FT_E_OK;
-  }
+  } else {
+    FT_REQUIRE((D == 64 || D == 128) && D == Dv, "ft_paged_decode: head sizes %d / %d not supported (multiples of 16 up to 128, 16-byte aligned rows)", D, Dv);
 #define FT_PD_LAUNCH(DD, GG)                                                                                   \
   paged_decode_kernel<DD, GG><<<grid, PD_THREADS, 0, stream>>>(                                                \
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),                        \
-      static_cast<const __nv_bfloat16*>(v_cache), block_table, ctx_len, static_cast<__nv_bfloat16*>(out),      \
-      part_o, part_ml, Hq, Hkv, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits)
+      static_cast<const __nv_bfloat16*>(v_cache), block_table, row_slot, ctx_len, static_cast<__nv_bfloat16*>(out), \
+      part_o, part_ml, Hq, Hkv, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, hg)
 #define FT_PD_BY_G(DD)                                             \
   switch (G) {                                                     \
     case 1: FT_PD_LAUNCH(DD, 1); break;                            \
@@ -662,19 +799,47 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
       set_last_error("ft_paged_decode: group size %d not supported (1, 2, 4, 8)", G); \
       return FT_E_BAD_ARG;                                         \
   }
-  if (D == 128) { FT_PD_BY_G(128) } else { FT_PD_BY_G(64) }
+    if (D == 128) { FT_PD_BY_G(128) } else { FT_PD_BY_G(64) }
 #undef FT_PD_BY_G
 #undef FT_PD_LAUNCH
+  }
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   if (n_splits > 1) {
     dim3 g2(Hq, B);
-    if (D == 128)
-      paged_decode_combine_kernel<128><<<g2, 128, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, ldo, n_splits);
-    else
-      paged_decode_combine_kernel<64><<<g2, 64, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, ldo, n_splits);
+    paged_decode_combine_kernel<<<g2, Dv <= 64 ? 64 : 128, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, Dv, ldo, n_splits, hg);
     FT_CUDA_CHECK(cudaGetLastError());
     count_launch();
   }
+  return FT_E_OK;
+}
+
+// Attention of arbitrary rows over the paged cache (see paged_rows_kernel): q [rows, Hq, D], out
+// [rows, Hq, Dv], row_slot / visible int32 [rows].  All tensors bf16, or fp32 with f32.
+FT_API int ft_paged_rows(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* row_slot,
+                         const int* visible, const void* gate, void* out, int rows, int Hq, int Hkv, int D, int Dv,
+                         long long ldq, long long ldg, long long ldo, int block_size, int max_blocks, int num_blocks,
+                         float scale, int f32, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(q && k_cache && v_cache && block_table && row_slot && visible && out, "ft_paged_rows: null pointer");
+  FT_REQUIRE(Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && D > 0 && Dv > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0, "ft_paged_rows: bad shape");
+  if (rows <= 0) return FT_E_OK;
+  const int groups = (Hq / Hkv + PR_HEADS - 1) / PR_HEADS;
+  const size_t smem = sizeof(float) * (static_cast<size_t>(PR_HEADS) * D + static_cast<size_t>(PD_WARPS) * PR_HEADS * Dv +
+                                       PD_WARPS * PR_HEADS * 32 + 2 * PD_WARPS * PR_HEADS);
+  FT_REQUIRE(smem <= 200 * 1024 && static_cast<long long>(Hkv) * groups < 65536, "ft_paged_rows: head sizes %d / %d are too large", D, Dv);
+  const dim3 grid(rows < 65536 ? rows : 65536, Hkv * groups);
+  const HeadGate hg = {gate, ldg};
+#define FT_PR_LAUNCH(T)                                                                                                      \
+  {                                                                                                                          \
+    FT_CUDA_CHECK(cudaFuncSetAttribute(paged_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
+    paged_rows_kernel<T><<<grid, PD_THREADS, smem, stream>>>(static_cast<const T*>(q), static_cast<const T*>(k_cache),       \
+        static_cast<const T*>(v_cache), block_table, row_slot, visible, hg, static_cast<T*>(out), rows, Hq, Hkv, D, Dv, ldq, \
+        ldo, block_size, max_blocks, num_blocks, scale, groups);                                                             \
+  }
+  if (f32) FT_PR_LAUNCH(float) else FT_PR_LAUNCH(__nv_bfloat16)
+#undef FT_PR_LAUNCH
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
   return FT_E_OK;
 }

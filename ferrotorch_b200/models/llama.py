@@ -242,6 +242,36 @@ class LlamaForCausalLM(nn.Module):
             h = h[:, -1:]
         return self.lm_head(h)
 
+    # ------------------------------------------------------------------ ragged batches over a paged cache (models.serving)
+    def make_paged_cache(self, num_blocks: int, block_size: int, max_seqs: int, max_seq_len: int):
+        from ..nn.paged import PagedKVCache
+
+        c, p = self.config, next(self.parameters())
+        return PagedKVCache(c.num_hidden_layers, c.num_key_value_heads, c.head_dim, num_blocks, max_seqs, max_seq_len, block_size,
+                            device=p.device, dtype=p.dtype)
+
+    @torch.no_grad()
+    def paged_forward(self, batch, cache) -> torch.Tensor:
+        """One pass over a :class:`~ferrotorch_b200.nn.paged.RaggedBatch`: logits of its wanted rows ``[wanted, vocab]``."""
+        m = self.model
+        x, delta = m.embed_tokens(batch.tokens[None]), None
+        for li, layer in enumerate(m.layers):
+            if delta is None:
+                h = layer.input_layernorm(x)
+            else:
+                h, x = layer.input_layernorm(x, delta)
+            attn = layer.self_attn
+            Hq, Hkv, D, T = attn.n_heads, attn.n_kv_heads, attn.head_dim, batch.n_rows
+            qkv = attn.qkv_proj(h).view(1, T, Hq + 2 * Hkv, D)
+            if attn.rope is not None:
+                qkv = attn.rope(qkv, positions=batch.positions, n_rot_heads=Hq + Hkv)
+            cache.append(li, qkv[0, :, Hq:Hq + Hkv], qkv[0, :, Hq + Hkv:], batch.positions, batch.slots)
+            a = cache.attend(li, qkv[0, :, :Hq], batch)
+            h, x = layer.post_attention_layernorm(x, attn.o_proj(a.view(1, T, Hq * D)))
+            delta = layer.mlp(h)
+        h, _ = m.norm(x, delta)
+        return self.lm_head(h[0].index_select(0, batch.last))
+
     # ------------------------------------------------------------------ the reference's id-level entry points
     def forward_from_ids(self, ids) -> torch.Tensor:
         """Logits ``[1, S, V]`` for one sequence of token ids (ferrotorch-llama/src/model.rs:223)."""

@@ -8,9 +8,9 @@ sequences and gives every step one flat token batch:
 
 * each running sequence contributes the tokens whose keys and values are not in the cache yet: one token when
   it is decoding, a chunk of its prompt (``prefill_chunk``) when it has just been admitted or was preempted;
-* the projections, the MLP and the norms run once over the flat batch; attention reads the pages: decoding
-  rows through :meth:`PagedKVCache.decode` (the paged-decode kernel on a device, row b reading the block table
-  of the sequence that owns it), prompt chunks through flash attention over the sequence's gathered pages;
+* the projections, the MLP and the norms run once over the flat batch; attention reads the pages
+  (:meth:`PagedKVCache.attend`): decoding rows through the paged-decode kernel, row b reading the block table of
+  the sequence that owns it, prompt chunks through the paged-prefill kernel;
 * pages are reserved as sequences grow; when the pool runs dry the most recently admitted sequence is preempted
   (its pages are freed, it re-enters the queue at the front and recomputes its prompt plus what it has generated),
   so the earliest requests always finish and the pool can be smaller than the sum of all contexts;
@@ -25,6 +25,10 @@ sequences and gives every step one flat token batch:
   of their tokens; a new request whose prompt starts with the same tokens adopts those pages (reference-counted
   in the pool) and computes only the rest.  Unused entries are evicted, deepest page of the least recently used
   chain first, before any sequence is preempted.
+
+The batcher schedules; :class:`PagedStepper` owns the cache and runs the steps.  It serves every model that offers
+``make_paged_cache`` and ``paged_forward`` (:mod:`~ferrotorch_b200.models.registry` lists them) and replays a step of
+single tokens as a captured CUDA graph when asked to.
 
 Greedy requests are sampled on the device in one ``argmax``; sampled requests carry their own generator, so
 the tokens of a request do not depend on which other requests share its steps.
@@ -43,8 +47,7 @@ from typing import Callable
 
 import torch
 
-from ..nn.paged import OutOfPages, PagedAttentionManager, PagedKVCache
-from ..ops.attention import flash_attention
+from ..nn.paged import DecodeBatch, OutOfPages, PagedAttentionManager, RaggedBatch
 from .generation import apply_repetition_penalty, filter_top_k_top_p
 
 
@@ -198,9 +201,82 @@ class PrefixCache:
         self._table.clear()
 
 
+class PagedStepper:
+    """The step function of a decoder over a paged cache: sequences are admitted, fed any number of tokens per step beside
+    one another, and released.  ``cuda_graph`` (device only): steps in which every sequence brings one token are captured
+    once per batch size (rounded up to a power of two, or a multiple of eight) and replayed."""
+
+    def __init__(self, model, num_blocks: int, block_size: int = 16, max_seqs: int = 64, max_seq_len: int | None = None,
+                 cuda_graph: bool = False):
+        self.model = model
+        self.max_seq_len = max_seq_len or model.config.max_position_embeddings or num_blocks * block_size
+        self.cache = model.make_paged_cache(num_blocks, block_size, max_seqs, self.max_seq_len)
+        self.manager = PagedAttentionManager(self.cache)
+        self.max_seqs = max_seqs
+        self.cuda_graph = cuda_graph and self.cache.device.type == "cuda"
+        self._graphs: dict = {}                           # rows -> (batch, graph, logits)
+        self.graph_replays = 0
+
+    def admit(self) -> int:
+        return self.manager.add_sequence(0)
+
+    def release(self, slot: int) -> None:
+        self.manager.remove_sequence(slot)
+
+    def length(self, slot: int) -> int:
+        return self.manager.active[slot]
+
+    def reserve(self, slot: int, new_len: int) -> None:
+        """Pages for the first ``new_len`` tokens of the sequence; raises :class:`OutOfPages`."""
+        self.cache.reserve(slot, new_len)
+        self.manager.active[slot] = max(self.manager.active[slot], new_len)
+
+    def feed(self, parts: list) -> torch.Tensor:
+        """``parts``: ``(slot, tokens, want)`` -- the next tokens of sequences and the places among them whose logits are
+        asked for.  Reserves their pages and runs one step; logits ``[wanted, vocab]`` in the order of the parts."""
+        entries = []
+        for slot, tokens, want in parts:
+            start = self.length(slot)
+            self.reserve(slot, start + len(tokens))
+            entries.append((slot, list(tokens), start, list(want)))
+        return self.step(entries)
+
+    def step(self, entries: list) -> torch.Tensor:
+        """One forward pass over ``(slot, tokens, first position, wanted places)`` entries whose pages are reserved."""
+        if self.cuda_graph and all(len(e[1]) == 1 and len(e[3]) == 1 for e in entries):
+            return self._step_graph(entries)
+        return self.model.paged_forward(RaggedBatch(entries, self.cache.device), self.cache)
+
+    def _graph_rows(self, n: int) -> int:
+        rows = 1 << max(0, n - 1).bit_length()
+        return rows if rows <= 8 else (n + 7) // 8 * 8
+
+    def _step_graph(self, entries: list) -> torch.Tensor:
+        n = len(entries)
+        rows = self._graph_rows(n)
+        self.cache.sync_table()                           # the only copy that a step makes outside the graph
+        got = self._graphs.get(rows)
+        if got is None:
+            batch = DecodeBatch(rows, self.cache.pad_slot, self.cache.device)
+            side = torch.cuda.Stream()
+            side.wait_stream(torch.cuda.current_stream())
+            with torch.cuda.stream(side):                 # sizes every scratch buffer; rows of no sequence write nothing
+                self.model.paged_forward(batch, self.cache)
+            torch.cuda.current_stream().wait_stream(side)
+            graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(graph):
+                logits = self.model.paged_forward(batch, self.cache)
+            got = self._graphs[rows] = (batch, graph, logits)
+        batch, graph, logits = got
+        batch.load([e[1][0] for e in entries], [e[2] for e in entries], [e[0] for e in entries])
+        graph.replay()
+        self.graph_replays += 1
+        return logits[:n].clone()
+
+
 class ContinuousBatcher:
-    """Serve requests on ``model`` (a :class:`~ferrotorch_b200.models.llama.LlamaForCausalLM`) with a paged cache
-    of ``num_blocks`` pages of ``block_size`` tokens.
+    """Serve requests on ``model`` (a :class:`~ferrotorch_b200.models.llama.LlamaForCausalLM` or any other that
+    :class:`PagedStepper` can run) with a paged cache of ``num_blocks`` pages of ``block_size`` tokens.
 
     ``max_running``: sequence slots; ``max_tokens_per_step``: size limit of a step's flat batch;
     ``prefill_chunk``: most prompt tokens one sequence contributes to one step (long prompts are spread over
@@ -209,14 +285,10 @@ class ContinuousBatcher:
 
     def __init__(self, model, num_blocks: int, block_size: int = 16, max_running: int = 64, max_seq_len: int | None = None,
                  max_tokens_per_step: int = 2048, prefill_chunk: int = 512, watermark: float = 0.01,
-                 prefix_caching: bool = False):
-        cfg = model.config
-        p = next(model.parameters())
+                 prefix_caching: bool = False, cuda_graph: bool = False):
         self.model = model
-        self.max_seq_len = max_seq_len or cfg.max_position_embeddings
-        self.cache = PagedKVCache(cfg.num_hidden_layers, cfg.num_key_value_heads, cfg.head_dim, num_blocks, max_running,
-                                  self.max_seq_len, block_size, device=p.device, dtype=p.dtype)
-        self.manager = PagedAttentionManager(self.cache)
+        self.stepper = PagedStepper(model, num_blocks, block_size, max_running, max_seq_len, cuda_graph)
+        self.max_seq_len, self.cache, self.manager = self.stepper.max_seq_len, self.stepper.cache, self.stepper.manager
         self.max_running, self.max_tokens_per_step, self.prefill_chunk = max_running, max_tokens_per_step, prefill_chunk
         if max_tokens_per_step < 1 or prefill_chunk < 1:
             raise ValueError("ContinuousBatcher: max_tokens_per_step and prefill_chunk must be at least 1")
@@ -301,8 +373,7 @@ class ContinuousBatcher:
         False if ``r`` itself had to give way."""
         while True:
             try:
-                self.cache.reserve(r.slot, new_len)
-                self.manager.active[r.slot] = max(self.manager.active[r.slot], new_len)
+                self.stepper.reserve(r.slot, new_len)
                 return True
             except OutOfPages:
                 if self.prefix is not None and self.prefix.evict(1):
@@ -368,12 +439,11 @@ class ContinuousBatcher:
             if need > self.manager.free_pages:
                 break
             self.waiting.popleft()
-            r.slot = self.manager.add_sequence(0)
+            r.slot = self.stepper.admit()
             if shared:
                 self.cache.adopt(r.slot, shared, start)
                 self.stats.prefix_hit_tokens += start
-            self.cache.reserve(r.slot, start + n)
-            self.manager.active[r.slot] = start + n
+            self.stepper.reserve(r.slot, start + n)
             r.computed = start
             r.state, r._admitted_at = RequestState.RUNNING, self.stats.steps
             self.running.append(r)
@@ -382,55 +452,13 @@ class ContinuousBatcher:
         return runs
 
     # ------------------------------------------------------------------ one forward over the flat batch
-    def _attention(self, attn, layer: int, h: torch.Tensor, pos: torch.Tensor, sid: torch.Tensor, spans: list) -> torch.Tensor:
-        T = h.shape[1]
-        Hq, Hkv, D = attn.n_heads, attn.n_kv_heads, attn.head_dim
-        qkv = attn.qkv_proj(h).view(1, T, Hq + 2 * Hkv, D)
-        if attn.rope is not None:
-            qkv = attn.rope(qkv, positions=pos, n_rot_heads=Hq + Hkv)
-        q, k, v = qkv[0, :, :Hq], qkv[0, :, Hq:Hq + Hkv], qkv[0, :, Hq + Hkv:]
-        self.cache.append(layer, k, v, pos, sid)
-        out = torch.empty((T, Hq, D), device=h.device, dtype=h.dtype)
-        single = [row for (_, row, _, n) in spans if n == 1]
-        if single:
-            idx = torch.tensor(single, device=h.device, dtype=torch.long)
-            qd = q.index_select(0, idx).contiguous()
-            out[idx] = self.cache.decode(layer, qd, (pos.index_select(0, idx) + 1).to(torch.int32), seq_ids=sid.index_select(0, idx))
-        for slot, row, start, n in spans:
-            if n > 1:
-                kk, vv = self.cache.gather(layer, slot, start + n)
-                out[row:row + n] = flash_attention(q[None, row:row + n].contiguous(), kk[None], vv[None], causal=True)[0]
-        return attn.o_proj(out.reshape(1, T, Hq * D))
-
-    @torch.no_grad()
     def _forward(self, runs: list) -> torch.Tensor:
         """Logits of the last token of every run (of its last ``1 + len(draft)`` tokens when it speculates), run after run."""
-        dev = self.cache.device
-        toks, poss, sids, spans, last, row = [], [], [], [], [], 0
+        entries = []
         for r, start, n in runs:
             draft = self._drafts.get(r.id, [])
-            seq = r.tokens() + draft
-            toks += seq[start:start + n]
-            poss += range(start, start + n)
-            sids += [r.slot] * n
-            spans.append((r.slot, row, start, n))
-            row += n
-            last += range(row - 1 - len(draft), row)
-        tok = torch.tensor(toks, dtype=torch.long, device=dev)
-        pos = torch.tensor(poss, dtype=torch.int32, device=dev)
-        sid = torch.tensor(sids, dtype=torch.int32, device=dev)
-        m = self.model.model
-        x, delta = m.embed_tokens(tok[None]), None
-        for li, layer in enumerate(m.layers):
-            if delta is None:
-                h = layer.input_layernorm(x)
-            else:
-                h, x = layer.input_layernorm(x, delta)
-            a = self._attention(layer.self_attn, li, h, pos, sid, spans)
-            h, x = layer.post_attention_layernorm(x, a)
-            delta = layer.mlp(h)
-        h, _ = m.norm(x, delta)
-        return self.model.lm_head(h[0, torch.tensor(last, device=dev)])
+            entries.append((r.slot, (r.tokens() + draft)[start:start + n], start, list(range(n - 1 - len(draft), n))))
+        return self.stepper.step(entries)
 
     def _sample(self, requests: list, logits: torch.Tensor) -> list:
         greedy = [i for i, r in enumerate(requests)

@@ -4,7 +4,11 @@ Bookkeeping mirrors the reference (ferrotorch-nn/src/paged_attention.rs:155-532)
 ``PagePool`` with O(1) allocate / free, a per-sequence page list, and a manager that adds,
 extends and drops sequences.  Unlike the reference, the pages are device memory
 (``[num_blocks, block_size, n_kv_heads, head_dim]`` for K and for V, per layer) and the block
-table is a device tensor read by ``ft_kv_append`` / ``ft_paged_decode`` (``csrc/paged_attn.cu``).
+table is a device tensor read by ``ft_kv_append`` / ``ft_paged_decode`` (``csrc/paged_attn.cu``) and
+``ft_paged_prefill`` (``csrc/paged_prefill.cu``).
+
+A forward pass over the cache works on a :class:`RaggedBatch`: any number of sequences, each with any number
+of new tokens, as one flat list of rows.  :meth:`PagedKVCache.attend` is its attention.
 """
 from __future__ import annotations
 
@@ -12,12 +16,16 @@ import torch
 
 from .. import _native
 from ..ops import functional as F
+from ..ops import reference as ref
 
 _i, _ll, _f, _vp = _native._i, _native._ll, _native._f, _native._vp
 _native.register_protos({
     "ft_kv_append": (_i, [_vp] * 7 + [_i, _i, _i, _i, _ll, _ll, _i, _i, _i, _i, _vp]),
     "ft_paged_decode_scratch": (_ll, [_i, _i, _i, _i]),
-    "ft_paged_decode": (_i, [_vp] * 7 + [_i, _i, _i, _i, _ll, _ll, _i, _i, _i, _f, _i, _i, _vp]),
+    "ft_paged_decode": (_i, [_vp] * 9 + [_i] * 5 + [_ll] * 3 + [_i, _i, _i, _f, _i, _i, _vp]),
+    "ft_paged_rows": (_i, [_vp] * 8 + [_i] * 5 + [_ll] * 3 + [_i, _i, _i, _f, _i, _i, _vp]),
+    "ft_paged_prefill_tile": (_i, [_i]),
+    "ft_paged_prefill": (_i, [_vp] * 7 + [_i] * 6 + [_ll] * 3 + [_i, _i, _i, _f, _i, _vp]),
 })
 
 
@@ -79,21 +87,107 @@ class PagePool:
         return self.num_pages
 
 
+class RaggedBatch:
+    """The rows of one forward pass: ``entries`` are ``(slot, tokens, start, want)`` -- a sequence slot, its next
+    token ids, the position of the first of them, and the places among them whose logits are asked for.
+
+    Entries of one token come first (:attr:`n_single` rows, the decode kernel's batch), longer ones after them
+    (:attr:`spans`, the prefill kernel's portions); ``last`` lists the wanted rows in the order of the entries as
+    they were given.  Everything the kernels read is copied to the device in one transfer."""
+
+    def __init__(self, entries: list, device):
+        self.device = torch.device(device)
+        order = [i for i, e in enumerate(entries) if len(e[1]) == 1]
+        self.n_single = len(order)
+        order += [i for i, e in enumerate(entries) if len(e[1]) > 1]
+        toks, pos, slots, self.spans, first_row, row = [], [], [], [], {}, 0
+        for i in order:
+            slot, tokens, start, _ = entries[i]
+            n = len(tokens)
+            first_row[i] = row
+            toks += tokens
+            pos += range(start, start + n)
+            slots += [slot] * n
+            if n > 1:
+                self.spans.append((slot, row, start, n))
+            row += n
+        want = [first_row[i] + w for i, e in enumerate(entries) if len(e[1]) for w in e[3]]
+        self.n_rows, self.n_want = row, len(want)
+        self._fill(toks, pos, slots, [p + 1 for p in pos], want)
+        self._items: dict = {}
+
+    def _fill(self, toks, pos, slots, visible, want) -> None:
+        """One buffer: token ids and wanted rows as int64, then positions, slots and visible-key counts as int32."""
+        n, m = len(toks), len(want)
+        host = torch.empty(n + m + (3 * n + 1) // 2, dtype=torch.long, pin_memory=self.device.type == "cuda")
+        host[:n + m] = torch.tensor(toks + want, dtype=torch.long)
+        host[n + m:].view(torch.int32)[:3 * n] = torch.tensor(pos + slots + visible, dtype=torch.int32)
+        self._buf = host.to(self.device, non_blocking=True)
+        self._host = host                                  # the pinned source lives as long as the batch
+        ints = self._buf[n + m:].view(torch.int32)
+        self.tokens, self.last = self._buf[:n], self._buf[n:n + m]
+        self.positions, self.slots, self.visible = ints[:n], ints[n:2 * n], ints[2 * n:3 * n]
+
+    def work_items(self, tile_tokens: int):
+        """The portions cut into work items of the prefill kernel (``[n, 4]`` int32 on the device: slot, first row,
+        tokens, first position; at most ``2 * tile_tokens`` tokens each), longest key range first."""
+        got = self._items.get(tile_tokens)
+        if got is None:
+            rows, step = [], 2 * tile_tokens
+            for slot, row, start, n in self.spans:
+                rows += [(slot, row + o, min(step, n - o), start + o) for o in range(0, n, step)]
+            rows.sort(key=lambda r: -(r[2] + r[3]))
+            host = torch.tensor(rows, dtype=torch.int32)
+            got = host.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else host
+            self._items[tile_tokens] = got
+        return got
+
+
+class DecodeBatch(RaggedBatch):
+    """A batch of single-token rows whose device tensors keep their addresses, for captured decode steps: ``rows``
+    rows, of which :meth:`load` fills some; the others belong to no sequence (no visible key, no page)."""
+
+    def __init__(self, rows: int, pad_slot: int, device):
+        self.device = torch.device(device)
+        self.n_single = self.n_rows = self.n_want = rows
+        self.spans, self._items, self.pad_slot = [], {}, pad_slot
+        self._fill([0] * rows, [0] * rows, [pad_slot] * rows, [0] * rows, list(range(rows)))
+        self._static = self._buf
+
+    def load(self, tokens: list, positions: list, slots: list) -> None:
+        pad = self.n_rows - len(tokens)
+        views = (self.tokens, self.last, self.positions, self.slots, self.visible)
+        self._fill(tokens + [0] * pad, positions + [0] * pad, slots + [self.pad_slot] * pad,
+                   [p + 1 for p in positions] + [0] * pad, list(range(self.n_rows)))
+        self._static.copy_(self._buf)
+        self._buf = self._static
+        self.tokens, self.last, self.positions, self.slots, self.visible = views
+
+
 class PagedKVCache:
     """Block tables for up to ``max_seqs`` sequences over one :class:`PagePool`, plus the device
-    K/V pages of every layer.  ``block_size`` tokens per page (16 in the benchmark configs)."""
+    K/V pages of every layer.  ``block_size`` tokens per page (16 in the benchmark configs).
+    ``n_kv_heads``, ``head_dim`` and ``v_head_dim`` (default: ``head_dim``) are numbers, or one number per layer."""
 
-    def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, num_blocks: int, max_seqs: int,
-                 max_seq_len: int, block_size: int = 16, device="cuda", dtype=torch.bfloat16):
-        self.n_layers, self.n_kv_heads, self.head_dim = n_layers, n_kv_heads, head_dim
+    def __init__(self, n_layers: int, n_kv_heads, head_dim, num_blocks: int, max_seqs: int,
+                 max_seq_len: int, block_size: int = 16, device="cuda", dtype=torch.bfloat16, v_head_dim=None):
+        def per_layer(v):
+            return [int(v)] * n_layers if isinstance(v, int) else [int(x) for x in v]
+
+        self.shapes = list(zip(per_layer(n_kv_heads), per_layer(head_dim), per_layer(head_dim if v_head_dim is None else v_head_dim)))
+        if len(self.shapes) != n_layers:
+            raise ValueError("PagedKVCache: %d layer shapes for %d layers" % (len(self.shapes), n_layers))
+        self.n_layers, self.dtype = n_layers, dtype
+        self.n_kv_heads, self.head_dim = self.shapes[0][:2] if self.shapes else (0, 0)
         self.block_size, self.num_blocks, self.max_seqs = block_size, num_blocks, max_seqs
         self.max_blocks = (max_seq_len + block_size - 1) // block_size
         self.device = torch.device(device)
         self.pool = PagePool(num_blocks)
-        shape = (num_blocks, block_size, n_kv_heads, head_dim)
-        self.k = [torch.zeros(shape, device=self.device, dtype=dtype) for _ in range(n_layers)]
-        self.v = [torch.zeros(shape, device=self.device, dtype=dtype) for _ in range(n_layers)]
-        self._table_host = torch.full((max_seqs, self.max_blocks), -1, dtype=torch.int32)
+        self.k = [torch.zeros((num_blocks, block_size, h, d), device=self.device, dtype=dtype) for h, d, _ in self.shapes]
+        self.v = [torch.zeros((num_blocks, block_size, h, dv), device=self.device, dtype=dtype) for h, _, dv in self.shapes]
+        # one row more than there are sequences: the padding rows of a captured decode step own no page
+        self.pad_slot = max_seqs
+        self._table_host = torch.full((max_seqs + 1, self.max_blocks), -1, dtype=torch.int32)
         self.block_table = self._table_host.to(self.device)
         self._pages: list[list[int]] = [[] for _ in range(max_seqs)]
         self.lengths = [0] * max_seqs
@@ -150,10 +244,11 @@ class PagedKVCache:
         sequence ``seq_ids[i]`` or ``i // tokens_per_seq``.  Pages must have been reserved."""
         T = k_new.shape[0]
         table = self.sync_table()
-        if not k_new.is_cuda:
-            sid = (seq_ids if seq_ids is not None else torch.arange(T) // tokens_per_seq).long()
+        Hkv, D, Dv = self.shapes[layer]
+        if not k_new.is_cuda or self.dtype != torch.bfloat16 or D != Dv:
+            sid = (seq_ids if seq_ids is not None else torch.arange(T, device=k_new.device) // tokens_per_seq).long()
             pos = positions.long()
-            blk = self._table_host[sid, pos // self.block_size].long()
+            blk = self._table_host[sid.cpu(), (pos // self.block_size).cpu()].long().to(k_new.device)
             if bool((blk < 0).any()):
                 raise ValueError("PagedKVCache.append: a position has no page (reserve the sequence first)")
             self.k[layer][blk, pos % self.block_size] = k_new.to(self.k[layer].dtype)
@@ -164,43 +259,107 @@ class PagedKVCache:
         rc = _native.kernels().ft_kv_append(
             k_new.data_ptr(), v_new.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(),
             table.data_ptr(), positions.data_ptr(), seq_ids.data_ptr() if seq_ids is not None else None, T,
-            tokens_per_seq, self.n_kv_heads, self.head_dim, ldk, ldv, self.block_size, self.max_blocks,
+            tokens_per_seq, Hkv, D, ldk, ldv, self.block_size, self.max_blocks,
             self.num_blocks, F._dev(k_new), F._stream())
         _native.check(rc, "ft_kv_append")
 
+    def _tensor_core_ok(self, layer: int, q: torch.Tensor, max_group: int) -> bool:
+        Hkv, D, Dv = self.shapes[layer]
+        return (q.dtype == torch.bfloat16 and D % 16 == 0 and Dv % 16 == 0 and D <= 128 and Dv <= 128
+                and q.shape[1] // Hkv <= max_group and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0)
+
+    def _rows(self, layer: int, q, visible, slots, scale, gate, out) -> None:
+        """Attention of arbitrary rows, any head sizes, bf16 or fp32 (the simple kernel)."""
+        T, Hq, D = q.shape
+        Hkv, _, Dv = self.shapes[layer]
+        rc = _native.kernels().ft_paged_rows(
+            q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), self.block_table.data_ptr(), slots.data_ptr(),
+            visible.data_ptr(), gate.data_ptr() if gate is not None else None, out.data_ptr(), T, Hq, Hkv, D, Dv, q.stride(0),
+            gate.stride(0) if gate is not None else 0, out.stride(0), self.block_size, self.max_blocks, self.num_blocks, float(scale),
+            int(q.dtype == torch.float32), F._dev(q), F._stream())
+        _native.check(rc, "ft_paged_rows")
+
     def decode(self, layer: int, q: torch.Tensor, ctx_len: torch.Tensor, scale: float | None = None,
-               n_splits: int = 0, seq_ids: torch.Tensor | None = None) -> torch.Tensor:
-        """One query token per sequence: ``q [B, Hq, D]``, ``ctx_len [B]`` int32 -> ``[B, Hq, D]``.  Row b
-        reads sequence b, or sequence ``seq_ids[b]`` (a batch of any subset of the live sequences: the rows of
-        the block table are gathered in that order)."""
+               n_splits: int = 0, seq_ids: torch.Tensor | None = None, gate: torch.Tensor | None = None,
+               out: torch.Tensor | None = None) -> torch.Tensor:
+        """One query token per sequence: ``q [B, Hq, D]``, ``ctx_len [B]`` int32 -> ``[B, Hq, Dv]``.  Row b
+        reads sequence b, or sequence ``seq_ids[b]`` (int32; a batch of any subset of the live sequences).
+        ``gate [B, Hq]``: output heads are multiplied by its sigmoid.  ``out``: where the result goes (the heads of a
+        row packed, any row stride)."""
         B, Hq, D = q.shape
+        Hkv, _, Dv = self.shapes[layer]
         scale = scale if scale is not None else D ** -0.5
         table = self.sync_table()
         if not q.is_cuda:
-            return self._decode_reference(layer, q, ctx_len, scale, seq_ids)
-        if seq_ids is not None:
-            table = table.index_select(0, seq_ids.to(device=table.device, dtype=torch.long)).contiguous()
+            o = self._decode_reference(layer, q, ctx_len, scale, seq_ids)
+            o = o if gate is None else ref.head_gate(o, gate)
+            return o if out is None else out.copy_(o)
+        if out is None:
+            out = torch.empty((B, Hq, Dv), device=q.device, dtype=q.dtype)
+        seq_ids = seq_ids.to(device=q.device, dtype=torch.int32) if seq_ids is not None else None
+        if not self._tensor_core_ok(layer, q, 16) and (q.dtype != torch.bfloat16 or D != Dv or D not in (64, 128)
+                                                       or Hq // Hkv not in (1, 2, 4, 8)):
+            rows = seq_ids if seq_ids is not None else torch.arange(B, device=q.device, dtype=torch.int32)
+            self._rows(layer, q, ctx_len, rows, scale, gate, out)
+            return out
         lib = _native.kernels()
         if n_splits <= 0:
-            ctas = B * self.n_kv_heads
+            ctas = B * Hkv
             n_splits = 1 if ctas >= 256 else max(1, min(8, 296 // max(ctas, 1)))
-        out = torch.empty(q.shape, device=q.device, dtype=q.dtype)
-        n_scr = int(lib.ft_paged_decode_scratch(B, Hq, D, n_splits))
+        n_scr = int(lib.ft_paged_decode_scratch(B, Hq, Dv, n_splits))
         scratch = F._get_scratch("paged_decode", n_scr, q.device) if n_scr else None
         rc = lib.ft_paged_decode(q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), table.data_ptr(),
-                                 ctx_len.data_ptr(), out.data_ptr(), scratch.data_ptr() if scratch is not None else None,
-                                 B, Hq, self.n_kv_heads, D, q.stride(0), out.stride(0), self.block_size,
+                                 seq_ids.data_ptr() if seq_ids is not None else None, ctx_len.data_ptr(),
+                                 gate.data_ptr() if gate is not None else None, out.data_ptr(),
+                                 scratch.data_ptr() if scratch is not None else None, B, Hq, Hkv, D, Dv, q.stride(0),
+                                 gate.stride(0) if gate is not None else 0, out.stride(0), self.block_size,
                                  self.max_blocks, self.num_blocks, float(scale), n_splits, F._dev(q), F._stream())
         _native.check(rc, "ft_paged_decode")
         return out
 
+    def attend(self, layer: int, q: torch.Tensor, batch: RaggedBatch, scale: float | None = None,
+               gate: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+        """Causal attention of a whole :class:`RaggedBatch` (its keys and values already appended): ``q [T, Hq, D]`` ->
+        ``[T, Hq, Dv]``.  Single tokens run on the decode kernel, longer portions on the prefill kernel; head sizes or
+        types that those do not cover run on the simple kernel."""
+        T, Hq, D = q.shape
+        Hkv, _, Dv = self.shapes[layer]
+        scale = scale if scale is not None else D ** -0.5
+        if out is None:
+            out = torch.empty((T, Hq, Dv), device=q.device, dtype=q.dtype)
+        table = self.sync_table()
+        n1 = batch.n_single
+        if n1:
+            self.decode(layer, q[:n1], batch.visible[:n1], scale, seq_ids=batch.slots[:n1],
+                        gate=gate[:n1] if gate is not None else None, out=out[:n1])
+        if not batch.spans:
+            return out
+        if not q.is_cuda:
+            for slot, row, start, n in batch.spans:
+                k, v = self.gather(layer, slot, start + n)
+                o = ref.attention(q[None, row:row + n], k[None], v[None], True, scale, start)[0][0]
+                out[row:row + n] = o if gate is None else ref.head_gate(o, gate[row:row + n])
+            return out
+        bs = self.block_size
+        if not (self._tensor_core_ok(layer, q, 128) and scale > 0 and bs >= 8 and (128 % bs == 0 or bs % 128 == 0)):
+            self._rows(layer, q[n1:], batch.visible[n1:], batch.slots[n1:], scale, gate[n1:] if gate is not None else None, out[n1:])
+            return out
+        lib = _native.kernels()
+        items = batch.work_items(int(lib.ft_paged_prefill_tile(Hq // Hkv)))
+        rc = lib.ft_paged_prefill(q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), table.data_ptr(), items.data_ptr(),
+                                  gate.data_ptr() if gate is not None else None, out.data_ptr(), items.shape[0], T, Hq, Hkv, D, Dv,
+                                  q.stride(0), gate.stride(0) if gate is not None else 0, out.stride(0), bs, self.max_blocks,
+                                  self.num_blocks, float(scale), F._dev(q), F._stream())
+        _native.check(rc, "ft_paged_prefill")
+        return out
+
     def gather(self, layer: int, seq: int, length: int):
-        """Contiguous ``[length, Hkv, D]`` K and V of one sequence (debug / reference path;
+        """Contiguous ``[length, Hkv, D]`` K and ``[length, Hkv, Dv]`` V of one sequence (debug / reference path;
         paged_attention.rs ``get_keys`` / ``get_values``)."""
         pages = self._pages[seq][: (length + self.block_size - 1) // self.block_size]
         idx = torch.tensor(pages, device=self.k[layer].device, dtype=torch.long)
-        k = self.k[layer][idx].reshape(-1, self.n_kv_heads, self.head_dim)[:length]
-        v = self.v[layer][idx].reshape(-1, self.n_kv_heads, self.head_dim)[:length]
+        k = self.k[layer][idx].flatten(0, 1)[:length]
+        v = self.v[layer][idx].flatten(0, 1)[:length]
         return k, v
 
     # ---- accessors under the reference's names (paged_attention.rs:359-395; there one object per
@@ -235,15 +394,15 @@ class PagedKVCache:
         ctx = ctx_len.long().cpu()
         n_blk = int((int(ctx.max()) + self.block_size - 1) // self.block_size)
         pages = self._table_host[rows, :n_blk].long().clamp_(min=0)          # unreserved slots read page 0 and are masked
-        k = self.k[layer][pages].reshape(B, n_blk * self.block_size, self.n_kv_heads, D).float()
-        v = self.v[layer][pages].reshape(B, n_blk * self.block_size, self.n_kv_heads, D).float()
-        g = Hq // self.n_kv_heads
-        qf = q.float().reshape(B, self.n_kv_heads, g, D)
+        Hkv, _, Dv = self.shapes[layer]
+        k = self.k[layer][pages].reshape(B, n_blk * self.block_size, Hkv, D).float()
+        v = self.v[layer][pages].reshape(B, n_blk * self.block_size, Hkv, Dv).float()
+        qf = q.float().reshape(B, Hkv, Hq // Hkv, D)
         s = torch.einsum("bhgd,blhd->bhgl", qf, k) * scale
         dead = torch.arange(n_blk * self.block_size)[None] >= ctx[:, None]
         s = s.masked_fill(dead[:, None, None, :], float("-inf"))
         o = torch.einsum("bhgl,blhd->bhgd", torch.softmax(s, -1), v)
-        return o.reshape(B, Hq, D).to(q.dtype)
+        return o.reshape(B, Hq, Dv).to(q.dtype)
 
 
 class PagedAttentionManager:
@@ -325,3 +484,29 @@ class PagedAttentionManager:
         if seq_id not in self.active:
             raise ValueError("PagedAttentionManager: invalid sequence id %d" % seq_id)
         return self.cache.gather(layer, seq_id, self._filled.get(seq_id, {}).get(layer, self.active[seq_id]))
+
+
+class PagedSession:
+    """A fixed set of equally long sequences on a paged cache of their own, for callers that think in ``[B, S]`` tensors
+    (``models.generation``).  ``model`` offers ``make_paged_cache`` and ``paged_forward``."""
+
+    def __init__(self, model, batch: int, max_len: int, block_size: int = 16):
+        pages = batch * ((max_len + block_size - 1) // block_size)
+        self.model, self.len = model, 0
+        self.cache = model.make_paged_cache(pages, block_size, batch, max_len)
+        self.manager = PagedAttentionManager(self.cache)
+        self.slots = [self.manager.add_sequence(0) for _ in range(batch)]
+
+    def extend(self, input_ids: torch.Tensor, last_token_only: bool = False) -> torch.Tensor:
+        """Append ``input_ids [B, S]`` to the sequences; logits ``[B, S or 1, V]``."""
+        B, S = input_ids.shape
+        if B != len(self.slots):
+            raise ValueError("PagedSession: %d sequences, got a batch of %d" % (len(self.slots), B))
+        want = [S - 1] if last_token_only else list(range(S))
+        entries = []
+        for slot, tokens in zip(self.slots, input_ids.tolist()):
+            self.manager.extend(slot, S)
+            entries.append((slot, tokens, self.len, want))
+        self.len += S
+        logits = self.model.paged_forward(RaggedBatch(entries, self.cache.device), self.cache)
+        return logits.view(B, len(want), -1)

@@ -331,6 +331,140 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float = 1e-5,
     return _RMSNormFn.apply(x, weight, eps, residual)
 
 
+# --------------------------------------------------------------------------- dynamic tanh and packed decoder rows
+_native.register_protos({
+    "ft_dyt_fwd": (_native._i, [_native._vp] * 2 + [_native._i] * 2 + [_native._vp] * 5 + [_native._i] * 3 + [_native._ll] * 2 +
+                   [_native._f, _native._i, _native._vp]),
+    "ft_qkv_finish": (_native._i, [_native._vp, _native._ll] + [_native._vp] * 8 + [_native._ll] + [_native._i] * 11 + [_native._f] * 3 +
+                      [_native._i] * 6 + [_native._vp]),
+    "ft_gemm_small_m_f32": (_native._i, [_native._vp] * 3 + [_native._i] + [_native._vp] * 4 + [_native._f, _native._vp] + [_native._i] * 3 +
+                            [_native._ll] * 4 + [_native._i] * 2 + [_native._vp]),
+})
+
+
+def dynamic_tanh(x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, *, scale: float = 1.0,
+                 out_dtype: torch.dtype | None = None) -> torch.Tensor:
+    """``(tanh(alpha x) w + b) * scale`` of the fp32 residual rows ``x [T, H]`` (parameters fp32, ``alpha`` a scalar)."""
+    dt = out_dtype or x.dtype
+    if not x.is_cuda:
+        return ref.dynamic_tanh(x, alpha, weight, bias, scale).to(dt)
+    y = torch.empty(x.shape, device=x.device, dtype=dt)
+    rc = _native.kernels().ft_dyt_fwd(x.data_ptr(), None, 0, int(x.dtype == torch.bfloat16), None, alpha.data_ptr(), weight.data_ptr(),
+                                      bias.data_ptr(), y.data_ptr(), int(dt == torch.float32), x.shape[0], x.shape[1], x.stride(0),
+                                      y.stride(0), float(scale), _dev(x), _stream())
+    _native.check(rc, "ft_dyt_fwd")
+    return y
+
+
+def embedding_dynamic_tanh(ids: torch.Tensor, table: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, *,
+                           out_dtype: torch.dtype | None = None):
+    """The gathered rows as the fp32 residual stream, and their dynamic tanh, from one kernel: ``(x, h)``."""
+    dt = out_dtype or table.dtype
+    if not table.is_cuda:
+        x = table[ids].float()
+        return x, ref.dynamic_tanh(x, alpha, weight, bias).to(dt)
+    T, H = ids.numel(), table.shape[1]
+    x = torch.empty((T, H), device=table.device, dtype=torch.float32)
+    h = torch.empty((T, H), device=table.device, dtype=dt)
+    rc = _native.kernels().ft_dyt_fwd(table.data_ptr(), ids.data_ptr(), table.shape[0], int(table.dtype == torch.bfloat16), x.data_ptr(),
+                                      alpha.data_ptr(), weight.data_ptr(), bias.data_ptr(), h.data_ptr(), int(dt == torch.float32), T, H,
+                                      table.stride(0), h.stride(0), 1.0, _dev(table), _stream())
+    _native.check(rc, "ft_dyt_fwd")
+    return x, h
+
+
+def qkv_finish(packed: torch.Tensor, cache, layer: int, batch, *, q: tuple, k: tuple, v: tuple, up: tuple = (0, 0),
+               q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, q_count: int = 0, k_count: int = 0,
+               eps: float = 1e-5, temp_coef: float = 0.0, temp_every: float = 1.0, act_out: torch.Tensor | None = None,
+               activation: str = "gelu") -> None:
+    """Everything between a layer's packed input projection ``[T, N]`` and its attention, in one kernel.  ``q``, ``k``, ``v``,
+    ``up`` are ``(offset, size)`` of the segments of a row: q and k are RMS-normalised over the whole projection (``q_count`` /
+    ``k_count`` true elements, the rest zero padding), q is scaled by the query temperature in place, k and v go to their cache
+    pages, ``activation(up)`` goes to ``act_out``."""
+    cache.sync_table()
+    if not packed.is_cuda:
+        qs, ks, vs = (packed[:, o:o + n] for o, n in (q, k, v))
+        qf, kf = qs.float(), ks.float()
+        if q_weight is not None:
+            qf = ref.projection_rms(qs, q_weight, eps, q_count)
+        if k_weight is not None:
+            kf = ref.projection_rms(ks, k_weight, eps, k_count)
+        if temp_coef:
+            qf = qf * ref.query_temperature(batch.positions, temp_coef, temp_every)[:, None]
+        if up[1]:
+            act_out.copy_(ref._ACTS[_ACT_ID[activation]](packed[:, up[0]:up[0] + up[1]].float()))
+        Hkv, D, Dv = cache.shapes[layer]
+        cache.append(layer, kf.view(-1, Hkv, D), vs.reshape(-1, Hkv, Dv), batch.positions, batch.slots)
+        qs.copy_(qf)
+        return
+    rc = _native.kernels().ft_qkv_finish(
+        packed.data_ptr(), packed.stride(0), batch.positions.data_ptr(), batch.slots.data_ptr(), cache.block_table.data_ptr(),
+        cache.k[layer].data_ptr(), cache.v[layer].data_ptr(), q_weight.data_ptr() if q_weight is not None else None,
+        k_weight.data_ptr() if k_weight is not None else None, act_out.data_ptr() if up[1] else None,
+        act_out.stride(0) if up[1] else 0, packed.shape[0], q[0], q[1], k[0], k[1], v[0], v[1], up[0], up[1],
+        q_count or q[1], k_count or k[1], float(eps), float(temp_coef), float(temp_every), _ACT_ID[activation],
+        int(packed.dtype == torch.float32), cache.block_size, cache.max_blocks, cache.num_blocks, _dev(packed), _stream())
+    _native.check(rc, "ft_qkv_finish")
+
+
+def _mm_f32(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``a @ w.T`` in true 32-bit, whatever the process allows for fp32 matrix products."""
+    old = torch.backends.cuda.matmul.allow_tf32
+    torch.backends.cuda.matmul.allow_tf32 = False
+    try:
+        return torch.matmul(a, w.t())
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = old
+
+
+def linear_rows(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``a [T, K] @ w.T`` for inference in the type of its operands (bf16 on the tcgen05 GEMM, fp32 as true fp32)."""
+    return gemm_nt(a, w) if a.dtype == torch.bfloat16 else _mm_f32(a, w)
+
+
+def _small_m_shape(a: torch.Tensor, w: torch.Tensor) -> bool:
+    return a.is_cuda and a.dtype == torch.bfloat16 and a.shape[0] <= 128 and w.shape[0] >= 1024 and w.shape[1] >= 512
+
+
+def _small_m_f32(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool, norm: tuple | None) -> torch.Tensor | None:
+    (M, K), N = a.shape, w.shape[0]
+    lib = _native.kernels()
+    ws = _small_m_workspace(int(lib.ft_gemm_small_m_workspace(M, N)), a.device)
+    h = torch.empty((M, N), device=a.device, dtype=torch.bfloat16) if norm is not None else None
+    alpha, nw, nb, scale = norm if norm is not None else (None, None, None, 1.0)
+    rc = lib.ft_gemm_small_m_f32(a.data_ptr(), w.data_ptr(), out.data_ptr(), int(accumulate),
+                                 *(t.data_ptr() if t is not None else None for t in (alpha, nw, nb, h)), float(scale), ws.data_ptr(),
+                                 M, N, K, a.stride(0), w.stride(0), out.stride(0), N, 0, _dev(a), _stream())
+    _native.check(rc, "ft_gemm_small_m_f32")
+    stats["gemm_small_m"] += 1
+    return h
+
+
+def linear_f32_out(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``a @ w.T`` with an fp32 result (logits)."""
+    if a.dtype != torch.bfloat16:
+        return _mm_f32(a, w)
+    if _small_m_shape(a, w):
+        out = torch.empty((a.shape[0], w.shape[0]), device=a.device, dtype=torch.float32)
+        _small_m_f32(a, w, out, False, None)
+        return out
+    return gemm_nt(a, w, out_dtype=torch.float32)
+
+
+def residual_linear_(x: torch.Tensor, a: torch.Tensor, w: torch.Tensor, norm: tuple | None = None) -> torch.Tensor | None:
+    """``x += a @ w.T`` on the fp32 residual stream, in place; with ``norm = (alpha, weight, bias, scale)`` also returns the
+    dynamic tanh of the new ``x`` in the type of ``a`` (decode-sized batches: from the same kernel that adds the product)."""
+    if _small_m_shape(a, w):
+        return _small_m_f32(a, w, x, True, norm)
+    if a.dtype == torch.bfloat16:
+        gemm_nt(a, w, out=x, accumulate=True)
+    else:
+        x += _mm_f32(a, w)
+    if norm is None:
+        return None
+    return dynamic_tanh(x, norm[0], norm[1], norm[2], scale=norm[3], out_dtype=a.dtype)
+
+
 # --------------------------------------------------------------------------- RoPE
 def _rope_launch(x, cos, sin, positions, n_rot_heads, seq_len, pos_offset, interleaved, backward):
     T = x.numel() // (x.shape[-1] * x.shape[-2])

@@ -25,6 +25,27 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float = 1e-5, residual: 
     return (y, x) if residual is not None else y
 
 
+def dynamic_tanh(x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, scale: float = 1.0):
+    """``(tanh(alpha * x) * w + b) * scale`` in fp32: the norm without a statistic of the row."""
+    return (torch.tanh(alpha.float() * x.float()) * weight.float() + bias.float()) * scale
+
+
+def projection_rms(x: torch.Tensor, weight: torch.Tensor, eps: float, count: int):
+    """RMS norm of whole rows of a projection whose padding (beyond ``count`` elements) is zero, fp32."""
+    xf = x.float()
+    return xf * torch.rsqrt(xf.pow(2).sum(-1, keepdim=True) / count + eps) * weight.float()
+
+
+def query_temperature(positions: torch.Tensor, coef: float, every: float) -> torch.Tensor:
+    """``1 + coef * ln(floor((p + 1) / every) + 1)``, fp32: queries grow slowly with their position."""
+    return 1.0 + coef * torch.log(torch.floor((positions.double() + 1) / every).float() + 1.0)
+
+
+def head_gate(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """``o [T, H, D]`` times ``sigmoid(gate [T, H])``, one number per head."""
+    return (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
+
+
 def rope_tables(head_dim: int, max_pos: int, theta: float = 10000.0, scaling: dict | None = None,
                 device=None):
     """cos/sin tables ``[max_pos, head_dim/2]`` in fp32.

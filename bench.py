@@ -64,6 +64,11 @@ def parse_args():
     ap.add_argument("--measure-exposed", action="store_true",
                     help="record how long the compute stream waits for the gradient exchange at the end of a step")
     ap.add_argument("--comm", default="fused", choices=["fused", "nccl"])
+    ap.add_argument("--workload", default="train", choices=["train", "decoder-serving"],
+                    help="decoder-serving: prefill / decode throughput of the decoder families side by side on one GPU "
+                    "(benchmarks/decoder_serving.py) instead of the training step")
+    ap.add_argument("--serving-sizes", default="1b,3b,8b")
+    ap.add_argument("--serving-kernels", action="store_true", help="also time every kernel of a layer against its roofline")
     return ap.parse_args()
 
 
@@ -297,6 +302,11 @@ def main() -> None:
     args = parse_args()
     if args.impl == "reference":
         reference_unavailable()
+        return
+    if args.workload == "decoder-serving":
+        from benchmarks import decoder_serving
+
+        print(json.dumps(decoder_serving.run(args, ClockSampler)))
         return
 
     import torch

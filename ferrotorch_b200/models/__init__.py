@@ -1,4 +1,4 @@
-"""Model families: Llama (single-GPU, tensor-parallel training, inference engine), ResNet, and the
+"""Model families: Llama (single-GPU, tensor-parallel training, inference engine), Bopudra, ResNet, and the
 small zoo (BERT, Whisper encoder, GCN, PPO policy) and the latent-diffusion stack (``diffusion``)."""
 from .llama import LlamaConfig, LlamaForCausalLM, LlamaModel  # noqa: F401
 from .llama_compat import (AwqQ4, GptqQ4, HqqQ4Axis1, LlamaActivation, LlamaAttention, LlamaGpuLayer, LlamaMLP,  # noqa: F401
@@ -24,7 +24,15 @@ def __getattr__(name):
         from . import spec_decode
 
         return getattr(spec_decode, name)
-    if name in ("ContinuousBatcher", "Request", "RequestState", "SamplingParams", "ServingStats"):
+    if name in ("BopudraConfig", "BopudraForCausalLM"):
+        from . import bopudra
+
+        return getattr(bopudra, name)
+    if name in ("load_causal_lm", "register_causal_lm", "list_causal_lms"):
+        from . import registry
+
+        return getattr(registry, name)
+    if name in ("PagedStepper", "ContinuousBatcher", "Request", "RequestState", "SamplingParams", "ServingStats"):
         from . import serving
 
         return getattr(serving, name)

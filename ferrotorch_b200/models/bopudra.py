@@ -56,6 +56,11 @@ class BopudraConfig:
         return cls.uniform(128256, 4096, 32, 32, 8, 128, 21504)
 
     @classmethod
+    def tiny(cls) -> "BopudraConfig":
+        """A few layers for smoke tests."""
+        return cls.uniform(1000, 128, 3, 4, 1, 32, 352, vdim=48)
+
+    @classmethod
     def from_dict(cls, cfg: dict | str) -> "BopudraConfig":
         """Build from a ``config.json`` dict or path."""
         if isinstance(cfg, str):
@@ -162,6 +167,34 @@ class BopudraForCausalLM(nn.Module):
         for block in self.blocks:
             block.random_(std, g)
         return self
+
+    @classmethod
+    def tiny_random(cls, dtype: torch.dtype = torch.bfloat16, device="cpu") -> "BopudraForCausalLM":
+        return cls(BopudraConfig.tiny(), dtype, device).random_()
+
+    def checkpoint_tensors(self) -> dict:
+        """The weights under their checkpoint names, in their true sizes."""
+        c = self.config
+        out = {"embed": self.embed[:, :c.hidden_size], "head": self.head[:c.vocab_size, :c.hidden_size]}
+        named = [("final.norm", self.final_norm)] + [("l%d.norm1" % i, n) for i, n in enumerate(self.norms)]
+        for name, n in named:
+            out.update({name: n.weight[:c.hidden_size], name + ".b": n.bias[:c.hidden_size], name + ".alpha": n.alpha})
+        for i, block in enumerate(self.blocks):
+            parts = block.unpack()
+            for name, key in (("q", "q"), ("k", "k"), ("v", "v"), ("o", "o"), ("g", "gate"), ("q.norm", "q_norm"), ("k.norm", "k_norm")):
+                out["l%d.mix.%s" % (i, name)] = parts[key]
+            if block.ff:
+                out.update({"l%d.mlp.up" % i: parts["up"], "l%d.mlp.down" % i: parts["down"]})
+        return {k: v.contiguous() for k, v in out.items()}
+
+    def save_pretrained(self, path: str) -> None:
+        """Write ``config.json`` and ``model.safetensors``."""
+        from ..serialize.state import save_safetensors
+
+        os.makedirs(path, exist_ok=True)
+        with open(os.path.join(path, "config.json"), "w") as f:
+            json.dump(self.config.to_dict(), f, indent=1)
+        save_safetensors(self.checkpoint_tensors(), os.path.join(path, "model.safetensors"))
 
     @classmethod
     def from_pretrained(cls, path: str, dtype: torch.dtype = torch.bfloat16, device="cpu") -> "BopudraForCausalLM":

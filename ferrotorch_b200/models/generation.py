@@ -110,7 +110,7 @@ def generate(model, input_ids: torch.Tensor, cfg: GenerationConfig | None = None
     gen = None
     if cfg.seed is not None:
         gen = torch.Generator(device=dev).manual_seed(cfg.seed)
-    caches = model.make_caches(B, S + cfg.max_new_tokens, device=dev, dtype=next(model.parameters()).dtype)
+    caches = model.make_caches(B, S + cfg.max_new_tokens, device=dev, dtype=getattr(model, "dtype", None) or next(model.parameters()).dtype)
     logits = model(input_ids, caches=caches, last_token_only=True)[:, -1]
     out = input_ids
     done = torch.zeros(B, dtype=torch.bool, device=dev)

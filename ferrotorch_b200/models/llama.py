@@ -309,6 +309,10 @@ class LlamaForCausalLM(nn.Module):
         return [KVCache(batch, max_len, c.num_key_value_heads, c.head_dim, device, dtype)
                 for _ in range(c.num_hidden_layers)]
 
+    @classmethod
+    def tiny_random(cls, dtype: torch.dtype = torch.bfloat16, device="cpu") -> "LlamaForCausalLM":
+        return cls(LlamaConfig.tiny()).to(device=device, dtype=dtype)
+
     # ------------------------------------------------------------------ model directories and files
     @classmethod
     def from_pretrained(cls, path: str, dtype: torch.dtype = torch.bfloat16, device="cpu") -> "LlamaForCausalLM":

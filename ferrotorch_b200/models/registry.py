@@ -1,7 +1,7 @@
 """Registry of decoder families: which class loads the model of a directory, chosen by its ``config.json``.
 
 A family registers a predicate on the configuration and the class that serves it.  The class offers
-``from_pretrained(path, dtype, device)``, ``config`` (with ``vocab_size``, ``max_position_embeddings`` or ``None``),
+``from_pretrained(path, dtype, device)``, ``tiny_random(dtype, device)``, ``config`` (with ``vocab_size``, ``max_position_embeddings`` or ``None``),
 ``make_paged_cache`` and ``paged_forward``: what :class:`~ferrotorch_b200.models.serving.PagedStepper` and the server need."""
 from __future__ import annotations
 
@@ -17,7 +17,6 @@ class CausalLMFamily:
     name: str
     matches: Callable[[dict], bool]
     model: str                    # "module:class"
-    float32: bool = True          # runs with 32-bit weights, cache and activations on a GPU
 
     def model_class(self):
         mod, cls = self.model.split(":")
@@ -34,6 +33,13 @@ def register_causal_lm(family: CausalLMFamily) -> None:
 
 def list_causal_lms() -> list[str]:
     return sorted(f.name for f in _FAMILIES)
+
+
+def family_named(name: str) -> CausalLMFamily:
+    for fam in _FAMILIES:
+        if fam.name == name:
+            return fam
+    raise ValueError("no decoder family %r (known: %s)" % (name, ", ".join(list_causal_lms())))
 
 
 def family_of(cfg: dict | str) -> CausalLMFamily:

@@ -204,20 +204,23 @@ class ServingApp:
 
 
 def main(argv=None) -> int:
-    """``python -m ferrotorch_b200.models.server --model DIR [--device cuda] [--port 8000]``: serve a Hugging Face
-    Llama directory (``config.json``, weights, ``tokenizer.json``).  ``--tiny`` serves a random tiny model on
-    token ids (a smoke test that needs no files)."""
+    """``python -m ferrotorch_b200.models.server --model DIR [--device cuda] [--port 8000]``: serve a model directory
+    (``config.json``, SafeTensors weights, ``tokenizer.json`` when there is one) of any registered decoder family.
+    ``--tiny`` serves a random tiny model of ``--family`` on token ids (a smoke test that needs no files)."""
     import argparse
     import os
     import time
 
     import torch
 
-    from .llama import LlamaConfig, LlamaForCausalLM
+    from .registry import family_named, list_causal_lms, load_causal_lm
 
     ap = argparse.ArgumentParser(description=main.__doc__)
     ap.add_argument("--model")
     ap.add_argument("--tiny", action="store_true")
+    ap.add_argument("--family", default="llama", choices=list_causal_lms(), help="family of the --tiny model")
+    ap.add_argument("--dtype", choices=("bfloat16", "float32"), default=None, help="default: bfloat16, on the CPU float32")
+    ap.add_argument("--cuda-graph", action="store_true", help="replay decode steps as captured CUDA graphs")
     ap.add_argument("--device", default="cuda" if torch.cuda.is_available() else "cpu")
     ap.add_argument("--host", default="127.0.0.1")
     ap.add_argument("--port", type=int, default=8000)
@@ -232,13 +235,13 @@ def main(argv=None) -> int:
     args = ap.parse_args(argv)
     if not args.tiny and not args.model:
         ap.error("give --model DIR or --tiny")
-    dtype = torch.bfloat16 if args.device != "cpu" else torch.float32
+    dtype = getattr(torch, args.dtype or ("bfloat16" if args.device != "cpu" else "float32"))
     encode = decode = None
     if args.tiny:
         torch.manual_seed(0)
-        model = LlamaForCausalLM(LlamaConfig.tiny()).to(device=args.device, dtype=dtype)
+        model = family_named(args.family).model_class().tiny_random(dtype=dtype, device=args.device)
     else:
-        model = LlamaForCausalLM.from_pretrained(args.model, dtype=dtype, device=args.device)
+        model = load_causal_lm(args.model, dtype=dtype, device=args.device)
         tok_path = os.path.join(args.model, "tokenizer.json")
         if os.path.exists(tok_path):
             from ..utils import text
@@ -246,8 +249,10 @@ def main(argv=None) -> int:
             tok = text.load_tokenizer(tok_path)
             encode, decode = (lambda s: text.encode(tok, s)), (lambda ids: text.decode(tok, ids))
     batcher = ContinuousBatcher(model.eval(), args.kv_pages, args.page_size, args.max_running,
-                                args.max_seq_len or min(model.config.max_position_embeddings, args.kv_pages * args.page_size),
-                                args.max_tokens_per_step, args.prefill_chunk, prefix_caching=not args.no_prefix_caching)
+                                args.max_seq_len or min(model.config.max_position_embeddings or args.kv_pages * args.page_size,
+                                                        args.kv_pages * args.page_size),
+                                args.max_tokens_per_step, args.prefill_chunk, prefix_caching=not args.no_prefix_caching,
+                                cuda_graph=args.cuda_graph)
     app = ServingApp(batcher, encode, decode, os.path.basename(os.path.normpath(args.model)) if args.model else "tiny").start(args.host, args.port)
     print("serving on http://%s:%d (POST /v1/completions, GET /health, GET /metrics)" % (app.host, app.port), flush=True)
     try:

@@ -14,7 +14,8 @@ from .fake_quant import FakeQuantize, MinMaxObserver, MovingAverageObserver, Qat
 from .extra import (HookedModule, HookHandle, LoRALinear, SqueezeExcitation, flash_attention,  # noqa: F401,E402
                     standard_attention)
 from ..core import BlockMask, flex_attention  # noqa: F401,E402
-from .paged import OutOfPages, PagedAttentionManager, PagedKVCache  # noqa: F401,E402
+from .paged import OutOfPages, PagedAttentionManager, PagedKVCache, PagedSession, RaggedBatch  # noqa: F401,E402
+from .packed_block import AttentionSpec, DynamicTanh, PackedParallelBlock  # noqa: F401,E402
 from ..ops.conv import IgemmConv2d, convert_convs  # noqa: F401,E402  (implicit-GEMM convolution; opt-in, see ops.conv)
 from ..ops.pool import MaxPool2d as NhwcMaxPool2d  # noqa: F401,E402
 from .compat import *  # noqa: F401,F403,E402

@@ -141,6 +141,25 @@ class PackedParallelBlock(nn.Module):
             self.q_norm.copy_(pad_heads(q_norm.float(), H, a.padded_dim))
             self.k_norm.copy_(pad_heads(k_norm.float(), G, a.padded_dim))
 
+    def unpack(self) -> dict:
+        """The inverse of :meth:`load`: views and copies of the true sizes."""
+        a, W = self.attn, self.hidden_size
+        (qo, qn), (ko, kn), (vo, vn), (uo, un), (go, gn) = self.segments
+
+        def heads(t, n, d):
+            return t.unflatten(0, (n, -1))[:, :d].flatten(0, 1)
+
+        w = self.in_proj[:, :W]
+        out = {"q": heads(w[qo:qo + qn], a.heads, a.dim), "k": heads(w[ko:ko + kn], a.kv_heads, a.dim), "v": heads(w[vo:vo + vn], a.kv_heads, a.vdim),
+               "o": heads(self.out_proj[:W, :self.value_width].t(), a.heads, a.vdim).t()}
+        if self.ff:
+            out.update(up=w[uo:uo + self.ff], down=self.out_proj[:W, self.value_width:self.value_width + self.ff])
+        if self.head_gate:
+            out.update(gate=w[go:go + a.heads])
+        if self.qk_norm:
+            out.update(q_norm=heads(self.q_norm, a.heads, a.dim), k_norm=heads(self.k_norm, a.kv_heads, a.dim))
+        return out
+
     def random_(self, std: float, generator: torch.Generator | None = None) -> None:
         """Random weights of the true sizes (benchmarks and smoke tests)."""
         a, W = self.attn, self.hidden_size

@@ -1,0 +1,65 @@
+"""Attention over the paged cache where one key stands out: queries that match exactly one key each."""
+import torch
+
+import bopudra_oracle as O
+from ferrotorch_b200.nn.paged import PagedAttentionManager, PagedKVCache, RaggedBatch
+
+
+def check_planted_keys(Hq, Hkv, D, Dv, block, dtype, device, length, tolerance=None):
+    """Keys are unit-scale noise; query i is a multiple of one key's direction, so that key's score stands out by tens.
+    Targets walk over the first keys, page and tile borders, the query's own key, and the key just after it (which a
+    query in a portion must not see although it is in the cache)."""
+    g = torch.Generator().manual_seed(length + D)
+    tol = tolerance or (1e-4 if dtype == torch.float32 else 3e-2)
+    cache = PagedKVCache(1, Hkv, D, 2 * ((length + block - 1) // block) + 3, 3, length + block, block, device, dtype, v_head_dim=Dv)
+    mgr = PagedAttentionManager(cache)
+    other, slot = mgr.add_sequence(0), mgr.add_sequence(0)
+    for n in range(1, length + 1, max(1, block - 1)):     # pages of two sequences interleave, not in order
+        for s in (other, slot):
+            cache.reserve(s, min(n + block, length))
+    cache.reserve(slot, length)
+    k = torch.randn(length, Hkv, D, generator=g).to(dtype)
+    v = torch.randn(length, Hkv, Dv, generator=g).to(dtype)
+    pos = torch.arange(length, dtype=torch.int32, device=device)
+    for s, sign in ((other, -1.0), (slot, 1.0)):
+        n = cache.lengths[s]
+        cache.append(0, (sign * k[:n]).to(device), (sign * v[:n]).to(device), pos[:n], torch.full((n,), s, dtype=torch.int32, device=device))
+    group, scale = Hq // Hkv, 0.25
+    edges = sorted({e for b in (block, 128) for m in range(0, length + b, b) for e in (m - 1, m, m + 1)} | {0, 1, 2, length - 1, length - 2})
+    edges = [e for e in edges if 0 <= e < length]
+    q, target = torch.zeros(length, Hq, D), {}
+    for i in range(length):
+        for h in range(Hq):
+            t = (edges + [i, i + 1])[(i * 7 + h * 3) % (len(edges) + 2)]
+            t = min(t, length - 1)
+            kt = k[t, h // group].float()
+            q[i, h] = kt * (50.0 / scale / kt.pow(2).sum())
+            target[i, h] = t
+    q = q.to(dtype)
+    gate = torch.randn(length, Hq, generator=g).to(dtype)
+    want = torch.zeros(length, Hq, Dv, dtype=torch.float64)
+    for i in range(length):
+        for h in range(Hq):
+            c = h // group
+            o = O.head_attention(q[i, h].double(), k[:i + 1, c].double(), v[:i + 1, c].double(), scale)
+            want[i, h] = o * torch.sigmoid(gate[i, h].double())
+            if target[i, h] <= i and D >= 32:             # the case is what it claims: that key carries the softmax
+                assert (o - v[target[i, h], c].double()).abs().max() < 0.2
+    for cuts in ([length], [1], [2, 1, 3, block, 1, 128, 5, 1]):
+        entries, at, n = [], 0, 0
+        while at < length:
+            step = min(cuts[n % len(cuts)], length - at)
+            entries.append((slot, [0] * step, at, []))
+            at, n = at + step, n + 1
+        batch = RaggedBatch(entries, device)
+        rows = batch.positions.long().cpu()
+        # rows lie in a wider buffer, as in a packed projection
+        buf = torch.zeros(length, Hq * D + 8, dtype=dtype)
+        buf[:, :Hq * D] = q[rows].flatten(1)
+        buf = buf.to(device)
+        out = torch.full((length, Hq * Dv + 16), 7.0, dtype=dtype, device=device)
+        cache.attend(0, buf[:, :Hq * D].unflatten(1, (Hq, D)), batch, scale, gate=gate[rows].to(device),
+                     out=out[:, :Hq * Dv].unflatten(1, (Hq, Dv)))
+        err = (out[:, :Hq * Dv].double().cpu().view(length, Hq, Dv) - want[rows]).abs().amax((1, 2))
+        assert float(err.max()) < tol, "cuts %s: error %.3g at position %d" % (cuts, float(err.max()), int(rows[err.argmax()]))
+        assert bool((out[:, Hq * Dv:] == 7.0).all())

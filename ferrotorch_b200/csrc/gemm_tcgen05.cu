@@ -1203,6 +1203,30 @@ static int small_m_pick_split(int N, int K, int ksplit, int min_split, int devic
   return ksplit > SMALL_M_MAX_SPLIT ? SMALL_M_MAX_SPLIT : ksplit;
 }
 
+// The whole contraction in one pass, C written transposed by the epilogue (bf16, or fp32 with GEMM_OUT_F32).
+static int small_m_single(const void* X, const void* W, void* C, const void* bias, int M, int N, int K, long long ldx,
+                          long long ldw, long long ldc, int flags, int device, cudaStream_t stream) {
+  const int bn = M <= 64 ? 64 : 128;
+  GemmParams p;
+  p.bias = bias; p.M = N; p.N = M; p.K = K;   // tile space: rows of W x batch
+  p.status = device_status_word(device);
+  p.taps = 0; p.cblocks = 0; p.ksplit = 1;
+  for (int t = 0; t < GEMM_MAX_TAPS; ++t) p.shift[t] = 0;
+  p.gHp = p.gWp = p.cHo = p.cWo = p.c_oh = p.c_ow = 0; p.split_rows = 0;
+  p.C = C; p.ldc = ldc;
+  p.flags = flags | GEMM_EPI_TRANSPOSED;
+  CUtensorMap tmA, tmB, tmC;
+  int rc = make_tmap_2d(&tmA, W, 2, K, N, ldw * 2, GEMM_BK, GEMM_BM, 3);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tmB, X, 2, K, M, ldx * 2, GEMM_BK, bn / 2, 3);
+  if (rc) return rc;
+  // the store map is not used by the transposed epilogue; point it at W so that it is valid
+  rc = make_tmap_2d(&tmC, W, 2, K, N, ldw * 2, 64, 32, 3);
+  if (rc) return rc;
+  return bn == 64 ? launch_pair<64, false, false, 0>(tmA, tmB, tmC, p, device, 0, stream)
+                  : launch_pair<128, false, false, 0>(tmA, tmB, tmC, p, device, 0, stream);
+}
+
 // Launch the split contraction of a small-batch GEMM into `workspace` (slices of ceil(N / 256) * 256 rows
 // x 64 or 128 columns); *ksplit returns the number of slices.
 static int small_m_split(const void* X, const void* W, float* workspace, int M, int N, int K, long long ldx, long long ldw,
@@ -1263,28 +1287,8 @@ FT_API int ft_gemm_small_m(const void* X, const void* W, void* C, const void* bi
   if (residual && ksplit == 1 && workspace && k_blocks >= 2) ksplit = 2;
   FT_REQUIRE(ksplit == 1 || workspace, "ft_gemm_small_m: a split contraction needs the workspace");
   FT_REQUIRE(ksplit > 1 || !residual, "ft_gemm_small_m: the residual is added by the split path only");
-  int rc;
-  if (ksplit == 1) {
-    GemmParams p;
-    p.bias = bias; p.M = N; p.N = M; p.K = K;   // tile space: rows of W x batch
-    p.status = device_status_word(device);
-    p.taps = 0; p.cblocks = 0; p.ksplit = 1;
-    for (int t = 0; t < GEMM_MAX_TAPS; ++t) p.shift[t] = 0;
-    p.gHp = p.gWp = p.cHo = p.cWo = p.c_oh = p.c_ow = 0; p.split_rows = 0;
-    p.C = C; p.ldc = ldc;
-    p.flags = (flags & 0xFFFF) | GEMM_EPI_TRANSPOSED;
-    CUtensorMap tmA, tmB, tmC;
-    rc = make_tmap_2d(&tmA, W, 2, K, N, ldw * 2, GEMM_BK, GEMM_BM, 3);
-    if (rc) return rc;
-    rc = make_tmap_2d(&tmB, X, 2, K, M, ldx * 2, GEMM_BK, bn / 2, 3);
-    if (rc) return rc;
-    // the store map is not used by the transposed epilogue; point it at W so that it is valid
-    rc = make_tmap_2d(&tmC, W, 2, K, N, ldw * 2, 64, 32, 3);
-    if (rc) return rc;
-    return bn == 64 ? launch_pair<64, false, false, 0>(tmA, tmB, tmC, p, device, 0, stream)
-                    : launch_pair<128, false, false, 0>(tmA, tmB, tmC, p, device, 0, stream);
-  }
-  rc = small_m_split(X, W, workspace, M, N, K, ldx, ldw, &ksplit, 2, device, stream);
+  if (ksplit == 1) return small_m_single(X, W, C, bias, M, N, K, ldx, ldw, ldc, flags & 0xFFFF, device, stream);
+  int rc = small_m_split(X, W, workspace, M, N, K, ldx, ldw, &ksplit, 2, device, stream);
   if (rc) return rc;
   dim3 grid((N + 31) / 32, (M + 31) / 32), block(32, 8);
   small_m_finalize_kernel<<<grid, block, 0, stream>>>(workspace, static_cast<__nv_bfloat16*>(C),
@@ -1296,8 +1300,8 @@ FT_API int ft_gemm_small_m(const void* X, const void* W, void* C, const void* bi
   return FT_E_OK;
 }
 
-// C[M, N] (fp32) (+)= X[M, K] W[N, K]^T for a small batch M <= 128, always through the split contraction
-// and its finalize pass (see ft_gemm_small_m), which also writes dyt_out[M, N] = (tanh(alpha C) w + b) * dyt_scale
+// C[M, N] (fp32) (+)= X[M, K] W[N, K]^T for a small batch M <= 128: in one pass when W alone fills the GPU and
+// nothing is added, else through the split contraction and its finalize pass (see ft_gemm_small_m), which also writes dyt_out[M, N] = (tanh(alpha C) w + b) * dyt_scale
 // as bf16 when dyt_out is given.  workspace: ft_gemm_small_m_workspace(M, N) floats.
 FT_API int ft_gemm_small_m_f32(const void* X, const void* W, float* C, int accumulate, const float* alpha, const float* dyt_w,
                                const float* dyt_b, void* dyt_out, float dyt_scale, float* workspace, int M, int N, int K,
@@ -1309,6 +1313,8 @@ FT_API int ft_gemm_small_m_f32(const void* X, const void* W, float* C, int accum
   FT_REQUIRE(M > 0 && M <= 128 && N > 0 && K > GEMM_BK, "ft_gemm_small_m_f32: M=%d must be in 1..128, K=%d above %d (N=%d)", M, K, GEMM_BK, N);
   FT_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0, "ft_gemm_small_m_f32: strides must be multiples of 8");
   FT_REQUIRE(!dyt_out || (alpha && dyt_w && dyt_b), "ft_gemm_small_m_f32: the fused norm needs its parameters");
+  if (!accumulate && !dyt_out && small_m_pick_split(N, K, ksplit, 1, device) == 1)
+    return small_m_single(X, W, C, nullptr, M, N, K, ldx, ldw, ldc, GEMM_OUT_F32, device, stream);
   int rc = small_m_split(X, W, workspace, M, N, K, ldx, ldw, &ksplit, 2, device, stream);
   if (rc) return rc;
   dim3 grid((N + 31) / 32, (M + 31) / 32), block(32, 8);

@@ -467,6 +467,14 @@ dyt_kernel(const TI* __restrict__ x, const long long* __restrict__ ids, int voca
   }
 }
 
+// The activation ahead of a bf16 store: 0.5 (1 + tanh u) = 1 / (1 + exp(-2 u)) needs one exponential and one
+// approximate division, where tanhf makes the kernel compute-bound.  fp32 rows keep act_fwd.
+__device__ __forceinline__ float act_row(float g, int act, const __nv_bfloat16*) {
+  if (act != 2) return act_fwd(g, act);
+  return g * __fdividef(1.f, 1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
+}
+__device__ __forceinline__ float act_row(float g, int act, const float*) { return act_fwd(g, act); }
+
 // ---------------------------------------------------------------- packed projection -> attention
 // One pass over a row of the packed input projection [ .. q .. k .. v .. up .. ] of a decoder layer
 // whose attention and feed-forward read the same input:
@@ -501,8 +509,30 @@ qkv_finish_kernel(const QkvFinishParams p) {
   __shared__ float red[2][NORM_THREADS / 32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float* nul = nullptr;
+  // blockIdx.y: part of the row.  Part 0 does q, k and v; the activation is spread over the others (over part 0
+  // when there is only one), because it is most of the row and waits for nothing.
+  const int act_parts = max(static_cast<int>(gridDim.y) - 1, 1), act_part = gridDim.y > 1 ? static_cast<int>(blockIdx.y) - 1 : 0;
   for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
     T* y = static_cast<T*>(p.packed) + static_cast<long long>(row) * p.ld;
+    if (act_part >= 0) {
+      T* up_out = static_cast<T*>(p.act_out) + static_cast<long long>(row) * p.ld_act;
+      const int stride = act_parts * NORM_THREADS * 8;
+      for (int i = (act_part * NORM_THREADS + threadIdx.x) * 8; i < p.up_n; i += 2 * stride) {   // two loads in flight
+        const int i2 = i + stride < p.up_n ? i + stride : i;
+        float f[8], g[8];
+        load8(y + p.up_off + i, f);
+        load8(y + p.up_off + i2, g);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = act_row(f[j], p.act, y);
+        store8(up_out + i, f);
+        if (i2 != i) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) g[j] = act_row(g[j], p.act, y);
+          store8(up_out + i2, g);
+        }
+      }
+    }
+    if (blockIdx.y > 0) continue;
     const int position = p.pos[row];
     float sq = 0.f, sk = 0.f;
     if (p.q_weight != nul)
@@ -523,14 +553,6 @@ qkv_finish_kernel(const QkvFinishParams p) {
     sk = warp_sum(sk);
     __syncthreads();                       // the previous row's sums have been read
     if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
-    // the MLP activation does not wait for the sums
-    for (int i = threadIdx.x * 8; i < p.up_n; i += NORM_THREADS * 8) {
-      float f[8];
-      load8(y + p.up_off + i, f);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) f[j] = act_fwd(f[j], p.act);
-      store8(static_cast<T*>(p.act_out) + static_cast<long long>(row) * p.ld_act + i, f);
-    }
     const int blk = p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + position / p.block_size];
     const bool cached = blk >= 0 && blk < p.num_blocks;    // host validates; never write out of range
     const long long token = static_cast<long long>(blk) * p.block_size + position % p.block_size;
@@ -741,12 +763,13 @@ FT_API int ft_dyt_fwd(const void* x, const long long* ids, int vocab, int in_bf1
 }
 
 // The pass between a packed input projection and its attention (see qkv_finish_kernel).  packed, caches
-// and act_out are bf16, or fp32 with f32.  Offsets and sizes in elements, multiples of 8.
+// and act_out are bf16, or fp32 with f32.  Offsets and sizes in elements, multiples of 8.  row_parts: blocks that
+// share a row (0: chosen here).
 FT_API int ft_qkv_finish(void* packed, long long ld, const int* pos, const int* slots, const int* block_table, void* k_cache,
                          void* v_cache, const float* q_weight, const float* k_weight, void* act_out, long long ld_act,
                          int rows, int q_off, int q_n, int k_off, int k_n, int v_off, int v_n, int up_off, int up_n,
                          int q_count, int k_count, float eps, float temp_coef, float temp_every, int act, int f32,
-                         int block_size, int max_blocks, int num_blocks, int device, cudaStream_t stream) {
+                         int block_size, int max_blocks, int num_blocks, int row_parts, int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(packed && pos && slots && block_table && k_cache && v_cache, "ft_qkv_finish: null pointer");
   FT_REQUIRE(((q_off | q_n | k_off | k_n | v_off | v_n | up_off | up_n) & 7) == 0 && ld % 8 == 0 && ld_act % 8 == 0,
@@ -768,7 +791,15 @@ FT_API int ft_qkv_finish(void* packed, long long ld, const int* pos, const int* 
   p.up_off = up_off; p.up_n = up_n; p.q_count = q_count; p.k_count = k_count;
   p.eps = eps; p.temp_coef = temp_coef; p.temp_every = temp_every;
   p.act = act; p.block_size = block_size; p.max_blocks = max_blocks; p.num_blocks = num_blocks;
-  const int grid = rows < sm_count(device) * 8 ? rows : sm_count(device) * 8;
+  // a batch that does not fill the GPU is cut into one more part per pass of a block over the activation
+  const int wave = sm_count(device) * 8;
+  if (row_parts <= 0) {
+    row_parts = up_n > 0 ? 1 + (up_n + NORM_THREADS * 8 - 1) / (NORM_THREADS * 8) : 1;
+    if (row_parts > wave / rows) row_parts = wave / rows > 1 ? wave / rows : 1;
+  }
+  if (row_parts > 64) row_parts = 64;
+  int per_part = wave / row_parts > 0 ? wave / row_parts : 1;
+  const dim3 grid(rows < per_part ? rows : per_part, row_parts);
   if (f32) qkv_finish_kernel<float><<<grid, NORM_THREADS, 0, stream>>>(p);
   else qkv_finish_kernel<__nv_bfloat16><<<grid, NORM_THREADS, 0, stream>>>(p);
   FT_CUDA_CHECK(cudaGetLastError());

@@ -39,27 +39,22 @@ __device__ __forceinline__ float head_gate_bf16(const HeadGate& gt, int row, int
   return gate_value(__bfloat162float(static_cast<const __nv_bfloat16*>(gt.g)[static_cast<long long>(row) * gt.ld + head]));
 }
 
-// k_new / v_new: [T, Hkv, D] rows with token stride ld (elements).  Token i goes to sequence
-// seq_ids[i] (or i / tokens_per_seq when null) at position pos[i].
-__global__ void kv_append_kernel(const __nv_bfloat16* __restrict__ k_new, const __nv_bfloat16* __restrict__ v_new,
-                                 __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache,
-                                 const int* __restrict__ block_table, const int* __restrict__ pos,
-                                 const int* __restrict__ seq_ids, int T, int tokens_per_seq, int Hkv, int D,
-                                 long long ldk, long long ldv, int block_size, int max_blocks, int num_blocks) {
-  const int row_vec = (Hkv * D) >> 3;
+// k_new / v_new: rows of kv16 / vv16 16-byte units (all KV heads of a token) with token strides ldk16 / ldv16 units.
+// Token i goes to sequence seq_ids[i] (or i / tokens_per_seq when null) at position pos[i].
+__global__ void kv_append_kernel(const uint4* __restrict__ k_new, const uint4* __restrict__ v_new, uint4* __restrict__ k_cache,
+                                 uint4* __restrict__ v_cache, const int* __restrict__ block_table,
+                                 const int* __restrict__ pos, const int* __restrict__ seq_ids, int T, int tokens_per_seq,
+                                 int kv16, int vv16, long long ldk16, long long ldv16, int block_size, int max_blocks,
+                                 int num_blocks) {
   for (int t = blockIdx.x; t < T; t += gridDim.x) {
     const int b = seq_ids ? seq_ids[t] : t / tokens_per_seq;
     const int p = pos[t];
     const int blk = block_table[static_cast<long long>(b) * max_blocks + p / block_size];
     if (blk < 0 || blk >= num_blocks) continue;  // host validates; never write out of range
-    const long long dst = (static_cast<long long>(blk) * block_size + p % block_size) * Hkv * D;
-    const uint4* ks = reinterpret_cast<const uint4*>(k_new + static_cast<long long>(t) * ldk);
-    const uint4* vs = reinterpret_cast<const uint4*>(v_new + static_cast<long long>(t) * ldv);
-    uint4* kd = reinterpret_cast<uint4*>(k_cache + dst);
-    uint4* vd = reinterpret_cast<uint4*>(v_cache + dst);
-    for (int i = threadIdx.x; i < row_vec; i += blockDim.x) {
-      kd[i] = ks[i];
-      vd[i] = vs[i];
+    const long long token = static_cast<long long>(blk) * block_size + p % block_size;
+    for (int i = threadIdx.x; i < max(kv16, vv16); i += blockDim.x) {
+      if (i < kv16) k_cache[token * kv16 + i] = k_new[t * ldk16 + i];
+      if (i < vv16) v_cache[token * vv16 + i] = v_new[t * ldv16 + i];
     }
   }
 }
@@ -712,20 +707,25 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
 
 using namespace ft;
 
+// Append keys [T, Hkv, D] and values [T, Hkv, Dv] of elem_bytes-sized elements (2 or 4; strides in elements).
 FT_API int ft_kv_append(const void* k_new, const void* v_new, void* k_cache, void* v_cache, const int* block_table,
-                        const int* pos, const int* seq_ids, int T, int tokens_per_seq, int Hkv, int D,
+                        const int* pos, const int* seq_ids, int T, int tokens_per_seq, int Hkv, int D, int Dv, int elem_bytes,
                         long long ldk, long long ldv, int block_size, int max_blocks, int num_blocks,
                         int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(k_new && v_new && k_cache && v_cache && block_table && pos, "ft_kv_append: null pointer");
-  FT_REQUIRE((Hkv * D) % 8 == 0 && ldk % 8 == 0 && ldv % 8 == 0 && block_size > 0 && (seq_ids || tokens_per_seq > 0),
-             "ft_kv_append: bad layout");
+  FT_REQUIRE(elem_bytes == 2 || elem_bytes == 4, "ft_kv_append: element size %d", elem_bytes);
+  const int unit = 16 / elem_bytes;
+  FT_REQUIRE((Hkv * D) % unit == 0 && (Hkv * Dv) % unit == 0 && ldk % unit == 0 && ldv % unit == 0 && block_size > 0 &&
+                 (seq_ids || tokens_per_seq > 0), "ft_kv_append: bad layout");
+  FT_REQUIRE(((reinterpret_cast<uintptr_t>(k_new) | reinterpret_cast<uintptr_t>(v_new) | reinterpret_cast<uintptr_t>(k_cache) |
+               reinterpret_cast<uintptr_t>(v_cache)) & 15) == 0, "ft_kv_append: pointers must be 16-byte aligned");
   if (T <= 0) return FT_E_OK;
   const int grid = T < sm_count(device) * 8 ? T : sm_count(device) * 8;
-  kv_append_kernel<<<grid, 128, 0, stream>>>(static_cast<const __nv_bfloat16*>(k_new), static_cast<const __nv_bfloat16*>(v_new),
-                                             static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache),
-                                             block_table, pos, seq_ids, T, tokens_per_seq, Hkv, D, ldk, ldv, block_size,
-                                             max_blocks, num_blocks);
+  kv_append_kernel<<<grid, 128, 0, stream>>>(static_cast<const uint4*>(k_new), static_cast<const uint4*>(v_new),
+                                             static_cast<uint4*>(k_cache), static_cast<uint4*>(v_cache), block_table, pos,
+                                             seq_ids, T, tokens_per_seq, Hkv * D / unit, Hkv * Dv / unit, ldk / unit, ldv / unit,
+                                             block_size, max_blocks, num_blocks);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

@@ -20,7 +20,7 @@ from ..ops import reference as ref
 
 _i, _ll, _f, _vp = _native._i, _native._ll, _native._f, _native._vp
 _native.register_protos({
-    "ft_kv_append": (_i, [_vp] * 7 + [_i, _i, _i, _i, _ll, _ll, _i, _i, _i, _i, _vp]),
+    "ft_kv_append": (_i, [_vp] * 7 + [_i] * 6 + [_ll, _ll, _i, _i, _i, _i, _vp]),
     "ft_paged_decode_scratch": (_ll, [_i, _i, _i, _i]),
     "ft_paged_decode": (_i, [_vp] * 9 + [_i] * 5 + [_ll] * 3 + [_i, _i, _i, _f, _i, _i, _vp]),
     "ft_paged_rows": (_i, [_vp] * 8 + [_i] * 5 + [_ll] * 3 + [_i, _i, _i, _f, _i, _i, _vp]),
@@ -245,21 +245,26 @@ class PagedKVCache:
         T = k_new.shape[0]
         table = self.sync_table()
         Hkv, D, Dv = self.shapes[layer]
-        if not k_new.is_cuda or self.dtype != torch.bfloat16 or D != Dv:
-            sid = (seq_ids if seq_ids is not None else torch.arange(T, device=k_new.device) // tokens_per_seq).long()
+        if not k_new.is_cuda:
+            sid = (seq_ids if seq_ids is not None else torch.arange(T) // tokens_per_seq).long()
             pos = positions.long()
-            blk = self._table_host[sid.cpu(), (pos // self.block_size).cpu()].long().to(k_new.device)
+            blk = self._table_host[sid, pos // self.block_size].long()
             if bool((blk < 0).any()):
                 raise ValueError("PagedKVCache.append: a position has no page (reserve the sequence first)")
             self.k[layer][blk, pos % self.block_size] = k_new.to(self.k[layer].dtype)
             self.v[layer][blk, pos % self.block_size] = v_new.to(self.v[layer].dtype)
             return
+        if k_new.dtype != self.dtype or v_new.dtype != self.dtype:
+            raise ValueError("PagedKVCache.append: the cache holds %s, got %s / %s" % (self.dtype, k_new.dtype, v_new.dtype))
+        unit = 16 // k_new.element_size()
+        k_new, v_new = (t if t.stride(-1) == 1 and t.stride(1) == t.shape[2] and t.stride(0) % unit == 0 and t.data_ptr() % 16 == 0
+                        else t.contiguous() for t in (k_new, v_new))
         ldk = k_new.stride(0)
         ldv = v_new.stride(0)
         rc = _native.kernels().ft_kv_append(
             k_new.data_ptr(), v_new.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(),
             table.data_ptr(), positions.data_ptr(), seq_ids.data_ptr() if seq_ids is not None else None, T,
-            tokens_per_seq, Hkv, D, ldk, ldv, self.block_size, self.max_blocks,
+            tokens_per_seq, Hkv, D, Dv, k_new.element_size(), ldk, ldv, self.block_size, self.max_blocks,
             self.num_blocks, F._dev(k_new), F._stream())
         _native.check(rc, "ft_kv_append")
 

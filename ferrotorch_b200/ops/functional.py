@@ -336,7 +336,7 @@ _native.register_protos({
     "ft_dyt_fwd": (_native._i, [_native._vp] * 2 + [_native._i] * 2 + [_native._vp] * 5 + [_native._i] * 3 + [_native._ll] * 2 +
                    [_native._f, _native._i, _native._vp]),
     "ft_qkv_finish": (_native._i, [_native._vp, _native._ll] + [_native._vp] * 8 + [_native._ll] + [_native._i] * 11 + [_native._f] * 3 +
-                      [_native._i] * 6 + [_native._vp]),
+                      [_native._i] * 7 + [_native._vp]),
     "ft_gemm_small_m_f32": (_native._i, [_native._vp] * 3 + [_native._i] + [_native._vp] * 4 + [_native._f, _native._vp] + [_native._i] * 3 +
                             [_native._ll] * 4 + [_native._i] * 2 + [_native._vp]),
 })
@@ -376,7 +376,7 @@ def embedding_dynamic_tanh(ids: torch.Tensor, table: torch.Tensor, alpha: torch.
 def qkv_finish(packed: torch.Tensor, cache, layer: int, batch, *, q: tuple, k: tuple, v: tuple, up: tuple = (0, 0),
                q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, q_count: int = 0, k_count: int = 0,
                eps: float = 1e-5, temp_coef: float = 0.0, temp_every: float = 1.0, act_out: torch.Tensor | None = None,
-               activation: str = "gelu") -> None:
+               activation: str = "gelu", row_parts: int = 0) -> None:
     """Everything between a layer's packed input projection ``[T, N]`` and its attention, in one kernel.  ``q``, ``k``, ``v``,
     ``up`` are ``(offset, size)`` of the segments of a row: q and k are RMS-normalised over the whole projection (``q_count`` /
     ``k_count`` true elements, the rest zero padding), q is scaled by the query temperature in place, k and v go to their cache
@@ -403,7 +403,7 @@ def qkv_finish(packed: torch.Tensor, cache, layer: int, batch, *, q: tuple, k: t
         k_weight.data_ptr() if k_weight is not None else None, act_out.data_ptr() if up[1] else None,
         act_out.stride(0) if up[1] else 0, packed.shape[0], q[0], q[1], k[0], k[1], v[0], v[1], up[0], up[1],
         q_count or q[1], k_count or k[1], float(eps), float(temp_coef), float(temp_every), _ACT_ID[activation],
-        int(packed.dtype == torch.float32), cache.block_size, cache.max_blocks, cache.num_blocks, _dev(packed), _stream())
+        int(packed.dtype == torch.float32), cache.block_size, cache.max_blocks, cache.num_blocks, row_parts, _dev(packed), _stream())
     _native.check(rc, "ft_qkv_finish")
 
 

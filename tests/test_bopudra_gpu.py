@@ -119,6 +119,9 @@ def test_small_batch_gemm_adds_to_the_residual_and_normalises(M):
     assert torch.allclose(F.linear_f32_out(a, w).double(), want - x.double(), atol=1e-4)
     h = F.residual_linear_(x, a, w, (alpha, nw, nb, 1.5))
     assert x.dtype == torch.float32 and torch.allclose(x.double(), want, atol=1e-4)
+    wide = (torch.randn(20008, K, device="cuda") * K ** -0.5).bfloat16()       # fills the GPU without a split
+    got = F.linear_f32_out(a, wide)
+    assert got.dtype == torch.float32 and torch.allclose(got.double(), a.double() @ wide.double().t(), atol=1e-4)
     assert torch.allclose(h.double(), (O.dynamic_tanh(want, 0.6, nw.double(), nb.double()) * 1.5), atol=3e-2, rtol=8e-3)
 
 

@@ -33,7 +33,7 @@ OUT = _PKG / "_C"
 KERNELS_SO = OUT / "libft_kernels.so"
 # Programs that only serve decoders (bin/trace_run) need a part of the sources: with FT_KERNEL_SET=decoder a checkout
 # without a built library compiles these alone.  A library that is already complete is used as it is.
-KERNEL_SETS = {"decoder": ("ft_host", "gemm_tcgen05", "norm_act", "paged_attn", "paged_prefill")}
+KERNEL_SETS = {"decoder": ("ft_host", "gemm_tcgen05", "norm_act", "decoder_rows", "recurrent", "grouped_gemm", "paged_attn", "paged_prefill")}
 HOST_SO = OUT / "libft_host.so"
 
 NVCC_FLAGS = [

@@ -1,5 +1,5 @@
-// Softmax arithmetic on one row of a 128 x 128 score tile, shared by the forward attention kernels that
-// keep the row in registers (attn_fwd.cu, paged_prefill.cu).
+// Arithmetic that attention kernels share: one row of a 128 x 128 score tile kept in registers (attn_fwd.cu,
+// paged_prefill.cu); windows, sinks and output gates (paged_attn.cu, paged_prefill.cu).
 #pragma once
 #include "ft_ptx.cuh"
 
@@ -64,6 +64,18 @@ __device__ __forceinline__ void att2_mask_row(f32x2 (&sp)[ATT_BN / 2], int kv0, 
   }
 }
 
+// Keys ahead of the first visible one (kv0 + c < first) get -inf.
+__device__ __forceinline__ void att2_mask_ahead(f32x2 (&sp)[ATT_BN / 2], int kv0, int first) {
+#pragma unroll
+  for (int i = 0; i < ATT_BN / 2; ++i) {
+    float a, b;
+    f2_unpack(sp[i], a, b);
+    if (kv0 + 2 * i < first) a = -INFINITY;
+    if (kv0 + 2 * i + 1 < first) b = -INFINITY;
+    sp[i] = f2_pack(a, b);
+  }
+}
+
 __device__ __forceinline__ float att2_row_max(const f32x2 (&sp)[ATT_BN / 2]) {
   float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;   // four independent chains
 #pragma unroll
@@ -79,6 +91,37 @@ __device__ __forceinline__ float att2_row_max(const f32x2 (&sp)[ATT_BN / 2]) {
     m3 = max3(m3, a, b);
   }
   return fmaxf(max3(m0, m1, m2), m3);
+}
+
+// ---------------------------------------------------------------- window, sink, output gate
+// A query that sees `len` keys through a window sees keys first_visible .. len - 1 (window 0: all of them).
+__device__ __forceinline__ int first_visible(int len, int window) { return window > 0 ? max(0, len - window) : 0; }
+
+// A head's sink joins the softmax: exp(sink) in the denominator, no key, no value, no scale.  m, l and acc are the
+// running maximum (in powers of two), the sum and an output element relative to that maximum.
+__device__ __forceinline__ void sink_join(const float* sink, int head, float& m, float& l, float& acc) {
+  if (!sink) return;
+  const float s2 = sink[head] * 1.4426950408889634f;
+  const float mm = fmaxf(m, s2);
+  const float sc = m == -INFINITY ? 0.f : exp2f(m - mm);
+  l = l * sc + exp2f(s2 - mm);
+  acc *= sc;
+  m = mm;
+}
+
+// Output gate: element d of head h of a row is multiplied by sigmoid(g[row * ld + h * head + d * elem]).
+struct HeadGate {
+  const void* g;       // null: no gate
+  long long ld;
+  int head, elem;      // strides; elem 0: one number per head
+  __device__ __forceinline__ long long at(int row, int h, int d) const {
+    return row * ld + static_cast<long long>(h) * head + static_cast<long long>(d) * elem;
+  }
+};
+__device__ __forceinline__ float gate_value(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float head_gate_bf16(const HeadGate& gt, int row, int head, int d) {
+  if (!gt.g) return 1.f;
+  return gate_value(__bfloat162float(static_cast<const __nv_bfloat16*>(gt.g)[gt.at(row, head, d)]));
 }
 
 }  // namespace ft

@@ -1,0 +1,284 @@
+// Row kernels of pre-norm decoders with an fp32 residual stream:
+//
+//   ft_rms_rows        RMS norm of residual rows, optionally gathering the rows first (the embedding,
+//                      or the rows whose logits are wanted) and optionally adding pending terms to the
+//                      residual (the outputs of a token's experts), all in one pass over the row.
+//   ft_qkv_head_finish everything between a packed projection [ q | k | v | .. ] and its attention:
+//                      per-head RMS norm of q and k, rotation of the first 2 * half elements of a head
+//                      by a cos / sin table, k and v into their cache pages.
+//
+// Rows are bf16 or fp32, arithmetic is fp32.
+#include <initializer_list>
+
+#include "row_vec.cuh"
+
+namespace ft {
+
+constexpr int ROW_THREADS = 256;
+constexpr int ROW_WARPS = ROW_THREADS / 32;
+constexpr int ROW_KEEP = 2;   // vectors of eight elements a thread keeps in registers (rows up to 4096 wide)
+
+struct RmsRowsParams {
+  const void* x;            // [n_src, ldx]
+  const long long* ids;     // row i reads x[ids[i]] (null: x[i])
+  float* x_out;             // fp32 [rows, ldo]: the row with its terms (may be x itself); null: not written
+  const void* terms;        // [.., ldt]: row i gains terms[where[source row * n_terms + j]], j < n_terms
+  const int* where;
+  const float* w;
+  void* y;                  // [rows, ldy]
+  long long ldx, ldo, ldt, ldy;
+  int rows, n_src, H, count, n_terms, term_rows;
+  float eps, offset;
+};
+
+// y = x / sqrt(sum(x^2) / count + eps) * (offset + w).  One block per row.
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(ROW_THREADS)
+rms_rows_kernel(const RmsRowsParams p) {
+  __shared__ float red[ROW_WARPS];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    long long src = row;
+    if (p.ids) {
+      src = p.ids[row];
+      if (src < 0 || src >= p.n_src) src = 0;    // host validates; never read out of range
+    }
+    const TI* xr = static_cast<const TI*>(p.x) + src * p.ldx;
+    float* xo = p.x_out ? p.x_out + static_cast<long long>(row) * p.ldo : nullptr;
+    TO* yr = static_cast<TO*>(p.y) + static_cast<long long>(row) * p.ldy;
+    auto fetch = [&](int i, float (&f)[8]) {
+      load8(xr + i, f);
+      for (int j = 0; j < p.n_terms; ++j) {
+        const int t = p.where[src * p.n_terms + j];
+        if (t < 0 || t >= p.term_rows) continue;
+        float g[8];
+        load8(static_cast<const TO*>(p.terms) + static_cast<long long>(t) * p.ldt + i, g);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] += g[e];
+      }
+    };
+    float kept[ROW_KEEP][8];
+    float sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < ROW_KEEP; ++k) {
+      const int i = (k * ROW_THREADS + threadIdx.x) * 8;
+      if (i < p.H) {
+        fetch(i, kept[k]);
+        if (xo) store8(xo + i, kept[k]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += kept[k][e] * kept[k][e];
+      }
+    }
+    const int rest = ROW_KEEP * ROW_THREADS * 8 + threadIdx.x * 8;
+    // wider rows: the tail is summed here and fetched once more below (a thread owns the same columns in both
+    // passes, so with x_out == x it must not add the terms again)
+    for (int i = rest; i < p.H; i += ROW_THREADS * 8) {
+      float f[8];
+      fetch(i, f);
+      if (xo) store8(xo + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum += f[e] * f[e];
+    }
+    sum = warp_sum(sum);
+    __syncthreads();                       // the previous row's sums have been read
+    if (lane == 0) red[warp] = sum;
+    __syncthreads();
+    sum = 0.f;
+#pragma unroll
+    for (int w = 0; w < ROW_WARPS; ++w) sum += red[w];
+    const float r = 1.f / sqrtf(sum / static_cast<float>(p.count) + p.eps);
+#pragma unroll
+    for (int k = 0; k < ROW_KEEP; ++k) {
+      const int i = (k * ROW_THREADS + threadIdx.x) * 8;
+      if (i < p.H) {
+        float w[8];
+        load8(p.w + i, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[e] = kept[k][e] * r * (p.offset + w[e]);
+        store8(yr + i, w);
+      }
+    }
+    for (int i = rest; i < p.H; i += ROW_THREADS * 8) {
+      float f[8], w[8];
+      if (xo) load8(static_cast<const float*>(xo) + i, f); else fetch(i, f);
+      load8(p.w + i, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[e] = f[e] * r * (p.offset + w[e]);
+      store8(yr + i, w);
+    }
+  }
+}
+
+// ---------------------------------------------------------------- packed projection -> attention, per head
+struct HeadFinishParams {
+  void* packed;             // [rows, ld]
+  long long ld;
+  const int* pos;
+  const int* slots;
+  const int* block_table;
+  void* k_cache;            // null: the layer has queries only (it reads another layer's pages)
+  void* v_cache;
+  const float* q_weight;    // [D]; null: no norm
+  const float* k_weight;
+  const float2* table;      // [positions, half]: cos, sin; null: no rotation
+  int rows, q_off, Hq, k_off, v_off, Hkv, D, Dv, d_true, half, positions;
+  float eps;
+  int block_size, max_blocks, num_blocks;
+};
+
+// A warp owns one head of one row at a time: q heads, then k heads, then v heads.  The head goes through shared
+// memory in fp32 because rotation pairs element i with i + half, in another lane.
+template <typename T>
+__global__ void __launch_bounds__(ROW_THREADS)
+qkv_head_finish_kernel(const HeadFinishParams p) {
+  extern __shared__ float head_sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* s = head_sm + warp * p.D;
+  const int tasks = p.Hq + (p.k_cache ? 2 * p.Hkv : 0);
+  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    T* y = static_cast<T*>(p.packed) + static_cast<long long>(row) * p.ld;
+    const int position = p.pos[row];
+    long long token = -1;
+    if (p.k_cache) {
+      const int blk = p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + position / p.block_size];
+      if (blk >= 0 && blk < p.num_blocks) token = static_cast<long long>(blk) * p.block_size + position % p.block_size;
+    }
+    const float2* cs = p.table ? p.table + static_cast<long long>(min(position, p.positions - 1)) * p.half : nullptr;
+    for (int task = blockIdx.y * ROW_WARPS + warp; task < tasks; task += gridDim.y * ROW_WARPS) {
+      if (task >= p.Hq + p.Hkv) {
+        const int h = task - p.Hq - p.Hkv;
+        if (token >= 0)
+          for (int i = lane * 8; i < p.Dv; i += 256) {
+            float f[8];
+            load8(y + p.v_off + h * p.Dv + i, f);
+            store8(static_cast<T*>(p.v_cache) + (token * p.Hkv + h) * p.Dv + i, f);
+          }
+        continue;
+      }
+      const bool is_q = task < p.Hq;
+      const int h = is_q ? task : task - p.Hq;
+      if (!is_q && token < 0) continue;
+      T* src = y + (is_q ? p.q_off : p.k_off) + h * p.D;
+      T* dst = is_q ? src : static_cast<T*>(p.k_cache) + (token * p.Hkv + h) * p.D;
+      const float* w = is_q ? p.q_weight : p.k_weight;
+      float sum = 0.f;
+      for (int i = lane * 8; i < p.D; i += 256) {
+        float f[8];
+        load8(src + i, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          sum += f[e] * f[e];
+          s[i + e] = f[e];
+        }
+      }
+      float r = 1.f;
+      if (w) r = 1.f / sqrtf(warp_sum(sum) / static_cast<float>(p.d_true) + p.eps);
+      __syncwarp();
+      for (int i = lane * 8; i < p.D; i += 256) {
+        float f[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const int d = i + e;
+          float v = w ? s[d] * r * w[d] : s[d];
+          if (cs && d < 2 * p.half) {
+            const int j = d < p.half ? d : d - p.half, o = d < p.half ? d + p.half : j;
+            const float other = w ? s[o] * r * w[o] : s[o];
+            const float2 t = cs[j];
+            v = d < p.half ? v * t.x - other * t.y : v * t.x + other * t.y;
+          }
+          f[e] = v;
+        }
+        store8(dst + i, f);
+      }
+      __syncwarp();
+    }
+  }
+}
+
+}  // namespace ft
+
+using namespace ft;
+
+static bool row_aligned(std::initializer_list<const void*> ps) {
+  uintptr_t v = 0;
+  for (const void* p : ps) v |= reinterpret_cast<uintptr_t>(p);
+  return (v & 15) == 0;
+}
+
+// y[rows, H] (bf16, or fp32 with out_f32) = RMS norm of x rows times (offset + w).  x: fp32, or bf16 with in_bf16,
+// [n_src, ldx]; ids (int64 [rows] or null): the rows to take.  terms ([term_rows, ldt], type of y) and where (int32
+// [n_src, n_terms]; entries outside 0 .. term_rows - 1 add nothing): added to the row first.  x_out: fp32 [rows,
+// ldo] receives the row with its terms, and may be x when ids is null.  count: true width (padding is zero).
+FT_API int ft_rms_rows(const void* x, const long long* ids, int n_src, int in_bf16, float* x_out, const void* terms,
+                       const int* where, int n_terms, int term_rows, const float* w, void* y, int out_f32, int rows, int H,
+                       int count, long long ldx, long long ldo, long long ldt, long long ldy, float eps, float offset,
+                       int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(x && w && y, "ft_rms_rows: null pointer");
+  FT_REQUIRE(H > 0 && H % 8 == 0 && count > 0 && count <= H && ((ldx | ldo | ldt | ldy) & 7) == 0 && ldx >= H && ldy >= H,
+             "ft_rms_rows: H=%d and strides must be multiples of 8", H);
+  FT_REQUIRE(n_terms == 0 || (terms && where && n_terms > 0 && ldt >= H && term_rows > 0), "ft_rms_rows: terms without their rows");
+  FT_REQUIRE(!x_out || ldo >= H, "ft_rms_rows: row stride of the residual");
+  FT_REQUIRE(row_aligned({x, x_out, terms, w, y}), "ft_rms_rows: pointers must be 16-byte aligned");
+  FT_REQUIRE(n_src > 0 && (ids || rows <= n_src), "ft_rms_rows: %d source rows", n_src);
+  if (rows <= 0) return FT_E_OK;
+  RmsRowsParams p;
+  p.x = x; p.ids = ids; p.x_out = x_out; p.terms = terms; p.where = where; p.w = w; p.y = y;
+  p.ldx = ldx; p.ldo = ldo; p.ldt = ldt; p.ldy = ldy;
+  p.rows = rows; p.n_src = n_src; p.H = H; p.count = count; p.n_terms = n_terms; p.term_rows = term_rows;
+  p.eps = eps; p.offset = offset;
+  const int cap = sm_count(device) * 8;
+  const int grid = rows < cap ? rows : cap;
+  if (in_bf16) {
+    if (out_f32) rms_rows_kernel<__nv_bfloat16, float><<<grid, ROW_THREADS, 0, stream>>>(p);
+    else rms_rows_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, ROW_THREADS, 0, stream>>>(p);
+  } else {
+    if (out_f32) rms_rows_kernel<float, float><<<grid, ROW_THREADS, 0, stream>>>(p);
+    else rms_rows_kernel<float, __nv_bfloat16><<<grid, ROW_THREADS, 0, stream>>>(p);
+  }
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// The pass between a packed projection and its attention (see qkv_head_finish_kernel).  packed and caches are bf16, or
+// fp32 with f32; offsets in elements, multiples of 8; head sizes D / Dv multiples of 8 of which d_true elements of a q
+// or k head exist (padding is zero).  k_cache null: no keys and values in the row.  table: fp32 pairs (cos, sin)
+// [positions, half] or null.
+FT_API int ft_qkv_head_finish(void* packed, long long ld, const int* pos, const int* slots, const int* block_table,
+                              void* k_cache, void* v_cache, const float* q_weight, const float* k_weight, const void* table,
+                              int rows, int q_off, int Hq, int k_off, int v_off, int Hkv, int D, int Dv, int d_true, int half,
+                              int positions, float eps, int f32, int block_size, int max_blocks, int num_blocks, int device,
+                              cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(packed && pos && (!k_cache || (v_cache && slots && block_table)), "ft_qkv_head_finish: null pointer");
+  FT_REQUIRE(((q_off | k_off | v_off | D | Dv) & 7) == 0 && ld % 8 == 0, "ft_qkv_head_finish: offsets, sizes and strides must be multiples of 8");
+  FT_REQUIRE(Hq > 0 && D > 0 && D <= 1024 && d_true > 0 && d_true <= D && q_off >= 0 && q_off + static_cast<long long>(Hq) * D <= ld,
+             "ft_qkv_head_finish: the queries lie outside the row");
+  FT_REQUIRE(!k_cache || (Hkv > 0 && Dv > 0 && k_off >= 0 && v_off >= 0 && k_off + static_cast<long long>(Hkv) * D <= ld &&
+                          v_off + static_cast<long long>(Hkv) * Dv <= ld && block_size > 0 && max_blocks > 0 && num_blocks > 0),
+             "ft_qkv_head_finish: the keys or values lie outside the row");
+  FT_REQUIRE(!table || (half > 0 && 2 * half <= d_true && positions > 0), "ft_qkv_head_finish: rotation of %d elements of %d", 2 * half, d_true);
+  FT_REQUIRE(row_aligned({packed, k_cache, v_cache}) && (reinterpret_cast<uintptr_t>(table) & 7) == 0,
+             "ft_qkv_head_finish: pointers must be 16-byte aligned");
+  if (rows <= 0) return FT_E_OK;
+  HeadFinishParams p;
+  p.packed = packed; p.ld = ld; p.pos = pos; p.slots = slots; p.block_table = block_table;
+  p.k_cache = k_cache; p.v_cache = v_cache; p.q_weight = q_weight; p.k_weight = k_weight;
+  p.table = static_cast<const float2*>(table);
+  p.rows = rows; p.q_off = q_off; p.Hq = Hq; p.k_off = k_off; p.v_off = v_off; p.Hkv = k_cache ? Hkv : 0;
+  p.D = D; p.Dv = Dv; p.d_true = d_true; p.half = half; p.positions = positions; p.eps = eps;
+  p.block_size = block_size; p.max_blocks = max_blocks; p.num_blocks = num_blocks;
+  // heads of a row are spread over blocks when the rows alone do not fill the GPU
+  const int wave = sm_count(device) * 8;
+  const int tasks = Hq + 2 * p.Hkv;
+  int parts = (tasks + ROW_WARPS - 1) / ROW_WARPS;
+  if (parts > wave / rows) parts = wave / rows > 1 ? wave / rows : 1;
+  const dim3 grid(rows < wave ? rows : wave, parts);
+  const size_t smem = static_cast<size_t>(ROW_WARPS) * D * sizeof(float);
+  if (f32) qkv_head_finish_kernel<float><<<grid, ROW_THREADS, smem, stream>>>(p);
+  else qkv_head_finish_kernel<__nv_bfloat16><<<grid, ROW_THREADS, smem, stream>>>(p);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}

@@ -44,6 +44,8 @@ enum GemmFlags : int {
   GEMM_RELU = 16,       // activation fused in the epilogue (after bias)
   GEMM_GELU = 32,
   GEMM_SILU = 64,
+  GEMM_RELU2 = 128,     // max(v, 0)^2
+  GEMM_ACT_MASK = GEMM_RELU | GEMM_GELU | GEMM_SILU | GEMM_RELU2,
   GEMM_EPI_DIRECT = 1 << 16,  // internal: per-lane read-modify-write epilogue
   GEMM_EPI_TRANSPOSED = 1 << 17,  // internal: the tile holds C^T; lane = column of C, register = row of C
 };
@@ -98,6 +100,7 @@ __device__ __forceinline__ float apply_act(float v, int flags) {
   if (flags & GEMM_RELU) return fmaxf(v, 0.f);
   if (flags & GEMM_GELU) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
   if (flags & GEMM_SILU) return v / (1.f + __expf(-v));
+  if (flags & GEMM_RELU2) return fmaxf(v, 0.f) * fmaxf(v, 0.f);
   return v;
 }
 
@@ -112,7 +115,7 @@ __device__ __forceinline__ void epilogue_direct(const GemmParams& p, uint32_t t_
   const bool out_f32 = (p.flags & GEMM_OUT_F32) != 0;
   const bool accumulate = (p.flags & GEMM_ACCUMULATE) != 0;
   const bool has_bias = (p.flags & (GEMM_BIAS | GEMM_BIAS_F32)) != 0;
-  const bool has_act = (p.flags & (GEMM_RELU | GEMM_GELU | GEMM_SILU)) != 0;
+  const bool has_act = (p.flags & GEMM_ACT_MASK) != 0;
 #pragma unroll 1
   for (int c = 0; c < BN / 32; ++c) {
     uint32_t r[32];
@@ -189,7 +192,7 @@ template <int BN>
 __device__ __forceinline__ void epilogue_crop(const GemmParams& p, uint32_t t_row, int row, int n0) {
   const bool out_f32 = (p.flags & GEMM_OUT_F32) != 0;
   const bool has_bias = (p.flags & (GEMM_BIAS | GEMM_BIAS_F32)) != 0;
-  const bool has_act = (p.flags & (GEMM_RELU | GEMM_GELU | GEMM_SILU)) != 0;
+  const bool has_act = (p.flags & GEMM_ACT_MASK) != 0;
   bool row_ok = row < p.M;
   long long dst_row = 0;
   {
@@ -255,7 +258,7 @@ template <int BN>
 __device__ __forceinline__ void epilogue_transposed(const GemmParams& p, uint32_t t_row, int n_idx, int m0) {
   const bool n_ok = n_idx < p.M;
   const bool has_bias = (p.flags & (GEMM_BIAS | GEMM_BIAS_F32)) != 0;
-  const bool has_act = (p.flags & (GEMM_RELU | GEMM_GELU | GEMM_SILU)) != 0;
+  const bool has_act = (p.flags & GEMM_ACT_MASK) != 0;
   float bias = 0.f;
   if (has_bias && n_ok)
     bias = (p.flags & GEMM_BIAS_F32) ? static_cast<const float*>(p.bias)[n_idx]
@@ -705,7 +708,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
     const bool out_f32 = (p.flags & GEMM_OUT_F32) != 0;
     const bool accumulate = (p.flags & GEMM_ACCUMULATE) != 0;
     const bool has_bias = (p.flags & (GEMM_BIAS | GEMM_BIAS_F32)) != 0;
-    const bool has_act = (p.flags & (GEMM_RELU | GEMM_GELU | GEMM_SILU)) != 0;
+    const bool has_act = (p.flags & GEMM_ACT_MASK) != 0;
     const bool direct = (p.flags & GEMM_EPI_DIRECT) != 0;
     const uint32_t stage_tiles = smem_u32(epi) + static_cast<uint32_t>(ew) * 2u * Cfg::EPI_TILE_BYTES;
     int buf = 0;
@@ -921,7 +924,7 @@ FT_API int ft_gemm_bf16(const void* A, const void* B, void* C, const void* bias,
   FT_REQUIRE(!(flags & (GEMM_BIAS | GEMM_BIAS_F32)) || bias, "ft_gemm_bf16: bias flag without bias");
   const bool force_single = bn < 0;
   if (force_single) bn = -bn;
-  const bool has_act = (flags & (GEMM_RELU | GEMM_GELU | GEMM_SILU)) != 0;
+  const bool has_act = (flags & GEMM_ACT_MASK) != 0;
   const bool accumulate = (flags & GEMM_ACCUMULATE) != 0;
   flags &= 0xFFFF;
 
@@ -1106,11 +1109,11 @@ FT_API int ft_conv_shift_wgrad(const void* dyp, const void* xp, float* dw, long 
 namespace ft {
 
 // ws holds the pieces of the split contraction: C^T as fp32 [ksplit][slice_rows >= N, ld_ws].  Write
-// C[m, n] = sum_ks ws[ks][n, m] (+ bias[n]) (+ residual[m, n]) as bf16; the pieces are summed in
+// C[m, n] = act(sum_ks ws[ks][n, m] (+ bias[n]) (+ residual[m, n])) as bf16; the pieces are summed in
 // index order, so the result does not depend on which CTA finished first.
 __global__ void small_m_finalize_kernel(const float* __restrict__ ws, __nv_bfloat16* __restrict__ C,
                                         const __nv_bfloat16* __restrict__ residual, const void* __restrict__ bias,
-                                        int bias_f32, int M, int N, int ld_ws, int ksplit, int slice_rows,
+                                        int flags, int M, int N, int ld_ws, int ksplit, int slice_rows,
                                         long long ldc, long long ldr) {
   // block = 32 x 8 threads over a 32 (n) x 32 (m) patch, transposed through shared memory
   __shared__ float tile[32][33];
@@ -1130,9 +1133,9 @@ __global__ void small_m_finalize_kernel(const float* __restrict__ ws, __nv_bfloa
     const int m = m0 + i, n = n0 + threadIdx.x;
     if (m < M && n < N) {
       float v = tile[threadIdx.x][i];
-      if (bias) v += bias_f32 ? static_cast<const float*>(bias)[n] : __bfloat162float(static_cast<const __nv_bfloat16*>(bias)[n]);
+      if (bias) v += (flags & GEMM_BIAS_F32) ? static_cast<const float*>(bias)[n] : __bfloat162float(static_cast<const __nv_bfloat16*>(bias)[n]);
       if (residual) v += __bfloat162float(residual[static_cast<long long>(m) * ldr + n]);
-      C[static_cast<long long>(m) * ldc + n] = __float2bfloat16(v);
+      C[static_cast<long long>(m) * ldc + n] = __float2bfloat16(apply_act(v, flags));
     }
   }
 }
@@ -1293,7 +1296,7 @@ FT_API int ft_gemm_small_m(const void* X, const void* W, void* C, const void* bi
   dim3 grid((N + 31) / 32, (M + 31) / 32), block(32, 8);
   small_m_finalize_kernel<<<grid, block, 0, stream>>>(workspace, static_cast<__nv_bfloat16*>(C),
                                                       static_cast<const __nv_bfloat16*>(residual), bias,
-                                                      (flags & GEMM_BIAS_F32) ? 1 : 0, M, N, bn, ksplit,
+                                                      flags, M, N, bn, ksplit,
                                                       (N + 255) / 256 * 256, ldc, ldr);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();

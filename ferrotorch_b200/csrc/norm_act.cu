@@ -13,8 +13,7 @@
 // Unlike the reference (one launch per op, 256-thread 1-D grids) every kernel moves
 // 16-byte vectors, keeps the row in registers between the statistics pass and the
 // scale pass, and fuses the neighbouring residual add / gate multiply.
-#include "ft_host.h"
-#include "ft_ptx.cuh"
+#include "row_vec.cuh"
 
 namespace ft {
 
@@ -50,16 +49,6 @@ __device__ __forceinline__ float block_max(float v, float* red) {
   return red[0];
 }
 
-__device__ __forceinline__ void unpack8(const uint4& u, float* f) {
-  float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y), c = unpack_bf16x2(u.z), d = unpack_bf16x2(u.w);
-  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
-}
-__device__ __forceinline__ uint4 pack8(const float* f) {
-  uint4 u;
-  u.x = pack_bf16x2(f[0], f[1]); u.y = pack_bf16x2(f[2], f[3]);
-  u.z = pack_bf16x2(f[4], f[5]); u.w = pack_bf16x2(f[6], f[7]);
-  return u;
-}
 
 // ---------------------------------------------------------------- RMSNorm forward
 // y = (x [+ delta]) * rstd * w ; if delta != null also writes res_out = x + delta.
@@ -422,20 +411,6 @@ __global__ void embedding_bwd_kernel(const long long* __restrict__ ids, const __
   }
 }
 
-// ---------------------------------------------------------------- 8-element rows of either dtype
-__device__ __forceinline__ void load8(const __nv_bfloat16* p, float* f) {
-  unpack8(*reinterpret_cast<const uint4*>(p), f);
-}
-__device__ __forceinline__ void load8(const float* p, float* f) {
-  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-}
-__device__ __forceinline__ void store8(__nv_bfloat16* p, const float* f) { *reinterpret_cast<uint4*>(p) = pack8(f); }
-__device__ __forceinline__ void store8(float* p, const float* f) {
-  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
-  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
-}
-
 // ---------------------------------------------------------------- dynamic tanh
 // y = (tanh(alpha * x) * w + b) * scale, element by element (no row statistic), fp32 input and
 // parameters.  With `ids` the input row is table[ids[row]] (a row of the embedding, TI) and is also
@@ -593,14 +568,6 @@ qkv_finish_kernel(const QkvFinishParams p) {
       }
     }
   }
-}
-
-static inline int blocks_for(long long work, int threads, int device, int per_sm = 8) {
-  long long b = (work + threads - 1) / threads;
-  const long long cap = static_cast<long long>(sm_count(device)) * per_sm;
-  if (b > cap) b = cap;
-  if (b < 1) b = 1;
-  return static_cast<int>(b);
 }
 
 }  // namespace ft

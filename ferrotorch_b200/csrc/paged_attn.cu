@@ -13,6 +13,8 @@
 //                       context, GQA (all query heads of a KV group share one pass over K/V),
 //                       flash-decoding split over the context with a second combine pass, and an
 //                       optional output gate per head.
+//                       A row may see a window of the most recent keys only, and a learned number
+//                       per head (a sink) may join the denominator.
 //   ft_paged_rows       the same for any mixture of rows (each with its own sequence and number of
 //                       visible keys), any head sizes, bf16 or fp32: the exact, simple kernel.
 // Decode attention is bandwidth bound (every cached byte is read once per step).  Key / value head
@@ -20,24 +22,13 @@
 // (paged_decode_tc_kernel: cp.async rows -> shared memory -> tcgen05.mma).  The CUDA-core kernel for
 // equal sizes of 64 or 128 reads K with one key per lane (full rows, no shuffles in the dot products)
 // and V with one row per warp step; it serves size 64, and queries that are not 16-byte aligned.
+#include "attn_row.cuh"
 #include "ft_host.h"
-#include "ft_ptx.cuh"
 
 namespace ft {
 
 constexpr int PD_THREADS = 128;
 constexpr int PD_WARPS = PD_THREADS / 32;
-
-// Output gate: head h of a row is multiplied by sigmoid(gate[row, h]) when a gate is given.
-struct HeadGate {
-  const void* g;       // null: no gate
-  long long ld;        // row stride in elements
-};
-__device__ __forceinline__ float gate_value(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float head_gate_bf16(const HeadGate& gt, int row, int head) {
-  if (!gt.g) return 1.f;
-  return gate_value(__bfloat162float(static_cast<const __nv_bfloat16*>(gt.g)[static_cast<long long>(row) * gt.ld + head]));
-}
 
 // k_new / v_new: rows of kv16 / vv16 16-byte units (all KV heads of a token) with token strides ldk16 / ldv16 units.
 // Token i goes to sequence seq_ids[i] (or i / tokens_per_seq when null) at position pos[i].
@@ -70,15 +61,17 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
                     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_table,
                     const int* __restrict__ row_slot, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
                     float* __restrict__ part_o, float* __restrict__ part_ml, int Hq, int Hkv, long long ldq, long long ldo,
-                    int block_size, int max_blocks, int num_blocks, float scale_log2, int n_splits, HeadGate gate) {
+                    int block_size, int max_blocks, int num_blocks, float scale_log2, int n_splits, int window,
+                    const float* __restrict__ sink, HeadGate gate) {
   constexpr int DV = D / 16;  // dims per lane in the PV phase (half-warp covers D)
   const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int half = lane >> 4, hl = lane & 15;
   const int len = ctx_len[b];
-  const int tiles_total = (len + 31) >> 5;
-  const int tiles_per_split = (tiles_total + n_splits - 1) / n_splits;
-  const int tile_lo = split * tiles_per_split, tile_hi = min(tiles_total, tile_lo + tiles_per_split);
+  const int first = first_visible(len, window);
+  const int tiles_end = (len + 31) >> 5;
+  const int tiles_per_split = (tiles_end - (first >> 5) + n_splits - 1) / n_splits;
+  const int tile_lo = (first >> 5) + split * tiles_per_split, tile_hi = min(tiles_end, tile_lo + tiles_per_split);
 
   __shared__ __align__(16) float s_q[G][D];          // q * scale * log2(e)
   __shared__ float s_p[PD_WARPS][G][32];             // probabilities of the current tile
@@ -106,12 +99,12 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     const int key0 = tile << 5;
     // ---- scores: lane j owns key key0 + j; issue the whole row's loads, then the dot products
     const int key = key0 + lane;
-    const bool valid = key < len;
+    const bool valid = key < len && key >= first;
     float s[G];
 #pragma unroll
     for (int g = 0; g < G; ++g) s[g] = 0.f;
     {
-      const int kk = valid ? key : key0;
+      const int kk = key < len ? key : key0;
       int blk = bt[kk / block_size];
       blk = min(max(blk, 0), num_blocks - 1);
       const uint4* kr = reinterpret_cast<const uint4*>(
@@ -216,8 +209,9 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     }
     const int hq = kvh * G + g;
     if (n_splits == 1) {
+      sink_join(sink, hq, mm, ll, acc);
       out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] =
-          __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq) : 0.f);
+          __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq, d) : 0.f);
     } else {
       const long long pidx = (static_cast<long long>(b) * Hq + hq) * n_splits + split;
       part_o[pidx * D + d] = acc;
@@ -228,7 +222,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 
 __global__ void paged_decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                             __nv_bfloat16* __restrict__ out, int Hq, int D, long long ldo, int n_splits,
-                                            HeadGate gate) {
+                                            const float* __restrict__ sink, HeadGate gate) {
   const int hq = blockIdx.x, b = blockIdx.y;
   const long long base = (static_cast<long long>(b) * Hq + hq) * n_splits;
   float mm = -INFINITY;
@@ -241,8 +235,10 @@ __global__ void paged_decode_combine_kernel(const float* __restrict__ part_o, co
       ll += part_ml[(base + s) * 2 + 1] * sc;
       acc += part_o[(base + s) * D + d] * sc;
     }
+    float m = mm;
+    sink_join(sink, hq, m, ll, acc);
     out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] =
-        __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq) : 0.f);
+        __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq, d) : 0.f);
   }
 }
 
@@ -299,7 +295,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
                        const int* __restrict__ row_slot, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
                        float* __restrict__ part_o, float* __restrict__ part_ml, int Hq, int Hkv, int D, int Dv, int g_real,
                        long long ldq, long long ldo, int block_size, int max_blocks, int num_blocks, float scale_log2,
-                       int n_splits, HeadGate gate, int* status) {
+                       int n_splits, int window, const float* __restrict__ sink, HeadGate gate, int* status) {
   using Cfg = PtCfg<HD>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -317,10 +313,11 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
   const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int len = ctx_len[b];
-  const int tiles_total = (len + PT_TILE - 1) / PT_TILE;
-  const int tiles_per_split = (tiles_total + n_splits - 1) / n_splits;
-  const int tile_lo = split * tiles_per_split;
-  const int n_tiles = max(0, min(tiles_total, tile_lo + tiles_per_split) - tile_lo);
+  const int first = first_visible(len, window);
+  const int tiles_end = (len + PT_TILE - 1) / PT_TILE;
+  const int tiles_per_split = (tiles_end - first / PT_TILE + n_splits - 1) / n_splits;
+  const int tile_lo = first / PT_TILE + split * tiles_per_split;
+  const int n_tiles = max(0, min(tiles_end, tile_lo + tiles_per_split) - tile_lo);
 
   if (threadIdx.x == 0) {
     *abort_word = 0;
@@ -481,7 +478,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
         tmem_ld_wait();
       }
       const int key = (tile_lo + t) * PT_TILE + r;
-      const bool valid = key < len;
+      const bool valid = key < len && key >= first;
       float s[G], mx[G];
 #pragma unroll
       for (int g = 0; g < G; ++g) {
@@ -565,8 +562,10 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
         const int hq = kvh * g_real + g;
         const float acc = __uint_as_float(ov[g]);
         if (n_splits == 1) {
+          float mm = m_ref[g], ll = l_tot[g], o = acc;
+          sink_join(sink, hq, mm, ll, o);
           out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * Dv + r] =
-              __float2bfloat16(l_tot[g] > 0.f ? acc / l_tot[g] * head_gate_bf16(gate, b, hq) : 0.f);
+              __float2bfloat16(ll > 0.f ? o / ll * head_gate_bf16(gate, b, hq, r) : 0.f);
         } else {
           const long long pidx = (static_cast<long long>(b) * Hq + hq) * n_splits + split;
           part_o[pidx * Dv + r] = acc;
@@ -586,7 +585,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
 }
 
 // ----------------------------------------------------------------------------- any rows, any sizes
-// Row i attends to keys 0 .. visible[i] - 1 of sequence row_slot[i].  A CTA owns one row and up to
+// Row i attends to keys 0 .. visible[i] - 1 of sequence row_slot[i] (the last `window` of them).  A CTA owns one row and up to
 // PR_HEADS query heads of one KV head; its four warps walk tiles of 32 keys (lane = key while scoring,
 // lane = value dim while accumulating) with an fp32 online softmax each, merged at the end.
 constexpr int PR_HEADS = 8;
@@ -601,7 +600,8 @@ __global__ void __launch_bounds__(PD_THREADS)
 paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                   const int* __restrict__ block_table, const int* __restrict__ row_slot, const int* __restrict__ visible,
                   HeadGate gate, T* __restrict__ out, int rows, int Hq, int Hkv, int D, int Dv, long long ldq, long long ldo,
-                  int block_size, int max_blocks, int num_blocks, float scale, int head_groups) {
+                  int block_size, int max_blocks, int num_blocks, float scale, int window, const float* __restrict__ sink,
+                  int head_groups) {
   extern __shared__ float sm[];
   const int g_all = Hq / Hkv;
   const int kvh = blockIdx.y / head_groups, h0 = (blockIdx.y % head_groups) * PR_HEADS;
@@ -615,6 +615,7 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
   for (int row = blockIdx.x; row < rows; row += gridDim.x) {
     __syncthreads();
     const int len = min(visible[row], max_blocks * block_size);
+    const int first = first_visible(len, window);
     const int* bt = block_table + static_cast<long long>(row_slot[row]) * max_blocks;
     for (int i = threadIdx.x; i < g * D; i += PD_THREADS) {
       const int h = i / D, d = i - h * D;
@@ -626,10 +627,10 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
 #pragma unroll
     for (int h = 0; h < PR_HEADS; ++h) { m[h] = -INFINITY; l[h] = 0.f; }
     __syncthreads();
-    for (int key0 = warp * 32; key0 < len; key0 += PD_WARPS * 32) {
+    for (int key0 = first / 32 * 32 + warp * 32; key0 < len; key0 += PD_WARPS * 32) {
       const int key = key0 + lane;
-      const bool valid = key < len;
-      const int kk = valid ? key : key0;
+      const bool valid = key < len && key >= first;
+      const int kk = key < len ? key : key0;
       const int blk = min(max(bt[kk / block_size], 0), num_blocks - 1);
       const T* kr = k_cache + ((static_cast<long long>(blk) * block_size + kk % block_size) * Hkv + kvh) * D;
       float s[PR_HEADS];
@@ -696,8 +697,9 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
         acc += s_o[(w * PR_HEADS + h) * Dv + d] * sc;
       }
       const int hq = kvh * g_all + h0 + h;
+      sink_join(sink, hq, mm, ll, acc);
       float v = ll > 0.f ? acc / ll : 0.f;
-      if (gate.g) v *= gate_value(to_f32(static_cast<const T*>(gate.g)[static_cast<long long>(row) * gate.ld + hq]));
+      if (gate.g) v *= gate_value(to_f32(static_cast<const T*>(gate.g)[gate.at(row, hq, d)]));
       from_f32(v, out + static_cast<long long>(row) * ldo + static_cast<long long>(hq) * Dv + d);
     }
   }
@@ -737,16 +739,19 @@ FT_API long long ft_paged_decode_scratch(int B, int Hq, int Dv, int n_splits) {
 }
 
 // q: [B, Hq, D] (row stride ldq), out: [B, Hq, Dv] (row stride ldo), ctx_len: int32 [B] = number of
-// cached tokens to attend to (including the current one, which must already be appended).  Row b reads
-// sequence row_slot[b] of the block table (null: sequence b).  gate (bf16 [B, Hq], row stride ldg, or
-// null): output heads are multiplied by sigmoid(gate).
+// cached tokens to attend to (including the current one, which must already be appended), of which the last
+// `window` are visible (0: all).  Row b reads sequence row_slot[b] of the block table (null: sequence b).  sink
+// (fp32 [Hq] or null): exp(sink) joins a head's denominator.  gate (bf16 or null): element d of head h of row b is
+// multiplied by sigmoid(gate[b * ldg + h * gate_head + d * gate_elem]); one number per head with gate_elem 0.
 FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
-                           const int* row_slot, const int* ctx_len, const void* gate, void* out, float* scratch, int B,
-                           int Hq, int Hkv, int D, int Dv, long long ldq, long long ldg, long long ldo, int block_size,
-                           int max_blocks, int num_blocks, float scale, int n_splits, int device, cudaStream_t stream) {
+                           const int* row_slot, const int* ctx_len, const void* gate, const float* sink, void* out,
+                           float* scratch, int B, int Hq, int Hkv, int D, int Dv, long long ldq, long long ldg,
+                           int gate_head, int gate_elem, long long ldo, int block_size, int max_blocks, int num_blocks,
+                           float scale, int window, int n_splits, int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(q && k_cache && v_cache && block_table && ctx_len && out, "ft_paged_decode: null pointer");
   FT_REQUIRE(B >= 0 && Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0, "ft_paged_decode: bad shape");
+  FT_REQUIRE(window >= 0, "ft_paged_decode: negative window");
   FT_REQUIRE(n_splits >= 1 && (n_splits == 1 || scratch), "ft_paged_decode: splits need scratch");
   if (B == 0) return FT_E_OK;
   const float sl2 = scale * 1.4426950408889634f;
@@ -754,7 +759,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
   float* part_ml = scratch ? scratch + static_cast<long long>(B) * Hq * n_splits * Dv : nullptr;
   dim3 grid(n_splits, Hkv, B);
   const int G = Hq / Hkv;
-  const HeadGate hg = {gate, ldg};
+  const HeadGate hg = {gate, ldg, gate_head, gate_elem};
   // equal head sizes of 64 half fill the tensor-core kernel's value tile: the CUDA-core kernel is faster there
   // (127 against 156 us at 64 rows x 2048 keys x 8 KV heads) and keeps P in fp32
   const bool core64 = D == 64 && Dv == 64 && (G == 1 || G == 2 || G == 4 || G == 8) &&
@@ -775,7 +780,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
     kern<<<grid, PT_THREADS, PtCfg<HH>::SMEM_BYTES, stream>>>(                                                  \
         static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache),                \
         static_cast<const __nv_bfloat16*>(q), block_table, row_slot, ctx_len, static_cast<__nv_bfloat16*>(out), \
-        part_o, part_ml, Hq, Hkv, D, Dv, G, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, hg, status); \
+        part_o, part_ml, Hq, Hkv, D, Dv, G, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, window, sink, hg, status); \
   }
 #define FT_PT_BY_G(HH)                     \
   if (G == 1) FT_PT_LAUNCH(HH, 1)          \
@@ -792,7 +797,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
   paged_decode_kernel<DD, GG><<<grid, PD_THREADS, 0, stream>>>(                                                \
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),                        \
       static_cast<const __nv_bfloat16*>(v_cache), block_table, row_slot, ctx_len, static_cast<__nv_bfloat16*>(out), \
-      part_o, part_ml, Hq, Hkv, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, hg)
+      part_o, part_ml, Hq, Hkv, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, window, sink, hg)
 #define FT_PD_BY_G(DD)                                             \
   switch (G) {                                                     \
     case 1: FT_PD_LAUNCH(DD, 1); break;                            \
@@ -811,7 +816,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
   count_launch();
   if (n_splits > 1) {
     dim3 g2(Hq, B);
-    paged_decode_combine_kernel<<<g2, Dv <= 64 ? 64 : 128, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, Dv, ldo, n_splits, hg);
+    paged_decode_combine_kernel<<<g2, Dv <= 64 ? 64 : 128, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, Dv, ldo, n_splits, sink, hg);
     FT_CUDA_CHECK(cudaGetLastError());
     count_launch();
   }
@@ -819,27 +824,29 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
 }
 
 // Attention of arbitrary rows over the paged cache (see paged_rows_kernel): q [rows, Hq, D], out
-// [rows, Hq, Dv], row_slot / visible int32 [rows].  All tensors bf16, or fp32 with f32.
+// [rows, Hq, Dv], row_slot / visible int32 [rows]; window, sink (always fp32) and gate as in ft_paged_decode.  All
+// other tensors bf16, or fp32 with f32.
 FT_API int ft_paged_rows(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* row_slot,
-                         const int* visible, const void* gate, void* out, int rows, int Hq, int Hkv, int D, int Dv,
-                         long long ldq, long long ldg, long long ldo, int block_size, int max_blocks, int num_blocks,
-                         float scale, int f32, int device, cudaStream_t stream) {
+                         const int* visible, const void* gate, const float* sink, void* out, int rows, int Hq, int Hkv,
+                         int D, int Dv, long long ldq, long long ldg, int gate_head, int gate_elem, long long ldo,
+                         int block_size, int max_blocks, int num_blocks, float scale, int window, int f32, int device,
+                         cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(q && k_cache && v_cache && block_table && row_slot && visible && out, "ft_paged_rows: null pointer");
-  FT_REQUIRE(Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && D > 0 && Dv > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0, "ft_paged_rows: bad shape");
+  FT_REQUIRE(Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && D > 0 && Dv > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0 && window >= 0, "ft_paged_rows: bad shape");
   if (rows <= 0) return FT_E_OK;
   const int groups = (Hq / Hkv + PR_HEADS - 1) / PR_HEADS;
   const size_t smem = sizeof(float) * (static_cast<size_t>(PR_HEADS) * D + static_cast<size_t>(PD_WARPS) * PR_HEADS * Dv +
                                        PD_WARPS * PR_HEADS * 32 + 2 * PD_WARPS * PR_HEADS);
   FT_REQUIRE(smem <= 200 * 1024 && static_cast<long long>(Hkv) * groups < 65536, "ft_paged_rows: head sizes %d / %d are too large", D, Dv);
   const dim3 grid(rows < 65536 ? rows : 65536, Hkv * groups);
-  const HeadGate hg = {gate, ldg};
+  const HeadGate hg = {gate, ldg, gate_head, gate_elem};
 #define FT_PR_LAUNCH(T)                                                                                                      \
   {                                                                                                                          \
     FT_CUDA_CHECK(cudaFuncSetAttribute(paged_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     paged_rows_kernel<T><<<grid, PD_THREADS, smem, stream>>>(static_cast<const T*>(q), static_cast<const T*>(k_cache),       \
         static_cast<const T*>(v_cache), block_table, row_slot, visible, hg, static_cast<T*>(out), rows, Hq, Hkv, D, Dv, ldq, \
-        ldo, block_size, max_blocks, num_blocks, scale, groups);                                                             \
+        ldo, block_size, max_blocks, num_blocks, scale, window, sink, groups);                                                             \
   }
   if (f32) FT_PR_LAUNCH(float) else FT_PR_LAUNCH(__nv_bfloat16)
 #undef FT_PR_LAUNCH

@@ -1,8 +1,9 @@
 // Causal attention of prompt portions over the paged KV cache on tcgen05 / TMEM (bf16).
 //
 // A portion is a run of consecutive tokens of one sequence whose keys and values are already in the
-// cache (ft_qkv_finish / ft_kv_append); query token at position p sees keys 0 .. p, which lie in pages
-// named by the block table.  A step holds any number of portions of any lengths, so the work comes as a
+// cache (ft_qkv_finish / ft_qkv_head_finish / ft_kv_append); query token at position p sees keys 0 .. p, or
+// the last `window` of them, which lie in pages named by the block table.  With a window an item starts at the
+// key block of its first token's first visible key.  A step holds any number of portions of any lengths, so the work comes as a
 // list of items: up to 2 * tpt consecutive tokens of one sequence, with all query heads of a KV group
 // packed into the rows of the tile (row r = token r / group, head r % group; tpt = 128 / group tokens per
 // 128-row tile).  Packing the group means that K and V are read once per group instead of once per head
@@ -16,8 +17,8 @@
 //   warp 1      MMA issuer, alternating between the tiles: O_i += P_i V, then S_i = Q_i K_next^T
 //   warp 2      TMEM allocator
 //   warps 4-11  softmax groups of the two tiles (thread = query row), P written back over S in TMEM
-// The epilogue divides by the row sum, multiplies by the head's output gate when there is one, and
-// stores bf16.  Head sizes are multiples of 16 up to 128 and may differ between keys and values: the
+// The epilogue adds the head's sink to the row sum, divides by it, multiplies by the output gate (per head
+// or per element) and stores bf16.  Head sizes are multiples of 16 up to 128 and may differ between keys and values: the
 // tensor maps end at the head's size, so the columns up to the tile's 64 or 128 are filled with zeros.
 // All waits are bounded and report through the device status word.
 #include "attn_row.cuh"
@@ -45,9 +46,11 @@ struct PpCfg {
 struct PpParams {
   const int* items;         // [n_items, 4]: sequence slot, first query row, tokens, position of the first token
   const int* block_table;
-  const __nv_bfloat16* gate;
+  HeadGate gate;            // bf16
+  const float* sink;
   __nv_bfloat16* out;
-  long long ldg, ldo;
+  long long ldo;
+  int window;
   int Hkv, group, tpt, D, Dv;
   int block_size, rows_per_box, boxes, max_blocks, num_blocks;
   float scale_log2;
@@ -77,10 +80,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int n_tok = p.items[4 * blockIdx.x + 2], pos0 = p.items[4 * blockIdx.x + 3];
   // tokens and key blocks of each tile
   int nt[2], nb[2];
+  const int j0 = first_visible(pos0 + 1, p.window) / ATT_BN;   // block 0 of this item is key block j0
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     nt[i] = min(max(n_tok - i * p.tpt, 0), p.tpt);
-    nb[i] = nt[i] > 0 ? (pos0 + i * p.tpt + nt[i] + ATT_BN - 1) / ATT_BN : 0;
+    nb[i] = nt[i] > 0 ? (pos0 + i * p.tpt + nt[i] + ATT_BN - 1) / ATT_BN - j0 : 0;
   }
   const int n_blocks = max(nb[0], nb[1]);
 
@@ -128,7 +132,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const int* bt = p.block_table + static_cast<long long>(slot) * p.max_blocks;
       // box `lane` of key block j: rows_per_box keys of one page, as a row of the [num_blocks * block_size] axis
       auto page_row = [&](int j) {
-        const int key = j * ATT_BN + lane * p.rows_per_box;
+        const int key = (j0 + j) * ATT_BN + lane * p.rows_per_box;
         const int page = min(key / p.block_size, p.max_blocks - 1);
         const int blk = min(max(lane < p.boxes ? __ldg(bt + page) : 0, 0), p.num_blocks - 1);
         return blk * p.block_size + key % p.block_size;
@@ -254,13 +258,16 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const int tile_pos = pos0 + ti * p.tpt;
     const int limit = tile_pos + tok;                              // last visible key
     const int warp_limit = tile_pos + (ew * 32) / p.group;         // of this warp's first row
+    const int first = first_visible(limit + 1, p.window);          // first visible key
+    const int warp_first = first_visible(tile_pos + (ew * 32 + 31) / p.group + 1, p.window);   // of its last row
     for (int j = 0; j < my_nb && ok; ++j) {
       if (!mbar_wait(bar(S_FULL + ti), j & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) { ok = false; break; }
       tc_fence_after();
       f32x2 sp[ATT_BN / 2];
       att2_load_row(s_addr, sp);
-      const int kv0 = j * ATT_BN;
-      if (kv0 + ATT_BN - 1 > warp_limit) att2_mask_row(sp, kv0, limit);   // warp-uniform branch
+      const int kv0 = (j0 + j) * ATT_BN;
+      if (kv0 + ATT_BN - 1 > warp_limit) att2_mask_row(sp, kv0, limit);   // warp-uniform branches
+      if (kv0 < warp_first) att2_mask_ahead(sp, kv0, first);              // a row may see nothing of its first blocks
       const float mx = att2_row_max(sp) * p.scale_log2;  // scale > 0, so the maximum commutes with it
       float alpha = 1.f;
       if (mx > m_ref + ATT2_RESCALE_THRESHOLD) {
@@ -305,8 +312,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const bool row_ok = tok < nt[ti];
       const long long row = static_cast<long long>(row0) + ti * p.tpt + tok;
       const int hq = kvh * p.group + head;
-      float inv_l = l > 0.f ? 1.f / l : 0.f;
-      if (p.gate && row_ok) inv_l /= 1.f + expf(-__bfloat162float(p.gate[row * p.ldg + hq]));
+      float m = m_ref, num = 1.f;
+      sink_join(p.sink, min(hq, p.Hkv * p.group - 1), m, l, num);
+      float inv_l = l > 0.f ? num / l : 0.f;
+      if (p.gate.g && row_ok && p.gate.elem == 0) inv_l *= head_gate_bf16(p.gate, static_cast<int>(row), hq, 0);
+      const bool elem_gate = p.gate.g && p.gate.elem != 0;
       __nv_bfloat16* orow = p.out + row * p.ldo + static_cast<long long>(hq) * p.Dv;
 #pragma unroll
       for (int c = 0; c < VD / 32; ++c) {
@@ -316,12 +326,23 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (row_ok) {
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
-            if (c * 32 + g * 8 >= p.Dv) continue;
+            const int d = c * 32 + g * 8;
+            if (d >= p.Dv) continue;
+            float f[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]) * inv_l;
+            if (elem_gate) {
+              const uint4 z = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.gate.g) +
+                                                              p.gate.at(static_cast<int>(row), hq, d));
+              const float2 z0 = unpack_bf16x2(z.x), z1 = unpack_bf16x2(z.y), z2 = unpack_bf16x2(z.z), z3 = unpack_bf16x2(z.w);
+              f[0] *= gate_value(z0.x); f[1] *= gate_value(z0.y); f[2] *= gate_value(z1.x); f[3] *= gate_value(z1.y);
+              f[4] *= gate_value(z2.x); f[5] *= gate_value(z2.y); f[6] *= gate_value(z3.x); f[7] *= gate_value(z3.y);
+            }
             uint4 o;
-            o.x = pack_bf16x2(__uint_as_float(t[g * 8 + 0]) * inv_l, __uint_as_float(t[g * 8 + 1]) * inv_l);
-            o.y = pack_bf16x2(__uint_as_float(t[g * 8 + 2]) * inv_l, __uint_as_float(t[g * 8 + 3]) * inv_l);
-            o.z = pack_bf16x2(__uint_as_float(t[g * 8 + 4]) * inv_l, __uint_as_float(t[g * 8 + 5]) * inv_l);
-            o.w = pack_bf16x2(__uint_as_float(t[g * 8 + 6]) * inv_l, __uint_as_float(t[g * 8 + 7]) * inv_l);
+            o.x = pack_bf16x2(f[0], f[1]);
+            o.y = pack_bf16x2(f[2], f[3]);
+            o.z = pack_bf16x2(f[4], f[5]);
+            o.w = pack_bf16x2(f[6], f[7]);
             *reinterpret_cast<uint4*>(orow + c * 32 + g * 8) = o;
           }
         }
@@ -360,14 +381,15 @@ static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, co
 FT_API int ft_paged_prefill_tile(int group) { return group > 0 && group <= ft::ATT_BM ? ft::ATT_BM / group : 0; }
 
 // Attention of prompt portions (see the top of this file).  q: [rows, Hq, D] (row stride ldq), out: [rows,
-// Hq, Dv] (row stride ldo), gate: bf16 [rows, Hq] (row stride ldg) or null.  items: int32 [n_items, 4] on the
+// Hq, Dv] (row stride ldo); window, sink and gate as in ft_paged_decode (a gate per element has unit element stride
+// and 16-byte aligned heads).  items: int32 [n_items, 4] on the
 // device: slot, first query row, number of tokens (<= 2 * ft_paged_prefill_tile), position of the first token;
 // keys 0 .. position of a token must be in the cache.  Page sizes: a divisor of 128 of at least 8, or a
 // multiple of 128.  scale > 0.
 FT_API int ft_paged_prefill(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* items,
-                            const void* gate, void* out, int n_items, int rows, int Hq, int Hkv, int D, int Dv,
-                            long long ldq, long long ldg, long long ldo, int block_size, int max_blocks, int num_blocks,
-                            float scale, int device, cudaStream_t stream) {
+                            const void* gate, const float* sink, void* out, int n_items, int rows, int Hq, int Hkv, int D,
+                            int Dv, long long ldq, long long ldg, int gate_head, int gate_elem, long long ldo, int block_size,
+                            int max_blocks, int num_blocks, float scale, int window, int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   using namespace ft;
   FT_REQUIRE(q && k_cache && v_cache && block_table && items && out, "ft_paged_prefill: null pointer");
@@ -380,10 +402,14 @@ FT_API int ft_paged_prefill(const void* q, const void* k_cache, const void* v_ca
              "ft_paged_prefill: strides must be multiples of 8 elements and the scale positive");
   FT_REQUIRE(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) |
                reinterpret_cast<uintptr_t>(out)) & 15) == 0, "ft_paged_prefill: pointers must be 16-byte aligned");
+  FT_REQUIRE(window >= 0 && (!gate || gate_elem == 0 || (gate_elem == 1 && gate_head % 8 == 0 && ldg % 8 == 0 &&
+                                                         (reinterpret_cast<uintptr_t>(gate) & 15) == 0)),
+             "ft_paged_prefill: the window is negative or the gate's elements are not packed and aligned");
   if (n_items <= 0) return FT_E_OK;
   PpParams p;
-  p.items = items; p.block_table = block_table; p.gate = static_cast<const __nv_bfloat16*>(gate);
-  p.out = static_cast<__nv_bfloat16*>(out); p.ldg = ldg; p.ldo = ldo;
+  p.items = items; p.block_table = block_table; p.gate = HeadGate{gate, ldg, gate_head, gate_elem};
+  p.sink = sink; p.window = window;
+  p.out = static_cast<__nv_bfloat16*>(out); p.ldo = ldo;
   p.Hkv = Hkv; p.group = Hq / Hkv; p.tpt = ATT_BM / p.group; p.D = D; p.Dv = Dv;
   p.block_size = block_size;
   p.rows_per_box = block_size < ATT_BN ? block_size : ATT_BN;

@@ -1,0 +1,202 @@
+// Recurrent decoder blocks: short causal convolutions with carried inputs, and linear recurrences over prompt portions.
+//
+//   ft_causal_conv   per channel, over the rows of a ragged batch; the inputs ahead of a portion come from the
+//                    sequence's slot, the rows that are a sequence's only token store their own inputs there
+//   ft_rglru_scan    S_t = a_t S_(t-1) + x_t over the rows of every portion, out = S * gelu(y); the final state and
+//                    the convolution's last inputs go to the slot
+//
+// A slot needs no clearing: what a sequence has seen follows from its positions, and position 0 starts from zero.
+#include <initializer_list>
+
+#include "recurrent.cuh"
+
+namespace ft {
+
+constexpr int CV_THREADS = 128;
+constexpr int CV_ROWS = 8;       // consecutive rows a thread walks (their inputs overlap)
+
+struct ConvParams {
+  const void* x;            // [rows, ldx]
+  const float* w;           // [taps, C]: w[taps - 1] weighs the row itself
+  const float* bias;        // [C]
+  void* state;              // [slots, taps - 1, C]: the last inputs of a sequence, the most recent one last
+  void* u;                  // [rows, ldu]
+  const int* pos;
+  const int* slots;
+  const int* starts;        // position of the first row of the row's portion
+  long long ldx, ldu;
+  int rows, n_single, C, taps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(CV_THREADS)
+causal_conv_kernel(const ConvParams p) {
+  const int c = (blockIdx.x * CV_THREADS + threadIdx.x) * 8;
+  if (c >= p.C) return;
+  const int keep = p.taps - 1;
+  float bias[8];
+  load8(p.bias + c, bias);
+  const T* x = static_cast<const T*>(p.x) + c;
+  for (int r0 = blockIdx.y * CV_ROWS; r0 < p.rows; r0 += gridDim.y * CV_ROWS)
+    for (int row = r0; row < min(r0 + CV_ROWS, p.rows); ++row) {
+      const int pos = p.pos[row], back = pos - p.starts[row];       // rows of this portion ahead of this one
+      T* st = static_cast<T*>(p.state) + static_cast<long long>(p.slots[row]) * keep * p.C + c;
+      float acc[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = bias[e];
+      for (int d = keep; d >= 0; --d) {                             // d rows back
+        if (pos - d < 0) continue;
+        float v[8], w[8];
+        if (d <= back) load8(x + static_cast<long long>(row - d) * p.ldx, v);
+        else load8(static_cast<const T*>(st) + static_cast<long long>(keep - (d - back)) * p.C, v);
+        load8(p.w + static_cast<long long>(keep - d) * p.C + c, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] += w[e] * v[e];
+      }
+      store8(static_cast<T*>(p.u) + static_cast<long long>(row) * p.ldu + c, acc);
+      if (row < p.n_single) {                                       // this thread is the only one at these inputs
+        float v[8];
+        for (int m = 0; m + 1 < keep; ++m) {
+          load8(static_cast<const T*>(st) + static_cast<long long>(m + 1) * p.C, v);
+          store8(st + static_cast<long long>(m) * p.C, v);
+        }
+        if (keep > 0) {
+          load8(x + static_cast<long long>(row) * p.ldx, v);
+          store8(st + static_cast<long long>(keep - 1) * p.C, v);
+        }
+      }
+    }
+}
+
+// ---------------------------------------------------------------- scan
+// One block per (32 channels, portion): lane = channel, a warp takes SC_STEP consecutive rows of a tile of
+// SC_WARPS * SC_STEP.  Every warp folds its rows into (product of decays, state from zero), the folds of a tile are
+// combined through shared memory, then every warp walks its rows again from its true state.  Each input is read once.
+constexpr int SC_WARPS = 8;
+constexpr int SC_STEP = 16;
+
+struct ScanParams {
+  const float* a;           // [rows, C]
+  const float* x;
+  const void* y;            // [rows, ldy]: the other branch
+  void* out;                // [rows, ldo]
+  float* state;             // [slots, C]
+  const int* spans;         // [n, 4]: slot, first row, first position, rows
+  const void* conv_x;       // [rows, ldc] inputs of the convolution, and its state (null: no convolution)
+  void* conv_state;
+  long long ldy, ldo, ldc;
+  int C, keep;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(SC_WARPS * 32)
+rglru_scan_kernel(const ScanParams p) {
+  __shared__ float fold_a[2][SC_WARPS][32], fold_s[2][SC_WARPS][32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = blockIdx.x * 32 + lane;
+  const bool c_ok = c < p.C;
+  const int cc = c_ok ? c : p.C - 1;
+  const int* span = p.spans + 4 * blockIdx.y;
+  const int slot = span[0], row0 = span[1], pos0 = span[2], n = span[3];
+  float* st = p.state + static_cast<long long>(slot) * p.C + cc;
+  float carry = pos0 == 0 ? 0.f : *st;
+  int buf = 0;
+  for (int base = 0; base < n; base += SC_WARPS * SC_STEP, buf ^= 1) {
+    const int t0 = base + warp * SC_STEP;
+    float a[SC_STEP], x[SC_STEP], y[SC_STEP];
+#pragma unroll
+    for (int i = 0; i < SC_STEP; ++i) {
+      const bool ok = t0 + i < n;
+      const long long row = row0 + (ok ? t0 + i : 0);
+      a[i] = ok ? __ldg(p.a + row * p.C + cc) : 1.f;
+      x[i] = ok ? __ldg(p.x + row * p.C + cc) : 0.f;
+      y[i] = ok ? static_cast<float>(static_cast<const T*>(p.y)[row * p.ldy + cc]) : 0.f;
+    }
+    float fa = 1.f, fs = 0.f;
+#pragma unroll
+    for (int i = 0; i < SC_STEP; ++i) {
+      fs = a[i] * fs + x[i];
+      fa *= a[i];
+    }
+    fold_a[buf][warp][lane] = fa;
+    fold_s[buf][warp][lane] = fs;
+    __syncthreads();          // one barrier per tile: the next tile folds into the other buffer
+    float s = carry;
+#pragma unroll
+    for (int w = 0; w < SC_WARPS; ++w) {
+      const float next = fold_a[buf][w][lane] * carry + fold_s[buf][w][lane];
+      if (w < warp) s = next;
+      carry = next;
+    }
+#pragma unroll
+    for (int i = 0; i < SC_STEP; ++i) {
+      s = a[i] * s + x[i];
+      if (t0 + i < n && c_ok)
+        static_cast<T*>(p.out)[(row0 + t0 + i) * p.ldo + c] = static_cast<T>(s * gelu_row(y[i], static_cast<const T*>(nullptr)));
+    }
+  }
+  if (warp == 0 && c_ok) *st = carry;
+  if (warp == SC_WARPS - 1 && c_ok && p.conv_state) {
+    // the last inputs of the sequence: from this portion, or what the slot held (moved down; m + n > m is still old)
+    T* cs = static_cast<T*>(p.conv_state) + static_cast<long long>(slot) * p.keep * p.C + c;
+    for (int m = 0; m < p.keep; ++m) {
+      const int o = n - p.keep + m;
+      cs[static_cast<long long>(m) * p.C] = o >= 0 ? static_cast<const T*>(p.conv_x)[(row0 + o) * p.ldc + c]
+                                                   : cs[static_cast<long long>(m + n) * p.C];
+    }
+  }
+}
+
+static bool rc_aligned(std::initializer_list<const void*> ps) {
+  uintptr_t v = 0;
+  for (const void* p : ps) v |= reinterpret_cast<uintptr_t>(p);
+  return (v & 15) == 0;
+}
+
+}  // namespace ft
+
+using namespace ft;
+
+// u = causal convolution of x over the rows of a ragged batch (see ConvParams).  x, state and u are bf16, or fp32
+// with f32; w [taps, C] and bias [C] fp32; C a multiple of 8.
+FT_API int ft_causal_conv(const void* x, long long ldx, const float* w, const float* bias, void* state, void* u, long long ldu,
+                          const int* pos, const int* slots, const int* starts, int rows, int n_single, int C, int taps, int f32,
+                          int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(x && w && bias && u && pos && slots && starts && (state || taps == 1), "ft_causal_conv: null pointer");
+  FT_REQUIRE(C > 0 && C % 8 == 0 && taps >= 1 && ((ldx | ldu) & 7) == 0 && ldx >= C && ldu >= C, "ft_causal_conv: %d channels, %d taps", C, taps);
+  FT_REQUIRE(rc_aligned({x, w, bias, state, u}) && n_single >= 0 && n_single <= rows, "ft_causal_conv: pointers must be 16-byte aligned");
+  if (rows <= 0) return FT_E_OK;
+  ConvParams p;
+  p.x = x; p.w = w; p.bias = bias; p.state = state; p.u = u; p.pos = pos; p.slots = slots; p.starts = starts;
+  p.ldx = ldx; p.ldu = ldu; p.rows = rows; p.n_single = n_single; p.C = C; p.taps = taps;
+  const int need = (rows + CV_ROWS - 1) / CV_ROWS;
+  const dim3 grid((C / 8 + CV_THREADS - 1) / CV_THREADS, need < 65535 ? need : 65535);
+  if (f32) causal_conv_kernel<float><<<grid, CV_THREADS, 0, stream>>>(p);
+  else causal_conv_kernel<__nv_bfloat16><<<grid, CV_THREADS, 0, stream>>>(p);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// The recurrence over n_spans portions (spans int32 [n_spans, 4]: slot, first row, first position, rows): a, x fp32
+// [rows, C], y / out [rows, ldy / ldo], state fp32 [slots, C].  conv_x [rows, ldc] and conv_state [slots, keep, C]: the
+// inputs of the block's convolution, whose last `keep` are stored (null: none).  bf16, or fp32 with f32.
+FT_API int ft_rglru_scan(const float* a, const float* x, const void* y, long long ldy, void* out, long long ldo, float* state,
+                         const int* spans, int n_spans, const void* conv_x, long long ldc, void* conv_state, int keep, int C,
+                         int f32, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(a && x && y && out && state && spans, "ft_rglru_scan: null pointer");
+  FT_REQUIRE(C > 0 && ldy >= C && ldo >= C && (!conv_state || (conv_x && keep >= 0 && ldc >= C)), "ft_rglru_scan: bad shape");
+  if (n_spans <= 0) return FT_E_OK;
+  FT_REQUIRE(n_spans < 65536, "ft_rglru_scan: %d portions", n_spans);
+  ScanParams p;
+  p.a = a; p.x = x; p.y = y; p.out = out; p.state = state; p.spans = spans;
+  p.conv_x = conv_x; p.conv_state = keep > 0 ? conv_state : nullptr; p.ldy = ldy; p.ldo = ldo; p.ldc = ldc; p.C = C; p.keep = keep;
+  const dim3 grid((C + 31) / 32, n_spans);
+  if (f32) rglru_scan_kernel<float><<<grid, SC_WARPS * 32, 0, stream>>>(p);
+  else rglru_scan_kernel<__nv_bfloat16><<<grid, SC_WARPS * 32, 0, stream>>>(p);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}

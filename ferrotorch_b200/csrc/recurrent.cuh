@@ -1,0 +1,83 @@
+// Real-gated linear recurrence with diagonal state (RG-LRU), the arithmetic shared by its kernels.
+//
+//   r = sigmoid(zr), i = sigmoid(zi)                 gates, from a block-diagonal product of u
+//   log a = -c r softplus(lam)                       decay
+//   S_t = a S_(t-1) + sqrt(1 - a^2) i u              state, fp32
+//   out = S_t gelu(y)                                with the other branch of the block
+#pragma once
+#include "row_vec.cuh"
+
+namespace ft {
+
+struct RglruGateParams {
+  const void* u;            // [rows, ldu]: the convolved branch
+  const float* r_bias;      // [channels]
+  const float* i_bias;
+  const float* decay;       // [channels]: -c softplus(lam)
+  float* a;                 // fp32 [rows, channels]: decay of the row
+  float* x;                 // fp32 [rows, channels]: input term of the row
+  long long ldu;
+  int channels;
+  // rows 0 .. n_single - 1 are the only new token of their sequence: their recurrence is one step, taken at once
+  int n_single;
+  const int* pos;
+  const int* slots;
+  float* state;             // fp32 [slots, channels]
+  const void* y;            // [rows, ldy]: the other branch ahead of its activation
+  void* out;                // [rows, ldo]
+  long long ldy, ldo;
+};
+
+__device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_f32(float g) {
+  const float k = 0.7978845608028654f * (g + 0.044715f * g * g * g);
+  return 0.5f * g * (1.f + tanhf(k));
+}
+// gelu ahead of a bf16 store: 0.5 (1 + tanh k) = 1 / (1 + exp(-2 k))
+__device__ __forceinline__ float gelu_row(float g, const __nv_bfloat16*) {
+  return g * __fdividef(1.f, 1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
+}
+__device__ __forceinline__ float gelu_row(float g, const float*) { return gelu_tanh_f32(g); }
+
+// a = exp(log_a) and sqrt(1 - a^2).  Close to a = 1 the difference is summed as the series of 1 - exp(z), z = 2 log a.
+__device__ __forceinline__ void decay_and_gain(float log_a, float& a, float& gain) {
+  a = expf(log_a);
+  const float z = 2.f * log_a;
+  const float near = -z * (1.f + z * (0.5f + z * (1.f / 6 + z * (1.f / 24 + z * (1.f / 120 + z * (1.f / 720))))));
+  gain = sqrtf(z > -0.25f ? near : 1.f - a * a);
+}
+
+// Eight channels c .. c + 7 of one row: gate pre-activations zr, zi without bias.
+template <typename T>
+__device__ __forceinline__ void rglru_gates8(const RglruGateParams& p, long long row, int c, const float* zr, const float* zi) {
+  float u[8], br[8], bi[8], dec[8], a[8], x[8];
+  load8(static_cast<const T*>(p.u) + row * p.ldu + c, u);
+  load8(p.r_bias + c, br);
+  load8(p.i_bias + c, bi);
+  load8(p.decay + c, dec);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    float gain;
+    decay_and_gain(dec[e] * sigmoid_f32(zr[e] + br[e]), a[e], gain);
+    x[e] = gain * sigmoid_f32(zi[e] + bi[e]) * u[e];
+  }
+  if (row >= p.n_single) {
+    store8(p.a + row * p.channels + c, a);
+    store8(p.x + row * p.channels + c, x);
+    return;
+  }
+  float* st = p.state + static_cast<long long>(p.slots[row]) * p.channels + c;
+  float s[8], y[8];
+  load8(static_cast<const T*>(p.y) + row * p.ldy + c, y);
+  load8(static_cast<const float*>(st), s);
+  const bool fresh = p.pos[row] == 0;       // a sequence starts from zero, whatever the slot held before
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    s[e] = fresh ? x[e] : a[e] * s[e] + x[e];
+    y[e] = s[e] * gelu_row(y[e], static_cast<const T*>(nullptr));
+  }
+  store8(st, s);
+  store8(static_cast<T*>(p.out) + row * p.ldo + c, y);
+}
+
+}  // namespace ft

@@ -1,4 +1,4 @@
-"""Model families: Llama (single-GPU, tensor-parallel training, inference engine), Bopudra, ResNet, and the
+"""Model families: Llama (single-GPU, tensor-parallel training, inference engine), Bopudra, Zolorax, ResNet, and the
 small zoo (BERT, Whisper encoder, GCN, PPO policy) and the latent-diffusion stack (``diffusion``)."""
 from .llama import LlamaConfig, LlamaForCausalLM, LlamaModel  # noqa: F401
 from .llama_compat import (AwqQ4, GptqQ4, HqqQ4Axis1, LlamaActivation, LlamaAttention, LlamaGpuLayer, LlamaMLP,  # noqa: F401
@@ -28,6 +28,10 @@ def __getattr__(name):
         from . import bopudra
 
         return getattr(bopudra, name)
+    if name in ("ZoloraxConfig", "ZoloraxForCausalLM"):
+        from . import zolorax
+
+        return getattr(zolorax, name)
     if name in ("load_causal_lm", "register_causal_lm", "list_causal_lms"):
         from . import registry
 

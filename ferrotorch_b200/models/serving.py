@@ -24,7 +24,9 @@ sequences and gives every step one flat token batch:
 * with ``prefix_caching`` whole pages of finished (or still running) prompts stay in a table keyed by a hash chain
   of their tokens; a new request whose prompt starts with the same tokens adopts those pages (reference-counted
   in the pool) and computes only the rest.  Unused entries are evicted, deepest page of the least recently used
-  chain first, before any sequence is preempted.
+  chain first, before any sequence is preempted;
+* a model with recurrent states (``cache.rewindable`` false) is scheduled the same way, except that its states can neither
+  come with the pages of a prefix nor be wound back: prefix caching and ``lookahead`` do nothing for it.
 
 The batcher schedules; :class:`PagedStepper` owns the cache and runs the steps.  It serves every model that offers
 ``make_paged_cache`` and ``paged_forward`` (:mod:`~ferrotorch_b200.models.registry` lists them) and replays a step of
@@ -293,7 +295,7 @@ class ContinuousBatcher:
         if max_tokens_per_step < 1 or prefill_chunk < 1:
             raise ValueError("ContinuousBatcher: max_tokens_per_step and prefill_chunk must be at least 1")
         self.watermark_pages = max(1, int(watermark * num_blocks)) if watermark > 0 else 0
-        self.prefix = PrefixCache(self.cache.pool, block_size) if prefix_caching else None
+        self.prefix = PrefixCache(self.cache.pool, block_size) if prefix_caching and self.cache.rewindable else None
         self._drafts: dict = {}
         self.waiting: collections.deque = collections.deque()
         self.running: list = []                           # in admission order
@@ -410,7 +412,7 @@ class ContinuousBatcher:
                 continue
             n = min(len(r.prompt) + len(r.output) - r.computed, self.prefill_chunk, budget)
             draft = []
-            if (r.lookahead > 0 and r.output and r.computed == len(r.prompt) + len(r.output) - 1 and r.sampling.temperature == 0.0
+            if (r.lookahead > 0 and self.cache.rewindable and r.output and r.computed == len(r.prompt) + len(r.output) - 1 and r.sampling.temperature == 0.0
                     and r.sampling.repetition_penalty == 1.0 and r.logits_processor is None):
                 k = min(r.lookahead, r.max_new_tokens - len(r.output) - 1, budget - 1, self.prefill_chunk - 1)
                 draft = self._look_up(r.tokens(), r.ngram, k) if k > 0 else []

@@ -16,6 +16,7 @@ import torch
 from torch import nn
 
 from ..ops import functional as F
+from ..ops import reference as ref
 
 
 def round_up(n: int, m: int) -> int:
@@ -37,10 +38,37 @@ def pad_heads(t: torch.Tensor, heads: int, padded: int) -> torch.Tensor:
     return pad_to(t.reshape(heads, d, *t.shape[1:]), heads, padded, *t.shape[1:]).flatten(0, 1)
 
 
+@dataclass(frozen=True)
+class YarnScaling:
+    """Interpolation of slow rotary dimensions for contexts ``factor`` times as long as ``original``: dimensions that turn
+    more than ``fast`` times over it keep their frequency, less than ``slow`` times have it divided, a linear ramp between."""
+    factor: float
+    original: float
+    fast: float = 32.0
+    slow: float = 1.0
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotation of the first ``dims`` elements of a head, pairs ``(i, i + dims / 2)``, frequencies ``base ** (-2 i / dims)``."""
+    dims: int
+    base: float
+    scaling: YarnScaling | None = None
+
+    def table(self, positions: int, device="cpu") -> torch.Tensor:
+        """cos and sin of every position, ``[positions, dims / 2, 2]`` fp32 (angles are computed in 64-bit)."""
+        sc = self.scaling
+        kind = None if sc is None else {"type": "yarn", "factor": sc.factor, "original_max": sc.original, "beta_fast": sc.fast,
+                                        "beta_slow": sc.slow, "full_range": True, "mscale": "always"}
+        return torch.stack(ref.rope_tables(self.dims, positions, self.base, kind), -1).contiguous().to(device)
+
+
 @dataclass
 class AttentionSpec:
     """One attention sublayer: ``heads`` query heads over ``kv_heads`` key/value heads of sizes ``dim`` / ``vdim``,
-    ``score = (q . k) * scale``; ``temp_coef`` / ``temp_every``: query temperature (coef 0: none)."""
+    ``score = (q . k) * scale``; ``temp_coef`` / ``temp_every``: query temperature (coef 0: none); ``window``: a query sees
+    its last so many positions, its own included (``None``: all); ``rotary``: rotation of queries and keys; ``kv_from``:
+    the layer whose keys and values this one reads instead of having its own."""
     heads: int
     kv_heads: int
     dim: int
@@ -48,12 +76,19 @@ class AttentionSpec:
     scale: float
     temp_coef: float = 0.0
     temp_every: float = 1.0
+    window: int | None = None
+    rotary: RotarySpec | None = None
+    kv_from: int | None = None
 
     def validate(self) -> None:
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
             raise ValueError("AttentionSpec: %d heads of %d / %d over %d key/value heads" % (self.heads, self.dim, self.vdim, self.kv_heads))
         if not self.temp_every > 0:
             raise ValueError("AttentionSpec: temp_every must be positive")
+        if self.window is not None and self.window < 1:
+            raise ValueError("AttentionSpec: window must be positive or absent")
+        if self.rotary is not None and (self.rotary.dims % 2 or not 0 < self.rotary.dims <= self.dim or self.rotary.base <= 1):
+            raise ValueError("AttentionSpec: rotation of %d elements of %d" % (self.rotary.dims, self.dim))
 
     @property
     def padded_dim(self) -> int:

@@ -22,11 +22,22 @@ _i, _ll, _f, _vp = _native._i, _native._ll, _native._f, _native._vp
 _native.register_protos({
     "ft_kv_append": (_i, [_vp] * 7 + [_i] * 6 + [_ll, _ll, _i, _i, _i, _i, _vp]),
     "ft_paged_decode_scratch": (_ll, [_i, _i, _i, _i]),
-    "ft_paged_decode": (_i, [_vp] * 9 + [_i] * 5 + [_ll] * 3 + [_i, _i, _i, _f, _i, _i, _vp]),
-    "ft_paged_rows": (_i, [_vp] * 8 + [_i] * 5 + [_ll] * 3 + [_i, _i, _i, _f, _i, _i, _vp]),
+    "ft_paged_decode": (_i, [_vp] * 10 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _i, _vp]),
+    "ft_paged_rows": (_i, [_vp] * 9 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _i, _vp]),
     "ft_paged_prefill_tile": (_i, [_i]),
-    "ft_paged_prefill": (_i, [_vp] * 7 + [_i] * 6 + [_ll] * 3 + [_i, _i, _i, _f, _i, _vp]),
+    "ft_paged_prefill": (_i, [_vp] * 8 + [_i] * 6 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp]),
 })
+
+
+def _gate_args(gate: torch.Tensor | None) -> tuple:
+    """Row, head and element stride of an output gate ``[T, Hq]`` (one number per head) or ``[T, Hq, Dv]``."""
+    if gate is None:
+        return 0, 0, 0
+    return (gate.stride(0), gate.stride(1), gate.stride(2)) if gate.dim() == 3 else (gate.stride(0), gate.stride(1), 0)
+
+
+def _ptr(t: torch.Tensor | None):
+    return t.data_ptr() if t is not None else None
 
 
 class OutOfPages(RuntimeError):
@@ -92,15 +103,16 @@ class RaggedBatch:
     token ids, the position of the first of them, and the places among them whose logits are asked for.
 
     Entries of one token come first (:attr:`n_single` rows, the decode kernel's batch), longer ones after them
-    (:attr:`spans`, the prefill kernel's portions); ``last`` lists the wanted rows in the order of the entries as
-    they were given.  Everything the kernels read is copied to the device in one transfer."""
+    (:attr:`spans`, the prefill kernel's portions); ``starts`` holds the first position of every row's entry; ``last``
+    lists the wanted rows in the order of the entries as they were given.  Everything the kernels read is copied to the
+    device in one transfer."""
 
     def __init__(self, entries: list, device):
         self.device = torch.device(device)
         order = [i for i, e in enumerate(entries) if len(e[1]) == 1]
         self.n_single = len(order)
         order += [i for i, e in enumerate(entries) if len(e[1]) > 1]
-        toks, pos, slots, self.spans, first_row, row = [], [], [], [], {}, 0
+        toks, pos, slots, starts, self.spans, first_row, row = [], [], [], [], [], {}, 0
         for i in order:
             slot, tokens, start, _ = entries[i]
             n = len(tokens)
@@ -108,25 +120,29 @@ class RaggedBatch:
             toks += tokens
             pos += range(start, start + n)
             slots += [slot] * n
+            starts += [start] * n
             if n > 1:
                 self.spans.append((slot, row, start, n))
             row += n
         want = [first_row[i] + w for i, e in enumerate(entries) if len(e[1]) for w in e[3]]
         self.n_rows, self.n_want = row, len(want)
-        self._fill(toks, pos, slots, [p + 1 for p in pos], want)
+        self._fill(toks, pos, slots, [p + 1 for p in pos], starts, want)
         self._items: dict = {}
 
-    def _fill(self, toks, pos, slots, visible, want) -> None:
-        """One buffer: token ids and wanted rows as int64, then positions, slots and visible-key counts as int32."""
-        n, m = len(toks), len(want)
-        host = torch.empty(n + m + (3 * n + 1) // 2, dtype=torch.long, pin_memory=self.device.type == "cuda")
+    def _fill(self, toks, pos, slots, visible, starts, want) -> None:
+        """One buffer: token ids and wanted rows as int64, then positions, slots, visible-key counts, entry starts and
+        the portions (slot, first row, first position, tokens) as int32."""
+        n, m, k = len(toks), len(want), len(self.spans)
+        ints = pos + slots + visible + starts + [v for span in self.spans for v in span]
+        host = torch.empty(n + m + (len(ints) + 1) // 2, dtype=torch.long, pin_memory=self.device.type == "cuda")
         host[:n + m] = torch.tensor(toks + want, dtype=torch.long)
-        host[n + m:].view(torch.int32)[:3 * n] = torch.tensor(pos + slots + visible, dtype=torch.int32)
+        host[n + m:].view(torch.int32)[:len(ints)] = torch.tensor(ints, dtype=torch.int32)
         self._buf = host.to(self.device, non_blocking=True)
         self._host = host                                  # the pinned source lives as long as the batch
         ints = self._buf[n + m:].view(torch.int32)
         self.tokens, self.last = self._buf[:n], self._buf[n:n + m]
-        self.positions, self.slots, self.visible = ints[:n], ints[n:2 * n], ints[2 * n:3 * n]
+        self.positions, self.slots, self.visible, self.starts = ints[:n], ints[n:2 * n], ints[2 * n:3 * n], ints[3 * n:4 * n]
+        self.span_table = ints[4 * n:4 * n + 4 * k].view(k, 4)
 
     def work_items(self, tile_tokens: int):
         """The portions cut into work items of the prefill kernel (``[n, 4]`` int32 on the device: slot, first row,
@@ -151,23 +167,26 @@ class DecodeBatch(RaggedBatch):
         self.device = torch.device(device)
         self.n_single = self.n_rows = self.n_want = rows
         self.spans, self._items, self.pad_slot = [], {}, pad_slot
-        self._fill([0] * rows, [0] * rows, [pad_slot] * rows, [0] * rows, list(range(rows)))
+        self._fill([0] * rows, [0] * rows, [pad_slot] * rows, [0] * rows, [0] * rows, list(range(rows)))
         self._static = self._buf
 
     def load(self, tokens: list, positions: list, slots: list) -> None:
         pad = self.n_rows - len(tokens)
-        views = (self.tokens, self.last, self.positions, self.slots, self.visible)
+        views = (self.tokens, self.last, self.positions, self.slots, self.visible, self.starts, self.span_table)
         self._fill(tokens + [0] * pad, positions + [0] * pad, slots + [self.pad_slot] * pad,
-                   [p + 1 for p in positions] + [0] * pad, list(range(self.n_rows)))
+                   [p + 1 for p in positions] + [0] * pad, positions + [0] * pad, list(range(self.n_rows)))
         self._static.copy_(self._buf)
         self._buf = self._static
-        self.tokens, self.last, self.positions, self.slots, self.visible = views
+        self.tokens, self.last, self.positions, self.slots, self.visible, self.starts, self.span_table = views
 
 
 class PagedKVCache:
     """Block tables for up to ``max_seqs`` sequences over one :class:`PagePool`, plus the device
     K/V pages of every layer.  ``block_size`` tokens per page (16 in the benchmark configs).
-    ``n_kv_heads``, ``head_dim`` and ``v_head_dim`` (default: ``head_dim``) are numbers, or one number per layer."""
+    ``n_kv_heads``, ``head_dim`` and ``v_head_dim`` (default: ``head_dim``) are numbers, or one number per layer.
+
+    ``states``: what layers keep per sequence slot besides keys and values (recurrent states, by layer).  A state holds
+    the whole sequence so far, so such a cache cannot take tokens back (:attr:`rewindable`) nor start from shared pages."""
 
     def __init__(self, n_layers: int, n_kv_heads, head_dim, num_blocks: int, max_seqs: int,
                  max_seq_len: int, block_size: int = 16, device="cuda", dtype=torch.bfloat16, v_head_dim=None):
@@ -192,6 +211,20 @@ class PagedKVCache:
         self._pages: list[list[int]] = [[] for _ in range(max_seqs)]
         self.lengths = [0] * max_seqs
         self._dirty = False
+        self.states: dict = {}
+        self._rotary: dict = {}
+
+    def rotary_table(self, spec) -> torch.Tensor:
+        """The table of a :class:`~ferrotorch_b200.nn.packed_block.RotarySpec` for every position the cache can hold."""
+        got = self._rotary.get(spec)
+        if got is None:
+            got = self._rotary[spec] = spec.table(self.max_blocks * self.block_size, self.device)
+        return got
+
+    @property
+    def rewindable(self) -> bool:
+        """Whether a sequence can drop its latest tokens or adopt a prefix: yes while pages are all it has."""
+        return not self.states
 
     # ------------------------------------------------------------------ bookkeeping (host)
     def reserve(self, seq: int, new_len: int) -> None:
@@ -210,6 +243,8 @@ class PagedKVCache:
     def adopt(self, seq: int, pages: list, length: int) -> None:
         """Start sequence ``seq`` on pages that already hold its first ``length`` tokens (whole pages that
         another sequence filled; every one gains a holder).  The sequence must be empty."""
+        if not self.rewindable:
+            raise ValueError("adopt: recurrent states do not come with the pages of a prefix")
         if self._pages[seq]:
             raise ValueError("adopt: sequence %d already has pages" % seq)
         if length != len(pages) * self.block_size or len(pages) > self.max_blocks:
@@ -273,30 +308,31 @@ class PagedKVCache:
         return (q.dtype == torch.bfloat16 and D % 16 == 0 and Dv % 16 == 0 and D <= 128 and Dv <= 128
                 and q.shape[1] // Hkv <= max_group and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0)
 
-    def _rows(self, layer: int, q, visible, slots, scale, gate, out) -> None:
+    def _rows(self, layer: int, q, visible, slots, scale, gate, out, window, sink) -> None:
         """Attention of arbitrary rows, any head sizes, bf16 or fp32 (the simple kernel)."""
         T, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
         rc = _native.kernels().ft_paged_rows(
             q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), self.block_table.data_ptr(), slots.data_ptr(),
-            visible.data_ptr(), gate.data_ptr() if gate is not None else None, out.data_ptr(), T, Hq, Hkv, D, Dv, q.stride(0),
-            gate.stride(0) if gate is not None else 0, out.stride(0), self.block_size, self.max_blocks, self.num_blocks, float(scale),
+            visible.data_ptr(), _ptr(gate), _ptr(sink), out.data_ptr(), T, Hq, Hkv, D, Dv, q.stride(0),
+            *_gate_args(gate), out.stride(0), self.block_size, self.max_blocks, self.num_blocks, float(scale), int(window or 0),
             int(q.dtype == torch.float32), F._dev(q), F._stream())
         _native.check(rc, "ft_paged_rows")
 
     def decode(self, layer: int, q: torch.Tensor, ctx_len: torch.Tensor, scale: float | None = None,
                n_splits: int = 0, seq_ids: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-               out: torch.Tensor | None = None) -> torch.Tensor:
+               out: torch.Tensor | None = None, window: int | None = None, sink: torch.Tensor | None = None) -> torch.Tensor:
         """One query token per sequence: ``q [B, Hq, D]``, ``ctx_len [B]`` int32 -> ``[B, Hq, Dv]``.  Row b
         reads sequence b, or sequence ``seq_ids[b]`` (int32; a batch of any subset of the live sequences).
-        ``gate [B, Hq]``: output heads are multiplied by its sigmoid.  ``out``: where the result goes (the heads of a
+        ``gate [B, Hq]`` or ``[B, Hq, Dv]``: output heads or elements are multiplied by its sigmoid.  ``window``: only the
+        last so many keys are visible.  ``sink [Hq]`` (fp32): its exponential joins a head's denominator.  ``out``: where the result goes (the heads of a
         row packed, any row stride)."""
         B, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
         scale = scale if scale is not None else D ** -0.5
         table = self.sync_table()
         if not q.is_cuda:
-            o = self._decode_reference(layer, q, ctx_len, scale, seq_ids)
+            o = self._decode_reference(layer, q, ctx_len, scale, seq_ids, window, sink)
             o = o if gate is None else ref.head_gate(o, gate)
             return o if out is None else out.copy_(o)
         if out is None:
@@ -305,28 +341,31 @@ class PagedKVCache:
         if not self._tensor_core_ok(layer, q, 16) and (q.dtype != torch.bfloat16 or D != Dv or D not in (64, 128)
                                                        or Hq // Hkv not in (1, 2, 4, 8)):
             rows = seq_ids if seq_ids is not None else torch.arange(B, device=q.device, dtype=torch.int32)
-            self._rows(layer, q, ctx_len, rows, scale, gate, out)
+            self._rows(layer, q, ctx_len, rows, scale, gate, out, window, sink)
             return out
         lib = _native.kernels()
         if n_splits <= 0:
             ctas = B * Hkv
             n_splits = 1 if ctas >= 256 else max(1, min(8, 296 // max(ctas, 1)))
+            if window:
+                n_splits = min(n_splits, (window + 126) // 128 + 1)          # tiles of 128 keys that a window can touch
         n_scr = int(lib.ft_paged_decode_scratch(B, Hq, Dv, n_splits))
         scratch = F._get_scratch("paged_decode", n_scr, q.device) if n_scr else None
         rc = lib.ft_paged_decode(q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), table.data_ptr(),
                                  seq_ids.data_ptr() if seq_ids is not None else None, ctx_len.data_ptr(),
-                                 gate.data_ptr() if gate is not None else None, out.data_ptr(),
+                                 _ptr(gate), _ptr(sink), out.data_ptr(),
                                  scratch.data_ptr() if scratch is not None else None, B, Hq, Hkv, D, Dv, q.stride(0),
-                                 gate.stride(0) if gate is not None else 0, out.stride(0), self.block_size,
-                                 self.max_blocks, self.num_blocks, float(scale), n_splits, F._dev(q), F._stream())
+                                 *_gate_args(gate), out.stride(0), self.block_size, self.max_blocks, self.num_blocks,
+                                 float(scale), int(window or 0), n_splits, F._dev(q), F._stream())
         _native.check(rc, "ft_paged_decode")
         return out
 
     def attend(self, layer: int, q: torch.Tensor, batch: RaggedBatch, scale: float | None = None,
-               gate: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+               gate: torch.Tensor | None = None, out: torch.Tensor | None = None, window: int | None = None,
+               sink: torch.Tensor | None = None) -> torch.Tensor:
         """Causal attention of a whole :class:`RaggedBatch` (its keys and values already appended): ``q [T, Hq, D]`` ->
         ``[T, Hq, Dv]``.  Single tokens run on the decode kernel, longer portions on the prefill kernel; head sizes or
-        types that those do not cover run on the simple kernel."""
+        types that those do not cover run on the simple kernel.  ``gate``, ``window`` and ``sink`` as in :meth:`decode`."""
         T, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
         scale = scale if scale is not None else D ** -0.5
@@ -336,25 +375,26 @@ class PagedKVCache:
         n1 = batch.n_single
         if n1:
             self.decode(layer, q[:n1], batch.visible[:n1], scale, seq_ids=batch.slots[:n1],
-                        gate=gate[:n1] if gate is not None else None, out=out[:n1])
+                        gate=gate[:n1] if gate is not None else None, out=out[:n1], window=window, sink=sink)
         if not batch.spans:
             return out
         if not q.is_cuda:
             for slot, row, start, n in batch.spans:
                 k, v = self.gather(layer, slot, start + n)
-                o = ref.attention(q[None, row:row + n], k[None], v[None], True, scale, start)[0][0]
+                o = ref.attention(q[None, row:row + n], k[None], v[None], True, scale, start, window, sink)[0][0]
                 out[row:row + n] = o if gate is None else ref.head_gate(o, gate[row:row + n])
             return out
         bs = self.block_size
         if not (self._tensor_core_ok(layer, q, 128) and scale > 0 and bs >= 8 and (128 % bs == 0 or bs % 128 == 0)):
-            self._rows(layer, q[n1:], batch.visible[n1:], batch.slots[n1:], scale, gate[n1:] if gate is not None else None, out[n1:])
+            self._rows(layer, q[n1:], batch.visible[n1:], batch.slots[n1:], scale, gate[n1:] if gate is not None else None, out[n1:],
+                       window, sink)
             return out
         lib = _native.kernels()
         items = batch.work_items(int(lib.ft_paged_prefill_tile(Hq // Hkv)))
         rc = lib.ft_paged_prefill(q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), table.data_ptr(), items.data_ptr(),
-                                  gate.data_ptr() if gate is not None else None, out.data_ptr(), items.shape[0], T, Hq, Hkv, D, Dv,
-                                  q.stride(0), gate.stride(0) if gate is not None else 0, out.stride(0), bs, self.max_blocks,
-                                  self.num_blocks, float(scale), F._dev(q), F._stream())
+                                  _ptr(gate), _ptr(sink), out.data_ptr(), items.shape[0], T, Hq, Hkv, D, Dv, q.stride(0),
+                                  *_gate_args(gate), out.stride(0), bs, self.max_blocks, self.num_blocks, float(scale),
+                                  int(window or 0), F._dev(q), F._stream())
         _native.check(rc, "ft_paged_prefill")
         return out
 
@@ -391,7 +431,7 @@ class PagedKVCache:
             if self._pages[s]:
                 self.free_sequence(s)
 
-    def _decode_reference(self, layer, q, ctx_len, scale, seq_ids=None):
+    def _decode_reference(self, layer, q, ctx_len, scale, seq_ids=None, window=None, sink=None):
         """Host form of the paged-decode kernel, all rows at once: the pages of every row are gathered through
         the block table into a padded ``[B, L, Hkv, D]`` view and positions past a row's length are masked."""
         B, Hq, D = q.shape
@@ -404,9 +444,14 @@ class PagedKVCache:
         v = self.v[layer][pages].reshape(B, n_blk * self.block_size, Hkv, Dv).float()
         qf = q.float().reshape(B, Hkv, Hq // Hkv, D)
         s = torch.einsum("bhgd,blhd->bhgl", qf, k) * scale
-        dead = torch.arange(n_blk * self.block_size)[None] >= ctx[:, None]
+        at = torch.arange(n_blk * self.block_size)[None]
+        dead = at >= ctx[:, None]
+        if window:
+            dead = dead | (at < ctx[:, None] - window)
         s = s.masked_fill(dead[:, None, None, :], float("-inf"))
-        o = torch.einsum("bhgl,blhd->bhgd", torch.softmax(s, -1), v)
+        if sink is not None:                              # one more column of the softmax, without a value
+            s = torch.cat([s, sink.float().view(1, Hkv, Hq // Hkv, 1).expand(B, -1, -1, 1)], -1)
+        o = torch.einsum("bhgl,blhd->bhgd", torch.softmax(s, -1)[..., :v.shape[1]], v)
         return o.reshape(B, Hq, Dv).to(q.dtype)
 
 

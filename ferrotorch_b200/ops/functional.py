@@ -19,8 +19,8 @@ from .. import _native
 from . import reference as ref
 
 GEMM_OUT_F32, GEMM_ACCUMULATE, GEMM_BIAS, GEMM_BIAS_F32 = 1, 2, 4, 8
-GEMM_RELU, GEMM_GELU, GEMM_SILU = 16, 32, 64
-_ACT_FLAGS = {None: 0, "relu": GEMM_RELU, "gelu": GEMM_GELU, "silu": GEMM_SILU}
+GEMM_RELU, GEMM_GELU, GEMM_SILU, GEMM_RELU2 = 16, 32, 64, 128
+_ACT_FLAGS = {None: 0, "relu": GEMM_RELU, "gelu": GEMM_GELU, "silu": GEMM_SILU, "relu2": GEMM_RELU2}      # gelu: the erf form
 
 stats = {"gemm_native": 0, "gemm_library": 0, "gemm_small_m": 0}
 
@@ -59,8 +59,6 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, *, bias: torch.Tensor | None 
         flags |= GEMM_BIAS_F32 if bias.dtype == torch.float32 else GEMM_BIAS
         bias_ptr = bias.data_ptr()
     lib = _native.kernels()
-    if activation is not None:
-        ksplit = 1                      # the activation is applied by the single-pass epilogue only
     if residual is not None and ksplit == 1:
         raise ValueError("gemm_small_m: a residual needs the split path (ksplit != 1)")
     ws = None
@@ -147,7 +145,7 @@ def gemm_nt(a: torch.Tensor, b: torch.Tensor, *, bias: torch.Tensor | None = Non
         if accumulate:
             r = r + out.float()
         if activation:
-            r = getattr(torch.nn.functional, activation)(r)
+            r = ref.activation(r, activation)
         out.copy_(r.to(out.dtype))
         return out
     la, lb = _layout(a), _layout(b)
@@ -166,7 +164,7 @@ def gemm_nt(a: torch.Tensor, b: torch.Tensor, *, bias: torch.Tensor | None = Non
         if accumulate:
             r = r + out.float()
         if activation:
-            r = getattr(torch.nn.functional, activation)(r)
+            r = ref.activation(r, activation)
         out.copy_(r.to(out.dtype))
         return out
     if (M <= 128 and N >= 1024 and K >= 512 and not accumulate and out.dtype == torch.bfloat16 and la[0] == 0
@@ -417,9 +415,15 @@ def _mm_f32(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         torch.backends.cuda.matmul.allow_tf32 = old
 
 
-def linear_rows(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """``a [T, K] @ w.T`` for inference in the type of its operands (bf16 on the tcgen05 GEMM, fp32 as true fp32)."""
-    return gemm_nt(a, w) if a.dtype == torch.bfloat16 else _mm_f32(a, w)
+def linear_rows(a: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, activation: str | None = None) -> torch.Tensor:
+    """``act(a [T, K] @ w.T + bias)`` for inference in the type of its operands (bf16 on the tcgen05 GEMM, fp32 as true
+    fp32); ``bias`` fp32."""
+    if a.dtype == torch.bfloat16:
+        return gemm_nt(a, w, bias=bias, activation=activation)
+    y = _mm_f32(a, w)
+    if bias is not None:
+        y += bias
+    return y if activation is None else ref.activation(y, activation)
 
 
 def _small_m_shape(a: torch.Tensor, w: torch.Tensor) -> bool:

@@ -42,8 +42,9 @@ def query_temperature(positions: torch.Tensor, coef: float, every: float) -> tor
 
 
 def head_gate(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
-    """``o [T, H, D]`` times ``sigmoid(gate [T, H])``, one number per head."""
-    return (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
+    """``o [T, H, D]`` times ``sigmoid(gate)``: one number per head (``[T, H]``) or per element (``[T, H, D]``)."""
+    g = torch.sigmoid(gate.float())
+    return (o.float() * (g if gate.dim() == o.dim() else g[..., None])).to(o.dtype)
 
 
 def rope_tables(head_dim: int, max_pos: int, theta: float = 10000.0, scaling: dict | None = None,
@@ -70,7 +71,9 @@ def rope_tables(head_dim: int, max_pos: int, theta: float = 10000.0, scaling: di
         # The reference's schedule (transformer.rs:357-392): correction range found on the full
         # dimension and halved onto the inv_freq index space, no attention temperature.  The
         # Hugging Face variant differs in both points: ``"hf_range": True`` keeps the range
-        # un-halved, ``"mscale": True`` multiplies cos / sin by 0.1 ln(factor) + 1.
+        # un-halved, ``"mscale": True`` multiplies cos / sin by 0.1 ln(factor) + 1.  ``"full_range": True``
+        # also lets the range reach the last dimension rather than the last frequency, and
+        # ``"mscale": "always"`` applies the multiplier whatever the factor.
         f = float(scaling["factor"])
         orig = float(scaling.get("original_max", max_pos))
         bf, bs = float(scaling.get("beta_fast", 32.0)), float(scaling.get("beta_slow", 1.0))
@@ -80,7 +83,9 @@ def rope_tables(head_dim: int, max_pos: int, theta: float = 10000.0, scaling: di
 
         low = max(float(math.floor(corr_dim(bf))), 0.0)
         high = min(float(math.ceil(corr_dim(bs))), float(head_dim - 1))
-        if scaling.get("hf_range", False):
+        if scaling.get("full_range", False):
+            high = max(high, low + 0.001)
+        elif scaling.get("hf_range", False):
             high = min(high, float(half - 1))
         else:
             low, high = low / 2.0, high / 2.0
@@ -88,7 +93,7 @@ def rope_tables(head_dim: int, max_pos: int, theta: float = 10000.0, scaling: di
         ramp = ((idx - low) / denom).clamp(0, 1)
         mask = 1.0 - ramp  # 1 -> keep extrapolated (high freq), 0 -> interpolate
         inv_freq = inv_freq / f * (1 - mask) + inv_freq * mask
-        mscale = 0.1 * math.log(f) + 1.0 if (scaling.get("mscale", False) and f > 1) else 1.0
+        mscale = 0.1 * math.log(f) + 1.0 if scaling.get("mscale") == "always" or (scaling.get("mscale", False) and f > 1) else 1.0
     elif kind == "llama3":
         f = float(scaling.get("factor", 8.0))
         lo_f, hi_f = float(scaling.get("low_freq_factor", 1.0)), float(scaling.get("high_freq_factor", 4.0))
@@ -131,6 +136,48 @@ def rope(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, positions: torch
 _ACTS = {0: F.silu, 1: F.relu, 2: lambda g: F.gelu(g, approximate="tanh")}
 
 
+def activation(x: torch.Tensor, name: str) -> torch.Tensor:
+    """The activations that GEMM epilogues apply: relu, gelu (erf form), silu, relu2 (the square of relu)."""
+    return F.relu(x).square() if name == "relu2" else getattr(F, name)(x)
+
+
+def rms_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, count: int, offset: float = 0.0) -> torch.Tensor:
+    """``x / sqrt(mean(x^2) + eps) * (offset + w)`` in fp32 for rows padded with zeros beyond ``count`` elements."""
+    xf = x.float()
+    return xf / torch.sqrt(xf.pow(2).sum(-1, keepdim=True) / count + eps) * (offset + weight.float())
+
+
+def rotate_leading(x: torch.Tensor, table: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """Rotate the first ``2 * half`` elements of every head of ``x [T, H, D]`` (pairs ``i, i + half``) by the rows
+    ``table[position] [half, 2]`` of cos and sin; the rest pass."""
+    half = table.shape[1]
+    c, s = table[positions.long()].unsqueeze(1).unbind(-1)
+    u, v, rest = x[..., :half], x[..., half:2 * half], x[..., 2 * half:]
+    return torch.cat([u * c - v * s, v * c + u * s, rest], -1)
+
+
+def decay_and_gain(log_a: torch.Tensor):
+    """``a`` and ``sqrt(1 - a^2)`` of a gated linear recurrence."""
+    return torch.exp(log_a), torch.sqrt(-torch.expm1(2.0 * log_a))
+
+
+def linear_recurrence(a: torch.Tensor, x: torch.Tensor, state: torch.Tensor) -> torch.Tensor:
+    """``S_t = a_t S_(t-1) + x_t`` over the rows of ``a``, ``x [T, C]`` from ``state [C]``: all states ``[T, C]``, fp32."""
+    out, s = torch.empty_like(x), state
+    for t in range(x.shape[0]):
+        s = a[t] * s + x[t]
+        out[t] = s
+    return out
+
+
+def top_experts(logits: torch.Tensor, top: int):
+    """The ``top`` experts of every row with the largest logits (the lower index of equals) and the sigmoid of theirs:
+    ``(index [T, top], weight [T, top])``."""
+    z = logits.float()
+    index = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, :top]
+    return index, torch.sigmoid(z.gather(1, index))
+
+
 def swiglu(gu: torch.Tensor, act: int = 0) -> torch.Tensor:
     """``act(gate) * up`` for ``gu = [gate | up]`` on the last dim (ferrotorch-llama/src/gpu.rs:696-703;
     relu / gelu variants: ferrotorch-nn/src/transformer.rs:693-764)."""
@@ -155,12 +202,14 @@ def repeat_kv(x: torch.Tensor, n_rep: int) -> torch.Tensor:
 
 
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = True,
-              scale: float | None = None, q_offset: int | None = None):
+              scale: float | None = None, q_offset: int | None = None, window: int | None = None,
+              sink: torch.Tensor | None = None):
     """GQA attention on ``[B, S, H, D]`` tensors, returns ``(out [B,Sq,Hq,D], lse [B,Hq,Sq])``.
 
     Scores scaled by ``1/sqrt(D)``, causal mask hides ``j > i + q_offset`` where the default
     offset aligns the last query with the last key (for Sq == Sk this is the reference's
-    top-left mask, ferrotorch-nn/src/flash_attention.rs:647-746), max-subtracted softmax."""
+    top-left mask, ferrotorch-nn/src/flash_attention.rs:647-746), max-subtracted softmax.  With ``window`` a query
+    sees only its last so many keys; with ``sink [Hq]`` a head's denominator gains ``exp(sink)``."""
     B, Sq, Hq, D = q.shape
     Sk, Hkv = k.shape[1], k.shape[2]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -173,7 +222,11 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = 
         i = torch.arange(Sq, device=q.device)[:, None] + off
         j = torch.arange(Sk, device=q.device)[None, :]
         s = s.masked_fill(j > i, float("-inf"))
+        if window:
+            s = s.masked_fill(i - j >= window, float("-inf"))
     lse = torch.logsumexp(s, dim=-1)
+    if sink is not None:
+        lse = torch.logaddexp(lse, sink.float().view(1, Hq, 1))
     p = torch.exp(s - lse.unsqueeze(-1))
     o = torch.matmul(p, vf).permute(0, 2, 1, 3)
     return o.to(q.dtype), lse

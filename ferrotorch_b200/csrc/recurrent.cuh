@@ -39,12 +39,12 @@ __device__ __forceinline__ float gelu_row(float g, const __nv_bfloat16*) {
 }
 __device__ __forceinline__ float gelu_row(float g, const float*) { return gelu_tanh_f32(g); }
 
-// a = exp(log_a) and sqrt(1 - a^2).  Close to a = 1 the difference is summed as the series of 1 - exp(z), z = 2 log a.
+// a = exp(log_a) and sqrt(1 - a^2) from q = a - 1: decays are often within 1e-3 of one, where an error in the last place
+// of exp would change the length of the memory, and the difference 1 - a^2 would cancel.
 __device__ __forceinline__ void decay_and_gain(float log_a, float& a, float& gain) {
-  a = expf(log_a);
-  const float z = 2.f * log_a;
-  const float near = -z * (1.f + z * (0.5f + z * (1.f / 6 + z * (1.f / 24 + z * (1.f / 120 + z * (1.f / 720))))));
-  gain = sqrtf(z > -0.25f ? near : 1.f - a * a);
+  const float q = expm1f(log_a);
+  a = 1.f + q;
+  gain = sqrtf(-q * (2.f + q));
 }
 
 // Eight channels c .. c + 7 of one row: gate pre-activations zr, zi without bias.

@@ -1,14 +1,15 @@
 """Attention over the paged cache where one key stands out: queries that match exactly one key each."""
 import torch
 
-import bopudra_oracle as O
+import zolorax_oracle as O
 from ferrotorch_b200.nn.paged import PagedAttentionManager, PagedKVCache, RaggedBatch
 
 
-def check_planted_keys(Hq, Hkv, D, Dv, block, dtype, device, length, tolerance=None):
+def check_planted_keys(Hq, Hkv, D, Dv, block, dtype, device, length, tolerance=None, window=None, sink=False, elem_gate=False):
     """Keys are unit-scale noise; query i is a multiple of one key's direction, so that key's score stands out by tens.
     Targets walk over the first keys, page and tile borders, the query's own key, and the key just after it (which a
-    query in a portion must not see although it is in the cache)."""
+    query in a portion must not see although it is in the cache); with a window also over the keys just inside and just
+    outside it.  ``sink``: every other head has a sink about as large as the planted score, the others a small one."""
     g = torch.Generator().manual_seed(length + D)
     tol = tolerance or (1e-4 if dtype == torch.float32 else 3e-2)
     cache = PagedKVCache(1, Hkv, D, 2 * ((length + block - 1) // block) + 3, 3, length + block, block, device, dtype, v_head_dim=Dv)
@@ -30,20 +31,25 @@ def check_planted_keys(Hq, Hkv, D, Dv, block, dtype, device, length, tolerance=N
     q, target = torch.zeros(length, Hq, D), {}
     for i in range(length):
         for h in range(Hq):
-            t = (edges + [i, i + 1])[(i * 7 + h * 3) % (len(edges) + 2)]
-            t = min(t, length - 1)
+            near = [i, i + 1] + ([i - window, i - window + 1, i - window - 1, i - window + 2] if window else [])
+            t = (edges + near)[(i * 7 + h * 3) % (len(edges) + len(near))]
+            if window and (i + h) % 3 == 0:
+                t = near[(i // 3 + h) % len(near)]
+            t = min(max(t, 0), length - 1)
             kt = k[t, h // group].float()
             q[i, h] = kt * (50.0 / scale / kt.pow(2).sum())
             target[i, h] = t
     q = q.to(dtype)
-    gate = torch.randn(length, Hq, generator=g).to(dtype)
+    gate = torch.randn(length, Hq, *([Dv] if elem_gate else []), generator=g).to(dtype)
+    sinks = torch.tensor([50.5 if h % 2 else 3.0 for h in range(Hq)]) if sink else None
     want = torch.zeros(length, Hq, Dv, dtype=torch.float64)
     for i in range(length):
         for h in range(Hq):
             c = h // group
-            o = O.head_attention(q[i, h].double(), k[:i + 1, c].double(), v[:i + 1, c].double(), scale)
+            lo, hi = O.visible_keys(i, window)
+            o = O.sink_attention(q[i, h].double(), k[lo:hi, c].double(), v[lo:hi, c].double(), scale, sinks[h].double() if sink else None)
             want[i, h] = o * torch.sigmoid(gate[i, h].double())
-            if target[i, h] <= i and D >= 32:             # the case is what it claims: that key carries the softmax
+            if lo <= target[i, h] < hi and D >= 32 and not (sink and h % 2):             # the case is what it claims: that key carries the softmax
                 assert (o - v[target[i, h], c].double()).abs().max() < 0.2
     for cuts in ([length], [1], [2, 1, 3, block, 1, 128, 5, 1]):
         entries, at, n = [], 0, 0
@@ -58,8 +64,8 @@ def check_planted_keys(Hq, Hkv, D, Dv, block, dtype, device, length, tolerance=N
         buf[:, :Hq * D] = q[rows].flatten(1)
         buf = buf.to(device)
         out = torch.full((length, Hq * Dv + 16), 7.0, dtype=dtype, device=device)
-        cache.attend(0, buf[:, :Hq * D].unflatten(1, (Hq, D)), batch, scale, gate=gate[rows].to(device),
-                     out=out[:, :Hq * Dv].unflatten(1, (Hq, Dv)))
+        cache.attend(0, buf[:, :Hq * D].unflatten(1, (Hq, D)), batch, scale, gate=gate[rows].to(device), window=window,
+                     sink=sinks.to(device) if sink else None, out=out[:, :Hq * Dv].unflatten(1, (Hq, Dv)))
         err = (out[:, :Hq * Dv].double().cpu().view(length, Hq, Dv) - want[rows]).abs().amax((1, 2))
         assert float(err.max()) < tol, "cuts %s: error %.3g at position %d" % (cuts, float(err.max()), int(rows[err.argmax()]))
         assert bool((out[:, Hq * Dv:] == 7.0).all())

@@ -3,7 +3,7 @@
     python bench.py --workload decoder-serving                 # all families and sizes below
     python bench.py --workload decoder-serving --serving-sizes 8b --serving-kernels
 
-Random weights.  Both families run on ``models.serving.PagedStepper``: prefill feeds prompts of ``prompt`` tokens in steps
+Random weights.  All families run on ``models.serving.PagedStepper``: prefill feeds prompts of ``prompt`` tokens in steps
 of at most 8192 tokens, decode replays the captured single-token step of ``batch`` sequences at contexts around
 ``prompt``.  Times are CUDA events around whole steps after warm-up (weights and cache exceed L2 at these sizes);
 ``--serving-kernels`` times every kernel of one layer with a 512 MB write between launches and relates it to the
@@ -18,12 +18,25 @@ import statistics
 import torch
 
 # name: (hidden, layers, heads, kv heads, head size, SwiGLU width, vocabulary, prompt, batch).  The parallel family's
-# two-matrix MLP is 1.5 x as wide, so both have the same number of parameters and matrix-product FLOPs.
+# two-matrix MLP is 1.5 x as wide, so both have the same number of parameters and matrix-product FLOPs.  Zolorax has the
+# same dense MLP in every other layer and eight experts of half the SwiGLU width, two of them used, in the others: equal
+# FLOPs per token, but more weights to read in a decode step.
 SIZES = {"1b": (2048, 16, 32, 8, 64, 8192, 128256, 2048, 64),
          "3b": (3072, 28, 24, 8, 128, 8192, 128256, 2048, 64),
          "8b": (4096, 32, 32, 8, 128, 14336, 128256, 2048, 64)}
-FAMILIES = ("llama", "bopudra")
+FAMILIES = ("llama", "bopudra", "zolorax")
 PAGE = 16
+EXPERTS, TOP, WINDOW = 8, 2, 1024
+
+
+def zolorax_config(size: str, n: int):
+    from ferrotorch_b200.models.zolorax import ZoloraxConfig, ZoloraxLayerConfig
+    from ferrotorch_b200.nn.feed_forward import ExpertSpec
+
+    hidden, _, heads, kv, dim, ff, vocab, _, _ = SIZES[size]
+    cfg = ZoloraxConfig.pattern(vocab, hidden, n, heads, kv, dim, ff, experts=0, window=WINDOW)
+    cfg.layers = [ZoloraxLayerConfig(s.mixer, ExpertSpec(EXPERTS, TOP, ff // TOP) if i % 2 else ff * 3 // 2) for i, s in enumerate(cfg.layers)]
+    return cfg
 
 
 def build(family: str, size: str, layers: int | None = None):
@@ -33,6 +46,10 @@ def build(family: str, size: str, layers: int | None = None):
         from ferrotorch_b200.models.bopudra import BopudraConfig, BopudraForCausalLM
 
         return BopudraForCausalLM(BopudraConfig.uniform(vocab, hidden, n, heads, kv, dim, ff * 3 // 2), device="cuda").random_()
+    if family == "zolorax":
+        from ferrotorch_b200.models.zolorax import ZoloraxConfig, ZoloraxForCausalLM
+
+        return ZoloraxForCausalLM(zolorax_config(size, n), device="cuda").random_()
     from ferrotorch_b200.models.llama import LlamaConfig, LlamaForCausalLM
 
     cfg = LlamaConfig(vocab_size=vocab, hidden_size=hidden, intermediate_size=ff, num_hidden_layers=n, num_attention_heads=heads,
@@ -77,17 +94,18 @@ def throughput(model, size: str, steps: int, warmup: int) -> dict:
     pre_ms = _event_ms(lambda: model.paged_forward(chunk, st.cache), warmup, steps)
 
     def decode():
-        st.feed([(s, [7], [0]) for s in slots])
+        st.feed([(s, [p[0]], [0]) for s, p in zip(slots, prompts)])
 
     dec_host_ms = _event_ms(decode, warmup, steps)         # as served: bookkeeping, one upload, replay
     graph = next(iter(st._graphs.values()))[1]
     dec_ms = _event_ms(graph.replay, warmup, steps)
-    return {"prefill_tok_s": round(per * prompt / pre_ms * 1e3), "prefill_ms": round(pre_ms, 3), "prefill_tokens_per_step": per * prompt,
+    weights = sum(t.numel() for t in {t.data_ptr(): t for t in [*model.parameters(), *model.buffers()]}.values())
+    return {"parameters_billions": round(weights / 1e9, 2), "prefill_tok_s": round(per * prompt / pre_ms * 1e3), "prefill_ms": round(pre_ms, 3), "prefill_tokens_per_step": per * prompt,
             "decode_tok_s": round(batch / dec_ms * 1e3), "decode_ms": round(dec_ms, 3), "decode_step_as_served_ms": round(dec_host_ms, 3),
             "decode_batch": batch, "context": prompt}
 
 
-def kernel_table(size: str, peaks: dict, steps: int) -> list:
+def kernel_table(size: str, peaks: dict, steps: int, families=FAMILIES) -> list:
     """Device time and roofline fraction of the kernels of one layer of each family: ``(family, phase, kernel, us, bound, frac)``."""
     from ferrotorch_b200 import _native
     from ferrotorch_b200.nn.paged import RaggedBatch
@@ -120,15 +138,16 @@ def kernel_table(size: str, peaks: dict, steps: int) -> list:
                      "of_measured": round(max(t_f, t_b) / us, 3)})
 
     lib = _native.kernels()
-    for family in FAMILIES:
-        model = build(family, size, layers=2)
+    for family in families:
+        model = build(family, size, layers=6 if family == "zolorax" else 2)
         cache = model.make_paged_cache(batch * ((prompt + 16) // PAGE + 1), PAGE, batch, prompt + 16)
         for s in range(batch):
             cache.reserve(s, prompt + 1)
         cache.sync_table()
         per = max(1, 8192 // prompt)
-        pre = RaggedBatch([(s, [1] * prompt, 0, [prompt - 1]) for s in range(per)], "cuda")
-        dec = RaggedBatch([(s, [1], prompt - 1, [0]) for s in range(batch)], "cuda")
+        ids = torch.randint(0, vocab, (max(per, batch), prompt), generator=torch.Generator().manual_seed(0)).tolist()
+        pre = RaggedBatch([(s, ids[s], 0, [prompt - 1]) for s in range(per)], "cuda")
+        dec = RaggedBatch([(s, ids[s][:1], prompt - 1, [0]) for s in range(batch)], "cuda")
         for phase, b in (("prefill", pre), ("decode", dec)):
             T = b.n_rows
             kvb = batch * prompt * kv * 2 * dim * 2
@@ -138,7 +157,9 @@ def kernel_table(size: str, peaks: dict, steps: int) -> list:
             def gemm(name, a, w, fn):
                 add(family, phase, name, fn, 2 * T * w.shape[0] * w.shape[1], 2 * (w.numel() + a.numel()))
 
-            if family == "bopudra":
+            if family == "zolorax":
+                _zolorax_kernels(lambda *a: add(family, phase, *a), gemm, model, cache, b, phase == "prefill", (hidden, heads, kv, dim, prompt, per, batch))
+            elif family == "bopudra":
                 blk, nrm = model.blocks[0], model.norms[0]
                 x, h = F.embedding_dynamic_tanh(b.tokens, model.embed, nrm.alpha, nrm.weight, nrm.bias, out_dtype=torch.bfloat16)
                 packed = F.linear_rows(h, blk.in_proj)
@@ -203,6 +224,71 @@ def kernel_table(size: str, peaks: dict, steps: int) -> list:
     return rows
 
 
+def _zolorax_kernels(add, gemm, model, cache, b, prefill: bool, sizes: tuple) -> None:
+    """The kernels of a recurrent, an attention, a dense and a routed sublayer."""
+    from ferrotorch_b200.ops import decoder as D
+    from ferrotorch_b200.ops import functional as F
+
+    hidden, heads, kv, dim, prompt, per, batch = sizes
+    T, dt = b.n_rows, torch.bfloat16
+    rec, att, routed = model.layers[0], model.layers[2], model.layers[1]
+    C = rec.mixer.spec.padded_width
+    x, h = rec.norm1.gather(b.tokens, model.embed, dt)
+    add("embedding + norm", lambda: rec.norm1.gather(b.tokens, model.embed, dt), 0, T * hidden * 8)
+    add("rms norm", lambda: rec.norm1(x, out_dtype=dt), 0, T * hidden * 6)
+    # recurrent mixer
+    m, st = rec.mixer, cache.states[0]
+    packed = F.linear_rows(h, m.in_proj, m.in_bias)
+    y, cx = packed[:, :C], packed[:, C:]
+    gemm("recurrent in_proj (y|x) + bias", h, m.in_proj, lambda: F.linear_rows(h, m.in_proj, m.in_bias))
+    add("causal conv", lambda: D.causal_conv(cx, m.conv_weight, m.conv_bias, st.conv, b), 0, 4 * T * C)
+    u = D.causal_conv(cx, m.conv_weight, m.conv_bias, st.conv, b)
+    out = torch.empty((T, C), device="cuda", dtype=dt)
+    n, a, z = m.gates.shape[-1], torch.rand((T, C), device="cuda"), torch.randn((T, C), device="cuda")
+
+    def gates():                                          # the portions left out: product and gates alone
+        spans, b.spans = b.spans, []
+        D.gated_recurrence(u, y, m.gates, m.r_bias, m.i_bias, m.decay, st.state, b, cx, st.conv, out)
+        b.spans = spans
+
+    add("gates" + ("" if prefill else " + step"), gates, 4 * T * C * n, 10 * T * C if prefill else 14 * T * C + 2 * m.gates.numel())
+    if prefill:
+        add("scan * gelu", lambda: D.rglru_scan(a, z, y, out, st.state, b, cx, st.conv), 0, 12 * T * C)
+    gemm("recurrent out_proj + residual", out, m.out_proj, lambda: F.residual_linear_(x, out, m.out_proj))
+    # attention mixer
+    m, s = att.mixer, att.mixer.attn
+    (qo, qn), (ko, kn), (vo, vn), (go, gn) = m.segments
+    packed = F.linear_rows(h, m.in_proj)
+    gemm("attention in_proj (q|k|v|g)", h, m.in_proj, lambda: F.linear_rows(h, m.in_proj))
+    add("head norms, rotation, append", lambda: D.qkv_head_finish(
+        packed, cache, 0, b, heads=heads, dim=dim, q_off=qo, k_off=ko, v_off=vo, q_weight=m.q_norm, k_weight=m.k_norm, eps=m.eps,
+        table=cache.rotary_table(s.rotary)), 0, 4 * T * (qn + kn + vn))
+    q, gate = packed[:, qo:qo + qn].unflatten(1, (heads, dim)), packed[:, go:go + gn].unflatten(1, (heads, dim))
+    o = torch.empty((T, heads, dim), device="cuda", dtype=dt)
+    seen = sum(min(i + 1, s.window) for i in range(prompt))
+    add("attention (window %d, sink, gated)" % s.window, lambda: cache.attend(0, q, b, s.scale, gate=gate, out=o, window=s.window, sink=m.sink),
+        4 * heads * dim * per * seen if prefill else 0,
+        2 * T * (3 * heads + 2 * kv) * dim if prefill else batch * min(prompt, s.window) * kv * 2 * dim * 2)
+    gemm("attention out_proj + residual", o.flatten(1), m.out_proj, lambda: F.residual_linear_(x, o.flatten(1), m.out_proj))
+    # feed-forwards
+    m = rec.mlp
+    act = F.linear_rows(h, m.up, activation="relu2")
+    gemm("dense up + squared relu", h, m.up, lambda: F.linear_rows(h, m.up, activation="relu2"))
+    gemm("dense down + residual", act, m.down, lambda: F.residual_linear_(x, act, m.down))
+    m = routed.mlp
+    E, top, ff = m.spec.experts, m.spec.top, m.spec.ff
+    r = D.moe_route(h, m.router, E, top)
+    add("routing (logits, choice, sort, gather)", lambda: D.moe_route(h, m.router, E, top), 2 * T * hidden * E, 2 * T * hidden * (1 + top))
+    eact = D.grouped_linear(r.sorted, m.gate_up, r, glu="silu", seg_rows=T)
+    yt = D.grouped_linear(eact, m.down, r, seg_rows=T)
+    add("experts gate|up + silu", lambda: D.grouped_linear(r.sorted, m.gate_up, r, glu="silu", seg_rows=T), 4 * T * top * hidden * ff,
+        2 * (m.gate_up.numel() + T * top * (hidden + ff)))
+    add("experts down", lambda: D.grouped_linear(eact, m.down, r, seg_rows=T), 2 * T * top * hidden * ff, 2 * (m.down.numel() + T * top * (hidden + ff)))
+    add("rms norm + experts' terms", lambda: rec.norm1(x, pending=(yt, r.place), update=True, out_dtype=dt), 0, T * hidden * (10 + 2 * top))
+    if not prefill:
+        gemm("head", h, model.head, lambda: F.linear_f32_out(h, model.head))
+
+
 def run(args, sampler_cls) -> dict:
     root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
     try:
@@ -212,7 +298,7 @@ def run(args, sampler_cls) -> dict:
         peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
     from ferrotorch_b200 import _native
 
-    sizes = args.serving_sizes.split(",")
+    sizes, families = args.serving_sizes.split(","), tuple(args.serving_families.split(","))
     out = {"metric": "decoder_serving_tokens_per_s", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup),
            "dtype": "bf16", "data": "synthetic", "weights": "random", "higher_is_better": True, "sizes": {}, "kernels": {}}
     launches = _native.launch_count()
@@ -220,16 +306,16 @@ def run(args, sampler_cls) -> dict:
     sampler.start()
     for size in sizes:
         out["sizes"][size] = {}
-        for family in FAMILIES:
+        for family in families:
             model = build(family, size)
             out["sizes"][size][family] = throughput(model, size, args.steps, max(3, args.warmup))
             del model
             gc.collect()
             torch.cuda.empty_cache()
         if args.serving_kernels:
-            out["kernels"][size] = kernel_table(size, peaks, args.steps)
+            out["kernels"][size] = kernel_table(size, peaks, args.steps, families)
     out["clocks"] = sampler.stop()
     out["gpu_launches"] = _native.launch_count() - launches
     out["device_status"] = _native.device_status(0)
-    out["value"] = out["sizes"][sizes[-1]]["bopudra"]["decode_tok_s"]
+    out["value"] = out["sizes"][sizes[-1]][families[-1]]["decode_tok_s"]
     return out

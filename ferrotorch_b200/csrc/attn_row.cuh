@@ -119,9 +119,11 @@ struct HeadGate {
   }
 };
 __device__ __forceinline__ float gate_value(float z) { return 1.f / (1.f + expf(-z)); }
+// The same ahead of a bf16 store: approximate exponential and division (an epilogue applies it to every output element).
+__device__ __forceinline__ float gate_value_bf16(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 __device__ __forceinline__ float head_gate_bf16(const HeadGate& gt, int row, int head, int d) {
   if (!gt.g) return 1.f;
-  return gate_value(__bfloat162float(static_cast<const __nv_bfloat16*>(gt.g)[gt.at(row, head, d)]));
+  return gate_value_bf16(__bfloat162float(static_cast<const __nv_bfloat16*>(gt.g)[gt.at(row, head, d)]));
 }
 
 }  // namespace ft

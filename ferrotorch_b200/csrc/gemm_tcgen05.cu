@@ -105,6 +105,48 @@ __device__ __forceinline__ float apply_act(float v, int flags) {
 }
 
 
+// Bias and activation on 32 accumulator columns.  The kind of both is decided once, outside the unrolled loops: with
+// the choice inside, the epilogue's code no longer fits the instruction cache and outlasts the main loop.
+__device__ __forceinline__ void add_bias32(const GemmParams& p, uint32_t (&r)[32], int col0) {
+  if (p.flags & GEMM_BIAS_F32) {
+    const float* b = static_cast<const float*>(p.bias) + col0;
+    if ((reinterpret_cast<uintptr_t>(b) & 15) == 0) {
+#pragma unroll
+      for (int j = 0; j < 32; j += 4)
+        if (col0 + j + 4 <= p.N) {
+          const float4 v = __ldg(reinterpret_cast<const float4*>(b + j));
+          r[j] = __float_as_uint(__uint_as_float(r[j]) + v.x);
+          r[j + 1] = __float_as_uint(__uint_as_float(r[j + 1]) + v.y);
+          r[j + 2] = __float_as_uint(__uint_as_float(r[j + 2]) + v.z);
+          r[j + 3] = __float_as_uint(__uint_as_float(r[j + 3]) + v.w);
+        }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 32; ++j)
+        if (col0 + j < p.N) r[j] = __float_as_uint(__uint_as_float(r[j]) + __ldg(b + j));
+    }
+    return;
+  }
+  const __nv_bfloat16* b = static_cast<const __nv_bfloat16*>(p.bias) + col0;
+#pragma unroll
+  for (int j = 0; j < 32; ++j)
+    if (col0 + j < p.N) r[j] = __float_as_uint(__uint_as_float(r[j]) + __bfloat162float(b[j]));
+}
+
+__device__ __forceinline__ void act32(uint32_t (&r)[32], int flags) {
+  if (flags & (GEMM_RELU | GEMM_RELU2)) {
+    const bool square = flags & GEMM_RELU2;
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+      const float v = fmaxf(__uint_as_float(r[j]), 0.f);
+      r[j] = __float_as_uint(square ? v * v : v);
+    }
+    return;
+  }
+#pragma unroll
+  for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(apply_act(__uint_as_float(r[j]), flags));
+}
+
 // Epilogue that writes straight to global memory, one accumulator row per lane.  Used where the
 // output needs a read-modify-write in fp32 before rounding (bf16 accumulate) or an activation
 // after the accumulation.  `t_row` addresses this warp's 32 TMEM lanes at the tile's first
@@ -270,11 +312,13 @@ __device__ __forceinline__ void epilogue_transposed(const GemmParams& p, uint32_
     tmem_ld_wait();
     if (!n_ok) continue;
 #pragma unroll
+    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) + bias);
+    if (has_act) act32(r, p.flags);
+#pragma unroll
     for (int j = 0; j < 32; ++j) {
       const int m = m0 + c * 32 + j;
       if (m < p.N) {
-        float v = __uint_as_float(r[j]) + bias;
-        if (has_act) v = apply_act(v, p.flags);
+        const float v = __uint_as_float(r[j]);
         if (p.flags & GEMM_OUT_F32)
           static_cast<float*>(p.C)[static_cast<long long>(m) * p.ldc + n_idx] = v;
         else
@@ -760,25 +804,12 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
           const int col0 = n0 + c * step_cols;
           if (m0 >= p.M || col0 >= p.N) continue;  // warp-uniform: nothing of this piece is inside C
           if (has_bias) {
-#pragma unroll
-            for (int j = 0; j < 64; ++j) {
-              const int col = col0 + j;
-              if (j < step_cols && col < p.N) {
-                const float b = (p.flags & GEMM_BIAS_F32)
-                                    ? static_cast<const float*>(p.bias)[col]
-                                    : __bfloat162float(static_cast<const __nv_bfloat16*>(p.bias)[col]);
-                uint32_t& x = j < 32 ? r0[j & 31] : r1[j & 31];
-                x = __float_as_uint(__uint_as_float(x) + b);
-              }
-            }
+            add_bias32(p, r0, col0);
+            if (!out_f32) add_bias32(p, r1, col0 + 32);
           }
           if (has_act) {
-#pragma unroll
-            for (int j = 0; j < 64; ++j)
-              if (j < step_cols) {
-                uint32_t& x = j < 32 ? r0[j & 31] : r1[j & 31];
-                x = __float_as_uint(apply_act(__uint_as_float(x), p.flags));
-              }
+            act32(r0, p.flags);
+            if (!out_f32) act32(r1, p.flags);
           }
           // the store issued two steps ago has finished reading this staging tile
           if (lane == 0) tma_store_wait_read<1>();

@@ -8,7 +8,8 @@
 //   EPI_GLU    two parts: C = act(r sum_0) * (r sum_1), r a factor per row (a routed token's weight: scaling the
 //              two sums is scaling the input)
 //   EPI_RGLRU  two parts: the gates of a real-gated linear recurrence (see recurrent.cuh), recurrence and all for
-//              rows that are a sequence's only token, decay and input term for the others
+//              rows that are a sequence's only token, decay and input term for the others (32 channels at a time
+//              through a swizzled staging tile per warp and TMA stores, because a lane holds a row)
 //
 // Groups are either segments of rows (a mixture of experts: rows sorted by expert, segments listed on the device by
 // moe_build_kernel, so that no launch depends on the host knowing the counts) or blocks of columns (a block-diagonal
@@ -90,28 +91,32 @@ __device__ __forceinline__ float glu_act(float g, int act) {
     const float k = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return 0.5f * g * (1.f + tanhf(k));
   }
-  return g / (1.f + __expf(-g));
+  return __fdividef(g, 1.f + __expf(-g));
 }
 
-template <int BN>
+template <int BN, int EPI>
 struct GgCfg {
+  // EPI_RGLRU: two staging tiles (decay, input term) of 32 rows x 32 fp32 per epilogue warp
+  static constexpr int STAGING = EPI == EPI_RGLRU ? 8 * 2 * 4096 : 0;
   static constexpr int A_BYTES = GG_BM * GG_BK * 2;
   static constexpr int B_BYTES = BN * GG_BK * 2;
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
-  static constexpr int STAGES = (200 * 1024) / STAGE_BYTES > 6 ? 6 : (200 * 1024) / STAGE_BYTES;
+  static constexpr int STAGES = (216 * 1024 - STAGING) / STAGE_BYTES > 6 ? 6 : (216 * 1024 - STAGING) / STAGE_BYTES;
   static constexpr int TMEM_COLS = 2 * BN;
-  static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 + 256;
+  static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + STAGING + 1024 + 256;
 };
 
 template <int BN, int EPI>
 __global__ void __launch_bounds__(GG_THREADS, 1)
-grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const GroupedParams p) {
-  using Cfg = GgCfg<BN>;
+grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
+                    const __grid_constant__ CUtensorMap tmDecay, const __grid_constant__ CUtensorMap tmInput, const GroupedParams p) {
+  using Cfg = GgCfg<BN, EPI>;
   constexpr int STAGES = Cfg::STAGES;
   constexpr int NW = EPI == EPI_STORE ? BN : BN / 2;    // output columns of a tile
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + STAGES * Cfg::STAGE_BYTES);
+  uint8_t* staging = smem + STAGES * Cfg::STAGE_BYTES;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(staging + Cfg::STAGING);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2 * STAGES + 4);
   volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -216,33 +221,76 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       float scale = 1.f;
       if constexpr (EPI == EPI_GLU)
         if (p.row_scale && row_ok) scale = p.row_scale[row];
-      if (warp_ok) {
+      if constexpr (EPI == EPI_RGLRU) {
+        const uint32_t tile_s = smem_u32(staging) + static_cast<uint32_t>(warp - 4) * 8192u;
+        const uint32_t row_s = tile_s + static_cast<uint32_t>(lane) * 128u, sw = static_cast<uint32_t>(lane & 7);
+        const bool stored = warp_ok && row + (t.rows - 1 - r) >= p.gates.n_single;      // some row of the tile leaves its terms
+        for (int c = wg * 32; warp_ok && c < NW; c += 64) {
+          const int n = t.n0 + c;
+          if (n >= p.N) break;
+          if (lane == 0) tma_store_wait_read<0>();       // the previous stores have read the staging tiles
+          __syncwarp();
+          const int ch = t.group * p.a_col + n;
+#pragma unroll 1
+          for (int h = 0; h < 2; ++h) {
+            uint32_t za[16], zb[16];
+            tmem_ld_32x16(t_row + c + h * 16, za);
+            tmem_ld_32x16(t_row + NW + c + h * 16, zb);
+            tmem_ld_wait();
+#pragma unroll
+            for (int g = 0; g < 2; ++g) {
+              const int o = h * 16 + g * 8;
+              float a8[8], x8[8];
+              if (row_ok && n + o < p.N) {
+                float zr[8], zi[8];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) { zr[e] = __uint_as_float(za[g * 8 + e]); zi[e] = __uint_as_float(zb[g * 8 + e]); }
+                rglru_gates8<__nv_bfloat16>(p.gates, row, ch + o, zr, zi, a8, x8);
+                if (row < p.gates.n_single) rglru_step8<__nv_bfloat16>(p.gates, row, ch + o, a8, x8);
+              } else {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) a8[e] = x8[e] = 0.f;
+              }
+#pragma unroll
+              for (int v = 0; v < 2; ++v) {
+                const uint32_t dst = row_s + ((static_cast<uint32_t>(o / 4 + v) ^ sw) << 4);
+                asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst), "f"(a8[4 * v]), "f"(a8[4 * v + 1]), "f"(a8[4 * v + 2]),
+                             "f"(a8[4 * v + 3]) : "memory");
+                asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst + 4096u), "f"(x8[4 * v]), "f"(x8[4 * v + 1]),
+                             "f"(x8[4 * v + 2]), "f"(x8[4 * v + 3]) : "memory");
+              }
+            }
+          }
+          fence_proxy_async_smem();
+          __syncwarp();
+          if (lane == 0 && stored) {
+            // the maps are [blocks, rows, n]: channels past the block and rows past the last are not written (rows of
+            // single tokens are: nothing reads them)
+            tma_store_3d(&tmDecay, tile_s, n, t.row0 + ew * 32, t.group);
+            tma_store_3d(&tmInput, tile_s + 4096u, n, t.row0 + ew * 32, t.group);
+            tma_store_commit();
+          }
+        }
+      } else if (warp_ok) {
 #pragma unroll 1
         for (int c = wg * 16; c < NW; c += 32) {
           const int n = t.n0 + c;
           if (n >= p.N) break;
           uint32_t a[16], b[16];
           tmem_ld_32x16(t_row + c, a);
-          if constexpr (EPI != EPI_STORE) tmem_ld_32x16(t_row + NW + c, b);
+          if constexpr (EPI == EPI_GLU) tmem_ld_32x16(t_row + NW + c, b);
           tmem_ld_wait();
           if (!row_ok) continue;
 #pragma unroll
           for (int h = 0; h < 2; ++h) {
             if (n + h * 8 >= p.N) continue;            // N is a multiple of 8
             float f[8];
-            if constexpr (EPI == EPI_RGLRU) {
-              float g[8];
 #pragma unroll
-              for (int e = 0; e < 8; ++e) { f[e] = __uint_as_float(a[h * 8 + e]); g[e] = __uint_as_float(b[h * 8 + e]); }
-              rglru_gates8<__nv_bfloat16>(p.gates, row, t.group * p.a_col + n + h * 8, f, g);
-            } else {
-#pragma unroll
-              for (int e = 0; e < 8; ++e) {
-                f[e] = __uint_as_float(a[h * 8 + e]);
-                if constexpr (EPI == EPI_GLU) f[e] = glu_act(scale * f[e], p.act) * (scale * __uint_as_float(b[h * 8 + e]));
-              }
-              store8(static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + n + h * 8, f);
+            for (int e = 0; e < 8; ++e) {
+              f[e] = __uint_as_float(a[h * 8 + e]);
+              if constexpr (EPI == EPI_GLU) f[e] = glu_act(scale * f[e], p.act) * (scale * __uint_as_float(b[h * 8 + e]));
             }
+            store8(static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + n + h * 8, f);
           }
         }
       }
@@ -251,6 +299,10 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       if (lane == 0) mbar_arrive(tempty_bar(acc));
       acc ^= 1;
       if (acc == 0) acc_phase ^= 1u;
+    }
+    if constexpr (EPI == EPI_RGLRU) {
+      if (lane == 0) tma_store_wait<0>();      // shared memory must outlive the stores that read it
+      __syncwarp();
     }
   }
 
@@ -328,7 +380,16 @@ grouped_gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W
             zr[e] = e & 1 ? r1v : r0v;
             zi[e] = e & 1 ? i1v : i0v;
           }
-          if (j == 0 && (threadIdx.x & 3) == 0 && ok) rglru_gates8<float>(p.gates, row, t.group * p.a_col + n, zr, zi);
+          if (j == 0 && (threadIdx.x & 3) == 0 && ok) {
+            const int c = t.group * p.a_col + n;
+            float a8[8], x8[8];
+            rglru_gates8<float>(p.gates, row, c, zr, zi, a8, x8);
+            if (row < p.gates.n_single) rglru_step8<float>(p.gates, row, c, a8, x8);
+            else {
+              store8(p.gates.a + row * p.gates.channels + c, a8);
+              store8(p.gates.x + row * p.gates.channels + c, x8);
+            }
+          }
         } else if (ok) {
           float v = acc[0][i][j];
           if constexpr (EPI == EPI_GLU) {
@@ -478,9 +539,9 @@ __global__ void moe_permute_kernel(const uint4* __restrict__ h, long long ldh16,
 }
 
 template <int BN, int EPI>
-static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tb, const GroupedParams& p, long long tiles, int device,
-                          cudaStream_t stream) {
-  using Cfg = GgCfg<BN>;
+static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tb, const CUtensorMap& tdecay, const CUtensorMap& tinput,
+                          const GroupedParams& p, long long tiles, int device, cudaStream_t stream) {
+  using Cfg = GgCfg<BN, EPI>;
   auto kern = grouped_gemm_kernel<BN, EPI>;
   static bool attr_set[64] = {false};
   if (!attr_set[device]) {
@@ -488,7 +549,7 @@ static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tb, const Gr
     attr_set[device] = true;
   }
   const int sms = sm_count(device);
-  kern<<<tiles < sms ? static_cast<int>(tiles) : sms, GG_THREADS, Cfg::SMEM_BYTES, stream>>>(ta, tb, p);
+  kern<<<tiles < sms ? static_cast<int>(tiles) : sms, GG_THREADS, Cfg::SMEM_BYTES, stream>>>(ta, tb, tdecay, tinput, p);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;
@@ -523,9 +584,18 @@ static int run_grouped(const void* A, long long lda, int total_rows, const void*
   if (rc) return rc;
   rc = make_tmap_2d(&tb, W, 2, p.K, static_cast<uint64_t>(p.groups) * p.parts * p.N, static_cast<uint64_t>(p.K) * 2, GG_BK, bn / 2, 3);
   if (rc) return rc;
-  if (bn == 256) return launch_grouped<256, EPI>(ta, tb, p, tiles_at(256), device, stream);
-  if (bn == 128) return launch_grouped<128, EPI>(ta, tb, p, tiles_at(128), device, stream);
-  return launch_grouped<64, EPI>(ta, tb, p, tiles_at(64), device, stream);
+  CUtensorMap td = ta, ti = ta;             // only EPI_RGLRU stores through its maps
+  if (EPI == EPI_RGLRU) {
+    const RglruGateParams& g = p.gates;
+    const uint64_t block = static_cast<uint64_t>(p.N) * 4, row = static_cast<uint64_t>(g.channels) * 4;
+    rc = make_tmap_3d(&td, g.a, 4, p.N, p.rows, p.groups, row, block, 32, 32, 1, 3, false);
+    if (rc) return rc;
+    rc = make_tmap_3d(&ti, g.x, 4, p.N, p.rows, p.groups, row, block, 32, 32, 1, 3, false);
+    if (rc) return rc;
+  }
+  if (bn == 256) return launch_grouped<256, EPI>(ta, tb, td, ti, p, tiles_at(256), device, stream);
+  if (bn == 128) return launch_grouped<128, EPI>(ta, tb, td, ti, p, tiles_at(128), device, stream);
+  return launch_grouped<64, EPI>(ta, tb, td, ti, p, tiles_at(64), device, stream);
 }
 
 static bool gg_aligned(std::initializer_list<const void*> ps) {

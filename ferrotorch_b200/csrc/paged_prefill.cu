@@ -335,8 +335,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
               const uint4 z = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.gate.g) +
                                                               p.gate.at(static_cast<int>(row), hq, d));
               const float2 z0 = unpack_bf16x2(z.x), z1 = unpack_bf16x2(z.y), z2 = unpack_bf16x2(z.z), z3 = unpack_bf16x2(z.w);
-              f[0] *= gate_value(z0.x); f[1] *= gate_value(z0.y); f[2] *= gate_value(z1.x); f[3] *= gate_value(z1.y);
-              f[4] *= gate_value(z2.x); f[5] *= gate_value(z2.y); f[6] *= gate_value(z3.x); f[7] *= gate_value(z3.y);
+              f[0] *= gate_value_bf16(z0.x); f[1] *= gate_value_bf16(z0.y); f[2] *= gate_value_bf16(z1.x); f[3] *= gate_value_bf16(z1.y);
+              f[4] *= gate_value_bf16(z2.x); f[5] *= gate_value_bf16(z2.y); f[6] *= gate_value_bf16(z3.x); f[7] *= gate_value_bf16(z3.y);
             }
             uint4 o;
             o.x = pack_bf16x2(f[0], f[1]);

@@ -13,7 +13,7 @@
 namespace ft {
 
 constexpr int CV_THREADS = 128;
-constexpr int CV_ROWS = 8;       // consecutive rows a thread walks (their inputs overlap)
+constexpr int CV_ROWS = 16;      // most consecutive rows a thread walks (their inputs overlap)
 
 struct ConvParams {
   const void* x;            // [rows, ldx]
@@ -25,8 +25,62 @@ struct ConvParams {
   const int* slots;
   const int* starts;        // position of the first row of the row's portion
   long long ldx, ldu;
-  int rows, n_single, C, taps;
+  int rows, n_single, C, taps, walk;
 };
+
+// The input d rows ahead of a row (d <= taps - 1): of the same portion, of the slot, or zero ahead of the sequence.
+template <typename T>
+__device__ __forceinline__ void conv_input(const ConvParams& p, const T* x, const T* st, int row, int pos, int back, int d, float (&v)[8]) {
+  if (pos - d < 0) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = 0.f;
+  } else if (d <= back) {
+    load8(x + static_cast<long long>(row - d) * p.ldx, v);
+  } else {
+    load8(st + static_cast<long long>(p.taps - 1 - (d - back)) * p.C, v);
+  }
+}
+
+// Up to four taps: weights and the sliding inputs stay in registers while the thread walks down its rows.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(CV_THREADS)
+short_conv_kernel(const ConvParams p) {
+  const int c = (blockIdx.x * CV_THREADS + threadIdx.x) * 8;
+  if (c >= p.C) return;
+  float w[TAPS][8], bias[8], in[TAPS][8];      // in[d]: the input d rows ahead
+  load8(p.bias + c, bias);
+#pragma unroll
+  for (int d = 0; d < TAPS; ++d) load8(p.w + static_cast<long long>(TAPS - 1 - d) * p.C + c, w[d]);
+  const T* x = static_cast<const T*>(p.x) + c;
+  for (int r0 = blockIdx.y * p.walk; r0 < p.rows; r0 += gridDim.y * p.walk) {
+    const int r1 = min(r0 + p.walk, p.rows);
+    for (int row = r0; row < r1; ++row) {
+      const int pos = p.pos[row], back = pos - p.starts[row];
+      T* st = static_cast<T*>(p.state) + static_cast<long long>(p.slots[row]) * (TAPS - 1) * p.C + c;
+      if (row == r0 || back == 0) {            // a walk or a portion begins: fetch what lies ahead of this row
+#pragma unroll
+        for (int d = 1; d < TAPS; ++d) conv_input(p, x, static_cast<const T*>(st), row, pos, back, d, in[d]);
+      }
+      load8(x + static_cast<long long>(row) * p.ldx, in[0]);
+      float acc[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = bias[e];
+#pragma unroll
+      for (int d = TAPS - 1; d >= 0; --d)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] += w[d][e] * in[d][e];
+      store8(static_cast<T*>(p.u) + static_cast<long long>(row) * p.ldu + c, acc);
+      if (TAPS > 1 && row < p.n_single) {      // this thread is the only one at these inputs
+#pragma unroll
+        for (int d = 0; d < TAPS - 1; ++d) store8(st + static_cast<long long>(TAPS - 2 - d) * p.C, in[d]);
+      }
+#pragma unroll
+      for (int d = TAPS - 1; d > 0; --d)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) in[d][e] = in[d - 1][e];
+    }
+  }
+}
 
 template <typename T>
 __global__ void __launch_bounds__(CV_THREADS)
@@ -37,18 +91,16 @@ causal_conv_kernel(const ConvParams p) {
   float bias[8];
   load8(p.bias + c, bias);
   const T* x = static_cast<const T*>(p.x) + c;
-  for (int r0 = blockIdx.y * CV_ROWS; r0 < p.rows; r0 += gridDim.y * CV_ROWS)
-    for (int row = r0; row < min(r0 + CV_ROWS, p.rows); ++row) {
+  for (int r0 = blockIdx.y * p.walk; r0 < p.rows; r0 += gridDim.y * p.walk)
+    for (int row = r0; row < min(r0 + p.walk, p.rows); ++row) {
       const int pos = p.pos[row], back = pos - p.starts[row];       // rows of this portion ahead of this one
       T* st = static_cast<T*>(p.state) + static_cast<long long>(p.slots[row]) * keep * p.C + c;
       float acc[8];
 #pragma unroll
       for (int e = 0; e < 8; ++e) acc[e] = bias[e];
-      for (int d = keep; d >= 0; --d) {                             // d rows back
-        if (pos - d < 0) continue;
+      for (int d = keep; d >= 0; --d) {
         float v[8], w[8];
-        if (d <= back) load8(x + static_cast<long long>(row - d) * p.ldx, v);
-        else load8(static_cast<const T*>(st) + static_cast<long long>(keep - (d - back)) * p.C, v);
+        conv_input(p, x, static_cast<const T*>(st), row, pos, back, d, v);
         load8(p.w + static_cast<long long>(keep - d) * p.C + c, w);
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[e] += w[e] * v[e];
@@ -104,17 +156,18 @@ rglru_scan_kernel(const ScanParams p) {
   for (int base = 0; base < n; base += SC_WARPS * SC_STEP, buf ^= 1) {
     const int t0 = base + warp * SC_STEP;
     float a[SC_STEP], x[SC_STEP], y[SC_STEP];
+    // every load is issued (past the end: of the last row), so that all of a tile are in flight together
 #pragma unroll
     for (int i = 0; i < SC_STEP; ++i) {
-      const bool ok = t0 + i < n;
-      const long long row = row0 + (ok ? t0 + i : 0);
-      a[i] = ok ? __ldg(p.a + row * p.C + cc) : 1.f;
-      x[i] = ok ? __ldg(p.x + row * p.C + cc) : 0.f;
-      y[i] = ok ? static_cast<float>(static_cast<const T*>(p.y)[row * p.ldy + cc]) : 0.f;
+      const long long row = row0 + min(t0 + i, n - 1);
+      a[i] = __ldg(p.a + row * p.C + cc);
+      x[i] = __ldg(p.x + row * p.C + cc);
+      y[i] = static_cast<float>(static_cast<const T*>(p.y)[row * p.ldy + cc]);
     }
     float fa = 1.f, fs = 0.f;
 #pragma unroll
     for (int i = 0; i < SC_STEP; ++i) {
+      if (t0 + i >= n) { a[i] = 1.f; x[i] = 0.f; }
       fs = a[i] * fs + x[i];
       fa *= a[i];
     }
@@ -170,10 +223,21 @@ FT_API int ft_causal_conv(const void* x, long long ldx, const float* w, const fl
   ConvParams p;
   p.x = x; p.w = w; p.bias = bias; p.state = state; p.u = u; p.pos = pos; p.slots = slots; p.starts = starts;
   p.ldx = ldx; p.ldu = ldu; p.rows = rows; p.n_single = n_single; p.C = C; p.taps = taps;
-  const int need = (rows + CV_ROWS - 1) / CV_ROWS;
-  const dim3 grid((C / 8 + CV_THREADS - 1) / CV_THREADS, need < 65535 ? need : 65535);
-  if (f32) causal_conv_kernel<float><<<grid, CV_THREADS, 0, stream>>>(p);
-  else causal_conv_kernel<__nv_bfloat16><<<grid, CV_THREADS, 0, stream>>>(p);
+  const int gx = (C / 8 + CV_THREADS - 1) / CV_THREADS;
+  p.walk = rows / (sm_count(device) * 8 / gx + 1);         // enough blocks for the GPU, then longer walks
+  p.walk = p.walk < 1 ? 1 : (p.walk > CV_ROWS ? CV_ROWS : p.walk);
+  const int need = (rows + p.walk - 1) / p.walk;
+  const dim3 grid(gx, need < 65535 ? need : 65535);
+#define FT_CONV(T)                                                                    \
+  switch (taps) {                                                                     \
+    case 1: short_conv_kernel<T, 1><<<grid, CV_THREADS, 0, stream>>>(p); break;       \
+    case 2: short_conv_kernel<T, 2><<<grid, CV_THREADS, 0, stream>>>(p); break;       \
+    case 3: short_conv_kernel<T, 3><<<grid, CV_THREADS, 0, stream>>>(p); break;       \
+    case 4: short_conv_kernel<T, 4><<<grid, CV_THREADS, 0, stream>>>(p); break;       \
+    default: causal_conv_kernel<T><<<grid, CV_THREADS, 0, stream>>>(p);               \
+  }
+  if (f32) { FT_CONV(float) } else { FT_CONV(__nv_bfloat16) }
+#undef FT_CONV
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

@@ -28,29 +28,41 @@ struct RglruGateParams {
   long long ldy, ldo;
 };
 
-__device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float gelu_tanh_f32(float g) {
+// Each function comes in two forms: for fp32 models with CUDA's accurate functions, ahead of bf16 operands and results
+// with the approximate instructions (both work in 32-bit; the second is good to a few units in the last place).
+__device__ __forceinline__ float sigmoid_row(float z, const float*) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_row(float z, const __nv_bfloat16*) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float gelu_row(float g, const float*) {
   const float k = 0.7978845608028654f * (g + 0.044715f * g * g * g);
   return 0.5f * g * (1.f + tanhf(k));
 }
-// gelu ahead of a bf16 store: 0.5 (1 + tanh k) = 1 / (1 + exp(-2 k))
+// 0.5 (1 + tanh k) = 1 / (1 + exp(-2 k))
 __device__ __forceinline__ float gelu_row(float g, const __nv_bfloat16*) {
   return g * __fdividef(1.f, 1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
 }
-__device__ __forceinline__ float gelu_row(float g, const float*) { return gelu_tanh_f32(g); }
 
 // a = exp(log_a) and sqrt(1 - a^2) from q = a - 1: decays are often within 1e-3 of one, where an error in the last place
 // of exp would change the length of the memory, and the difference 1 - a^2 would cancel.
-__device__ __forceinline__ void decay_and_gain(float log_a, float& a, float& gain) {
+__device__ __forceinline__ void decay_and_gain(float log_a, float& a, float& gain, const float*) {
   const float q = expm1f(log_a);
   a = 1.f + q;
   gain = sqrtf(-q * (2.f + q));
 }
+// The same with q from the Taylor series of exp(z) - 1 near zero (seven terms: 3e-9 of q at 0.25) and a plain difference away from it.
+__device__ __forceinline__ void decay_and_gain(float log_a, float& a, float& gain, const __nv_bfloat16*) {
+  const float z = log_a;
+  const float near = z * (1.f + z * (0.5f + z * (1.f / 6 + z * (1.f / 24 + z * (1.f / 120 + z * (1.f / 720 + z * (1.f / 5040)))))));
+  const float q = z > -0.25f ? near : __expf(z) - 1.f;
+  a = 1.f + q;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(gain) : "f"(-q * (2.f + q)));
+}
 
-// Eight channels c .. c + 7 of one row: gate pre-activations zr, zi without bias.
+// Decay and input term of eight channels c .. c + 7 of one row from the gates' pre-activations zr, zi without bias.
 template <typename T>
-__device__ __forceinline__ void rglru_gates8(const RglruGateParams& p, long long row, int c, const float* zr, const float* zi) {
-  float u[8], br[8], bi[8], dec[8], a[8], x[8];
+__device__ __forceinline__ void rglru_gates8(const RglruGateParams& p, long long row, int c, const float* zr, const float* zi, float* a,
+                                             float* x) {
+  const T* kind = nullptr;
+  float u[8], br[8], bi[8], dec[8];
   load8(static_cast<const T*>(p.u) + row * p.ldu + c, u);
   load8(p.r_bias + c, br);
   load8(p.i_bias + c, bi);
@@ -58,14 +70,14 @@ __device__ __forceinline__ void rglru_gates8(const RglruGateParams& p, long long
 #pragma unroll
   for (int e = 0; e < 8; ++e) {
     float gain;
-    decay_and_gain(dec[e] * sigmoid_f32(zr[e] + br[e]), a[e], gain);
-    x[e] = gain * sigmoid_f32(zi[e] + bi[e]) * u[e];
+    decay_and_gain(dec[e] * sigmoid_row(zr[e] + br[e], kind), a[e], gain, kind);
+    x[e] = gain * sigmoid_row(zi[e] + bi[e], kind) * u[e];
   }
-  if (row >= p.n_single) {
-    store8(p.a + row * p.channels + c, a);
-    store8(p.x + row * p.channels + c, x);
-    return;
-  }
+}
+
+// One step of the recurrence for eight channels of a row that is its sequence's only token.
+template <typename T>
+__device__ __forceinline__ void rglru_step8(const RglruGateParams& p, long long row, int c, const float* a, const float* x) {
   float* st = p.state + static_cast<long long>(p.slots[row]) * p.channels + c;
   float s[8], y[8];
   load8(static_cast<const T*>(p.y) + row * p.ldy + c, y);

@@ -195,36 +195,25 @@ qkv_head_finish_kernel(const HeadFinishParams p) {
   }
 }
 
-// The same for heads of 4 * L elements, L = 8 .. 32 lanes with four elements each, when the rotated half is a multiple of
-// four: a lane keeps its elements in registers, its weights over all rows and its angles over all heads of a row; the
+// The same for heads of 8 * L elements, L = 4 .. 16 lanes with eight elements each, when the rotated half is a multiple of
+// eight: a lane keeps its elements in registers, its weights over all rows and its angles over all heads of a row; the
 // partner of an element lies in another lane at the same place.  A warp takes 32 / L heads at a time, HF_BATCH loads ahead.
-constexpr int HF_BATCH = 4;
-
-__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
-  const uint2 u = *reinterpret_cast<const uint2*>(p);
-  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
-  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
-}
-__device__ __forceinline__ void load4(const float* p, float (&f)[4]) {
-  const float4 a = *reinterpret_cast<const float4*>(p);
-  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-}
-__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&f)[4]) {
-  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
-}
-__device__ __forceinline__ void store4(float* p, const float (&f)[4]) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+constexpr int HF_BATCH = 2;
 
 template <typename T, int L>
 __global__ void __launch_bounds__(ROW_THREADS)
 qkv_head_lanes_kernel(const HeadFinishParams p) {
-  constexpr int HPW = 32 / L, D = 4 * L;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hl = lane % L, d = hl * 4;
-  float wq[4] = {1.f, 1.f, 1.f, 1.f}, wk[4] = {1.f, 1.f, 1.f, 1.f};
-  if (p.q_weight) load4(p.q_weight + d, wq);
-  if (p.k_weight) load4(p.k_weight + d, wk);
+  constexpr int HPW = 32 / L, D = 8 * L;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hl = lane % L, d = hl * 8;
+  float wq[8], wk[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) wq[e] = wk[e] = 1.f;
+  if (p.q_weight) load8(p.q_weight + d, wq);
+  if (p.k_weight) load8(p.k_weight + d, wk);
+  const float inv_count = 1.f / static_cast<float>(p.d_true);
   const bool rotated = p.table && d < 2 * p.half, first = d < p.half;
   const int j = first ? d : d - p.half;
-  const int partner = (lane - hl) + (rotated ? (first ? hl + p.half / 4 : hl - p.half / 4) : hl);
+  const int partner = (lane - hl) + (rotated ? (first ? hl + p.half / 8 : hl - p.half / 8) : hl);
   const int q_tasks = (p.Hq + HPW - 1) / HPW, k_tasks = (p.Hkv + HPW - 1) / HPW;
   // a warp takes tasks part * HF_BATCH .. of a row: queries, then keys
   const int parts = gridDim.y * ROW_WARPS, chunk = (q_tasks + k_tasks + HF_BATCH - 1) / HF_BATCH;
@@ -234,60 +223,72 @@ qkv_head_lanes_kernel(const HeadFinishParams p) {
   if (sub >= rows_per_pass) return;
   for (int row = blockIdx.x * rows_per_pass + sub; row < p.rows; row += gridDim.x * rows_per_pass) {
     T* y = static_cast<T*>(p.packed) + static_cast<long long>(row) * p.ld;
-    const int position = p.pos[row];
-    long long token = -1;
-    if (p.k_cache) {
-      const int blk = p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + position / p.block_size];
-      if (blk >= 0 && blk < p.num_blocks) token = static_cast<long long>(blk) * p.block_size + position % p.block_size;
-    }
-    float cs[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
-    if (rotated) {
-      const float4* t = reinterpret_cast<const float4*>(p.table + static_cast<long long>(min(position, p.positions - 1)) * p.half + j);
-      const float4 a = __ldg(t), b = __ldg(t + 1);
-      cs[0] = a.x; cs[1] = a.z; cs[2] = b.x; cs[3] = b.z;
-      const float sg = first ? -1.f : 1.f;
-      sn[0] = sg * a.y; sn[1] = sg * a.w; sn[2] = sg * b.y; sn[3] = sg * b.w;
-    }
-    for (int t0 = part * HF_BATCH; t0 < q_tasks + k_tasks; t0 += warps_per_row * HF_BATCH) {
-      float v[HF_BATCH][4];
+    float v[HF_BATCH][8];
+    auto fetch = [&](int t0) {
 #pragma unroll
       for (int i = 0; i < HF_BATCH; ++i) {
         const int t = t0 + i;
         const bool is_q = t < q_tasks;
         const int h = (is_q ? t : t - q_tasks) * HPW + lane / L;
         const bool ok = t < q_tasks + k_tasks && h < (is_q ? p.Hq : p.Hkv);
-        load4(y + (is_q ? p.q_off : p.k_off) + (ok ? h : 0) * D + d, v[i]);
+        load8(y + (is_q ? p.q_off : p.k_off) + (ok ? h : 0) * D + d, v[i]);
       }
+    };
+    // what does not depend on the position is asked for first
+    fetch(part * HF_BATCH);
+    const int n_values = p.Hkv * p.Dv, v0 = (part * 32 + lane) * 8;
+    float value[8];
+    if (v0 < n_values) load8(y + p.v_off + v0, value);
+    const int position = p.pos[row];
+    long long token = -1;
+    if (p.k_cache) {
+      const int blk = p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + position / p.block_size];
+      if (blk >= 0 && blk < p.num_blocks) token = static_cast<long long>(blk) * p.block_size + position % p.block_size;
+    }
+    float cs[8], sn[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { cs[e] = 1.f; sn[e] = 0.f; }
+    if (rotated) {
+      const float4* t = reinterpret_cast<const float4*>(p.table + static_cast<long long>(min(position, p.positions - 1)) * p.half + j);
+      const float sg = first ? -1.f : 1.f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float4 a = __ldg(t + e);
+        cs[2 * e] = a.x; cs[2 * e + 1] = a.z;
+        sn[2 * e] = sg * a.y; sn[2 * e + 1] = sg * a.w;
+      }
+    }
+    for (int t0 = part * HF_BATCH; t0 < q_tasks + k_tasks; t0 += warps_per_row * HF_BATCH) {
+      if (t0 > part * HF_BATCH) fetch(t0);
 #pragma unroll
       for (int i = 0; i < HF_BATCH; ++i) {
         const int t = t0 + i;
         const bool is_q = t < q_tasks;
         const int h = (is_q ? t : t - q_tasks) * HPW + lane / L;
         const bool ok = t < q_tasks + k_tasks && h < (is_q ? p.Hq : p.Hkv) && (is_q || token >= 0);
-        float sum = v[i][0] * v[i][0] + v[i][1] * v[i][1] + v[i][2] * v[i][2] + v[i][3] * v[i][3];
+        float sum = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += v[i][e] * v[i][e];
 #pragma unroll
         for (int o = L / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
         const bool norm = is_q ? p.q_weight != nullptr : p.k_weight != nullptr;
-        const float r = norm ? 1.f / sqrtf(sum / static_cast<float>(p.d_true) + p.eps) : 1.f;
-        float f[4];
+        const float r = norm ? rsqrtf(sum * inv_count + p.eps) : 1.f;
+        float f[8];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) f[e] = v[i][e] * r * (is_q ? wq[e] : wk[e]);
+        for (int e = 0; e < 8; ++e) f[e] = v[i][e] * r * (is_q ? wq[e] : wk[e]);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
+        for (int e = 0; e < 8; ++e) {
           const float other = __shfl_sync(0xffffffffu, f[e], partner);
           v[i][e] = f[e] * cs[e] + other * sn[e];
         }
-        if (ok) store4((is_q ? y + p.q_off + h * D : static_cast<T*>(p.k_cache) + (token * p.Hkv + h) * D) + d, v[i]);
+        if (ok) store8((is_q ? y + p.q_off + h * D : static_cast<T*>(p.k_cache) + (token * p.Hkv + h) * D) + d, v[i]);
       }
     }
-    if (token >= 0) {                            // values: one run in the row, one in the cache
-      const int n = p.Hkv * p.Dv;
-      for (int i = (part * 32 + lane) * 8; i < n; i += warps_per_row * 256) {
-        float f[8];
-        load8(y + p.v_off + i, f);
-        store8(static_cast<T*>(p.v_cache) + token * n + i, f);
+    if (token >= 0)                              // values: one run in the row, one in the cache
+      for (int i = v0; i < n_values; i += warps_per_row * 256) {
+        if (i > v0) load8(y + p.v_off + i, value);
+        store8(static_cast<T*>(p.v_cache) + token * n_values + i, value);
       }
-    }
   }
 }
 
@@ -323,7 +324,7 @@ FT_API int ft_rms_rows(const void* x, const long long* ids, int n_src, int in_bf
   p.ldx = ldx; p.ldo = ldo; p.ldt = ldt; p.ldy = ldy;
   p.rows = rows; p.n_src = n_src; p.H = H; p.count = count; p.n_terms = n_terms; p.term_rows = term_rows;
   p.eps = eps; p.offset = offset;
-  const int cap = sm_count(device) * 8;
+  const int cap = sm_count(device) * 32;
   const int grid = rows < cap ? rows : cap;
   if (in_bf16) {
     if (out_f32) rms_rows_kernel<__nv_bfloat16, float><<<grid, ROW_THREADS, 0, stream>>>(p);
@@ -366,15 +367,15 @@ FT_API int ft_qkv_head_finish(void* packed, long long ld, const int* pos, const 
   p.D = D; p.Dv = Dv; p.d_true = d_true; p.half = half; p.positions = positions; p.eps = eps;
   p.block_size = block_size; p.max_blocks = max_blocks; p.num_blocks = num_blocks;
   const int wave = sm_count(device) * 8;
-  if ((D == 32 || D == 64 || D == 128) && (!table || (half % 4 == 0 && (reinterpret_cast<uintptr_t>(table) & 15) == 0)) &&
+  if ((D == 32 || D == 64 || D == 128) && (!table || (half % 8 == 0 && (reinterpret_cast<uintptr_t>(table) & 15) == 0)) &&
       row_aligned({q_weight, k_weight})) {
-    const int blocks = rows < wave ? rows : wave;      // a block holds one row or several, by the number of heads
+    const int blocks = rows < 4 * wave ? rows : 4 * wave;      // a block holds one row or several, by the number of heads
     const dim3 grid(blocks, 1);
 #define FT_HL(T, LL) qkv_head_lanes_kernel<T, LL><<<grid, ROW_THREADS, 0, stream>>>(p)
     if (f32) {
-      if (D == 32) FT_HL(float, 8); else if (D == 64) FT_HL(float, 16); else FT_HL(float, 32);
+      if (D == 32) FT_HL(float, 4); else if (D == 64) FT_HL(float, 8); else FT_HL(float, 16);
     } else {
-      if (D == 32) FT_HL(__nv_bfloat16, 8); else if (D == 64) FT_HL(__nv_bfloat16, 16); else FT_HL(__nv_bfloat16, 32);
+      if (D == 32) FT_HL(__nv_bfloat16, 4); else if (D == 64) FT_HL(__nv_bfloat16, 8); else FT_HL(__nv_bfloat16, 16);
     }
 #undef FT_HL
     FT_CUDA_CHECK(cudaGetLastError());

@@ -207,10 +207,21 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
     }
   } else if (warp >= 4) {
     const int ew = warp & 3, wg = (warp - 4) >> 2;   // TMEM lane quarter; which chunks of the columns
+    uint4 u_next[4];                                 // EPI_RGLRU: 32 channels of this lane's row, loaded ahead of the accumulator
+    auto fetch_u = [&](const GroupedTile& t, int n, int r) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        u_next[q] = make_uint4(0u, 0u, 0u, 0u);
+        if (r < t.rows && n + 8 * q < p.N)
+          u_next[q] = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.gates.u) +
+                                                      (static_cast<long long>(t.row0) + r) * p.gates.ldu + t.group * p.a_col + n + 8 * q);
+      }
+    };
     int acc = 0;
     uint32_t acc_phase = 0;
     for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x) {
       const GroupedTile t = grouped_tile(p, tile, m_items, n_blocks, NW);
+      if constexpr (EPI == EPI_RGLRU) fetch_u(t, t.n0 + wg * 32, ew * 32 + lane);
       if (!mbar_wait(tfull_bar(acc), acc_phase, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) break;
       tc_fence_after();
       const uint32_t t_row = tmem_base + (static_cast<uint32_t>(ew * 32) << 16) + static_cast<uint32_t>(acc * BN);
@@ -228,10 +239,11 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
         for (int c = wg * 32; warp_ok && c < NW; c += 64) {
           const int n = t.n0 + c;
           if (n >= p.N) break;
+          if (c > wg * 32) fetch_u(t, n, r);
           if (lane == 0) tma_store_wait_read<0>();       // the previous stores have read the staging tiles
           __syncwarp();
           const int ch = t.group * p.a_col + n;
-#pragma unroll 1
+#pragma unroll
           for (int h = 0; h < 2; ++h) {
             uint32_t za[16], zb[16];
             tmem_ld_32x16(t_row + c + h * 16, za);
@@ -245,7 +257,9 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 float zr[8], zi[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) { zr[e] = __uint_as_float(za[g * 8 + e]); zi[e] = __uint_as_float(zb[g * 8 + e]); }
-                rglru_gates8<__nv_bfloat16>(p.gates, row, ch + o, zr, zi, a8, x8);
+                float u8[8];
+                unpack8(u_next[g + 2 * h], u8);
+                rglru_gates8<__nv_bfloat16>(p.gates, ch + o, zr, zi, u8, a8, x8);
                 if (row < p.gates.n_single) rglru_step8<__nv_bfloat16>(p.gates, row, ch + o, a8, x8);
               } else {
 #pragma unroll
@@ -382,8 +396,9 @@ grouped_gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W
           }
           if (j == 0 && (threadIdx.x & 3) == 0 && ok) {
             const int c = t.group * p.a_col + n;
-            float a8[8], x8[8];
-            rglru_gates8<float>(p.gates, row, c, zr, zi, a8, x8);
+            float u8[8], a8[8], x8[8];
+            load8(static_cast<const float*>(p.gates.u) + row * p.gates.ldu + c, u8);
+            rglru_gates8<float>(p.gates, c, zr, zi, u8, a8, x8);
             if (row < p.gates.n_single) rglru_step8<float>(p.gates, row, c, a8, x8);
             else {
               store8(p.gates.a + row * p.gates.channels + c, a8);

@@ -13,6 +13,7 @@
 namespace ft {
 
 constexpr int CV_THREADS = 128;
+constexpr int CV_BATCH = 4;      // rows loaded together
 constexpr int CV_ROWS = 16;      // most consecutive rows a thread walks (their inputs overlap)
 
 struct ConvParams {
@@ -43,7 +44,7 @@ __device__ __forceinline__ void conv_input(const ConvParams& p, const T* x, cons
 
 // Up to four taps: weights and the sliding inputs stay in registers while the thread walks down its rows.
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(CV_THREADS)
+__global__ void __launch_bounds__(CV_THREADS, 5)
 short_conv_kernel(const ConvParams p) {
   const int c = (blockIdx.x * CV_THREADS + threadIdx.x) * 8;
   if (c >= p.C) return;
@@ -54,30 +55,44 @@ short_conv_kernel(const ConvParams p) {
   const T* x = static_cast<const T*>(p.x) + c;
   for (int r0 = blockIdx.y * p.walk; r0 < p.rows; r0 += gridDim.y * p.walk) {
     const int r1 = min(r0 + p.walk, p.rows);
-    for (int row = r0; row < r1; ++row) {
-      const int pos = p.pos[row], back = pos - p.starts[row];
-      T* st = static_cast<T*>(p.state) + static_cast<long long>(p.slots[row]) * (TAPS - 1) * p.C + c;
-      if (row == r0 || back == 0) {            // a walk or a portion begins: fetch what lies ahead of this row
+    for (int rb = r0; rb < r1; rb += CV_BATCH) {
+      float now[CV_BATCH][8];
+      int pos[CV_BATCH], back[CV_BATCH];
 #pragma unroll
-        for (int d = 1; d < TAPS; ++d) conv_input(p, x, static_cast<const T*>(st), row, pos, back, d, in[d]);
-      }
-      load8(x + static_cast<long long>(row) * p.ldx, in[0]);
-      float acc[8];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = bias[e];
-#pragma unroll
-      for (int d = TAPS - 1; d >= 0; --d)
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] += w[d][e] * in[d][e];
-      store8(static_cast<T*>(p.u) + static_cast<long long>(row) * p.ldu + c, acc);
-      if (TAPS > 1 && row < p.n_single) {      // this thread is the only one at these inputs
-#pragma unroll
-        for (int d = 0; d < TAPS - 1; ++d) store8(st + static_cast<long long>(TAPS - 2 - d) * p.C, in[d]);
+      for (int i = 0; i < CV_BATCH; ++i) {     // past the end: the last row again
+        const int row = min(rb + i, r1 - 1);
+        load8(x + static_cast<long long>(row) * p.ldx, now[i]);
+        pos[i] = __ldg(p.pos + row);
+        back[i] = pos[i] - __ldg(p.starts + row);
       }
 #pragma unroll
-      for (int d = TAPS - 1; d > 0; --d)
+      for (int i = 0; i < CV_BATCH; ++i) {
+        const int row = rb + i;
+        if (row >= r1) break;
+        const bool single = row < p.n_single;
+        T* st = static_cast<T*>(p.state);
+        if (single || back[i] < TAPS - 1) st += static_cast<long long>(p.slots[row]) * (TAPS - 1) * p.C + c;
+        if (row == r0 || back[i] == 0) {       // a walk or a portion begins: fetch what lies ahead of this row
 #pragma unroll
-        for (int e = 0; e < 8; ++e) in[d][e] = in[d - 1][e];
+          for (int d = 1; d < TAPS; ++d) conv_input(p, x, static_cast<const T*>(st), row, pos[i], back[i], d, in[d]);
+        }
+        float acc[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { in[0][e] = now[i][e]; acc[e] = bias[e]; }
+#pragma unroll
+        for (int d = TAPS - 1; d >= 0; --d)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[e] += w[d][e] * in[d][e];
+        store8(static_cast<T*>(p.u) + static_cast<long long>(row) * p.ldu + c, acc);
+        if (TAPS > 1 && single) {              // this thread is the only one at these inputs
+#pragma unroll
+          for (int d = 0; d < TAPS - 1; ++d) store8(st + static_cast<long long>(TAPS - 2 - d) * p.C, in[d]);
+        }
+#pragma unroll
+        for (int d = TAPS - 1; d > 0; --d)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) in[d][e] = in[d - 1][e];
+      }
     }
   }
 }
@@ -123,9 +138,10 @@ causal_conv_kernel(const ConvParams p) {
 // ---------------------------------------------------------------- scan
 // One block per (32 channels, portion): lane = channel, a warp takes SC_STEP consecutive rows of a tile of
 // SC_WARPS * SC_STEP.  Every warp folds its rows into (product of decays, state from zero), the folds of a tile are
-// combined through shared memory, then every warp walks its rows again from its true state.  Each input is read once.
+// combined through shared memory, then every warp walks its rows again from its true state.  Each input is read once;
+// the next tile is loaded while one is computed.
 constexpr int SC_WARPS = 8;
-constexpr int SC_STEP = 16;
+constexpr int SC_STEP = 8;
 
 struct ScanParams {
   const float* a;           // [rows, C]
@@ -141,7 +157,7 @@ struct ScanParams {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(SC_WARPS * 32)
+__global__ void __launch_bounds__(SC_WARPS * 32, 3)
 rglru_scan_kernel(const ScanParams p) {
   __shared__ float fold_a[2][SC_WARPS][32], fold_s[2][SC_WARPS][32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -151,26 +167,36 @@ rglru_scan_kernel(const ScanParams p) {
   const int* span = p.spans + 4 * blockIdx.y;
   const int slot = span[0], row0 = span[1], pos0 = span[2], n = span[3];
   float* st = p.state + static_cast<long long>(slot) * p.C + cc;
-  float carry = pos0 == 0 ? 0.f : *st;
-  int buf = 0;
-  for (int base = 0; base < n; base += SC_WARPS * SC_STEP, buf ^= 1) {
-    const int t0 = base + warp * SC_STEP;
-    float a[SC_STEP], x[SC_STEP], y[SC_STEP];
-    // every load is issued (past the end: of the last row), so that all of a tile are in flight together
+  float a[SC_STEP], x[SC_STEP];
+  T y[SC_STEP];
+  // every load is issued (past the end: of the last row), so that all of a tile are in flight together
+  auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < SC_STEP; ++i) {
       const long long row = row0 + min(t0 + i, n - 1);
       a[i] = __ldg(p.a + row * p.C + cc);
       x[i] = __ldg(p.x + row * p.C + cc);
-      y[i] = static_cast<float>(static_cast<const T*>(p.y)[row * p.ldy + cc]);
+      y[i] = static_cast<const T*>(p.y)[row * p.ldy + cc];
     }
+  };
+  fetch(warp * SC_STEP);
+  float carry = pos0 == 0 ? 0.f : *st;
+  int buf = 0;
+  for (int base = 0; base < n; base += SC_WARPS * SC_STEP, buf ^= 1) {
+    const int t0 = base + warp * SC_STEP;
+    float ca[SC_STEP], cx[SC_STEP];
+    T cy[SC_STEP];
     float fa = 1.f, fs = 0.f;
 #pragma unroll
     for (int i = 0; i < SC_STEP; ++i) {
-      if (t0 + i >= n) { a[i] = 1.f; x[i] = 0.f; }
-      fs = a[i] * fs + x[i];
-      fa *= a[i];
+      const bool ok = t0 + i < n;
+      ca[i] = ok ? a[i] : 1.f;
+      cx[i] = ok ? x[i] : 0.f;
+      cy[i] = y[i];
+      fs = ca[i] * fs + cx[i];
+      fa *= ca[i];
     }
+    if (base + SC_WARPS * SC_STEP < n) fetch(t0 + SC_WARPS * SC_STEP);
     fold_a[buf][warp][lane] = fa;
     fold_s[buf][warp][lane] = fs;
     __syncthreads();          // one barrier per tile: the next tile folds into the other buffer
@@ -183,9 +209,9 @@ rglru_scan_kernel(const ScanParams p) {
     }
 #pragma unroll
     for (int i = 0; i < SC_STEP; ++i) {
-      s = a[i] * s + x[i];
+      s = ca[i] * s + cx[i];
       if (t0 + i < n && c_ok)
-        static_cast<T*>(p.out)[(row0 + t0 + i) * p.ldo + c] = static_cast<T>(s * gelu_row(y[i], static_cast<const T*>(nullptr)));
+        static_cast<T*>(p.out)[(row0 + t0 + i) * p.ldo + c] = static_cast<T>(s * gelu_row(static_cast<float>(cy[i]), static_cast<const T*>(nullptr)));
     }
   }
   if (warp == 0 && c_ok) *st = carry;

@@ -31,14 +31,21 @@ struct RglruGateParams {
 // Each function comes in two forms: for fp32 models with CUDA's accurate functions, ahead of bf16 operands and results
 // with the approximate instructions (both work in 32-bit; the second is good to a few units in the last place).
 __device__ __forceinline__ float sigmoid_row(float z, const float*) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float sigmoid_row(float z, const __nv_bfloat16*) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float fast_rcp(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+__device__ __forceinline__ float sigmoid_row(float z, const __nv_bfloat16*) {
+  return fast_rcp(1.f + fast_exp2(-1.4426950408889634f * z));
+}
 __device__ __forceinline__ float gelu_row(float g, const float*) {
   const float k = 0.7978845608028654f * (g + 0.044715f * g * g * g);
   return 0.5f * g * (1.f + tanhf(k));
 }
 // 0.5 (1 + tanh k) = 1 / (1 + exp(-2 k))
 __device__ __forceinline__ float gelu_row(float g, const __nv_bfloat16*) {
-  return g * __fdividef(1.f, 1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
+  return g * sigmoid_row(1.5957691216057308f * (g + 0.044715f * g * g * g), static_cast<const __nv_bfloat16*>(nullptr));
 }
 
 // a = exp(log_a) and sqrt(1 - a^2) from q = a - 1: decays are often within 1e-3 of one, where an error in the last place
@@ -52,18 +59,18 @@ __device__ __forceinline__ void decay_and_gain(float log_a, float& a, float& gai
 __device__ __forceinline__ void decay_and_gain(float log_a, float& a, float& gain, const __nv_bfloat16*) {
   const float z = log_a;
   const float near = z * (1.f + z * (0.5f + z * (1.f / 6 + z * (1.f / 24 + z * (1.f / 120 + z * (1.f / 720 + z * (1.f / 5040)))))));
-  const float q = z > -0.25f ? near : __expf(z) - 1.f;
+  const float q = z > -0.25f ? near : fast_exp2(1.4426950408889634f * z) - 1.f;
   a = 1.f + q;
-  asm("sqrt.approx.f32 %0, %1;" : "=f"(gain) : "f"(-q * (2.f + q)));
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(gain) : "f"(-q * (2.f + q)));
 }
 
-// Decay and input term of eight channels c .. c + 7 of one row from the gates' pre-activations zr, zi without bias.
+// Decay and input term of eight channels c .. c + 7 of one row from its gates' pre-activations zr, zi (without bias) and its
+// convolved branch u.
 template <typename T>
-__device__ __forceinline__ void rglru_gates8(const RglruGateParams& p, long long row, int c, const float* zr, const float* zi, float* a,
+__device__ __forceinline__ void rglru_gates8(const RglruGateParams& p, int c, const float* zr, const float* zi, const float* u, float* a,
                                              float* x) {
   const T* kind = nullptr;
-  float u[8], br[8], bi[8], dec[8];
-  load8(static_cast<const T*>(p.u) + row * p.ldu + c, u);
+  float br[8], bi[8], dec[8];
   load8(p.r_bias + c, br);
   load8(p.i_bias + c, bi);
   load8(p.decay + c, dec);

@@ -139,12 +139,6 @@ __device__ __forceinline__ void tma_store_2d(const CUtensorMap* m, uint32_t src,
                : "l"(reinterpret_cast<uint64_t>(m)), "r"(src), "r"(x), "r"(y)
                : "memory");
 }
-__device__ __forceinline__ void tma_store_3d(const CUtensorMap* m, uint32_t src, int x, int y, int z) {
-  asm volatile("cp.async.bulk.tensor.3d.global.shared::cta.bulk_group [%0, {%2, %3, %4}], [%1];"
-               :
-               : "l"(reinterpret_cast<uint64_t>(m)), "r"(src), "r"(x), "r"(y), "r"(z)
-               : "memory");
-}
 __device__ __forceinline__ void tma_store_commit() {
   asm volatile("cp.async.bulk.commit_group;" ::: "memory");
 }

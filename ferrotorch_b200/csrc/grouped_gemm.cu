@@ -8,19 +8,18 @@
 //   EPI_GLU    two parts: C = act(r sum_0) * (r sum_1), r a factor per row (a routed token's weight: scaling the
 //              two sums is scaling the input)
 //   EPI_RGLRU  two parts: the gates of a real-gated linear recurrence (see recurrent.cuh), recurrence and all for
-//              rows that are a sequence's only token, decay and input term for the others (32 channels at a time
-//              through a swizzled staging tile per warp and TMA stores, because a lane holds a row)
+//              rows that are a sequence's only token, decay and input term for the others
 //
 // Groups are either segments of rows (a mixture of experts: rows sorted by expert, segments listed on the device by
 // moe_build_kernel, so that no launch depends on the host knowing the counts) or blocks of columns (a block-diagonal
 // matrix: every row takes part in every group with its own columns).
 //
-// The kernel is persistent, one CTA per SM, 384 threads:
+// The kernel is persistent, one CTA per SM, 384 threads (EPI_RGLRU: 640):
 //   warp 0     TMA producer: a ring of {A 128 x 64, W BN x 64} tiles; the A box has only as many rows as the caller
 //              says a segment can have (a decode step: 16 or 32), so small batches move little besides weights
 //   warp 1     MMA issuer
 //   warp 2     TMEM allocator (two accumulators of BN columns)
-//   warps 4-11 epilogue, two warpgroups that share a tile's columns
+//   warps 4-   epilogue, two warpgroups that share a tile's columns (EPI_RGLRU: four, its arithmetic is the bound)
 // Rows of a tile past the end of its segment hold other rows or stale shared memory; rows of an MMA are independent
 // and those are not stored.  All waits are bounded and report through the device status word.
 //
@@ -32,7 +31,6 @@
 
 namespace ft {
 
-constexpr int GG_THREADS = 384;
 constexpr int GG_BM = 128;
 constexpr int GG_BK = 64;
 constexpr int GG_GROUP_M = 16;
@@ -96,27 +94,25 @@ __device__ __forceinline__ float glu_act(float g, int act) {
 
 template <int BN, int EPI>
 struct GgCfg {
-  // EPI_RGLRU: two staging tiles (decay, input term) of 32 rows x 32 fp32 per epilogue warp
-  static constexpr int STAGING = EPI == EPI_RGLRU ? 8 * 2 * 4096 : 0;
+  static constexpr int EPI_WARPS = EPI == EPI_RGLRU ? 16 : 8;
+  static constexpr int THREADS = 128 + 32 * EPI_WARPS;
   static constexpr int A_BYTES = GG_BM * GG_BK * 2;
   static constexpr int B_BYTES = BN * GG_BK * 2;
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
-  static constexpr int STAGES = (216 * 1024 - STAGING) / STAGE_BYTES > 6 ? 6 : (216 * 1024 - STAGING) / STAGE_BYTES;
+  static constexpr int STAGES = (216 * 1024) / STAGE_BYTES > 6 ? 6 : (216 * 1024) / STAGE_BYTES;
   static constexpr int TMEM_COLS = 2 * BN;
-  static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + STAGING + 1024 + 256;
+  static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 + 256;
 };
 
 template <int BN, int EPI>
-__global__ void __launch_bounds__(GG_THREADS, 1)
-grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
-                    const __grid_constant__ CUtensorMap tmDecay, const __grid_constant__ CUtensorMap tmInput, const GroupedParams p) {
+__global__ void __launch_bounds__(GgCfg<BN, EPI>::THREADS, 1)
+grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const GroupedParams p) {
   using Cfg = GgCfg<BN, EPI>;
   constexpr int STAGES = Cfg::STAGES;
   constexpr int NW = EPI == EPI_STORE ? BN : BN / 2;    // output columns of a tile
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-  uint8_t* staging = smem + STAGES * Cfg::STAGE_BYTES;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(staging + Cfg::STAGING);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + STAGES * Cfg::STAGE_BYTES);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2 * STAGES + 4);
   volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -134,7 +130,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
     }
     for (int a = 0; a < 2; ++a) {
       mbar_init(tfull_bar(a), 1);
-      mbar_init(tempty_bar(a), 8);   // one arrival per epilogue warp
+      mbar_init(tempty_bar(a), Cfg::EPI_WARPS);   // one arrival per epilogue warp
     }
     fence_mbar_init();
     tma_prefetch_desc(&tmA);
@@ -207,10 +203,10 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
     }
   } else if (warp >= 4) {
     const int ew = warp & 3, wg = (warp - 4) >> 2;   // TMEM lane quarter; which chunks of the columns
-    uint4 u_next[4];                                 // EPI_RGLRU: 32 channels of this lane's row, loaded ahead of the accumulator
+    uint4 u_next[2];                                 // EPI_RGLRU: 16 channels of this lane's row, loaded ahead of the accumulator
     auto fetch_u = [&](const GroupedTile& t, int n, int r) {
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
+      for (int q = 0; q < 2; ++q) {
         u_next[q] = make_uint4(0u, 0u, 0u, 0u);
         if (r < t.rows && n + 8 * q < p.N)
           u_next[q] = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.gates.u) +
@@ -221,7 +217,7 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
     uint32_t acc_phase = 0;
     for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x) {
       const GroupedTile t = grouped_tile(p, tile, m_items, n_blocks, NW);
-      if constexpr (EPI == EPI_RGLRU) fetch_u(t, t.n0 + wg * 32, ew * 32 + lane);
+      if constexpr (EPI == EPI_RGLRU) fetch_u(t, t.n0 + wg * 16, ew * 32 + lane);
       if (!mbar_wait(tfull_bar(acc), acc_phase, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) break;
       tc_fence_after();
       const uint32_t t_row = tmem_base + (static_cast<uint32_t>(ew * 32) << 16) + static_cast<uint32_t>(acc * BN);
@@ -233,57 +229,30 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       if constexpr (EPI == EPI_GLU)
         if (p.row_scale && row_ok) scale = p.row_scale[row];
       if constexpr (EPI == EPI_RGLRU) {
-        const uint32_t tile_s = smem_u32(staging) + static_cast<uint32_t>(warp - 4) * 8192u;
-        const uint32_t row_s = tile_s + static_cast<uint32_t>(lane) * 128u, sw = static_cast<uint32_t>(lane & 7);
-        const bool stored = warp_ok && row + (t.rows - 1 - r) >= p.gates.n_single;      // some row of the tile leaves its terms
-        for (int c = wg * 32; warp_ok && c < NW; c += 64) {
+        for (int c = wg * 16; warp_ok && c < NW; c += 64) {
           const int n = t.n0 + c;
           if (n >= p.N) break;
-          if (c > wg * 32) fetch_u(t, n, r);
-          if (lane == 0) tma_store_wait_read<0>();       // the previous stores have read the staging tiles
-          __syncwarp();
-          const int ch = t.group * p.a_col + n;
+          uint32_t za[16], zb[16];
+          tmem_ld_32x16(t_row + c, za);
+          tmem_ld_32x16(t_row + NW + c, zb);
+          tmem_ld_wait();
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            uint32_t za[16], zb[16];
-            tmem_ld_32x16(t_row + c + h * 16, za);
-            tmem_ld_32x16(t_row + NW + c + h * 16, zb);
-            tmem_ld_wait();
+          for (int g = 0; g < 2; ++g) {
+            if (!row_ok || n + g * 8 >= p.N) continue;
+            const int ch = t.group * p.a_col + n + g * 8;
+            float zr[8], zi[8], u8[8], a8[8], x8[8];
 #pragma unroll
-            for (int g = 0; g < 2; ++g) {
-              const int o = h * 16 + g * 8;
-              float a8[8], x8[8];
-              if (row_ok && n + o < p.N) {
-                float zr[8], zi[8];
-#pragma unroll
-                for (int e = 0; e < 8; ++e) { zr[e] = __uint_as_float(za[g * 8 + e]); zi[e] = __uint_as_float(zb[g * 8 + e]); }
-                float u8[8];
-                unpack8(u_next[g + 2 * h], u8);
-                rglru_gates8<__nv_bfloat16>(p.gates, ch + o, zr, zi, u8, a8, x8);
-                if (row < p.gates.n_single) rglru_step8<__nv_bfloat16>(p.gates, row, ch + o, a8, x8);
-              } else {
-#pragma unroll
-                for (int e = 0; e < 8; ++e) a8[e] = x8[e] = 0.f;
-              }
-#pragma unroll
-              for (int v = 0; v < 2; ++v) {
-                const uint32_t dst = row_s + ((static_cast<uint32_t>(o / 4 + v) ^ sw) << 4);
-                asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst), "f"(a8[4 * v]), "f"(a8[4 * v + 1]), "f"(a8[4 * v + 2]),
-                             "f"(a8[4 * v + 3]) : "memory");
-                asm volatile("st.shared.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(dst + 4096u), "f"(x8[4 * v]), "f"(x8[4 * v + 1]),
-                             "f"(x8[4 * v + 2]), "f"(x8[4 * v + 3]) : "memory");
-              }
+            for (int e = 0; e < 8; ++e) { zr[e] = __uint_as_float(za[g * 8 + e]); zi[e] = __uint_as_float(zb[g * 8 + e]); }
+            unpack8(u_next[g], u8);
+            rglru_gates8<__nv_bfloat16>(p.gates, ch, zr, zi, u8, a8, x8);
+            if (row < p.gates.n_single) {
+              rglru_step8<__nv_bfloat16>(p.gates, row, ch, a8, x8);
+            } else {
+              store8_sector(p.gates.a + row * p.gates.channels + ch, a8);
+              store8_sector(p.gates.x + row * p.gates.channels + ch, x8);
             }
           }
-          fence_proxy_async_smem();
-          __syncwarp();
-          if (lane == 0 && stored) {
-            // the maps are [blocks, rows, n]: channels past the block and rows past the last are not written (rows of
-            // single tokens are: nothing reads them)
-            tma_store_3d(&tmDecay, tile_s, n, t.row0 + ew * 32, t.group);
-            tma_store_3d(&tmInput, tile_s + 4096u, n, t.row0 + ew * 32, t.group);
-            tma_store_commit();
-          }
+          if (c + 64 < NW) fetch_u(t, n + 64, r);
         }
       } else if (warp_ok) {
 #pragma unroll 1
@@ -313,10 +282,6 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       if (lane == 0) mbar_arrive(tempty_bar(acc));
       acc ^= 1;
       if (acc == 0) acc_phase ^= 1u;
-    }
-    if constexpr (EPI == EPI_RGLRU) {
-      if (lane == 0) tma_store_wait<0>();      // shared memory must outlive the stores that read it
-      __syncwarp();
     }
   }
 
@@ -554,8 +519,8 @@ __global__ void moe_permute_kernel(const uint4* __restrict__ h, long long ldh16,
 }
 
 template <int BN, int EPI>
-static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tb, const CUtensorMap& tdecay, const CUtensorMap& tinput,
-                          const GroupedParams& p, long long tiles, int device, cudaStream_t stream) {
+static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tb, const GroupedParams& p, long long tiles, int device,
+                          cudaStream_t stream) {
   using Cfg = GgCfg<BN, EPI>;
   auto kern = grouped_gemm_kernel<BN, EPI>;
   static bool attr_set[64] = {false};
@@ -564,7 +529,7 @@ static int launch_grouped(const CUtensorMap& ta, const CUtensorMap& tb, const CU
     attr_set[device] = true;
   }
   const int sms = sm_count(device);
-  kern<<<tiles < sms ? static_cast<int>(tiles) : sms, GG_THREADS, Cfg::SMEM_BYTES, stream>>>(ta, tb, tdecay, tinput, p);
+  kern<<<tiles < sms ? static_cast<int>(tiles) : sms, Cfg::THREADS, Cfg::SMEM_BYTES, stream>>>(ta, tb, p);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;
@@ -599,18 +564,9 @@ static int run_grouped(const void* A, long long lda, int total_rows, const void*
   if (rc) return rc;
   rc = make_tmap_2d(&tb, W, 2, p.K, static_cast<uint64_t>(p.groups) * p.parts * p.N, static_cast<uint64_t>(p.K) * 2, GG_BK, bn / 2, 3);
   if (rc) return rc;
-  CUtensorMap td = ta, ti = ta;             // only EPI_RGLRU stores through its maps
-  if (EPI == EPI_RGLRU) {
-    const RglruGateParams& g = p.gates;
-    const uint64_t block = static_cast<uint64_t>(p.N) * 4, row = static_cast<uint64_t>(g.channels) * 4;
-    rc = make_tmap_3d(&td, g.a, 4, p.N, p.rows, p.groups, row, block, 32, 32, 1, 3, false);
-    if (rc) return rc;
-    rc = make_tmap_3d(&ti, g.x, 4, p.N, p.rows, p.groups, row, block, 32, 32, 1, 3, false);
-    if (rc) return rc;
-  }
-  if (bn == 256) return launch_grouped<256, EPI>(ta, tb, td, ti, p, tiles_at(256), device, stream);
-  if (bn == 128) return launch_grouped<128, EPI>(ta, tb, td, ti, p, tiles_at(128), device, stream);
-  return launch_grouped<64, EPI>(ta, tb, td, ti, p, tiles_at(64), device, stream);
+  if (bn == 256) return launch_grouped<256, EPI>(ta, tb, p, tiles_at(256), device, stream);
+  if (bn == 128) return launch_grouped<128, EPI>(ta, tb, p, tiles_at(128), device, stream);
+  return launch_grouped<64, EPI>(ta, tb, p, tiles_at(64), device, stream);
 }
 
 static bool gg_aligned(std::initializer_list<const void*> ps) {
@@ -705,7 +661,9 @@ FT_API int ft_rglru_gates(const void* u, long long ldu, const void* W, const flo
   FT_REQUIRE(blocks > 0 && n > 0 && n % 8 == 0 && ((ldu | ldy | ldo) & 7) == 0 && ldu >= static_cast<long long>(blocks) * n &&
                  ldy >= static_cast<long long>(blocks) * n && ldo >= static_cast<long long>(blocks) * n,
              "ft_rglru_gates: block size %d and strides must be multiples of 8", n);
-  FT_REQUIRE(gg_aligned({u, W, r_bias, i_bias, decay, a, x, state, y, out}), "ft_rglru_gates: pointers must be 16-byte aligned");
+  FT_REQUIRE(gg_aligned({u, W, r_bias, i_bias, decay, state, y, out}) &&
+                 ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(x)) & 31) == 0,
+             "ft_rglru_gates: pointers must be 16-byte aligned, a and x 32-byte");
   FT_REQUIRE(n_single >= 0 && n_single <= rows, "ft_rglru_gates: %d single rows of %d", n_single, rows);
   if (rows <= 0) return FT_E_OK;
   GroupedParams p = {};

@@ -29,6 +29,12 @@ __device__ __forceinline__ void store8(float* p, const float* f) {
   reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
 }
 
+// Eight fp32 as one 32-byte store (a whole sector): for lanes that each hold a row.  p 32-byte aligned.
+__device__ __forceinline__ void store8_sector(float* p, const float* f) {
+  asm volatile("st.global.v8.f32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "f"(f[0]), "f"(f[1]), "f"(f[2]), "f"(f[3]), "f"(f[4]),
+               "f"(f[5]), "f"(f[6]), "f"(f[7]) : "memory");
+}
+
 static inline int blocks_for(long long work, int threads, int device, int per_sm = 8) {
   long long b = (work + threads - 1) / threads;
   const long long cap = static_cast<long long>(sm_count(device)) * per_sm;

@@ -196,99 +196,91 @@ qkv_head_finish_kernel(const HeadFinishParams p) {
 }
 
 // The same for heads of 8 * L elements, L = 4 .. 16 lanes with eight elements each, when the rotated half is a multiple of
-// eight: a lane keeps its elements in registers, its weights over all rows and its angles over all heads of a row; the
-// partner of an element lies in another lane at the same place.  A warp takes 32 / L heads at a time, HF_BATCH loads ahead.
+// eight: elements stay in registers, the partner of an element lies in another lane at the same place.  A warp takes one
+// item at a time: HF_BATCH times 32 / L heads of one row's queries or keys, or a run of its values.
 constexpr int HF_BATCH = 2;
 
 template <typename T, int L>
-__global__ void __launch_bounds__(ROW_THREADS)
+__global__ void __launch_bounds__(ROW_THREADS, 4)
 qkv_head_lanes_kernel(const HeadFinishParams p) {
-  constexpr int HPW = 32 / L, D = 8 * L;
+  constexpr int HPW = 32 / L, D = 8 * L, ITEM_HEADS = HPW * HF_BATCH, ITEM_VALUES = 256 * HF_BATCH;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, hl = lane % L, d = hl * 8;
-  float wq[8], wk[8];
-#pragma unroll
-  for (int e = 0; e < 8; ++e) wq[e] = wk[e] = 1.f;
-  if (p.q_weight) load8(p.q_weight + d, wq);
-  if (p.k_weight) load8(p.k_weight + d, wk);
-  const float inv_count = 1.f / static_cast<float>(p.d_true);
   const bool rotated = p.table && d < 2 * p.half, first = d < p.half;
   const int j = first ? d : d - p.half;
   const int partner = (lane - hl) + (rotated ? (first ? hl + p.half / 8 : hl - p.half / 8) : hl);
-  const int q_tasks = (p.Hq + HPW - 1) / HPW, k_tasks = (p.Hkv + HPW - 1) / HPW;
-  // a warp takes tasks part * HF_BATCH .. of a row: queries, then keys
-  const int parts = gridDim.y * ROW_WARPS, chunk = (q_tasks + k_tasks + HF_BATCH - 1) / HF_BATCH;
-  const int warps_per_row = min(parts, chunk);
-  const int rows_per_pass = parts / warps_per_row;
-  const int me = blockIdx.y * ROW_WARPS + warp, sub = me / warps_per_row, part = me - sub * warps_per_row;
-  if (sub >= rows_per_pass) return;
-  for (int row = blockIdx.x * rows_per_pass + sub; row < p.rows; row += gridDim.x * rows_per_pass) {
+  const float inv_count = 1.f / static_cast<float>(p.d_true), sign = first ? -1.f : 1.f;
+  const int n_values = p.Hkv * p.Dv;
+  const int q_items = (p.Hq + ITEM_HEADS - 1) / ITEM_HEADS, k_items = (p.Hkv + ITEM_HEADS - 1) / ITEM_HEADS;
+  const int row_items = q_items + k_items + (n_values + ITEM_VALUES - 1) / ITEM_VALUES;
+  const long long items = static_cast<long long>(p.rows) * row_items;
+  for (long long item = static_cast<long long>(blockIdx.x) * ROW_WARPS + warp; item < items; item += static_cast<long long>(gridDim.x) * ROW_WARPS) {
+    const int row = static_cast<int>(item / row_items), kind = static_cast<int>(item - static_cast<long long>(row) * row_items);
     T* y = static_cast<T*>(p.packed) + static_cast<long long>(row) * p.ld;
+    const bool is_q = kind < q_items, is_v = kind >= q_items + k_items;
+    const int h0 = (is_q ? kind : kind - q_items) * ITEM_HEADS + lane / L, heads = is_q ? p.Hq : p.Hkv;
+    const int v0 = (kind - q_items - k_items) * ITEM_VALUES + lane * 8;
+    const T* src = y + (is_v ? p.v_off + v0 : (is_q ? p.q_off : p.k_off) + h0 * D + d);
+    const int step = is_v ? 256 : HPW * D;
     float v[HF_BATCH][8];
-    auto fetch = [&](int t0) {
+    bool ok[HF_BATCH];
 #pragma unroll
-      for (int i = 0; i < HF_BATCH; ++i) {
-        const int t = t0 + i;
-        const bool is_q = t < q_tasks;
-        const int h = (is_q ? t : t - q_tasks) * HPW + lane / L;
-        const bool ok = t < q_tasks + k_tasks && h < (is_q ? p.Hq : p.Hkv);
-        load8(y + (is_q ? p.q_off : p.k_off) + (ok ? h : 0) * D + d, v[i]);
-      }
-    };
-    // what does not depend on the position is asked for first
-    fetch(part * HF_BATCH);
-    const int n_values = p.Hkv * p.Dv, v0 = (part * 32 + lane) * 8;
-    float value[8];
-    if (v0 < n_values) load8(y + p.v_off + v0, value);
-    const int position = p.pos[row];
-    long long token = -1;
-    if (p.k_cache) {
-      const int blk = p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + position / p.block_size];
-      if (blk >= 0 && blk < p.num_blocks) token = static_cast<long long>(blk) * p.block_size + position % p.block_size;
+    for (int i = 0; i < HF_BATCH; ++i) {           // what does not depend on the position is asked for first
+      ok[i] = is_v ? v0 + i * 256 < n_values : h0 + i * HPW < heads;
+      if (ok[i]) load8(src + i * step, v[i]);
+      else
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = 0.f;
     }
-    float cs[8], sn[8];
+    const int position = p.pos[row];
+    long long token = 0;
+    if (!is_q) {
+      const int blk = p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + position / p.block_size];
+      if (blk < 0 || blk >= p.num_blocks) continue;
+      token = static_cast<long long>(blk) * p.block_size + position % p.block_size;
+    }
+    if (is_v) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) { cs[e] = 1.f; sn[e] = 0.f; }
+      for (int i = 0; i < HF_BATCH; ++i)
+        if (ok[i]) store8(static_cast<T*>(p.v_cache) + token * n_values + v0 + i * 256, v[i]);
+      continue;
+    }
+    float cs[8], sn[8], w[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { cs[e] = w[e] = 1.f; sn[e] = 0.f; }
     if (rotated) {
       const float4* t = reinterpret_cast<const float4*>(p.table + static_cast<long long>(min(position, p.positions - 1)) * p.half + j);
-      const float sg = first ? -1.f : 1.f;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float4 a = __ldg(t + e);
         cs[2 * e] = a.x; cs[2 * e + 1] = a.z;
-        sn[2 * e] = sg * a.y; sn[2 * e + 1] = sg * a.w;
+        sn[2 * e] = sign * a.y; sn[2 * e + 1] = sign * a.w;
       }
     }
-    for (int t0 = part * HF_BATCH; t0 < q_tasks + k_tasks; t0 += warps_per_row * HF_BATCH) {
-      if (t0 > part * HF_BATCH) fetch(t0);
+    const float* weight = is_q ? p.q_weight : p.k_weight;
+    if (weight) load8(weight + d, w);
+    T* dst = is_q ? y + p.q_off + h0 * D + d : static_cast<T*>(p.k_cache) + (token * p.Hkv + h0) * D + d;
 #pragma unroll
-      for (int i = 0; i < HF_BATCH; ++i) {
-        const int t = t0 + i;
-        const bool is_q = t < q_tasks;
-        const int h = (is_q ? t : t - q_tasks) * HPW + lane / L;
-        const bool ok = t < q_tasks + k_tasks && h < (is_q ? p.Hq : p.Hkv) && (is_q || token >= 0);
+    for (int i = 0; i < HF_BATCH; ++i) {
+      float r = 1.f;
+      if (weight) {                                 // the same in every lane of the warp
         float sum = 0.f;
 #pragma unroll
         for (int e = 0; e < 8; ++e) sum += v[i][e] * v[i][e];
 #pragma unroll
         for (int o = L / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        const bool norm = is_q ? p.q_weight != nullptr : p.k_weight != nullptr;
-        const float r = norm ? rsqrtf(sum * inv_count + p.eps) : 1.f;
-        float f[8];
+        r = rsqrtf(sum * inv_count + p.eps);
+      }
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[e] = v[i][e] * r * (is_q ? wq[e] : wk[e]);
+      for (int e = 0; e < 8; ++e) v[i][e] *= r * w[e];
+      if (p.table) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-          const float other = __shfl_sync(0xffffffffu, f[e], partner);
-          v[i][e] = f[e] * cs[e] + other * sn[e];
+          const float other = __shfl_sync(0xffffffffu, v[i][e], partner);
+          v[i][e] = v[i][e] * cs[e] + other * sn[e];
         }
-        if (ok) store8((is_q ? y + p.q_off + h * D : static_cast<T*>(p.k_cache) + (token * p.Hkv + h) * D) + d, v[i]);
       }
+      if (ok[i]) store8(dst + i * step, v[i]);
     }
-    if (token >= 0)                              // values: one run in the row, one in the cache
-      for (int i = v0; i < n_values; i += warps_per_row * 256) {
-        if (i > v0) load8(y + p.v_off + i, value);
-        store8(static_cast<T*>(p.v_cache) + token * n_values + i, value);
-      }
   }
 }
 
@@ -369,8 +361,11 @@ FT_API int ft_qkv_head_finish(void* packed, long long ld, const int* pos, const 
   const int wave = sm_count(device) * 8;
   if ((D == 32 || D == 64 || D == 128) && (!table || (half % 8 == 0 && (reinterpret_cast<uintptr_t>(table) & 15) == 0)) &&
       row_aligned({q_weight, k_weight})) {
-    const int blocks = rows < 4 * wave ? rows : 4 * wave;      // a block holds one row or several, by the number of heads
-    const dim3 grid(blocks, 1);
+    const int per_pass = 32 / (D / 8) * HF_BATCH;
+    const long long items = static_cast<long long>(rows) * ((Hq + per_pass - 1) / per_pass + (p.Hkv + per_pass - 1) / per_pass +
+                                                            (p.Hkv * Dv + 256 * HF_BATCH - 1) / (256 * HF_BATCH));
+    const long long need = (items + ROW_WARPS - 1) / ROW_WARPS;
+    const int grid = need < 4 * wave ? static_cast<int>(need) : 4 * wave;
 #define FT_HL(T, LL) qkv_head_lanes_kernel<T, LL><<<grid, ROW_THREADS, 0, stream>>>(p)
     if (f32) {
       if (D == 32) FT_HL(float, 4); else if (D == 64) FT_HL(float, 8); else FT_HL(float, 16);

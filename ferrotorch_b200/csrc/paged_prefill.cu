@@ -57,7 +57,8 @@ struct PpParams {
   int* status;
 };
 
-template <int HD, int VD>
+// EXTRAS: a window, sinks or a gate per element (they cost registers that the plain kernel does not have to spare).
+template <int HD, int VD, bool EXTRAS>
 __global__ void __launch_bounds__(PP_THREADS, 1)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                      const __grid_constant__ CUtensorMap tmV, const PpParams p) {
@@ -80,7 +81,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int n_tok = p.items[4 * blockIdx.x + 2], pos0 = p.items[4 * blockIdx.x + 3];
   // tokens and key blocks of each tile
   int nt[2], nb[2];
-  const int j0 = first_visible(pos0 + 1, p.window) / ATT_BN;   // block 0 of this item is key block j0
+  const int j0 = EXTRAS ? first_visible(pos0 + 1, p.window) / ATT_BN : 0;   // block 0 of this item is key block j0
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     nt[i] = min(max(n_tok - i * p.tpt, 0), p.tpt);
@@ -258,8 +259,6 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const int tile_pos = pos0 + ti * p.tpt;
     const int limit = tile_pos + tok;                              // last visible key
     const int warp_limit = tile_pos + (ew * 32) / p.group;         // of this warp's first row
-    const int first = first_visible(limit + 1, p.window);          // first visible key
-    const int warp_first = first_visible(tile_pos + (ew * 32 + 31) / p.group + 1, p.window);   // of its last row
     for (int j = 0; j < my_nb && ok; ++j) {
       if (!mbar_wait(bar(S_FULL + ti), j & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) { ok = false; break; }
       tc_fence_after();
@@ -267,7 +266,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       att2_load_row(s_addr, sp);
       const int kv0 = (j0 + j) * ATT_BN;
       if (kv0 + ATT_BN - 1 > warp_limit) att2_mask_row(sp, kv0, limit);   // warp-uniform branches
-      if (kv0 < warp_first) att2_mask_ahead(sp, kv0, first);              // a row may see nothing of its first blocks
+      // no row of the warp is more than 31 positions past its first; a row may see nothing of its first blocks
+      if (EXTRAS && kv0 < first_visible(warp_limit + 32, p.window)) att2_mask_ahead(sp, kv0, first_visible(limit + 1, p.window));
       const float mx = att2_row_max(sp) * p.scale_log2;  // scale > 0, so the maximum commutes with it
       float alpha = 1.f;
       if (mx > m_ref + ATT2_RESCALE_THRESHOLD) {
@@ -313,10 +313,10 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const long long row = static_cast<long long>(row0) + ti * p.tpt + tok;
       const int hq = kvh * p.group + head;
       float m = m_ref, num = 1.f;
-      sink_join(p.sink, min(hq, p.Hkv * p.group - 1), m, l, num);
+      if constexpr (EXTRAS) sink_join(p.sink, min(hq, p.Hkv * p.group - 1), m, l, num);
       float inv_l = l > 0.f ? num / l : 0.f;
       if (p.gate.g && row_ok && p.gate.elem == 0) inv_l *= head_gate_bf16(p.gate, static_cast<int>(row), hq, 0);
-      const bool elem_gate = p.gate.g && p.gate.elem != 0;
+      const bool elem_gate = EXTRAS && p.gate.g && p.gate.elem != 0;
       __nv_bfloat16* orow = p.out + row * p.ldo + static_cast<long long>(hq) * p.Dv;
 #pragma unroll
       for (int c = 0; c < VD / 32; ++c) {
@@ -359,11 +359,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   if (threadIdx.x == 0 && *abort_word != 0 && p.status) atomicCAS(p.status, 0, *abort_word);
 }
 
-template <int HD, int VD>
-static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PpParams& p,
+template <int HD, int VD, bool EXTRAS>
+static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PpParams& p,
                                 int n_items, int device, cudaStream_t stream) {
   using Cfg = PpCfg<HD, VD>;
-  auto kern = paged_prefill_kernel<HD, VD>;
+  auto kern = paged_prefill_kernel<HD, VD, EXTRAS>;
   static bool attr_set[64] = {false};
   if (!attr_set[device]) {
     FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));
@@ -373,6 +373,14 @@ static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, co
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;
+}
+
+template <int HD, int VD>
+static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PpParams& p,
+                                int n_items, int device, cudaStream_t stream) {
+  const bool extras = p.window > 0 || p.sink || (p.gate.g && p.gate.elem != 0);
+  return extras ? launch_prefill<HD, VD, true>(tq, tk, tv, p, n_items, device, stream)
+                : launch_prefill<HD, VD, false>(tq, tk, tv, p, n_items, device, stream);
 }
 
 }  // namespace ft

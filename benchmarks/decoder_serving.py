@@ -47,7 +47,7 @@ def build(family: str, size: str, layers: int | None = None):
 
         return BopudraForCausalLM(BopudraConfig.uniform(vocab, hidden, n, heads, kv, dim, ff * 3 // 2), device="cuda").random_()
     if family == "zolorax":
-        from ferrotorch_b200.models.zolorax import ZoloraxConfig, ZoloraxForCausalLM
+        from ferrotorch_b200.models.zolorax import ZoloraxForCausalLM
 
         return ZoloraxForCausalLM(zolorax_config(size, n), device="cuda").random_()
     from ferrotorch_b200.models.llama import LlamaConfig, LlamaForCausalLM

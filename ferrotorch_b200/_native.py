@@ -33,7 +33,8 @@ OUT = _PKG / "_C"
 KERNELS_SO = OUT / "libft_kernels.so"
 # Programs that only serve decoders (bin/trace_run) need a part of the sources: with FT_KERNEL_SET=decoder a checkout
 # without a built library compiles these alone.  A library that is already complete is used as it is.
-KERNEL_SETS = {"decoder": ("ft_host", "gemm_tcgen05", "norm_act", "decoder_rows", "recurrent", "grouped_gemm", "paged_attn", "paged_prefill")}
+KERNEL_SETS = {"decoder": ("ft_host", "gemm_tcgen05", "norm_act", "decoder_rows", "streams", "recurrent", "matrix_memory",
+                           "grouped_gemm", "paged_attn", "paged_prefill", "latent_attn")}
 HOST_SO = OUT / "libft_host.so"
 
 NVCC_FLAGS = [

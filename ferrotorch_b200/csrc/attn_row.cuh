@@ -93,9 +93,17 @@ __device__ __forceinline__ float att2_row_max(const f32x2 (&sp)[ATT_BN / 2]) {
   return fmaxf(max3(m0, m1, m2), m3);
 }
 
-// ---------------------------------------------------------------- window, sink, output gate
-// A query that sees `len` keys through a window sees keys first_visible .. len - 1 (window 0: all of them).
-__device__ __forceinline__ int first_visible(int len, int window) { return window > 0 ? max(0, len - window) : 0; }
+// ---------------------------------------------------------------- visible keys, distance bias, sink, output gate
+// A query at position len - 1 sees keys first_visible .. len - 1: with a window the last so many, with chunks (counted from
+// position 0) those of its own chunk; 0: no such limit.
+struct KeyRange {
+  int window, chunk;
+  __device__ __forceinline__ int first_visible(int len) const {
+    const int lo = window > 0 ? max(0, len - window) : 0;
+    return chunk > 0 ? max(lo, max(len - 1, 0) / chunk * chunk) : lo;
+  }
+};
+constexpr float ATT_LOG2E = 1.4426950408889634f;
 
 // A head's sink joins the softmax: exp(sink) in the denominator, no key, no value, no scale.  m, l and acc are the
 // running maximum (in powers of two), the sum and an output element relative to that maximum.

@@ -4,7 +4,7 @@
 //
 // W is [groups, parts, N, K] (bf16, K-major).  With two parts a tile accumulates both products of the same rows, so
 // that the epilogue can combine them:
-//   EPI_STORE  one part:  C = sum
+//   EPI_STORE  one part:  C = sum, optionally times the sigmoid of a gate per element
 //   EPI_GLU    two parts: C = act(r sum_0) * (r sum_1), r a factor per row (a routed token's weight: scaling the
 //              two sums is scaling the input)
 //   EPI_RGLRU  two parts: the gates of a real-gated linear recurrence (see recurrent.cuh), recurrence and all for
@@ -12,7 +12,7 @@
 //
 // Groups are either segments of rows (a mixture of experts: rows sorted by expert, segments listed on the device by
 // moe_build_kernel, so that no launch depends on the host knowing the counts) or blocks of columns (a block-diagonal
-// matrix: every row takes part in every group with its own columns).
+// matrix: every row takes part in every group with its own columns, and the results of group g begin at column g * out_col).
 //
 // The kernel is persistent, one CTA per SM, 384 threads (EPI_RGLRU: 640):
 //   warp 0     TMA producer: a ring of {A 128 x 64, W BN x 64} tiles; the A box has only as many rows as the caller
@@ -46,6 +46,9 @@ struct GroupedParams {
   int N, K, parts;
   void* out;                 // EPI_STORE / EPI_GLU: [rows, ldo]
   long long ldo;
+  int out_col;
+  const void* gate;          // EPI_STORE: element (row, column) is multiplied by sigmoid(gate[row * ldgate + column]); null: not
+  long long ldgate;
   const float* row_scale;    // EPI_GLU: per row, or null
   int act;
   RglruGateParams gates;     // EPI_RGLRU
@@ -273,7 +276,16 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
               f[e] = __uint_as_float(a[h * 8 + e]);
               if constexpr (EPI == EPI_GLU) f[e] = glu_act(scale * f[e], p.act) * (scale * __uint_as_float(b[h * 8 + e]));
             }
-            store8(static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + n + h * 8, f);
+            const long long col = static_cast<long long>(t.group) * p.out_col + n + h * 8;
+            if constexpr (EPI == EPI_STORE) {
+              if (p.gate) {
+                float z[8];
+                load8(static_cast<const __nv_bfloat16*>(p.gate) + row * p.ldgate + col, z);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) f[e] *= sigmoid_row(z[e], static_cast<const __nv_bfloat16*>(nullptr));
+              }
+            }
+            store8(static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + col, f);
           }
         }
       }
@@ -377,7 +389,10 @@ grouped_gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W
             const float g = s * v;
             v = (p.act == 0 ? g / (1.f + expf(-g)) : glu_act(g, p.act)) * (s * acc[1][i][j]);
           }
-          static_cast<float*>(p.out)[row * p.ldo + n] = v;
+          const long long col = static_cast<long long>(t.group) * p.out_col + n;
+          if constexpr (EPI == EPI_STORE)
+            if (p.gate) v *= sigmoid_row(static_cast<const float*>(p.gate)[row * p.ldgate + col], static_cast<const float*>(nullptr));
+          static_cast<float*>(p.out)[row * p.ldo + col] = v;
         }
       }
     }
@@ -385,17 +400,46 @@ grouped_gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W
 }
 
 // ----------------------------------------------------------------------------- routing
-// The experts of a row: the `top` largest router logits (the lower index of equals), their sigmoid as weights.  One
-// warp per row.  With h the logits are computed here, from the row and the router's matrix in fp32 (batches too small
-// for a product of their own); else they are read.
+// The experts of a row and their weights from its router logits z.  One warp per row.
+//   SCORE_SIGMOID  the `top` largest logits (the lower index of equals), weighted by their sigmoid
+//   SCORE_SOFTMAX  scores s = softmax(z) over all outputs; the `top` largest s + correction, weighted by their s, divided by the
+//                  sum of these (+ 1e-20) when normalised
+// With h the logits are computed here, from the row and the router's matrix in fp32 (batches too small for a product of
+// their own); else they are read.
 constexpr int MR_THREADS = 256;
 constexpr int MR_MAX_EXPERTS = 1024;
 
-__device__ __forceinline__ void choose_experts(float* z, int experts, int top, int lane, int* index, float* weight) {
-  for (int k = 0; k < top; ++k) {
+enum : int { SCORE_SIGMOID = 0, SCORE_SOFTMAX = 1 };
+
+struct RouteRule {
+  int outputs, top, score, normalize;   // outputs: router logits of a row
+  const float* correction;              // [outputs] or null
+};
+
+// z [outputs] in shared memory is overwritten (softmax scores take a second array of the same size behind it).
+__device__ __forceinline__ void choose_experts(float* z, const RouteRule& rule, int lane, int* index, float* weight) {
+  const int n = rule.outputs;
+  float* s = z + n;
+  if (rule.score == SCORE_SOFTMAX) {
+    float m = -INFINITY, sum = 0.f;
+    for (int e = lane; e < n; e += 32) m = fmaxf(m, z[e]);
+    m = warp_max(m);
+    for (int e = lane; e < n; e += 32) {
+      s[e] = expf(z[e] - m);
+      sum += s[e];
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < n; e += 32) {
+      s[e] /= sum;
+      z[e] = s[e] + (rule.correction ? rule.correction[e] : 0.f);
+    }
+    __syncwarp();
+  }
+  float total = 0.f;
+  for (int k = 0; k < rule.top; ++k) {
     float best = -INFINITY;
     int at = 0x7fffffff;
-    for (int e = lane; e < experts; e += 32)
+    for (int e = lane; e < n; e += 32)
       if (z[e] > best || (z[e] == best && e < at && best > -INFINITY)) { best = z[e]; at = e; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -403,36 +447,41 @@ __device__ __forceinline__ void choose_experts(float* z, int experts, int top, i
       const int i = __shfl_xor_sync(0xffffffffu, at, o);
       if (b > best || (b == best && i < at)) { best = b; at = i; }
     }
-    if (at >= experts) at = k < experts ? k : 0;     // logits that are not numbers: still an expert that exists
+    if (at >= n) at = k < n ? k : 0;     // logits that are not numbers: still an expert that exists
+    const float w = rule.score == SCORE_SOFTMAX ? s[at] : 1.f / (1.f + expf(-best));
+    total += w;
     if (lane == 0) {
       index[k] = at;
-      weight[k] = 1.f / (1.f + expf(-best));
+      weight[k] = w;
       z[at] = -INFINITY;
     }
     __syncwarp();
   }
+  if (rule.normalize && lane == 0)
+    for (int k = 0; k < rule.top; ++k) weight[k] /= total + 1e-20f;
+  __syncwarp();
 }
 
 __global__ void __launch_bounds__(MR_THREADS)
-moe_choose_kernel(const float* __restrict__ logits, long long ldl, int rows, int experts, int top, int* __restrict__ index,
+moe_choose_kernel(const float* __restrict__ logits, long long ldl, int rows, const RouteRule rule, int* __restrict__ index,
                   float* __restrict__ weight) {
   extern __shared__ float mr_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float* z = mr_sm + warp * experts;
+  float* z = mr_sm + warp * 2 * rule.outputs;
   for (int row = blockIdx.x * (MR_THREADS / 32) + warp; row < rows; row += gridDim.x * (MR_THREADS / 32)) {
-    for (int e = lane; e < experts; e += 32) z[e] = logits[row * ldl + e];
+    for (int e = lane; e < rule.outputs; e += 32) z[e] = logits[row * ldl + e];
     __syncwarp();
-    choose_experts(z, experts, top, lane, index + static_cast<long long>(row) * top, weight + static_cast<long long>(row) * top);
+    choose_experts(z, rule, lane, index + static_cast<long long>(row) * rule.top, weight + static_cast<long long>(row) * rule.top);
   }
 }
 
 // One block per row: the row in registers of all warps in turn, one expert per warp at a time.
 template <typename T>
 __global__ void __launch_bounds__(MR_THREADS)
-moe_route_rows_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ router, int rows, int H, int experts,
-                      int top, int* __restrict__ index, float* __restrict__ weight) {
+moe_route_rows_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ router, int rows, int H, const RouteRule rule,
+                      int* __restrict__ index, float* __restrict__ weight) {
   extern __shared__ float mr_sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, experts = rule.outputs;
   for (int row = blockIdx.x; row < rows; row += gridDim.x) {
     const T* hr = h + row * ldh;
     for (int e0 = warp * 2; e0 < experts; e0 += MR_THREADS / 16) {
@@ -457,14 +506,15 @@ moe_route_rows_kernel(const T* __restrict__ h, long long ldh, const T* __restric
     }
     __syncthreads();
     if (warp == 0)
-      choose_experts(mr_sm, experts, top, lane, index + static_cast<long long>(row) * top, weight + static_cast<long long>(row) * top);
+      choose_experts(mr_sm, rule, lane, index + static_cast<long long>(row) * rule.top, weight + static_cast<long long>(row) * rule.top);
     __syncthreads();
   }
 }
 
 // Sort the (row, choice) pairs by expert.  One block: count, prefix sum, place.  place[i] = sorted position of pair
 // i = row * top + k; scale[position] = its weight; items = (expert, first position, rows) with at most GG_BM rows each,
-// n_items how many.  The order inside an expert is not fixed; every row is computed on its own.
+// n_items how many.  Choices of outputs from `experts` on have no rows and place -1.  The order inside an expert is not
+// fixed; every row is computed on its own.
 __global__ void __launch_bounds__(1024)
 moe_build_kernel(const int* __restrict__ index, const float* __restrict__ weight, int pairs, int experts,
                  int* __restrict__ place, float* __restrict__ scale, int* __restrict__ items, int max_items,
@@ -473,7 +523,8 @@ moe_build_kernel(const int* __restrict__ index, const float* __restrict__ weight
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   count[threadIdx.x] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += 1024) atomicAdd(&count[min(max(index[i], 0), experts - 1)], 1);
+  for (int i = threadIdx.x; i < pairs; i += 1024)
+    if (index[i] < experts) atomicAdd(&count[max(index[i], 0)], 1);
   __syncthreads();
   // exclusive prefix sums of rows and items over the experts (thread = expert)
   const int rows = static_cast<int>(threadIdx.x) < experts ? count[threadIdx.x] : 0;
@@ -498,7 +549,11 @@ moe_build_kernel(const int* __restrict__ index, const float* __restrict__ weight
   if (threadIdx.x == 1023) *n_items = min(i0 + its, max_items);
   __syncthreads();
   for (int i = threadIdx.x; i < pairs; i += 1024) {
-    const int e = min(max(index[i], 0), experts - 1);
+    const int e = max(index[i], 0);
+    if (e >= experts) {
+      place[i] = -1;
+      continue;
+    }
     const int at = base[e] + atomicAdd(&count[e], 1);
     place[i] = at;
     scale[at] = weight[i];
@@ -559,7 +614,7 @@ static int run_grouped(const void* A, long long lda, int total_rows, const void*
   }
   FT_REQUIRE(bn == 64 || bn == 128 || bn == 256, "grouped gemm: tile width %d", bn);
   CUtensorMap ta, tb;
-  const uint64_t inner = p.a_col ? static_cast<uint64_t>(p.groups) * p.a_col : p.K;
+  const uint64_t inner = p.a_col ? static_cast<uint64_t>(p.groups - 1) * p.a_col + p.K : p.K;
   int rc = make_tmap_2d(&ta, A, 2, inner, total_rows, static_cast<uint64_t>(lda) * 2, GG_BK, p.a_rows, 3);
   if (rc) return rc;
   rc = make_tmap_2d(&tb, W, 2, p.K, static_cast<uint64_t>(p.groups) * p.parts * p.N, static_cast<uint64_t>(p.K) * 2, GG_BK, bn / 2, 3);
@@ -582,34 +637,38 @@ using namespace ft;
 // Work items that ft_moe_route can list for `pairs` (row, choice) pairs over `experts`.
 FT_API int ft_moe_max_items(int pairs, int experts) { return (pairs < experts ? pairs : experts) + pairs / GG_BM; }
 
-// Routing of `rows` rows: the experts of every row and their weights (sigmoid of the logit), rows sorted by expert.
-// logits: fp32 [rows, ldl] or null (then computed from h and router [experts, H], the type of h).  Outputs: index
-// int32 [rows, top], weight fp32 [rows, top], place int32 [rows, top] (sorted position), scale fp32 [rows * top] (by
-// position), items int32 [max_items, 3] and n_items for ft_grouped_gemm, sorted [rows * top, H] (the rows of h).
-// h: bf16, or fp32 with f32; H a multiple of 8; experts <= 1024.
+// Routing of `rows` rows (see RouteRule): the choices of every row and their weights, rows sorted by expert.  The router has
+// outputs >= experts logits; choices from `experts` on have no matrices: place -1.  logits: fp32 [rows, ldl] or null (then
+// computed from h and router [outputs, H], the type of h).  Outputs: index int32 [rows, top], weight fp32 [rows, top], place
+// int32 [rows, top] (sorted position), scale fp32 [rows * top] (by position), items int32 [max_items, 3] and n_items for
+// ft_grouped_gemm, sorted [rows * top, H] (the rows of h).  h: bf16, or fp32 with f32; H a multiple of 8; outputs <= 1024.
 FT_API int ft_moe_route(const void* h, long long ldh, const void* router, const float* logits, long long ldl, int rows, int H,
-                        int experts, int top, int f32, int* index, float* weight, int* place, float* scale, int* items,
-                        int max_items, int* n_items, void* sorted, int device, cudaStream_t stream) {
+                        int experts, int outputs, int top, int score, const float* correction, int normalize, int f32, int* index,
+                        float* weight, int* place, float* scale, int* items, int max_items, int* n_items, void* sorted, int device,
+                        cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(h && (router || logits) && index && weight && place && scale && items && n_items && sorted, "ft_moe_route: null pointer");
-  FT_REQUIRE(experts >= 1 && experts <= MR_MAX_EXPERTS && top >= 1 && top <= experts, "ft_moe_route: %d of %d experts", top, experts);
+  FT_REQUIRE(experts >= 1 && outputs >= experts && outputs <= MR_MAX_EXPERTS && top >= 1 && top <= outputs, "ft_moe_route: %d of %d outputs, %d experts", top, outputs, experts);
+  FT_REQUIRE(score == SCORE_SOFTMAX || (score == SCORE_SIGMOID && !correction), "ft_moe_route: score %d", score);
   FT_REQUIRE(H > 0 && H % 8 == 0 && ldh % 8 == 0 && gg_aligned({h, router, sorted}), "ft_moe_route: H=%d and strides must be multiples of 8", H);
   FT_REQUIRE(static_cast<long long>(rows) * top < (1ll << 31) && max_items >= ft_moe_max_items(rows * top, experts), "ft_moe_route: %d items are too few", max_items);
   if (rows <= 0) return FT_E_OK;
   const int sms = sm_count(device);
+  const RouteRule rule = {outputs, top, score, normalize, correction};
   if (logits) {
-    const size_t smem = static_cast<size_t>(MR_THREADS / 32) * experts * sizeof(float);
+    const size_t smem = static_cast<size_t>(MR_THREADS / 32) * 2 * outputs * sizeof(float);
     const int need = (rows + MR_THREADS / 32 - 1) / (MR_THREADS / 32), cap = sms * 8;
-    moe_choose_kernel<<<need < cap ? need : cap, MR_THREADS, smem, stream>>>(logits, ldl, rows, experts, top, index, weight);
+    FT_CUDA_CHECK(cudaFuncSetAttribute(moe_choose_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+    moe_choose_kernel<<<need < cap ? need : cap, MR_THREADS, smem, stream>>>(logits, ldl, rows, rule, index, weight);
   } else {
     const int cap = sms * 8;
-    const size_t smem = static_cast<size_t>(experts) * sizeof(float);
+    const size_t smem = static_cast<size_t>(outputs) * 2 * sizeof(float);
     if (f32)
       moe_route_rows_kernel<float><<<rows < cap ? rows : cap, MR_THREADS, smem, stream>>>(
-          static_cast<const float*>(h), ldh, static_cast<const float*>(router), rows, H, experts, top, index, weight);
+          static_cast<const float*>(h), ldh, static_cast<const float*>(router), rows, H, rule, index, weight);
     else
       moe_route_rows_kernel<__nv_bfloat16><<<rows < cap ? rows : cap, MR_THREADS, smem, stream>>>(
-          static_cast<const __nv_bfloat16*>(h), ldh, static_cast<const __nv_bfloat16*>(router), rows, H, experts, top, index, weight);
+          static_cast<const __nv_bfloat16*>(h), ldh, static_cast<const __nv_bfloat16*>(router), rows, H, rule, index, weight);
   }
   FT_CUDA_CHECK(cudaGetLastError());
   moe_build_kernel<<<1, 1024, 0, stream>>>(index, weight, rows * top, experts, place, scale, items, max_items, n_items);
@@ -646,6 +705,29 @@ FT_API int ft_grouped_gemm(const void* A, long long lda, int total_rows, const v
   p.N = N; p.K = K; p.out = out; p.ldo = ldo; p.row_scale = row_scale; p.act = act;
   return glu ? run_grouped<EPI_GLU>(A, lda, total_rows, W, p, f32, bn, device, stream)
              : run_grouped<EPI_STORE>(A, lda, total_rows, W, p, f32, bn, device, stream);
+}
+
+// The same product over blocks of columns: group g multiplies columns g * a_col .. g * a_col + K - 1 of every row of A [rows, lda]
+// by W [groups, parts, N, K] into columns g * out_col .. of out.  glu as in ft_grouped_gemm; gate (glu 0; [rows, ldgate], null: none):
+// every result is multiplied by the sigmoid of the gate at its row and column.  Sizes and strides multiples of 8.
+FT_API int ft_block_linear(const void* A, long long lda, int rows, const void* W, int groups, int a_col, int N, int K, int glu, int act,
+                           void* out, long long ldo, int out_col, const void* gate, long long ldgate, int f32, int bn, int device,
+                           cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(A && W && out && !(gate && glu), "ft_block_linear: null pointer, or a gate with glu");
+  FT_REQUIRE(groups > 0 && N > 0 && K > 0 && ((N | K | a_col | out_col) & 7) == 0 && ((lda | ldo | ldgate) & 7) == 0 && K <= a_col &&
+                 (out_col >= N || groups == 1) && lda >= static_cast<long long>(groups - 1) * a_col + K &&
+                 ldo >= static_cast<long long>(groups - 1) * out_col + N && (!gate || ldgate >= static_cast<long long>(groups - 1) * out_col + N),
+             "ft_block_linear: %d blocks of N=%d, K=%d", groups, N, K);
+  FT_REQUIRE(gg_aligned({A, W, out, gate}), "ft_block_linear: pointers must be 16-byte aligned");
+  FT_REQUIRE(act >= 0 && act <= 2 && static_cast<long long>(groups) * 2 * N < (1ll << 31), "ft_block_linear: bad argument");
+  if (rows <= 0) return FT_E_OK;
+  GroupedParams p = {};
+  p.rows = rows; p.groups = groups; p.a_col = a_col; p.a_rows = GG_BM; p.N = N; p.K = K;
+  while (p.a_rows > 16 && p.a_rows / 2 >= rows) p.a_rows >>= 1;
+  p.out = out; p.ldo = ldo; p.out_col = out_col; p.act = act; p.gate = gate; p.ldgate = ldgate;
+  return glu ? run_grouped<EPI_GLU>(A, lda, rows, W, p, f32, bn, device, stream)
+             : run_grouped<EPI_STORE>(A, lda, rows, W, p, f32, bn, device, stream);
 }
 
 // Gates of a real-gated linear recurrence for all rows, from u [rows, ldu] (blocks * n channels) and W [blocks, 2, n, n]

@@ -13,7 +13,8 @@
 //                       context, GQA (all query heads of a KV group share one pass over K/V),
 //                       flash-decoding split over the context with a second combine pass, and an
 //                       optional output gate per head.
-//                       A row may see a window of the most recent keys only, and a learned number
+//                       A row may see a window of the most recent keys only, or those of its own chunk; a
+//                       bias that grows with the distance may be taken off the scores, and a learned number
 //                       per head (a sink) may join the denominator.
 //   ft_paged_rows       the same for any mixture of rows (each with its own sequence and number of
 //                       visible keys), any head sizes, bf16 or fp32: the exact, simple kernel.
@@ -61,14 +62,14 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
                     const __nv_bfloat16* __restrict__ v_cache, const int* __restrict__ block_table,
                     const int* __restrict__ row_slot, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
                     float* __restrict__ part_o, float* __restrict__ part_ml, int Hq, int Hkv, long long ldq, long long ldo,
-                    int block_size, int max_blocks, int num_blocks, float scale_log2, int n_splits, int window,
-                    const float* __restrict__ sink, HeadGate gate) {
+                    int block_size, int max_blocks, int num_blocks, float scale_log2, int n_splits, KeyRange range,
+                    const float* __restrict__ slopes, const float* __restrict__ sink, HeadGate gate, float out_scale) {
   constexpr int DV = D / 16;  // dims per lane in the PV phase (half-warp covers D)
   const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int half = lane >> 4, hl = lane & 15;
   const int len = ctx_len[b];
-  const int first = first_visible(len, window);
+  const int first = range.first_visible(len);
   const int tiles_end = (len + 31) >> 5;
   const int tiles_per_split = (tiles_end - (first >> 5) + n_splits - 1) / n_splits;
   const int tile_lo = (first >> 5) + split * tiles_per_split, tile_hi = min(tiles_end, tile_lo + tiles_per_split);
@@ -84,10 +85,11 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   }
   __syncthreads();
 
-  float m[G], l[G], o[G][DV];
+  float m[G], l[G], o[G][DV], slope[G];
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     m[g] = -INFINITY; l[g] = 0.f;
+    slope[g] = slopes ? slopes[kvh * G + g] * ATT_LOG2E : 0.f;
 #pragma unroll
     for (int j = 0; j < DV; ++j) o[g][j] = 0.f;
   }
@@ -128,7 +130,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     float alpha[G];
 #pragma unroll
     for (int g = 0; g < G; ++g) {
-      const float sv = valid ? s[g] : -INFINITY;
+      const float sv = valid ? s[g] - slope[g] * static_cast<float>(len - 1 - key) : -INFINITY;
       const float mx = warp_max(sv);
       const float m_new = fmaxf(m[g], mx);
       const float pv = valid ? fast_exp2(sv - m_new) : 0.f;
@@ -211,7 +213,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     if (n_splits == 1) {
       sink_join(sink, hq, mm, ll, acc);
       out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] =
-          __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq, d) : 0.f);
+          __float2bfloat16(ll > 0.f ? acc / ll * out_scale * head_gate_bf16(gate, b, hq, d) : 0.f);
     } else {
       const long long pidx = (static_cast<long long>(b) * Hq + hq) * n_splits + split;
       part_o[pidx * D + d] = acc;
@@ -222,7 +224,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 
 __global__ void paged_decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                             __nv_bfloat16* __restrict__ out, int Hq, int D, long long ldo, int n_splits,
-                                            const float* __restrict__ sink, HeadGate gate) {
+                                            const float* __restrict__ sink, HeadGate gate, float out_scale) {
   const int hq = blockIdx.x, b = blockIdx.y;
   const long long base = (static_cast<long long>(b) * Hq + hq) * n_splits;
   float mm = -INFINITY;
@@ -238,7 +240,7 @@ __global__ void paged_decode_combine_kernel(const float* __restrict__ part_o, co
     float m = mm;
     sink_join(sink, hq, m, ll, acc);
     out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * D + d] =
-        __float2bfloat16(ll > 0.f ? acc / ll * head_gate_bf16(gate, b, hq, d) : 0.f);
+        __float2bfloat16(ll > 0.f ? acc / ll * out_scale * head_gate_bf16(gate, b, hq, d) : 0.f);
   }
 }
 
@@ -295,7 +297,8 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
                        const int* __restrict__ row_slot, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
                        float* __restrict__ part_o, float* __restrict__ part_ml, int Hq, int Hkv, int D, int Dv, int g_real,
                        long long ldq, long long ldo, int block_size, int max_blocks, int num_blocks, float scale_log2,
-                       int n_splits, int window, const float* __restrict__ sink, HeadGate gate, int* status) {
+                       int n_splits, KeyRange range, const float* __restrict__ slopes, const float* __restrict__ sink, HeadGate gate,
+                       float out_scale, int* status) {
   using Cfg = PtCfg<HD>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -313,7 +316,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
   const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int len = ctx_len[b];
-  const int first = first_visible(len, window);
+  const int first = range.first_visible(len);
   const int tiles_end = (len + PT_TILE - 1) / PT_TILE;
   const int tiles_per_split = (tiles_end - first / PT_TILE + n_splits - 1) / n_splits;
   const int tile_lo = first / PT_TILE + split * tiles_per_split;
@@ -460,9 +463,13 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
     const int ew = warp & 3;
     const int r = ew * 32 + lane;   // key of the tile while scoring, output dim in the epilogue
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(ew * 32) << 16);
-    float m_ref[G], l_part[G];
+    float m_ref[G], l_part[G], slope[G];
 #pragma unroll
-    for (int g = 0; g < G; ++g) { m_ref[g] = -INFINITY; l_part[g] = 0.f; }
+    for (int g = 0; g < G; ++g) {
+      m_ref[g] = -INFINITY;
+      l_part[g] = 0.f;
+      slope[g] = slopes && g < g_real ? slopes[kvh * g_real + g] * ATT_LOG2E : 0.f;
+    }
     bool ok = true;
     // Every softmax thread runs every iteration down to the named barriers, also after a failed
     // wait (later waits then fail at once), so no barrier is ever left short of arrivals.
@@ -482,7 +489,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
       float s[G], mx[G];
 #pragma unroll
       for (int g = 0; g < G; ++g) {
-        s[g] = valid ? __uint_as_float(sv[g]) * scale_log2 : -INFINITY;
+        s[g] = valid ? __uint_as_float(sv[g]) * scale_log2 - slope[g] * static_cast<float>(len - 1 - key) : -INFINITY;
         mx[g] = warp_max(s[g]);
       }
       if (lane == 0) {
@@ -565,7 +572,7 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
           float mm = m_ref[g], ll = l_tot[g], o = acc;
           sink_join(sink, hq, mm, ll, o);
           out[static_cast<long long>(b) * ldo + static_cast<long long>(hq) * Dv + r] =
-              __float2bfloat16(ll > 0.f ? o / ll * head_gate_bf16(gate, b, hq, r) : 0.f);
+              __float2bfloat16(ll > 0.f ? o / ll * out_scale * head_gate_bf16(gate, b, hq, r) : 0.f);
         } else {
           const long long pidx = (static_cast<long long>(b) * Hq + hq) * n_splits + split;
           part_o[pidx * Dv + r] = acc;
@@ -600,8 +607,8 @@ __global__ void __launch_bounds__(PD_THREADS)
 paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                   const int* __restrict__ block_table, const int* __restrict__ row_slot, const int* __restrict__ visible,
                   HeadGate gate, T* __restrict__ out, int rows, int Hq, int Hkv, int D, int Dv, long long ldq, long long ldo,
-                  int block_size, int max_blocks, int num_blocks, float scale, int window, const float* __restrict__ sink,
-                  int head_groups) {
+                  int ldv, int block_size, int max_blocks, int num_blocks, float scale, KeyRange range, const float* __restrict__ slopes,
+                  const float* __restrict__ sink, float out_scale, int head_groups) {
   extern __shared__ float sm[];
   const int g_all = Hq / Hkv;
   const int kvh = blockIdx.y / head_groups, h0 = (blockIdx.y % head_groups) * PR_HEADS;
@@ -615,7 +622,7 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
   for (int row = blockIdx.x; row < rows; row += gridDim.x) {
     __syncthreads();
     const int len = min(visible[row], max_blocks * block_size);
-    const int first = first_visible(len, window);
+    const int first = range.first_visible(len);
     const int* bt = block_table + static_cast<long long>(row_slot[row]) * max_blocks;
     for (int i = threadIdx.x; i < g * D; i += PD_THREADS) {
       const int h = i / D, d = i - h * D;
@@ -649,7 +656,8 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
       for (int h = 0; h < PR_HEADS; ++h) {
         alpha[h] = 1.f;
         if (h >= g) continue;
-        const float sv = valid ? s[h] : -INFINITY;
+        const float bias = slopes ? slopes[kvh * g_all + h0 + h] * ATT_LOG2E * static_cast<float>(len - 1 - key) : 0.f;
+        const float sv = valid ? s[h] - bias : -INFINITY;
         const float m_new = fmaxf(m[h], warp_max(sv));
         const float pv = valid ? exp2f(sv - m_new) : 0.f;
         alpha[h] = exp2f(m[h] - m_new);              // first tile: exp2(-inf) = 0
@@ -666,7 +674,7 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
         for (int j = 0; j < n_keys; ++j) {
           const int kj = key0 + j;
           const int bj = min(max(bt[kj / block_size], 0), num_blocks - 1);
-          const float vd = to_f32(v_cache[((static_cast<long long>(bj) * block_size + kj % block_size) * Hkv + kvh) * Dv + d]);
+          const float vd = to_f32(v_cache[((static_cast<long long>(bj) * block_size + kj % block_size) * Hkv + kvh) * ldv + d]);
 #pragma unroll
           for (int h = 0; h < PR_HEADS; ++h)
             if (h < g) acc[h] += pr[h * 32 + j] * vd;
@@ -698,7 +706,7 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
       }
       const int hq = kvh * g_all + h0 + h;
       sink_join(sink, hq, mm, ll, acc);
-      float v = ll > 0.f ? acc / ll : 0.f;
+      float v = ll > 0.f ? acc / ll * out_scale : 0.f;
       if (gate.g) v *= gate_value(to_f32(static_cast<const T*>(gate.g)[gate.at(row, hq, d)]));
       from_f32(v, out + static_cast<long long>(row) * ldo + static_cast<long long>(hq) * Dv + d);
     }
@@ -740,18 +748,21 @@ FT_API long long ft_paged_decode_scratch(int B, int Hq, int Dv, int n_splits) {
 
 // q: [B, Hq, D] (row stride ldq), out: [B, Hq, Dv] (row stride ldo), ctx_len: int32 [B] = number of
 // cached tokens to attend to (including the current one, which must already be appended), of which the last
-// `window` are visible (0: all).  Row b reads sequence row_slot[b] of the block table (null: sequence b).  sink
+// `window` are visible (0: all), or those of the row's own chunk of `chunk` positions (0: all).  slopes (fp32 [Hq] or null): a
+// head's slope times the distance of a key is taken off its score.  The result is multiplied by out_scale.  Row b reads sequence row_slot[b] of the block table (null: sequence b).  sink
 // (fp32 [Hq] or null): exp(sink) joins a head's denominator.  gate (bf16 or null): element d of head h of row b is
 // multiplied by sigmoid(gate[b * ldg + h * gate_head + d * gate_elem]); one number per head with gate_elem 0.
 FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                            const int* row_slot, const int* ctx_len, const void* gate, const float* sink, void* out,
                            float* scratch, int B, int Hq, int Hkv, int D, int Dv, long long ldq, long long ldg,
                            int gate_head, int gate_elem, long long ldo, int block_size, int max_blocks, int num_blocks,
-                           float scale, int window, int n_splits, int device, cudaStream_t stream) {
+                           float scale, int window, int chunk, const float* slopes, float out_scale, int n_splits, int device,
+                           cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(q && k_cache && v_cache && block_table && ctx_len && out, "ft_paged_decode: null pointer");
   FT_REQUIRE(B >= 0 && Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0, "ft_paged_decode: bad shape");
-  FT_REQUIRE(window >= 0, "ft_paged_decode: negative window");
+  FT_REQUIRE(window >= 0 && chunk >= 0, "ft_paged_decode: negative window or chunk");
+  const KeyRange range = {window, chunk};
   FT_REQUIRE(n_splits >= 1 && (n_splits == 1 || scratch), "ft_paged_decode: splits need scratch");
   if (B == 0) return FT_E_OK;
   const float sl2 = scale * 1.4426950408889634f;
@@ -780,7 +791,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
     kern<<<grid, PT_THREADS, PtCfg<HH>::SMEM_BYTES, stream>>>(                                                  \
         static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache),                \
         static_cast<const __nv_bfloat16*>(q), block_table, row_slot, ctx_len, static_cast<__nv_bfloat16*>(out), \
-        part_o, part_ml, Hq, Hkv, D, Dv, G, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, window, sink, hg, status); \
+        part_o, part_ml, Hq, Hkv, D, Dv, G, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, range, slopes, sink, hg, out_scale, status); \
   }
 #define FT_PT_BY_G(HH)                     \
   if (G == 1) FT_PT_LAUNCH(HH, 1)          \
@@ -797,7 +808,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
   paged_decode_kernel<DD, GG><<<grid, PD_THREADS, 0, stream>>>(                                                \
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),                        \
       static_cast<const __nv_bfloat16*>(v_cache), block_table, row_slot, ctx_len, static_cast<__nv_bfloat16*>(out), \
-      part_o, part_ml, Hq, Hkv, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, window, sink, hg)
+      part_o, part_ml, Hq, Hkv, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, range, slopes, sink, hg, out_scale)
 #define FT_PD_BY_G(DD)                                             \
   switch (G) {                                                     \
     case 1: FT_PD_LAUNCH(DD, 1); break;                            \
@@ -816,7 +827,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
   count_launch();
   if (n_splits > 1) {
     dim3 g2(Hq, B);
-    paged_decode_combine_kernel<<<g2, Dv <= 64 ? 64 : 128, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, Dv, ldo, n_splits, sink, hg);
+    paged_decode_combine_kernel<<<g2, Dv <= 64 ? 64 : 128, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), Hq, Dv, ldo, n_splits, sink, hg, out_scale);
     FT_CUDA_CHECK(cudaGetLastError());
     count_launch();
   }
@@ -824,16 +835,17 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
 }
 
 // Attention of arbitrary rows over the paged cache (see paged_rows_kernel): q [rows, Hq, D], out
-// [rows, Hq, Dv], row_slot / visible int32 [rows]; window, sink (always fp32) and gate as in ft_paged_decode.  All
-// other tensors bf16, or fp32 with f32.
+// [rows, Hq, Dv], row_slot / visible int32 [rows]; window, chunk, slopes, sink (always fp32) and gate as in
+// ft_paged_decode.  A cached value has Dv elements, the next head's begins ldv later (values that are the leading elements of
+// the keys: v_cache = k_cache, ldv = D).  All other tensors bf16, or fp32 with f32.
 FT_API int ft_paged_rows(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* row_slot,
                          const int* visible, const void* gate, const float* sink, void* out, int rows, int Hq, int Hkv,
                          int D, int Dv, long long ldq, long long ldg, int gate_head, int gate_elem, long long ldo,
-                         int block_size, int max_blocks, int num_blocks, float scale, int window, int f32, int device,
-                         cudaStream_t stream) {
+                         int ldv, int block_size, int max_blocks, int num_blocks, float scale, int window, int chunk,
+                         const float* slopes, float out_scale, int f32, int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(q && k_cache && v_cache && block_table && row_slot && visible && out, "ft_paged_rows: null pointer");
-  FT_REQUIRE(Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && D > 0 && Dv > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0 && window >= 0, "ft_paged_rows: bad shape");
+  FT_REQUIRE(Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && D > 0 && Dv > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0 && window >= 0 && chunk >= 0 && ldv >= Dv, "ft_paged_rows: bad shape");
   if (rows <= 0) return FT_E_OK;
   const int groups = (Hq / Hkv + PR_HEADS - 1) / PR_HEADS;
   const size_t smem = sizeof(float) * (static_cast<size_t>(PR_HEADS) * D + static_cast<size_t>(PD_WARPS) * PR_HEADS * Dv +
@@ -846,7 +858,7 @@ FT_API int ft_paged_rows(const void* q, const void* k_cache, const void* v_cache
     FT_CUDA_CHECK(cudaFuncSetAttribute(paged_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     paged_rows_kernel<T><<<grid, PD_THREADS, smem, stream>>>(static_cast<const T*>(q), static_cast<const T*>(k_cache),       \
         static_cast<const T*>(v_cache), block_table, row_slot, visible, hg, static_cast<T*>(out), rows, Hq, Hkv, D, Dv, ldq, \
-        ldo, block_size, max_blocks, num_blocks, scale, window, sink, groups);                                                             \
+        ldo, ldv, block_size, max_blocks, num_blocks, scale, KeyRange{window, chunk}, slopes, sink, out_scale, groups);       \
   }
   if (f32) FT_PR_LAUNCH(float) else FT_PR_LAUNCH(__nv_bfloat16)
 #undef FT_PR_LAUNCH

@@ -1,9 +1,9 @@
 // Causal attention of prompt portions over the paged KV cache on tcgen05 / TMEM (bf16).
 //
 // A portion is a run of consecutive tokens of one sequence whose keys and values are already in the
-// cache (ft_qkv_finish / ft_qkv_head_finish / ft_kv_append); query token at position p sees keys 0 .. p, or
-// the last `window` of them, which lie in pages named by the block table.  With a window an item starts at the
-// key block of its first token's first visible key.  A step holds any number of portions of any lengths, so the work comes as a
+// cache (ft_qkv_finish / ft_qkv_head_finish / ft_kv_append); query token at position p sees keys 0 .. p,
+// the last `window` of them, or those of its own chunk, which lie in pages named by the block table.  An item starts at
+// the key block of its first token's first visible key.  A bias that grows with the distance (a slope per head) may be taken off the scores.  A step holds any number of portions of any lengths, so the work comes as a
 // list of items: up to 2 * tpt consecutive tokens of one sequence, with all query heads of a KV group
 // packed into the rows of the tile (row r = token r / group, head r % group; tpt = 128 / group tokens per
 // 128-row tile).  Packing the group means that K and V are read once per group instead of once per head
@@ -49,20 +49,25 @@ struct PpParams {
   HeadGate gate;            // bf16
   const float* sink;
   __nv_bfloat16* out;
+  const float* slopes;
   long long ldo;
-  int window;
+  KeyRange range;
   int Hkv, group, tpt, D, Dv;
   int block_size, rows_per_box, boxes, max_blocks, num_blocks;
-  float scale_log2;
+  float scale_log2, out_scale;
   int* status;
 };
 
-// EXTRAS: a window, sinks or a gate per element (they cost registers that the plain kernel does not have to spare).
-template <int HD, int VD, bool EXTRAS>
+// What an instance can do beside plain causal attention (it costs registers that the plain kernel does not have to spare):
+// PP_EXTRAS a window, chunks, sinks or a gate per element; PP_BIAS the distance bias as well.
+enum : int { PP_PLAIN = 0, PP_EXTRAS = 1, PP_BIAS = 2 };
+
+template <int HD, int VD, int KIND>
 __global__ void __launch_bounds__(PP_THREADS, 1)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                      const __grid_constant__ CUtensorMap tmV, const PpParams p) {
   using Cfg = PpCfg<HD, VD>;
+  constexpr bool EXTRAS = KIND != PP_PLAIN;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
@@ -81,7 +86,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int n_tok = p.items[4 * blockIdx.x + 2], pos0 = p.items[4 * blockIdx.x + 3];
   // tokens and key blocks of each tile
   int nt[2], nb[2];
-  const int j0 = EXTRAS ? first_visible(pos0 + 1, p.window) / ATT_BN : 0;   // block 0 of this item is key block j0
+  const int j0 = EXTRAS ? p.range.first_visible(pos0 + 1) / ATT_BN : 0;   // block 0 of this item is key block j0
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     nt[i] = min(max(n_tok - i * p.tpt, 0), p.tpt);
@@ -259,16 +264,29 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const int tile_pos = pos0 + ti * p.tpt;
     const int limit = tile_pos + tok;                              // last visible key
     const int warp_limit = tile_pos + (ew * 32) / p.group;         // of this warp's first row
+    float slope = 0.f;                                             // in powers of two per position
+    if constexpr (KIND == PP_BIAS)
+      if (p.slopes) slope = p.slopes[min(kvh * p.group + head, p.Hkv * p.group - 1)] * ATT_LOG2E;
+    const float row_scale = KIND == PP_BIAS ? 1.f : p.scale_log2;  // what a score is still to be multiplied by
     for (int j = 0; j < my_nb && ok; ++j) {
       if (!mbar_wait(bar(S_FULL + ti), j & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) { ok = false; break; }
       tc_fence_after();
       f32x2 sp[ATT_BN / 2];
       att2_load_row(s_addr, sp);
       const int kv0 = (j0 + j) * ATT_BN;
+      if constexpr (KIND == PP_BIAS) {                             // score * scale - slope * (limit - key)
+        const f32x2 sc = f2_pack(p.scale_log2, p.scale_log2), two = f2_pack(2.f * slope, 2.f * slope);
+        const float b0 = slope * static_cast<float>(kv0 - limit);
+        f32x2 bias = f2_pack(b0, b0 + slope);
+#pragma unroll
+        for (int i = 0; i < ATT_BN / 2; ++i) {
+          sp[i] = f2_fma(sp[i], sc, f2_fma(two, f2_pack(static_cast<float>(i), static_cast<float>(i)), bias));
+        }
+      }
       if (kv0 + ATT_BN - 1 > warp_limit) att2_mask_row(sp, kv0, limit);   // warp-uniform branches
       // no row of the warp is more than 31 positions past its first; a row may see nothing of its first blocks
-      if (EXTRAS && kv0 < first_visible(warp_limit + 32, p.window)) att2_mask_ahead(sp, kv0, first_visible(limit + 1, p.window));
-      const float mx = att2_row_max(sp) * p.scale_log2;  // scale > 0, so the maximum commutes with it
+      if (EXTRAS && kv0 < p.range.first_visible(warp_limit + 32)) att2_mask_ahead(sp, kv0, p.range.first_visible(limit + 1));
+      const float mx = att2_row_max(sp) * row_scale;     // scale > 0, so the maximum commutes with it
       float alpha = 1.f;
       if (mx > m_ref + ATT2_RESCALE_THRESHOLD) {
         alpha = fast_exp2(m_ref - mx);  // m_ref = -inf on the first block -> 0
@@ -276,7 +294,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       }
       const float m_use = (m_ref == -INFINITY) ? 0.f : m_ref;
       uint32_t pk[ATT_BN / 2];
-      const float rowsum = att2_exp_row(sp, p.scale_log2, -m_use, pk);
+      const float rowsum = att2_exp_row(sp, row_scale, -m_use, pk);
       l = l * alpha + rowsum;
       if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
         // O of the previous blocks is relative to the old reference: bring it to the new one
@@ -314,7 +332,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const int hq = kvh * p.group + head;
       float m = m_ref, num = 1.f;
       if constexpr (EXTRAS) sink_join(p.sink, min(hq, p.Hkv * p.group - 1), m, l, num);
-      float inv_l = l > 0.f ? num / l : 0.f;
+      float inv_l = l > 0.f ? num / l * p.out_scale : 0.f;
       if (p.gate.g && row_ok && p.gate.elem == 0) inv_l *= head_gate_bf16(p.gate, static_cast<int>(row), hq, 0);
       const bool elem_gate = EXTRAS && p.gate.g && p.gate.elem != 0;
       __nv_bfloat16* orow = p.out + row * p.ldo + static_cast<long long>(hq) * p.Dv;
@@ -359,11 +377,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   if (threadIdx.x == 0 && *abort_word != 0 && p.status) atomicCAS(p.status, 0, *abort_word);
 }
 
-template <int HD, int VD, bool EXTRAS>
+template <int HD, int VD, int KIND>
 static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PpParams& p,
                                 int n_items, int device, cudaStream_t stream) {
   using Cfg = PpCfg<HD, VD>;
-  auto kern = paged_prefill_kernel<HD, VD, EXTRAS>;
+  auto kern = paged_prefill_kernel<HD, VD, KIND>;
   static bool attr_set[64] = {false};
   if (!attr_set[device]) {
     FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));
@@ -378,9 +396,10 @@ static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CU
 template <int HD, int VD>
 static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PpParams& p,
                                 int n_items, int device, cudaStream_t stream) {
-  const bool extras = p.window > 0 || p.sink || (p.gate.g && p.gate.elem != 0);
-  return extras ? launch_prefill<HD, VD, true>(tq, tk, tv, p, n_items, device, stream)
-                : launch_prefill<HD, VD, false>(tq, tk, tv, p, n_items, device, stream);
+  if (p.slopes) return launch_prefill<HD, VD, PP_BIAS>(tq, tk, tv, p, n_items, device, stream);
+  const bool extras = p.range.window > 0 || p.range.chunk > 0 || p.sink || (p.gate.g && p.gate.elem != 0);
+  return extras ? launch_prefill<HD, VD, PP_EXTRAS>(tq, tk, tv, p, n_items, device, stream)
+                : launch_prefill<HD, VD, PP_PLAIN>(tq, tk, tv, p, n_items, device, stream);
 }
 
 }  // namespace ft
@@ -389,7 +408,7 @@ static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, co
 FT_API int ft_paged_prefill_tile(int group) { return group > 0 && group <= ft::ATT_BM ? ft::ATT_BM / group : 0; }
 
 // Attention of prompt portions (see the top of this file).  q: [rows, Hq, D] (row stride ldq), out: [rows,
-// Hq, Dv] (row stride ldo); window, sink and gate as in ft_paged_decode (a gate per element has unit element stride
+// Hq, Dv] (row stride ldo); window, chunk, slopes, sink, gate and out_scale as in ft_paged_decode (a gate per element has unit element stride
 // and 16-byte aligned heads).  items: int32 [n_items, 4] on the
 // device: slot, first query row, number of tokens (<= 2 * ft_paged_prefill_tile), position of the first token;
 // keys 0 .. position of a token must be in the cache.  Page sizes: a divisor of 128 of at least 8, or a
@@ -397,7 +416,8 @@ FT_API int ft_paged_prefill_tile(int group) { return group > 0 && group <= ft::A
 FT_API int ft_paged_prefill(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* items,
                             const void* gate, const float* sink, void* out, int n_items, int rows, int Hq, int Hkv, int D,
                             int Dv, long long ldq, long long ldg, int gate_head, int gate_elem, long long ldo, int block_size,
-                            int max_blocks, int num_blocks, float scale, int window, int device, cudaStream_t stream) {
+                            int max_blocks, int num_blocks, float scale, int window, int chunk, const float* slopes, float out_scale, int device,
+                            cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   using namespace ft;
   FT_REQUIRE(q && k_cache && v_cache && block_table && items && out, "ft_paged_prefill: null pointer");
@@ -410,13 +430,13 @@ FT_API int ft_paged_prefill(const void* q, const void* k_cache, const void* v_ca
              "ft_paged_prefill: strides must be multiples of 8 elements and the scale positive");
   FT_REQUIRE(((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) |
                reinterpret_cast<uintptr_t>(out)) & 15) == 0, "ft_paged_prefill: pointers must be 16-byte aligned");
-  FT_REQUIRE(window >= 0 && (!gate || gate_elem == 0 || (gate_elem == 1 && gate_head % 8 == 0 && ldg % 8 == 0 &&
+  FT_REQUIRE(window >= 0 && chunk >= 0 && (!gate || gate_elem == 0 || (gate_elem == 1 && gate_head % 8 == 0 && ldg % 8 == 0 &&
                                                          (reinterpret_cast<uintptr_t>(gate) & 15) == 0)),
              "ft_paged_prefill: the window is negative or the gate's elements are not packed and aligned");
   if (n_items <= 0) return FT_E_OK;
   PpParams p;
   p.items = items; p.block_table = block_table; p.gate = HeadGate{gate, ldg, gate_head, gate_elem};
-  p.sink = sink; p.window = window;
+  p.sink = sink; p.slopes = slopes; p.range = KeyRange{window, chunk}; p.out_scale = out_scale;
   p.out = static_cast<__nv_bfloat16*>(out); p.ldo = ldo;
   p.Hkv = Hkv; p.group = Hq / Hkv; p.tpt = ATT_BM / p.group; p.D = D; p.Dv = Dv;
   p.block_size = block_size;

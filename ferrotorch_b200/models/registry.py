@@ -69,3 +69,4 @@ def _is_llama(cfg: dict) -> bool:
 register_causal_lm(CausalLMFamily("llama", _is_llama, "ferrotorch_b200.models.llama:LlamaForCausalLM"))
 register_causal_lm(CausalLMFamily("bopudra", lambda c: c.get("architecture") == "Bopudra", "ferrotorch_b200.models.bopudra:BopudraForCausalLM"))
 register_causal_lm(CausalLMFamily("zolorax", lambda c: c.get("architecture") == "Zolorax", "ferrotorch_b200.models.zolorax:ZoloraxForCausalLM"))
+register_causal_lm(CausalLMFamily("tenalorn", lambda c: c.get("architecture") == "Tenalorn", "ferrotorch_b200.models.tenalorn:TenalornForCausalLM"))

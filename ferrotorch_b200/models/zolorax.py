@@ -326,7 +326,8 @@ class ZoloraxForCausalLM(nn.Module):
             else:
                 layer.mixer(x, h, batch, cache.states[i])
             if layer.mlp is not None:
-                pending = layer.mlp(x, layer.norm2(x, out_dtype=self.dtype))
+                h = layer.norm2(x, out_dtype=self.dtype)
+                pending = layer.mlp(h) if isinstance(layer.mlp, RoutedExperts) else layer.mlp(x, h)
             if on_layer is not None:
                 on_layer(i, x if pending is None else x + pending[0][pending[1].long()].float().sum(1))
         if batch.n_want == 0:

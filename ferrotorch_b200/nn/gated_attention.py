@@ -133,6 +133,8 @@ class GatedAttention(nn.Module):
     def forward(self, x: torch.Tensor, h: torch.Tensor, batch, cache, layer: int) -> None:
         """Adds the sublayer of input ``h`` to the fp32 residual ``x``; ``layer``: its (or its source's) place in the cache."""
         a = self.attn
+        if a.chunk is not None or a.distance_bias or (a.rotary is not None and a.rotary.interleaved):
+            raise ValueError("GatedAttention: no chunks, distance bias or rotation of neighbours")
         (qo, qn), (ko, _), (vo, _), (go, gn) = self.segments
         packed = F.linear_rows(h, self.in_proj)
         D.qkv_head_finish(packed, cache, layer, batch, heads=a.heads, dim=a.padded_dim, q_off=qo, k_off=ko, v_off=vo,

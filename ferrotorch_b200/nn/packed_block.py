@@ -50,10 +50,12 @@ class YarnScaling:
 
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotation of the first ``dims`` elements of a head, pairs ``(i, i + dims / 2)``, frequencies ``base ** (-2 i / dims)``."""
+    """Rotation of the first ``dims`` elements of a head, frequencies ``base ** (-2 i / dims)``; pairs ``(i, i + dims / 2)``, or
+    neighbours ``(2 i, 2 i + 1)`` when ``interleaved``."""
     dims: int
     base: float
     scaling: YarnScaling | None = None
+    interleaved: bool = False
 
     def table(self, positions: int, device="cpu") -> torch.Tensor:
         """cos and sin of every position, ``[positions, dims / 2, 2]`` fp32 (angles are computed in 64-bit)."""
@@ -63,12 +65,19 @@ class RotarySpec:
         return torch.stack(ref.rope_tables(self.dims, positions, self.base, kind), -1).contiguous().to(device)
 
 
+def head_slopes(heads: int) -> torch.Tensor:
+    """Slopes of a distance bias: ``2 ** (-8 (h + 1) / heads)`` for head h, fp32."""
+    return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float64).float()
+
+
 @dataclass
 class AttentionSpec:
     """One attention sublayer: ``heads`` query heads over ``kv_heads`` key/value heads of sizes ``dim`` / ``vdim``,
     ``score = (q . k) * scale``; ``temp_coef`` / ``temp_every``: query temperature (coef 0: none); ``window``: a query sees
-    its last so many positions, its own included (``None``: all); ``rotary``: rotation of queries and keys; ``kv_from``:
-    the layer whose keys and values this one reads instead of having its own."""
+    its last so many positions, its own included (``None``: all); ``chunk``: it sees those of its own chunk of so many positions,
+    chunks counted from position 0 (``None``: all); ``distance_bias``: the distance of a key times the head's slope (:func:`head_slopes`)
+    is taken off its score; ``rotary``: rotation of queries and keys; ``kv_from``: the layer whose keys and values this one reads
+    instead of having its own."""
     heads: int
     kv_heads: int
     dim: int
@@ -79,6 +88,8 @@ class AttentionSpec:
     window: int | None = None
     rotary: RotarySpec | None = None
     kv_from: int | None = None
+    chunk: int | None = None
+    distance_bias: bool = False
 
     def validate(self) -> None:
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
@@ -87,6 +98,8 @@ class AttentionSpec:
             raise ValueError("AttentionSpec: temp_every must be positive")
         if self.window is not None and self.window < 1:
             raise ValueError("AttentionSpec: window must be positive or absent")
+        if self.chunk is not None and self.chunk < 1:
+            raise ValueError("AttentionSpec: chunk must be positive or absent")
         if self.rotary is not None and (self.rotary.dims % 2 or not 0 < self.rotary.dims <= self.dim or self.rotary.base <= 1):
             raise ValueError("AttentionSpec: rotation of %d elements of %d" % (self.rotary.dims, self.dim))
 

@@ -22,10 +22,10 @@ _i, _ll, _f, _vp = _native._i, _native._ll, _native._f, _native._vp
 _native.register_protos({
     "ft_kv_append": (_i, [_vp] * 7 + [_i] * 6 + [_ll, _ll, _i, _i, _i, _i, _vp]),
     "ft_paged_decode_scratch": (_ll, [_i, _i, _i, _i]),
-    "ft_paged_decode": (_i, [_vp] * 10 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _i, _vp]),
-    "ft_paged_rows": (_i, [_vp] * 9 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _i, _vp]),
+    "ft_paged_decode": (_i, [_vp] * 10 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp, _f, _i, _i, _vp]),
+    "ft_paged_rows": (_i, [_vp] * 9 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _i, _f, _i, _i, _vp, _f, _i, _i, _vp]),
     "ft_paged_prefill_tile": (_i, [_i]),
-    "ft_paged_prefill": (_i, [_vp] * 8 + [_i] * 6 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp]),
+    "ft_paged_prefill": (_i, [_vp] * 8 + [_i] * 6 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp, _f, _i, _vp]),
 })
 
 
@@ -185,11 +185,15 @@ class PagedKVCache:
     K/V pages of every layer.  ``block_size`` tokens per page (16 in the benchmark configs).
     ``n_kv_heads``, ``head_dim`` and ``v_head_dim`` (default: ``head_dim``) are numbers, or one number per layer.
 
+    ``values_in_keys`` (per layer, default none): a layer without values of its own; its values are the leading ``v_head_dim``
+    elements of its keys (latent attention).
+
     ``states``: what layers keep per sequence slot besides keys and values (recurrent states, by layer).  A state holds
     the whole sequence so far, so such a cache cannot take tokens back (:attr:`rewindable`) nor start from shared pages."""
 
     def __init__(self, n_layers: int, n_kv_heads, head_dim, num_blocks: int, max_seqs: int,
-                 max_seq_len: int, block_size: int = 16, device="cuda", dtype=torch.bfloat16, v_head_dim=None):
+                 max_seq_len: int, block_size: int = 16, device="cuda", dtype=torch.bfloat16, v_head_dim=None,
+                 values_in_keys: list | None = None):
         def per_layer(v):
             return [int(v)] * n_layers if isinstance(v, int) else [int(x) for x in v]
 
@@ -203,7 +207,10 @@ class PagedKVCache:
         self.device = torch.device(device)
         self.pool = PagePool(num_blocks)
         self.k = [torch.zeros((num_blocks, block_size, h, d), device=self.device, dtype=dtype) for h, d, _ in self.shapes]
-        self.v = [torch.zeros((num_blocks, block_size, h, dv), device=self.device, dtype=dtype) for h, _, dv in self.shapes]
+        self.values_in_keys = list(values_in_keys) if values_in_keys is not None else [False] * n_layers
+        self.v = [k[..., :dv] if shared else torch.zeros((num_blocks, block_size, h, dv), device=self.device, dtype=dtype)
+                  for (h, _, dv), k, shared in zip(self.shapes, self.k, self.values_in_keys)]
+        self.token_pages: torch.Tensor | None = None
         # one row more than there are sequences: the padding rows of a captured decode step own no page
         self.pad_slot = max_seqs
         self._table_host = torch.full((max_seqs + 1, self.max_blocks), -1, dtype=torch.int32)
@@ -220,6 +227,10 @@ class PagedKVCache:
         if got is None:
             got = self._rotary[spec] = spec.table(self.max_blocks * self.block_size, self.device)
         return got
+
+    def keep_tokens(self) -> None:
+        """Also keep the token of every position in the pages (for embeddings that look back)."""
+        self.token_pages = torch.zeros((self.num_blocks, self.block_size), device=self.device, dtype=torch.int32)
 
     @property
     def rewindable(self) -> bool:
@@ -305,43 +316,45 @@ class PagedKVCache:
 
     def _tensor_core_ok(self, layer: int, q: torch.Tensor, max_group: int) -> bool:
         Hkv, D, Dv = self.shapes[layer]
-        return (q.dtype == torch.bfloat16 and D % 16 == 0 and Dv % 16 == 0 and D <= 128 and Dv <= 128
+        return (q.dtype == torch.bfloat16 and not self.values_in_keys[layer] and D % 16 == 0 and Dv % 16 == 0 and D <= 128 and Dv <= 128
                 and q.shape[1] // Hkv <= max_group and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0)
 
-    def _rows(self, layer: int, q, visible, slots, scale, gate, out, window, sink) -> None:
+    def _rows(self, layer: int, q, visible, slots, scale, gate, out, window, sink, chunk=None, slopes=None, out_scale=1.0) -> None:
         """Attention of arbitrary rows, any head sizes, bf16 or fp32 (the simple kernel)."""
         T, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
         rc = _native.kernels().ft_paged_rows(
             q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), self.block_table.data_ptr(), slots.data_ptr(),
             visible.data_ptr(), _ptr(gate), _ptr(sink), out.data_ptr(), T, Hq, Hkv, D, Dv, q.stride(0),
-            *_gate_args(gate), out.stride(0), self.block_size, self.max_blocks, self.num_blocks, float(scale), int(window or 0),
-            int(q.dtype == torch.float32), F._dev(q), F._stream())
+            *_gate_args(gate), out.stride(0), self.v[layer].stride(2), self.block_size, self.max_blocks, self.num_blocks, float(scale),
+            int(window or 0), int(chunk or 0), _ptr(slopes), float(out_scale), int(q.dtype == torch.float32), F._dev(q), F._stream())
         _native.check(rc, "ft_paged_rows")
 
     def decode(self, layer: int, q: torch.Tensor, ctx_len: torch.Tensor, scale: float | None = None,
                n_splits: int = 0, seq_ids: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-               out: torch.Tensor | None = None, window: int | None = None, sink: torch.Tensor | None = None) -> torch.Tensor:
+               out: torch.Tensor | None = None, window: int | None = None, sink: torch.Tensor | None = None,
+               chunk: int | None = None, slopes: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
         """One query token per sequence: ``q [B, Hq, D]``, ``ctx_len [B]`` int32 -> ``[B, Hq, Dv]``.  Row b
         reads sequence b, or sequence ``seq_ids[b]`` (int32; a batch of any subset of the live sequences).
         ``gate [B, Hq]`` or ``[B, Hq, Dv]``: output heads or elements are multiplied by its sigmoid.  ``window``: only the
-        last so many keys are visible.  ``sink [Hq]`` (fp32): its exponential joins a head's denominator.  ``out``: where the result goes (the heads of a
-        row packed, any row stride)."""
+        last so many keys are visible; ``chunk``: those of the query's own chunk of so many positions, counted from 0.  ``sink
+        [Hq]`` (fp32): its exponential joins a head's denominator.  ``slopes [Hq]`` (fp32): times the distance of a key, taken off
+        its score.  ``out_scale``: factor of the result.  ``out``: where the result goes (the heads of a row packed, any row stride)."""
         B, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
         scale = scale if scale is not None else D ** -0.5
         table = self.sync_table()
         if not q.is_cuda:
-            o = self._decode_reference(layer, q, ctx_len, scale, seq_ids, window, sink)
-            o = o if gate is None else ref.head_gate(o, gate)
+            o = self._decode_reference(layer, q, ctx_len, scale, seq_ids, window, sink, chunk, slopes)
+            o = self._finish_reference(o, gate, out_scale)
             return o if out is None else out.copy_(o)
         if out is None:
             out = torch.empty((B, Hq, Dv), device=q.device, dtype=q.dtype)
         seq_ids = seq_ids.to(device=q.device, dtype=torch.int32) if seq_ids is not None else None
-        if not self._tensor_core_ok(layer, q, 16) and (q.dtype != torch.bfloat16 or D != Dv or D not in (64, 128)
+        if not self._tensor_core_ok(layer, q, 16) and (q.dtype != torch.bfloat16 or self.values_in_keys[layer] or D != Dv or D not in (64, 128)
                                                        or Hq // Hkv not in (1, 2, 4, 8)):
             rows = seq_ids if seq_ids is not None else torch.arange(B, device=q.device, dtype=torch.int32)
-            self._rows(layer, q, ctx_len, rows, scale, gate, out, window, sink)
+            self._rows(layer, q, ctx_len, rows, scale, gate, out, window, sink, chunk, slopes, out_scale)
             return out
         lib = _native.kernels()
         if n_splits <= 0:
@@ -349,6 +362,8 @@ class PagedKVCache:
             n_splits = 1 if ctas >= 256 else max(1, min(8, 296 // max(ctas, 1)))
             if window:
                 n_splits = min(n_splits, (window + 126) // 128 + 1)          # tiles of 128 keys that a window can touch
+            if chunk:
+                n_splits = min(n_splits, (chunk + 126) // 128 + 1)
         n_scr = int(lib.ft_paged_decode_scratch(B, Hq, Dv, n_splits))
         scratch = F._get_scratch("paged_decode", n_scr, q.device) if n_scr else None
         rc = lib.ft_paged_decode(q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), table.data_ptr(),
@@ -356,16 +371,17 @@ class PagedKVCache:
                                  _ptr(gate), _ptr(sink), out.data_ptr(),
                                  scratch.data_ptr() if scratch is not None else None, B, Hq, Hkv, D, Dv, q.stride(0),
                                  *_gate_args(gate), out.stride(0), self.block_size, self.max_blocks, self.num_blocks,
-                                 float(scale), int(window or 0), n_splits, F._dev(q), F._stream())
+                                 float(scale), int(window or 0), int(chunk or 0), _ptr(slopes), float(out_scale), n_splits, F._dev(q), F._stream())
         _native.check(rc, "ft_paged_decode")
         return out
 
     def attend(self, layer: int, q: torch.Tensor, batch: RaggedBatch, scale: float | None = None,
                gate: torch.Tensor | None = None, out: torch.Tensor | None = None, window: int | None = None,
-               sink: torch.Tensor | None = None) -> torch.Tensor:
+               sink: torch.Tensor | None = None, chunk: int | None = None, slopes: torch.Tensor | None = None,
+               out_scale: float = 1.0) -> torch.Tensor:
         """Causal attention of a whole :class:`RaggedBatch` (its keys and values already appended): ``q [T, Hq, D]`` ->
         ``[T, Hq, Dv]``.  Single tokens run on the decode kernel, longer portions on the prefill kernel; head sizes or
-        types that those do not cover run on the simple kernel.  ``gate``, ``window`` and ``sink`` as in :meth:`decode`."""
+        types that those do not cover run on the simple kernel.  The other arguments as in :meth:`decode`."""
         T, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
         scale = scale if scale is not None else D ** -0.5
@@ -375,26 +391,27 @@ class PagedKVCache:
         n1 = batch.n_single
         if n1:
             self.decode(layer, q[:n1], batch.visible[:n1], scale, seq_ids=batch.slots[:n1],
-                        gate=gate[:n1] if gate is not None else None, out=out[:n1], window=window, sink=sink)
+                        gate=gate[:n1] if gate is not None else None, out=out[:n1], window=window, sink=sink, chunk=chunk, slopes=slopes,
+                        out_scale=out_scale)
         if not batch.spans:
             return out
         if not q.is_cuda:
             for slot, row, start, n in batch.spans:
                 k, v = self.gather(layer, slot, start + n)
-                o = ref.attention(q[None, row:row + n], k[None], v[None], True, scale, start, window, sink)[0][0]
-                out[row:row + n] = o if gate is None else ref.head_gate(o, gate[row:row + n])
+                o = ref.attention(q[None, row:row + n], k[None], v[None], True, scale, start, window, sink, chunk, slopes)[0][0]
+                out[row:row + n] = self._finish_reference(o, gate[row:row + n] if gate is not None else None, out_scale)
             return out
         bs = self.block_size
         if not (self._tensor_core_ok(layer, q, 128) and scale > 0 and bs >= 8 and (128 % bs == 0 or bs % 128 == 0)):
             self._rows(layer, q[n1:], batch.visible[n1:], batch.slots[n1:], scale, gate[n1:] if gate is not None else None, out[n1:],
-                       window, sink)
+                       window, sink, chunk, slopes, out_scale)
             return out
         lib = _native.kernels()
         items = batch.work_items(int(lib.ft_paged_prefill_tile(Hq // Hkv)))
         rc = lib.ft_paged_prefill(q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), table.data_ptr(), items.data_ptr(),
                                   _ptr(gate), _ptr(sink), out.data_ptr(), items.shape[0], T, Hq, Hkv, D, Dv, q.stride(0),
                                   *_gate_args(gate), out.stride(0), bs, self.max_blocks, self.num_blocks, float(scale),
-                                  int(window or 0), F._dev(q), F._stream())
+                                  int(window or 0), int(chunk or 0), _ptr(slopes), float(out_scale), F._dev(q), F._stream())
         _native.check(rc, "ft_paged_prefill")
         return out
 
@@ -431,7 +448,12 @@ class PagedKVCache:
             if self._pages[s]:
                 self.free_sequence(s)
 
-    def _decode_reference(self, layer, q, ctx_len, scale, seq_ids=None, window=None, sink=None):
+    @staticmethod
+    def _finish_reference(o, gate, out_scale):
+        o = o if gate is None else ref.head_gate(o, gate)
+        return o if out_scale == 1.0 else (o.float() * out_scale).to(o.dtype)
+
+    def _decode_reference(self, layer, q, ctx_len, scale, seq_ids=None, window=None, sink=None, chunk=None, slopes=None):
         """Host form of the paged-decode kernel, all rows at once: the pages of every row are gathered through
         the block table into a padded ``[B, L, Hkv, D]`` view and positions past a row's length are masked."""
         B, Hq, D = q.shape
@@ -448,6 +470,10 @@ class PagedKVCache:
         dead = at >= ctx[:, None]
         if window:
             dead = dead | (at < ctx[:, None] - window)
+        if chunk:
+            dead = dead | (at < (ctx[:, None] - 1) // chunk * chunk)
+        if slopes is not None:
+            s = s - slopes.float().view(1, Hkv, Hq // Hkv, 1) * (ctx[:, None] - 1 - at).float()[:, None, None, :]
         s = s.masked_fill(dead[:, None, None, :], float("-inf"))
         if sink is not None:                              # one more column of the softmax, without a value
             s = torch.cat([s, sink.float().view(1, Hkv, Hq // Hkv, 1).expand(B, -1, -1, 1)], -1)

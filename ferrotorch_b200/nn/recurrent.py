@@ -1,5 +1,6 @@
 """Recurrent sublayers of decoders: a gated branch, a short causal convolution and a real-gated linear recurrence with
-diagonal state.  What a sequence has seen lives in its slot of an :class:`RGLRUState`."""
+diagonal state, whose sequences live in the slots of an :class:`RGLRUState`; sizes and state of matrix memories
+(:class:`MatrixMemorySpec`, :class:`MatrixMemoryState`), which :mod:`~ferrotorch_b200.nn.parallel_mixer` runs beside attention."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -42,6 +43,38 @@ class RGLRUState:
     def __init__(self, slots: int, spec: RGLRUSpec, device, dtype: torch.dtype):
         self.state = torch.zeros((slots, spec.padded_width), device=device, dtype=torch.float32)
         self.conv = torch.zeros((slots, spec.conv - 1, spec.padded_width), device=device, dtype=dtype)
+
+
+@dataclass
+class MatrixMemorySpec:
+    """``heads`` memories of ``dim x vdim`` with exponential gates, whose logarithms are capped at ``gate_cap``."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    def validate(self) -> None:
+        if min(self.heads, self.dim, self.vdim) < 1 or not self.gate_cap > 0:
+            raise ValueError("MatrixMemorySpec: %d heads of %d x %d, gates capped at %g" % (self.heads, self.dim, self.vdim, self.gate_cap))
+
+    @property
+    def padded_dim(self) -> int:
+        return round_up(self.dim, 16)
+
+    @property
+    def padded_vdim(self) -> int:
+        return round_up(self.vdim, 16)
+
+
+class MatrixMemoryState:
+    """State of one layer for every sequence slot, fp32: the memories ``S [slots, heads, dim, vdim]``, their normalisers ``n [slots,
+    heads, dim]`` and the running maxima ``m [slots, heads]`` that both are relative to (padded sizes).  A slot is not cleared between
+    sequences: position 0 starts from zero."""
+
+    def __init__(self, slots: int, spec: MatrixMemorySpec, device):
+        self.S = torch.zeros((slots, spec.heads, spec.padded_dim, spec.padded_vdim), device=device)
+        self.n = torch.zeros((slots, spec.heads, spec.padded_dim), device=device)
+        self.m = torch.zeros((slots, spec.heads), device=device)
 
 
 class RGLRUBlock(nn.Module):

@@ -1,13 +1,15 @@
 """Front ends of the kernels that pre-norm decoders over paged caches use beside the projections and the attention: RMS
-norm of fp32 residual rows, the per-head pass between projection and attention (``csrc/decoder_rows.cu``), short
-convolution and gated linear recurrence (``csrc/recurrent.cu``), routing and grouped products of expert layers
-(``csrc/grouped_gemm.cu``).
+norm of fp32 residual rows, the per-head pass between projection and attention (``csrc/decoder_rows.cu``), residuals of
+several streams and n-gram embeddings (``csrc/streams.cu``), short convolution and gated linear recurrence
+(``csrc/recurrent.cu``), matrix memories (``csrc/matrix_memory.cu``), the pass ahead of latent attention
+(``csrc/latent_attn.cu``), routing and grouped products of expert layers and products by blocks (``csrc/grouped_gemm.cu``).
 
 CUDA tensors run the kernels (bf16 on the tensor cores where there is a product, fp32 in true 32-bit); CPU tensors run
 the plain forms of :mod:`ferrotorch_b200.ops.reference`."""
 from __future__ import annotations
 
 from dataclasses import dataclass
+from typing import NamedTuple
 
 import torch
 
@@ -23,7 +25,13 @@ _native.register_protos({
     "ft_rglru_gates": (_i, [_vp, _ll] + [_vp] * 4 + [_i] * 3 + [_vp, _vp, _i] + [_vp] * 4 + [_ll, _vp, _ll] + [_i] * 3 + [_vp]),
     "ft_rglru_scan": (_i, [_vp] * 3 + [_ll, _vp, _ll, _vp, _vp, _i, _vp, _ll, _vp] + [_i] * 4 + [_vp]),
     "ft_moe_max_items": (_i, [_i, _i]),
-    "ft_moe_route": (_i, [_vp, _ll, _vp, _vp, _ll] + [_i] * 5 + [_vp] * 5 + [_i, _vp, _vp, _i, _vp]),
+    "ft_moe_route": (_i, [_vp, _ll, _vp, _vp, _ll] + [_i] * 6 + [_vp, _i, _i] + [_vp] * 5 + [_i, _vp, _vp, _i, _vp]),
+    "ft_block_linear": (_i, [_vp, _ll, _i, _vp] + [_i] * 6 + [_vp, _ll, _i, _vp, _ll] + [_i] * 3 + [_vp]),
+    "ft_stream_step": (_i, [_vp, _ll, _ll, _vp, _i] + [_vp] * 4 + [_i, _vp, _ll, _vp, _ll, _i, _vp, _vp, _i, _vp, _ll, _vp, _vp, _ll] + [_i] * 3 + [_f, _i, _i, _vp]),
+    "ft_embed_bigram": (_i, [_vp] * 8 + [_ll, _i, _i, _ll, _ll, _f, _vp, _i] + [_vp] * 3 + [_i] * 3 + [_f] + [_i] * 5 + [_vp]),
+    "ft_softcap": (_i, [_vp, _ll, _f, _i, _vp]),
+    "ft_latent_finish": (_i, [_vp, _ll, _vp, _i] + [_vp] * 6 + [_i] * 11 + [_f] + [_i] * 5 + [_vp]),
+    "ft_memory_steps": (_i, [_vp] * 4 + [_ll, _vp, _ll, _i] + [_vp] * 7 + [_ll] + [_i] * 4 + [_f] * 4 + [_vp] * 3 + [_i] * 3 + [_vp]),
     "ft_grouped_gemm": (_i, [_vp, _ll, _i] + [_vp] * 3 + [_i] * 5 + [_vp, _i, _vp, _ll] + [_i] * 4 + [_vp]),
 })
 
@@ -49,7 +57,7 @@ def rms_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, *, count: int | 
         return ref.rms_rows(xs, weight, eps, count, offset).to(dt)
     n = x.shape[0] if rows is None else rows.numel()
     y = torch.empty((n, x.shape[1]), device=x.device, dtype=dt)
-    terms, where = pending if pending is not None else (None, None)
+    terms, where = pending[:2] if pending is not None else (None, None)
     rc = _native.kernels().ft_rms_rows(
         x.data_ptr(), _ptr(rows), x.shape[0], 0, x.data_ptr() if update else None, _ptr(terms), _ptr(where),
         where.shape[1] if where is not None else 0, terms.shape[0] if terms is not None else 0, weight.data_ptr(), y.data_ptr(),
@@ -75,6 +83,93 @@ def embedding_rms(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, 
         float(offset), F._dev(table), F._stream())
     _native.check(rc, "ft_rms_rows")
     return x, h
+
+
+# --------------------------------------------------------------------------- residuals of several streams
+class SublayerTerms(NamedTuple):
+    """What a sublayer adds to the residual, not yet summed: rows ``terms[where[i, j]]`` for all j (times ``weight[i, j]``), a dense
+    row ``dense[i]``; where ``where[i, j]`` is negative, ``weight[i, j]`` times the sublayer's own input ``own[i]``."""
+    terms: torch.Tensor | None = None
+    where: torch.Tensor | None = None
+    weight: torch.Tensor | None = None
+    dense: torch.Tensor | None = None
+    own: torch.Tensor | None = None
+
+    def total(self) -> torch.Tensor:
+        """The sum, fp32."""
+        y = self.dense.float() if self.dense is not None else 0.0
+        if self.terms is None:
+            return y
+        t, w = self.terms[self.where.clamp(min=0).long()].float(), self.weight if self.weight is not None else torch.ones_like(self.where, dtype=torch.float32)
+        if self.own is not None:
+            t = torch.where(self.where[..., None] < 0, self.own.float()[:, None], t)
+        return y + (t * w[..., None]).sum(1)
+
+
+def stream_step(x: torch.Tensor, y: SublayerTerms, mix: torch.Tensor, out: torch.Tensor, into: torch.Tensor, weight: torch.Tensor, eps: float,
+                *, count: int, out_dtype: torch.dtype, rows: torch.Tensor | None = None, update: bool = True):
+    """All streams of the residual at once after a sublayer, and the next sublayer's input from them: ``(x', h)``.
+
+    ``x [T, S, H]`` fp32 (a broadcast view when the streams are still equal): ``x'_t = sum_s mix[s, t] x_s + out[t] y``, in place
+    where ``x`` is dense; ``h`` the RMS norm of ``sum_t into[t] x'_t`` times ``weight``.  ``rows``: only these rows; without
+    ``update`` (always with ``rows``) the streams are not written."""
+    T, S, H = x.shape
+    if not x.is_cuda:
+        new = torch.einsum("nsh,st->nth", x, mix) + out[:, None] * y.total()[:, None, :]
+        u = torch.einsum("nth,t->nh", new if rows is None else new[rows], into)
+        return new, ref.rms_rows(u, weight, eps, count).to(out_dtype)
+    n = T if rows is None else rows.numel()
+    update = update and rows is None
+    dest = None
+    if update:
+        dest = x if x.is_contiguous() else torch.empty((T, S, H), device=x.device, dtype=torch.float32)
+    h = torch.empty((n, H), device=x.device, dtype=out_dtype)
+    t, own, dense = y.terms, y.own, y.dense
+    rc = _native.kernels().ft_stream_step(
+        x.data_ptr(), x.stride(0), x.stride(1) if S > 1 else 0, _ptr(rows), T, _ptr(dest), mix.data_ptr(), out.data_ptr(), into.data_ptr(), S, _ptr(dense),
+        dense.stride(0) if dense is not None else 0, _ptr(t), t.stride(0) if t is not None else 0, t.shape[0] if t is not None else 0,
+        _ptr(y.where), _ptr(y.weight), y.where.shape[1] if t is not None else 0, _ptr(own), own.stride(0) if own is not None else 0,
+        weight.data_ptr(), h.data_ptr(), h.stride(0), n, H, count, float(eps), int(out_dtype == torch.float32), F._dev(x), F._stream())
+    _native.check(rc, "ft_stream_step")
+    return (dest if update else x), h
+
+
+def embed_bigram(batch, cache, table: torch.Tensor, bigram: torch.Tensor, scale: float, mul_prev: int, mul_cur: int, into: torch.Tensor,
+                 weight: torch.Tensor, eps: float, *, count: int, out_dtype: torch.dtype):
+    """``x = scale * table[token] + bigram[row]`` of a ragged batch (fp32 ``[T, H]``) and the RMS norm of ``sum(into) x``: ``(x, h)``.
+
+    ``row = (previous * mul_prev + token * mul_cur) mod buckets``, the last row of ``bigram [buckets + 1, H]`` for the first token of
+    a sequence.  The cache keeps the tokens (:meth:`PagedKVCache.keep_tokens`): a portion finds its previous token there."""
+    T, H, buckets = batch.n_rows, table.shape[1], bigram.shape[0] - 1
+    pages = cache.token_pages
+    cache.sync_table()
+    if not table.is_cuda:
+        pos, slots, bs = batch.positions.long(), batch.slots.long(), cache.block_size
+        before = (pos - 1).clamp(min=0)
+        held = pages[cache._table_host[slots, before // bs].long().clamp(min=0), before % bs].long()
+        prev = torch.where(pos > batch.starts, torch.cat([batch.tokens[:1], batch.tokens[:-1]]), held)
+        row = torch.where(pos > 0, (prev * mul_prev + batch.tokens * mul_cur) % buckets, buckets)
+        pages[cache._table_host[slots, pos // bs].long(), pos % bs] = batch.tokens.int()
+        x = scale * table[batch.tokens].float() + bigram[row].float()
+        return x, ref.rms_rows(x * into.sum(), weight, eps, count).to(out_dtype)
+    x = torch.empty((T, H), device=table.device, dtype=torch.float32)
+    h = torch.empty((T, H), device=table.device, dtype=out_dtype)
+    rc = _native.kernels().ft_embed_bigram(
+        batch.tokens.data_ptr(), batch.positions.data_ptr(), batch.starts.data_ptr(), batch.slots.data_ptr(), cache.block_table.data_ptr(),
+        pages.data_ptr(), table.data_ptr(), bigram.data_ptr(), table.stride(0), table.shape[0], buckets, mul_prev, mul_cur, float(scale),
+        into.data_ptr(), into.numel(), weight.data_ptr(), x.data_ptr(), h.data_ptr(), T, H, count, float(eps), int(out_dtype == torch.float32),
+        cache.block_size, cache.max_blocks, cache.num_blocks, F._dev(table), F._stream())
+    _native.check(rc, "ft_embed_bigram")
+    return x, h
+
+
+def softcap_(z: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap * tanh(z / cap)`` on contiguous fp32 logits, in place."""
+    if not z.is_cuda:
+        return z.copy_(cap * torch.tanh(z / cap))
+    rc = _native.kernels().ft_softcap(z.data_ptr(), z.numel(), float(cap), F._dev(z), F._stream())
+    _native.check(rc, "ft_softcap")
+    return z
 
 
 # --------------------------------------------------------------------------- projection -> attention, per head
@@ -110,6 +205,63 @@ def qkv_head_finish(packed: torch.Tensor, cache, layer: int, batch, *, heads: in
         table.shape[1] if table is not None else 0, table.shape[0] if table is not None else 0, float(eps),
         int(packed.dtype == torch.float32), cache.block_size, cache.max_blocks, cache.num_blocks, F._dev(packed), F._stream())
     _native.check(rc, "ft_qkv_head_finish")
+
+
+def latent_finish(packed: torch.Tensor, cache, layer: int, batch, *, heads: int, q_off: int, q_head: int, q_rot: int, c_off: int, rank: int,
+                  rank_pad: int, weight: torch.Tensor, eps: float, table: torch.Tensor, q_lat: torch.Tensor | None = None) -> None:
+    """Everything between a packed projection and its latent attention, in one kernel: RMS norm of the latent (``rank`` of ``rank_pad``
+    elements at ``c_off``, ``weight [rank_pad]``), rotation of the key part behind it and of the part at ``q_rot`` of every query
+    head (heads of ``q_head`` elements from ``q_off``; pairs of neighbours, ``table [positions, half, 2]``), the row into its page.
+    Latent and key part change in place; so do the queries, except that the first rows' rotated parts go to ``q_lat [rows, heads,
+    rank_pad + rot_pad]``, behind the place of their latent part."""
+    width = cache.shapes[layer][1]
+    rot_pad, half = width - rank_pad, table.shape[1]
+    n_lat = q_lat.shape[0] if q_lat is not None else 0
+    cache.sync_table()
+    if not packed.is_cuda:
+        row = packed[:, c_off:c_off + width].float()
+        c = ref.rms_rows(row[:, :rank_pad], weight, eps, rank)
+        row = torch.cat([c, ref.rotate_pairs(row[:, None, rank_pad:], table, batch.positions)[:, 0]], 1).to(packed.dtype)
+        packed[:, c_off:c_off + width] = row
+        pos = batch.positions.long()
+        cache.k[layer][cache._table_host[batch.slots.long(), pos // cache.block_size].long(), pos % cache.block_size, 0] = row
+        q = packed[:, q_off:q_off + heads * q_head].unflatten(1, (heads, q_head))[:, :, q_rot:q_rot + rot_pad]
+        turned = ref.rotate_pairs(q.float(), table, batch.positions).to(packed.dtype)
+        if n_lat:
+            q_lat[:, :, rank_pad:] = turned[:n_lat]
+        q[n_lat:] = turned[n_lat:]
+        return
+    rc = _native.kernels().ft_latent_finish(
+        packed.data_ptr(), packed.stride(0), _ptr(q_lat), n_lat, batch.positions.data_ptr(), batch.slots.data_ptr(), cache.block_table.data_ptr(),
+        cache.k[layer].data_ptr(), weight.data_ptr(), table.data_ptr(), packed.shape[0], heads, q_off, q_head, q_rot, c_off, rank_pad, rank, rot_pad,
+        half, table.shape[0], float(eps), int(packed.dtype == torch.float32), cache.block_size, cache.max_blocks, cache.num_blocks,
+        F._dev(packed), F._stream())
+    _native.check(rc, "ft_latent_finish")
+
+
+def block_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, a_col: int = 0, out_col: int = 0, gate: torch.Tensor | None = None,
+                 glu: str | None = None, bn: int = 0) -> torch.Tensor:
+    """Product by blocks of columns: block g of ``w [blocks, parts, N, K]`` takes columns ``g * a_col ..`` of ``a [T, ..]`` into columns
+    ``g * out_col ..`` of ``out``.  One part: the product, times the sigmoid of ``gate`` (laid out like ``out``) when given; two
+    parts with ``glu`` naming the activation: ``act(gate a) * (up a)``."""
+    G, parts, N, K = w.shape
+    T = a.shape[0]
+    a_col, out_col = a_col or K, out_col or N
+    if parts != (2 if glu else 1):
+        raise ValueError("block_linear: %d parts with activation %r" % (parts, glu))
+    if not a.is_cuda:
+        for g in range(G):
+            z = torch.einsum("tk,pnk->ptn", a[:, g * a_col:g * a_col + K].float(), w[g].float())
+            z = z[0] if not glu else ref._ACTS[F._ACT_ID[glu]](z[0]) * z[1]
+            if gate is not None:
+                z = z * torch.sigmoid(gate[:, g * out_col:g * out_col + N].float())
+            out[:, g * out_col:g * out_col + N] = z.to(out.dtype)
+        return out
+    rc = _native.kernels().ft_block_linear(
+        a.data_ptr(), a.stride(0), T, w.data_ptr(), G, a_col, N, K, int(glu is not None), F._ACT_ID[glu] if glu else 0, out.data_ptr(),
+        out.stride(0), out_col, _ptr(gate), gate.stride(0) if gate is not None else 0, int(a.dtype == torch.float32), bn, F._dev(a), F._stream())
+    _native.check(rc, "ft_block_linear")
+    return out
 
 
 # --------------------------------------------------------------------------- recurrent blocks
@@ -190,11 +342,51 @@ def rglru_scan(a: torch.Tensor, x: torch.Tensor, y: torch.Tensor, out: torch.Ten
     _native.check(rc, "ft_rglru_scan")
 
 
+def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, z: torch.Tensor, i_bias: torch.Tensor,
+                  f_bias: torch.Tensor, norm: torch.Tensor, state, batch, out: torch.Tensor, *, heads: int, dim: int, vdim: int, cap: float,
+                  eps: float, out_scale: float = 1.0) -> torch.Tensor:
+    """Matrix memories over the rows of a ragged batch: ``out = norm(o) * weight * sigmoid(gate) * out_scale`` per head (see
+    ``csrc/matrix_memory.cu``).
+
+    ``q, k [T, heads * dp]``, ``v, gate [T, heads * vp]``: parts of one packed projection (one row stride), heads padded from ``dim``
+    and ``vdim``; ``z [T, 2 * n]`` fp32: pre-activations of the input gates and, from column n, of the forget gates; ``state``: what
+    the sequences' slots hold (:class:`~ferrotorch_b200.nn.recurrent.MatrixMemoryState`)."""
+    T, n_gate = q.shape[0], z.shape[1] // 2
+    if not q.is_cuda:
+        qs, ks = (t.float().unflatten(1, (heads, -1)) for t in (q, k))
+        vs = v.float().unflatten(1, (heads, -1))
+        gi, gf = ref.memory_gates(z[:, :heads] + i_bias, z[:, n_gate:n_gate + heads] + f_bias, cap)
+        for slot, row, start, n in _span_list(batch):
+            if start == 0:
+                for t in (state.S, state.n, state.m):
+                    t[slot].zero_()
+            r = slice(row, row + n)
+            o = ref.matrix_memory(qs[r] * dim ** -0.5, ks[r], vs[r], gi[r], gf[r], state.S[slot], state.n[slot], state.m[slot])
+            o = o / torch.sqrt(o.pow(2).sum(-1, keepdim=True) / vdim + eps)
+            out[r] = (o.flatten(1) * norm * torch.sigmoid(gate[r].float()) * out_scale).to(out.dtype)
+        return out
+    dp, vp = state.S.shape[2:]
+
+    def steps(spans, items):
+        rc = _native.kernels().ft_memory_steps(
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), gate.data_ptr(), q.stride(0), z.data_ptr(), z.stride(0), n_gate, i_bias.data_ptr(),
+            f_bias.data_ptr(), norm.data_ptr(), state.S.data_ptr(), state.n.data_ptr(), state.m.data_ptr(), out.data_ptr(), out.stride(0), heads, dp, vp,
+            vdim, dim ** -0.5, float(cap), float(eps), float(out_scale), _ptr(spans), batch.positions.data_ptr(), batch.slots.data_ptr(), items,
+            int(q.dtype == torch.float32), F._dev(q), F._stream())
+        _native.check(rc, "ft_memory_steps")
+
+    if batch.n_single:
+        steps(None, batch.n_single)
+    if batch.spans:
+        steps(batch.span_table, len(batch.spans))
+    return out
+
+
 # --------------------------------------------------------------------------- expert layers
 @dataclass
 class Routing:
-    """Rows sorted by expert: ``sorted [T * top, H]``, ``place [T, top]`` (where a row's copies lie), ``scale [T * top]``
-    (their weights), ``items`` / ``n_items`` (segments, on the device)."""
+    """Rows sorted by expert: ``sorted [T * top, H]``, ``place [T, top]`` (where a row's copies lie; -1: a choice without
+    matrices), ``scale [T * top]`` (their weights), ``items`` / ``n_items`` (segments, on the device)."""
     index: torch.Tensor
     weight: torch.Tensor
     place: torch.Tensor
@@ -204,19 +396,28 @@ class Routing:
     sorted: torch.Tensor
 
 
+_SCORES = {"sigmoid": 0, "softmax": 1}
 ROUTE_ROWS = 512      # up to so many rows the routing kernel computes the logits itself
 
 
-def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, top: int) -> Routing:
-    """The ``top`` experts of every row of ``h [T, H]`` with the largest logits ``router h`` (fp32), weighted by the sigmoid of
-    the logit, and the rows sorted by expert.  ``router [>= experts, H]`` (padded rows are ignored)."""
+def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, top: int, *, identity: int = 0, score: str = "sigmoid",
+              correction: torch.Tensor | None = None, normalize: bool = False) -> Routing:
+    """The ``top`` choices of every row of ``h [T, H]`` by its logits ``router h`` (fp32), and the rows sorted by expert.
+
+    ``score``: ``sigmoid`` (the largest logits, weighted by their sigmoid) or ``softmax`` over all logits (the largest scores after
+    adding ``correction``, weighted by the score itself; ``normalize``: over the sum of the chosen ones).  The router's first
+    ``experts`` outputs are experts, ``identity`` more have no matrices.  ``router [>= experts + identity, H]`` (padded rows are
+    ignored)."""
     T, H = h.shape
+    outputs = experts + identity
     if not h.is_cuda:
-        index, weight = ref.top_experts(h.float() @ router[:experts].float().t(), top)
+        index, weight = ref.top_experts(h.float() @ router[:outputs].float().t(), top, score, correction, normalize)
         order = index.flatten().argsort(stable=True)
         place = torch.empty_like(order)
         place[order] = torch.arange(order.numel())
-        return Routing(index, weight, place.view(T, top).int(), weight.flatten()[order], index.flatten()[order], torch.tensor(T * top),
+        place[index.flatten() >= experts] = -1
+        real = int((index < experts).sum())
+        return Routing(index, weight, place.view(T, top).int(), weight.flatten()[order], index.flatten()[order][:real], torch.tensor(real),
                        h[order // top])
     lib, dev = _native.kernels(), h.device
     cap = int(lib.ft_moe_max_items(T * top, experts))
@@ -227,17 +428,17 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, top: int) -> 
     rows = torch.empty((T * top, H), device=dev, dtype=h.dtype)
     logits = F.linear_f32_out(h, router) if T > ROUTE_ROWS else None
     rc = lib.ft_moe_route(h.data_ptr(), h.stride(0), router.data_ptr(), _ptr(logits), logits.stride(0) if logits is not None else 0, T, H,
-                          experts, top, int(h.dtype == torch.float32), index.data_ptr(), weight.data_ptr(), place.data_ptr(),
+                          experts, outputs, top, _SCORES[score], _ptr(correction), int(normalize), int(h.dtype == torch.float32), index.data_ptr(), weight.data_ptr(), place.data_ptr(),
                           scale.data_ptr(), items.data_ptr(), cap, n_items.data_ptr(), rows.data_ptr(), F._dev(h), F._stream())
     _native.check(rc, "ft_moe_route")
     return Routing(index, weight.view(T, top), place, scale, items, n_items, rows)
 
 
 def grouped_linear(a: torch.Tensor, w: torch.Tensor, routing: Routing, *, glu: str | None = None, seg_rows: int = 0,
-                   bn: int = 0) -> torch.Tensor:
+                   bn: int = 0, scaled: bool = True) -> torch.Tensor:
     """Rows sorted by expert through their expert's matrix: ``a [R, K]``, ``w [experts, parts, N, K]`` -> ``[R, N]``.  One part: the
     product.  Two parts (gate, up) with ``glu`` naming the activation: ``act(gate r a) * (up r a)`` with r the row's routing
-    weight.  ``seg_rows``: an upper bound of the rows of one expert."""
+    weight (``scaled`` false: 1).  ``seg_rows``: an upper bound of the rows of one expert."""
     E, parts, N, K = w.shape
     R = a.shape[0]
     if parts != (2 if glu else 1):
@@ -245,17 +446,17 @@ def grouped_linear(a: torch.Tensor, w: torch.Tensor, routing: Routing, *, glu: s
     out = torch.empty((R, N), device=a.device, dtype=a.dtype)
     if not a.is_cuda:
         for e in routing.items.unique().tolist():
-            rows = routing.items == e
+            rows = (routing.items == e).nonzero().flatten()
             z = torch.einsum("rk,pnk->prn", a[rows].float(), w[e].float())
             if glu:
-                s = routing.scale[rows][:, None]
+                s = routing.scale[rows][:, None] if scaled else 1.0
                 out[rows] = (ref._ACTS[F._ACT_ID[glu]](s * z[0]) * (s * z[1])).to(out.dtype)
             else:
                 out[rows] = z[0].to(out.dtype)
         return out
     rc = _native.kernels().ft_grouped_gemm(
         a.data_ptr(), a.stride(0), R, w.data_ptr(), routing.items.data_ptr(), routing.n_items.data_ptr(), routing.items.shape[0], E, N, K,
-        int(glu is not None), routing.scale.data_ptr() if glu else None, F._ACT_ID[glu] if glu else 0, out.data_ptr(), out.stride(0),
+        int(glu is not None), routing.scale.data_ptr() if glu and scaled else None, F._ACT_ID[glu] if glu else 0, out.data_ptr(), out.stride(0),
         seg_rows, int(a.dtype == torch.float32), bn, F._dev(a), F._stream())
     _native.check(rc, "ft_grouped_gemm")
     return out

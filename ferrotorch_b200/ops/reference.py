@@ -170,12 +170,47 @@ def linear_recurrence(a: torch.Tensor, x: torch.Tensor, state: torch.Tensor) -> 
     return out
 
 
-def top_experts(logits: torch.Tensor, top: int):
-    """The ``top`` experts of every row with the largest logits (the lower index of equals) and the sigmoid of theirs:
-    ``(index [T, top], weight [T, top])``."""
+def top_experts(logits: torch.Tensor, top: int, score: str = "sigmoid", correction: torch.Tensor | None = None,
+                normalize: bool = False):
+    """The ``top`` experts of every row with the largest scores (the lower index of equals) and their weights: ``(index [T, top],
+    weight [T, top])``.  Scores: the sigmoid of the logit, or the softmax over all logits, to which the choice adds
+    ``correction``; ``normalize``: weights divided by their sum."""
     z = logits.float()
-    index = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, :top]
-    return index, torch.sigmoid(z.gather(1, index))
+    s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, -1)
+    choice = (z if score == "sigmoid" else s) if correction is None else s + correction.float()
+    index = torch.sort(choice, dim=-1, descending=True, stable=True).indices[:, :top]
+    w = s.gather(1, index)
+    return index, w / (w.sum(-1, keepdim=True) + 1e-20) if normalize else w
+
+
+def rotate_pairs(x: torch.Tensor, table: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
+    """Rotate the first ``2 * half`` elements of ``x [T, H, D]`` (pairs ``2i, 2i + 1``) by the rows ``table[position] [half, 2]``."""
+    half = table.shape[1]
+    c, s = table[positions.long()].unsqueeze(1).unbind(-1)
+    u, v = x[..., 0:2 * half:2], x[..., 1:2 * half:2]
+    return torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., 2 * half:]], -1)
+
+
+def memory_gates(zi: torch.Tensor, zf: torch.Tensor, cap: float):
+    """Logarithmic input and forget gate of a matrix memory from their pre-activations, fp32."""
+    return cap * torch.tanh(zi / cap), F.logsigmoid(cap * torch.tanh(zf / cap))
+
+
+def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Tensor, f: torch.Tensor, S: torch.Tensor,
+                  n: torch.Tensor, m: torch.Tensor) -> torch.Tensor:
+    """The recurrence of a matrix memory over rows ``q, k [T, H, D]``, ``v [T, H, V]`` with log gates ``i, f [T, H]``, from (and
+    into) ``S [H, D, V]``, ``n [H, D]``, ``m [H]``: outputs ``[T, H, V]``, fp32."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        new = torch.maximum(f[t] + m, i[t])
+        keep, add = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+        ka = add[:, None] * k[t]
+        S.mul_(keep[:, None, None]).add_(ka[:, :, None] * v[t][:, None, :])
+        n.mul_(keep[:, None]).add_(ka)
+        m.copy_(new)
+        den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        out[t] = torch.einsum("hdv,hd->hv", S, q[t]) / den[:, None]
+    return out
 
 
 def swiglu(gu: torch.Tensor, act: int = 0) -> torch.Tensor:
@@ -203,13 +238,14 @@ def repeat_kv(x: torch.Tensor, n_rep: int) -> torch.Tensor:
 
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = True,
               scale: float | None = None, q_offset: int | None = None, window: int | None = None,
-              sink: torch.Tensor | None = None):
+              sink: torch.Tensor | None = None, chunk: int | None = None, slopes: torch.Tensor | None = None):
     """GQA attention on ``[B, S, H, D]`` tensors, returns ``(out [B,Sq,Hq,D], lse [B,Hq,Sq])``.
 
     Scores scaled by ``1/sqrt(D)``, causal mask hides ``j > i + q_offset`` where the default
     offset aligns the last query with the last key (for Sq == Sk this is the reference's
     top-left mask, ferrotorch-nn/src/flash_attention.rs:647-746), max-subtracted softmax.  With ``window`` a query
-    sees only its last so many keys; with ``sink [Hq]`` a head's denominator gains ``exp(sink)``."""
+    sees only its last so many keys, with ``chunk`` those of its own chunk of so many positions; ``slopes [Hq]`` times the
+    distance of a key is taken off its score; with ``sink [Hq]`` a head's denominator gains ``exp(sink)``."""
     B, Sq, Hq, D = q.shape
     Sk, Hkv = k.shape[1], k.shape[2]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -221,7 +257,11 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = 
         off = (Sk - Sq) if q_offset is None else q_offset
         i = torch.arange(Sq, device=q.device)[:, None] + off
         j = torch.arange(Sk, device=q.device)[None, :]
+        if slopes is not None:
+            s = s - slopes.float().view(1, Hq, 1, 1) * (i - j).float()
         s = s.masked_fill(j > i, float("-inf"))
+        if chunk:
+            s = s.masked_fill(j < i // chunk * chunk, float("-inf"))
         if window:
             s = s.masked_fill(i - j >= window, float("-inf"))
     lse = torch.logsumexp(s, dim=-1)

@@ -289,6 +289,8 @@ class PagedKVCache:
         """Write ``k_new / v_new [T, Hkv, D]`` at ``positions [T]`` (int32).  Token i belongs to
         sequence ``seq_ids[i]`` or ``i // tokens_per_seq``.  Pages must have been reserved."""
         T = k_new.shape[0]
+        if self.values_in_keys[layer]:
+            raise ValueError("PagedKVCache.append: layer %d has no values of its own" % layer)
         table = self.sync_table()
         Hkv, D, Dv = self.shapes[layer]
         if not k_new.is_cuda:

@@ -4,6 +4,20 @@
 //   ft_latent_finish   everything between the packed projection [ q heads | latent | rotated key part | .. ] and the
 //                      attention: RMS norm of the latent, rotation of the key part and of every head's rotated
 //                      query part (neighbouring elements are pairs), the row into its cache page
+//   ft_latent_decode   one query token per row, queries already in the latent space: all heads of a row attend to the cached
+//                      rows themselves, o = softmax(scale * q . row) row[0 .. rank), split over the context (bf16)
+//   ft_latent_gather   the cached rows of portions' contexts, contiguous: the operand from which the keys and values of
+//                      a prompt portion are formed
+//
+// Decoding reads every cached row once for up to 32 heads.  A CTA owns (context split, group of heads, row) and walks the keys in
+// tiles of 128, the layout of paged_decode_tc_kernel (paged_attn.cu) with the values inside the keys:
+//     S^T[key, head]  = sum over 64-column pieces of the tile  (M = 128 keys, N = heads)
+//     O^T[d, head]   += tile[:, d]^T P^T                       (one MMA chain per 128 latent columns)
+// A tile of 576 columns takes 144 KB, so there is one; its pieces are ring slots of their own: a piece is loaded again as soon as
+// the last product that reads it has finished, while the others are still in use.
+//   warp 0  producer: one TMA box per page and piece     warp 1  MMA issuer     warp 2  TMEM allocator
+//   warps 4-7  softmax (thread = key) and epilogue (thread = latent column)
+// All waits are bounded and report through the device status word.
 #include <initializer_list>
 
 #include "row_vec.cuh"
@@ -93,6 +107,336 @@ latent_finish_kernel(const LatentFinishParams p) {
   }
 }
 
+// ---------------------------------------------------------------- decode
+constexpr int LD_THREADS = 256;
+constexpr int LD_TILE = 128;               // keys
+constexpr int LD_PIECE = LD_TILE * 128;    // bytes of 64 columns
+constexpr int LD_MAX_PIECES = 9;
+constexpr float LD_RESCALE = 8.f;
+
+template <int N>
+struct LdCfg {
+  static constexpr int Q_PIECE = N * 128;
+  static constexpr int P_BYTES = 2 * N * 128;             // two pieces of 64 keys
+  static constexpr int OFF_Q = LD_MAX_PIECES * LD_PIECE;
+  static constexpr int OFF_P = OFF_Q + LD_MAX_PIECES * Q_PIECE;
+  static constexpr int OFF_RED = OFF_P + P_BYTES;         // [4 warps][N] floats, then [N] references
+  static constexpr int OFF_BAR = OFF_RED + 5 * N * 4;
+  static constexpr int SMEM_BYTES = OFF_BAR + 256 + 1024;
+  static constexpr uint32_t TMEM_COLS = N * 5 <= 128 ? 128 : 256;
+};
+
+struct LatentDecodeParams {
+  const __nv_bfloat16* q;    // [B, H, width]
+  const int* block_table;
+  const int* row_slot;
+  const int* ctx_len;
+  __nv_bfloat16* out;        // [B, H, rank] (row stride ldo)
+  float* part_o;
+  float* part_ml;
+  long long ldo;
+  int H, width, rank, pieces, v_pieces;      // v_pieces: 64-column pieces that the value products read (even)
+  int block_size, rows_per_box, boxes, max_blocks, num_blocks, n_splits;
+  float scale_log2;
+  int* status;
+};
+
+template <int N>
+__global__ void __launch_bounds__(LD_THREADS, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecodeParams p) {
+  using Cfg = LdCfg<N>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const uint32_t sbase = smem_u32(smem);
+  float* s_red = reinterpret_cast<float*>(smem + Cfg::OFF_RED);
+  float* s_ref = s_red + 4 * N;
+  enum { FULL = 0, EMPTY = FULL + LD_MAX_PIECES, S_FULL = EMPTY + LD_MAX_PIECES, P_FULL, O_DONE, NBARS };
+  const uint32_t bar0 = sbase + Cfg::OFF_BAR;
+  auto bar = [&](int i) { return bar0 + 8u * i; };
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + Cfg::OFF_BAR + 8 * NBARS);
+  volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  const int split = blockIdx.x, h0 = blockIdx.y * N, b = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int heads = min(N, p.H - h0);
+  const int len = min(p.ctx_len[b], p.max_blocks * p.block_size);
+  const int tiles = (len + LD_TILE - 1) / LD_TILE, per_split = (tiles + p.n_splits - 1) / p.n_splits;
+  const int tile_lo = split * per_split, n_tiles = max(0, min(tiles, tile_lo + per_split) - tile_lo);
+  const int blocks = p.v_pieces / 2;         // 128-column blocks of the latent
+
+  if (threadIdx.x == 0) {
+    *abort_word = 0;
+    for (int i = 0; i < LD_MAX_PIECES; ++i) {
+      mbar_init(bar(FULL + i), 1);
+      mbar_init(bar(EMPTY + i), 1);
+    }
+    mbar_init(bar(S_FULL), 1);
+    mbar_init(bar(P_FULL), 4);
+    mbar_init(bar(O_DONE), 1);
+    fence_mbar_init();
+    tma_prefetch_desc(&tmC);
+  }
+  if (warp == 2) {
+    tmem_alloc(smem_u32(tmem_slot), Cfg::TMEM_COLS);
+    tmem_relinquish();
+  }
+  // the queries as the B operand (rows past the heads and columns past the width zero)
+  for (int i = threadIdx.x; i < N * LD_MAX_PIECES * 8; i += LD_THREADS) {
+    const int h = i / (LD_MAX_PIECES * 8), u = i - h * (LD_MAX_PIECES * 8);
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (h < heads && u * 8 < p.width) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(b) * p.H + h0 + h) * p.width + u * 8);
+    *reinterpret_cast<uint4*>(smem + Cfg::OFF_Q + (u >> 3) * Cfg::Q_PIECE + h * 128 + (((u & 7) ^ (h & 7)) << 4)) = v;
+  }
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  const uint32_t COL_S = 0, COL_O = N;       // O^T of block i at COL_O + i * N
+
+  if (warp == 0) {
+    // ------------------------------------------------------------------ producer (whole warp)
+    const int* bt = p.block_table + static_cast<long long>(p.row_slot ? p.row_slot[b] : b) * p.max_blocks;
+    bool ok = true;
+    for (int t = 0; t < n_tiles && ok; ++t) {
+      const int key = (tile_lo + t) * LD_TILE + lane * p.rows_per_box;     // rows past the context: finite values of other tokens
+      const int page = min(key / p.block_size, p.max_blocks - 1);
+      const int blk = min(max(lane < p.boxes ? __ldg(bt + page) : 0, 0), p.num_blocks - 1);
+      const int row = blk * p.block_size + key % p.block_size;
+      for (int c = 0; c < p.pieces; ++c) {
+        ok = mbar_wait(bar(EMPTY + c), (t & 1) ^ 1u, abort_word, FT_ERR_TIMEOUT_PRODUCER);
+        if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+        if (lane == 0) mbar_expect_tx(bar(FULL + c), LD_PIECE);
+        __syncwarp();
+        if (lane < p.boxes) tma_load_2d(sbase + c * LD_PIECE + lane * p.rows_per_box * 128, &tmC, bar(FULL + c), c * 64, row);
+      }
+    }
+    if (*abort_word) {   // let copies in flight land before the CTA leaves
+      const unsigned long long t0 = globaltimer_ns();
+      while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = make_idesc_f16(LD_TILE, N, 1, 0, 0);
+      constexpr uint32_t idesc_o = make_idesc_f16(128, N, 1, 1, 0);
+      bool ok = true;
+      for (int t = 0; t < n_tiles && ok; ++t) {
+        for (int c = 0; c < p.pieces; ++c) {
+          ok = mbar_wait(bar(FULL + c), t & 1, abort_word, FT_ERR_TIMEOUT_MMA);
+          if (!ok) break;
+          tc_fence_after();
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk)
+            umma_f16_ss(tmem + COL_S, make_smem_desc_sw128(sbase + c * LD_PIECE + kk * 32, 16, 1024),
+                        make_smem_desc_sw128(sbase + Cfg::OFF_Q + c * Cfg::Q_PIECE + kk * 32, 16, 1024), idesc_s, (c > 0 || kk > 0) ? 1u : 0u);
+          if (c >= p.v_pieces) umma_commit(bar(EMPTY + c));
+        }
+        if (!ok) break;
+        umma_commit(bar(S_FULL));
+        ok = mbar_wait(bar(P_FULL), t & 1, abort_word, FT_ERR_TIMEOUT_MMA);
+        if (!ok) break;
+        tc_fence_after();
+        for (int i = 0; i < blocks; ++i) {
+#pragma unroll
+          for (int kk = 0; kk < LD_TILE / 16; ++kk)
+            umma_f16_ss(tmem + COL_O + i * N, make_smem_desc_sw128(sbase + 2 * i * LD_PIECE + kk * 2048, LD_PIECE, 1024),
+                        make_smem_desc_sw128(sbase + Cfg::OFF_P + (kk >> 2) * Cfg::Q_PIECE + (kk & 3) * 32, 16, 1024), idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
+          umma_commit(bar(EMPTY + 2 * i));
+          umma_commit(bar(EMPTY + 2 * i + 1));
+        }
+        umma_commit(bar(O_DONE));
+      }
+    }
+  } else if (warp >= 4) {
+    // ------------------------------------------------------------------ softmax / epilogue
+    const int ew = warp & 3, r = ew * 32 + lane;
+    const uint32_t lane_addr = tmem + (static_cast<uint32_t>(ew * 32) << 16);
+    float l_part[N];
+#pragma unroll
+    for (int g = 0; g < N; ++g) l_part[g] = 0.f;
+    if (r < N) s_ref[r] = -INFINITY;
+    bool ok = true;
+    // every thread runs every iteration down to the named barriers, also after a failed wait
+    for (int t = 0; t < n_tiles; ++t) {
+      if (ok && !mbar_wait(bar(S_FULL), t & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) ok = false;
+      ok = __all_sync(0xffffffffu, ok);
+      float s[N];
+      {
+        uint32_t raw[N];
+#pragma unroll
+        for (int g = 0; g < N; ++g) raw[g] = 0u;
+        if (ok) {
+          tc_fence_after();
+#pragma unroll
+          for (int g = 0; g < N; g += 16) tmem_ld_32x16(lane_addr + COL_S + g, *reinterpret_cast<uint32_t(*)[16]>(&raw[g]));
+          tmem_ld_wait();
+        }
+        const bool valid = (tile_lo + t) * LD_TILE + r < len;
+#pragma unroll
+        for (int g = 0; g < N; ++g) s[g] = valid ? __uint_as_float(raw[g]) * p.scale_log2 : -INFINITY;
+      }
+      // maxima over the warp's keys: halve the heads a lane holds while doubling the keys it covers; lane g ends with head g
+      {
+        float v[N];
+#pragma unroll
+        for (int g = 0; g < N; ++g) v[g] = s[g];
+#pragma unroll
+        for (int w = N / 2; w >= 1; w >>= 1) {
+          const bool upper = lane & w;
+#pragma unroll
+          for (int g = 0; g < w; ++g) {
+            const float send = upper ? v[g] : v[g + w], keep = upper ? v[g + w] : v[g];
+            v[g] = fmaxf(keep, __shfl_xor_sync(0xffffffffu, send, w));
+          }
+        }
+        if (N == 16) v[0] = fmaxf(v[0], __shfl_xor_sync(0xffffffffu, v[0], 16));
+        if (lane < N) s_red[ew * N + lane] = v[0];
+      }
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+      // every thread makes the same decision; the references are replaced after all have read them
+      const float tile_max = lane < N ? fmaxf(fmaxf(s_red[lane], s_red[N + lane]), fmaxf(s_red[2 * N + lane], s_red[3 * N + lane])) : -INFINITY;
+      const float old_ref = lane < N ? s_ref[lane] : 0.f;
+      const bool moves = lane < N && tile_max > old_ref + LD_RESCALE;
+      const float my_ref = moves ? tile_max : old_ref, my_alpha = moves ? fast_exp2(old_ref - tile_max) : 1.f;   // first tile: 0
+      const bool any = __any_sync(0xffffffffu, moves);
+      // O of the earlier tiles and the P buffer are free once the products of tile t - 1 have finished
+      if (t > 0 && ok && !mbar_wait(bar(O_DONE), (t - 1) & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) ok = false;
+      ok = __all_sync(0xffffffffu, ok);
+      if (any) {
+        float alpha[N];
+#pragma unroll
+        for (int g = 0; g < N; ++g) {
+          alpha[g] = __shfl_sync(0xffffffffu, my_alpha, g);
+          l_part[g] *= alpha[g];
+        }
+        if (t > 0 && ok) {
+          tc_fence_after();
+          for (int i = 0; i < blocks; ++i)
+#pragma unroll
+            for (int g0 = 0; g0 < N; g0 += 16) {
+              uint32_t ov[16];
+              tmem_ld_32x16(lane_addr + COL_O + i * N + g0, ov);
+              tmem_ld_wait();
+#pragma unroll
+              for (int g = 0; g < 16; ++g) ov[g] = __float_as_uint(__uint_as_float(ov[g]) * alpha[g0 + g]);
+              tmem_st_32x16(lane_addr + COL_O + i * N + g0, ov);
+            }
+          tmem_st_wait();
+        }
+      }
+      {
+        uint8_t* pb = smem + Cfg::OFF_P + (r >> 6) * Cfg::Q_PIECE;
+        const int kc = r & 63;
+#pragma unroll
+        for (int g = 0; g < N; ++g) {
+          const float ref = __shfl_sync(0xffffffffu, my_ref, g);
+          const float pv = s[g] == -INFINITY ? 0.f : fast_exp2(s[g] - ref);
+          const __nv_bfloat16 pb16 = __float2bfloat16(pv);
+          l_part[g] += __bfloat162float(pb16);     // the sum of what the MMA will actually use
+          *reinterpret_cast<__nv_bfloat16*>(pb + g * 128 + (((kc >> 3) ^ (g & 7)) << 4) + (kc & 7) * 2) = pb16;
+        }
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      __syncwarp();
+      if (ok && lane == 0) mbar_arrive(bar(P_FULL));
+      asm volatile("bar.sync 1, 128;" ::: "memory");      // s_red and the old references have been read by all
+      if (ew == 0 && lane < N) s_ref[lane] = my_ref;
+    }
+    if (ok && n_tiles > 0) ok = mbar_wait(bar(O_DONE), (n_tiles - 1) & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE);
+    ok = __all_sync(0xffffffffu, ok);
+    tc_fence_after();
+#pragma unroll
+    for (int g = 0; g < N; ++g) {
+      const float ws = warp_sum(l_part[g]);
+      if (lane == 0) s_red[ew * N + g] = ws;
+    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    if (ok)
+      for (int i = 0; i < blocks; ++i)
+#pragma unroll
+        for (int g0 = 0; g0 < N; g0 += 16) {
+          uint32_t ov[16];
+#pragma unroll
+          for (int g = 0; g < 16; ++g) ov[g] = 0u;
+          if (n_tiles > 0) {
+            tmem_ld_32x16(lane_addr + COL_O + i * N + g0, ov);
+            tmem_ld_wait();
+          }
+          const int d = i * 128 + r;
+#pragma unroll
+          for (int g = 0; g < 16; ++g) {
+            const int h = g0 + g;
+            if (h >= heads || d >= p.rank) continue;
+            const float l = s_red[h] + s_red[N + h] + s_red[2 * N + h] + s_red[3 * N + h], o = __uint_as_float(ov[g]);
+            if (p.n_splits == 1) {
+              p.out[b * p.ldo + static_cast<long long>(h0 + h) * p.rank + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+            } else {
+              const long long at = (static_cast<long long>(b) * p.H + h0 + h) * p.n_splits + split;
+              p.part_o[at * p.rank + d] = o;
+              if (d == 0) { p.part_ml[at * 2] = s_ref[h]; p.part_ml[at * 2 + 1] = l; }
+            }
+          }
+        }
+  }
+
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 2) {
+    tc_fence_after();
+    tmem_dealloc(tmem, Cfg::TMEM_COLS);
+  }
+  if (threadIdx.x == 0 && *abort_word != 0 && p.status) atomicCAS(p.status, 0, *abort_word);
+}
+
+// One block per (head, row): the splits' factors once, then their rows in vectors of four.
+constexpr int LC_MAX_SPLITS = 32;
+__global__ void __launch_bounds__(128)
+latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out, int H, int rank,
+                      long long ldo, int n_splits) {
+  __shared__ float s_f[LC_MAX_SPLITS];
+  const int h = blockIdx.x, b = blockIdx.y;
+  const long long base = (static_cast<long long>(b) * H + h) * n_splits;
+  if (threadIdx.x < 32) {
+    const int s = threadIdx.x;
+    const float m = s < n_splits ? part_ml[(base + s) * 2] : -INFINITY;
+    const float mm = warp_max(m);
+    const float f = m == -INFINITY ? 0.f : fast_exp2(m - mm);
+    const float l = warp_sum(s < n_splits ? part_ml[(base + s) * 2 + 1] * f : 0.f);
+    s_f[s] = l > 0.f ? f / l : 0.f;
+  }
+  __syncthreads();
+  for (int d = threadIdx.x * 4; d < rank; d += 512) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < n_splits; ++s) {
+      const float f = s_f[s];
+      if (f == 0.f) continue;                      // a split without keys left its partial result unwritten or zero
+      const float4 o = *reinterpret_cast<const float4*>(part_o + (base + s) * rank + d);
+      acc.x += f * o.x; acc.y += f * o.y; acc.z += f * o.z; acc.w += f * o.w;
+    }
+    *reinterpret_cast<uint2*>(out + b * ldo + static_cast<long long>(h) * rank + d) = make_uint2(pack_bf16x2(acc.x, acc.y), pack_bf16x2(acc.z, acc.w));
+  }
+}
+
+// out[first + i] = cached row of token i of sequence slot, i < n, for every (slot, first, n) of `spans`; zeros up to the next
+// multiple of `pad` rows.
+__global__ void latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table, const int* __restrict__ spans,
+                                     uint4* __restrict__ out, int units, int pad, int block_size, int max_blocks, int num_blocks) {
+  const int* span = spans + 3 * blockIdx.y;
+  const int slot = span[0], first = span[1], n = span[2];
+  for (int i = blockIdx.x * blockDim.y + threadIdx.y; i < (n + pad - 1) / pad * pad; i += gridDim.x * blockDim.y) {
+    if (i >= n) {
+      for (int u = threadIdx.x; u < units; u += blockDim.x) out[(static_cast<long long>(first) + i) * units + u] = make_uint4(0u, 0u, 0u, 0u);
+      continue;
+    }
+    const int page = i / block_size;
+    int blk = page < max_blocks ? __ldg(block_table + static_cast<long long>(slot) * max_blocks + page) : 0;
+    blk = min(max(blk, 0), num_blocks - 1);
+    const uint4* src = cache + (static_cast<long long>(blk) * block_size + i % block_size) * units;
+    for (int u = threadIdx.x; u < units; u += blockDim.x) out[(static_cast<long long>(first) + i) * units + u] = src[u];
+  }
+}
+
 static bool la_aligned(std::initializer_list<const void*> ps) {
   uintptr_t v = 0;
   for (const void* p : ps) v |= reinterpret_cast<uintptr_t>(p);
@@ -129,6 +473,77 @@ FT_API int ft_latent_finish(void* packed, long long ld, void* q_lat, int n_lat, 
   const int cap = sm_count(device) * 16, grid = rows < cap ? rows : cap;
   if (f32) latent_finish_kernel<float><<<grid, LF_THREADS, 0, stream>>>(p);
   else latent_finish_kernel<__nv_bfloat16><<<grid, LF_THREADS, 0, stream>>>(p);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// Decode attention over latent rows (see the top of this file): q [B, H, width] bf16, cache [num_blocks, block_size, width], out
+// [B, H, rank] (row stride ldo), width and rank multiples of 16, width up to 576 and rank up to 512.  Row b reads its first
+// ctx_len[b] tokens of sequence row_slot[b] (null: b).  scratch: B * H * n_splits * (rank + 2) floats when n_splits > 1.  Page
+// sizes: a divisor of 128 of at least 8, or a multiple of 128.
+FT_API int ft_latent_decode(const void* q, const void* cache, const int* block_table, const int* row_slot, const int* ctx_len, void* out,
+                            float* scratch, int B, int H, int width, int rank, long long ldo, int block_size, int max_blocks,
+                            int num_blocks, float scale, int n_splits, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(q && cache && block_table && ctx_len && out, "ft_latent_decode: null pointer");
+  FT_REQUIRE(H > 0 && width >= 16 && width % 16 == 0 && width <= LD_MAX_PIECES * 64 && rank >= 16 && rank % 16 == 0 && rank <= width && rank <= 512,
+             "ft_latent_decode: rows of %d with a latent of %d", width, rank);
+  FT_REQUIRE(block_size >= 8 && (LD_TILE % block_size == 0 || block_size % LD_TILE == 0) && max_blocks > 0 && num_blocks > 0 &&
+                 static_cast<long long>(num_blocks) * block_size < (1ll << 31), "ft_latent_decode: page size %d", block_size);
+  FT_REQUIRE(n_splits >= 1 && n_splits <= LC_MAX_SPLITS && (n_splits == 1 || scratch), "ft_latent_decode: %d splits", n_splits);
+  FT_REQUIRE(la_aligned({q, cache, out, scratch}) && ldo % 8 == 0 && ldo >= static_cast<long long>(H) * rank, "ft_latent_decode: pointers must be 16-byte aligned");
+  if (B <= 0) return FT_E_OK;
+  FT_REQUIRE(B < 65536, "ft_latent_decode: %d rows", B);
+  LatentDecodeParams p;
+  p.q = static_cast<const __nv_bfloat16*>(q); p.block_table = block_table; p.row_slot = row_slot; p.ctx_len = ctx_len;
+  p.out = static_cast<__nv_bfloat16*>(out); p.part_o = scratch;
+  p.part_ml = scratch ? scratch + static_cast<long long>(B) * H * n_splits * rank : nullptr;
+  p.ldo = ldo; p.H = H; p.width = width; p.rank = rank; p.v_pieces = 2 * ((rank + 127) / 128);
+  p.pieces = (width + 63) / 64;
+  if (p.pieces < p.v_pieces) p.pieces = p.v_pieces;          // a piece past the row: zeros
+  p.block_size = block_size; p.rows_per_box = block_size < LD_TILE ? block_size : LD_TILE; p.boxes = LD_TILE / p.rows_per_box;
+  p.max_blocks = max_blocks; p.num_blocks = num_blocks; p.n_splits = n_splits;
+  p.scale_log2 = scale * 1.4426950408889634f; p.status = device_status_word(device);
+  CUtensorMap tc;
+  if (int rc = make_tmap_2d(&tc, cache, 2, width, static_cast<uint64_t>(num_blocks) * block_size, static_cast<uint64_t>(width) * 2, 64, p.rows_per_box, 3))
+    return rc;
+  const int N = H <= 16 ? 16 : 32;
+  const dim3 grid(n_splits, (H + N - 1) / N, B);
+#define FT_LD(NN)                                                                                                                   \
+  {                                                                                                                                 \
+    static bool attr_set[64] = {false};                                                                                             \
+    if (!attr_set[device]) {                                                                                                        \
+      FT_CUDA_CHECK(cudaFuncSetAttribute(latent_decode_kernel<NN>, cudaFuncAttributeMaxDynamicSharedMemorySize, LdCfg<NN>::SMEM_BYTES)); \
+      attr_set[device] = true;                                                                                                      \
+    }                                                                                                                               \
+    latent_decode_kernel<NN><<<grid, LD_THREADS, LdCfg<NN>::SMEM_BYTES, stream>>>(tc, p);                                           \
+  }
+  if (N == 16) FT_LD(16) else FT_LD(32)
+#undef FT_LD
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  if (n_splits > 1) {
+    latent_combine_kernel<<<dim3(H, B), 128, 0, stream>>>(p.part_o, p.part_ml, p.out, H, rank, ldo, n_splits);
+    FT_CUDA_CHECK(cudaGetLastError());
+    count_launch();
+  }
+  return FT_E_OK;
+}
+
+// The cached rows of contexts, contiguous: spans int32 [n_spans, 3] (sequence slot, first row of out, tokens), rows of
+// row_bytes (a multiple of 16); every span is filled up with zero rows to a multiple of `pad`.  longest: most tokens of a span.
+FT_API int ft_latent_gather(const void* cache, const int* block_table, const int* spans, int n_spans, int longest, void* out, int row_bytes,
+                            int pad, int block_size, int max_blocks, int num_blocks, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(cache && block_table && spans && out && row_bytes > 0 && row_bytes % 16 == 0 && pad > 0 && la_aligned({cache, out}), "ft_latent_gather: null or unaligned pointer");
+  FT_REQUIRE(block_size > 0 && max_blocks > 0 && num_blocks > 0 && n_spans < 65536, "ft_latent_gather: bad shape");
+  if (n_spans <= 0 || longest <= 0) return FT_E_OK;
+  int gx = (longest + 3) / 4;
+  const int cap = sm_count(device) * 16 / n_spans + 1;
+  if (gx > cap) gx = cap;
+  latent_gather_kernel<<<dim3(gx, n_spans), dim3(64, 4), 0, stream>>>(static_cast<const uint4*>(cache), block_table, spans,
+                                                                      static_cast<uint4*>(out), row_bytes / 16, pad, block_size, max_blocks, num_blocks);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

@@ -9,6 +9,20 @@
 // and all arithmetic of the recurrence are fp32; q, k, v and the output gate come from a packed projection.
 //
 //   ft_memory_steps   token by token: rows that are their sequence's only token, short portions, any sizes, bf16 or fp32
+//   ft_memory_chunks  whole portions in chunks of 128 tokens on tcgen05 / TMEM (bf16, dim up to 128, vdim up to 256)
+//
+// Chunks.  Let b_t be the sum of f over a chunk's tokens up to t, a_t = i_t - b_t, M the maximum before the chunk and x_t =
+// max(M, a_1 .. a_t).  Then m_t = b_t + x_t and
+//   S_t = e^(M - x_t) S + sum_(s <= t) e^(a_s - x_t) k_s v_s^T,
+// so a chunk's outputs are a causal product of scores like attention's plus q times the state at its start, and its
+// contribution to the next state is one product over its tokens, independent of all other chunks.  Four passes:
+//   memory_gates_kernel   a, x, e^-m of every token and M of every chunk (fp32; a warp scans a chunk)
+//   memory_update_kernel  U = sum_s e^(a_s - x_end) k_s v_s^T of every (chunk, head): tcgen05 product with the weighted keys
+//                         as high and low bf16 halves, so that the state keeps about 16 bits more than its operands
+//   memory_carry_kernel   S' = e^(M - x_end) S + U over the chunks of a portion, element by element in fp32; leaves every
+//                         chunk's starting state in bf16 and the final one in the slot
+//   memory_output_kernel  P = causal e^(a_s - x_t) q.k and e^(M - x_t) q written over the scores in TMEM as operands of
+//                         one accumulator, O = P V + (..q) S; denominator, norm, gate and store
 //
 // A slot needs no clearing: what a sequence has seen follows from its positions, and position 0 starts from zero.
 #include <initializer_list>
@@ -162,6 +176,486 @@ memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
     for (int i = tid * 4; i < p.dp * p.vp; i += MS_THREADS * 4) *reinterpret_cast<float4*>(S_mem + i) = *reinterpret_cast<const float4*>(s_state + i);
 }
 
+// ---------------------------------------------------------------- chunks
+constexpr int MC_ROWS = 128;      // tokens of a chunk
+constexpr int MC_CHUNK = MC_ROWS * 128;          // bytes of a 64-column tile of 128 rows
+constexpr int MC_GATE_WARPS = 32;
+constexpr int MC_UPDATE_THREADS = 256;
+constexpr int MC_OUT_THREADS = 128;
+
+struct MemoryChunks {
+  const int* spans;         // [n_spans, 4]: slot, first row, first position, rows
+  const int* span_chunks;   // [n_spans]: first chunk
+  const int* chunks;        // [n_chunks, 4]: span, first row, rows, number within the portion
+  float* a2;                // [H, ldt] fp32, in powers of two: a_t
+  float* x2;                // x_t
+  float* floor;             // e^-m_t
+  float* start2;            // [n_chunks, H]: M
+  float* end2;              // [n_chunks, H]: x of the last token
+  float* U;                 // [n_chunks, H, dp, vw]
+  float* Un;                // [n_chunks, H, dp]
+  __nv_bfloat16* Sb;        // [n_chunks, H, dp, vw]: states at the chunks' starts
+  float* nb;                // [n_chunks, H, dp]
+  long long ldt;
+  int n_spans, n_chunks, vw;      // vw: vp rounded up to 64
+  int* status;
+};
+
+// One block per (head, portion), a warp per chunk, up to MC_GATE_WARPS chunks at a time.
+__global__ void __launch_bounds__(MC_GATE_WARPS * 32)
+memory_gates_kernel(const MemoryParams p, const MemoryChunks c) {
+  __shared__ float s_sum[MC_GATE_WARPS], s_max[MC_GATE_WARPS], s_start[MC_GATE_WARPS];
+  __shared__ float s_carry;
+  const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int* span = c.spans + 4 * blockIdx.y;
+  const int slot = span[0], row0 = span[1], pos0 = span[2], rows = span[3];
+  const int n_chunks = (rows + MC_ROWS - 1) / MC_ROWS, first = c.span_chunks[blockIdx.y];
+  float* m_slot = p.m + static_cast<long long>(slot) * p.H + h;
+  const float bi = p.i_bias[h], bf = p.f_bias[h];
+  if (threadIdx.x == 0) s_carry = pos0 == 0 ? 0.f : *m_slot;
+  for (int base = 0; base < n_chunks; base += MC_GATE_WARPS) {
+    const int k = base + warp, t0 = k * MC_ROWS + lane * 4;
+    float b[4], a[4], x[4];
+    float sum = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float f = 0.f;
+      a[e] = -INFINITY;
+      if (k < n_chunks && t0 + e < rows) {
+        const float* z = p.z + (static_cast<long long>(row0) + t0 + e) * p.ldz;
+        f = mem_forget_gate(z[p.f_off + h] + bf, p.cap);
+        a[e] = mem_input_gate(z[h] + bi, p.cap);
+      }
+      sum += f;
+      b[e] = sum;
+    }
+    float before = sum;                                // sums of the lanes ahead
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, before, o);
+      if (lane >= o) before += v;
+    }
+    const float total = __shfl_sync(0xffffffffu, before, 31);
+    before = __shfl_up_sync(0xffffffffu, before, 1);
+    if (lane == 0) before = 0.f;
+    float mx = -INFINITY;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      b[e] += before;
+      a[e] -= b[e];
+      mx = fmaxf(mx, a[e]);
+      x[e] = mx;
+    }
+    float ahead = mx;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, ahead, o);
+      if (lane >= o) ahead = fmaxf(ahead, v);
+    }
+    const float top = __shfl_sync(0xffffffffu, ahead, 31);
+    ahead = __shfl_up_sync(0xffffffffu, ahead, 1);
+    if (lane == 0) ahead = -INFINITY;
+    if (lane == 0) { s_sum[warp] = total; s_max[warp] = top; }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+      float m = s_carry;
+      for (int w = 0; w < MC_GATE_WARPS && base + w < n_chunks; ++w) {
+        s_start[w] = m;
+        m = s_sum[w] + fmaxf(m, s_max[w]);
+      }
+      s_carry = m;
+    }
+    __syncthreads();
+    if (k < n_chunks) {
+      const float start = s_start[warp];
+      const long long at = static_cast<long long>(h) * c.ldt + row0 + t0;
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (t0 + e < rows) {
+          const float xe = fmaxf(start, fmaxf(ahead, x[e]));
+          c.a2[at + e] = a[e] * 1.4426950408889634f;
+          c.x2[at + e] = xe * 1.4426950408889634f;
+          c.floor[at + e] = expf(-(b[e] + xe));
+        }
+      if (lane == 0) {
+        c.start2[static_cast<long long>(first + k) * p.H + h] = start * 1.4426950408889634f;
+        c.end2[static_cast<long long>(first + k) * p.H + h] = fmaxf(start, top) * 1.4426950408889634f;
+      }
+    }
+    __syncthreads();                                   // s_start has been read
+  }
+  if (threadIdx.x == 0) *m_slot = s_carry;
+}
+
+// 16-byte unit `unit` of row `row` in a tile of 64-column pieces with 128-byte swizzle.
+__device__ __forceinline__ uint32_t mc_unit(int row, int unit) {
+  return static_cast<uint32_t>(unit >> 3) * MC_CHUNK + static_cast<uint32_t>(row) * 128u + (static_cast<uint32_t>((unit & 7) ^ (row & 7)) << 4);
+}
+
+// U of one (chunk, head).  The keys' tile [128 tokens, 128] is weighted in place (its low halves go to a second tile) and
+// multiplied as the transposed A operand with V.
+template <int VC>
+__global__ void __launch_bounds__(MC_UPDATE_THREADS)
+memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const MemoryParams p, const MemoryChunks c) {
+  constexpr int OFF_LO = 2 * MC_CHUNK, OFF_V = 4 * MC_CHUNK, OFF_N = OFF_V + VC * MC_CHUNK, OFF_W = OFF_N + 16 * 128 * 4, OFF_BAR = OFF_W + MC_ROWS * 4;
+  constexpr uint32_t COLS = VC == 1 ? 64 : (VC == 2 ? 128 : 256);
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const uint32_t sbase = smem_u32(smem);
+  float* s_n = reinterpret_cast<float*>(smem + OFF_N);             // [16][128]
+  float* s_w = reinterpret_cast<float*>(smem + OFF_W);
+  const uint32_t bar_k = sbase + OFF_BAR, bar_v = bar_k + 8, bar_m = bar_k + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + OFF_BAR + 24);
+  volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
+  const int h = blockIdx.y;
+  const int* ch = c.chunks + 4 * blockIdx.x;
+  const int row0 = ch[1], rows = ch[2];
+  const long long ph = static_cast<long long>(blockIdx.x) * p.H + h;
+  if (tid == 0) {
+    *abort_word = 0;
+    mbar_init(bar_k, 1);
+    mbar_init(bar_v, 1);
+    mbar_init(bar_m, 1);
+    fence_mbar_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(smem_u32(tmem_slot), COLS);
+    tmem_relinquish();
+  }
+  const float end2 = c.end2[ph];
+  if (tid < MC_ROWS) s_w[tid] = tid < rows ? exp2f(c.a2[static_cast<long long>(h) * c.ldt + row0 + tid] - end2) : 0.f;
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  if (tid == 0) {
+    mbar_expect_tx(bar_k, 2 * MC_CHUNK);
+    for (int i = 0; i < 2; ++i) tma_load_2d(sbase + i * MC_CHUNK, &tmK, bar_k, h * p.dp + i * 64, row0);
+    mbar_expect_tx(bar_v, VC * MC_CHUNK);
+    for (int i = 0; i < VC; ++i) tma_load_2d(sbase + OFF_V + i * MC_CHUNK, &tmV, bar_v, h * p.vp + i * 64, row0);
+  }
+  bool ok = mbar_wait(bar_k, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE);
+  if (ok) {
+    const int unit = tid & 15, r0 = tid >> 4;
+    float acc[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+#pragma unroll
+    for (int i = 0; i < MC_ROWS / 16; ++i) {
+      const int row = r0 + 16 * i;
+      uint4* at = reinterpret_cast<uint4*>(smem + mc_unit(row, unit));
+      const float w = s_w[row];
+      float f[8], hi[8];
+      unpack8(*at, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        f[e] *= w;
+        acc[e] += f[e];
+      }
+      const uint4 packed = pack8(f);
+      unpack8(packed, hi);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] -= hi[e];
+      *at = packed;
+      *reinterpret_cast<uint4*>(smem + OFF_LO + mc_unit(row, unit)) = pack8(f);
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s_n[r0 * 128 + unit * 8 + e] = acc[e];
+  }
+  fence_proxy_async_smem();
+  __syncthreads();
+  if (tid == 0 && ok && mbar_wait(bar_v, 0, abort_word, FT_ERR_TIMEOUT_MMA)) {
+    constexpr uint32_t idesc = make_idesc_f16(128, VC * 64, 1, 1, 1);
+#pragma unroll
+    for (int half = 0; half < 2; ++half)
+#pragma unroll
+      for (int kk = 0; kk < MC_ROWS / 16; ++kk)
+        umma_f16_ss(tmem, make_smem_desc_sw128(sbase + half * OFF_LO + kk * 2048, MC_CHUNK, 1024),
+                    make_smem_desc_sw128(sbase + OFF_V + kk * 2048, MC_CHUNK, 1024), idesc, (half > 0 || kk > 0) ? 1u : 0u);
+    umma_commit(bar_m);
+  }
+  if (tid < p.dp && ok) {
+    float n = 0.f;
+#pragma unroll
+    for (int g = 0; g < 16; ++g) n += s_n[g * 128 + tid];
+    c.Un[ph * p.dp + tid] = n;
+  }
+  ok = mbar_wait(bar_m, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE) && ok;
+  ok = __all_sync(0xffffffffu, ok);
+  if (ok) {
+    tc_fence_after();
+    const int ew = warp & 3, d = ew * 32 + lane;
+    if (ew * 32 < p.dp) {                              // whole warps: the TMEM load is a warp-wide instruction
+      float* dst = c.U + (ph * p.dp + d) * c.vw;
+      for (int col = (warp >> 2) * 32; col < VC * 64; col += 64) {
+        uint32_t t[32];
+        tmem_ld_32x32(tmem + (static_cast<uint32_t>(ew * 32) << 16) + col, t);
+        tmem_ld_wait();
+        if (d < p.dp) {
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            float f[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]);
+            store8_sector(dst + col + g * 8, f);
+          }
+        }
+      }
+    }
+  } else if (tid == 0) {                               // let copies in flight land before the block leaves
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tmem, COLS);
+  }
+  if (tid == 0 && *abort_word != 0 && c.status) atomicCAS(c.status, 0, *abort_word);
+}
+
+// The states of a portion's chunks, one after another: a thread owns four elements of S (and the first block one of n).
+constexpr int MC_AHEAD = 4;       // contributions loaded together
+__global__ void __launch_bounds__(256)
+memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
+  const int h = blockIdx.y;
+  const int* span = c.spans + 4 * blockIdx.z;
+  const int slot = span[0], pos0 = span[2], rows = span[3];
+  const int n_chunks = (rows + MC_ROWS - 1) / MC_ROWS, first = c.span_chunks[blockIdx.z];
+  const long long sh = static_cast<long long>(slot) * p.H + h;
+  const int i = (blockIdx.x * 256 + threadIdx.x) * 4;
+  const long long per = static_cast<long long>(p.dp) * c.vw;
+  auto factor = [&](int k) {
+    const long long at = static_cast<long long>(first + k) * p.H + h;
+    return exp2f(c.start2[at] - c.end2[at]);
+  };
+  if (i < p.dp * c.vw) {
+    const int d = i / c.vw, col = i - d * c.vw;
+    float4* S = reinterpret_cast<float4*>(p.S + (sh * p.dp + d) * p.vp + col);
+    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (col < p.vp && pos0 > 0) s = *S;
+    for (int k0 = 0; k0 < n_chunks; k0 += MC_AHEAD) {
+      float4 u[MC_AHEAD];
+      float g[MC_AHEAD];
+#pragma unroll
+      for (int j = 0; j < MC_AHEAD; ++j)
+        if (k0 + j < n_chunks) {
+          u[j] = __ldcs(reinterpret_cast<const float4*>(c.U + (static_cast<long long>(first + k0 + j) * p.H + h) * per + i));
+          g[j] = factor(k0 + j);
+        }
+#pragma unroll
+      for (int j = 0; j < MC_AHEAD; ++j)
+        if (k0 + j < n_chunks) {
+          *reinterpret_cast<uint2*>(c.Sb + (static_cast<long long>(first + k0 + j) * p.H + h) * per + i) = make_uint2(pack_bf16x2(s.x, s.y), pack_bf16x2(s.z, s.w));
+          s.x = g[j] * s.x + u[j].x; s.y = g[j] * s.y + u[j].y; s.z = g[j] * s.z + u[j].z; s.w = g[j] * s.w + u[j].w;
+        }
+    }
+    if (col < p.vp) *S = s;
+  }
+  if (blockIdx.x == 0 && static_cast<int>(threadIdx.x) < p.dp) {
+    float n = pos0 > 0 ? p.n[sh * p.dp + threadIdx.x] : 0.f;
+    for (int k = 0; k < n_chunks; ++k) {
+      const long long at = (static_cast<long long>(first + k) * p.H + h) * p.dp + threadIdx.x;
+      c.nb[at] = n;
+      n = factor(k) * n + c.Un[at];
+    }
+    p.n[sh * p.dp + threadIdx.x] = n;
+  }
+}
+
+// Outputs of one (chunk, head): thread = token.  Shared memory: Q and K (later the starting state), V.
+template <int DC, int VC>
+__global__ void __launch_bounds__(MC_OUT_THREADS)
+memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                     const __grid_constant__ CUtensorMap tmS, const MemoryParams p, const MemoryChunks c) {
+  constexpr int FRONT = (2 * DC > VC ? 2 * DC : VC) * MC_CHUNK;
+  constexpr int OFF_K = DC * MC_CHUNK, OFF_V = FRONT, OFF_A = OFF_V + VC * MC_CHUNK, OFF_NB = OFF_A + MC_ROWS * 4, OFF_BAR = OFF_NB + 128 * 4;
+  constexpr uint32_t COLS = VC <= 2 ? 256 : 512, COL_O = 128, COL_Q = 64;      // scores (then P | weighted q), outputs
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const uint32_t sbase = smem_u32(smem);
+  float* s_a = reinterpret_cast<float*>(smem + OFF_A);
+  float* s_nb = reinterpret_cast<float*>(smem + OFF_NB);
+  const uint32_t bar_qk = sbase + OFF_BAR, bar_v = bar_qk + 8, bar_s = bar_qk + 16, bar_score = bar_qk + 24, bar_out = bar_qk + 32;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + OFF_BAR + 40);
+  volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  const int warp = threadIdx.x >> 5, tid = threadIdx.x;
+  const int h = blockIdx.y;
+  const int* ch = c.chunks + 4 * blockIdx.x;
+  const int row0 = ch[1], rows = ch[2];
+  const bool fresh = ch[3] == 0 && c.spans[4 * ch[0] + 2] == 0;                 // nothing ahead of this chunk
+  const long long ph = static_cast<long long>(blockIdx.x) * p.H + h, gate_at = static_cast<long long>(h) * c.ldt + row0;
+  if (tid == 0) {
+    *abort_word = 0;
+    for (int i = 0; i < 5; ++i) mbar_init(bar_qk + 8 * i, 1);
+    fence_mbar_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(smem_u32(tmem_slot), COLS);
+    tmem_relinquish();
+  }
+  s_a[tid] = tid < rows ? c.a2[gate_at + tid] : -INFINITY;
+  if (tid < p.dp) s_nb[tid] = fresh ? 0.f : c.nb[ph * p.dp + tid];
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  if (tid == 0) {
+    mbar_expect_tx(bar_qk, 2 * DC * MC_CHUNK);
+    for (int i = 0; i < DC; ++i) {
+      tma_load_2d(sbase + i * MC_CHUNK, &tmQ, bar_qk, h * p.dp + i * 64, row0);
+      tma_load_2d(sbase + OFF_K + i * MC_CHUNK, &tmK, bar_qk, h * p.dp + i * 64, row0);
+    }
+    mbar_expect_tx(bar_v, VC * MC_CHUNK);
+    for (int i = 0; i < VC; ++i) tma_load_2d(sbase + OFF_V + i * MC_CHUNK, &tmV, bar_v, h * p.vp + i * 64, row0);
+    if (mbar_wait(bar_qk, 0, abort_word, FT_ERR_TIMEOUT_MMA)) {
+      constexpr uint32_t idesc = make_idesc_f16(128, 128, 1, 0, 0);
+      for (int kk = 0; kk < p.dp / 16; ++kk) {
+        const uint32_t off = (kk >> 2) * MC_CHUNK + (kk & 3) * 32;
+        umma_f16_ss(tmem, make_smem_desc_sw128(sbase + off, 16, 1024), make_smem_desc_sw128(sbase + OFF_K + off, 16, 1024), idesc, kk > 0 ? 1u : 0u);
+      }
+      umma_commit(bar_score);
+    }
+  }
+  const bool row_ok = tid < rows;
+  const float x2 = row_ok ? c.x2[gate_at + tid] : 0.f, floor_m = row_ok ? c.floor[gate_at + tid] : 1.f;
+  const float inter = (fresh || !row_ok) ? 0.f : exp2f(c.start2[ph] - x2) * p.q_scale;
+  const long long row = static_cast<long long>(row0) + (row_ok ? tid : 0);
+  const __nv_bfloat16* q_row = static_cast<const __nv_bfloat16*>(p.q) + row * p.ld + static_cast<long long>(h) * p.dp;
+  const uint32_t lane_addr = tmem + (static_cast<uint32_t>(warp * 32) << 16);
+  float den = 0.f;
+  bool ok = mbar_wait(bar_score, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE);
+  if (tid == 0 && ok && !fresh) {                      // the scores are done: Q and K make room for the state
+    mbar_expect_tx(bar_s, static_cast<uint32_t>(p.dp) * 128u * VC);
+    for (int i = 0; i < VC; ++i) tma_load_2d(sbase + i * MC_CHUNK, &tmS, bar_s, i * 64, static_cast<int>(ph * p.dp));
+  }
+  ok = __all_sync(0xffffffffu, ok);
+  if (ok) {
+    tc_fence_after();
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {                      // 32 keys at a time; P of a group lies over scores already read
+      uint32_t pk[16];
+      if (j <= warp) {
+        uint32_t t[32];
+        tmem_ld_32x32(lane_addr + j * 32, t);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          float v[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int key = j * 32 + 2 * i + e;
+            const float w = fast_exp2(s_a[key] - x2);
+            v[e] = key <= tid ? __uint_as_float(t[2 * i + e]) * p.q_scale * w : 0.f;
+            den += v[e];
+          }
+          pk[i] = pack_bf16x2(v[0], v[1]);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) pk[i] = 0u;
+      }
+      tmem_st_32x16(lane_addr + j * 16, pk);
+    }
+    if (!fresh) {
+      for (int d = 0; d < p.dp; d += 32) {             // the weighted query, an operand like P
+        uint32_t pk[16];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          float f[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = 0.f;
+          if (d + u * 8 < p.dp) load8(q_row + d + u * 8, f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            f[e] *= inter;
+            if (d + u * 8 < p.dp) den += f[e] * s_nb[d + u * 8 + e];
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) pk[u * 4 + e] = pack_bf16x2(f[2 * e], f[2 * e + 1]);
+        }
+        tmem_st_32x16(lane_addr + COL_Q + d / 2, pk);
+      }
+    }
+    tmem_st_wait();
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (tid == 0 && ok) {
+    tc_fence_after();
+    bool go = mbar_wait(bar_v, 0, abort_word, FT_ERR_TIMEOUT_MMA);
+    if (go && !fresh) go = mbar_wait(bar_s, 0, abort_word, FT_ERR_TIMEOUT_MMA);
+    if (go) {
+      constexpr uint32_t idesc = make_idesc_f16(128, VC * 64, 1, 0, 1);
+#pragma unroll
+      for (int kk = 0; kk < MC_ROWS / 16; ++kk)
+        umma_f16_ts(tmem + COL_O, tmem + kk * 8, make_smem_desc_sw128(sbase + OFF_V + kk * 2048, MC_CHUNK, 1024), idesc, kk > 0 ? 1u : 0u);
+      if (!fresh)
+        for (int kk = 0; kk < p.dp / 16; ++kk)
+          umma_f16_ts(tmem + COL_O, tmem + COL_Q + kk * 8, make_smem_desc_sw128(sbase + kk * 2048, MC_CHUNK, 1024), idesc, 1u);
+      umma_commit(bar_out);
+    }
+  }
+  ok = mbar_wait(bar_out, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE) && ok;
+  ok = __all_sync(0xffffffffu, ok);
+  if (ok) {
+    tc_fence_after();
+    const float inv = 1.f / (fmaxf(fabsf(den), floor_m) + 1e-6f);
+    float sum = 0.f;
+#pragma unroll
+    for (int col = 0; col < VC * 64; col += 32) {
+      uint32_t t[32];
+      tmem_ld_32x32(lane_addr + COL_O + col, t);
+      tmem_ld_wait();
+#pragma unroll
+      for (int e = 0; e < 32; ++e) {
+        const float o = __uint_as_float(t[e]);
+        if (col + e < p.vp) sum += o * o;
+      }
+    }
+    // rms norm of o * inv: the factor of a column is inv / sqrt(mean(o^2) inv^2 + eps)
+    const float r = p.out_scale * inv * rsqrtf(sum * inv * inv / static_cast<float>(p.vdim) + p.eps);
+    const __nv_bfloat16* g_row = static_cast<const __nv_bfloat16*>(p.gate) + row * p.ld + static_cast<long long>(h) * p.vp;
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.vp;
+    const float* norm = p.norm + static_cast<long long>(h) * p.vp;
+#pragma unroll 1
+    for (int col = 0; col < VC * 64; col += 32) {
+      if (col >= p.vp) break;
+      uint32_t t[32];
+      tmem_ld_32x32(lane_addr + COL_O + col, t);
+      tmem_ld_wait();
+      if (!row_ok) continue;
+#pragma unroll
+      for (int g = 0; g < 4; ++g) {
+        const int j = col + g * 8;
+        if (j >= p.vp) continue;
+        float f[8], w[8], z[8];
+        load8(norm + j, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]) * r * w[e];
+        if (p.gate) {
+          load8(g_row + j, z);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-z[e]));
+        }
+        store8(out + j, f);
+      }
+    }
+  } else if (tid == 0) {                               // let copies in flight land before the block leaves
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tmem, COLS);
+  }
+  if (tid == 0 && *abort_word != 0 && c.status) atomicCAS(c.status, 0, *abort_word);
+}
+
 static bool mem_aligned(std::initializer_list<const void*> ps) {
   uintptr_t v = 0;
   for (const void* p : ps) v |= reinterpret_cast<uintptr_t>(p);
@@ -217,4 +711,84 @@ FT_API int ft_memory_steps(const void* q, const void* k, const void* v, const vo
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;
+}
+
+// Whole portions of bf16 rows in chunks (see the top of this file): dp up to 128, vp up to 256.  rows: rows of the packed
+// projection.  spans [n_spans, 4] and chunks [n_chunks, 4] (span, first row, rows up to 128, number within the portion;
+// portion after portion) int32, span_chunks [n_spans]: first chunk of a portion.  scratch: ft_memory_scratch bytes.
+static long long memory_scratch_at(int rows, int H, int dp, int vp, int n_chunks, long long* at) {
+  const long long vw = (vp + 63) / 64 * 64, ldt = (rows + 31) / 32 * 32, ch = static_cast<long long>(n_chunks) * H;
+  const long long sizes[9] = {H * ldt * 4, H * ldt * 4, H * ldt * 4, ch * 4, ch * 4, ch * dp * vw * 4, ch * dp * 4, ch * dp * vw * 2, ch * dp * 4};
+  long long total = 0;
+  for (int i = 0; i < 9; ++i) {
+    if (at) at[i] = total;
+    total += (sizes[i] + 255) / 256 * 256;
+  }
+  return total;
+}
+
+FT_API long long ft_memory_scratch(int rows, int H, int dp, int vp, int n_chunks) { return memory_scratch_at(rows, H, dp, vp, n_chunks, nullptr); }
+
+template <int DC, int VC>
+static int launch_memory(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const MemoryParams& p,
+                         const MemoryChunks& c, int device, cudaStream_t stream) {
+  constexpr int UPDATE_SMEM = (4 + VC) * MC_CHUNK + 16 * 128 * 4 + MC_ROWS * 4 + 64 + 1024;
+  constexpr int OUT_SMEM = ((2 * DC > VC ? 2 * DC : VC) + VC) * MC_CHUNK + MC_ROWS * 4 + 128 * 4 + 64 + 1024;
+  static bool attr_set[64] = {false};
+  if (!attr_set[device]) {
+    FT_CUDA_CHECK(cudaFuncSetAttribute(memory_update_kernel<VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, UPDATE_SMEM));
+    FT_CUDA_CHECK(cudaFuncSetAttribute(memory_output_kernel<DC, VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, OUT_SMEM));
+    attr_set[device] = true;
+  }
+  memory_gates_kernel<<<dim3(p.H, c.n_spans), MC_GATE_WARPS * 32, 0, stream>>>(p, c);
+  FT_CUDA_CHECK(cudaGetLastError());
+  memory_update_kernel<VC><<<dim3(c.n_chunks, p.H), MC_UPDATE_THREADS, UPDATE_SMEM, stream>>>(tk, tv, p, c);
+  FT_CUDA_CHECK(cudaGetLastError());
+  memory_carry_kernel<<<dim3((p.dp * c.vw / 4 + 255) / 256, p.H, c.n_spans), 256, 0, stream>>>(p, c);
+  FT_CUDA_CHECK(cudaGetLastError());
+  memory_output_kernel<DC, VC><<<dim3(c.n_chunks, p.H), MC_OUT_THREADS, OUT_SMEM, stream>>>(tq, tk, tv, ts, p, c);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch(4);
+  return FT_E_OK;
+}
+
+FT_API int ft_memory_chunks(const void* q, const void* k, const void* v, const void* gate, long long ld, const float* z, long long ldz,
+                            int f_off, const float* i_bias, const float* f_bias, const float* norm, float* S, float* n, float* m,
+                            void* out, long long ldo, int H, int dp, int vp, int vdim, float q_scale, float cap, float eps,
+                            float out_scale, int rows, const int* spans, int n_spans, const int* span_chunks, const int* chunks,
+                            int n_chunks, void* scratch, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  MemoryParams p;
+  if (int rc = memory_params(p, q, k, v, gate, ld, z, ldz, f_off, i_bias, f_bias, norm, S, n, m, out, ldo, H, dp, vp, vdim, q_scale, cap, eps, out_scale))
+    return rc;
+  FT_REQUIRE(dp <= 128 && vp <= 256, "ft_memory_chunks: heads of %d x %d are too large", dp, vp);
+  FT_REQUIRE(rows > 0 && spans && span_chunks && chunks && scratch && (reinterpret_cast<uintptr_t>(scratch) & 255) == 0, "ft_memory_chunks: null pointer or unaligned scratch");
+  if (n_spans <= 0 || n_chunks <= 0) return FT_E_OK;
+  FT_REQUIRE(n_spans < 65536 && static_cast<long long>(n_chunks) * H * dp < (1ll << 31), "ft_memory_chunks: too many portions or chunks");
+  long long at[9];
+  memory_scratch_at(rows, H, dp, vp, n_chunks, at);
+  char* base = static_cast<char*>(scratch);
+  MemoryChunks c;
+  c.spans = spans; c.span_chunks = span_chunks; c.chunks = chunks;
+  c.a2 = reinterpret_cast<float*>(base + at[0]); c.x2 = reinterpret_cast<float*>(base + at[1]); c.floor = reinterpret_cast<float*>(base + at[2]);
+  c.start2 = reinterpret_cast<float*>(base + at[3]); c.end2 = reinterpret_cast<float*>(base + at[4]); c.U = reinterpret_cast<float*>(base + at[5]);
+  c.Un = reinterpret_cast<float*>(base + at[6]); c.Sb = reinterpret_cast<__nv_bfloat16*>(base + at[7]); c.nb = reinterpret_cast<float*>(base + at[8]);
+  c.ldt = (rows + 31) / 32 * 32; c.n_spans = n_spans; c.n_chunks = n_chunks; c.vw = (vp + 63) / 64 * 64;
+  c.status = device_status_word(device);
+  CUtensorMap tq, tk, tv, ts;
+  const uint64_t stride = static_cast<uint64_t>(ld) * 2;
+  if (int rc = make_tmap_2d(&tq, q, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
+  if (int rc = make_tmap_2d(&tk, k, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
+  if (int rc = make_tmap_2d(&tv, v, 2, static_cast<uint64_t>(H) * vp, rows, stride, 64, MC_ROWS, 3)) return rc;
+  if (int rc = make_tmap_2d(&ts, c.Sb, 2, c.vw, static_cast<uint64_t>(n_chunks) * H * dp, static_cast<uint64_t>(c.vw) * 2, 64, dp, 3)) return rc;
+#define FT_MC(DCN)                                                              \
+  switch (c.vw / 64) {                                                          \
+    case 1: return launch_memory<DCN, 1>(tq, tk, tv, ts, p, c, device, stream); \
+    case 2: return launch_memory<DCN, 2>(tq, tk, tv, ts, p, c, device, stream); \
+    case 3: return launch_memory<DCN, 3>(tq, tk, tv, ts, p, c, device, stream); \
+    default: return launch_memory<DCN, 4>(tq, tk, tv, ts, p, c, device, stream); \
+  }
+  if (dp <= 64) { FT_MC(1) }
+  FT_MC(2)
+#undef FT_MC
 }

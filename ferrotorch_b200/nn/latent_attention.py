@@ -9,10 +9,15 @@ from dataclasses import dataclass
 import torch
 from torch import nn
 
+from .. import _native
 from ..ops import decoder as D
 from ..ops import functional as F
 from .gated_attention import checked, unpad_heads
 from .packed_block import RotarySpec, pad_heads, pad_to, round_up
+from .paged import prefill_pages
+
+FORMED_PAGE = 128    # rows of a page of formed keys
+ABSORB_ROWS = 16     # a step whose portions have at most so many tokens treats their rows like single tokens
 
 
 @dataclass
@@ -63,9 +68,11 @@ class LatentSpec:
 class LatentAttention(nn.Module):
     """``W_o (attention(h) * sigmoid(W_g h))``, element by element.
 
-    One packed product ``[q | latent, rotated key | g]`` and one pass for norm, rotation and cache.  Queries are brought into the
-    latent space (``W_uk`` applied to them instead of to every key), so that all heads attend to the cached rows themselves, and
-    the gated product with ``W_uv`` follows."""
+    One packed product ``[q | latent, rotated key | g]`` and one pass for norm, rotation and cache.  Then, for single tokens, short
+    portions and in fp32: queries are brought into the latent space (``W_uk`` applied to them instead of to every key), so that all
+    heads attend to the cached rows themselves, and the gated product with ``W_uv`` follows.  For longer portions: keys and values of
+    their contexts are formed from the cached rows by one product each (the rotated key part passes through it by a unit
+    matrix), and the portions run on the prefill kernel, gate included."""
 
     def __init__(self, hidden_size: int, spec: LatentSpec, eps: float):
         super().__init__()
@@ -77,6 +84,19 @@ class LatentAttention(nn.Module):
         self.register_buffer("to_latent", torch.zeros(s.heads, 1, s.padded_rank, s.padded_dim))      # W_uk of a head, transposed
         self.register_buffer("to_value", torch.zeros(s.heads, 1, s.padded_vdim, s.padded_rank))      # W_uv of a head
         self.register_buffer("out_proj", torch.zeros(width, self.value_width))
+        self.register_buffer("key_proj", None, persistent=False)         # all heads' keys and values from a cached row
+        self.register_buffer("value_proj", None, persistent=False)
+
+    def _form_keys(self) -> None:
+        s, t = self.spec, self.to_latent
+        if t.dtype != torch.bfloat16 or s.head_size > 128 or s.padded_vdim > 128:
+            return
+        key = torch.zeros(s.heads, s.head_size, s.row_size, dtype=t.dtype, device=t.device)
+        key[:, :s.padded_dim, :s.padded_rank] = t[:, 0].transpose(1, 2)
+        unit = torch.arange(s.rot_dim, device=t.device)
+        key[:, s.padded_dim + unit, s.padded_rank + unit] = 1.0
+        self.key_proj = key.flatten(0, 1)
+        self.value_proj = pad_to(self.to_value[:, 0].flatten(0, 1), self.value_width, s.row_size)
 
     def _shapes(self) -> dict:
         W, s = self.hidden_size, self.spec
@@ -107,6 +127,7 @@ class LatentAttention(nn.Module):
         self.to_latent[:, 0].copy_(pad_to(uk.transpose(1, 2), s.heads, s.padded_rank, s.padded_dim))
         self.to_value[:, 0].copy_(pad_to(uv, s.heads, s.padded_vdim, s.padded_rank))
         self.out_proj.copy_(pad_to(pad_heads(sd["o"].t(), s.heads, s.padded_vdim).t(), width, self.value_width))
+        self._form_keys()
 
     def unpack(self) -> dict:
         s, W = self.spec, self.hidden_size
@@ -132,11 +153,23 @@ class LatentAttention(nn.Module):
         """The sublayer's output for input ``h``; ``layer``: its place in the cache."""
         s, T = self.spec, h.shape[0]
         packed = F.linear_rows(h, self.in_proj)
-        q_lat = torch.empty((T, s.heads, s.row_size), device=h.device, dtype=h.dtype)
+        formed = self.key_proj is not None and h.is_cuda and batch.longest > ABSORB_ROWS
+        n = batch.n_single if formed else T               # rows that attend in the latent space
+        q_lat = torch.empty((n, s.heads, s.row_size), device=h.device, dtype=h.dtype)
         D.latent_finish(packed, cache, layer, batch, heads=s.heads, q_off=0, q_head=s.head_size, q_rot=s.padded_dim, c_off=self.q_width,
                         rank=s.rank, rank_pad=s.padded_rank, weight=self.latent_norm, eps=self.eps, table=cache.rotary_table(s.rotary), q_lat=q_lat)
-        D.block_linear(packed[:, :self.q_width], self.to_latent, q_lat.flatten(1), a_col=s.head_size, out_col=s.row_size)
-        o_lat = cache.attend(layer, q_lat, batch, s.scale)
         heads = torch.empty((T, self.value_width), device=h.device, dtype=h.dtype)
-        D.block_linear(o_lat.flatten(1), self.to_value, heads, gate=packed[:, self.q_width + s.row_size:])
+        gate = packed[:, self.q_width + s.row_size:]
+        if n:
+            D.block_linear(packed[:n, :self.q_width], self.to_latent, q_lat.flatten(1), a_col=s.head_size, out_col=s.row_size)
+            o_lat = cache.decode(layer, q_lat, batch.visible[:n], s.scale, seq_ids=batch.slots[:n]) if formed else cache.attend(layer, q_lat, batch, s.scale)
+            D.block_linear(o_lat.flatten(1), self.to_value, heads[:n], gate=gate[:n])
+        if formed:
+            q, g, out = (t.unflatten(1, (s.heads, -1)) for t in (packed[:, :self.q_width], gate, heads))
+            for rows, spans, longest, table, items in batch.contexts(int(_native.kernels().ft_paged_prefill_tile(1)), FORMED_PAGE):
+                ctx = torch.empty((rows, s.row_size), device=h.device, dtype=h.dtype)
+                cache.gather_contexts(layer, spans, longest, ctx, FORMED_PAGE)
+                k, v = F.linear_rows(ctx, self.key_proj), F.linear_rows(ctx, self.value_proj)
+                prefill_pages(q, k.view(-1, FORMED_PAGE, s.heads, s.head_size), v.view(-1, FORMED_PAGE, s.heads, s.padded_vdim), table, items, s.scale,
+                              out=out, gate=g)
         return D.SublayerTerms(dense=F.linear_rows(heads, self.out_proj))

@@ -24,6 +24,8 @@ _native.register_protos({
     "ft_paged_decode_scratch": (_ll, [_i, _i, _i, _i]),
     "ft_paged_decode": (_i, [_vp] * 10 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp, _f, _i, _i, _vp]),
     "ft_paged_rows": (_i, [_vp] * 9 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _i, _f, _i, _i, _vp, _f, _i, _i, _vp]),
+    "ft_latent_decode": (_i, [_vp] * 7 + [_i] * 4 + [_ll, _i, _i, _i, _f, _i, _i, _vp]),
+    "ft_latent_gather": (_i, [_vp] * 3 + [_i, _i, _vp] + [_i] * 6 + [_vp]),
     "ft_paged_prefill_tile": (_i, [_i]),
     "ft_paged_prefill": (_i, [_vp] * 8 + [_i] * 6 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp, _f, _i, _vp]),
 })
@@ -38,6 +40,20 @@ def _gate_args(gate: torch.Tensor | None) -> tuple:
 
 def _ptr(t: torch.Tensor | None):
     return t.data_ptr() if t is not None else None
+
+
+def prefill_pages(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, table: torch.Tensor, items: torch.Tensor, scale: float, *,
+                  out: torch.Tensor, gate: torch.Tensor | None = None, window: int | None = None, sink: torch.Tensor | None = None,
+                  chunk: int | None = None, slopes: torch.Tensor | None = None, out_scale: float = 1.0) -> None:
+    """Attention of the portions listed in ``items`` (device only): ``q [T, Hq, D]``, pages ``k [pages, tokens, Hkv, D]`` and ``v``,
+    block table ``[sequences, pages of one]``."""
+    T, Hq, D = q.shape
+    pages, bs, Hkv, Dv = v.shape
+    rc = _native.kernels().ft_paged_prefill(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), table.data_ptr(), items.data_ptr(), _ptr(gate), _ptr(sink), out.data_ptr(), items.shape[0], T, Hq, Hkv, D,
+        Dv, q.stride(0), *_gate_args(gate), out.stride(0), bs, table.shape[1], pages, float(scale), int(window or 0), int(chunk or 0), _ptr(slopes),
+        float(out_scale), F._dev(q), F._stream())
+    _native.check(rc, "ft_paged_prefill")
 
 
 class OutOfPages(RuntimeError):
@@ -144,6 +160,11 @@ class RaggedBatch:
         self.positions, self.slots, self.visible, self.starts = ints[:n], ints[n:2 * n], ints[2 * n:3 * n], ints[3 * n:4 * n]
         self.span_table = ints[4 * n:4 * n + 4 * k].view(k, 4)
 
+    @property
+    def longest(self) -> int:
+        """Tokens of the longest portion."""
+        return max((s[3] for s in self.spans), default=0)
+
     def work_items(self, tile_tokens: int):
         """The portions cut into work items of the prefill kernel (``[n, 4]`` int32 on the device: slot, first row,
         tokens, first position; at most ``2 * tile_tokens`` tokens each), longest key range first."""
@@ -157,6 +178,54 @@ class RaggedBatch:
             got = host.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else host
             self._items[tile_tokens] = got
         return got
+
+
+    def contexts(self, tile_tokens: int, page: int = 128, limit: int = 32768) -> list:
+        """The portions' contexts laid out one after another in pages of ``page`` rows of their own, for attention over keys that are
+        formed for this step: groups ``(rows, spans [n, 3], longest, block table [n, pages], work items [m, 4])`` of at most ``limit``
+        rows (a longer context is a group of its own); spans are ``(slot, first row, tokens)``, items as in :meth:`work_items` with
+        the place in the group's table instead of the slot."""
+        key = ("contexts", tile_tokens, page, limit)
+        got = self._items.get(key)
+        if got is None:
+            got, group, rows = [], [], 0
+            for span in self.spans:
+                need = (span[2] + span[3] + page - 1) // page * page
+                if group and rows + need > limit:
+                    got.append(self._context_group(group, rows, tile_tokens, page))
+                    group, rows = [], 0
+                group.append((*span, rows))
+                rows += need
+            got.append(self._context_group(group, rows, tile_tokens, page))
+            self._items[key] = got
+        return got
+
+    def _context_group(self, group: list, rows: int, tile_tokens: int, page: int) -> tuple:
+        step, n = 2 * tile_tokens, len(group)
+        longest = max(s[2] + s[3] for s in group)
+        width = (longest + page - 1) // page
+        spans = [v for slot, _, start, k, first in group for v in (slot, first, start + k)]
+        table = [min(first // page + j, rows // page - 1) for *_, first in group for j in range(width)]
+        items = [(i, row + o, min(step, k - o), start + o) for i, (_, row, start, k, _) in enumerate(group) for o in range(0, k, step)]
+        items.sort(key=lambda r: -(r[2] + r[3]))
+        host = torch.tensor(spans + table + [v for r in items for v in r], dtype=torch.int32)
+        buf = host.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else host
+        a, b = 3 * n, 3 * n + n * width
+        return rows, buf[:a].view(n, 3), longest, buf[a:b].view(n, width), buf[b:].view(-1, 4)
+
+    def chunk_table(self, rows: int):
+        """The portions cut into chunks of ``rows`` tokens, portion after portion: ``(first chunk of every portion [n_spans], chunks
+        [n, 4])``, int32 on the device; a chunk is portion, first row, rows, number within the portion."""
+        got = self._items.get(("chunks", rows))
+        if got is None:
+            first, chunks = [], []
+            for i, (_, row, _, n) in enumerate(self.spans):
+                first.append(len(chunks))
+                chunks += [(i, row + o, min(rows, n - o), o // rows) for o in range(0, n, rows)]
+            host = torch.tensor(first + [v for c in chunks for v in c], dtype=torch.int32)
+            buf = host.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else host
+            got = self._items[("chunks", rows)] = (buf[:len(first)], buf[len(first):].view(-1, 4), host)
+        return got[:2]
 
 
 class DecodeBatch(RaggedBatch):
@@ -353,6 +422,9 @@ class PagedKVCache:
         if out is None:
             out = torch.empty((B, Hq, Dv), device=q.device, dtype=q.dtype)
         seq_ids = seq_ids.to(device=q.device, dtype=torch.int32) if seq_ids is not None else None
+        plain = gate is None and not window and sink is None and not chunk and slopes is None and out_scale == 1.0
+        if plain and self._latent_ok(layer, q):
+            return self._latent_rows(layer, q, ctx_len, seq_ids, scale, out, n_splits)
         if not self._tensor_core_ok(layer, q, 16) and (q.dtype != torch.bfloat16 or self.values_in_keys[layer] or D != Dv or D not in (64, 128)
                                                        or Hq // Hkv not in (1, 2, 4, 8)):
             rows = seq_ids if seq_ids is not None else torch.arange(B, device=q.device, dtype=torch.int32)
@@ -404,18 +476,48 @@ class PagedKVCache:
                 out[row:row + n] = self._finish_reference(o, gate[row:row + n] if gate is not None else None, out_scale)
             return out
         bs = self.block_size
+        if self.values_in_keys[layer]:                    # a portion's rows are as good as single ones
+            self.decode(layer, q[n1:], batch.visible[n1:], scale, seq_ids=batch.slots[n1:], gate=gate[n1:] if gate is not None else None, out=out[n1:],
+                        window=window, sink=sink, chunk=chunk, slopes=slopes, out_scale=out_scale)
+            return out
         if not (self._tensor_core_ok(layer, q, 128) and scale > 0 and bs >= 8 and (128 % bs == 0 or bs % 128 == 0)):
             self._rows(layer, q[n1:], batch.visible[n1:], batch.slots[n1:], scale, gate[n1:] if gate is not None else None, out[n1:],
                        window, sink, chunk, slopes, out_scale)
             return out
-        lib = _native.kernels()
-        items = batch.work_items(int(lib.ft_paged_prefill_tile(Hq // Hkv)))
-        rc = lib.ft_paged_prefill(q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), table.data_ptr(), items.data_ptr(),
-                                  _ptr(gate), _ptr(sink), out.data_ptr(), items.shape[0], T, Hq, Hkv, D, Dv, q.stride(0),
-                                  *_gate_args(gate), out.stride(0), bs, self.max_blocks, self.num_blocks, float(scale),
-                                  int(window or 0), int(chunk or 0), _ptr(slopes), float(out_scale), F._dev(q), F._stream())
-        _native.check(rc, "ft_paged_prefill")
+        items = batch.work_items(int(_native.kernels().ft_paged_prefill_tile(Hq // Hkv)))
+        prefill_pages(q, self.k[layer], self.v[layer], table, items, scale, out=out, gate=gate, window=window, sink=sink, chunk=chunk, slopes=slopes,
+                      out_scale=out_scale)
         return out
+
+    def _latent_ok(self, layer: int, q: torch.Tensor) -> bool:
+        _, D, Dv = self.shapes[layer]
+        bs = self.block_size
+        return (self.values_in_keys[layer] and q.dtype == torch.bfloat16 and q.is_contiguous() and D <= 576 and Dv <= 512 and q.shape[0] < 65536
+                and bs >= 8 and (128 % bs == 0 or bs % 128 == 0))
+
+    def _latent_rows(self, layer: int, q: torch.Tensor, visible: torch.Tensor, slots: torch.Tensor | None, scale: float, out: torch.Tensor,
+                     n_splits: int = 0) -> torch.Tensor:
+        """Rows of queries in the latent space over latent rows (the tensor-core kernel)."""
+        B, H, W = q.shape
+        Dv = self.shapes[layer][2]
+        if n_splits <= 0:
+            n_splits = max(1, min(16, 148 // (B * ((H + 31) // 32))))
+        lib = _native.kernels()
+        n_scr = int(lib.ft_paged_decode_scratch(B, H, Dv, n_splits))
+        scratch = F._get_scratch("paged_decode", n_scr, q.device) if n_scr else None
+        rc = lib.ft_latent_decode(q.data_ptr(), self.k[layer].data_ptr(), self.block_table.data_ptr(), _ptr(slots), visible.data_ptr(), out.data_ptr(),
+                                  _ptr(scratch), B, H, W, Dv, out.stride(0), self.block_size, self.max_blocks, self.num_blocks, float(scale), n_splits,
+                                  F._dev(q), F._stream())
+        _native.check(rc, "ft_latent_decode")
+        return out
+
+    def gather_contexts(self, layer: int, spans: torch.Tensor, longest: int, out: torch.Tensor, pad: int) -> None:
+        """Rows 0 .. n - 1 of a layer's keys of sequence ``slot``, contiguous from row ``first`` of ``out``, for every ``(slot, first, n)``
+        of ``spans``, and zero rows up to a multiple of ``pad`` (device only)."""
+        rc = _native.kernels().ft_latent_gather(self.k[layer].data_ptr(), self.sync_table().data_ptr(), spans.data_ptr(), spans.shape[0], longest,
+                                                out.data_ptr(), out.shape[1] * out.element_size(), pad, self.block_size, self.max_blocks, self.num_blocks,
+                                                F._dev(out), F._stream())
+        _native.check(rc, "ft_latent_gather")
 
     def gather(self, layer: int, seq: int, length: int):
         """Contiguous ``[length, Hkv, D]`` K and ``[length, Hkv, Dv]`` V of one sequence (debug / reference path;

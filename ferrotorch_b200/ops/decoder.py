@@ -31,6 +31,8 @@ _native.register_protos({
     "ft_embed_bigram": (_i, [_vp] * 8 + [_ll, _i, _i, _ll, _ll, _f, _vp, _i] + [_vp] * 3 + [_i] * 3 + [_f] + [_i] * 5 + [_vp]),
     "ft_softcap": (_i, [_vp, _ll, _f, _i, _vp]),
     "ft_latent_finish": (_i, [_vp, _ll, _vp, _i] + [_vp] * 6 + [_i] * 11 + [_f] + [_i] * 5 + [_vp]),
+    "ft_memory_scratch": (_ll, [_i] * 5),
+    "ft_memory_chunks": (_i, [_vp] * 4 + [_ll, _vp, _ll, _i] + [_vp] * 7 + [_ll] + [_i] * 4 + [_f] * 4 + [_i, _vp, _i, _vp, _vp, _i, _vp, _i, _vp]),
     "ft_memory_steps": (_i, [_vp] * 4 + [_ll, _vp, _ll, _i] + [_vp] * 7 + [_ll] + [_i] * 4 + [_f] * 4 + [_vp] * 3 + [_i] * 3 + [_vp]),
     "ft_grouped_gemm": (_i, [_vp, _ll, _i] + [_vp] * 3 + [_i] * 5 + [_vp, _i, _vp, _ll] + [_i] * 4 + [_vp]),
 })
@@ -342,15 +344,20 @@ def rglru_scan(a: torch.Tensor, x: torch.Tensor, y: torch.Tensor, out: torch.Ten
     _native.check(rc, "ft_rglru_scan")
 
 
+MEMORY_CHUNK = 128       # tokens of a chunk of ft_memory_chunks
+MEMORY_STEP_ROWS = 12    # a step whose portions have at most so many tokens runs them token by token
+
+
 def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, z: torch.Tensor, i_bias: torch.Tensor,
                   f_bias: torch.Tensor, norm: torch.Tensor, state, batch, out: torch.Tensor, *, heads: int, dim: int, vdim: int, cap: float,
-                  eps: float, out_scale: float = 1.0) -> torch.Tensor:
+                  eps: float, out_scale: float = 1.0, chunks: bool = False) -> torch.Tensor:
     """Matrix memories over the rows of a ragged batch: ``out = norm(o) * weight * sigmoid(gate) * out_scale`` per head (see
     ``csrc/matrix_memory.cu``).
 
     ``q, k [T, heads * dp]``, ``v, gate [T, heads * vp]``: parts of one packed projection (one row stride), heads padded from ``dim``
     and ``vdim``; ``z [T, 2 * n]`` fp32: pre-activations of the input gates and, from column n, of the forget gates; ``state``: what
-    the sequences' slots hold (:class:`~ferrotorch_b200.nn.recurrent.MatrixMemoryState`)."""
+    the sequences' slots hold (:class:`~ferrotorch_b200.nn.recurrent.MatrixMemoryState`).  Portions in bf16 run in chunks (short
+    ones only with ``chunks``), everything else token by token."""
     T, n_gate = q.shape[0], z.shape[1] // 2
     if not q.is_cuda:
         qs, ks = (t.float().unflatten(1, (heads, -1)) for t in (q, k))
@@ -366,19 +373,27 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch
             out[r] = (o.flatten(1) * norm * torch.sigmoid(gate[r].float()) * out_scale).to(out.dtype)
         return out
     dp, vp = state.S.shape[2:]
+    lib, f32 = _native.kernels(), q.dtype == torch.float32
+    args = (q.data_ptr(), k.data_ptr(), v.data_ptr(), gate.data_ptr(), q.stride(0), z.data_ptr(), z.stride(0), n_gate, i_bias.data_ptr(),
+            f_bias.data_ptr(), norm.data_ptr(), state.S.data_ptr(), state.n.data_ptr(), state.m.data_ptr(), out.data_ptr(), out.stride(0), heads, dp, vp,
+            vdim, dim ** -0.5, float(cap), float(eps), float(out_scale))
 
     def steps(spans, items):
-        rc = _native.kernels().ft_memory_steps(
-            q.data_ptr(), k.data_ptr(), v.data_ptr(), gate.data_ptr(), q.stride(0), z.data_ptr(), z.stride(0), n_gate, i_bias.data_ptr(),
-            f_bias.data_ptr(), norm.data_ptr(), state.S.data_ptr(), state.n.data_ptr(), state.m.data_ptr(), out.data_ptr(), out.stride(0), heads, dp, vp,
-            vdim, dim ** -0.5, float(cap), float(eps), float(out_scale), _ptr(spans), batch.positions.data_ptr(), batch.slots.data_ptr(), items,
-            int(q.dtype == torch.float32), F._dev(q), F._stream())
+        rc = lib.ft_memory_steps(*args, _ptr(spans), batch.positions.data_ptr(), batch.slots.data_ptr(), items, int(f32), F._dev(q), F._stream())
         _native.check(rc, "ft_memory_steps")
 
     if batch.n_single:
         steps(None, batch.n_single)
-    if batch.spans:
+    if not batch.spans:
+        return out
+    if f32 or dp > 128 or vp > 256 or (batch.longest <= MEMORY_STEP_ROWS and not chunks):
         steps(batch.span_table, len(batch.spans))
+        return out
+    first, table = batch.chunk_table(MEMORY_CHUNK)
+    scratch = F._get_scratch("matrix_memory", (int(lib.ft_memory_scratch(T, heads, dp, vp, table.shape[0])) + 3) // 4, q.device)
+    rc = lib.ft_memory_chunks(*args, T, batch.span_table.data_ptr(), len(batch.spans), first.data_ptr(), table.data_ptr(), table.shape[0], scratch.data_ptr(),
+                              F._dev(q), F._stream())
+    _native.check(rc, "ft_memory_chunks")
     return out
 
 

@@ -20,11 +20,12 @@ import torch
 # name: (hidden, layers, heads, kv heads, head size, SwiGLU width, vocabulary, prompt, batch).  The parallel family's
 # two-matrix MLP is 1.5 x as wide, so both have the same number of parameters and matrix-product FLOPs.  Zolorax has the
 # same dense MLP in every other layer and eight experts of half the SwiGLU width, two of them used, in the others: equal
-# FLOPs per token, but more weights to read in a decode step.
+# FLOPs per token, but more weights to read in a decode step.  Tenalorn has in every layer eight experts of a third of the
+# SwiGLU width, two of them used, and a shared one: again equal FLOPs; memories of 128 x 128 with half the width in all.
 SIZES = {"1b": (2048, 16, 32, 8, 64, 8192, 128256, 2048, 64),
          "3b": (3072, 28, 24, 8, 128, 8192, 128256, 2048, 64),
          "8b": (4096, 32, 32, 8, 128, 14336, 128256, 2048, 64)}
-FAMILIES = ("llama", "bopudra", "zolorax")
+FAMILIES = ("llama", "bopudra", "zolorax", "tenalorn")
 PAGE = 16
 EXPERTS, TOP, WINDOW = 8, 2, 1024
 
@@ -39,6 +40,14 @@ def zolorax_config(size: str, n: int):
     return cfg
 
 
+def tenalorn_config(size: str, n: int):
+    from ferrotorch_b200.models.tenalorn import BigramSpec, TenalornConfig
+
+    hidden, _, heads, kv, dim, ff, vocab, _, _ = SIZES[size]
+    return TenalornConfig.pattern(vocab, hidden, n, heads, kv, dim, ff // 3 // 64 * 64, chunk=WINDOW, memory_heads=hidden // 256, memory_dim=128,
+                                  memory_vdim=128, rank=512, experts=EXPERTS, top=TOP, identity=0, streams=2, bigram=BigramSpec(131071, 1031, 17))
+
+
 def build(family: str, size: str, layers: int | None = None):
     hidden, n, heads, kv, dim, ff, vocab, _, _ = SIZES[size]
     n = layers or n
@@ -50,6 +59,10 @@ def build(family: str, size: str, layers: int | None = None):
         from ferrotorch_b200.models.zolorax import ZoloraxForCausalLM
 
         return ZoloraxForCausalLM(zolorax_config(size, n), device="cuda").random_()
+    if family == "tenalorn":
+        from ferrotorch_b200.models.tenalorn import TenalornForCausalLM
+
+        return TenalornForCausalLM(tenalorn_config(size, n), device="cuda").random_()
     from ferrotorch_b200.models.llama import LlamaConfig, LlamaForCausalLM
 
     cfg = LlamaConfig(vocab_size=vocab, hidden_size=hidden, intermediate_size=ff, num_hidden_layers=n, num_attention_heads=heads,
@@ -139,7 +152,7 @@ def kernel_table(size: str, peaks: dict, steps: int, families=FAMILIES) -> list:
 
     lib = _native.kernels()
     for family in families:
-        model = build(family, size, layers=6 if family == "zolorax" else 2)
+        model = build(family, size, layers={"zolorax": 6, "tenalorn": 3}.get(family, 2))
         cache = model.make_paged_cache(batch * ((prompt + 16) // PAGE + 1), PAGE, batch, prompt + 16)
         for s in range(batch):
             cache.reserve(s, prompt + 1)
@@ -159,6 +172,8 @@ def kernel_table(size: str, peaks: dict, steps: int, families=FAMILIES) -> list:
 
             if family == "zolorax":
                 _zolorax_kernels(lambda *a: add(family, phase, *a), gemm, model, cache, b, phase == "prefill", (hidden, heads, kv, dim, prompt, per, batch))
+            elif family == "tenalorn":
+                _tenalorn_kernels(lambda *a: add(family, phase, *a), gemm, model, cache, b, phase == "prefill", (hidden, heads, kv, dim, prompt, per, batch))
             elif family == "bopudra":
                 blk, nrm = model.blocks[0], model.norms[0]
                 x, h = F.embedding_dynamic_tanh(b.tokens, model.embed, nrm.alpha, nrm.weight, nrm.bias, out_dtype=torch.bfloat16)
@@ -287,6 +302,105 @@ def _zolorax_kernels(add, gemm, model, cache, b, prefill: bool, sizes: tuple) ->
     add("rms norm + experts' terms", lambda: rec.norm1(x, pending=(yt, r.place), update=True, out_dtype=dt), 0, T * hidden * (10 + 2 * top))
     if not prefill:
         gemm("head", h, model.head, lambda: F.linear_f32_out(h, model.head))
+
+
+def _tenalorn_kernels(add, gemm, model, cache, b, prefill: bool, sizes: tuple) -> None:
+    """The kernels of a parallel and a latent mixer, the routed feed-forward and the streams."""
+    from ferrotorch_b200 import _native
+    from ferrotorch_b200.nn.latent_attention import FORMED_PAGE
+    from ferrotorch_b200.nn.paged import prefill_pages
+    from ferrotorch_b200.ops import decoder as D
+    from ferrotorch_b200.ops import functional as F
+
+    hidden, heads, kv, dim, prompt, per, batch = sizes
+    T, dt, c = b.n_rows, torch.bfloat16, model.config
+    S, par, lat = c.streams, model.layers[0], model.layers[1]
+
+    def embed():
+        return D.embed_bigram(b, cache, model.embed, model.bigram, c.embedding_scale, c.bigram.mul_prev, c.bigram.mul_cur, par.hc1.into, par.norm1.weight,
+                              c.norm_eps, count=hidden, out_dtype=dt)
+
+    x, h = embed()
+    add("embedding + bigram + norm", embed, 0, T * hidden * 10)
+    # attention beside memories
+    m, a, w = par.mixer, par.mixer.attn, par.mixer.memory
+    at = m.offsets
+    packed, z = F.linear_rows(h, m.in_proj), F.linear_f32_out(h, m.gate_proj)
+    gemm("parallel in_proj (q|k|v|q'|k'|v'|g')", h, m.in_proj, lambda: F.linear_rows(h, m.in_proj))
+    add("memory gates' product (fp32 out)", lambda: F.linear_f32_out(h, m.gate_proj), 0, 2 * T * hidden)
+    add("head norms, append", lambda: D.qkv_head_finish(packed, cache, 0, b, heads=heads, dim=dim, q_off=at["left.q"], k_off=at["left.k"], v_off=at["left.v"],
+                                                        q_weight=m.ones, k_weight=m.ones, true_dim=dim, eps=m.eps), 0, 4 * T * (heads + 2 * kv) * dim)
+    both = torch.empty((T, m.left_width + m.right_width), device="cuda", dtype=dt)
+    q, o = packed[:, at["left.q"]:at["left.k"]].unflatten(1, (heads, dim)), both[:, :m.left_width].unflatten(1, (heads, dim))
+    seen = sum(i % a.chunk + 1 for i in range(prompt))
+    now = (prompt - 1) % a.chunk + 1
+    add("attention (chunks of %d, distance bias)" % a.chunk, lambda: cache.attend(0, q, b, a.scale, out=o, chunk=a.chunk, slopes=m.slopes, out_scale=1.2),
+        4 * heads * dim * per * seen if prefill else 0, 2 * T * (2 * heads + 2 * kv) * dim if prefill else batch * now * kv * 2 * dim * 2)
+
+    def memory():
+        D.matrix_memory(packed[:, at["right.q"]:at["right.k"]], packed[:, at["right.k"]:at["right.v"]], packed[:, at["right.v"]:at["right.g"]],
+                        packed[:, at["right.g"]:], z, m.i_bias, m.f_bias, m.norm, cache.states[0], b, both[:, m.left_width:], heads=w.heads, dim=w.dim,
+                        vdim=w.vdim, cap=w.gate_cap, eps=m.eps)
+
+    inner = w.heads * (2 * w.dim + 3 * w.vdim) * 2 * T
+    flops = T * w.heads * (2 * 64 * (w.dim + w.vdim) + 4 * w.dim * w.vdim)
+    add("matrix memories" + (" (four passes)" if prefill else " (step)"), memory, flops if prefill else 0,
+        inner + (0 if prefill else 8 * T * w.heads * w.dim * (w.vdim + 1)))
+    gemm("parallel out_proj", both, m.out_proj, lambda: F.linear_rows(both, m.out_proj))
+    # latent attention
+    m, s = lat.mixer, lat.mixer.spec
+    packed = F.linear_rows(h, m.in_proj)
+    gemm("latent in_proj (q|latent|g)", h, m.in_proj, lambda: F.linear_rows(h, m.in_proj))
+    table, gate = cache.rotary_table(s.rotary), packed[:, m.q_width + s.row_size:]
+    q_lat = torch.randn((0 if prefill else T, s.heads, s.row_size), device="cuda").to(dt)
+    add("latent norm, rotation, append", lambda: D.latent_finish(
+        packed, cache, 1, b, heads=s.heads, q_off=0, q_head=s.head_size, q_rot=s.padded_dim, c_off=m.q_width, rank=s.rank, rank_pad=s.padded_rank,
+        weight=m.latent_norm, eps=m.eps, table=table, q_lat=q_lat), 0, 2 * T * (3 * s.row_size + 2 * s.heads * s.padded_rot))
+    out = torch.empty((T, m.value_width), device="cuda", dtype=dt)
+    if prefill:
+        rows, spans, longest, pages, items = b.contexts(int(_native.kernels().ft_paged_prefill_tile(1)), FORMED_PAGE)[0]
+        ctx = torch.empty((rows, s.row_size), device="cuda", dtype=dt)
+        add("latent rows of the contexts", lambda: cache.gather_contexts(1, spans, longest, ctx, FORMED_PAGE), 0, 4 * ctx.numel())
+        k, v = F.linear_rows(ctx, m.key_proj), F.linear_rows(ctx, m.value_proj)
+        gemm("keys from latents", ctx, m.key_proj, lambda: F.linear_rows(ctx, m.key_proj))
+        gemm("values from latents", ctx, m.value_proj, lambda: F.linear_rows(ctx, m.value_proj))
+        q4, g4, o4 = (t.unflatten(1, (s.heads, -1)) for t in (packed[:, :m.q_width], gate, out))
+        k, v = k.view(-1, FORMED_PAGE, s.heads, s.head_size), v.view(-1, FORMED_PAGE, s.heads, s.padded_vdim)
+        add("attention (formed keys, gated)", lambda: prefill_pages(q4, k, v, pages, items, s.scale, out=o4, gate=g4),
+            2 * s.heads * (s.head_size + s.padded_vdim) * per * prompt * (prompt + 1) // 2, 2 * T * s.heads * (2 * s.head_size + 3 * s.padded_vdim))
+    else:
+        add("queries into the latent space", lambda: D.block_linear(packed[:, :m.q_width], m.to_latent, q_lat.flatten(1), a_col=s.head_size, out_col=s.row_size),
+            2 * T * m.to_latent.numel(), 2 * (m.to_latent.numel() + T * s.heads * (s.padded_dim + s.padded_rank)))
+        o_lat = cache.decode(1, q_lat, b.visible, s.scale, seq_ids=b.slots)
+        add("attention (latent rows)", lambda: cache.decode(1, q_lat, b.visible, s.scale, seq_ids=b.slots), 2 * s.heads * (s.row_size + s.padded_rank) * batch * prompt,
+            batch * prompt * s.row_size * 2)
+        add("values from latents, gated", lambda: D.block_linear(o_lat.flatten(1), m.to_value, out, gate=gate), 2 * T * m.to_value.numel(),
+            2 * (m.to_value.numel() + T * s.heads * (s.padded_rank + 2 * s.padded_vdim)))
+    gemm("latent out_proj", out, m.out_proj, lambda: F.linear_rows(out, m.out_proj))
+    # feed-forward and streams
+    m, e = par.mlp, par.mlp.spec
+    n_act = T * e.top
+    kw = dict(identity=e.identity, score=e.score, correction=m.correction, normalize=e.normalize)
+    r = D.moe_route(h, m.router, e.experts, e.top, **kw)
+    add("routing (logits, choice, sort, gather)", lambda: D.moe_route(h, m.router, e.experts, e.top, **kw), 2 * T * hidden * e.outputs, 2 * T * hidden * (1 + e.top))
+    act = D.grouped_linear(r.sorted, m.gate_up, r, glu="silu", seg_rows=T, scaled=False)
+    yt = D.grouped_linear(act, m.down, r, seg_rows=T)
+    add("experts gate|up + silu", lambda: D.grouped_linear(r.sorted, m.gate_up, r, glu="silu", seg_rows=T, scaled=False), 4 * n_act * hidden * e.ff,
+        2 * (m.gate_up.numel() + n_act * (hidden + e.ff)))
+    add("experts down", lambda: D.grouped_linear(act, m.down, r, seg_rows=T), 2 * n_act * hidden * e.ff, 2 * (m.down.numel() + n_act * (hidden + e.ff)))
+    act = torch.empty((T, m.shared_down.shape[1]), device="cuda", dtype=dt)
+    add("shared expert gate|up + silu", lambda: D.block_linear(h, m.shared_gate_up, act, glu="silu"), 4 * T * hidden * e.shared_ff,
+        2 * (m.shared_gate_up.numel() + T * (hidden + e.shared_ff)))
+    gemm("shared expert down", act, m.shared_down, lambda: F.linear_rows(act, m.shared_down))
+    y = F.linear_rows(act, m.shared_down)
+    xs = x[:, None].repeat(1, S, 1)
+    add("streams + norm (mixer)", lambda: par.hc1.step(xs, D.SublayerTerms(dense=y), par.hc2.into, par.norm2, dt), 0, T * hidden * (8 * S + 4))
+    terms = D.SublayerTerms(yt, r.place, r.weight, y)
+    add("streams + norm (experts' terms)", lambda: par.hc2.step(xs, terms, lat.hc1.into, lat.norm1, dt), 0, T * hidden * (8 * S + 4 + 2 * e.top))
+    if not prefill:
+        gemm("head", h, model.head, lambda: F.linear_f32_out(h, model.head))
+        logits = F.linear_f32_out(h, model.head)
+        add("soft cap", lambda: D.softcap_(logits, 30.0), 0, 8 * logits.numel())
 
 
 def run(args, sampler_cls) -> dict:

@@ -20,9 +20,10 @@
 //   memory_update_kernel  U = sum_s e^(a_s - x_end) k_s v_s^T of every (chunk, head): tcgen05 product with the weighted keys
 //                         as high and low bf16 halves, so that the state keeps about 16 bits more than its operands
 //   memory_carry_kernel   S' = e^(M - x_end) S + U over the chunks of a portion, element by element in fp32; leaves every
-//                         chunk's starting state in bf16 and the final one in the slot
-//   memory_output_kernel  P = causal e^(a_s - x_t) q.k and e^(M - x_t) q written over the scores in TMEM as operands of
-//                         one accumulator, O = P V + (..q) S; denominator, norm, gate and store
+//                         chunk's starting state as high and low bf16 halves and the final one in the slot
+//   memory_output_kernel  O = q S, scaled row by row with e^(M - x_t) in TMEM, then + P V with the weights P = causal
+//                         e^(a_s - x_t) q.k written over the scores; denominator, norm, gate and store.  S and P are operands in
+//                         high and low halves: o is normed, so where keys nearly cancel, the error of a plain bf16 weight would grow
 //
 // A slot needs no clearing: what a sequence has seen follows from its positions, and position 0 starts from zero.
 #include <initializer_list>
@@ -181,7 +182,7 @@ constexpr int MC_ROWS = 128;      // tokens of a chunk
 constexpr int MC_CHUNK = MC_ROWS * 128;          // bytes of a 64-column tile of 128 rows
 constexpr int MC_GATE_WARPS = 32;
 constexpr int MC_UPDATE_THREADS = 256;
-constexpr int MC_OUT_THREADS = 128;
+constexpr int MC_OUT_THREADS = 160;
 
 struct MemoryChunks {
   const int* spans;         // [n_spans, 4]: slot, first row, first position, rows
@@ -194,7 +195,7 @@ struct MemoryChunks {
   float* end2;              // [n_chunks, H]: x of the last token
   float* U;                 // [n_chunks, H, dp, vw]
   float* Un;                // [n_chunks, H, dp]
-  __nv_bfloat16* Sb;        // [n_chunks, H, dp, vw]: states at the chunks' starts
+  __nv_bfloat16* Sb;        // [2, n_chunks, H, dp, vw]: states at the chunks' starts, high and low halves
   float* nb;                // [n_chunks, H, dp]
   long long ldt;
   int n_spans, n_chunks, vw;      // vw: vp rounded up to 64
@@ -426,7 +427,7 @@ memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
   const int n_chunks = (rows + MC_ROWS - 1) / MC_ROWS, first = c.span_chunks[blockIdx.z];
   const long long sh = static_cast<long long>(slot) * p.H + h;
   const int i = (blockIdx.x * 256 + threadIdx.x) * 4;
-  const long long per = static_cast<long long>(p.dp) * c.vw;
+  const long long per = static_cast<long long>(p.dp) * c.vw, low = static_cast<long long>(c.n_chunks) * p.H * per;
   auto factor = [&](int k) {
     const long long at = static_cast<long long>(first + k) * p.H + h;
     return exp2f(c.start2[at] - c.end2[at]);
@@ -448,7 +449,11 @@ memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
 #pragma unroll
       for (int j = 0; j < MC_AHEAD; ++j)
         if (k0 + j < n_chunks) {
-          *reinterpret_cast<uint2*>(c.Sb + (static_cast<long long>(first + k0 + j) * p.H + h) * per + i) = make_uint2(pack_bf16x2(s.x, s.y), pack_bf16x2(s.z, s.w));
+          __nv_bfloat16* at = c.Sb + (static_cast<long long>(first + k0 + j) * p.H + h) * per + i;
+          const uint32_t h0 = pack_bf16x2(s.x, s.y), h1 = pack_bf16x2(s.z, s.w);
+          const float2 f0 = unpack_bf16x2(h0), f1 = unpack_bf16x2(h1);
+          *reinterpret_cast<uint2*>(at) = make_uint2(h0, h1);
+          *reinterpret_cast<uint2*>(at + low) = make_uint2(pack_bf16x2(s.x - f0.x, s.y - f0.y), pack_bf16x2(s.z - f1.x, s.w - f1.y));
           s.x = g[j] * s.x + u[j].x; s.y = g[j] * s.y + u[j].y; s.z = g[j] * s.z + u[j].z; s.w = g[j] * s.w + u[j].w;
         }
     }
@@ -465,23 +470,31 @@ memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
   }
 }
 
-// Outputs of one (chunk, head): thread = token.  Shared memory: Q and K (later the starting state), V.
+// Outputs of one (chunk, head).  Warps 0-3: thread = token.  Warp 4: copies and products.  Shared memory: Q | K, then the low half
+// of the state | the high half of the state, then V.
+template <int DC, int VC>
+struct MemOut {
+  static constexpr int MID = DC > VC ? DC : VC;
+  static constexpr int OFF_K = DC * MC_CHUNK, OFF_V = OFF_K + MID * MC_CHUNK, OFF_A = OFF_V + VC * MC_CHUNK, OFF_NB = OFF_A + MC_ROWS * 4,
+                       OFF_BAR = OFF_NB + 128 * 4, SMEM = OFF_BAR + 128 + 1024;
+  static constexpr uint32_t COLS = VC <= 2 ? 256 : 512, COL_LOW = 64, COL_O = 128;      // scores (then P high | low), outputs
+};
+
 template <int DC, int VC>
 __global__ void __launch_bounds__(MC_OUT_THREADS)
 memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                      const __grid_constant__ CUtensorMap tmS, const MemoryParams p, const MemoryChunks c) {
-  constexpr int FRONT = (2 * DC > VC ? 2 * DC : VC) * MC_CHUNK;
-  constexpr int OFF_K = DC * MC_CHUNK, OFF_V = FRONT, OFF_A = OFF_V + VC * MC_CHUNK, OFF_NB = OFF_A + MC_ROWS * 4, OFF_BAR = OFF_NB + 128 * 4;
-  constexpr uint32_t COLS = VC <= 2 ? 256 : 512, COL_O = 128, COL_Q = 64;      // scores (then P | weighted q), outputs
+  using Cfg = MemOut<DC, VC>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-  const uint32_t sbase = smem_u32(smem);
-  float* s_a = reinterpret_cast<float*>(smem + OFF_A);
-  float* s_nb = reinterpret_cast<float*>(smem + OFF_NB);
-  const uint32_t bar_qk = sbase + OFF_BAR, bar_v = bar_qk + 8, bar_s = bar_qk + 16, bar_score = bar_qk + 24, bar_out = bar_qk + 32;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + OFF_BAR + 40);
+  const uint32_t sQ = smem_u32(smem), sK = sQ + Cfg::OFF_K, sV = sQ + Cfg::OFF_V;
+  float* s_a = reinterpret_cast<float*>(smem + Cfg::OFF_A);
+  float* s_nb = reinterpret_cast<float*>(smem + Cfg::OFF_NB);
+  enum { QK = 0, HIGH, LOW, V, SCORE, HIGH_DONE, INTER, P_FULL, OUT, NBARS };
+  auto bar = [&](int i) { return sQ + Cfg::OFF_BAR + 8u * i; };
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + Cfg::OFF_BAR + 8 * NBARS);
   volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  const int warp = threadIdx.x >> 5, tid = threadIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
   const int h = blockIdx.y;
   const int* ch = c.chunks + 4 * blockIdx.x;
   const int row0 = ch[1], rows = ch[2];
@@ -489,169 +502,213 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const long long ph = static_cast<long long>(blockIdx.x) * p.H + h, gate_at = static_cast<long long>(h) * c.ldt + row0;
   if (tid == 0) {
     *abort_word = 0;
-    for (int i = 0; i < 5; ++i) mbar_init(bar_qk + 8 * i, 1);
+    for (int i = 0; i < NBARS; ++i) mbar_init(bar(i), i == P_FULL ? 4 : 1);
     fence_mbar_init();
   }
-  if (warp == 0) {
-    tmem_alloc(smem_u32(tmem_slot), COLS);
+  if (warp == 4) {
+    tmem_alloc(smem_u32(tmem_slot), Cfg::COLS);
     tmem_relinquish();
   }
-  s_a[tid] = tid < rows ? c.a2[gate_at + tid] : -INFINITY;
+  if (tid < MC_ROWS) s_a[tid] = tid < rows ? c.a2[gate_at + tid] : -INFINITY;
   if (tid < p.dp) s_nb[tid] = fresh ? 0.f : c.nb[ph * p.dp + tid];
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot;
-  if (tid == 0) {
-    mbar_expect_tx(bar_qk, 2 * DC * MC_CHUNK);
-    for (int i = 0; i < DC; ++i) {
-      tma_load_2d(sbase + i * MC_CHUNK, &tmQ, bar_qk, h * p.dp + i * 64, row0);
-      tma_load_2d(sbase + OFF_K + i * MC_CHUNK, &tmK, bar_qk, h * p.dp + i * 64, row0);
-    }
-    mbar_expect_tx(bar_v, VC * MC_CHUNK);
-    for (int i = 0; i < VC; ++i) tma_load_2d(sbase + OFF_V + i * MC_CHUNK, &tmV, bar_v, h * p.vp + i * 64, row0);
-    if (mbar_wait(bar_qk, 0, abort_word, FT_ERR_TIMEOUT_MMA)) {
-      constexpr uint32_t idesc = make_idesc_f16(128, 128, 1, 0, 0);
-      for (int kk = 0; kk < p.dp / 16; ++kk) {
-        const uint32_t off = (kk >> 2) * MC_CHUNK + (kk & 3) * 32;
-        umma_f16_ss(tmem, make_smem_desc_sw128(sbase + off, 16, 1024), make_smem_desc_sw128(sbase + OFF_K + off, 16, 1024), idesc, kk > 0 ? 1u : 0u);
+
+  if (warp == 4) {
+    if (lane == 0) {
+      auto wait = [&](int i) { return mbar_wait(bar(i), 0, abort_word, FT_ERR_TIMEOUT_MMA); };
+      auto load_v = [&]() {
+        mbar_expect_tx(bar(V), VC * MC_CHUNK);
+        for (int i = 0; i < VC; ++i) tma_load_2d(sV + i * MC_CHUNK, &tmV, bar(V), h * p.vp + i * 64, row0);
+      };
+      auto load_state = [&](int b, uint32_t dst, long long row) {
+        mbar_expect_tx(bar(b), static_cast<uint32_t>(p.dp) * 128u * VC);
+        for (int i = 0; i < VC; ++i) tma_load_2d(dst + i * MC_CHUNK, &tmS, bar(b), i * 64, static_cast<int>(row));
+      };
+      constexpr uint32_t idesc_score = make_idesc_f16(128, 128, 1, 0, 0), idesc_out = make_idesc_f16(128, VC * 64, 1, 0, 1);
+      auto q_state = [&](uint32_t state, bool first) {                          // O (+)= Q times one half of the state
+        for (int kk = 0; kk < p.dp / 16; ++kk)
+          umma_f16_ss(tmem + Cfg::COL_O, make_smem_desc_sw128(sQ + (kk >> 2) * MC_CHUNK + (kk & 3) * 32, 16, 1024),
+                      make_smem_desc_sw128(state + kk * 2048, MC_CHUNK, 1024), idesc_out, (first && kk == 0) ? 0u : 1u);
+      };
+      mbar_expect_tx(bar(QK), 2 * DC * MC_CHUNK);
+      for (int i = 0; i < DC; ++i) {
+        tma_load_2d(sQ + i * MC_CHUNK, &tmQ, bar(QK), h * p.dp + i * 64, row0);
+        tma_load_2d(sK + i * MC_CHUNK, &tmK, bar(QK), h * p.dp + i * 64, row0);
       }
-      umma_commit(bar_score);
-    }
-  }
-  const bool row_ok = tid < rows;
-  const float x2 = row_ok ? c.x2[gate_at + tid] : 0.f, floor_m = row_ok ? c.floor[gate_at + tid] : 1.f;
-  const float inter = (fresh || !row_ok) ? 0.f : exp2f(c.start2[ph] - x2) * p.q_scale;
-  const long long row = static_cast<long long>(row0) + (row_ok ? tid : 0);
-  const __nv_bfloat16* q_row = static_cast<const __nv_bfloat16*>(p.q) + row * p.ld + static_cast<long long>(h) * p.dp;
-  const uint32_t lane_addr = tmem + (static_cast<uint32_t>(warp * 32) << 16);
-  float den = 0.f;
-  bool ok = mbar_wait(bar_score, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE);
-  if (tid == 0 && ok && !fresh) {                      // the scores are done: Q and K make room for the state
-    mbar_expect_tx(bar_s, static_cast<uint32_t>(p.dp) * 128u * VC);
-    for (int i = 0; i < VC; ++i) tma_load_2d(sbase + i * MC_CHUNK, &tmS, bar_s, i * 64, static_cast<int>(ph * p.dp));
-  }
-  ok = __all_sync(0xffffffffu, ok);
-  if (ok) {
-    tc_fence_after();
+      if (fresh) load_v();
+      else load_state(HIGH, sV, ph * p.dp);
+      bool ok = wait(QK);
+      if (ok) {
+        tc_fence_after();
+        for (int kk = 0; kk < p.dp / 16; ++kk) {
+          const uint32_t off = (kk >> 2) * MC_CHUNK + (kk & 3) * 32;
+          umma_f16_ss(tmem, make_smem_desc_sw128(sQ + off, 16, 1024), make_smem_desc_sw128(sK + off, 16, 1024), idesc_score, kk > 0 ? 1u : 0u);
+        }
+        umma_commit(bar(SCORE));
+      }
+      if (!fresh) {
+        if (ok && (ok = wait(HIGH))) {
+          tc_fence_after();
+          q_state(sV, true);
+          umma_commit(bar(HIGH_DONE));
+        }
+        if (ok && (ok = wait(SCORE))) load_state(LOW, sK, (static_cast<long long>(c.n_chunks) * p.H + ph) * p.dp);    // K has been read
+        if (ok && (ok = wait(HIGH_DONE))) load_v();
+        if (ok && (ok = wait(LOW))) {
+          tc_fence_after();
+          q_state(sK, false);
+          umma_commit(bar(INTER));
+        }
+      }
+      if (ok && (ok = wait(V)) && (ok = wait(P_FULL))) {
+        tc_fence_after();
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {                      // 32 keys at a time; P of a group lies over scores already read
-      uint32_t pk[16];
-      if (j <= warp) {
+        for (int half = 0; half < 2; ++half)
+#pragma unroll
+          for (int kk = 0; kk < MC_ROWS / 16; ++kk)
+            umma_f16_ts(tmem + Cfg::COL_O, tmem + half * Cfg::COL_LOW + kk * 8, make_smem_desc_sw128(sV + kk * 2048, MC_CHUNK, 1024), idesc_out,
+                        (fresh && half == 0 && kk == 0) ? 0u : 1u);
+        umma_commit(bar(OUT));
+      }
+      if (!ok) {                                       // let copies in flight land before the block leaves
+        const unsigned long long t0 = globaltimer_ns();
+        while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+      }
+    }
+  } else {
+    const bool row_ok = tid < rows;
+    const float x2 = row_ok ? c.x2[gate_at + tid] : 0.f, floor_m = row_ok ? c.floor[gate_at + tid] : 1.f;
+    const float inter = (fresh || !row_ok) ? 0.f : exp2f(c.start2[ph] - x2) * p.q_scale;
+    const long long row = static_cast<long long>(row0) + (row_ok ? tid : 0);
+    const uint32_t lane_addr = tmem + (static_cast<uint32_t>(warp * 32) << 16);
+    float den = 0.f;
+    if (!fresh) {                                      // q times the normaliser at the chunk's start
+      const __nv_bfloat16* q_row = static_cast<const __nv_bfloat16*>(p.q) + row * p.ld + static_cast<long long>(h) * p.dp;
+      for (int d = 0; d < p.dp; d += 8) {
+        float f[8];
+        load8(q_row + d, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) den += f[e] * s_nb[d + e];
+      }
+      den *= inter;
+    }
+    auto wait = [&](int i) { return __all_sync(0xffffffffu, mbar_wait(bar(i), 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE)); };
+    bool ok = wait(SCORE);
+    if (ok) {
+      tc_fence_after();
+      uint32_t lows[2][16];                            // low halves of the first two groups wait until their scores' place is free
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {                    // 32 keys at a time; the high halves of a group lie over scores already read
+        uint32_t hi[16], lo[16];
+        if (j <= warp) {
+          uint32_t t[32];
+          tmem_ld_32x32(lane_addr + j * 32, t);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            float v[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const int key = j * 32 + 2 * i + e;
+              const float w = fast_exp2(s_a[key] - x2);
+              v[e] = key <= tid ? __uint_as_float(t[2 * i + e]) * p.q_scale * w : 0.f;
+              den += v[e];
+            }
+            hi[i] = pack_bf16x2(v[0], v[1]);
+            const float2 r = unpack_bf16x2(hi[i]);
+            lo[i] = pack_bf16x2(v[0] - r.x, v[1] - r.y);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) hi[i] = lo[i] = 0u;
+        }
+        tmem_st_32x16(lane_addr + j * 16, hi);
+        if (j < 2) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) lows[j][i] = lo[i];
+        } else if (j == 2) {
+          tmem_st_32x16(lane_addr + Cfg::COL_LOW, lows[0]);          // scores 64 .. 95 have been read
+          tmem_st_32x16(lane_addr + Cfg::COL_LOW + 16, lows[1]);
+#pragma unroll
+          for (int i = 0; i < 16; ++i) lows[0][i] = lo[i];
+        } else {
+          tmem_st_32x16(lane_addr + Cfg::COL_LOW + 32, lows[0]);
+          tmem_st_32x16(lane_addr + Cfg::COL_LOW + 48, lo);
+        }
+      }
+      if (!fresh) {
+        ok = wait(INTER);
+        if (ok) {
+          tc_fence_after();
+#pragma unroll 1
+          for (int col = 0; col < VC * 64; col += 32) {
+            uint32_t t[32];
+            tmem_ld_32x32(lane_addr + Cfg::COL_O + col, t);
+            tmem_ld_wait();
+#pragma unroll
+            for (int e = 0; e < 32; ++e) t[e] = __float_as_uint(__uint_as_float(t[e]) * inter);
+            tmem_st_32x32(lane_addr + Cfg::COL_O + col, t);
+          }
+        }
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (ok && lane == 0) mbar_arrive(bar(P_FULL));
+    }
+    if (ok) ok = wait(OUT);
+    if (ok) {
+      tc_fence_after();
+      const float inv = 1.f / (fmaxf(fabsf(den), floor_m) + 1e-6f);
+      float sum = 0.f;
+#pragma unroll
+      for (int col = 0; col < VC * 64; col += 32) {
         uint32_t t[32];
-        tmem_ld_32x32(lane_addr + j * 32, t);
+        tmem_ld_32x32(lane_addr + Cfg::COL_O + col, t);
         tmem_ld_wait();
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          float v[2];
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const int key = j * 32 + 2 * i + e;
-            const float w = fast_exp2(s_a[key] - x2);
-            v[e] = key <= tid ? __uint_as_float(t[2 * i + e]) * p.q_scale * w : 0.f;
-            den += v[e];
-          }
-          pk[i] = pack_bf16x2(v[0], v[1]);
+        for (int e = 0; e < 32; ++e) {
+          const float o = __uint_as_float(t[e]) * inv;
+          if (col + e < p.vp) sum += o * o;
         }
-      } else {
-#pragma unroll
-        for (int i = 0; i < 16; ++i) pk[i] = 0u;
       }
-      tmem_st_32x16(lane_addr + j * 16, pk);
-    }
-    if (!fresh) {
-      for (int d = 0; d < p.dp; d += 32) {             // the weighted query, an operand like P
-        uint32_t pk[16];
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-          float f[8];
-#pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = 0.f;
-          if (d + u * 8 < p.dp) load8(q_row + d + u * 8, f);
-#pragma unroll
-          for (int e = 0; e < 8; ++e) {
-            f[e] *= inter;
-            if (d + u * 8 < p.dp) den += f[e] * s_nb[d + u * 8 + e];
-          }
-#pragma unroll
-          for (int e = 0; e < 4; ++e) pk[u * 4 + e] = pack_bf16x2(f[2 * e], f[2 * e + 1]);
-        }
-        tmem_st_32x16(lane_addr + COL_Q + d / 2, pk);
-      }
-    }
-    tmem_st_wait();
-  }
-  tc_fence_before();
-  __syncthreads();
-  if (tid == 0 && ok) {
-    tc_fence_after();
-    bool go = mbar_wait(bar_v, 0, abort_word, FT_ERR_TIMEOUT_MMA);
-    if (go && !fresh) go = mbar_wait(bar_s, 0, abort_word, FT_ERR_TIMEOUT_MMA);
-    if (go) {
-      constexpr uint32_t idesc = make_idesc_f16(128, VC * 64, 1, 0, 1);
-#pragma unroll
-      for (int kk = 0; kk < MC_ROWS / 16; ++kk)
-        umma_f16_ts(tmem + COL_O, tmem + kk * 8, make_smem_desc_sw128(sbase + OFF_V + kk * 2048, MC_CHUNK, 1024), idesc, kk > 0 ? 1u : 0u);
-      if (!fresh)
-        for (int kk = 0; kk < p.dp / 16; ++kk)
-          umma_f16_ts(tmem + COL_O, tmem + COL_Q + kk * 8, make_smem_desc_sw128(sbase + kk * 2048, MC_CHUNK, 1024), idesc, 1u);
-      umma_commit(bar_out);
-    }
-  }
-  ok = mbar_wait(bar_out, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE) && ok;
-  ok = __all_sync(0xffffffffu, ok);
-  if (ok) {
-    tc_fence_after();
-    const float inv = 1.f / (fmaxf(fabsf(den), floor_m) + 1e-6f);
-    float sum = 0.f;
-#pragma unroll
-    for (int col = 0; col < VC * 64; col += 32) {
-      uint32_t t[32];
-      tmem_ld_32x32(lane_addr + COL_O + col, t);
-      tmem_ld_wait();
-#pragma unroll
-      for (int e = 0; e < 32; ++e) {
-        const float o = __uint_as_float(t[e]);
-        if (col + e < p.vp) sum += o * o;
-      }
-    }
-    // rms norm of o * inv: the factor of a column is inv / sqrt(mean(o^2) inv^2 + eps)
-    const float r = p.out_scale * inv * rsqrtf(sum * inv * inv / static_cast<float>(p.vdim) + p.eps);
-    const __nv_bfloat16* g_row = static_cast<const __nv_bfloat16*>(p.gate) + row * p.ld + static_cast<long long>(h) * p.vp;
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.vp;
-    const float* norm = p.norm + static_cast<long long>(h) * p.vp;
+      const float r = p.out_scale * inv / sqrtf(sum / static_cast<float>(p.vdim) + p.eps);
+      const __nv_bfloat16* g_row = static_cast<const __nv_bfloat16*>(p.gate) + row * p.ld + static_cast<long long>(h) * p.vp;
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.vp;
+      const float* norm = p.norm + static_cast<long long>(h) * p.vp;
 #pragma unroll 1
-    for (int col = 0; col < VC * 64; col += 32) {
-      if (col >= p.vp) break;
-      uint32_t t[32];
-      tmem_ld_32x32(lane_addr + COL_O + col, t);
-      tmem_ld_wait();
-      if (!row_ok) continue;
+      for (int col = 0; col < VC * 64; col += 32) {
+        if (col >= p.vp) break;
+        uint32_t t[32];
+        tmem_ld_32x32(lane_addr + Cfg::COL_O + col, t);
+        tmem_ld_wait();
+        if (!row_ok) continue;
 #pragma unroll
-      for (int g = 0; g < 4; ++g) {
-        const int j = col + g * 8;
-        if (j >= p.vp) continue;
-        float f[8], w[8], z[8];
-        load8(norm + j, w);
+        for (int g = 0; g < 4; ++g) {
+          const int j = col + g * 8;
+          if (j >= p.vp) continue;
+          float f[8], w[8], z[8];
+          load8(norm + j, w);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]) * r * w[e];
-        if (p.gate) {
-          load8(g_row + j, z);
+          for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]) * r * w[e];
+          if (p.gate) {
+            load8(g_row + j, z);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-z[e]));
+            for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-z[e]));
+          }
+          store8(out + j, f);
         }
-        store8(out + j, f);
       }
     }
-  } else if (tid == 0) {                               // let copies in flight land before the block leaves
-    const unsigned long long t0 = globaltimer_ns();
-    while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 0) {
+  if (warp == 4) {
     tc_fence_after();
-    tmem_dealloc(tmem, COLS);
+    tmem_dealloc(tmem, Cfg::COLS);
   }
   if (tid == 0 && *abort_word != 0 && c.status) atomicCAS(c.status, 0, *abort_word);
 }
@@ -718,7 +775,7 @@ FT_API int ft_memory_steps(const void* q, const void* k, const void* v, const vo
 // portion after portion) int32, span_chunks [n_spans]: first chunk of a portion.  scratch: ft_memory_scratch bytes.
 static long long memory_scratch_at(int rows, int H, int dp, int vp, int n_chunks, long long* at) {
   const long long vw = (vp + 63) / 64 * 64, ldt = (rows + 31) / 32 * 32, ch = static_cast<long long>(n_chunks) * H;
-  const long long sizes[9] = {H * ldt * 4, H * ldt * 4, H * ldt * 4, ch * 4, ch * 4, ch * dp * vw * 4, ch * dp * 4, ch * dp * vw * 2, ch * dp * 4};
+  const long long sizes[9] = {H * ldt * 4, H * ldt * 4, H * ldt * 4, ch * 4, ch * 4, ch * dp * vw * 4, ch * dp * 4, ch * dp * vw * 4, ch * dp * 4};
   long long total = 0;
   for (int i = 0; i < 9; ++i) {
     if (at) at[i] = total;
@@ -733,7 +790,7 @@ template <int DC, int VC>
 static int launch_memory(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const MemoryParams& p,
                          const MemoryChunks& c, int device, cudaStream_t stream) {
   constexpr int UPDATE_SMEM = (4 + VC) * MC_CHUNK + 16 * 128 * 4 + MC_ROWS * 4 + 64 + 1024;
-  constexpr int OUT_SMEM = ((2 * DC > VC ? 2 * DC : VC) + VC) * MC_CHUNK + MC_ROWS * 4 + 128 * 4 + 64 + 1024;
+  constexpr int OUT_SMEM = MemOut<DC, VC>::SMEM;
   static bool attr_set[64] = {false};
   if (!attr_set[device]) {
     FT_CUDA_CHECK(cudaFuncSetAttribute(memory_update_kernel<VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, UPDATE_SMEM));
@@ -764,7 +821,7 @@ FT_API int ft_memory_chunks(const void* q, const void* k, const void* v, const v
   FT_REQUIRE(dp <= 128 && vp <= 256, "ft_memory_chunks: heads of %d x %d are too large", dp, vp);
   FT_REQUIRE(rows > 0 && spans && span_chunks && chunks && scratch && (reinterpret_cast<uintptr_t>(scratch) & 255) == 0, "ft_memory_chunks: null pointer or unaligned scratch");
   if (n_spans <= 0 || n_chunks <= 0) return FT_E_OK;
-  FT_REQUIRE(n_spans < 65536 && static_cast<long long>(n_chunks) * H * dp < (1ll << 31), "ft_memory_chunks: too many portions or chunks");
+  FT_REQUIRE(n_spans < 65536 && 2ll * n_chunks * H * dp < (1ll << 31), "ft_memory_chunks: too many portions or chunks");
   long long at[9];
   memory_scratch_at(rows, H, dp, vp, n_chunks, at);
   char* base = static_cast<char*>(scratch);
@@ -780,7 +837,7 @@ FT_API int ft_memory_chunks(const void* q, const void* k, const void* v, const v
   if (int rc = make_tmap_2d(&tq, q, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
   if (int rc = make_tmap_2d(&tk, k, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
   if (int rc = make_tmap_2d(&tv, v, 2, static_cast<uint64_t>(H) * vp, rows, stride, 64, MC_ROWS, 3)) return rc;
-  if (int rc = make_tmap_2d(&ts, c.Sb, 2, c.vw, static_cast<uint64_t>(n_chunks) * H * dp, static_cast<uint64_t>(c.vw) * 2, 64, dp, 3)) return rc;
+  if (int rc = make_tmap_2d(&ts, c.Sb, 2, c.vw, 2 * static_cast<uint64_t>(n_chunks) * H * dp, static_cast<uint64_t>(c.vw) * 2, 64, dp, 3)) return rc;
 #define FT_MC(DCN)                                                              \
   switch (c.vw / 64) {                                                          \
     case 1: return launch_memory<DCN, 1>(tq, tk, tv, ts, p, c, device, stream); \

@@ -55,7 +55,8 @@ def config_dict(case) -> dict:
 
 def random_weights(cfg: dict, seed: int = 0, close_calls: bool = True) -> dict:
     """Without ``close_calls`` the corrections of the router are far apart, so that the rounding of its input in bf16 changes
-    no choice; tests of whole models in bf16 use that."""
+    no choice, and the keys of memories resemble their queries: the direction of a memory's output hangs on the sign of
+    n.q, which rounding may turn where it is nearly zero.  Tests of whole models in bf16 use that."""
     g = torch.Generator().manual_seed(seed)
     W, V, S = cfg["width"], cfg["vocab"], cfg["streams"]
 
@@ -79,6 +80,8 @@ def random_weights(cfg: dict, seed: int = 0, close_calls: bool = True) -> dict:
             H, D, Dv = b["heads"], b["dim"], b["vdim"]
             for name, shape in (("q", (H * D, W)), ("k", (H * D, W)), ("v", (H * Dv, W)), ("g", (H * Dv, W)), ("i", (H, W)), ("f", (H, W))):
                 out[mix + "right." + name] = rnd(*shape, std=W ** -0.5)
+            if not close_calls:
+                out[mix + "right.k"] = (0.95 * out[mix + "right.q"].float() + 0.3 * out[mix + "right.k"].float()).bfloat16()
             out[mix + "right.o"], out[mix + "right.norm"] = rnd(W, H * Dv, std=2.0 * (H * Dv) ** -0.5), rnd(H * Dv, std=0.3, mean=1.0)
             out[mix + "right.i.b"], out[mix + "right.f.b"] = rnd(H), rnd(H, std=1.5, mean=3.0)
         else:
@@ -109,3 +112,4 @@ class Case(DecoderCase):
                 m["scale"] *= 0.5
         weights = random_weights(cfg, seed, dtype == torch.float32)
         super().__init__(cfg, weights, TenalornForCausalLM(TenalornConfig.from_dict(cfg), dtype, device), O.forward)
+        self.loose_rows = 0.0 if dtype == torch.float32 else 0.05

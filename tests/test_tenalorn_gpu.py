@@ -289,12 +289,12 @@ def test_stream_step_kernel(rows, S, H, count, dtype):
             new = O.streams_out([xs[:, s].double() for s in range(S)], mix.double(), out.double(), total)
             u = O.streams_in(new, into.double())
             want = u / torch.sqrt(u.pow(2).sum(-1, keepdim=True) / count + 1e-3) * w.double()
-            src = xs.clone() if xs is x else xs
+            src = xs.clone() if xs is x or S == 1 else xs
             gx, gh = D.stream_step(src, sub, mix, out, into, w, 1e-3, count=count, out_dtype=dt)
             assert gh.dtype == dt and torch.allclose(gx.double(), torch.stack(new, 1), atol=1e-4, rtol=1e-5)
             assert torch.allclose(gh.double(), want, atol=tol * 4, rtol=1e-2 if dtype == "bf16" else 1e-4)
             ids = torch.randint(0, rows, (4,), device="cuda")
-            src = xs.clone() if xs is x else xs
+            src = xs.clone() if xs is x or S == 1 else xs
             same, part = D.stream_step(src, sub, mix, out, into, w, 1e-3, count=count, out_dtype=dt, rows=ids)
             assert torch.equal(part, gh[ids]) and torch.equal(same, xs)
 

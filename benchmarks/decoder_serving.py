@@ -325,9 +325,9 @@ def _tenalorn_kernels(add, gemm, model, cache, b, prefill: bool, sizes: tuple) -
     # attention beside memories
     m, a, w = par.mixer, par.mixer.attn, par.mixer.memory
     at = m.offsets
-    packed, z = F.linear_rows(h, m.in_proj), F.linear_f32_out(h, m.gate_proj)
+    packed, z = F.linear_rows(h, m.in_proj), D.few_outputs(h, m.gate_proj)
     gemm("parallel in_proj (q|k|v|q'|k'|v'|g')", h, m.in_proj, lambda: F.linear_rows(h, m.in_proj))
-    add("memory gates' product (fp32 out)", lambda: F.linear_f32_out(h, m.gate_proj), 0, 2 * T * hidden)
+    add("memory gates' product (fp32 out)", lambda: D.few_outputs(h, m.gate_proj), 0, 2 * T * hidden)
     add("head norms, append", lambda: D.qkv_head_finish(packed, cache, 0, b, heads=heads, dim=dim, q_off=at["left.q"], k_off=at["left.k"], v_off=at["left.v"],
                                                         q_weight=m.ones, k_weight=m.ones, true_dim=dim, eps=m.eps), 0, 4 * T * (heads + 2 * kv) * dim)
     both = torch.empty((T, m.left_width + m.right_width), device="cuda", dtype=dt)
@@ -355,7 +355,7 @@ def _tenalorn_kernels(add, gemm, model, cache, b, prefill: bool, sizes: tuple) -
     q_lat = torch.randn((0 if prefill else T, s.heads, s.row_size), device="cuda").to(dt)
     add("latent norm, rotation, append", lambda: D.latent_finish(
         packed, cache, 1, b, heads=s.heads, q_off=0, q_head=s.head_size, q_rot=s.padded_dim, c_off=m.q_width, rank=s.rank, rank_pad=s.padded_rank,
-        weight=m.latent_norm, eps=m.eps, table=table, q_lat=q_lat), 0, 2 * T * (3 * s.row_size + 2 * s.heads * s.padded_rot))
+        weight=m.latent_norm, eps=m.eps, table=table, q_lat=q_lat), 0, 4 * T * (s.row_size + s.heads * s.padded_rot))
     out = torch.empty((T, m.value_width), device="cuda", dtype=dt)
     if prefill:
         rows, spans, longest, pages, items = b.contexts(int(_native.kernels().ft_paged_prefill_tile(1)), FORMED_PAGE)[0]

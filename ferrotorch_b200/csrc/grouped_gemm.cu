@@ -475,6 +475,38 @@ moe_choose_kernel(const float* __restrict__ logits, long long ldl, int rows, con
   }
 }
 
+// z[n] = w[n] . h for a row h and n outputs (fp32), in shared or global memory: a warp takes two outputs at a time.
+template <typename T>
+__device__ __forceinline__ void row_outputs(const T* h, const T* __restrict__ w, int H, int n, float* z) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int e0 = warp * 2; e0 < n; e0 += MR_THREADS / 16) {
+    const T* w0 = w + static_cast<long long>(e0) * H;
+    const T* w1 = e0 + 1 < n ? w0 + H : w0;
+    float s0 = 0.f, s1 = 0.f;
+#pragma unroll 4
+    for (int i = lane * 8; i < H; i += 256) {
+      float a[8], b[8], c[8];
+      load8(h + i, a);
+      load8(w0 + i, b);
+      load8(w1 + i, c);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) { s0 += a[e] * b[e]; s1 += a[e] * c[e]; }
+    }
+    s0 = warp_sum(s0);
+    s1 = warp_sum(s1);
+    if (lane == 0) {
+      z[e0] = s0;
+      if (e0 + 1 < n) z[e0 + 1] = s1;
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(MR_THREADS)
+few_outputs_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, float* __restrict__ z, int rows, int H, int n) {
+  for (int row = blockIdx.x; row < rows; row += gridDim.x) row_outputs(h + row * ldh, w, H, n, z + static_cast<long long>(row) * n);
+}
+
 // One block per row: the row in registers of all warps in turn, one expert per warp at a time.
 template <typename T>
 __global__ void __launch_bounds__(MR_THREADS)
@@ -483,27 +515,7 @@ moe_route_rows_kernel(const T* __restrict__ h, long long ldh, const T* __restric
   extern __shared__ float mr_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, experts = rule.outputs;
   for (int row = blockIdx.x; row < rows; row += gridDim.x) {
-    const T* hr = h + row * ldh;
-    for (int e0 = warp * 2; e0 < experts; e0 += MR_THREADS / 16) {
-      const T* w0 = router + static_cast<long long>(e0) * H;
-      const T* w1 = e0 + 1 < experts ? w0 + H : w0;
-      float s0 = 0.f, s1 = 0.f;
-#pragma unroll 4
-      for (int i = lane * 8; i < H; i += 256) {
-        float a[8], b[8], c[8];
-        load8(hr + i, a);
-        load8(w0 + i, b);
-        load8(w1 + i, c);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) { s0 += a[e] * b[e]; s1 += a[e] * c[e]; }
-      }
-      s0 = warp_sum(s0);
-      s1 = warp_sum(s1);
-      if (lane == 0) {
-        mr_sm[e0] = s0;
-        if (e0 + 1 < experts) mr_sm[e0 + 1] = s1;
-      }
-    }
+    row_outputs(h + row * ldh, router, H, experts, mr_sm);
     __syncthreads();
     if (warp == 0)
       choose_experts(mr_sm, rule, lane, index + static_cast<long long>(row) * rule.top, weight + static_cast<long long>(row) * rule.top);
@@ -633,6 +645,20 @@ static bool gg_aligned(std::initializer_list<const void*> ps) {
 }  // namespace ft
 
 using namespace ft;
+
+// z [rows, n] = h [rows, H] w^T, fp32 results for a few outputs n of few rows (more of either: a product of their own).  h and w bf16,
+// or fp32 with f32; H a multiple of 8.
+FT_API int ft_few_outputs(const void* h, long long ldh, const void* w, float* z, int rows, int H, int n, int f32, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(h && w && z && H > 0 && H % 8 == 0 && ldh % 8 == 0 && n > 0 && gg_aligned({h, w}), "ft_few_outputs: H=%d and strides must be multiples of 8", H);
+  if (rows <= 0) return FT_E_OK;
+  const int cap = sm_count(device) * 8, grid = rows < cap ? rows : cap;
+  if (f32) few_outputs_kernel<float><<<grid, MR_THREADS, 0, stream>>>(static_cast<const float*>(h), ldh, static_cast<const float*>(w), z, rows, H, n);
+  else few_outputs_kernel<__nv_bfloat16><<<grid, MR_THREADS, 0, stream>>>(static_cast<const __nv_bfloat16*>(h), ldh, static_cast<const __nv_bfloat16*>(w), z, rows, H, n);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
 
 // Work items that ft_moe_route can list for `pairs` (row, choice) pairs over `experts`.
 FT_API int ft_moe_max_items(int pairs, int experts) { return (pairs < experts ? pairs : experts) + pairs / GG_BM; }

@@ -24,11 +24,12 @@
 
 namespace ft {
 
-constexpr int LF_THREADS = 128;
+constexpr int LF_MAX_THREADS = 256;
+constexpr int LF_KEEP = 3;        // vectors of eight elements of the latent that a lane keeps
 
 struct LatentFinishParams {
   void* packed;             // [rows, ld]
-  void* q_lat;              // [n_lat, H, ldq_head]: rows 0 .. n_lat - 1 put their rotated query parts here, behind the latent part
+  void* q_lat;              // [n_lat, H, rank_pad + rot_pad]: rows 0 .. n_lat - 1 put their rotated query parts here, behind the latent part
   const int* pos;
   const int* slots;
   const int* block_table;
@@ -57,7 +58,7 @@ __device__ __forceinline__ void rotate8(float (&f)[8], int d, const float2* cs, 
 
 // One block per row: the first warp takes the latent and the key part, the others the queries.
 template <typename T>
-__global__ void __launch_bounds__(LF_THREADS)
+__global__ void __launch_bounds__(LF_MAX_THREADS)
 latent_finish_kernel(const LatentFinishParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int width = p.rank_pad + p.rot_pad;
@@ -66,22 +67,32 @@ latent_finish_kernel(const LatentFinishParams p) {
     const int position = p.pos[row];
     const float2* cs = p.table + static_cast<long long>(min(position, p.positions - 1)) * p.half;
     if (warp == 0) {
+      const T* c = y + p.c_off;
+      float kept[LF_KEEP][8];
+      float sum = 0.f;
+#pragma unroll
+      for (int k = 0; k < LF_KEEP; ++k) {
+        const int i = (k * 32 + lane) * 8;
+        if (i < width) load8(c + i, kept[k]);
+      }
       const int page = position / p.block_size;
       const int blk = page < p.max_blocks ? p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + page] : -1;
       T* dst = blk >= 0 && blk < p.num_blocks
                    ? static_cast<T*>(p.cache) + (static_cast<long long>(blk) * p.block_size + position % p.block_size) * width : nullptr;
-      T* c = y + p.c_off;
-      float sum = 0.f;
-      for (int i = lane * 8; i < p.rank_pad; i += 256) {
+#pragma unroll
+      for (int k = 0; k < LF_KEEP; ++k)
+        if ((k * 32 + lane) * 8 < p.rank_pad)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) sum += kept[k][e] * kept[k][e];
+      const int rest = (LF_KEEP * 32 + lane) * 8;      // wider rows are read twice
+      for (int i = rest; i < p.rank_pad; i += 256) {
         float f[8];
         load8(c + i, f);
 #pragma unroll
         for (int e = 0; e < 8; ++e) sum += f[e] * f[e];
       }
       const float r = 1.f / sqrtf(warp_sum(sum) / static_cast<float>(p.rank) + p.eps);
-      for (int i = lane * 8; i < width; i += 256) {
-        float f[8];
-        load8(c + i, f);
+      auto finish = [&](int i, float (&f)[8]) {
         if (i < p.rank_pad) {
           float w[8];
           load8(p.weight + i, w);
@@ -90,12 +101,23 @@ latent_finish_kernel(const LatentFinishParams p) {
         } else {
           rotate8(f, i - p.rank_pad, cs, p.half);
         }
-        store8(c + i, f);
-        if (dst) store8(dst + i, f);
+        store8(dst + i, f);
+      };
+      if (dst) {
+#pragma unroll
+        for (int k = 0; k < LF_KEEP; ++k) {
+          const int i = (k * 32 + lane) * 8;
+          if (i < width) finish(i, kept[k]);
+        }
+        for (int i = rest; i < width; i += 256) {
+          float f[8];
+          load8(c + i, f);
+          finish(i, f);
+        }
       }
     } else {
       const int units = p.rot_pad / 8;
-      for (int u = threadIdx.x - 32; u < p.H * units; u += LF_THREADS - 32) {
+      for (int u = threadIdx.x - 32; u < p.H * units; u += blockDim.x - 32) {
         const int h = u / units, d = (u - h * units) * 8;
         T* q = y + p.q_off + static_cast<long long>(h) * p.q_head + p.q_rot + d;
         float f[8];
@@ -420,20 +442,33 @@ latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
 
 // out[first + i] = cached row of token i of sequence slot, i < n, for every (slot, first, n) of `spans`; zeros up to the next
 // multiple of `pad` rows.
-__global__ void latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table, const int* __restrict__ spans,
-                                     uint4* __restrict__ out, int units, int pad, int block_size, int max_blocks, int num_blocks) {
+constexpr int LG_BATCH = 4;       // units loaded together
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table, const int* __restrict__ spans,
+                     uint4* __restrict__ out, int units, int pad, int block_size, int max_blocks, int num_blocks) {
   const int* span = spans + 3 * blockIdx.y;
-  const int slot = span[0], first = span[1], n = span[2];
-  for (int i = blockIdx.x * blockDim.y + threadIdx.y; i < (n + pad - 1) / pad * pad; i += gridDim.x * blockDim.y) {
-    if (i >= n) {
-      for (int u = threadIdx.x; u < units; u += blockDim.x) out[(static_cast<long long>(first) + i) * units + u] = make_uint4(0u, 0u, 0u, 0u);
-      continue;
+  const int n = span[2];
+  const int* bt = block_table + static_cast<long long>(span[0]) * max_blocks;
+  const long long total = static_cast<long long>((n + pad - 1) / pad * pad) * units;
+  uint4* dst = out + static_cast<long long>(span[1]) * units;
+  for (long long base = static_cast<long long>(blockIdx.x) * 256 * LG_BATCH; base < total; base += static_cast<long long>(gridDim.x) * 256 * LG_BATCH) {
+    uint4 v[LG_BATCH];
+#pragma unroll
+    for (int j = 0; j < LG_BATCH; ++j) {
+      const long long at = base + j * 256 + threadIdx.x;
+      const int i = static_cast<int>(at / units), u = static_cast<int>(at - static_cast<long long>(i) * units);
+      v[j] = make_uint4(0u, 0u, 0u, 0u);
+      if (at < total && i < n) {
+        const int page = i / block_size;
+        const int blk = min(max(page < max_blocks ? __ldg(bt + page) : 0, 0), num_blocks - 1);
+        v[j] = cache[(static_cast<long long>(blk) * block_size + i % block_size) * units + u];
+      }
     }
-    const int page = i / block_size;
-    int blk = page < max_blocks ? __ldg(block_table + static_cast<long long>(slot) * max_blocks + page) : 0;
-    blk = min(max(blk, 0), num_blocks - 1);
-    const uint4* src = cache + (static_cast<long long>(blk) * block_size + i % block_size) * units;
-    for (int u = threadIdx.x; u < units; u += blockDim.x) out[(static_cast<long long>(first) + i) * units + u] = src[u];
+#pragma unroll
+    for (int j = 0; j < LG_BATCH; ++j) {
+      const long long at = base + j * 256 + threadIdx.x;
+      if (at < total) dst[at] = v[j];
+    }
   }
 }
 
@@ -450,7 +485,8 @@ using namespace ft;
 // The pass between a packed projection and its latent attention (see the top of this file): query heads of q_head elements
 // from q_off, their rotated part of rot_pad elements at q_rot; latent and key part of rank_pad + rot_pad from c_off, of
 // which rank and 2 * half exist (padding is zero).  packed and cache bf16, or fp32 with f32; all sizes and offsets multiples of
-// 8.  Rows n_lat .. keep their rotated query parts in place, the rows ahead of them put theirs into q_lat.
+// 8.  Rows n_lat .. keep their rotated query parts in place, the rows ahead of them put theirs into q_lat; the latent and the
+// key part go to the page only.
 FT_API int ft_latent_finish(void* packed, long long ld, void* q_lat, int n_lat, const int* pos, const int* slots, const int* block_table,
                             void* cache, const float* weight, const void* table, int rows, int H, int q_off, int q_head, int q_rot,
                             int c_off, int rank_pad, int rank, int rot_pad, int half, int positions, float eps, int f32, int block_size,
@@ -470,9 +506,11 @@ FT_API int ft_latent_finish(void* packed, long long ld, void* q_lat, int n_lat, 
   p.table = static_cast<const float2*>(table); p.ld = ld; p.rows = rows; p.n_lat = n_lat; p.H = H; p.q_off = q_off; p.q_head = q_head;
   p.q_rot = q_rot; p.c_off = c_off; p.rank_pad = rank_pad; p.rank = rank; p.rot_pad = rot_pad; p.half = half; p.positions = positions;
   p.eps = eps; p.block_size = block_size; p.max_blocks = max_blocks; p.num_blocks = num_blocks;
-  const int cap = sm_count(device) * 16, grid = rows < cap ? rows : cap;
-  if (f32) latent_finish_kernel<float><<<grid, LF_THREADS, 0, stream>>>(p);
-  else latent_finish_kernel<__nv_bfloat16><<<grid, LF_THREADS, 0, stream>>>(p);
+  const int cap = sm_count(device) * 64, grid = rows < cap ? rows : cap;
+  int threads = 32 + (H * (rot_pad / 8) + 31) / 32 * 32;
+  if (threads > LF_MAX_THREADS) threads = LF_MAX_THREADS;
+  if (f32) latent_finish_kernel<float><<<grid, threads, 0, stream>>>(p);
+  else latent_finish_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>(p);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;
@@ -539,11 +577,12 @@ FT_API int ft_latent_gather(const void* cache, const int* block_table, const int
   FT_REQUIRE(cache && block_table && spans && out && row_bytes > 0 && row_bytes % 16 == 0 && pad > 0 && la_aligned({cache, out}), "ft_latent_gather: null or unaligned pointer");
   FT_REQUIRE(block_size > 0 && max_blocks > 0 && num_blocks > 0 && n_spans < 65536, "ft_latent_gather: bad shape");
   if (n_spans <= 0 || longest <= 0) return FT_E_OK;
-  int gx = (longest + 3) / 4;
-  const int cap = sm_count(device) * 16 / n_spans + 1;
+  const long long most = static_cast<long long>((longest + pad - 1) / pad * pad) * (row_bytes / 16);
+  long long gx = (most + 256 * LG_BATCH - 1) / (256 * LG_BATCH);
+  const long long cap = sm_count(device) * 32ll / n_spans + 1;
   if (gx > cap) gx = cap;
-  latent_gather_kernel<<<dim3(gx, n_spans), dim3(64, 4), 0, stream>>>(static_cast<const uint4*>(cache), block_table, spans,
-                                                                      static_cast<uint4*>(out), row_bytes / 16, pad, block_size, max_blocks, num_blocks);
+  latent_gather_kernel<<<dim3(static_cast<unsigned>(gx), n_spans), 256, 0, stream>>>(static_cast<const uint4*>(cache), block_table, spans,
+                                                                                     static_cast<uint4*>(out), row_bytes / 16, pad, block_size, max_blocks, num_blocks);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

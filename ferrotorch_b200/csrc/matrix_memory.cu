@@ -471,26 +471,28 @@ memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
 }
 
 // Outputs of one (chunk, head).  Warps 0-3: thread = token.  Warp 4: copies and products.  Shared memory: Q | K, then the low half
-// of the state | the high half of the state, then V.
+// of the state | the high half of the state, then V; at the end the gate lies over Q (and what follows), and the results over it.
 template <int DC, int VC>
 struct MemOut {
   static constexpr int MID = DC > VC ? DC : VC;
   static constexpr int OFF_K = DC * MC_CHUNK, OFF_V = OFF_K + MID * MC_CHUNK, OFF_A = OFF_V + VC * MC_CHUNK, OFF_NB = OFF_A + MC_ROWS * 4,
-                       OFF_BAR = OFF_NB + 128 * 4, SMEM = OFF_BAR + 128 + 1024;
+                       OFF_W = OFF_NB + 128 * 4, OFF_BAR = OFF_W + VC * 64 * 4, SMEM = OFF_BAR + 128 + 1024;
   static constexpr uint32_t COLS = VC <= 2 ? 256 : 512, COL_LOW = 64, COL_O = 128;      // scores (then P high | low), outputs
 };
 
 template <int DC, int VC>
 __global__ void __launch_bounds__(MC_OUT_THREADS)
 memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                     const __grid_constant__ CUtensorMap tmS, const MemoryParams p, const MemoryChunks c) {
+                     const __grid_constant__ CUtensorMap tmS, const __grid_constant__ CUtensorMap tmG, const MemoryParams p,
+                     const MemoryChunks c) {
   using Cfg = MemOut<DC, VC>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t sQ = smem_u32(smem), sK = sQ + Cfg::OFF_K, sV = sQ + Cfg::OFF_V;
   float* s_a = reinterpret_cast<float*>(smem + Cfg::OFF_A);
   float* s_nb = reinterpret_cast<float*>(smem + Cfg::OFF_NB);
-  enum { QK = 0, HIGH, LOW, V, SCORE, HIGH_DONE, INTER, P_FULL, OUT, NBARS };
+  float* s_w = reinterpret_cast<float*>(smem + Cfg::OFF_W);
+  enum { QK = 0, HIGH, LOW, V, SCORE, HIGH_DONE, INTER, Q_READ, P_FULL, GATE, OUT, NBARS };
   auto bar = [&](int i) { return sQ + Cfg::OFF_BAR + 8u * i; };
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + Cfg::OFF_BAR + 8 * NBARS);
   volatile int* abort_word = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -502,7 +504,7 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const long long ph = static_cast<long long>(blockIdx.x) * p.H + h, gate_at = static_cast<long long>(h) * c.ldt + row0;
   if (tid == 0) {
     *abort_word = 0;
-    for (int i = 0; i < NBARS; ++i) mbar_init(bar(i), i == P_FULL ? 4 : 1);
+    for (int i = 0; i < NBARS; ++i) mbar_init(bar(i), i == P_FULL || i == Q_READ ? 4 : 1);
     fence_mbar_init();
   }
   if (warp == 4) {
@@ -511,6 +513,7 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   }
   if (tid < MC_ROWS) s_a[tid] = tid < rows ? c.a2[gate_at + tid] : -INFINITY;
   if (tid < p.dp) s_nb[tid] = fresh ? 0.f : c.nb[ph * p.dp + tid];
+  for (int i = tid; i < p.vp; i += MC_OUT_THREADS) s_w[i] = p.norm[static_cast<long long>(h) * p.vp + i];
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -563,6 +566,11 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
           umma_commit(bar(INTER));
         }
       }
+      // the last product with Q has finished and every token has read its own: the gate takes the place
+      if (ok && p.gate && (ok = wait(fresh ? SCORE : INTER)) && (ok = wait(Q_READ))) {
+        mbar_expect_tx(bar(GATE), VC * MC_CHUNK);
+        for (int i = 0; i < VC; ++i) tma_load_2d(sQ + i * MC_CHUNK, &tmG, bar(GATE), h * p.vp + i * 64, row0);
+      }
       if (ok && (ok = wait(V)) && (ok = wait(P_FULL))) {
         tc_fence_after();
 #pragma unroll
@@ -582,21 +590,22 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const bool row_ok = tid < rows;
     const float x2 = row_ok ? c.x2[gate_at + tid] : 0.f, floor_m = row_ok ? c.floor[gate_at + tid] : 1.f;
     const float inter = (fresh || !row_ok) ? 0.f : exp2f(c.start2[ph] - x2) * p.q_scale;
-    const long long row = static_cast<long long>(row0) + (row_ok ? tid : 0);
     const uint32_t lane_addr = tmem + (static_cast<uint32_t>(warp * 32) << 16);
     float den = 0.f;
-    if (!fresh) {                                      // q times the normaliser at the chunk's start
-      const __nv_bfloat16* q_row = static_cast<const __nv_bfloat16*>(p.q) + row * p.ld + static_cast<long long>(h) * p.dp;
-      for (int d = 0; d < p.dp; d += 8) {
+    auto wait = [&](int i) { return __all_sync(0xffffffffu, mbar_wait(bar(i), 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE)); };
+    bool ok = wait(QK);
+    if (ok && !fresh) {                                // q times the normaliser at the chunk's start
+      for (int u = 0; u < p.dp / 8; ++u) {
         float f[8];
-        load8(q_row + d, f);
+        unpack8(*reinterpret_cast<const uint4*>(smem + mc_unit(tid, u)), f);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) den += f[e] * s_nb[d + e];
+        for (int e = 0; e < 8; ++e) den += f[e] * s_nb[u * 8 + e];
       }
       den *= inter;
     }
-    auto wait = [&](int i) { return __all_sync(0xffffffffu, mbar_wait(bar(i), 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE)); };
-    bool ok = wait(SCORE);
+    __syncwarp();
+    if (ok && lane == 0) mbar_arrive(bar(Q_READ));
+    ok = ok && wait(SCORE);
     if (ok) {
       tc_fence_after();
       uint32_t lows[2][16];                            // low halves of the first two groups wait until their scores' place is free
@@ -676,31 +685,34 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         }
       }
       const float r = p.out_scale * inv / sqrtf(sum / static_cast<float>(p.vdim) + p.eps);
-      const __nv_bfloat16* g_row = static_cast<const __nv_bfloat16*>(p.gate) + row * p.ld + static_cast<long long>(h) * p.vp;
-      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.vp;
-      const float* norm = p.norm + static_cast<long long>(h) * p.vp;
+      if (p.gate) ok = wait(GATE);
 #pragma unroll 1
       for (int col = 0; col < VC * 64; col += 32) {
         if (col >= p.vp) break;
         uint32_t t[32];
         tmem_ld_32x32(lane_addr + Cfg::COL_O + col, t);
         tmem_ld_wait();
-        if (!row_ok) continue;
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
-          const int j = col + g * 8;
-          if (j >= p.vp) continue;
-          float f[8], w[8], z[8];
-          load8(norm + j, w);
+          uint4* at = reinterpret_cast<uint4*>(smem + mc_unit(tid, col / 8 + g));
+          float f[8], z[8];
 #pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]) * r * w[e];
+          for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]) * r * s_w[col + g * 8 + e];
           if (p.gate) {
-            load8(g_row + j, z);
+            unpack8(*at, z);
 #pragma unroll
             for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-z[e]));
           }
-          store8(out + j, f);
+          *at = pack8(f);
         }
+      }
+      __syncwarp();
+      // the warp's rows, contiguous pieces of a row by neighbouring lanes
+      const int units = p.vp / 8, live = min(32, rows - warp * 32) * units;
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (static_cast<long long>(row0) + warp * 32) * p.ldo + static_cast<long long>(h) * p.vp;
+      for (int i = lane; ok && i < live; i += 32) {
+        const int rr = i / units, u = i - rr * units;
+        *reinterpret_cast<uint4*>(out + rr * p.ldo + u * 8) = *reinterpret_cast<const uint4*>(smem + mc_unit(warp * 32 + rr, u));
       }
     }
   }
@@ -787,8 +799,8 @@ static long long memory_scratch_at(int rows, int H, int dp, int vp, int n_chunks
 FT_API long long ft_memory_scratch(int rows, int H, int dp, int vp, int n_chunks) { return memory_scratch_at(rows, H, dp, vp, n_chunks, nullptr); }
 
 template <int DC, int VC>
-static int launch_memory(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const MemoryParams& p,
-                         const MemoryChunks& c, int device, cudaStream_t stream) {
+static int launch_memory(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const CUtensorMap& tg,
+                         const MemoryParams& p, const MemoryChunks& c, int device, cudaStream_t stream) {
   constexpr int UPDATE_SMEM = (4 + VC) * MC_CHUNK + 16 * 128 * 4 + MC_ROWS * 4 + 64 + 1024;
   constexpr int OUT_SMEM = MemOut<DC, VC>::SMEM;
   static bool attr_set[64] = {false};
@@ -803,7 +815,7 @@ static int launch_memory(const CUtensorMap& tq, const CUtensorMap& tk, const CUt
   FT_CUDA_CHECK(cudaGetLastError());
   memory_carry_kernel<<<dim3((p.dp * c.vw / 4 + 255) / 256, p.H, c.n_spans), 256, 0, stream>>>(p, c);
   FT_CUDA_CHECK(cudaGetLastError());
-  memory_output_kernel<DC, VC><<<dim3(c.n_chunks, p.H), MC_OUT_THREADS, OUT_SMEM, stream>>>(tq, tk, tv, ts, p, c);
+  memory_output_kernel<DC, VC><<<dim3(c.n_chunks, p.H), MC_OUT_THREADS, OUT_SMEM, stream>>>(tq, tk, tv, ts, tg, p, c);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch(4);
   return FT_E_OK;
@@ -832,18 +844,19 @@ FT_API int ft_memory_chunks(const void* q, const void* k, const void* v, const v
   c.Un = reinterpret_cast<float*>(base + at[6]); c.Sb = reinterpret_cast<__nv_bfloat16*>(base + at[7]); c.nb = reinterpret_cast<float*>(base + at[8]);
   c.ldt = (rows + 31) / 32 * 32; c.n_spans = n_spans; c.n_chunks = n_chunks; c.vw = (vp + 63) / 64 * 64;
   c.status = device_status_word(device);
-  CUtensorMap tq, tk, tv, ts;
+  CUtensorMap tq, tk, tv, ts, tg;
   const uint64_t stride = static_cast<uint64_t>(ld) * 2;
   if (int rc = make_tmap_2d(&tq, q, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
   if (int rc = make_tmap_2d(&tk, k, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
   if (int rc = make_tmap_2d(&tv, v, 2, static_cast<uint64_t>(H) * vp, rows, stride, 64, MC_ROWS, 3)) return rc;
+  if (int rc = make_tmap_2d(&tg, gate ? gate : v, 2, static_cast<uint64_t>(H) * vp, rows, stride, 64, MC_ROWS, 3)) return rc;
   if (int rc = make_tmap_2d(&ts, c.Sb, 2, c.vw, 2 * static_cast<uint64_t>(n_chunks) * H * dp, static_cast<uint64_t>(c.vw) * 2, 64, dp, 3)) return rc;
 #define FT_MC(DCN)                                                              \
   switch (c.vw / 64) {                                                          \
-    case 1: return launch_memory<DCN, 1>(tq, tk, tv, ts, p, c, device, stream); \
-    case 2: return launch_memory<DCN, 2>(tq, tk, tv, ts, p, c, device, stream); \
-    case 3: return launch_memory<DCN, 3>(tq, tk, tv, ts, p, c, device, stream); \
-    default: return launch_memory<DCN, 4>(tq, tk, tv, ts, p, c, device, stream); \
+    case 1: return launch_memory<DCN, 1>(tq, tk, tv, ts, tg, p, c, device, stream); \
+    case 2: return launch_memory<DCN, 2>(tq, tk, tv, ts, tg, p, c, device, stream); \
+    case 3: return launch_memory<DCN, 3>(tq, tk, tv, ts, tg, p, c, device, stream); \
+    default: return launch_memory<DCN, 4>(tq, tk, tv, ts, tg, p, c, device, stream); \
   }
   if (dp <= 64) { FT_MC(1) }
   FT_MC(2)

@@ -97,7 +97,7 @@ class AttentionMemoryMixer(nn.Module):
         """The sublayer's output for input ``h``; ``layer``: the attention's place in the cache; carries ``state`` on."""
         a, m, at = self.attn, self.memory, self.offsets
         packed = F.linear_rows(h, self.in_proj)
-        z = F.linear_f32_out(h, self.gate_proj)
+        z = D.few_outputs(h, self.gate_proj)
         D.qkv_head_finish(packed, cache, layer, batch, heads=a.heads, dim=a.padded_dim, q_off=at["left.q"], k_off=at["left.k"], v_off=at["left.v"],
                           q_weight=self.ones, k_weight=self.ones, true_dim=a.dim, eps=self.eps)
         heads = torch.empty((h.shape[0], self.left_width + self.right_width), device=h.device, dtype=h.dtype)

@@ -27,6 +27,7 @@ _native.register_protos({
     "ft_moe_max_items": (_i, [_i, _i]),
     "ft_moe_route": (_i, [_vp, _ll, _vp, _vp, _ll] + [_i] * 6 + [_vp, _i, _i] + [_vp] * 5 + [_i, _vp, _vp, _i, _vp]),
     "ft_block_linear": (_i, [_vp, _ll, _i, _vp] + [_i] * 6 + [_vp, _ll, _i, _vp, _ll] + [_i] * 3 + [_vp]),
+    "ft_few_outputs": (_i, [_vp, _ll, _vp, _vp] + [_i] * 5 + [_vp]),
     "ft_stream_step": (_i, [_vp, _ll, _ll, _vp, _i] + [_vp] * 4 + [_i, _vp, _ll, _vp, _ll, _i, _vp, _vp, _i, _vp, _ll, _vp, _vp, _ll] + [_i] * 3 + [_f, _i, _i, _vp]),
     "ft_embed_bigram": (_i, [_vp] * 8 + [_ll, _i, _i, _ll, _ll, _f, _vp, _i] + [_vp] * 3 + [_i] * 3 + [_f] + [_i] * 5 + [_vp]),
     "ft_softcap": (_i, [_vp, _ll, _f, _i, _vp]),
@@ -213,8 +214,8 @@ def latent_finish(packed: torch.Tensor, cache, layer: int, batch, *, heads: int,
                   rank_pad: int, weight: torch.Tensor, eps: float, table: torch.Tensor, q_lat: torch.Tensor | None = None) -> None:
     """Everything between a packed projection and its latent attention, in one kernel: RMS norm of the latent (``rank`` of ``rank_pad``
     elements at ``c_off``, ``weight [rank_pad]``), rotation of the key part behind it and of the part at ``q_rot`` of every query
-    head (heads of ``q_head`` elements from ``q_off``; pairs of neighbours, ``table [positions, half, 2]``), the row into its page.
-    Latent and key part change in place; so do the queries, except that the first rows' rotated parts go to ``q_lat [rows, heads,
+    head (heads of ``q_head`` elements from ``q_off``; pairs of neighbours, ``table [positions, half, 2]``), the row into its page
+    (and nowhere else).  The queries change in place, except that the first rows' rotated parts go to ``q_lat [rows, heads,
     rank_pad + rot_pad]``, behind the place of their latent part."""
     width = cache.shapes[layer][1]
     rot_pad, half = width - rank_pad, table.shape[1]
@@ -224,7 +225,6 @@ def latent_finish(packed: torch.Tensor, cache, layer: int, batch, *, heads: int,
         row = packed[:, c_off:c_off + width].float()
         c = ref.rms_rows(row[:, :rank_pad], weight, eps, rank)
         row = torch.cat([c, ref.rotate_pairs(row[:, None, rank_pad:], table, batch.positions)[:, 0]], 1).to(packed.dtype)
-        packed[:, c_off:c_off + width] = row
         pos = batch.positions.long()
         cache.k[layer][cache._table_host[batch.slots.long(), pos // cache.block_size].long(), pos % cache.block_size, 0] = row
         q = packed[:, q_off:q_off + heads * q_head].unflatten(1, (heads, q_head))[:, :, q_rot:q_rot + rot_pad]
@@ -264,6 +264,18 @@ def block_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, a_col: 
         out.stride(0), out_col, _ptr(gate), gate.stride(0) if gate is not None else 0, int(a.dtype == torch.float32), bn, F._dev(a), F._stream())
     _native.check(rc, "ft_block_linear")
     return out
+
+
+def few_outputs(h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``h @ w.T`` with fp32 results for a few outputs: small batches on a kernel of their own, large ones as an ordinary product."""
+    T, H = h.shape
+    if not h.is_cuda or T > ROUTE_ROWS or w.shape[0] > 256:
+        return F.linear_f32_out(h, w)
+    z = torch.empty((T, w.shape[0]), device=h.device, dtype=torch.float32)
+    rc = _native.kernels().ft_few_outputs(h.data_ptr(), h.stride(0), w.data_ptr(), z.data_ptr(), T, H, w.shape[0], int(h.dtype == torch.float32), F._dev(h),
+                                          F._stream())
+    _native.check(rc, "ft_few_outputs")
+    return z
 
 
 # --------------------------------------------------------------------------- recurrent blocks

@@ -355,7 +355,7 @@ def test_latent_finish_kernel(heads, dim, rot, dims, rank, dtype):
             D.latent_finish(t, c, 0, RaggedBatch(entries, dev), heads=heads, q_off=0, q_head=spec.head_size, q_rot=spec.padded_dim, c_off=qw, rank=rank,
                             rank_pad=spec.padded_rank, weight=weight.to(dev), eps=1e-3, table=table.to(dev), q_lat=ql)
         tol = dict(atol=2e-5, rtol=1e-5) if dtype == "fp32" else dict(atol=3e-2, rtol=1e-2)
-        assert torch.allclose(p[:, qw:].cpu().float(), r[:, qw:].float(), **tol) and torch.allclose(p[n_lat:, :qw].cpu().float(), r[n_lat:, :qw].float(), **tol)
+        assert torch.equal(p[:, qw:].cpu(), ref[:, qw:]) and torch.allclose(p[n_lat:, :qw].cpu().float(), r[n_lat:, :qw].float(), **tol)
         assert torch.allclose(lat[0].cpu().float(), lat[1].float(), **tol) and torch.allclose(caches[0].k[0].cpu().float(), caches[1].k[0].float(), **tol)
 
 
@@ -401,6 +401,8 @@ def test_products_by_blocks(T, G, K, N, a_col, out_col, bn, dtype):
                 want = want * torch.sigmoid(gate[:, g * out_col:g * out_col + N].double())
             assert torch.allclose(out[:, g * out_col:g * out_col + N].double(), want, **tol), g
             assert bool((out[:, g * out_col + N:(g + 1) * out_col] == 7.0).all())
+    few = D.few_outputs(a[:, :K].contiguous(), w[0, 0, :9])
+    assert few.dtype == torch.float32 and torch.allclose(few.double(), a[:, :K].double() @ w[0, 0, :9].double().t(), atol=1e-4)
     w2 = _rnd(1, 2, N, K, std=K ** -0.5, dtype=dt)
     out = D.block_linear(a[:, :K], w2, torch.empty(T, N, device="cuda", dtype=dt), glu="silu", bn=bn)
     z = a[:, :K].double()

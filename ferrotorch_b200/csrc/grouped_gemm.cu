@@ -501,10 +501,13 @@ __device__ __forceinline__ void row_outputs(const T* h, const T* __restrict__ w,
   }
 }
 
+constexpr int FEW_OUTPUTS = MR_THREADS / 16;       // of a block: two a warp
 template <typename T>
 __global__ void __launch_bounds__(MR_THREADS)
 few_outputs_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, float* __restrict__ z, int rows, int H, int n) {
-  for (int row = blockIdx.x; row < rows; row += gridDim.x) row_outputs(h + row * ldh, w, H, n, z + static_cast<long long>(row) * n);
+  const int e0 = blockIdx.y * FEW_OUTPUTS, m = min(FEW_OUTPUTS, n - e0);
+  for (int row = blockIdx.x; row < rows; row += gridDim.x)
+    row_outputs(h + row * ldh, w + static_cast<long long>(e0) * H, H, m, z + static_cast<long long>(row) * n + e0);
 }
 
 // One block per row: the row in registers of all warps in turn, one expert per warp at a time.
@@ -652,7 +655,8 @@ FT_API int ft_few_outputs(const void* h, long long ldh, const void* w, float* z,
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(h && w && z && H > 0 && H % 8 == 0 && ldh % 8 == 0 && n > 0 && gg_aligned({h, w}), "ft_few_outputs: H=%d and strides must be multiples of 8", H);
   if (rows <= 0) return FT_E_OK;
-  const int cap = sm_count(device) * 8, grid = rows < cap ? rows : cap;
+  const int cap = sm_count(device) * 8;
+  const dim3 grid(rows < cap ? rows : cap, (n + FEW_OUTPUTS - 1) / FEW_OUTPUTS);
   if (f32) few_outputs_kernel<float><<<grid, MR_THREADS, 0, stream>>>(static_cast<const float*>(h), ldh, static_cast<const float*>(w), z, rows, H, n);
   else few_outputs_kernel<__nv_bfloat16><<<grid, MR_THREADS, 0, stream>>>(static_cast<const __nv_bfloat16*>(h), ldh, static_cast<const __nv_bfloat16*>(w), z, rows, H, n);
   FT_CUDA_CHECK(cudaGetLastError());

@@ -16,7 +16,7 @@
 // A tile of 576 columns takes 144 KB, so there is one; its pieces are ring slots of their own: a piece is loaded again as soon as
 // the last product that reads it has finished, while the others are still in use.
 //   warp 0  producer: one TMA box per page and piece     warp 1  MMA issuer     warp 2  TMEM allocator
-//   warps 4-7  softmax (thread = key) and epilogue (thread = latent column)
+//   warps 4-   softmax (thread = key) and epilogue (thread = latent column), four warps for every 16 heads
 // All waits are bounded and report through the device status word.
 #include <initializer_list>
 
@@ -24,7 +24,8 @@
 
 namespace ft {
 
-constexpr int LF_MAX_THREADS = 256;
+constexpr int LF_ROWS = 4;        // rows of a block
+constexpr int LF_MAX_THREADS = 32 * LF_ROWS + 256;
 constexpr int LF_KEEP = 3;        // vectors of eight elements of the latent that a lane keeps
 
 struct LatentFinishParams {
@@ -56,81 +57,93 @@ __device__ __forceinline__ void rotate8(float (&f)[8], int d, const float2* cs, 
   }
 }
 
-// One block per row: the first warp takes the latent and the key part, the others the queries.
+// A block takes LF_ROWS rows: one warp each for their latents and key parts, the other threads their queries (a thread the same
+// place of every row, all loads in flight together).
 template <typename T>
 __global__ void __launch_bounds__(LF_MAX_THREADS)
 latent_finish_kernel(const LatentFinishParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int width = p.rank_pad + p.rot_pad;
-  for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
-    T* y = static_cast<T*>(p.packed) + static_cast<long long>(row) * p.ld;
-    const int position = p.pos[row];
-    const float2* cs = p.table + static_cast<long long>(min(position, p.positions - 1)) * p.half;
-    if (warp == 0) {
-      const T* c = y + p.c_off;
-      float kept[LF_KEEP][8];
-      float sum = 0.f;
+  const int row0 = blockIdx.x * LF_ROWS;
+  auto angles = [&](int row) { return p.table + static_cast<long long>(min(p.pos[row], p.positions - 1)) * p.half; };
+  if (warp < LF_ROWS) {
+    const int row = row0 + warp;
+    if (row >= p.rows) return;
+    const T* c = static_cast<const T*>(p.packed) + static_cast<long long>(row) * p.ld + p.c_off;
+    float kept[LF_KEEP][8];
+    float sum = 0.f;
 #pragma unroll
-      for (int k = 0; k < LF_KEEP; ++k) {
-        const int i = (k * 32 + lane) * 8;
-        if (i < width) load8(c + i, kept[k]);
+    for (int k = 0; k < LF_KEEP; ++k) {
+      const int i = (k * 32 + lane) * 8;
+      if (i < width) load8(c + i, kept[k]);
+    }
+    const int position = p.pos[row], page = position / p.block_size;
+    const float2* cs = angles(row);
+    const int blk = page < p.max_blocks ? p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + page] : -1;
+    if (blk < 0 || blk >= p.num_blocks) return;        // a row of no sequence
+    T* dst = static_cast<T*>(p.cache) + (static_cast<long long>(blk) * p.block_size + position % p.block_size) * width;
+#pragma unroll
+    for (int k = 0; k < LF_KEEP; ++k)
+      if ((k * 32 + lane) * 8 < p.rank_pad)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += kept[k][e] * kept[k][e];
+    const int rest = (LF_KEEP * 32 + lane) * 8;        // wider rows are read twice
+    for (int i = rest; i < p.rank_pad; i += 256) {
+      float f[8];
+      load8(c + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum += f[e] * f[e];
+    }
+    const float r = 1.f / sqrtf(warp_sum(sum) / static_cast<float>(p.rank) + p.eps);
+    auto finish = [&](int i, float (&f)[8]) {
+      if (i < p.rank_pad) {
+        float w[8];
+        load8(p.weight + i, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] *= r * w[e];
+      } else {
+        rotate8(f, i - p.rank_pad, cs, p.half);
       }
-      const int page = position / p.block_size;
-      const int blk = page < p.max_blocks ? p.block_table[static_cast<long long>(p.slots[row]) * p.max_blocks + page] : -1;
-      T* dst = blk >= 0 && blk < p.num_blocks
-                   ? static_cast<T*>(p.cache) + (static_cast<long long>(blk) * p.block_size + position % p.block_size) * width : nullptr;
+      store8(dst + i, f);
+    };
 #pragma unroll
-      for (int k = 0; k < LF_KEEP; ++k)
-        if ((k * 32 + lane) * 8 < p.rank_pad)
+    for (int k = 0; k < LF_KEEP; ++k) {
+      const int i = (k * 32 + lane) * 8;
+      if (i < width) finish(i, kept[k]);
+    }
+    for (int i = rest; i < width; i += 256) {
+      float f[8];
+      load8(c + i, f);
+      finish(i, f);
+    }
+  } else {
+    const int units = p.rot_pad / 8;
+    for (int u = threadIdx.x - 32 * LF_ROWS; u < p.H * units; u += blockDim.x - 32 * LF_ROWS) {
+      const int h = u / units, d = (u - h * units) * 8;
+      float f[LF_ROWS][8];
+      const float2* cs[LF_ROWS];
+      T* q[LF_ROWS];
 #pragma unroll
-          for (int e = 0; e < 8; ++e) sum += kept[k][e] * kept[k][e];
-      const int rest = (LF_KEEP * 32 + lane) * 8;      // wider rows are read twice
-      for (int i = rest; i < p.rank_pad; i += 256) {
-        float f[8];
-        load8(c + i, f);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) sum += f[e] * f[e];
+      for (int k = 0; k < LF_ROWS; ++k) {              // past the end: the last row again, not stored
+        const int row = min(row0 + k, p.rows - 1);
+        q[k] = static_cast<T*>(p.packed) + static_cast<long long>(row) * p.ld + p.q_off + static_cast<long long>(h) * p.q_head + p.q_rot + d;
+        load8(q[k], f[k]);
+        cs[k] = angles(row);
       }
-      const float r = 1.f / sqrtf(warp_sum(sum) / static_cast<float>(p.rank) + p.eps);
-      auto finish = [&](int i, float (&f)[8]) {
-        if (i < p.rank_pad) {
-          float w[8];
-          load8(p.weight + i, w);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] *= r * w[e];
-        } else {
-          rotate8(f, i - p.rank_pad, cs, p.half);
-        }
-        store8(dst + i, f);
-      };
-      if (dst) {
+      for (int k = 0; k < LF_ROWS; ++k) rotate8(f[k], d, cs[k], p.half);
 #pragma unroll
-        for (int k = 0; k < LF_KEEP; ++k) {
-          const int i = (k * 32 + lane) * 8;
-          if (i < width) finish(i, kept[k]);
-        }
-        for (int i = rest; i < width; i += 256) {
-          float f[8];
-          load8(c + i, f);
-          finish(i, f);
-        }
-      }
-    } else {
-      const int units = p.rot_pad / 8;
-      for (int u = threadIdx.x - 32; u < p.H * units; u += blockDim.x - 32) {
-        const int h = u / units, d = (u - h * units) * 8;
-        T* q = y + p.q_off + static_cast<long long>(h) * p.q_head + p.q_rot + d;
-        float f[8];
-        load8(q, f);
-        rotate8(f, d, cs, p.half);
-        store8(row < p.n_lat ? static_cast<T*>(p.q_lat) + (static_cast<long long>(row) * p.H + h) * width + p.rank_pad + d : q, f);
+      for (int k = 0; k < LF_ROWS; ++k) {
+        const int row = row0 + k;
+        if (row < p.rows)
+          store8(row < p.n_lat ? static_cast<T*>(p.q_lat) + (static_cast<long long>(row) * p.H + h) * width + p.rank_pad + d : q[k], f[k]);
       }
     }
   }
 }
 
 // ---------------------------------------------------------------- decode
-constexpr int LD_THREADS = 256;
+constexpr int LD_GROUP = 16;               // heads of a softmax group
 constexpr int LD_TILE = 128;               // keys
 constexpr int LD_PIECE = LD_TILE * 128;    // bytes of 64 columns
 constexpr int LD_MAX_PIECES = 9;
@@ -138,11 +151,13 @@ constexpr float LD_RESCALE = 8.f;
 
 template <int N>
 struct LdCfg {
+  static constexpr int GROUPS = N / LD_GROUP;
+  static constexpr int THREADS = 128 + 128 * GROUPS;
   static constexpr int Q_PIECE = N * 128;
   static constexpr int P_BYTES = 2 * N * 128;             // two pieces of 64 keys
   static constexpr int OFF_Q = LD_MAX_PIECES * LD_PIECE;
   static constexpr int OFF_P = OFF_Q + LD_MAX_PIECES * Q_PIECE;
-  static constexpr int OFF_RED = OFF_P + P_BYTES;         // [4 warps][N] floats, then [N] references
+  static constexpr int OFF_RED = OFF_P + P_BYTES;         // per group [4 warps][16] floats, then [16] references
   static constexpr int OFF_BAR = OFF_RED + 5 * N * 4;
   static constexpr int SMEM_BYTES = OFF_BAR + 256 + 1024;
   static constexpr uint32_t TMEM_COLS = N * 5 <= 128 ? 128 : 256;
@@ -164,14 +179,12 @@ struct LatentDecodeParams {
 };
 
 template <int N>
-__global__ void __launch_bounds__(LD_THREADS, 1)
+__global__ void __launch_bounds__(LdCfg<N>::THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecodeParams p) {
   using Cfg = LdCfg<N>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t sbase = smem_u32(smem);
-  float* s_red = reinterpret_cast<float*>(smem + Cfg::OFF_RED);
-  float* s_ref = s_red + 4 * N;
   enum { FULL = 0, EMPTY = FULL + LD_MAX_PIECES, S_FULL = EMPTY + LD_MAX_PIECES, P_FULL, O_DONE, NBARS };
   const uint32_t bar0 = sbase + Cfg::OFF_BAR;
   auto bar = [&](int i) { return bar0 + 8u * i; };
@@ -192,7 +205,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
       mbar_init(bar(EMPTY + i), 1);
     }
     mbar_init(bar(S_FULL), 1);
-    mbar_init(bar(P_FULL), 4);
+    mbar_init(bar(P_FULL), 4 * Cfg::GROUPS);
     mbar_init(bar(O_DONE), 1);
     fence_mbar_init();
     tma_prefetch_desc(&tmC);
@@ -202,7 +215,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     tmem_relinquish();
   }
   // the queries as the B operand (rows past the heads and columns past the width zero)
-  for (int i = threadIdx.x; i < N * LD_MAX_PIECES * 8; i += LD_THREADS) {
+  for (int i = threadIdx.x; i < N * LD_MAX_PIECES * 8; i += Cfg::THREADS) {
     const int h = i / (LD_MAX_PIECES * 8), u = i - h * (LD_MAX_PIECES * 8);
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
     if (h < heads && u * 8 < p.width) v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(b) * p.H + h0 + h) * p.width + u * 8);
@@ -271,39 +284,43 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     }
   } else if (warp >= 4) {
     // ------------------------------------------------------------------ softmax / epilogue
-    const int ew = warp & 3, r = ew * 32 + lane;
+    constexpr int G = LD_GROUP;
+    const int ew = warp & 3, r = ew * 32 + lane, group = (warp - 4) >> 2, hg = group * G;    // first head of the group
+    float* s_red = reinterpret_cast<float*>(smem + Cfg::OFF_RED) + group * 5 * G;
+    float* s_ref = s_red + 4 * G;
+    auto group_sync = [&]() { asm volatile("bar.sync %0, 128;" ::"r"(1 + group) : "memory"); };
     const uint32_t lane_addr = tmem + (static_cast<uint32_t>(ew * 32) << 16);
-    float l_part[N];
+    float l_part[G];
 #pragma unroll
-    for (int g = 0; g < N; ++g) l_part[g] = 0.f;
-    if (r < N) s_ref[r] = -INFINITY;
+    for (int g = 0; g < G; ++g) l_part[g] = 0.f;
+    if (r < G) s_ref[r] = -INFINITY;
     bool ok = true;
     // every thread runs every iteration down to the named barriers, also after a failed wait
     for (int t = 0; t < n_tiles; ++t) {
       if (ok && !mbar_wait(bar(S_FULL), t & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) ok = false;
       ok = __all_sync(0xffffffffu, ok);
-      float s[N];
+      float s[G];
       {
-        uint32_t raw[N];
+        uint32_t raw[G];
 #pragma unroll
-        for (int g = 0; g < N; ++g) raw[g] = 0u;
+        for (int g = 0; g < G; ++g) raw[g] = 0u;
         if (ok) {
           tc_fence_after();
 #pragma unroll
-          for (int g = 0; g < N; g += 16) tmem_ld_32x16(lane_addr + COL_S + g, *reinterpret_cast<uint32_t(*)[16]>(&raw[g]));
+          for (int g = 0; g < G; g += 16) tmem_ld_32x16(lane_addr + COL_S + hg + g, *reinterpret_cast<uint32_t(*)[16]>(&raw[g]));
           tmem_ld_wait();
         }
         const bool valid = (tile_lo + t) * LD_TILE + r < len;
 #pragma unroll
-        for (int g = 0; g < N; ++g) s[g] = valid ? __uint_as_float(raw[g]) * p.scale_log2 : -INFINITY;
+        for (int g = 0; g < G; ++g) s[g] = valid ? __uint_as_float(raw[g]) * p.scale_log2 : -INFINITY;
       }
       // maxima over the warp's keys: halve the heads a lane holds while doubling the keys it covers; lane g ends with head g
       {
-        float v[N];
+        float v[G];
 #pragma unroll
-        for (int g = 0; g < N; ++g) v[g] = s[g];
+        for (int g = 0; g < G; ++g) v[g] = s[g];
 #pragma unroll
-        for (int w = N / 2; w >= 1; w >>= 1) {
+        for (int w = G / 2; w >= 1; w >>= 1) {
           const bool upper = lane & w;
 #pragma unroll
           for (int g = 0; g < w; ++g) {
@@ -311,23 +328,23 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
             v[g] = fmaxf(keep, __shfl_xor_sync(0xffffffffu, send, w));
           }
         }
-        if (N == 16) v[0] = fmaxf(v[0], __shfl_xor_sync(0xffffffffu, v[0], 16));
-        if (lane < N) s_red[ew * N + lane] = v[0];
+        v[0] = fmaxf(v[0], __shfl_xor_sync(0xffffffffu, v[0], 16));
+        if (lane < G) s_red[ew * G + lane] = v[0];
       }
-      asm volatile("bar.sync 1, 128;" ::: "memory");
+      group_sync();
       // every thread makes the same decision; the references are replaced after all have read them
-      const float tile_max = lane < N ? fmaxf(fmaxf(s_red[lane], s_red[N + lane]), fmaxf(s_red[2 * N + lane], s_red[3 * N + lane])) : -INFINITY;
-      const float old_ref = lane < N ? s_ref[lane] : 0.f;
-      const bool moves = lane < N && tile_max > old_ref + LD_RESCALE;
+      const float tile_max = lane < G ? fmaxf(fmaxf(s_red[lane], s_red[G + lane]), fmaxf(s_red[2 * G + lane], s_red[3 * G + lane])) : -INFINITY;
+      const float old_ref = lane < G ? s_ref[lane] : 0.f;
+      const bool moves = lane < G && tile_max > old_ref + LD_RESCALE;
       const float my_ref = moves ? tile_max : old_ref, my_alpha = moves ? fast_exp2(old_ref - tile_max) : 1.f;   // first tile: 0
       const bool any = __any_sync(0xffffffffu, moves);
       // O of the earlier tiles and the P buffer are free once the products of tile t - 1 have finished
       if (t > 0 && ok && !mbar_wait(bar(O_DONE), (t - 1) & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE)) ok = false;
       ok = __all_sync(0xffffffffu, ok);
       if (any) {
-        float alpha[N];
+        float alpha[G];
 #pragma unroll
-        for (int g = 0; g < N; ++g) {
+        for (int g = 0; g < G; ++g) {
           alpha[g] = __shfl_sync(0xffffffffu, my_alpha, g);
           l_part[g] *= alpha[g];
         }
@@ -335,13 +352,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
           tc_fence_after();
           for (int i = 0; i < blocks; ++i)
 #pragma unroll
-            for (int g0 = 0; g0 < N; g0 += 16) {
+            for (int g0 = 0; g0 < G; g0 += 16) {
               uint32_t ov[16];
-              tmem_ld_32x16(lane_addr + COL_O + i * N + g0, ov);
+              tmem_ld_32x16(lane_addr + COL_O + i * N + hg + g0, ov);
               tmem_ld_wait();
 #pragma unroll
               for (int g = 0; g < 16; ++g) ov[g] = __float_as_uint(__uint_as_float(ov[g]) * alpha[g0 + g]);
-              tmem_st_32x16(lane_addr + COL_O + i * N + g0, ov);
+              tmem_st_32x16(lane_addr + COL_O + i * N + hg + g0, ov);
             }
           tmem_st_wait();
         }
@@ -350,51 +367,51 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
         uint8_t* pb = smem + Cfg::OFF_P + (r >> 6) * Cfg::Q_PIECE;
         const int kc = r & 63;
 #pragma unroll
-        for (int g = 0; g < N; ++g) {
+        for (int g = 0; g < G; ++g) {
           const float ref = __shfl_sync(0xffffffffu, my_ref, g);
           const float pv = s[g] == -INFINITY ? 0.f : fast_exp2(s[g] - ref);
           const __nv_bfloat16 pb16 = __float2bfloat16(pv);
           l_part[g] += __bfloat162float(pb16);     // the sum of what the MMA will actually use
-          *reinterpret_cast<__nv_bfloat16*>(pb + g * 128 + (((kc >> 3) ^ (g & 7)) << 4) + (kc & 7) * 2) = pb16;
+          *reinterpret_cast<__nv_bfloat16*>(pb + (hg + g) * 128 + (((kc >> 3) ^ (g & 7)) << 4) + (kc & 7) * 2) = pb16;
         }
       }
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
       if (ok && lane == 0) mbar_arrive(bar(P_FULL));
-      asm volatile("bar.sync 1, 128;" ::: "memory");      // s_red and the old references have been read by all
-      if (ew == 0 && lane < N) s_ref[lane] = my_ref;
+      group_sync();      // s_red and the old references have been read by all
+      if (ew == 0 && lane < G) s_ref[lane] = my_ref;
     }
     if (ok && n_tiles > 0) ok = mbar_wait(bar(O_DONE), (n_tiles - 1) & 1, abort_word, FT_ERR_TIMEOUT_EPILOGUE);
     ok = __all_sync(0xffffffffu, ok);
     tc_fence_after();
 #pragma unroll
-    for (int g = 0; g < N; ++g) {
+    for (int g = 0; g < G; ++g) {
       const float ws = warp_sum(l_part[g]);
-      if (lane == 0) s_red[ew * N + g] = ws;
+      if (lane == 0) s_red[ew * G + g] = ws;
     }
-    asm volatile("bar.sync 1, 128;" ::: "memory");
+    group_sync();
     if (ok)
       for (int i = 0; i < blocks; ++i)
 #pragma unroll
-        for (int g0 = 0; g0 < N; g0 += 16) {
+        for (int g0 = 0; g0 < G; g0 += 16) {
           uint32_t ov[16];
 #pragma unroll
           for (int g = 0; g < 16; ++g) ov[g] = 0u;
           if (n_tiles > 0) {
-            tmem_ld_32x16(lane_addr + COL_O + i * N + g0, ov);
+            tmem_ld_32x16(lane_addr + COL_O + i * N + hg + g0, ov);
             tmem_ld_wait();
           }
           const int d = i * 128 + r;
 #pragma unroll
           for (int g = 0; g < 16; ++g) {
             const int h = g0 + g;
-            if (h >= heads || d >= p.rank) continue;
-            const float l = s_red[h] + s_red[N + h] + s_red[2 * N + h] + s_red[3 * N + h], o = __uint_as_float(ov[g]);
+            if (hg + h >= heads || d >= p.rank) continue;
+            const float l = s_red[h] + s_red[G + h] + s_red[2 * G + h] + s_red[3 * G + h], o = __uint_as_float(ov[g]);
             if (p.n_splits == 1) {
-              p.out[b * p.ldo + static_cast<long long>(h0 + h) * p.rank + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+              p.out[b * p.ldo + static_cast<long long>(h0 + hg + h) * p.rank + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
             } else {
-              const long long at = (static_cast<long long>(b) * p.H + h0 + h) * p.n_splits + split;
+              const long long at = (static_cast<long long>(b) * p.H + h0 + hg + h) * p.n_splits + split;
               p.part_o[at * p.rank + d] = o;
               if (d == 0) { p.part_ml[at * 2] = s_ref[h]; p.part_ml[at * 2 + 1] = l; }
             }
@@ -506,8 +523,8 @@ FT_API int ft_latent_finish(void* packed, long long ld, void* q_lat, int n_lat, 
   p.table = static_cast<const float2*>(table); p.ld = ld; p.rows = rows; p.n_lat = n_lat; p.H = H; p.q_off = q_off; p.q_head = q_head;
   p.q_rot = q_rot; p.c_off = c_off; p.rank_pad = rank_pad; p.rank = rank; p.rot_pad = rot_pad; p.half = half; p.positions = positions;
   p.eps = eps; p.block_size = block_size; p.max_blocks = max_blocks; p.num_blocks = num_blocks;
-  const int cap = sm_count(device) * 64, grid = rows < cap ? rows : cap;
-  int threads = 32 + (H * (rot_pad / 8) + 31) / 32 * 32;
+  const int grid = (rows + LF_ROWS - 1) / LF_ROWS;
+  int threads = 32 * LF_ROWS + (H * (rot_pad / 8) + 31) / 32 * 32;
   if (threads > LF_MAX_THREADS) threads = LF_MAX_THREADS;
   if (f32) latent_finish_kernel<float><<<grid, threads, 0, stream>>>(p);
   else latent_finish_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>(p);
@@ -555,7 +572,7 @@ FT_API int ft_latent_decode(const void* q, const void* cache, const int* block_t
       FT_CUDA_CHECK(cudaFuncSetAttribute(latent_decode_kernel<NN>, cudaFuncAttributeMaxDynamicSharedMemorySize, LdCfg<NN>::SMEM_BYTES)); \
       attr_set[device] = true;                                                                                                      \
     }                                                                                                                               \
-    latent_decode_kernel<NN><<<grid, LD_THREADS, LdCfg<NN>::SMEM_BYTES, stream>>>(tc, p);                                           \
+    latent_decode_kernel<NN><<<grid, LdCfg<NN>::THREADS, LdCfg<NN>::SMEM_BYTES, stream>>>(tc, p);                                           \
   }
   if (N == 16) FT_LD(16) else FT_LD(32)
 #undef FT_LD

@@ -162,6 +162,8 @@ struct EmbedParams {
   float scale, eps;
 };
 
+constexpr int EB_KEEP = 2;        // vectors of eight elements a thread keeps
+
 template <typename T>
 __global__ void __launch_bounds__(ST_MAX_THREADS)
 embed_bigram_kernel(const EmbedParams p) {
@@ -169,6 +171,15 @@ embed_bigram_kernel(const EmbedParams p) {
   float in = 0.f;
   for (int s = 0; s < p.S; ++s) in += p.in[s];
   for (int row = blockIdx.x; row < p.rows; row += gridDim.x) {
+    long long token = p.tokens[row];
+    if (token < 0 || token >= p.vocab) token = 0;
+    const T* er = static_cast<const T*>(p.table) + token * p.ld;
+    float u[EB_KEEP][8];
+#pragma unroll
+    for (int k = 0; k < EB_KEEP; ++k) {              // the token's row is on its way while the previous token is looked up
+      const int i = (k * blockDim.x + threadIdx.x) * 8;
+      if (i < p.H) load8(er + i, u[k]);
+    }
     const int pos = p.pos[row];
     const int* bt = p.block_table + static_cast<long long>(p.slots[row]) * p.max_blocks;
     auto page_of = [&](int q) -> long long {
@@ -176,8 +187,6 @@ embed_bigram_kernel(const EmbedParams p) {
       const int blk = page < p.max_blocks ? bt[page] : -1;
       return blk < 0 || blk >= p.num_blocks ? -1 : static_cast<long long>(blk) * p.block_size + q % p.block_size;
     };
-    long long token = p.tokens[row];
-    if (token < 0 || token >= p.vocab) token = 0;
     long long bucket = p.buckets;
     if (pos > 0) {
       long long prev = 0;
@@ -189,32 +198,40 @@ embed_bigram_kernel(const EmbedParams p) {
       bucket = (prev * p.mul_prev + token * p.mul_cur) % p.buckets;
       if (bucket < 0) bucket += p.buckets;
     }
-    if (threadIdx.x == 0) {                      // no row reads a page place that a row of the same step writes
-      const long long at = page_of(pos);
-      if (at >= 0) p.token_pages[at] = static_cast<int>(token);
-    }
-    const T* er = static_cast<const T*>(p.table) + token * p.ld;
     const T* br = static_cast<const T*>(p.bigram) + bucket * p.ld;
-    float u[ST_KEEP][4];
     float sum = 0.f;
 #pragma unroll
-    for (int k = 0; k < ST_KEEP; ++k) {
-      const int i = (k * blockDim.x + threadIdx.x) * 4;
+    for (int k = 0; k < EB_KEEP; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 8;
       if (i >= p.H) continue;
-      float a[4], b[4];
-      load4(er + i, a);
-      load4(br + i, b);
+      float b[8];
+      load8(br + i, b);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) a[e] = a[e] * p.scale + b[e];
-      store4(p.x + static_cast<long long>(row) * p.H + i, a);
+      for (int e = 0; e < 8; ++e) b[e] = u[k][e] * p.scale + b[e];
+      store8(p.x + static_cast<long long>(row) * p.H + i, b);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        u[k][e] = in * a[e];
+      for (int e = 0; e < 8; ++e) {
+        u[k][e] = in * b[e];
         sum += u[k][e] * u[k][e];
       }
     }
+    if (threadIdx.x == 0) {                          // no row reads a page place that a row of the same step writes
+      const long long at = page_of(pos);
+      if (at >= 0) p.token_pages[at] = static_cast<int>(token);
+    }
     sum = block_total(sum, red);
-    store_normed(u, sum, p.w, static_cast<T*>(p.h) + static_cast<long long>(row) * p.H, p.H, p.count, p.eps);
+    const float r = 1.f / sqrtf(sum / static_cast<float>(p.count) + p.eps);
+    T* h = static_cast<T*>(p.h) + static_cast<long long>(row) * p.H;
+#pragma unroll
+    for (int k = 0; k < EB_KEEP; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 8;
+      if (i >= p.H) continue;
+      float w[8];
+      load8(p.w + i, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[e] = u[k][e] * r * w[e];
+      store8(h + i, w);
+    }
   }
 }
 
@@ -289,7 +306,7 @@ FT_API int ft_embed_bigram(const long long* tokens, const int* pos, const int* s
                            int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(tokens && pos && starts && slots && block_table && token_pages && table && bigram && in && w && x && h, "ft_embed_bigram: null pointer");
-  FT_REQUIRE(H > 0 && H % 8 == 0 && H <= ST_KEEP * 4 * ST_MAX_THREADS && count > 0 && count <= H && ld >= H && ld % 8 == 0, "ft_embed_bigram: rows of %d", H);
+  FT_REQUIRE(H > 0 && H % 8 == 0 && H <= EB_KEEP * 8 * ST_MAX_THREADS && count > 0 && count <= H && ld >= H && ld % 8 == 0, "ft_embed_bigram: rows of %d", H);
   FT_REQUIRE(vocab > 0 && buckets > 0 && S > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0, "ft_embed_bigram: bad shape");
   FT_REQUIRE(st_aligned({table, bigram, w, x, h}), "ft_embed_bigram: pointers must be 16-byte aligned");
   if (rows <= 0) return FT_E_OK;
@@ -298,7 +315,9 @@ FT_API int ft_embed_bigram(const long long* tokens, const int* pos, const int* s
   p.table = table; p.bigram = bigram; p.in = in; p.w = w; p.x = x; p.h = h; p.ld = ld; p.mul_prev = mul_prev; p.mul_cur = mul_cur;
   p.rows = rows; p.S = S; p.H = H; p.count = count; p.vocab = vocab; p.buckets = buckets; p.block_size = block_size;
   p.max_blocks = max_blocks; p.num_blocks = num_blocks; p.scale = scale; p.eps = eps;
-  const int cap = sm_count(device) * 32, grid = rows < cap ? rows : cap, threads = stream_threads(H);
+  const int cap = sm_count(device) * 32, grid = rows < cap ? rows : cap;
+  int threads = (H / 8 + EB_KEEP - 1) / EB_KEEP;
+  threads = threads < 64 ? 64 : (threads + 31) / 32 * 32;
   if (f32) embed_bigram_kernel<float><<<grid, threads, 0, stream>>>(p);
   else embed_bigram_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>(p);
   FT_CUDA_CHECK(cudaGetLastError());

@@ -153,7 +153,7 @@ class LatentAttention(nn.Module):
         """The sublayer's output for input ``h``; ``layer``: its place in the cache."""
         s, T = self.spec, h.shape[0]
         packed = F.linear_rows(h, self.in_proj)
-        formed = self.key_proj is not None and h.is_cuda and batch.longest > ABSORB_ROWS
+        formed = self.key_proj is not None and h.is_cuda and s.scale > 0 and batch.longest > ABSORB_ROWS
         n = batch.n_single if formed else T               # rows that attend in the latent space
         q_lat = torch.empty((n, s.heads, s.row_size), device=h.device, dtype=h.dtype)
         D.latent_finish(packed, cache, layer, batch, heads=s.heads, q_off=0, q_head=s.head_size, q_rot=s.padded_dim, c_off=self.q_width,

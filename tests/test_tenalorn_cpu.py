@@ -385,3 +385,16 @@ def test_server_command_line_serves_the_family(tmp_path):
     assert server.main(["--tiny", "--family", "tenalorn", *args]) == 0
     Case("mixed").save(tmp_path / "m")
     assert server.main(["--model", str(tmp_path / "m"), *args]) == 0
+
+
+def test_the_decoder_kernel_set_holds_every_kernel_the_cache_and_the_row_kernels_call():
+    import os
+    import re
+
+    from ferrotorch_b200 import _native
+    from ferrotorch_b200.nn import paged
+
+    text = "".join(open(os.path.join(_native.CSRC, n + ".cu")).read() for n in _native.KERNEL_SETS["decoder"])
+    have = set(re.findall(r"FT_API[^;{(]*?\b(ft_\w+)\s*\(", text))
+    need = {n for m in (paged, D) for n in re.findall(r"\.(ft_\w+)\(", open(m.__file__).read())}
+    assert {"ft_latent_decode", "ft_memory_chunks", "ft_stream_step"} <= need <= have, need - have

@@ -103,6 +103,25 @@ struct KeyRange {
     return chunk > 0 ? max(lo, max(len - 1, 0) / chunk * chunk) : lo;
   }
 };
+
+// Means of keys and values over blocks of `pool` consecutive positions (counted from 0), seen once a block lies wholly ahead of
+// the window.  Block b lies with the page that holds its last position: [num_blocks, per_page, Hkv, head size].
+struct PooledKeys {
+  const void* k;
+  const void* v;
+  int pool, per_page;      // pool 0: none
+  // Blocks that a query sees whose first visible key is `first`.
+  __device__ __forceinline__ int count(int first) const { return pool > 0 ? first / pool : 0; }
+  // Row of block b on the [num_blocks * per_page] axis; bt: the sequence's pages.
+  __device__ __forceinline__ long long row(int b, const int* bt, int block_size, int max_blocks, int num_blocks) const {
+    const int page = min((b * pool + pool - 1) / block_size, max_blocks - 1);
+    const int at = min(max(b - page * block_size / pool, 0), per_page - 1);
+    return static_cast<long long>(min(max(__ldg(bt + page), 0), num_blocks - 1)) * per_page + at;
+  }
+};
+static inline PooledKeys pooled_keys(const void* k, const void* v, int pool, int block_size) {
+  return PooledKeys{k, v, pool, pool > 0 ? (block_size - 1) / pool + 1 : 0};
+}
 constexpr float ATT_LOG2E = 1.4426950408889634f;
 
 // A head's sink joins the softmax: exp(sink) in the denominator, no key, no value, no scale.  m, l and acc are the

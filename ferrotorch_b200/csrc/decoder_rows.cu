@@ -1,8 +1,12 @@
-// Row kernels of pre-norm decoders with an fp32 residual stream:
+// Row kernels of decoders with an fp32 residual stream:
 //
 //   ft_rms_rows        RMS norm of residual rows, optionally gathering the rows first (the embedding,
 //                      or the rows whose logits are wanted) and optionally adding pending terms to the
 //                      residual (the outputs of a token's experts), all in one pass over the row.
+//   ft_sum_norm_rows   norm after the sum: a factor times the residual row plus a sublayer's terms times their gate,
+//                      RMS-normed back into the residual and into the next sublayer's input, in one pass.
+//   ft_part_norm       RMS norm of equal runs of a row on their own, in place.
+//   ft_poly_norm       sum of a row's first three powers, each over its own root mean square.
 //   ft_qkv_head_finish everything between a packed projection [ q | k | v | .. ] and its attention:
 //                      per-head RMS norm of q and k, rotation of the first 2 * half elements of a head
 //                      by a cos / sin table, k and v into their cache pages.
@@ -10,6 +14,7 @@
 // Rows are bf16 or fp32, arithmetic is fp32.
 #include <initializer_list>
 
+#include "recurrent.cuh"
 #include "row_vec.cuh"
 
 namespace ft {
@@ -105,6 +110,348 @@ rms_rows_kernel(const RmsRowsParams p) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) w[e] = f[e] * r * (p.offset + w[e]);
       store8(yr + i, w);
+    }
+  }
+}
+
+// ---------------------------------------------------------------- norm after the sum
+constexpr int SN_TERMS = 4;   // terms whose places and weights a thread keeps in registers
+
+struct SumNormParams {
+  const void* x;            // [n_src, ldx]
+  const long long* ids;     // token i has x[ids[i]] (null: x[i])
+  const long long* rows;    // row i is token rows[i] (null: token i)
+  const void* dense;        // [tokens, ldd] or null, times dense_weight[token] (null: 1)
+  const float* dense_weight;
+  const void* terms;        // [term_rows, ldt]: token i gains weight[i, j] (null: 1) times terms[where[i, j]], j < n_terms
+  const int* where;
+  const float* weight;
+  const void* gate;         // [tokens, ldg] or null: the terms' sum is multiplied by its sigmoid
+  const float* w;           // [H]
+  const float* w2;          // [H]: of a second norm ahead of h; null: none
+  float* x_out;             // fp32 [rows, ldo] or null; may be x when ids and rows are null
+  void* h;                  // [rows, ldh] or null
+  long long ldx, ldd, ldt, ldg, ldo, ldh;
+  int n_rows, tokens, n_src, H, count, n_terms, term_rows;
+  float alpha, eps;
+};
+
+__device__ __forceinline__ float block_total(float v, float* red) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  v = warp_sum(v);
+  __syncthreads();                         // the previous total has been read
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  v = 0.f;
+#pragma unroll
+  for (int w = 0; w < ROW_WARPS; ++w) v += red[w];
+  return v;
+}
+
+// One block per row.
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(ROW_THREADS)
+sum_norm_rows_kernel(const SumNormParams p) {
+  __shared__ float red[ROW_WARPS];
+  for (int row = blockIdx.x; row < p.n_rows; row += gridDim.x) {
+    long long token = row;
+    if (p.rows) {
+      token = p.rows[row];
+      if (token < 0 || token >= p.tokens) token = 0;    // host validates; never read out of range
+    }
+    long long src = token;
+    if (p.ids) {
+      src = p.ids[token];
+      if (src < 0 || src >= p.n_src) src = 0;
+    }
+    const TI* xr = static_cast<const TI*>(p.x) + src * p.ldx;
+    const TO* dr = p.dense ? static_cast<const TO*>(p.dense) + token * p.ldd : nullptr;
+    const TO* gr = p.gate ? static_cast<const TO*>(p.gate) + token * p.ldg : nullptr;
+    const float dw = p.dense_weight ? p.dense_weight[token] : 1.f;
+    const int* where = p.where + token * p.n_terms;
+    const float* weight = p.weight ? p.weight + token * p.n_terms : nullptr;
+    int at[SN_TERMS];
+    float tw[SN_TERMS];
+#pragma unroll
+    for (int j = 0; j < SN_TERMS; ++j) {
+      at[j] = j < p.n_terms ? where[j] : -1;
+      tw[j] = weight && j < p.n_terms ? weight[j] : 1.f;
+    }
+    float* xo = p.x_out ? p.x_out + static_cast<long long>(row) * p.ldo : nullptr;
+    TO* hr = p.h ? static_cast<TO*>(p.h) + static_cast<long long>(row) * p.ldh : nullptr;
+    auto add_term = [&](int t, float wt, int i, float (&y)[8]) {
+      if (t < 0 || t >= p.term_rows) return;
+      float g[8];
+      load8(static_cast<const TO*>(p.terms) + static_cast<long long>(t) * p.ldt + i, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] += wt * g[e];
+    };
+    auto fetch = [&](int i, float (&f)[8]) {
+      float y[8], g[8];
+      load8(xr + i, f);
+      if (gr) load8(gr + i, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = 0.f;
+      if (dr) {
+        load8(dr + i, y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] *= dw;
+      }
+#pragma unroll
+      for (int j = 0; j < SN_TERMS; ++j) add_term(at[j], tw[j], i, y);
+      for (int j = SN_TERMS; j < p.n_terms; ++j) add_term(where[j], weight ? weight[j] : 1.f, i, y);
+      if (gr) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] *= sigmoid_row(g[e], static_cast<const TO*>(nullptr));
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = p.alpha * f[e] + y[e];
+    };
+    float kept[ROW_KEEP][8];
+    float sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < ROW_KEEP; ++k) {
+      const int i = (k * ROW_THREADS + threadIdx.x) * 8;
+      if (i < p.H) {
+        fetch(i, kept[k]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += kept[k][e] * kept[k][e];
+      }
+    }
+    // wider rows: the tail's sum waits in x_out where there is one (a thread owns the same columns in every pass) and is formed
+    // anew where not
+    const int rest = ROW_KEEP * ROW_THREADS * 8 + threadIdx.x * 8;
+    for (int i = rest; i < p.H; i += ROW_THREADS * 8) {
+      float f[8];
+      fetch(i, f);
+      if (xo) store8(xo + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum += f[e] * f[e];
+    }
+    const float r = 1.f / sqrtf(block_total(sum, red) / static_cast<float>(p.count) + p.eps);
+    auto normed = [&](int i, const float (&f)[8], float (&o)[8]) {
+      float w[8];
+      load8(p.w + i, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] = f[e] * r * w[e];
+    };
+    float r2 = 1.f;
+    if (p.w2) {
+      sum = 0.f;
+#pragma unroll
+      for (int k = 0; k < ROW_KEEP; ++k) {
+        const int i = (k * ROW_THREADS + threadIdx.x) * 8;
+        if (i < p.H) {
+          float o[8];
+          normed(i, kept[k], o);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) sum += o[e] * o[e];
+        }
+      }
+      for (int i = rest; i < p.H; i += ROW_THREADS * 8) {
+        float f[8], o[8];
+        if (xo) load8(static_cast<const float*>(xo) + i, f); else fetch(i, f);
+        normed(i, f, o);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += o[e] * o[e];
+      }
+      r2 = 1.f / sqrtf(block_total(sum, red) / static_cast<float>(p.count) + p.eps);
+    }
+    auto store = [&](int i, const float (&f)[8]) {
+      float o[8];
+      normed(i, f, o);
+      if (xo) store8(xo + i, o);
+      if (!hr) return;
+      if (p.w2) {
+        float w[8];
+        load8(p.w2 + i, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] *= r2 * w[e];
+      }
+      store8(hr + i, o);
+    };
+#pragma unroll
+    for (int k = 0; k < ROW_KEEP; ++k) {
+      const int i = (k * ROW_THREADS + threadIdx.x) * 8;
+      if (i < p.H) store(i, kept[k]);
+    }
+    for (int i = rest; i < p.H; i += ROW_THREADS * 8) {
+      float f[8];
+      if (xo) load8(static_cast<const float*>(xo) + i, f); else fetch(i, f);
+      store(i, f);
+    }
+  }
+}
+
+// ---------------------------------------------------------------- norms inside sublayers
+constexpr int PN_KEEP = 4;      // vectors of eight elements a thread keeps in registers
+
+// `parts` runs of n elements per row, contiguous and whole vectors; GT threads take one run.
+template <typename T, int GT>
+__global__ void __launch_bounds__(ROW_THREADS)
+part_norm_kernel(T* __restrict__ y, long long ld, const float* __restrict__ w, int rows, int parts, int n, float eps) {
+  __shared__ float red[ROW_WARPS];
+  const int t = threadIdx.x % GT;
+  const long long tasks = static_cast<long long>(rows) * parts;
+  for (long long task = static_cast<long long>(blockIdx.x) * (ROW_THREADS / GT) + threadIdx.x / GT; task < tasks;
+       task += static_cast<long long>(gridDim.x) * (ROW_THREADS / GT)) {
+    const long long row = task / parts;
+    const int part = static_cast<int>(task - row * parts);
+    T* at = y + row * ld + static_cast<long long>(part) * n;
+    const float* wp = w + static_cast<long long>(part) * n;
+    float kept[PN_KEEP][8];
+    float sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < PN_KEEP; ++k) {
+      const int i = (k * GT + t) * 8;
+      if (i < n) {
+        load8(at + i, kept[k]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum += kept[k][e] * kept[k][e];
+      }
+    }
+    const int rest = (PN_KEEP * GT + t) * 8;
+    for (int i = rest; i < n; i += GT * 8) {
+      float f[8];
+      load8(at + i, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum += f[e] * f[e];
+    }
+    sum = GT == 32 ? warp_sum(sum) : block_total(sum, red);
+    const float r = 1.f / sqrtf(sum / static_cast<float>(n) + eps);
+    auto finish = [&](int i, float (&f)[8]) {
+      float g[8];
+      load8(wp + i, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] *= r * g[e];
+      store8(at + i, f);
+    };
+#pragma unroll
+    for (int k = 0; k < PN_KEEP; ++k) {
+      const int i = (k * GT + t) * 8;
+      if (i < n) finish(i, kept[k]);
+    }
+    for (int i = rest; i < n; i += GT * 8) {
+      float f[8];
+      load8(at + i, f);
+      finish(i, f);
+    }
+  }
+}
+
+// Any sizes: element i of a run is element i % vdim of a head padded to vp.  A warp takes one run.
+template <typename T>
+__global__ void __launch_bounds__(ROW_THREADS)
+part_norm_any_kernel(T* __restrict__ y, long long ld, const float* __restrict__ w, int rows, int parts, int n, int vdim, int vp, float eps) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long tasks = static_cast<long long>(rows) * parts;
+  for (long long task = static_cast<long long>(blockIdx.x) * ROW_WARPS + warp; task < tasks; task += static_cast<long long>(gridDim.x) * ROW_WARPS) {
+    const long long row = task / parts;
+    const int part = static_cast<int>(task - row * parts);
+    T* yr = y + row * ld;
+    auto column = [&](int i) {
+      const int c = part * n + i;
+      return c / vdim * vp + c % vdim;
+    };
+    float sum = 0.f;
+    for (int i = lane; i < n; i += 32) {
+      const float v = static_cast<float>(yr[column(i)]);
+      sum += v * v;
+    }
+    const float r = 1.f / sqrtf(warp_sum(sum) / static_cast<float>(n) + eps);
+    for (int i = lane; i < n; i += 32) {
+      const int c = column(i);
+      yr[c] = static_cast<T>(static_cast<float>(yr[c]) * r * w[c]);
+    }
+  }
+}
+
+__device__ __forceinline__ void raw_load(const __nv_bfloat16* p, uint4 (&v)[1]) { v[0] = *reinterpret_cast<const uint4*>(p); }
+__device__ __forceinline__ void raw_load(const float* p, uint4 (&v)[2]) {
+  v[0] = reinterpret_cast<const uint4*>(p)[0];
+  v[1] = reinterpret_cast<const uint4*>(p)[1];
+}
+__device__ __forceinline__ void raw_unpack(const uint4 (&v)[1], float (&f)[8]) { unpack8(v[0], f); }
+__device__ __forceinline__ void raw_unpack(const uint4 (&v)[2], float (&f)[8]) {
+  f[0] = __uint_as_float(v[0].x); f[1] = __uint_as_float(v[0].y); f[2] = __uint_as_float(v[0].z); f[3] = __uint_as_float(v[0].w);
+  f[4] = __uint_as_float(v[1].x); f[5] = __uint_as_float(v[1].y); f[6] = __uint_as_float(v[1].z); f[7] = __uint_as_float(v[1].w);
+}
+
+// out = a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e over rows of N elements of which `count` exist (the others are
+// zero).  One block per row; the first KEEP vectors of a thread stay in registers.
+template <typename T, int KEEP>
+__global__ void __launch_bounds__(ROW_THREADS)
+poly_norm_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo, const float* __restrict__ coef, int rows, int N, int count,
+                 float eps) {
+  __shared__ float red[3][ROW_WARPS];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int row = blockIdx.x; row < rows; row += gridDim.x) {
+    const T* zr = z + static_cast<long long>(row) * ldz;
+    T* yr = out + static_cast<long long>(row) * ldo;
+    uint4 kept[KEEP][sizeof(T) / 2];
+    float s[3] = {0.f, 0.f, 0.f};
+    auto add = [&](const float (&f)[8]) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float q = f[e] * f[e];
+        s[0] += q;
+        s[1] += q * q;
+        s[2] += q * q * q;
+      }
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = (k * ROW_THREADS + threadIdx.x) * 8;
+      if (i < N) raw_load(zr + i, kept[k]);
+    }
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      if ((k * ROW_THREADS + static_cast<int>(threadIdx.x)) * 8 < N) {
+        float f[8];
+        raw_unpack(kept[k], f);
+        add(f);
+      }
+    }
+    const int rest = (KEEP * ROW_THREADS + threadIdx.x) * 8;
+    for (int i = rest; i < N; i += ROW_THREADS * 8) {
+      float f[8];
+      load8(zr + i, f);
+      add(f);
+    }
+    __syncthreads();                       // the previous row's sums have been read
+#pragma unroll
+    for (int j = 0; j < 3; ++j) {
+      s[j] = warp_sum(s[j]);
+      if (lane == 0) red[j][warp] = s[j];
+    }
+    __syncthreads();
+    float c[3];
+#pragma unroll
+    for (int j = 0; j < 3; ++j) {
+      float v = 0.f;
+#pragma unroll
+      for (int w = 0; w < ROW_WARPS; ++w) v += red[j][w];
+      c[j] = coef[j] / sqrtf(v / static_cast<float>(count) + eps);
+    }
+    const float last = coef[3];
+    auto finish = [&](int i, float (&f)[8]) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = ((c[2] * f[e] + c[1]) * f[e] + c[0]) * f[e] + last;
+      store8(yr + i, f);
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+      const int i = (k * ROW_THREADS + threadIdx.x) * 8;
+      if (i < N) {
+        float f[8];
+        raw_unpack(kept[k], f);
+        finish(i, f);
+      }
+    }
+    for (int i = rest; i < N; i += ROW_THREADS * 8) {
+      float f[8];
+      load8(zr + i, f);
+      finish(i, f);
     }
   }
 }
@@ -325,6 +672,92 @@ FT_API int ft_rms_rows(const void* x, const long long* ids, int n_src, int in_bf
     if (out_f32) rms_rows_kernel<float, float><<<grid, ROW_THREADS, 0, stream>>>(p);
     else rms_rows_kernel<float, __nv_bfloat16><<<grid, ROW_THREADS, 0, stream>>>(p);
   }
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// x' = norm(alpha x + sigmoid(gate) (dense_weight dense + sum_j weight_j terms[where_j])) * w for `n_rows` rows (see SumNormParams), RMS
+// over `count` elements, into x_out and, as bf16 or with out_f32 as fp32, into h; with w2 h goes through a second norm.  x: fp32, or
+// bf16 with in_bf16 (fp32 embeddings: in_bf16 0).  dense, terms and gate have the type of h.  H and strides multiples of 8.
+FT_API int ft_sum_norm_rows(const void* x, long long ldx, const long long* ids, int n_src, int in_bf16, const long long* rows, const void* dense,
+                            long long ldd, const float* dense_weight, const void* terms, long long ldt, int term_rows, const int* where,
+                            const float* weight, int n_terms, const void* gate, long long ldg, float alpha, const float* w, const float* w2,
+                            float* x_out, long long ldo, void* h, long long ldh, int out_f32, int n_rows, int tokens, int H, int count,
+                            float eps, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(x && w && (x_out || h) && (dense || n_terms > 0), "ft_sum_norm_rows: null pointer");
+  FT_REQUIRE(H > 0 && H % 8 == 0 && count > 0 && count <= H && ((ldx | ldd | ldt | ldg | ldo | ldh) & 7) == 0 && ldx >= H,
+             "ft_sum_norm_rows: H=%d and strides must be multiples of 8", H);
+  FT_REQUIRE(n_terms == 0 || (terms && where && n_terms > 0 && ldt >= H && term_rows > 0), "ft_sum_norm_rows: terms without their rows");
+  FT_REQUIRE((!dense || ldd >= H) && (!gate || ldg >= H) && (!x_out || ldo >= H) && (!h || ldh >= H), "ft_sum_norm_rows: row strides");
+  FT_REQUIRE(row_aligned({x, dense, terms, gate, w, w2, x_out, h}), "ft_sum_norm_rows: pointers must be 16-byte aligned");
+  FT_REQUIRE(n_src > 0 && (ids || tokens <= n_src) && (rows || n_rows <= tokens), "ft_sum_norm_rows: %d source rows", n_src);
+  FT_REQUIRE(x_out != x || (!ids && !rows && !in_bf16), "ft_sum_norm_rows: gathered rows cannot be updated in place");
+  if (n_rows <= 0) return FT_E_OK;
+  SumNormParams p;
+  p.x = x; p.ids = ids; p.rows = rows; p.dense = dense; p.dense_weight = dense_weight; p.terms = terms; p.where = where; p.weight = weight;
+  p.gate = gate; p.w = w; p.w2 = w2; p.x_out = x_out; p.h = h;
+  p.ldx = ldx; p.ldd = ldd; p.ldt = ldt; p.ldg = ldg; p.ldo = ldo; p.ldh = ldh;
+  p.n_rows = n_rows; p.tokens = tokens; p.n_src = n_src; p.H = H; p.count = count; p.n_terms = n_terms; p.term_rows = term_rows;
+  p.alpha = alpha; p.eps = eps;
+  const int cap = sm_count(device) * 32;
+  const int grid = n_rows < cap ? n_rows : cap;
+  if (in_bf16) {
+    if (out_f32) sum_norm_rows_kernel<__nv_bfloat16, float><<<grid, ROW_THREADS, 0, stream>>>(p);
+    else sum_norm_rows_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, ROW_THREADS, 0, stream>>>(p);
+  } else {
+    if (out_f32) sum_norm_rows_kernel<float, float><<<grid, ROW_THREADS, 0, stream>>>(p);
+    else sum_norm_rows_kernel<float, __nv_bfloat16><<<grid, ROW_THREADS, 0, stream>>>(p);
+  }
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// RMS norm, in place, of `parts` equal runs of rows y [rows, ld] on their own, times w [heads * vp].  A row is heads of vdim
+// elements padded to vp; runs count the elements that exist.  bf16, or fp32 with f32.
+FT_API int ft_part_norm(void* y, long long ld, const float* w, int rows, int heads, int vdim, int vp, int parts, float eps, int f32, int device,
+                        cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(y && w, "ft_part_norm: null pointer");
+  const long long inner = static_cast<long long>(heads) * vdim;
+  FT_REQUIRE(heads > 0 && vdim > 0 && vp >= vdim && parts > 0 && inner % parts == 0 && static_cast<long long>(heads) * vp < (1ll << 31) &&
+                 ld >= static_cast<long long>(heads) * vp, "ft_part_norm: %d heads of %d in %d parts", heads, vdim, parts);
+  if (rows <= 0) return FT_E_OK;
+  const int n = static_cast<int>(inner / parts), cap = sm_count(device) * 16;
+  const bool vectors = vp == vdim && n % 8 == 0 && ld % 8 == 0 && row_aligned({y, w});
+  const bool wide = vectors && n > PN_KEEP * 256;
+  const long long tasks = static_cast<long long>(rows) * parts, need = wide ? tasks : (tasks + ROW_WARPS - 1) / ROW_WARPS;
+  const int grid = need < cap ? static_cast<int>(need) : cap;
+#define FT_PN(T)                                                                                                        \
+  if (wide) part_norm_kernel<T, 256><<<grid, ROW_THREADS, 0, stream>>>(static_cast<T*>(y), ld, w, rows, parts, n, eps);  \
+  else if (vectors) part_norm_kernel<T, 32><<<grid, ROW_THREADS, 0, stream>>>(static_cast<T*>(y), ld, w, rows, parts, n, eps); \
+  else part_norm_any_kernel<T><<<grid, ROW_THREADS, 0, stream>>>(static_cast<T*>(y), ld, w, rows, parts, n, vdim, vp, eps);
+  if (f32) { FT_PN(float) } else { FT_PN(__nv_bfloat16) }
+#undef FT_PN
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// out [rows, N] = a N(z) + b N(z^2) + c N(z^3) + e with coef = (a, b, c, e) fp32, N dividing a row by its root mean square over `count`
+// elements (those behind them are zero; they become e).  bf16, or fp32 with f32; N and strides multiples of 8.
+FT_API int ft_poly_norm(const void* z, long long ldz, void* out, long long ldo, const float* coef, int rows, int N, int count, float eps, int f32,
+                        int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(z && out && coef, "ft_poly_norm: null pointer");
+  FT_REQUIRE(N > 0 && N % 8 == 0 && count > 0 && count <= N && ldz >= N && ldo >= N && ((ldz | ldo) & 7) == 0 && row_aligned({z, out}),
+             "ft_poly_norm: N=%d and strides must be multiples of 8", N);
+  if (rows <= 0) return FT_E_OK;
+  const int cap = sm_count(device) * 16, grid = rows < cap ? rows : cap;
+#define FT_PO(T, K) \
+  poly_norm_kernel<T, K><<<grid, ROW_THREADS, 0, stream>>>(static_cast<const T*>(z), ldz, static_cast<T*>(out), ldo, coef, rows, N, count, eps)
+  if (f32) FT_PO(float, 4);
+  else if (N <= 2 * ROW_THREADS * 8) FT_PO(__nv_bfloat16, 2);
+  else if (N <= 6 * ROW_THREADS * 8) FT_PO(__nv_bfloat16, 6);
+  else FT_PO(__nv_bfloat16, 12);
+#undef FT_PO
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

@@ -4,7 +4,7 @@
 //
 // W is [groups, parts, N, K] (bf16, K-major).  With two parts a tile accumulates both products of the same rows, so
 // that the epilogue can combine them:
-//   EPI_STORE  one part:  C = sum, optionally times the sigmoid of a gate per element
+//   EPI_STORE  one part:  C = sum, optionally the square of its relu, or times the sigmoid of a gate per element
 //   EPI_GLU    two parts: C = act(r sum_0) * (r sum_1), r a factor per row (a routed token's weight: scaling the
 //              two sums is scaling the input)
 //   EPI_RGLRU  two parts: the gates of a real-gated linear recurrence (see recurrent.cuh), recurrence and all for
@@ -36,6 +36,7 @@ constexpr int GG_BK = 64;
 constexpr int GG_GROUP_M = 16;
 
 enum : int { EPI_STORE = 0, EPI_GLU = 1, EPI_RGLRU = 2 };
+constexpr int GG_RELU2 = 3;
 
 struct GroupedParams {
   // segments: items[3 i ..] = group, first row, rows; n_items_dev on the device.  Column blocks: items null,
@@ -50,7 +51,7 @@ struct GroupedParams {
   const void* gate;          // EPI_STORE: element (row, column) is multiplied by sigmoid(gate[row * ldgate + column]); null: not
   long long ldgate;
   const float* row_scale;    // EPI_GLU: per row, or null
-  int act;
+  int act;                   // EPI_GLU: of the first sum; EPI_STORE: GG_RELU2 or 0
   RglruGateParams gates;     // EPI_RGLRU
   int* status;
 };
@@ -278,6 +279,10 @@ grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             }
             const long long col = static_cast<long long>(t.group) * p.out_col + n + h * 8;
             if constexpr (EPI == EPI_STORE) {
+              if (p.act == GG_RELU2) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) { f[e] = fmaxf(f[e], 0.f); f[e] *= f[e]; }
+              }
               if (p.gate) {
                 float z[8];
                 load8(static_cast<const __nv_bfloat16*>(p.gate) + row * p.ldgate + col, z);
@@ -390,6 +395,9 @@ grouped_gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W
             v = (p.act == 0 ? g / (1.f + expf(-g)) : glu_act(g, p.act)) * (s * acc[1][i][j]);
           }
           const long long col = static_cast<long long>(t.group) * p.out_col + n;
+          if constexpr (EPI == EPI_STORE) {
+            if (p.act == GG_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+          }
           if constexpr (EPI == EPI_STORE)
             if (p.gate) v *= sigmoid_row(static_cast<const float*>(p.gate)[row * p.ldgate + col], static_cast<const float*>(nullptr));
           static_cast<float*>(p.out)[row * p.ldo + col] = v;
@@ -403,7 +411,8 @@ grouped_gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ W
 // The experts of a row and their weights from its router logits z.  One warp per row.
 //   SCORE_SIGMOID  the `top` largest logits (the lower index of equals), weighted by their sigmoid
 //   SCORE_SOFTMAX  scores s = softmax(z) over all outputs; the `top` largest s + correction, weighted by their s, divided by the
-//                  sum of these (+ 1e-20) when normalised
+//                  sum of these (+ 1e-20) when normalised: the softmax over the chosen logits alone
+// A bias per output may join the logits.  One more output behind these may be a gate of the row: its sigmoid is stored.
 // With h the logits are computed here, from the row and the router's matrix in fp32 (batches too small for a product of
 // their own); else they are read.
 constexpr int MR_THREADS = 256;
@@ -414,12 +423,22 @@ enum : int { SCORE_SIGMOID = 0, SCORE_SOFTMAX = 1 };
 struct RouteRule {
   int outputs, top, score, normalize;   // outputs: router logits of a row
   const float* correction;              // [outputs] or null
+  const float* bias;                    // [outputs] or null
+  float* gate;                          // [rows] or null: sigmoid of output `outputs`
+  __host__ __device__ __forceinline__ int logits() const { return outputs + (gate ? 1 : 0); }
 };
 
-// z [outputs] in shared memory is overwritten (softmax scores take a second array of the same size behind it).
-__device__ __forceinline__ void choose_experts(float* z, const RouteRule& rule, int lane, int* index, float* weight) {
+// z [rule.logits()] in shared memory is overwritten (softmax scores take a second array of the same size behind it).
+__device__ __forceinline__ void choose_experts(float* z, const RouteRule& rule, int lane, long long row, int* index, float* weight) {
   const int n = rule.outputs;
-  float* s = z + n;
+  float* s = z + rule.logits();
+  index += row * rule.top;
+  weight += row * rule.top;
+  if (rule.gate && lane == 0) rule.gate[row] = 1.f / (1.f + expf(-z[n]));
+  if (rule.bias) {
+    for (int e = lane; e < n; e += 32) z[e] += rule.bias[e];
+    __syncwarp();
+  }
   if (rule.score == SCORE_SOFTMAX) {
     float m = -INFINITY, sum = 0.f;
     for (int e = lane; e < n; e += 32) m = fmaxf(m, z[e]);
@@ -467,11 +486,12 @@ moe_choose_kernel(const float* __restrict__ logits, long long ldl, int rows, con
                   float* __restrict__ weight) {
   extern __shared__ float mr_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float* z = mr_sm + warp * 2 * rule.outputs;
+  const int n = rule.logits();
+  float* z = mr_sm + warp * 2 * n;
   for (int row = blockIdx.x * (MR_THREADS / 32) + warp; row < rows; row += gridDim.x * (MR_THREADS / 32)) {
-    for (int e = lane; e < rule.outputs; e += 32) z[e] = logits[row * ldl + e];
+    for (int e = lane; e < n; e += 32) z[e] = logits[row * ldl + e];
     __syncwarp();
-    choose_experts(z, rule, lane, index + static_cast<long long>(row) * rule.top, weight + static_cast<long long>(row) * rule.top);
+    choose_experts(z, rule, lane, row, index, weight);
   }
 }
 
@@ -516,12 +536,11 @@ __global__ void __launch_bounds__(MR_THREADS)
 moe_route_rows_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ router, int rows, int H, const RouteRule rule,
                       int* __restrict__ index, float* __restrict__ weight) {
   extern __shared__ float mr_sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, experts = rule.outputs;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int row = blockIdx.x; row < rows; row += gridDim.x) {
-    row_outputs(h + row * ldh, router, H, experts, mr_sm);
+    row_outputs(h + row * ldh, router, H, rule.logits(), mr_sm);
     __syncthreads();
-    if (warp == 0)
-      choose_experts(mr_sm, rule, lane, index + static_cast<long long>(row) * rule.top, weight + static_cast<long long>(row) * rule.top);
+    if (warp == 0) choose_experts(mr_sm, rule, lane, row, index, weight);
     __syncthreads();
   }
 }
@@ -669,30 +688,32 @@ FT_API int ft_moe_max_items(int pairs, int experts) { return (pairs < experts ? 
 
 // Routing of `rows` rows (see RouteRule): the choices of every row and their weights, rows sorted by expert.  The router has
 // outputs >= experts logits; choices from `experts` on have no matrices: place -1.  logits: fp32 [rows, ldl] or null (then
-// computed from h and router [outputs, H], the type of h).  Outputs: index int32 [rows, top], weight fp32 [rows, top], place
+// computed from h and router [outputs, H], the type of h).  bias fp32 [outputs] or null joins the logits.  gate fp32 [rows] or null: the
+// router has one more output, whose sigmoid this receives.  Outputs: index int32 [rows, top], weight fp32 [rows, top], place
 // int32 [rows, top] (sorted position), scale fp32 [rows * top] (by position), items int32 [max_items, 3] and n_items for
 // ft_grouped_gemm, sorted [rows * top, H] (the rows of h).  h: bf16, or fp32 with f32; H a multiple of 8; outputs <= 1024.
 FT_API int ft_moe_route(const void* h, long long ldh, const void* router, const float* logits, long long ldl, int rows, int H,
-                        int experts, int outputs, int top, int score, const float* correction, int normalize, int f32, int* index,
-                        float* weight, int* place, float* scale, int* items, int max_items, int* n_items, void* sorted, int device,
+                        int experts, int outputs, int top, int score, const float* correction, const float* bias, int normalize,
+                        float* gate, int f32, int* index, float* weight, int* place, float* scale, int* items, int max_items, int* n_items, void* sorted, int device,
                         cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(h && (router || logits) && index && weight && place && scale && items && n_items && sorted, "ft_moe_route: null pointer");
   FT_REQUIRE(experts >= 1 && outputs >= experts && outputs <= MR_MAX_EXPERTS && top >= 1 && top <= outputs, "ft_moe_route: %d of %d outputs, %d experts", top, outputs, experts);
+  FT_REQUIRE(outputs + (gate ? 1 : 0) <= MR_MAX_EXPERTS, "ft_moe_route: %d outputs and a gate", outputs);
   FT_REQUIRE(score == SCORE_SOFTMAX || (score == SCORE_SIGMOID && !correction), "ft_moe_route: score %d", score);
   FT_REQUIRE(H > 0 && H % 8 == 0 && ldh % 8 == 0 && gg_aligned({h, router, sorted}), "ft_moe_route: H=%d and strides must be multiples of 8", H);
   FT_REQUIRE(static_cast<long long>(rows) * top < (1ll << 31) && max_items >= ft_moe_max_items(rows * top, experts), "ft_moe_route: %d items are too few", max_items);
   if (rows <= 0) return FT_E_OK;
   const int sms = sm_count(device);
-  const RouteRule rule = {outputs, top, score, normalize, correction};
+  const RouteRule rule = {outputs, top, score, normalize, correction, bias, gate};
   if (logits) {
-    const size_t smem = static_cast<size_t>(MR_THREADS / 32) * 2 * outputs * sizeof(float);
+    const size_t smem = static_cast<size_t>(MR_THREADS / 32) * 2 * rule.logits() * sizeof(float);
     const int need = (rows + MR_THREADS / 32 - 1) / (MR_THREADS / 32), cap = sms * 8;
     FT_CUDA_CHECK(cudaFuncSetAttribute(moe_choose_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     moe_choose_kernel<<<need < cap ? need : cap, MR_THREADS, smem, stream>>>(logits, ldl, rows, rule, index, weight);
   } else {
     const int cap = sms * 8;
-    const size_t smem = static_cast<size_t>(outputs) * 2 * sizeof(float);
+    const size_t smem = static_cast<size_t>(rule.logits()) * 2 * sizeof(float);
     if (f32)
       moe_route_rows_kernel<float><<<rows < cap ? rows : cap, MR_THREADS, smem, stream>>>(
           static_cast<const float*>(h), ldh, static_cast<const float*>(router), rows, H, rule, index, weight);
@@ -715,7 +736,7 @@ FT_API int ft_moe_route(const void* h, long long ldh, const void* router, const 
 }
 
 // out = epilogue(A W^T) over segments of rows: A [total_rows, K], W [groups, parts, N, K], items / n_items as
-// ft_moe_route writes them (at most max_items).  glu 0: one part, out = the sum; glu 1: two parts (gate, up), out =
+// ft_moe_route writes them (at most max_items).  glu 0: one part, out = the sum, or with act 3 the square of its relu; glu 1: two parts (gate, up), out =
 // act(r gate) * (r up) with r = row_scale (null: 1), act 0 silu / 1 relu / 2 gelu (tanh form).  seg_rows: an upper
 // bound of the rows of a segment (0: none known).  All bf16, or fp32 with f32.  N and K multiples of 8.
 FT_API int ft_grouped_gemm(const void* A, long long lda, int total_rows, const void* W, const int* items, const int* n_items,
@@ -726,7 +747,7 @@ FT_API int ft_grouped_gemm(const void* A, long long lda, int total_rows, const v
   FT_REQUIRE(groups > 0 && N > 0 && K > 0 && ((N | K) & 7) == 0 && lda % 8 == 0 && ldo % 8 == 0 && lda >= K && ldo >= N,
              "ft_grouped_gemm: N=%d, K=%d and strides must be multiples of 8", N, K);
   FT_REQUIRE(gg_aligned({A, W, out}), "ft_grouped_gemm: pointers must be 16-byte aligned");
-  FT_REQUIRE(act >= 0 && act <= 2 && static_cast<long long>(groups) * 2 * N < (1ll << 31), "ft_grouped_gemm: bad argument");
+  FT_REQUIRE((glu ? act >= 0 && act <= 2 : act == 0 || act == GG_RELU2) && static_cast<long long>(groups) * 2 * N < (1ll << 31), "ft_grouped_gemm: bad argument");
   GroupedParams p = {};
   p.items = items; p.n_items_dev = n_items; p.max_items = max_items; p.groups = groups;
   p.a_rows = GG_BM;

@@ -1,21 +1,32 @@
-// Matrix memories (the recurrence of xLSTM's mLSTM): per head a state S [dim, vdim] and a normaliser n [dim], both relative
-// to a running maximum m of the logarithmic gates,
+// Recurrences whose state is a matrix per head, S [dim, vdim], and changes by outer products k v^T.  Two rules:
+//
+// MEMORY, the recurrence of xLSTM's mLSTM: S and a normaliser n [dim], both relative to a running maximum m of the logarithmic gates,
 //
 //   i = cap tanh((zi + bi) / cap),  f = logsigmoid(cap tanh((zf + bf) / cap))
 //   m' = max(f + m, i),  S' = e^(f + m - m') S + e^(i - m') k v^T,  n' likewise with k alone
 //   o = S'^T q / (max(|n'.q|, e^-m') + 1e-6)
 //
-// followed by an RMS norm of every head's o, a weight, the sigmoid of an output gate and a constant factor.  Gates, states
-// and all arithmetic of the recurrence are fp32; q, k, v and the output gate come from a packed projection.
+// followed by an RMS norm of every head's o, a weight, the sigmoid of an output gate and a constant factor.
 //
-//   ft_memory_steps   token by token: rows that are their sequence's only token, short portions, any sizes, bf16 or fp32
-//   ft_memory_chunks  whole portions in chunks of 128 tokens on tcgen05 / TMEM (bf16, dim up to 128, vdim up to 256)
+// STATE_SPACE, state-space duality (Mamba-2): with step sizes dt = softplus(z + b) and a rate per head,
+//
+//   S' = e^(-rate dt) S + dt k v^T,  o = (S'^T q + skip v) silu(gate)
+//
+// where k, q (B and C there) are shared by the heads of a group.
+//
+// Gates, step sizes, states and all arithmetic of the recurrence are fp32; q, k, v and the output gate come from packed rows.
+//
+//   ft_memory_steps, ft_state_steps    token by token: rows that are their sequence's only token, short portions, any sizes,
+//                                      bf16 or fp32
+//   ft_memory_chunks, ft_state_chunks  whole portions in chunks of 128 tokens on tcgen05 / TMEM (bf16, dim up to 128, vdim up
+//                                      to 256)
 //
 // Chunks.  Let b_t be the sum of f over a chunk's tokens up to t, a_t = i_t - b_t, M the maximum before the chunk and x_t =
 // max(M, a_1 .. a_t).  Then m_t = b_t + x_t and
 //   S_t = e^(M - x_t) S + sum_(s <= t) e^(a_s - x_t) k_s v_s^T,
 // so a chunk's outputs are a causal product of scores like attention's plus q times the state at its start, and its
-// contribution to the next state is one product over its tokens, independent of all other chunks.  Four passes:
+// contribution to the next state is one product over its tokens, independent of all other chunks.  With b the sum of -rate dt, a =
+// log dt - b, x = -b and M = 0 this is the state-space rule, whose exponents never are positive where they count.  Four passes:
 //   memory_gates_kernel   a, x, e^-m of every token and M of every chunk (fp32; a warp scans a chunk)
 //   memory_update_kernel  U = sum_s e^(a_s - x_end) k_s v_s^T of every (chunk, head): tcgen05 product with the weighted keys
 //                         as high and low bf16 halves, so that the state keeps about 16 bits more than its operands
@@ -23,7 +34,8 @@
 //                         chunk's starting state as high and low bf16 halves and the final one in the slot
 //   memory_output_kernel  O = q S, scaled row by row with e^(M - x_t) in TMEM, then + P V with the weights P = causal
 //                         e^(a_s - x_t) q.k written over the scores; denominator, norm, gate and store.  S and P are operands in
-//                         high and low halves: o is normed, so where keys nearly cancel, the error of a plain bf16 weight would grow
+//                         high and low halves: o is normed, so where keys nearly cancel, the error of a plain bf16 weight would grow.
+//                         STATE_SPACE adds skip times the token's own v, which is still in shared memory
 //
 // A slot needs no clearing: what a sequence has seen follows from its positions, and position 0 starts from zero.
 #include <initializer_list>
@@ -32,21 +44,25 @@
 
 namespace ft {
 
+enum : int { MEMORY = 0, STATE_SPACE = 1 };
+
 struct MemoryParams {
-  const void* q;            // rows of a packed projection with stride ld: head h at q + row * ld + h * dp
+  const void* q;            // packed rows with stride ld: head h at q + row * ld + h / group * dp
   const void* k;
   const void* v;            // head h at v + row * ld + h * vp
-  const void* gate;         // like v; null: no output gate
+  const void* gate;         // rows with stride ldg, heads like v's; null: no output gate
   const float* z;           // [rows, ldz]: gate pre-activations without bias, input gates at [h], forget gates at [f_off + h]
   const float* i_bias;      // [H]
   const float* f_bias;
   const float* norm;        // [H, vp]
+  const float* rate;        // STATE_SPACE (which has z and i_bias for the step sizes, and neither f_bias, norm, n nor m): [H]
+  const float* skip;        // [H]
   float* S;                 // [slots, H, dp, vp]
   float* n;                 // [slots, H, dp]
   float* m;                 // [slots, H]
   void* out;                // [rows, ldo], head h at h * vp
-  long long ld, ldz, ldo;
-  int f_off, H, dp, vp, vdim;
+  long long ld, ldg, ldz, ldo;
+  int f_off, H, group, dp, vp, vdim;   // group: heads that share q and k
   float q_scale, cap, eps, out_scale;
 };
 
@@ -61,6 +77,11 @@ __device__ __forceinline__ float mem_forget_gate(float z, float cap) {
   return fminf(c, 0.f) - log1pf(expf(-fabsf(c)));
 }
 
+// softplus and the decay of a step; decays are often within 1e-3 of one, where an error in the last place of exp would change the
+// length of the memory.
+__device__ __forceinline__ float state_step(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float state_decay(float rate, float dt) { return 1.f + expm1f(-rate * dt); }
+
 // ---------------------------------------------------------------- token by token
 // One block per (item, head).  Thread (r, c): rows r, r + groups, .. of the state and columns 4 c .. 4 c + 3 of each run of
 // 4 * lanes columns.  Items are portions (spans) or, with spans null, single rows.  The state of a longer portion is kept
@@ -74,7 +95,7 @@ struct MemoryItems {
   int in_smem;
 };
 
-template <typename T>
+template <typename T, int RULE>
 __global__ void __launch_bounds__(MS_THREADS)
 memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
   extern __shared__ float ms_sm[];
@@ -98,36 +119,49 @@ memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
   const long long sh = static_cast<long long>(slot) * p.H + h;
   float* S_mem = p.S + sh * p.dp * p.vp;
   float* S = it.in_smem ? s_state : S_mem;
+  const long long qk = static_cast<long long>(h / p.group) * p.dp;
   bool fresh = pos0 == 0;
-  float m = fresh ? 0.f : p.m[sh];
-  for (int d = tid; d < p.dp; d += MS_THREADS) s_n[d] = fresh ? 0.f : p.n[sh * p.dp + d];
+  float m = 0.f;
+  if constexpr (RULE == MEMORY) {
+    m = fresh ? 0.f : p.m[sh];
+    for (int d = tid; d < p.dp; d += MS_THREADS) s_n[d] = fresh ? 0.f : p.n[sh * p.dp + d];
+  }
   if (it.in_smem) {
     for (int i = tid * 4; i < p.dp * p.vp; i += MS_THREADS * 4)
       *reinterpret_cast<float4*>(s_state + i) = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(S_mem + i);
     fresh = false;
   }
-  const float bi = p.i_bias[h], bf = p.f_bias[h];
+  const float bi = p.i_bias[h], bf = RULE == MEMORY ? p.f_bias[h] : p.rate[h], skip = RULE == MEMORY ? 0.f : p.skip[h];
   for (int t = 0; t < rows; ++t, fresh = false) {
     const long long row = row0 + t;
     __syncthreads();                     // the state has been loaded; the previous row's vectors have been read
     for (int d = tid; d < p.dp; d += MS_THREADS) {
-      s_q[d] = mem_f32(static_cast<const T*>(p.q)[row * p.ld + static_cast<long long>(h) * p.dp + d]) * p.q_scale;
-      s_k[d] = mem_f32(static_cast<const T*>(p.k)[row * p.ld + static_cast<long long>(h) * p.dp + d]);
+      s_q[d] = mem_f32(static_cast<const T*>(p.q)[row * p.ld + qk + d]) * p.q_scale;
+      s_k[d] = mem_f32(static_cast<const T*>(p.k)[row * p.ld + qk + d]);
     }
     for (int d = tid; d < p.vp; d += MS_THREADS) s_v[d] = mem_f32(static_cast<const T*>(p.v)[row * p.ld + static_cast<long long>(h) * p.vp + d]);
-    const float gi = mem_input_gate(p.z[row * p.ldz + h] + bi, p.cap), gf = mem_forget_gate(p.z[row * p.ldz + p.f_off + h] + bf, p.cap);
-    const float mm = fmaxf(gf + m, gi);
-    const float keep = expf(gf + m - mm), add = expf(gi - mm);
-    m = mm;
-    __syncthreads();
-    float dot = 0.f;
-    for (int d = tid; d < p.dp; d += MS_THREADS) {
-      const float nn = keep * s_n[d] + add * s_k[d];
-      s_n[d] = nn;
-      dot += nn * s_q[d];
+    float keep, add;
+    if constexpr (RULE == MEMORY) {
+      const float gi = mem_input_gate(p.z[row * p.ldz + h] + bi, p.cap), gf = mem_forget_gate(p.z[row * p.ldz + p.f_off + h] + bf, p.cap);
+      const float mm = fmaxf(gf + m, gi);
+      keep = expf(gf + m - mm);
+      add = expf(gi - mm);
+      m = mm;
+    } else {
+      add = state_step(p.z[row * p.ldz + h] + bi);
+      keep = state_decay(bf, add);
     }
-    dot = warp_sum(dot);
-    if (lane == 0) s_red[warp] = dot;
+    __syncthreads();
+    if constexpr (RULE == MEMORY) {
+      float dot = 0.f;
+      for (int d = tid; d < p.dp; d += MS_THREADS) {
+        const float nn = keep * s_n[d] + add * s_k[d];
+        s_n[d] = nn;
+        dot += nn * s_q[d];
+      }
+      dot = warp_sum(dot);
+      if (lane == 0) s_red[warp] = dot;
+    }
     if (r < groups)
       for (int j = c * 4; j < p.vp; j += lanes * 4) {
         const float4 v4 = *reinterpret_cast<const float4*>(s_v + j);
@@ -145,7 +179,19 @@ memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
         *reinterpret_cast<float4*>(s_part + r * p.vp + j) = acc;
       }
     __syncthreads();
-    dot = 0.f;
+    if constexpr (RULE == STATE_SPACE) {
+      for (int j = tid; j < p.vp; j += MS_THREADS) {
+        float o = skip * s_v[j];
+        for (int g = 0; g < groups; ++g) o += s_part[g * p.vp + j];
+        if (p.gate) {
+          const float z = mem_f32(static_cast<const T*>(p.gate)[row * p.ldg + static_cast<long long>(h) * p.vp + j]);
+          o *= z / (1.f + expf(-z));
+        }
+        mem_store(static_cast<T*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.vp + j, o);
+      }
+      continue;
+    }
+    float dot = 0.f;
 #pragma unroll
     for (int w = 0; w < MS_THREADS / 32; ++w) dot += s_red[w];
     const float inv = 1.f / (fmaxf(fabsf(dot), expf(-m)) + 1e-6f);
@@ -166,13 +212,15 @@ memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
     const float rn = p.out_scale / sqrtf(sum / static_cast<float>(p.vdim) + p.eps);
     for (int j = tid; j < p.vp; j += MS_THREADS) {
       float o = s_part[j] * rn * p.norm[static_cast<long long>(h) * p.vp + j];
-      if (p.gate) o *= 1.f / (1.f + expf(-mem_f32(static_cast<const T*>(p.gate)[row * p.ld + static_cast<long long>(h) * p.vp + j])));
+      if (p.gate) o *= 1.f / (1.f + expf(-mem_f32(static_cast<const T*>(p.gate)[row * p.ldg + static_cast<long long>(h) * p.vp + j])));
       mem_store(static_cast<T*>(p.out) + row * p.ldo + static_cast<long long>(h) * p.vp + j, o);
     }
   }
   __syncthreads();
-  for (int d = tid; d < p.dp; d += MS_THREADS) p.n[sh * p.dp + d] = s_n[d];
-  if (tid == 0) p.m[sh] = m;
+  if constexpr (RULE == MEMORY) {
+    for (int d = tid; d < p.dp; d += MS_THREADS) p.n[sh * p.dp + d] = s_n[d];
+    if (tid == 0) p.m[sh] = m;
+  }
   if (it.in_smem)
     for (int i = tid * 4; i < p.dp * p.vp; i += MS_THREADS * 4) *reinterpret_cast<float4*>(S_mem + i) = *reinterpret_cast<const float4*>(s_state + i);
 }
@@ -288,6 +336,46 @@ memory_gates_kernel(const MemoryParams p, const MemoryChunks c) {
   if (threadIdx.x == 0) *m_slot = s_carry;
 }
 
+// The same for the state-space rule, where chunks do not wait for one another: a warp per (head, chunk).
+__global__ void __launch_bounds__(256)
+state_gates_kernel(const MemoryParams p, const MemoryChunks c) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long tasks = static_cast<long long>(c.n_chunks) * p.H;
+  for (long long task = static_cast<long long>(blockIdx.x) * 8 + warp; task < tasks; task += static_cast<long long>(gridDim.x) * 8) {
+    const int k = static_cast<int>(task / p.H), h = static_cast<int>(task - static_cast<long long>(k) * p.H);
+    const int row0 = c.chunks[4 * k + 1], rows = c.chunks[4 * k + 2], t0 = lane * 4;
+    const float bias = p.i_bias[h], rate = p.rate[h];
+    float dt[4], b[4], sum = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      dt[e] = t0 + e < rows ? state_step(p.z[(static_cast<long long>(row0) + t0 + e) * p.ldz + h] + bias) : 0.f;
+      sum -= rate * dt[e];
+      b[e] = sum;
+    }
+    float before = sum;                                // sums of the lanes ahead
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, before, o);
+      if (lane >= o) before += v;
+    }
+    const float total = __shfl_sync(0xffffffffu, before, 31);
+    before = __shfl_up_sync(0xffffffffu, before, 1);
+    if (lane == 0) before = 0.f;
+    const long long at = static_cast<long long>(h) * c.ldt + row0 + t0;
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (t0 + e < rows) {
+        const float b2 = (b[e] + before) * 1.4426950408889634f;
+        c.a2[at + e] = log2f(dt[e]) - b2;              // a step of zero: -inf, a weight of zero
+        c.x2[at + e] = -b2;
+      }
+    if (lane == 0) {
+      c.start2[task] = 0.f;
+      c.end2[task] = -total * 1.4426950408889634f;
+    }
+  }
+}
+
 // 16-byte unit `unit` of row `row` in a tile of 64-column pieces with 128-byte swizzle.
 __device__ __forceinline__ uint32_t mc_unit(int row, int unit) {
   return static_cast<uint32_t>(unit >> 3) * MC_CHUNK + static_cast<uint32_t>(row) * 128u + (static_cast<uint32_t>((unit & 7) ^ (row & 7)) << 4);
@@ -295,7 +383,7 @@ __device__ __forceinline__ uint32_t mc_unit(int row, int unit) {
 
 // U of one (chunk, head).  The keys' tile [128 tokens, 128] is weighted in place (its low halves go to a second tile) and
 // multiplied as the transposed A operand with V.
-template <int VC>
+template <int VC, int RULE>
 __global__ void __launch_bounds__(MC_UPDATE_THREADS)
 memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const MemoryParams p, const MemoryChunks c) {
   constexpr int OFF_LO = 2 * MC_CHUNK, OFF_V = 4 * MC_CHUNK, OFF_N = OFF_V + VC * MC_CHUNK, OFF_W = OFF_N + 16 * 128 * 4, OFF_BAR = OFF_W + MC_ROWS * 4;
@@ -332,7 +420,7 @@ memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
   const uint32_t tmem = *tmem_slot;
   if (tid == 0) {
     mbar_expect_tx(bar_k, 2 * MC_CHUNK);
-    for (int i = 0; i < 2; ++i) tma_load_2d(sbase + i * MC_CHUNK, &tmK, bar_k, h * p.dp + i * 64, row0);
+    for (int i = 0; i < 2; ++i) tma_load_2d(sbase + i * MC_CHUNK, &tmK, bar_k, h / p.group * p.dp + i * 64, row0);
     mbar_expect_tx(bar_v, VC * MC_CHUNK);
     for (int i = 0; i < VC; ++i) tma_load_2d(sbase + OFF_V + i * MC_CHUNK, &tmV, bar_v, h * p.vp + i * 64, row0);
   }
@@ -352,7 +440,7 @@ memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         f[e] *= w;
-        acc[e] += f[e];
+        if constexpr (RULE == MEMORY) acc[e] += f[e];
       }
       const uint4 packed = pack8(f);
       unpack8(packed, hi);
@@ -361,8 +449,10 @@ memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
       *at = packed;
       *reinterpret_cast<uint4*>(smem + OFF_LO + mc_unit(row, unit)) = pack8(f);
     }
+    if constexpr (RULE == MEMORY) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) s_n[r0 * 128 + unit * 8 + e] = acc[e];
+      for (int e = 0; e < 8; ++e) s_n[r0 * 128 + unit * 8 + e] = acc[e];
+    }
   }
   fence_proxy_async_smem();
   __syncthreads();
@@ -376,7 +466,7 @@ memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
                     make_smem_desc_sw128(sbase + OFF_V + kk * 2048, MC_CHUNK, 1024), idesc, (half > 0 || kk > 0) ? 1u : 0u);
     umma_commit(bar_m);
   }
-  if (tid < p.dp && ok) {
+  if (RULE == MEMORY && tid < p.dp && ok) {
     float n = 0.f;
 #pragma unroll
     for (int g = 0; g < 16; ++g) n += s_n[g * 128 + tid];
@@ -419,6 +509,7 @@ memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
 
 // The states of a portion's chunks, one after another: a thread owns four elements of S (and the first block one of n).
 constexpr int MC_AHEAD = 4;       // contributions loaded together
+template <int RULE>
 __global__ void __launch_bounds__(256)
 memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
   const int h = blockIdx.y;
@@ -459,7 +550,7 @@ memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
     }
     if (col < p.vp) *S = s;
   }
-  if (blockIdx.x == 0 && static_cast<int>(threadIdx.x) < p.dp) {
+  if (RULE == MEMORY && blockIdx.x == 0 && static_cast<int>(threadIdx.x) < p.dp) {
     float n = pos0 > 0 ? p.n[sh * p.dp + threadIdx.x] : 0.f;
     for (int k = 0; k < n_chunks; ++k) {
       const long long at = (static_cast<long long>(first + k) * p.H + h) * p.dp + threadIdx.x;
@@ -480,7 +571,7 @@ struct MemOut {
   static constexpr uint32_t COLS = VC <= 2 ? 256 : 512, COL_LOW = 64, COL_O = 128;      // scores (then P high | low), outputs
 };
 
-template <int DC, int VC>
+template <int DC, int VC, int RULE>
 __global__ void __launch_bounds__(MC_OUT_THREADS)
 memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                      const __grid_constant__ CUtensorMap tmS, const __grid_constant__ CUtensorMap tmG, const MemoryParams p,
@@ -512,8 +603,8 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     tmem_relinquish();
   }
   if (tid < MC_ROWS) s_a[tid] = tid < rows ? c.a2[gate_at + tid] : -INFINITY;
-  if (tid < p.dp) s_nb[tid] = fresh ? 0.f : c.nb[ph * p.dp + tid];
-  for (int i = tid; i < p.vp; i += MC_OUT_THREADS) s_w[i] = p.norm[static_cast<long long>(h) * p.vp + i];
+  if (RULE == MEMORY && tid < p.dp) s_nb[tid] = fresh ? 0.f : c.nb[ph * p.dp + tid];
+  if (RULE == MEMORY) for (int i = tid; i < p.vp; i += MC_OUT_THREADS) s_w[i] = p.norm[static_cast<long long>(h) * p.vp + i];
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -538,8 +629,8 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       };
       mbar_expect_tx(bar(QK), 2 * DC * MC_CHUNK);
       for (int i = 0; i < DC; ++i) {
-        tma_load_2d(sQ + i * MC_CHUNK, &tmQ, bar(QK), h * p.dp + i * 64, row0);
-        tma_load_2d(sK + i * MC_CHUNK, &tmK, bar(QK), h * p.dp + i * 64, row0);
+        tma_load_2d(sQ + i * MC_CHUNK, &tmQ, bar(QK), h / p.group * p.dp + i * 64, row0);
+        tma_load_2d(sK + i * MC_CHUNK, &tmK, bar(QK), h / p.group * p.dp + i * 64, row0);
       }
       if (fresh) load_v();
       else load_state(HIGH, sV, ph * p.dp);
@@ -588,13 +679,14 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     }
   } else {
     const bool row_ok = tid < rows;
-    const float x2 = row_ok ? c.x2[gate_at + tid] : 0.f, floor_m = row_ok ? c.floor[gate_at + tid] : 1.f;
+    const float x2 = row_ok ? c.x2[gate_at + tid] : 0.f, floor_m = RULE == MEMORY && row_ok ? c.floor[gate_at + tid] : 1.f;
+    const float skip = RULE == STATE_SPACE ? p.skip[h] : 0.f;
     const float inter = (fresh || !row_ok) ? 0.f : exp2f(c.start2[ph] - x2) * p.q_scale;
     const uint32_t lane_addr = tmem + (static_cast<uint32_t>(warp * 32) << 16);
     float den = 0.f;
     auto wait = [&](int i) { return __all_sync(0xffffffffu, mbar_wait(bar(i), 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE)); };
     bool ok = wait(QK);
-    if (ok && !fresh) {                                // q times the normaliser at the chunk's start
+    if (RULE == MEMORY && ok && !fresh) {              // q times the normaliser at the chunk's start
       for (int u = 0; u < p.dp / 8; ++u) {
         float f[8];
         unpack8(*reinterpret_cast<const uint4*>(smem + mc_unit(tid, u)), f);
@@ -624,7 +716,7 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
               const int key = j * 32 + 2 * i + e;
               const float w = fast_exp2(s_a[key] - x2);
               v[e] = key <= tid ? __uint_as_float(t[2 * i + e]) * p.q_scale * w : 0.f;
-              den += v[e];
+              if constexpr (RULE == MEMORY) den += v[e];
             }
             hi[i] = pack_bf16x2(v[0], v[1]);
             const float2 r = unpack_bf16x2(hi[i]);
@@ -671,20 +763,23 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     if (ok) ok = wait(OUT);
     if (ok) {
       tc_fence_after();
-      const float inv = 1.f / (fmaxf(fabsf(den), floor_m) + 1e-6f);
-      float sum = 0.f;
+      float r = 1.f;
+      if constexpr (RULE == MEMORY) {
+        const float inv = 1.f / (fmaxf(fabsf(den), floor_m) + 1e-6f);
+        float sum = 0.f;
 #pragma unroll
-      for (int col = 0; col < VC * 64; col += 32) {
-        uint32_t t[32];
-        tmem_ld_32x32(lane_addr + Cfg::COL_O + col, t);
-        tmem_ld_wait();
+        for (int col = 0; col < VC * 64; col += 32) {
+          uint32_t t[32];
+          tmem_ld_32x32(lane_addr + Cfg::COL_O + col, t);
+          tmem_ld_wait();
 #pragma unroll
-        for (int e = 0; e < 32; ++e) {
-          const float o = __uint_as_float(t[e]) * inv;
-          if (col + e < p.vp) sum += o * o;
+          for (int e = 0; e < 32; ++e) {
+            const float o = __uint_as_float(t[e]) * inv;
+            if (col + e < p.vp) sum += o * o;
+          }
         }
+        r = p.out_scale * inv / sqrtf(sum / static_cast<float>(p.vdim) + p.eps);
       }
-      const float r = p.out_scale * inv / sqrtf(sum / static_cast<float>(p.vdim) + p.eps);
       if (p.gate) ok = wait(GATE);
 #pragma unroll 1
       for (int col = 0; col < VC * 64; col += 32) {
@@ -697,11 +792,16 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
           uint4* at = reinterpret_cast<uint4*>(smem + mc_unit(tid, col / 8 + g));
           float f[8], z[8];
 #pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(t[g * 8 + e]) * r * s_w[col + g * 8 + e];
+          for (int e = 0; e < 8; ++e) f[e] = RULE == MEMORY ? __uint_as_float(t[g * 8 + e]) * r * s_w[col + g * 8 + e] : __uint_as_float(t[g * 8 + e]);
+          if constexpr (RULE == STATE_SPACE) {
+            unpack8(*reinterpret_cast<const uint4*>(smem + Cfg::OFF_V + mc_unit(tid, col / 8 + g)), z);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] += skip * z[e];
+          }
           if (p.gate) {
             unpack8(*at, z);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-z[e]));
+            for (int e = 0; e < 8; ++e) f[e] = __fdividef(RULE == MEMORY ? f[e] : f[e] * z[e], 1.f + __expf(-z[e]));
           }
           *at = pack8(f);
         }
@@ -731,18 +831,55 @@ static bool mem_aligned(std::initializer_list<const void*> ps) {
   return (v & 15) == 0;
 }
 
-static int memory_params(MemoryParams& p, const void* q, const void* k, const void* v, const void* gate, long long ld, const float* z,
-                         long long ldz, int f_off, const float* i_bias, const float* f_bias, const float* norm, float* S, float* n,
-                         float* m, void* out, long long ldo, int H, int dp, int vp, int vdim, float q_scale, float cap, float eps,
-                         float out_scale) {
-  FT_REQUIRE(q && k && v && z && i_bias && f_bias && norm && S && n && m && out, "matrix memory: null pointer");
-  FT_REQUIRE(H > 0 && H < 65536 && dp > 0 && dp % 16 == 0 && vp > 0 && vp % 16 == 0 && vdim > 0 && vdim <= vp && ld % 8 == 0 && ldo % 8 == 0 &&
-                 ldo >= static_cast<long long>(H) * vp && f_off >= H && ldz >= f_off + H && cap > 0.f,
-             "matrix memory: %d heads of %d x %d", H, dp, vp);
-  FT_REQUIRE(mem_aligned({q, k, v, gate, S, n, out, norm}), "matrix memory: pointers must be 16-byte aligned");
-  p.q = q; p.k = k; p.v = v; p.gate = gate; p.z = z; p.i_bias = i_bias; p.f_bias = f_bias; p.norm = norm; p.S = S; p.n = n; p.m = m;
-  p.out = out; p.ld = ld; p.ldz = ldz; p.ldo = ldo; p.f_off = f_off; p.H = H; p.dp = dp; p.vp = vp; p.vdim = vdim;
+static int memory_params(MemoryParams& p, const void* q, const void* k, const void* v, long long ld, const void* gate, long long ldg, const float* z,
+                         long long ldz, const float* i_bias, float* S, void* out, long long ldo, int H, int group, int dp, int vp) {
+  FT_REQUIRE(q && k && v && z && i_bias && S && out, "matrix memory: null pointer");
+  FT_REQUIRE(H > 0 && H < 65536 && group > 0 && H % group == 0 && dp > 0 && dp % 16 == 0 && vp > 0 && vp % 16 == 0 && ld % 8 == 0 && ldo % 8 == 0 &&
+                 ldg % 8 == 0 && (!gate || ldg >= static_cast<long long>(H) * vp) && ldo >= static_cast<long long>(H) * vp && ldz >= H,
+             "matrix memory: %d heads of %d x %d in groups of %d", H, dp, vp, group);
+  FT_REQUIRE(mem_aligned({q, k, v, gate, S, out}), "matrix memory: pointers must be 16-byte aligned");
+  p = MemoryParams{};
+  p.q = q; p.k = k; p.v = v; p.gate = gate; p.z = z; p.i_bias = i_bias; p.S = S; p.out = out;
+  p.ld = ld; p.ldg = ldg; p.ldz = ldz; p.ldo = ldo; p.H = H; p.group = group; p.dp = dp; p.vp = vp; p.vdim = vp;
+  p.q_scale = 1.f; p.out_scale = 1.f; p.cap = 1.f;
+  return FT_E_OK;
+}
+
+// What the memory rule has beside the common operands.
+static int memory_gates(MemoryParams& p, int f_off, const float* f_bias, const float* norm, float* n, float* m, int vdim, float q_scale, float cap,
+                        float eps, float out_scale) {
+  FT_REQUIRE(f_bias && norm && n && m && vdim > 0 && vdim <= p.vp && f_off >= p.H && p.ldz >= f_off + p.H && cap > 0.f, "matrix memory: gates or null pointer");
+  FT_REQUIRE(mem_aligned({n, norm}), "matrix memory: pointers must be 16-byte aligned");
+  p.f_off = f_off; p.f_bias = f_bias; p.norm = norm; p.n = n; p.m = m; p.vdim = vdim;
   p.q_scale = q_scale; p.cap = cap; p.eps = eps; p.out_scale = out_scale;
+  return FT_E_OK;
+}
+
+static int state_rates(MemoryParams& p, const float* rate, const float* skip) {
+  FT_REQUIRE(rate && skip, "state space: null pointer");
+  p.rate = rate; p.skip = skip;
+  return FT_E_OK;
+}
+
+template <int RULE>
+static int run_steps(const MemoryParams& p, const int* spans, const int* pos, const int* slots, int n_items, int f32, cudaStream_t stream) {
+  FT_REQUIRE(spans || (pos && slots), "matrix memory: neither portions nor rows");
+  if (n_items <= 0) return FT_E_OK;
+  MemoryItems it = {spans, pos, slots, 0};
+  const int lanes = p.vp / 4 < MS_THREADS ? p.vp / 4 : MS_THREADS, groups = MS_THREADS / lanes;
+  size_t smem = sizeof(float) * (3 * static_cast<size_t>(p.dp) + p.vp + static_cast<size_t>(groups) * p.vp + 32);
+  const size_t state = sizeof(float) * static_cast<size_t>(p.dp) * p.vp;
+  if (spans && smem + state <= 200 * 1024) {
+    it.in_smem = 1;
+    smem += state;
+  }
+  FT_REQUIRE(smem <= 200 * 1024, "matrix memory: heads of %d x %d are too large", p.dp, p.vp);
+  const dim3 grid(n_items, p.H);
+  auto kern = f32 ? memory_steps_kernel<float, RULE> : memory_steps_kernel<__nv_bfloat16, RULE>;
+  FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  kern<<<grid, MS_THREADS, smem, stream>>>(p, it);
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
   return FT_E_OK;
 }
 
@@ -760,26 +897,22 @@ FT_API int ft_memory_steps(const void* q, const void* k, const void* v, const vo
                            cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   MemoryParams p;
-  if (int rc = memory_params(p, q, k, v, gate, ld, z, ldz, f_off, i_bias, f_bias, norm, S, n, m, out, ldo, H, dp, vp, vdim, q_scale, cap, eps, out_scale))
-    return rc;
-  FT_REQUIRE(spans || (pos && slots), "ft_memory_steps: neither portions nor rows");
-  if (n_items <= 0) return FT_E_OK;
-  MemoryItems it = {spans, pos, slots, 0};
-  const int lanes = vp / 4 < MS_THREADS ? vp / 4 : MS_THREADS, groups = MS_THREADS / lanes;
-  size_t smem = sizeof(float) * (3 * static_cast<size_t>(dp) + vp + static_cast<size_t>(groups) * vp + 32);
-  const size_t state = sizeof(float) * static_cast<size_t>(dp) * vp;
-  if (spans && smem + state <= 200 * 1024) {
-    it.in_smem = 1;
-    smem += state;
-  }
-  FT_REQUIRE(smem <= 200 * 1024, "ft_memory_steps: heads of %d x %d are too large", dp, vp);
-  const dim3 grid(n_items, H);
-  auto kern = f32 ? memory_steps_kernel<float> : memory_steps_kernel<__nv_bfloat16>;
-  FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-  kern<<<grid, MS_THREADS, smem, stream>>>(p, it);
-  FT_CUDA_CHECK(cudaGetLastError());
-  count_launch();
-  return FT_E_OK;
+  if (int rc = memory_params(p, q, k, v, ld, gate, ld, z, ldz, i_bias, S, out, ldo, H, 1, dp, vp)) return rc;
+  if (int rc = memory_gates(p, f_off, f_bias, norm, n, m, vdim, q_scale, cap, eps, out_scale)) return rc;
+  return run_steps<MEMORY>(p, spans, pos, slots, n_items, f32, stream);
+}
+
+// The state-space rule token by token: v (x) [rows, H * vp], k and q (B and C) [rows, H / group * dp] with row stride ld, gate [rows, ldg] or
+// null, z fp32 [rows, ldz] (step sizes ahead of bias and softplus), bias, rate and skip fp32 [H], S fp32 [slots, H, dp, vp].  Items as in
+// ft_memory_steps.
+FT_API int ft_state_steps(const void* q, const void* k, const void* v, long long ld, const void* gate, long long ldg, const float* z, long long ldz,
+                          const float* bias, const float* rate, const float* skip, float* S, void* out, long long ldo, int H, int group, int dp,
+                          int vp, const int* spans, const int* pos, const int* slots, int n_items, int f32, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  MemoryParams p;
+  if (int rc = memory_params(p, q, k, v, ld, gate, ldg, z, ldz, bias, S, out, ldo, H, group, dp, vp)) return rc;
+  if (int rc = state_rates(p, rate, skip)) return rc;
+  return run_steps<STATE_SPACE>(p, spans, pos, slots, n_items, f32, stream);
 }
 
 // Whole portions of bf16 rows in chunks (see the top of this file): dp up to 128, vp up to 256.  rows: rows of the packed
@@ -798,42 +931,44 @@ static long long memory_scratch_at(int rows, int H, int dp, int vp, int n_chunks
 
 FT_API long long ft_memory_scratch(int rows, int H, int dp, int vp, int n_chunks) { return memory_scratch_at(rows, H, dp, vp, n_chunks, nullptr); }
 
-template <int DC, int VC>
+template <int DC, int VC, int RULE>
 static int launch_memory(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const CUtensorMap& tg,
                          const MemoryParams& p, const MemoryChunks& c, int device, cudaStream_t stream) {
   constexpr int UPDATE_SMEM = (4 + VC) * MC_CHUNK + 16 * 128 * 4 + MC_ROWS * 4 + 64 + 1024;
   constexpr int OUT_SMEM = MemOut<DC, VC>::SMEM;
+  auto update = memory_update_kernel<VC, RULE>;
+  auto output = memory_output_kernel<DC, VC, RULE>;
   static bool attr_set[64] = {false};
   if (!attr_set[device]) {
-    FT_CUDA_CHECK(cudaFuncSetAttribute(memory_update_kernel<VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, UPDATE_SMEM));
-    FT_CUDA_CHECK(cudaFuncSetAttribute(memory_output_kernel<DC, VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, OUT_SMEM));
+    FT_CUDA_CHECK(cudaFuncSetAttribute(update, cudaFuncAttributeMaxDynamicSharedMemorySize, UPDATE_SMEM));
+    FT_CUDA_CHECK(cudaFuncSetAttribute(output, cudaFuncAttributeMaxDynamicSharedMemorySize, OUT_SMEM));
     attr_set[device] = true;
   }
-  memory_gates_kernel<<<dim3(p.H, c.n_spans), MC_GATE_WARPS * 32, 0, stream>>>(p, c);
+  if (RULE == MEMORY) {
+    memory_gates_kernel<<<dim3(p.H, c.n_spans), MC_GATE_WARPS * 32, 0, stream>>>(p, c);
+  } else {
+    const long long blocks = (static_cast<long long>(c.n_chunks) * p.H + 7) / 8, cap = sm_count(device) * 16;
+    state_gates_kernel<<<static_cast<int>(blocks < cap ? blocks : cap), 256, 0, stream>>>(p, c);
+  }
   FT_CUDA_CHECK(cudaGetLastError());
-  memory_update_kernel<VC><<<dim3(c.n_chunks, p.H), MC_UPDATE_THREADS, UPDATE_SMEM, stream>>>(tk, tv, p, c);
+  update<<<dim3(c.n_chunks, p.H), MC_UPDATE_THREADS, UPDATE_SMEM, stream>>>(tk, tv, p, c);
   FT_CUDA_CHECK(cudaGetLastError());
-  memory_carry_kernel<<<dim3((p.dp * c.vw / 4 + 255) / 256, p.H, c.n_spans), 256, 0, stream>>>(p, c);
+  memory_carry_kernel<RULE><<<dim3((p.dp * c.vw / 4 + 255) / 256, p.H, c.n_spans), 256, 0, stream>>>(p, c);
   FT_CUDA_CHECK(cudaGetLastError());
-  memory_output_kernel<DC, VC><<<dim3(c.n_chunks, p.H), MC_OUT_THREADS, OUT_SMEM, stream>>>(tq, tk, tv, ts, tg, p, c);
+  output<<<dim3(c.n_chunks, p.H), MC_OUT_THREADS, OUT_SMEM, stream>>>(tq, tk, tv, ts, tg, p, c);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch(4);
   return FT_E_OK;
 }
 
-FT_API int ft_memory_chunks(const void* q, const void* k, const void* v, const void* gate, long long ld, const float* z, long long ldz,
-                            int f_off, const float* i_bias, const float* f_bias, const float* norm, float* S, float* n, float* m,
-                            void* out, long long ldo, int H, int dp, int vp, int vdim, float q_scale, float cap, float eps,
-                            float out_scale, int rows, const int* spans, int n_spans, const int* span_chunks, const int* chunks,
-                            int n_chunks, void* scratch, int device, cudaStream_t stream) {
-  if (int _rc = ft::ensure_device(device)) return _rc;
-  MemoryParams p;
-  if (int rc = memory_params(p, q, k, v, gate, ld, z, ldz, f_off, i_bias, f_bias, norm, S, n, m, out, ldo, H, dp, vp, vdim, q_scale, cap, eps, out_scale))
-    return rc;
-  FT_REQUIRE(dp <= 128 && vp <= 256, "ft_memory_chunks: heads of %d x %d are too large", dp, vp);
-  FT_REQUIRE(rows > 0 && spans && span_chunks && chunks && scratch && (reinterpret_cast<uintptr_t>(scratch) & 255) == 0, "ft_memory_chunks: null pointer or unaligned scratch");
+template <int RULE>
+static int run_chunks(const MemoryParams& p, int rows, const int* spans, int n_spans, const int* span_chunks, const int* chunks, int n_chunks,
+                      void* scratch, int device, cudaStream_t stream) {
+  const int H = p.H, dp = p.dp, vp = p.vp;
+  FT_REQUIRE(dp <= 128 && vp <= 256, "matrix memory: heads of %d x %d are too large for chunks", dp, vp);
+  FT_REQUIRE(rows > 0 && spans && span_chunks && chunks && scratch && (reinterpret_cast<uintptr_t>(scratch) & 255) == 0, "matrix memory: null pointer or unaligned scratch");
   if (n_spans <= 0 || n_chunks <= 0) return FT_E_OK;
-  FT_REQUIRE(n_spans < 65536 && 2ll * n_chunks * H * dp < (1ll << 31), "ft_memory_chunks: too many portions or chunks");
+  FT_REQUIRE(n_spans < 65536 && 2ll * n_chunks * H * dp < (1ll << 31), "matrix memory: too many portions or chunks");
   long long at[9];
   memory_scratch_at(rows, H, dp, vp, n_chunks, at);
   char* base = static_cast<char*>(scratch);
@@ -845,20 +980,47 @@ FT_API int ft_memory_chunks(const void* q, const void* k, const void* v, const v
   c.ldt = (rows + 31) / 32 * 32; c.n_spans = n_spans; c.n_chunks = n_chunks; c.vw = (vp + 63) / 64 * 64;
   c.status = device_status_word(device);
   CUtensorMap tq, tk, tv, ts, tg;
-  const uint64_t stride = static_cast<uint64_t>(ld) * 2;
-  if (int rc = make_tmap_2d(&tq, q, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
-  if (int rc = make_tmap_2d(&tk, k, 2, static_cast<uint64_t>(H) * dp, rows, stride, 64, MC_ROWS, 3)) return rc;
-  if (int rc = make_tmap_2d(&tv, v, 2, static_cast<uint64_t>(H) * vp, rows, stride, 64, MC_ROWS, 3)) return rc;
-  if (int rc = make_tmap_2d(&tg, gate ? gate : v, 2, static_cast<uint64_t>(H) * vp, rows, stride, 64, MC_ROWS, 3)) return rc;
+  const uint64_t stride = static_cast<uint64_t>(p.ld) * 2, keys = static_cast<uint64_t>(H / p.group) * dp;
+  if (int rc = make_tmap_2d(&tq, p.q, 2, keys, rows, stride, 64, MC_ROWS, 3)) return rc;
+  if (int rc = make_tmap_2d(&tk, p.k, 2, keys, rows, stride, 64, MC_ROWS, 3)) return rc;
+  if (int rc = make_tmap_2d(&tv, p.v, 2, static_cast<uint64_t>(H) * vp, rows, stride, 64, MC_ROWS, 3)) return rc;
+  if (int rc = make_tmap_2d(&tg, p.gate ? p.gate : p.v, 2, static_cast<uint64_t>(H) * vp, rows, p.gate ? static_cast<uint64_t>(p.ldg) * 2 : stride, 64, MC_ROWS, 3)) return rc;
   if (int rc = make_tmap_2d(&ts, c.Sb, 2, c.vw, 2 * static_cast<uint64_t>(n_chunks) * H * dp, static_cast<uint64_t>(c.vw) * 2, 64, dp, 3)) return rc;
 #define FT_MC(DCN)                                                              \
   switch (c.vw / 64) {                                                          \
-    case 1: return launch_memory<DCN, 1>(tq, tk, tv, ts, tg, p, c, device, stream); \
-    case 2: return launch_memory<DCN, 2>(tq, tk, tv, ts, tg, p, c, device, stream); \
-    case 3: return launch_memory<DCN, 3>(tq, tk, tv, ts, tg, p, c, device, stream); \
-    default: return launch_memory<DCN, 4>(tq, tk, tv, ts, tg, p, c, device, stream); \
+    case 1: return launch_memory<DCN, 1, RULE>(tq, tk, tv, ts, tg, p, c, device, stream); \
+    case 2: return launch_memory<DCN, 2, RULE>(tq, tk, tv, ts, tg, p, c, device, stream); \
+    case 3: return launch_memory<DCN, 3, RULE>(tq, tk, tv, ts, tg, p, c, device, stream); \
+    default: return launch_memory<DCN, 4, RULE>(tq, tk, tv, ts, tg, p, c, device, stream); \
   }
   if (dp <= 64) { FT_MC(1) }
   FT_MC(2)
 #undef FT_MC
+}
+
+FT_API int ft_memory_chunks(const void* q, const void* k, const void* v, const void* gate, long long ld, const float* z, long long ldz,
+                            int f_off, const float* i_bias, const float* f_bias, const float* norm, float* S, float* n, float* m,
+                            void* out, long long ldo, int H, int dp, int vp, int vdim, float q_scale, float cap, float eps,
+                            float out_scale, int rows, const int* spans, int n_spans, const int* span_chunks, const int* chunks,
+                            int n_chunks, void* scratch, int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  MemoryParams p;
+  if (int rc = memory_params(p, q, k, v, ld, gate, ld, z, ldz, i_bias, S, out, ldo, H, 1, dp, vp)) return rc;
+  if (int rc = memory_gates(p, f_off, f_bias, norm, n, m, vdim, q_scale, cap, eps, out_scale)) return rc;
+  return run_chunks<MEMORY>(p, rows, spans, n_spans, span_chunks, chunks, n_chunks, scratch, device, stream);
+}
+
+// The state-space rule over whole portions of bf16 rows in chunks: operands as in ft_state_steps, portions and chunks as in
+// ft_memory_chunks, scratch of ft_state_scratch bytes.
+FT_API long long ft_state_scratch(int rows, int H, int dp, int vp, int n_chunks) { return memory_scratch_at(rows, H, dp, vp, n_chunks, nullptr); }
+
+FT_API int ft_state_chunks(const void* q, const void* k, const void* v, long long ld, const void* gate, long long ldg, const float* z, long long ldz,
+                           const float* bias, const float* rate, const float* skip, float* S, void* out, long long ldo, int H, int group, int dp,
+                           int vp, int rows, const int* spans, int n_spans, const int* span_chunks, const int* chunks, int n_chunks, void* scratch,
+                           int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  MemoryParams p;
+  if (int rc = memory_params(p, q, k, v, ld, gate, ldg, z, ldz, bias, S, out, ldo, H, group, dp, vp)) return rc;
+  if (int rc = state_rates(p, rate, skip)) return rc;
+  return run_chunks<STATE_SPACE>(p, rows, spans, n_spans, span_chunks, chunks, n_chunks, scratch, device, stream);
 }

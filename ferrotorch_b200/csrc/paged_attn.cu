@@ -15,7 +15,9 @@
 //                       optional output gate per head.
 //                       A row may see a window of the most recent keys only, or those of its own chunk; a
 //                       bias that grows with the distance may be taken off the scores, and a learned number
-//                       per head (a sink) may join the denominator.
+//                       per head (a sink) may join the denominator.  Ahead of a window it may see the means of
+//                       whole blocks of keys and values.
+//   ft_pool_blocks      these means, of the blocks that end among the rows of a step.
 //   ft_paged_rows       the same for any mixture of rows (each with its own sequence and number of
 //                       visible keys), any head sizes, bf16 or fp32: the exact, simple kernel.
 // Decode attention is bandwidth bound (every cached byte is read once per step).  Key / value head
@@ -25,6 +27,7 @@
 // and V with one row per warp step; it serves size 64, and queries that are not 16-byte aligned.
 #include "attn_row.cuh"
 #include "ft_host.h"
+#include "row_vec.cuh"
 
 namespace ft {
 
@@ -47,6 +50,45 @@ __global__ void kv_append_kernel(const uint4* __restrict__ k_new, const uint4* _
     for (int i = threadIdx.x; i < max(kv16, vv16); i += blockDim.x) {
       if (i < kv16) k_cache[token * kv16 + i] = k_new[t * ldk16 + i];
       if (i < vv16) v_cache[token * vv16 + i] = v_new[t * ldv16 + i];
+    }
+  }
+}
+
+// Row i ends a block when (pos[i] + 1) % pool == 0: the means of its pool keys and values (their rows are in the cache) go to the
+// block's place.  A thread owns eight elements of a token's keys or values.
+constexpr int PB_THREADS = 128;
+template <typename T>
+__global__ void __launch_bounds__(PB_THREADS)
+pool_blocks_kernel(const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ k_pool, T* __restrict__ v_pool,
+                   const int* __restrict__ block_table, const int* __restrict__ pos, const int* __restrict__ slots, int rows, int kw, int vw,
+                   int pool, int per_page, int block_size, int max_blocks, int num_blocks) {
+  const float inv = 1.f / static_cast<float>(pool);
+  for (int row = blockIdx.x; row < rows; row += gridDim.x) {
+    const int last = pos[row];
+    if ((last + 1) % pool != 0) continue;
+    const int* bt = block_table + static_cast<long long>(slots[row]) * max_blocks;
+    const int page = last / block_size, first = last + 1 - pool;
+    if (page >= max_blocks || bt[page] < 0 || bt[page] >= num_blocks) continue;   // a row of no sequence
+    const long long dst = static_cast<long long>(bt[page]) * per_page + (last / pool - page * block_size / pool);
+    for (int i = (blockIdx.y * PB_THREADS + threadIdx.x) * 8; i < kw + vw; i += gridDim.y * PB_THREADS * 8) {
+      const bool is_k = i < kw;
+      const int c = is_k ? i : i - kw, width = is_k ? kw : vw;
+      const T* src = is_k ? k_cache : v_cache;
+      float sum[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum[e] = 0.f;
+#pragma unroll 8
+      for (int j = 0; j < pool; ++j) {
+        const int p = first + j;
+        const int blk = min(max(__ldg(bt + p / block_size), 0), num_blocks - 1);
+        float f[8];
+        load8(src + (static_cast<long long>(blk) * block_size + p % block_size) * width + c, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum[e] += f[e];
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sum[e] *= inv;
+      store8((is_k ? k_pool : v_pool) + dst * width + c, sum);
     }
   }
 }
@@ -297,8 +339,8 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
                        const int* __restrict__ row_slot, const int* __restrict__ ctx_len, __nv_bfloat16* __restrict__ out,
                        float* __restrict__ part_o, float* __restrict__ part_ml, int Hq, int Hkv, int D, int Dv, int g_real,
                        long long ldq, long long ldo, int block_size, int max_blocks, int num_blocks, float scale_log2,
-                       int n_splits, KeyRange range, const float* __restrict__ slopes, const float* __restrict__ sink, HeadGate gate,
-                       float out_scale, int* status) {
+                       int n_splits, KeyRange range, PooledKeys pooled, const float* __restrict__ slopes, const float* __restrict__ sink,
+                       HeadGate gate, float out_scale, int* status) {
   using Cfg = PtCfg<HD>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -317,10 +359,13 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int len = ctx_len[b];
   const int first = range.first_visible(len);
-  const int tiles_end = (len + PT_TILE - 1) / PT_TILE;
-  const int tiles_per_split = (tiles_end - first / PT_TILE + n_splits - 1) / n_splits;
-  const int tile_lo = first / PT_TILE + split * tiles_per_split;
-  const int n_tiles = max(0, min(tiles_end, tile_lo + tiles_per_split) - tile_lo);
+  // tiles of pooled blocks, then tiles of keys from the first visible one's on; tile_lo counts in this order
+  const int n_pool = pooled.count(first), pool_tiles = (n_pool + PT_TILE - 1) / PT_TILE;
+  const int key_tile = first / PT_TILE - pool_tiles;             // tile t holds keys from (key_tile + t) * PT_TILE on
+  const int tiles_all = pool_tiles + max(0, (len + PT_TILE - 1) / PT_TILE - first / PT_TILE);
+  const int tiles_per_split = (tiles_all + n_splits - 1) / n_splits;
+  const int tile_lo = split * tiles_per_split;
+  const int n_tiles = max(0, min(tiles_all, tile_lo + tiles_per_split) - tile_lo);
 
   if (threadIdx.x == 0) {
     *abort_word = 0;
@@ -387,24 +432,38 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
         const int st = t % PT_STAGES;
         ok = mbar_wait(bar(ST_EMPTY + st), ((t / PT_STAGES) & 1) ^ 1u, abort_word, FT_ERR_TIMEOUT_PRODUCER);
         if (ok) {
-          const int key0 = (tile_lo + t) * PT_TILE;
           const uint32_t sK = sbase + st * Cfg::STAGE_BYTES + chunk_off, sV = sK + Cfg::K_BYTES;
-#pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            const int row = row0 + 8 * i;
-            const int key = key0 + row;
-            const int page = key / block_size;
-            int blk = (key < len && page < max_blocks) ? __ldg(bt + page) : 0;
-            blk = min(max(blk, 0), num_blocks - 1);
-            const long long src = ((static_cast<long long>(blk) * block_size + key % block_size) * Hkv + kvh);
+          auto copy = [&](int row, const __nv_bfloat16* k, const __nv_bfloat16* v, long long src, bool there) {
             const uint32_t dst = static_cast<uint32_t>(row) * 128u + (static_cast<uint32_t>((unit & 7) ^ (row & 7)) << 4);
-            const uint32_t nbytes = key < len ? 16u : 0u;   // rows past the context are zero-filled
+            const uint32_t nbytes = there ? 16u : 0u;       // rows past the context are zero-filled
             if (has_k)
               asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sK + dst),
-                           "l"(k_cache + src * D + unit * 8), "r"(nbytes) : "memory");
+                           "l"(k + src * D + unit * 8), "r"(nbytes) : "memory");
             if (has_v)
               asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sV + dst),
-                           "l"(v_cache + src * Dv + unit * 8), "r"(nbytes) : "memory");
+                           "l"(v + src * Dv + unit * 8), "r"(nbytes) : "memory");
+          };
+          if (tile_lo + t < pool_tiles) {
+            const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(pooled.k);
+            const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(pooled.v);
+#pragma unroll 4
+            for (int i = 0; i < 16; ++i) {
+              const int row = row0 + 8 * i, block = (tile_lo + t) * PT_TILE + row;
+              const bool there = block < n_pool;
+              const long long src = there ? pooled.row(block, bt, block_size, max_blocks, num_blocks) * Hkv + kvh : 0;
+              copy(row, kp, vp, src, there);
+            }
+          } else {
+            const int key0 = (key_tile + tile_lo + t) * PT_TILE;
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+              const int row = row0 + 8 * i;
+              const int key = key0 + row;
+              const int page = key / block_size;
+              int blk = (key < len && page < max_blocks) ? __ldg(bt + page) : 0;
+              blk = min(max(blk, 0), num_blocks - 1);
+              copy(row, k_cache, v_cache, (static_cast<long long>(blk) * block_size + key % block_size) * Hkv + kvh, key < len);
+            }
           }
         }
       }
@@ -484,8 +543,9 @@ paged_decode_tc_kernel(const __nv_bfloat16* __restrict__ k_cache, const __nv_bfl
         tmem_ld_32x16(lane_addr + COL_S + sb * PT_N, sv);
         tmem_ld_wait();
       }
-      const int key = (tile_lo + t) * PT_TILE + r;
-      const bool valid = key < len && key >= first;
+      const bool is_pool = tile_lo + t < pool_tiles;
+      const int key = (tile_lo + t + (is_pool ? 0 : key_tile)) * PT_TILE + r;
+      const bool valid = is_pool ? key < n_pool : key < len && key >= first;
       float s[G], mx[G];
 #pragma unroll
       for (int g = 0; g < G; ++g) {
@@ -607,8 +667,8 @@ __global__ void __launch_bounds__(PD_THREADS)
 paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                   const int* __restrict__ block_table, const int* __restrict__ row_slot, const int* __restrict__ visible,
                   HeadGate gate, T* __restrict__ out, int rows, int Hq, int Hkv, int D, int Dv, long long ldq, long long ldo,
-                  int ldv, int block_size, int max_blocks, int num_blocks, float scale, KeyRange range, const float* __restrict__ slopes,
-                  const float* __restrict__ sink, float out_scale, int head_groups) {
+                  int ldv, int block_size, int max_blocks, int num_blocks, float scale, KeyRange range, PooledKeys pooled,
+                  const float* __restrict__ slopes, const float* __restrict__ sink, float out_scale, int head_groups) {
   extern __shared__ float sm[];
   const int g_all = Hq / Hkv;
   const int kvh = blockIdx.y / head_groups, h0 = (blockIdx.y % head_groups) * PR_HEADS;
@@ -634,12 +694,20 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
 #pragma unroll
     for (int h = 0; h < PR_HEADS; ++h) { m[h] = -INFINITY; l[h] = 0.f; }
     __syncthreads();
-    for (int key0 = first / 32 * 32 + warp * 32; key0 < len; key0 += PD_WARPS * 32) {
-      const int key = key0 + lane;
-      const bool valid = key < len && key >= first;
-      const int kk = key < len ? key : key0;
+    // tiles of 32 pooled blocks, then tiles of 32 keys
+    const int n_pool = pooled.count(first), pool_tiles = (n_pool + 31) / 32, tiles = pool_tiles + max(0, (len - first / 32 * 32 + 31) / 32);
+    auto key_row = [&](int kk) {
       const int blk = min(max(bt[kk / block_size], 0), num_blocks - 1);
-      const T* kr = k_cache + ((static_cast<long long>(blk) * block_size + kk % block_size) * Hkv + kvh) * D;
+      return static_cast<long long>(blk) * block_size + kk % block_size;
+    };
+    for (int tile = warp; tile < tiles; tile += PD_WARPS) {
+      const bool is_pool = tile < pool_tiles;
+      const int key0 = is_pool ? tile * 32 : (first / 32 + tile - pool_tiles) * 32, end = is_pool ? n_pool : len;
+      const int key = key0 + lane;
+      const bool valid = key < end && (is_pool || key >= first);
+      const int kk = key < end ? key : key0;
+      const T* kr = is_pool ? static_cast<const T*>(pooled.k) + (pooled.row(kk, bt, block_size, max_blocks, num_blocks) * Hkv + kvh) * D
+                            : k_cache + (key_row(kk) * Hkv + kvh) * D;
       float s[PR_HEADS];
 #pragma unroll
       for (int h = 0; h < PR_HEADS; ++h) s[h] = 0.f;
@@ -666,15 +734,14 @@ paged_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const 
         pr[h * 32 + lane] = pv;
       }
       __syncwarp();
-      const int n_keys = min(32, len - key0);
+      const int n_keys = min(32, end - key0);
       for (int d = lane; d < Dv; d += 32) {
         float acc[PR_HEADS];
 #pragma unroll
         for (int h = 0; h < PR_HEADS; ++h) acc[h] = h < g ? o[h * Dv + d] * alpha[h] : 0.f;
         for (int j = 0; j < n_keys; ++j) {
-          const int kj = key0 + j;
-          const int bj = min(max(bt[kj / block_size], 0), num_blocks - 1);
-          const float vd = to_f32(v_cache[((static_cast<long long>(bj) * block_size + kj % block_size) * Hkv + kvh) * ldv + d]);
+          const float vd = is_pool ? to_f32(static_cast<const T*>(pooled.v)[(pooled.row(key0 + j, bt, block_size, max_blocks, num_blocks) * Hkv + kvh) * Dv + d])
+                                   : to_f32(v_cache[(key_row(key0 + j) * Hkv + kvh) * ldv + d]);
 #pragma unroll
           for (int h = 0; h < PR_HEADS; ++h)
             if (h < g) acc[h] += pr[h * 32 + j] * vd;
@@ -741,6 +808,33 @@ FT_API int ft_kv_append(const void* k_new, const void* v_new, void* k_cache, voi
   return FT_E_OK;
 }
 
+// Means of whole blocks of keys and values.  Block b of a sequence holds its positions b * pool .. b * pool + pool - 1 and lies with the
+// page of its last position: k_pool [num_blocks, (block_size - 1) / pool + 1, Hkv, D], place b - page * block_size / pool (v_pool
+// likewise).  For every one of `rows` rows (positions pos of sequences slots, already in the cache) that ends a block the means
+// are formed in fp32.  bf16, or fp32 with f32; head sizes such that a token's keys and values are whole 8-element vectors.
+FT_API int ft_pool_blocks(const void* k_cache, const void* v_cache, void* k_pool, void* v_pool, const int* block_table, const int* pos,
+                          const int* slots, int rows, int Hkv, int D, int Dv, int pool, int f32, int block_size, int max_blocks, int num_blocks,
+                          int device, cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(k_cache && v_cache && k_pool && v_pool && block_table && pos && slots, "ft_pool_blocks: null pointer");
+  FT_REQUIRE(Hkv > 0 && D > 0 && Dv > 0 && (Hkv * D) % 8 == 0 && (Hkv * Dv) % 8 == 0 && pool > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0,
+             "ft_pool_blocks: %d heads of %d / %d, blocks of %d", Hkv, D, Dv, pool);
+  FT_REQUIRE(((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(k_pool) |
+               reinterpret_cast<uintptr_t>(v_pool)) & 15) == 0, "ft_pool_blocks: pointers must be 16-byte aligned");
+  if (rows <= 0) return FT_E_OK;
+  const int kw = Hkv * D, vw = Hkv * Dv, per_page = (block_size - 1) / pool + 1, cap = sm_count(device) * 16;
+  const int parts = (kw + vw + PB_THREADS * 8 - 1) / (PB_THREADS * 8);
+  const dim3 grid(rows < cap ? rows : cap, parts);
+#define FT_PB(T) \
+  pool_blocks_kernel<T><<<grid, PB_THREADS, 0, stream>>>(static_cast<const T*>(k_cache), static_cast<const T*>(v_cache), static_cast<T*>(k_pool), \
+      static_cast<T*>(v_pool), block_table, pos, slots, rows, kw, vw, pool, per_page, block_size, max_blocks, num_blocks)
+  if (f32) FT_PB(float); else FT_PB(__nv_bfloat16);
+#undef FT_PB
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
 // Scratch floats needed for n_splits > 1: B * Hq * n_splits * (Dv + 2).
 FT_API long long ft_paged_decode_scratch(int B, int Hq, int Dv, int n_splits) {
   return n_splits > 1 ? static_cast<long long>(B) * Hq * n_splits * (Dv + 2) : 0;
@@ -751,17 +845,20 @@ FT_API long long ft_paged_decode_scratch(int B, int Hq, int Dv, int n_splits) {
 // `window` are visible (0: all), or those of the row's own chunk of `chunk` positions (0: all).  slopes (fp32 [Hq] or null): a
 // head's slope times the distance of a key is taken off its score.  The result is multiplied by out_scale.  Row b reads sequence row_slot[b] of the block table (null: sequence b).  sink
 // (fp32 [Hq] or null): exp(sink) joins a head's denominator.  gate (bf16 or null): element d of head h of row b is
-// multiplied by sigmoid(gate[b * ldg + h * gate_head + d * gate_elem]); one number per head with gate_elem 0.
+// multiplied by sigmoid(gate[b * ldg + h * gate_head + d * gate_elem]); one number per head with gate_elem 0.  pool (with a window, without
+// chunk and slopes; 0: none): the row also sees k_pool and v_pool (see ft_pool_blocks) of the blocks wholly ahead of its window.
 FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                            const int* row_slot, const int* ctx_len, const void* gate, const float* sink, void* out,
                            float* scratch, int B, int Hq, int Hkv, int D, int Dv, long long ldq, long long ldg,
                            int gate_head, int gate_elem, long long ldo, int block_size, int max_blocks, int num_blocks,
-                           float scale, int window, int chunk, const float* slopes, float out_scale, int n_splits, int device,
-                           cudaStream_t stream) {
+                           float scale, int window, int chunk, const void* k_pool, const void* v_pool, int pool, const float* slopes,
+                           float out_scale, int n_splits, int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(q && k_cache && v_cache && block_table && ctx_len && out, "ft_paged_decode: null pointer");
   FT_REQUIRE(B >= 0 && Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0, "ft_paged_decode: bad shape");
   FT_REQUIRE(window >= 0 && chunk >= 0, "ft_paged_decode: negative window or chunk");
+  FT_REQUIRE(pool == 0 || (pool > 0 && window > 0 && !chunk && !slopes && k_pool && v_pool), "ft_paged_decode: blocks of %d keys", pool);
+  const PooledKeys pooled = pooled_keys(k_pool, v_pool, pool, block_size);
   const KeyRange range = {window, chunk};
   FT_REQUIRE(n_splits >= 1 && (n_splits == 1 || scratch), "ft_paged_decode: splits need scratch");
   if (B == 0) return FT_E_OK;
@@ -773,7 +870,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
   const HeadGate hg = {gate, ldg, gate_head, gate_elem};
   // equal head sizes of 64 half fill the tensor-core kernel's value tile: the CUDA-core kernel is faster there
   // (127 against 156 us at 64 rows x 2048 keys x 8 KV heads) and keeps P in fp32
-  const bool core64 = D == 64 && Dv == 64 && (G == 1 || G == 2 || G == 4 || G == 8) &&
+  const bool core64 = pool == 0 && D == 64 && Dv == 64 && (G == 1 || G == 2 || G == 4 || G == 8) &&
                       ((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) == 0;
   const bool tensor_core = !core64 && D >= 16 && D <= 128 && D % 16 == 0 && Dv >= 16 && Dv <= 128 && Dv % 16 == 0 && G <= PT_N &&
                            (reinterpret_cast<uintptr_t>(q) & 15) == 0 && ldq % 8 == 0 &&
@@ -791,7 +888,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
     kern<<<grid, PT_THREADS, PtCfg<HH>::SMEM_BYTES, stream>>>(                                                  \
         static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache),                \
         static_cast<const __nv_bfloat16*>(q), block_table, row_slot, ctx_len, static_cast<__nv_bfloat16*>(out), \
-        part_o, part_ml, Hq, Hkv, D, Dv, G, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, range, slopes, sink, hg, out_scale, status); \
+        part_o, part_ml, Hq, Hkv, D, Dv, G, ldq, ldo, block_size, max_blocks, num_blocks, sl2, n_splits, range, pooled, slopes, sink, hg, out_scale, status); \
   }
 #define FT_PT_BY_G(HH)                     \
   if (G == 1) FT_PT_LAUNCH(HH, 1)          \
@@ -803,6 +900,7 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
 #undef FT_PT_BY_G
 #undef FT_PT_LAUNCH
   } else {
+    FT_REQUIRE(pool == 0, "ft_paged_decode: blocks of keys need head sizes that are multiples of 16 up to 128, 16-byte aligned rows");
     FT_REQUIRE((D == 64 || D == 128) && D == Dv, "ft_paged_decode: head sizes %d / %d not supported (multiples of 16 up to 128, 16-byte aligned rows)", D, Dv);
 #define FT_PD_LAUNCH(DD, GG)                                                                                   \
   paged_decode_kernel<DD, GG><<<grid, PD_THREADS, 0, stream>>>(                                                \
@@ -835,17 +933,19 @@ FT_API int ft_paged_decode(const void* q, const void* k_cache, const void* v_cac
 }
 
 // Attention of arbitrary rows over the paged cache (see paged_rows_kernel): q [rows, Hq, D], out
-// [rows, Hq, Dv], row_slot / visible int32 [rows]; window, chunk, slopes, sink (always fp32) and gate as in
+// [rows, Hq, Dv], row_slot / visible int32 [rows]; window, chunk, pool, slopes, sink (always fp32) and gate as in
 // ft_paged_decode.  A cached value has Dv elements, the next head's begins ldv later (values that are the leading elements of
 // the keys: v_cache = k_cache, ldv = D).  All other tensors bf16, or fp32 with f32.
 FT_API int ft_paged_rows(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* row_slot,
                          const int* visible, const void* gate, const float* sink, void* out, int rows, int Hq, int Hkv,
                          int D, int Dv, long long ldq, long long ldg, int gate_head, int gate_elem, long long ldo,
                          int ldv, int block_size, int max_blocks, int num_blocks, float scale, int window, int chunk,
-                         const float* slopes, float out_scale, int f32, int device, cudaStream_t stream) {
+                         const void* k_pool, const void* v_pool, int pool, const float* slopes, float out_scale, int f32, int device,
+                         cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(q && k_cache && v_cache && block_table && row_slot && visible && out, "ft_paged_rows: null pointer");
   FT_REQUIRE(Hkv > 0 && Hq > 0 && Hq % Hkv == 0 && D > 0 && Dv > 0 && block_size > 0 && max_blocks > 0 && num_blocks > 0 && window >= 0 && chunk >= 0 && ldv >= Dv, "ft_paged_rows: bad shape");
+  FT_REQUIRE(pool == 0 || (pool > 0 && window > 0 && !chunk && !slopes && k_pool && v_pool), "ft_paged_rows: blocks of %d keys", pool);
   if (rows <= 0) return FT_E_OK;
   const int groups = (Hq / Hkv + PR_HEADS - 1) / PR_HEADS;
   const size_t smem = sizeof(float) * (static_cast<size_t>(PR_HEADS) * D + static_cast<size_t>(PD_WARPS) * PR_HEADS * Dv +
@@ -858,7 +958,7 @@ FT_API int ft_paged_rows(const void* q, const void* k_cache, const void* v_cache
     FT_CUDA_CHECK(cudaFuncSetAttribute(paged_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem))); \
     paged_rows_kernel<T><<<grid, PD_THREADS, smem, stream>>>(static_cast<const T*>(q), static_cast<const T*>(k_cache),       \
         static_cast<const T*>(v_cache), block_table, row_slot, visible, hg, static_cast<T*>(out), rows, Hq, Hkv, D, Dv, ldq, \
-        ldo, ldv, block_size, max_blocks, num_blocks, scale, KeyRange{window, chunk}, slopes, sink, out_scale, groups);       \
+        ldo, ldv, block_size, max_blocks, num_blocks, scale, KeyRange{window, chunk}, pooled_keys(k_pool, v_pool, pool, block_size), slopes, sink, out_scale, groups); \
   }
   if (f32) FT_PR_LAUNCH(float) else FT_PR_LAUNCH(__nv_bfloat16)
 #undef FT_PR_LAUNCH

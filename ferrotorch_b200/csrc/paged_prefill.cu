@@ -20,6 +20,8 @@
 // The epilogue adds the head's sink to the row sum, divides by it, multiplies by the output gate (per head
 // or per element) and stores bf16.  Head sizes are multiples of 16 up to 128 and may differ between keys and values: the
 // tensor maps end at the head's size, so the columns up to the tile's 64 or 128 are filled with zeros.
+// Pooled blocks ahead of a window come first: tiles of 128 means, whose rows lie anywhere in the pooled pages, four to a
+// TMA gather.
 // All waits are bounded and report through the device status word.
 #include "attn_row.cuh"
 #include "ft_host.h"
@@ -52,6 +54,7 @@ struct PpParams {
   const float* slopes;
   long long ldo;
   KeyRange range;
+  PooledKeys pooled;
   int Hkv, group, tpt, D, Dv;
   int block_size, rows_per_box, boxes, max_blocks, num_blocks;
   float scale_log2, out_scale;
@@ -59,13 +62,15 @@ struct PpParams {
 };
 
 // What an instance can do beside plain causal attention (it costs registers that the plain kernel does not have to spare):
-// PP_EXTRAS a window, chunks, sinks or a gate per element; PP_BIAS the distance bias as well.
-enum : int { PP_PLAIN = 0, PP_EXTRAS = 1, PP_BIAS = 2 };
+// PP_EXTRAS a window, chunks, sinks or a gate per element; PP_BIAS the distance bias as well; PP_POOL what PP_EXTRAS can, and
+// pooled blocks.
+enum : int { PP_PLAIN = 0, PP_EXTRAS = 1, PP_BIAS = 2, PP_POOL = 3 };
 
 template <int HD, int VD, int KIND>
 __global__ void __launch_bounds__(PP_THREADS, 1)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                     const __grid_constant__ CUtensorMap tmV, const PpParams p) {
+                     const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmKp,
+                     const __grid_constant__ CUtensorMap tmVp, const PpParams p) {
   using Cfg = PpCfg<HD, VD>;
   constexpr bool EXTRAS = KIND != PP_PLAIN;
   extern __shared__ uint8_t smem_raw[];
@@ -86,11 +91,14 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int n_tok = p.items[4 * blockIdx.x + 2], pos0 = p.items[4 * blockIdx.x + 3];
   // tokens and key blocks of each tile
   int nt[2], nb[2];
-  const int j0 = EXTRAS ? p.range.first_visible(pos0 + 1) / ATT_BN : 0;   // block 0 of this item is key block j0
+  // blocks of pooled means, which the item's last token sees, then blocks of keys: number n_pool of this item is key block j0
+  const int pool_seen = KIND == PP_POOL ? p.pooled.count(p.range.first_visible(pos0 + n_tok)) : 0;
+  const int n_pool = (pool_seen + ATT_BN - 1) / ATT_BN;
+  const int j0 = EXTRAS ? p.range.first_visible(pos0 + 1) / ATT_BN : 0;
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     nt[i] = min(max(n_tok - i * p.tpt, 0), p.tpt);
-    nb[i] = nt[i] > 0 ? (pos0 + i * p.tpt + nt[i] + ATT_BN - 1) / ATT_BN - j0 : 0;
+    nb[i] = nt[i] > 0 ? (pos0 + i * p.tpt + nt[i] + ATT_BN - 1) / ATT_BN - j0 + n_pool : 0;
   }
   const int n_blocks = max(nb[0], nb[1]);
 
@@ -110,6 +118,10 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmV);
+    if (KIND == PP_POOL) {
+      tma_prefetch_desc(&tmKp);
+      tma_prefetch_desc(&tmVp);
+    }
   }
   if (warp == 2) {
     tmem_alloc(smem_u32(tmem_slot), Cfg::TMEM_COLS);
@@ -138,22 +150,37 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const int* bt = p.block_table + static_cast<long long>(slot) * p.max_blocks;
       // box `lane` of key block j: rows_per_box keys of one page, as a row of the [num_blocks * block_size] axis
       auto page_row = [&](int j) {
-        const int key = (j0 + j) * ATT_BN + lane * p.rows_per_box;
+        const int key = (j0 + j - n_pool) * ATT_BN + lane * p.rows_per_box;
         const int page = min(key / p.block_size, p.max_blocks - 1);
         const int blk = min(max(lane < p.boxes ? __ldg(bt + page) : 0, 0), p.num_blocks - 1);
         return blk * p.block_size + key % p.block_size;
       };
-      int row = page_row(0);
+      // pooled block 4 * lane + i of tile j, as a row of the [num_blocks * per_page * Hkv] axis; past the last one: that one again
+      auto pool_row = [&](int j, int i) {
+        const int b = min(j * ATT_BN + lane * 4 + i, pool_seen - 1);
+        return static_cast<int>(p.pooled.row(b, bt, p.block_size, p.max_blocks, p.num_blocks)) * p.Hkv + kvh;
+      };
+      int row = n_pool > 0 ? 0 : page_row(0);
       bool ok = true;
       for (int j = 0; j < n_blocks; ++j) {
         const int st = j & 1;
         const uint32_t par = ((j >> 1) & 1) ^ 1u;
-        const int next_row = j + 1 < n_blocks ? page_row(j + 1) : 0;
+        const int next_row = j + 1 < n_blocks && j + 1 >= n_pool ? page_row(j + 1) : 0;
+        const bool is_pool = KIND == PP_POOL && j < n_pool;
+        int pr[4];
+        if (is_pool) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) pr[i] = pool_row(j, i);
+        }
         ok = mbar_wait(bar(K_EMPTY + st), par, abort_word, FT_ERR_TIMEOUT_PRODUCER);
         if (!__all_sync(0xffffffffu, ok)) break;
         if (lane == 0) mbar_expect_tx(bar(K_FULL + st), Cfg::K_BYTES);
         __syncwarp();
-        if (lane < p.boxes) {
+        if (is_pool) {
+#pragma unroll
+          for (int c = 0; c < HD / 64; ++c)
+            tma_gather4_2d(sK + st * Cfg::K_BYTES + c * (ATT_BN * 128) + lane * 512, &tmKp, bar(K_FULL + st), c * 64, pr[0], pr[1], pr[2], pr[3]);
+        } else if (lane < p.boxes) {
 #pragma unroll
           for (int c = 0; c < HD / 64; ++c)
             tma_load_3d(sK + st * Cfg::K_BYTES + c * (ATT_BN * 128) + lane * p.rows_per_box * 128, &tmK, bar(K_FULL + st),
@@ -163,7 +190,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (!__all_sync(0xffffffffu, ok)) break;
         if (lane == 0) mbar_expect_tx(bar(V_FULL + st), Cfg::V_BYTES);
         __syncwarp();
-        if (lane < p.boxes) {
+        if (is_pool) {
+#pragma unroll
+          for (int c = 0; c < VD / 64; ++c)
+            tma_gather4_2d(sV + st * Cfg::V_BYTES + c * (ATT_BN * 128) + lane * 512, &tmVp, bar(V_FULL + st), c * 64, pr[0], pr[1], pr[2], pr[3]);
+        } else if (lane < p.boxes) {
 #pragma unroll
           for (int c = 0; c < VD / 64; ++c)
             tma_load_3d(sV + st * Cfg::V_BYTES + c * (ATT_BN * 128) + lane * p.rows_per_box * 128, &tmV, bar(V_FULL + st),
@@ -264,6 +295,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const int tile_pos = pos0 + ti * p.tpt;
     const int limit = tile_pos + tok;                              // last visible key
     const int warp_limit = tile_pos + (ew * 32) / p.group;         // of this warp's first row
+    const int pool_limit = KIND == PP_POOL ? p.pooled.count(p.range.first_visible(limit + 1)) - 1 : 0;       // last visible pooled block
+    const int warp_pool_limit = KIND == PP_POOL ? p.pooled.count(p.range.first_visible(warp_limit + 1)) - 1 : 0;
     float slope = 0.f;                                             // in powers of two per position
     if constexpr (KIND == PP_BIAS)
       if (p.slopes) slope = p.slopes[min(kvh * p.group + head, p.Hkv * p.group - 1)] * ATT_LOG2E;
@@ -273,7 +306,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       tc_fence_after();
       f32x2 sp[ATT_BN / 2];
       att2_load_row(s_addr, sp);
-      const int kv0 = (j0 + j) * ATT_BN;
+      const bool is_pool = KIND == PP_POOL && j < n_pool;
+      const int kv0 = is_pool ? j * ATT_BN : (j0 + j - n_pool) * ATT_BN;
       if constexpr (KIND == PP_BIAS) {                             // score * scale - slope * (limit - key)
         const f32x2 sc = f2_pack(p.scale_log2, p.scale_log2), two = f2_pack(2.f * slope, 2.f * slope);
         const float b0 = slope * static_cast<float>(kv0 - limit);
@@ -283,9 +317,10 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
           sp[i] = f2_fma(sp[i], sc, f2_fma(two, f2_pack(static_cast<float>(i), static_cast<float>(i)), bias));
         }
       }
-      if (kv0 + ATT_BN - 1 > warp_limit) att2_mask_row(sp, kv0, limit);   // warp-uniform branches
+      const int last_seen = is_pool ? pool_limit : limit;
+      if (kv0 + ATT_BN - 1 > (is_pool ? warp_pool_limit : warp_limit)) att2_mask_row(sp, kv0, last_seen);   // warp-uniform branches
       // no row of the warp is more than 31 positions past its first; a row may see nothing of its first blocks
-      if (EXTRAS && kv0 < p.range.first_visible(warp_limit + 32)) att2_mask_ahead(sp, kv0, p.range.first_visible(limit + 1));
+      if (EXTRAS && !is_pool && kv0 < p.range.first_visible(warp_limit + 32)) att2_mask_ahead(sp, kv0, p.range.first_visible(limit + 1));
       const float mx = att2_row_max(sp) * row_scale;     // scale > 0, so the maximum commutes with it
       float alpha = 1.f;
       if (mx > m_ref + ATT2_RESCALE_THRESHOLD) {
@@ -378,8 +413,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
 }
 
 template <int HD, int VD, int KIND>
-static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PpParams& p,
-                                int n_items, int device, cudaStream_t stream) {
+static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tkp, const CUtensorMap& tvp,
+                                const PpParams& p, int n_items, int device, cudaStream_t stream) {
   using Cfg = PpCfg<HD, VD>;
   auto kern = paged_prefill_kernel<HD, VD, KIND>;
   static bool attr_set[64] = {false};
@@ -387,19 +422,20 @@ static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CU
     FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));
     attr_set[device] = true;
   }
-  kern<<<dim3(n_items, p.Hkv), PP_THREADS, Cfg::SMEM_BYTES, stream>>>(tq, tk, tv, p);
+  kern<<<dim3(n_items, p.Hkv), PP_THREADS, Cfg::SMEM_BYTES, stream>>>(tq, tk, tv, tkp, tvp, p);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;
 }
 
 template <int HD, int VD>
-static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const PpParams& p,
-                                int n_items, int device, cudaStream_t stream) {
-  if (p.slopes) return launch_prefill<HD, VD, PP_BIAS>(tq, tk, tv, p, n_items, device, stream);
+static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tkp, const CUtensorMap& tvp,
+                                const PpParams& p, int n_items, int device, cudaStream_t stream) {
+  if (p.pooled.pool > 0) return launch_prefill<HD, VD, PP_POOL>(tq, tk, tv, tkp, tvp, p, n_items, device, stream);
+  if (p.slopes) return launch_prefill<HD, VD, PP_BIAS>(tq, tk, tv, tkp, tvp, p, n_items, device, stream);
   const bool extras = p.range.window > 0 || p.range.chunk > 0 || p.sink || (p.gate.g && p.gate.elem != 0);
-  return extras ? launch_prefill<HD, VD, PP_EXTRAS>(tq, tk, tv, p, n_items, device, stream)
-                : launch_prefill<HD, VD, PP_PLAIN>(tq, tk, tv, p, n_items, device, stream);
+  return extras ? launch_prefill<HD, VD, PP_EXTRAS>(tq, tk, tv, tkp, tvp, p, n_items, device, stream)
+                : launch_prefill<HD, VD, PP_PLAIN>(tq, tk, tv, tkp, tvp, p, n_items, device, stream);
 }
 
 }  // namespace ft
@@ -408,7 +444,7 @@ static int launch_paged_prefill(const CUtensorMap& tq, const CUtensorMap& tk, co
 FT_API int ft_paged_prefill_tile(int group) { return group > 0 && group <= ft::ATT_BM ? ft::ATT_BM / group : 0; }
 
 // Attention of prompt portions (see the top of this file).  q: [rows, Hq, D] (row stride ldq), out: [rows,
-// Hq, Dv] (row stride ldo); window, chunk, slopes, sink, gate and out_scale as in ft_paged_decode (a gate per element has unit element stride
+// Hq, Dv] (row stride ldo); window, chunk, pool, slopes, sink, gate and out_scale as in ft_paged_decode (a gate per element has unit element stride
 // and 16-byte aligned heads).  items: int32 [n_items, 4] on the
 // device: slot, first query row, number of tokens (<= 2 * ft_paged_prefill_tile), position of the first token;
 // keys 0 .. position of a token must be in the cache.  Page sizes: a divisor of 128 of at least 8, or a
@@ -416,8 +452,8 @@ FT_API int ft_paged_prefill_tile(int group) { return group > 0 && group <= ft::A
 FT_API int ft_paged_prefill(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* items,
                             const void* gate, const float* sink, void* out, int n_items, int rows, int Hq, int Hkv, int D,
                             int Dv, long long ldq, long long ldg, int gate_head, int gate_elem, long long ldo, int block_size,
-                            int max_blocks, int num_blocks, float scale, int window, int chunk, const float* slopes, float out_scale, int device,
-                            cudaStream_t stream) {
+                            int max_blocks, int num_blocks, float scale, int window, int chunk, const void* k_pool, const void* v_pool, int pool,
+                            const float* slopes, float out_scale, int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   using namespace ft;
   FT_REQUIRE(q && k_cache && v_cache && block_table && items && out, "ft_paged_prefill: null pointer");
@@ -433,10 +469,12 @@ FT_API int ft_paged_prefill(const void* q, const void* k_cache, const void* v_ca
   FT_REQUIRE(window >= 0 && chunk >= 0 && (!gate || gate_elem == 0 || (gate_elem == 1 && gate_head % 8 == 0 && ldg % 8 == 0 &&
                                                          (reinterpret_cast<uintptr_t>(gate) & 15) == 0)),
              "ft_paged_prefill: the window is negative or the gate's elements are not packed and aligned");
+  FT_REQUIRE(pool == 0 || (pool > 0 && window > 0 && !chunk && !slopes && k_pool && v_pool &&
+                           ((reinterpret_cast<uintptr_t>(k_pool) | reinterpret_cast<uintptr_t>(v_pool)) & 15) == 0), "ft_paged_prefill: blocks of %d keys", pool);
   if (n_items <= 0) return FT_E_OK;
   PpParams p;
   p.items = items; p.block_table = block_table; p.gate = HeadGate{gate, ldg, gate_head, gate_elem};
-  p.sink = sink; p.slopes = slopes; p.range = KeyRange{window, chunk}; p.out_scale = out_scale;
+  p.sink = sink; p.slopes = slopes; p.range = KeyRange{window, chunk}; p.pooled = pooled_keys(k_pool, v_pool, pool, block_size); p.out_scale = out_scale;
   p.out = static_cast<__nv_bfloat16*>(out); p.ldo = ldo;
   p.Hkv = Hkv; p.group = Hq / Hkv; p.tpt = ATT_BM / p.group; p.D = D; p.Dv = Dv;
   p.block_size = block_size;
@@ -455,9 +493,16 @@ FT_API int ft_paged_prefill(const void* q, const void* k_cache, const void* v_ca
   rc = make_tmap_3d(&tv, v_cache, 2, Dv, Hkv, n_rows, static_cast<uint64_t>(Dv) * 2, static_cast<uint64_t>(Hkv) * Dv * 2, 64, 1,
                     p.rows_per_box, 3);
   if (rc) return rc;
+  CUtensorMap tkp = tk, tvp = tv;
+  if (pool > 0) {
+    const uint64_t pool_rows = static_cast<uint64_t>(num_blocks) * p.pooled.per_page * Hkv;
+    FT_REQUIRE(pool_rows < (1ull << 31), "ft_paged_prefill: the cache is too large");
+    if (int rc2 = make_tmap_2d(&tkp, k_pool, 2, D, pool_rows, static_cast<uint64_t>(D) * 2, 64, 1, 3)) return rc2;
+    if (int rc2 = make_tmap_2d(&tvp, v_pool, 2, Dv, pool_rows, static_cast<uint64_t>(Dv) * 2, 64, 1, 3)) return rc2;
+  }
   if (D > 64)
-    return Dv > 64 ? launch_paged_prefill<128, 128>(tq, tk, tv, p, n_items, device, stream)
-                   : launch_paged_prefill<128, 64>(tq, tk, tv, p, n_items, device, stream);
-  return Dv > 64 ? launch_paged_prefill<64, 128>(tq, tk, tv, p, n_items, device, stream)
-                 : launch_paged_prefill<64, 64>(tq, tk, tv, p, n_items, device, stream);
+    return Dv > 64 ? launch_paged_prefill<128, 128>(tq, tk, tv, tkp, tvp, p, n_items, device, stream)
+                   : launch_paged_prefill<128, 64>(tq, tk, tv, tkp, tvp, p, n_items, device, stream);
+  return Dv > 64 ? launch_paged_prefill<64, 128>(tq, tk, tv, tkp, tvp, p, n_items, device, stream)
+                 : launch_paged_prefill<64, 64>(tq, tk, tv, tkp, tvp, p, n_items, device, stream);
 }

@@ -1,7 +1,9 @@
 // Recurrent decoder blocks: short causal convolutions with carried inputs, and linear recurrences over prompt portions.
 //
-//   ft_causal_conv   per channel, over the rows of a ragged batch; the inputs ahead of a portion come from the
-//                    sequence's slot, the rows that are a sequence's only token store their own inputs there
+//   ft_causal_conv   per channel, over the rows of a ragged batch, with or without a silu of the result; the inputs ahead of
+//                    a portion come from the sequence's slot, the rows that are a sequence's only token store their own
+//                    inputs there
+//   ft_conv_tail     the last inputs of portions into the slots, where no scan follows that does it
 //   ft_rglru_scan    S_t = a_t S_(t-1) + x_t over the rows of every portion, out = S * gelu(y); the final state and
 //                    the convolution's last inputs go to the slot
 //
@@ -26,8 +28,16 @@ struct ConvParams {
   const int* slots;
   const int* starts;        // position of the first row of the row's portion
   long long ldx, ldu;
-  int rows, n_single, C, taps, walk;
+  int rows, n_single, C, taps, walk, silu;
 };
+
+// The result of a channel: the sum itself or its silu (in the form of the type, see recurrent.cuh).
+template <typename T>
+__device__ __forceinline__ void conv_finish(const ConvParams& p, float (&v)[8]) {
+  if (!p.silu) return;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] *= sigmoid_row(v[e], static_cast<const T*>(nullptr));
+}
 
 // The input d rows ahead of a row (d <= taps - 1): of the same portion, of the slot, or zero ahead of the sequence.
 template <typename T>
@@ -83,6 +93,7 @@ short_conv_kernel(const ConvParams p) {
         for (int d = TAPS - 1; d >= 0; --d)
 #pragma unroll
           for (int e = 0; e < 8; ++e) acc[e] += w[d][e] * in[d][e];
+        conv_finish<T>(p, acc);
         store8(static_cast<T*>(p.u) + static_cast<long long>(row) * p.ldu + c, acc);
         if (TAPS > 1 && single) {              // this thread is the only one at these inputs
 #pragma unroll
@@ -120,6 +131,7 @@ causal_conv_kernel(const ConvParams p) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[e] += w[e] * v[e];
       }
+      conv_finish<T>(p, acc);
       store8(static_cast<T*>(p.u) + static_cast<long long>(row) * p.ldu + c, acc);
       if (row < p.n_single) {                                       // this thread is the only one at these inputs
         float v[8];
@@ -133,6 +145,25 @@ causal_conv_kernel(const ConvParams p) {
         }
       }
     }
+}
+
+// The last `keep` inputs of every portion into its slot: from the portion, or what the slot held (moved down; m + n > m is still
+// old).  A thread owns eight channels.
+template <typename T>
+__global__ void __launch_bounds__(CV_THREADS)
+conv_tail_kernel(const T* __restrict__ x, long long ldx, T* state, const int* __restrict__ spans, int C, int keep) {
+  const int c = (blockIdx.x * CV_THREADS + threadIdx.x) * 8;
+  if (c >= C) return;
+  const int* span = spans + 4 * blockIdx.y;
+  const int slot = span[0], row0 = span[1], n = span[3];
+  T* st = state + static_cast<long long>(slot) * keep * C + c;
+  for (int m = 0; m < keep; ++m) {
+    const int o = n - keep + m;
+    float v[8];
+    if (o >= 0) load8(x + static_cast<long long>(row0 + o) * ldx + c, v);
+    else load8(static_cast<const T*>(st) + static_cast<long long>(m + n) * C, v);
+    store8(st + static_cast<long long>(m) * C, v);
+  }
 }
 
 // ---------------------------------------------------------------- scan
@@ -237,9 +268,9 @@ static bool rc_aligned(std::initializer_list<const void*> ps) {
 using namespace ft;
 
 // u = causal convolution of x over the rows of a ragged batch (see ConvParams).  x, state and u are bf16, or fp32
-// with f32; w [taps, C] and bias [C] fp32; C a multiple of 8.
+// with f32; w [taps, C] and bias [C] fp32; C a multiple of 8.  silu: of the result.
 FT_API int ft_causal_conv(const void* x, long long ldx, const float* w, const float* bias, void* state, void* u, long long ldu,
-                          const int* pos, const int* slots, const int* starts, int rows, int n_single, int C, int taps, int f32,
+                          const int* pos, const int* slots, const int* starts, int rows, int n_single, int C, int taps, int silu, int f32,
                           int device, cudaStream_t stream) {
   if (int _rc = ft::ensure_device(device)) return _rc;
   FT_REQUIRE(x && w && bias && u && pos && slots && starts && (state || taps == 1), "ft_causal_conv: null pointer");
@@ -248,7 +279,7 @@ FT_API int ft_causal_conv(const void* x, long long ldx, const float* w, const fl
   if (rows <= 0) return FT_E_OK;
   ConvParams p;
   p.x = x; p.w = w; p.bias = bias; p.state = state; p.u = u; p.pos = pos; p.slots = slots; p.starts = starts;
-  p.ldx = ldx; p.ldu = ldu; p.rows = rows; p.n_single = n_single; p.C = C; p.taps = taps;
+  p.ldx = ldx; p.ldu = ldu; p.rows = rows; p.n_single = n_single; p.C = C; p.taps = taps; p.silu = silu;
   const int gx = (C / 8 + CV_THREADS - 1) / CV_THREADS;
   p.walk = rows / (sm_count(device) * 8 / gx + 1);         // enough blocks for the GPU, then longer walks
   p.walk = p.walk < 1 ? 1 : (p.walk > CV_ROWS ? CV_ROWS : p.walk);
@@ -264,6 +295,22 @@ FT_API int ft_causal_conv(const void* x, long long ldx, const float* w, const fl
   }
   if (f32) { FT_CONV(float) } else { FT_CONV(__nv_bfloat16) }
 #undef FT_CONV
+  FT_CUDA_CHECK(cudaGetLastError());
+  count_launch();
+  return FT_E_OK;
+}
+
+// The last `keep` rows of x [rows, ldx] of every portion (spans int32 [n_spans, 4]: slot, first row, first position, rows) into state
+// [slots, keep, C].  bf16, or fp32 with f32; C a multiple of 8.
+FT_API int ft_conv_tail(const void* x, long long ldx, void* state, const int* spans, int n_spans, int C, int keep, int f32, int device,
+                        cudaStream_t stream) {
+  if (int _rc = ft::ensure_device(device)) return _rc;
+  FT_REQUIRE(x && state && spans, "ft_conv_tail: null pointer");
+  FT_REQUIRE(C > 0 && C % 8 == 0 && keep > 0 && ldx >= C && ldx % 8 == 0 && n_spans < 65536 && rc_aligned({x, state}), "ft_conv_tail: %d channels", C);
+  if (n_spans <= 0) return FT_E_OK;
+  const dim3 grid((C / 8 + CV_THREADS - 1) / CV_THREADS, n_spans);
+  if (f32) conv_tail_kernel<float><<<grid, CV_THREADS, 0, stream>>>(static_cast<const float*>(x), ldx, static_cast<float*>(state), spans, C, keep);
+  else conv_tail_kernel<__nv_bfloat16><<<grid, CV_THREADS, 0, stream>>>(static_cast<const __nv_bfloat16*>(x), ldx, static_cast<__nv_bfloat16*>(state), spans, C, keep);
   FT_CUDA_CHECK(cudaGetLastError());
   count_launch();
   return FT_E_OK;

@@ -70,3 +70,4 @@ register_causal_lm(CausalLMFamily("llama", _is_llama, "ferrotorch_b200.models.ll
 register_causal_lm(CausalLMFamily("bopudra", lambda c: c.get("architecture") == "Bopudra", "ferrotorch_b200.models.bopudra:BopudraForCausalLM"))
 register_causal_lm(CausalLMFamily("zolorax", lambda c: c.get("architecture") == "Zolorax", "ferrotorch_b200.models.zolorax:ZoloraxForCausalLM"))
 register_causal_lm(CausalLMFamily("tenalorn", lambda c: c.get("architecture") == "Tenalorn", "ferrotorch_b200.models.tenalorn:TenalornForCausalLM"))
+register_causal_lm(CausalLMFamily("mogelix", lambda c: c.get("architecture") == "Mogelix", "ferrotorch_b200.models.mogelix:MogelixForCausalLM"))

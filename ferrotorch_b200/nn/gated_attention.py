@@ -1,5 +1,5 @@
-"""Parts of pre-norm decoders over a paged cache: RMS norm of the fp32 residual stream, and attention with per-head query /
-key norm, rotation, window, sink and an output gate per element, whose keys and values may be another layer's.
+"""Parts of decoders over a paged cache: RMS norm of the fp32 residual stream, and attention with per-head query / key norm,
+rotation, window, pooled blocks ahead of it, sink and an output gate per element, whose keys and values may be another layer's.
 
 Sizes are padded at load time with zero weights like those of :mod:`~ferrotorch_b200.nn.packed_block`."""
 from __future__ import annotations
@@ -48,15 +48,22 @@ class ResidualRMSNorm(nn.Module):
 
 
 class GatedAttention(nn.Module):
-    """``x += W_o (attention(h) * sigmoid(W_g h))`` over a paged cache.
+    """``W_o (attention(h) * sigmoid(W_g h))`` over a paged cache: added to the residual (:meth:`forward`) or left to the kernel that
+    does (:meth:`terms`).
 
-    One packed product ``[q | k | v | g]`` (``[q | g]`` when the keys are another layer's), one pass for norms, rotation and
-    cache, the attention with sink, window and gate, and the output product onto the residual.  ``qk_norm``: RMS norm per
-    head, weights shared by the heads; ``sink``: one learned number per head in the denominator; ``gate``: per element."""
+    One packed product ``[q | k | v | g | r]`` (``[q | g | r]`` when the keys are another layer's), one pass for norms, rotation and
+    cache, the attention with sink, window, pooled blocks and gate, and the output product.  ``qk_norm``: RMS norm per head, by
+    ``norm_weights`` with weights shared by the heads (a norm without weights and a rotation may change places); ``bias``: of queries,
+    keys and values; ``sink``: one learned number per head in the denominator; ``gate``: per element; ``residual_gate``: pre-activations
+    of a gate of the whole sublayer, ``rg`` with its bias ``rg.b``, ride along in the packed product."""
 
-    def __init__(self, hidden_size: int, attn: AttentionSpec, eps: float, qk_norm: bool = True, sink: bool = True, gate: bool = True):
+    def __init__(self, hidden_size: int, attn: AttentionSpec, eps: float, qk_norm: bool = True, sink: bool = True, gate: bool = True,
+                 norm_weights: bool = True, bias: bool = False, residual_gate: bool = False):
         super().__init__()
+        if attn.chunk is not None or attn.distance_bias or (attn.rotary is not None and attn.rotary.interleaved):
+            raise ValueError("GatedAttention: no chunks, distance bias or rotation of neighbours")
         self.attn, self.eps, self.hidden_size, self.qk_norm, self.gated = attn, eps, hidden_size, qk_norm, gate
+        self.norm_weights, self.bias, self.residual_gate = qk_norm and norm_weights, bias, residual_gate
         a, width = attn, round_up(hidden_size, 8)
         own = a.kv_from is None
         self.value_width = a.heads * a.padded_vdim
@@ -66,21 +73,37 @@ class GatedAttention(nn.Module):
         for n in sizes:
             self.segments.append((at, n))
             at += n
+        self.gate_at = at
+        at += width if residual_gate else 0
         self.register_buffer("in_proj", torch.zeros(at, width))
+        self.register_buffer("in_bias", torch.zeros(at) if bias or residual_gate else None)
         self.register_buffer("out_proj", torch.zeros(width, self.value_width))
-        self.register_buffer("q_norm", torch.zeros(a.padded_dim) if qk_norm else None)
-        self.register_buffer("k_norm", torch.zeros(a.padded_dim) if qk_norm and own else None)
+        ones = torch.ones(a.padded_dim)
+        self.register_buffer("q_norm", (torch.zeros(a.padded_dim) if self.norm_weights else ones) if qk_norm else None)
+        self.register_buffer("k_norm", (torch.zeros(a.padded_dim) if self.norm_weights else ones.clone()) if qk_norm and own else None)
         self.register_buffer("sink", torch.zeros(a.heads) if sink else None)
+
+    def _parts(self) -> list:
+        """``(name, first row of the packed product, heads, head size, padded head size, biased)`` of what it holds."""
+        a, at = self.attn, [off for off, _ in self.segments]
+        out = [("q", at[0], a.heads, a.dim, a.padded_dim, self.bias)]
+        if a.kv_from is None:
+            out += [("k", at[1], a.kv_heads, a.dim, a.padded_dim, self.bias), ("v", at[2], a.kv_heads, a.vdim, a.padded_vdim, self.bias)]
+        if self.gated:
+            out.append(("g", at[3], a.heads, a.vdim, a.padded_vdim, False))
+        if self.residual_gate:
+            out.append(("rg", self.gate_at, 1, self.hidden_size, self.in_proj.shape[1], True))
+        return out
 
     def _shapes(self) -> dict:
         """True shapes of the weights by name."""
         a, W = self.attn, self.hidden_size
-        out = {"q": (a.heads * a.dim, W), "o": (W, a.heads * a.vdim)}
-        if a.kv_from is None:
-            out.update(k=(a.kv_heads * a.dim, W), v=(a.kv_heads * a.vdim, W))
-        if self.gated:
-            out["g"] = (a.heads * a.vdim, W)
-        if self.qk_norm:
+        out = {"o": (W, a.heads * a.vdim)}
+        for name, _, heads, d, _, biased in self._parts():
+            out[name] = (heads * d, W)
+            if biased:
+                out[name + ".b"] = (heads * d,)
+        if self.norm_weights:
             out["q.norm"] = (a.dim,)
             if a.kv_from is None:
                 out["k.norm"] = (a.dim,)
@@ -97,26 +120,29 @@ class GatedAttention(nn.Module):
         for name, shape in self._shapes().items():
             checked("GatedAttention", name, sd.get(name), shape)
         width = self.in_proj.shape[1]
-        for (off, n), name, heads, d in zip(self.segments, ("q", "k", "v", "g"), (a.heads, a.kv_heads, a.kv_heads, a.heads),
-                                            (a.padded_dim, a.padded_dim, a.padded_vdim, a.padded_vdim)):
-            if n:
-                self.in_proj[off:off + n].copy_(pad_to(pad_heads(sd[name], heads, d), n, width))
+        for name, at, heads, _, padded, biased in self._parts():
+            n = heads * padded
+            self.in_proj[at:at + n].copy_(pad_to(pad_heads(sd[name], heads, padded), n, width))
+            if biased:
+                self.in_bias[at:at + n].copy_(pad_heads(sd[name + ".b"].float(), heads, padded))
         self.out_proj.copy_(pad_to(pad_heads(sd["o"].t(), a.heads, a.padded_vdim).t(), width, self.value_width))
-        for buf, name in ((self.q_norm, "q.norm"), (self.k_norm, "k.norm")):
-            if buf is not None:
-                buf.copy_(pad_to(sd[name].float(), a.padded_dim))
+        if self.norm_weights:
+            for buf, name in ((self.q_norm, "q.norm"), (self.k_norm, "k.norm")):
+                if buf is not None:
+                    buf.copy_(pad_to(sd[name].float(), a.padded_dim))
         if self.sink is not None:
             self.sink.copy_(sd["sink"].float())
 
     def unpack(self) -> dict:
         a, W = self.attn, self.hidden_size
         out = {}
-        for (off, n), name, heads, d in zip(self.segments, ("q", "k", "v", "g"), (a.heads, a.kv_heads, a.kv_heads, a.heads),
-                                            (a.dim, a.dim, a.vdim, a.vdim)):
-            if n:
-                out[name] = unpad_heads(self.in_proj[off:off + n, :W], heads, d)
+        for name, at, heads, d, padded, biased in self._parts():
+            out[name] = unpad_heads(self.in_proj[at:at + heads * padded, :W], heads, d)
+            if biased:
+                out[name + ".b"] = unpad_heads(self.in_bias[at:at + heads * padded], heads, d)
         out["o"] = unpad_heads(self.out_proj[:W].t(), a.heads, a.vdim).t()
-        for buf, name, n in ((self.q_norm, "q.norm", a.dim), (self.k_norm, "k.norm", a.dim), (self.sink, "sink", a.heads)):
+        for buf, name, n in ((self.q_norm if self.norm_weights else None, "q.norm", a.dim), (self.k_norm if self.norm_weights else None, "k.norm", a.dim),
+                             (self.sink, "sink", a.heads)):
             if buf is not None:
                 out[name] = buf[:n]
         return out
@@ -127,21 +153,31 @@ class GatedAttention(nn.Module):
                    for n, s in self._shapes().items()})
 
     def cast_(self, dtype: torch.dtype) -> None:
-        """The matrices in ``dtype``; norm weights and sinks stay fp32."""
+        """The matrices in ``dtype``; biases, norm weights and sinks stay fp32."""
         self.in_proj, self.out_proj = self.in_proj.to(dtype), self.out_proj.to(dtype)
 
-    def forward(self, x: torch.Tensor, h: torch.Tensor, batch, cache, layer: int) -> None:
-        """Adds the sublayer of input ``h`` to the fp32 residual ``x``; ``layer``: its (or its source's) place in the cache."""
+    def attend(self, h: torch.Tensor, batch, cache, layer: int) -> tuple:
+        """The heads' results ``[T, heads * padded_vdim]`` for input ``h`` and the packed product; ``layer``: the (or its source's)
+        place in the cache."""
         a = self.attn
-        if a.chunk is not None or a.distance_bias or (a.rotary is not None and a.rotary.interleaved):
-            raise ValueError("GatedAttention: no chunks, distance bias or rotation of neighbours")
         (qo, qn), (ko, _), (vo, _), (go, gn) = self.segments
-        packed = F.linear_rows(h, self.in_proj)
+        packed = F.linear_rows(h, self.in_proj, self.in_bias)
         D.qkv_head_finish(packed, cache, layer, batch, heads=a.heads, dim=a.padded_dim, q_off=qo, k_off=ko, v_off=vo,
                           own_keys=a.kv_from is None, q_weight=self.q_norm, k_weight=self.k_norm, true_dim=a.dim, eps=self.eps,
                           table=cache.rotary_table(a.rotary) if a.rotary is not None else None)
+        if a.kv_from is None:
+            cache.pool_blocks(layer, batch)
         heads = torch.empty((h.shape[0], a.heads, a.padded_vdim), device=h.device, dtype=h.dtype)
         gate = packed[:, go:go + gn].unflatten(1, (a.heads, a.padded_vdim)) if self.gated else None
         cache.attend(layer, packed[:, qo:qo + qn].unflatten(1, (a.heads, a.padded_dim)), batch, a.scale, gate=gate, out=heads,
-                     window=a.window, sink=self.sink)
-        F.residual_linear_(x, heads.flatten(1), self.out_proj)
+                     window=a.window, sink=self.sink, pool=a.pool)
+        return heads.flatten(1), packed
+
+    def forward(self, x: torch.Tensor, h: torch.Tensor, batch, cache, layer: int) -> None:
+        """Adds the sublayer of input ``h`` to the fp32 residual ``x``."""
+        F.residual_linear_(x, self.attend(h, batch, cache, layer)[0], self.out_proj)
+
+    def terms(self, h: torch.Tensor, batch, cache, layer: int) -> tuple:
+        """The sublayer's output and the pre-activations of its residual gate (a view; ``None`` without one)."""
+        heads, packed = self.attend(h, batch, cache, layer)
+        return D.SublayerTerms(dense=F.linear_rows(heads, self.out_proj)), packed[:, self.gate_at:] if self.residual_gate else None

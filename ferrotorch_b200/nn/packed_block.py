@@ -49,19 +49,32 @@ class YarnScaling:
 
 
 @dataclass(frozen=True)
+class WavelengthScaling:
+    """Interpolation by wavelength for contexts ``factor`` times as long as ``original`` (Llama 3.1): dimensions that turn more than
+    ``high`` times over it keep their frequency, less than ``low`` times have it divided, a linear transition between."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotation of the first ``dims`` elements of a head, frequencies ``base ** (-2 i / dims)``; pairs ``(i, i + dims / 2)``, or
     neighbours ``(2 i, 2 i + 1)`` when ``interleaved``."""
     dims: int
     base: float
-    scaling: YarnScaling | None = None
+    scaling: YarnScaling | WavelengthScaling | None = None
     interleaved: bool = False
 
     def table(self, positions: int, device="cpu") -> torch.Tensor:
         """cos and sin of every position, ``[positions, dims / 2, 2]`` fp32 (angles are computed in 64-bit)."""
         sc = self.scaling
-        kind = None if sc is None else {"type": "yarn", "factor": sc.factor, "original_max": sc.original, "beta_fast": sc.fast,
-                                        "beta_slow": sc.slow, "full_range": True, "mscale": "always"}
+        if isinstance(sc, WavelengthScaling):
+            kind = {"type": "llama3", "factor": sc.factor, "original_max": sc.original, "low_freq_factor": sc.low, "high_freq_factor": sc.high}
+        else:
+            kind = None if sc is None else {"type": "yarn", "factor": sc.factor, "original_max": sc.original, "beta_fast": sc.fast,
+                                            "beta_slow": sc.slow, "full_range": True, "mscale": "always"}
         return torch.stack(ref.rope_tables(self.dims, positions, self.base, kind), -1).contiguous().to(device)
 
 
@@ -77,7 +90,8 @@ class AttentionSpec:
     its last so many positions, its own included (``None``: all); ``chunk``: it sees those of its own chunk of so many positions,
     chunks counted from position 0 (``None``: all); ``distance_bias``: the distance of a key times the head's slope (:func:`head_slopes`)
     is taken off its score; ``rotary``: rotation of queries and keys; ``kv_from``: the layer whose keys and values this one reads
-    instead of having its own."""
+    instead of having its own; ``pool``: beside its window a query sees one key and value, their means, for each block of so many
+    positions (counted from 0) that lies wholly ahead of the window (``None``: nothing ahead of it)."""
     heads: int
     kv_heads: int
     dim: int
@@ -90,6 +104,7 @@ class AttentionSpec:
     kv_from: int | None = None
     chunk: int | None = None
     distance_bias: bool = False
+    pool: int | None = None
 
     def validate(self) -> None:
         if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
@@ -100,6 +115,8 @@ class AttentionSpec:
             raise ValueError("AttentionSpec: window must be positive or absent")
         if self.chunk is not None and self.chunk < 1:
             raise ValueError("AttentionSpec: chunk must be positive or absent")
+        if self.pool is not None and (self.pool < 1 or self.window is None or self.chunk is not None or self.distance_bias):
+            raise ValueError("AttentionSpec: pooled blocks of %d positions need a window, and neither chunks nor a distance bias" % self.pool)
         if self.rotary is not None and (self.rotary.dims % 2 or not 0 < self.rotary.dims <= self.dim or self.rotary.base <= 1):
             raise ValueError("AttentionSpec: rotation of %d elements of %d" % (self.rotary.dims, self.dim))
 

@@ -22,12 +22,13 @@ _i, _ll, _f, _vp = _native._i, _native._ll, _native._f, _native._vp
 _native.register_protos({
     "ft_kv_append": (_i, [_vp] * 7 + [_i] * 6 + [_ll, _ll, _i, _i, _i, _i, _vp]),
     "ft_paged_decode_scratch": (_ll, [_i, _i, _i, _i]),
-    "ft_paged_decode": (_i, [_vp] * 10 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp, _f, _i, _i, _vp]),
-    "ft_paged_rows": (_i, [_vp] * 9 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _i, _f, _i, _i, _vp, _f, _i, _i, _vp]),
+    "ft_paged_decode": (_i, [_vp] * 10 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i] + [_vp] * 2 + [_i, _vp, _f, _i, _i, _vp]),
+    "ft_paged_rows": (_i, [_vp] * 9 + [_i] * 5 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _i, _f, _i, _i] + [_vp] * 2 + [_i, _vp, _f, _i, _i, _vp]),
+    "ft_pool_blocks": (_i, [_vp] * 7 + [_i] * 5 + [_i] * 5 + [_vp]),
     "ft_latent_decode": (_i, [_vp] * 7 + [_i] * 4 + [_ll, _i, _i, _i, _f, _i, _i, _vp]),
     "ft_latent_gather": (_i, [_vp] * 3 + [_i, _i, _vp] + [_i] * 6 + [_vp]),
     "ft_paged_prefill_tile": (_i, [_i]),
-    "ft_paged_prefill": (_i, [_vp] * 8 + [_i] * 6 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i, _vp, _f, _i, _vp]),
+    "ft_paged_prefill": (_i, [_vp] * 8 + [_i] * 6 + [_ll, _ll, _i, _i, _ll] + [_i, _i, _i, _f, _i, _i] + [_vp] * 2 + [_i, _vp, _f, _i, _vp]),
 })
 
 
@@ -42,17 +43,23 @@ def _ptr(t: torch.Tensor | None):
     return t.data_ptr() if t is not None else None
 
 
+def _pool_args(pool: int | None, pooled: tuple | None) -> tuple:
+    """Pooled keys, pooled values and tokens of a block."""
+    return (pooled[0].data_ptr(), pooled[1].data_ptr(), pool) if pool else (None, None, 0)
+
+
 def prefill_pages(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, table: torch.Tensor, items: torch.Tensor, scale: float, *,
                   out: torch.Tensor, gate: torch.Tensor | None = None, window: int | None = None, sink: torch.Tensor | None = None,
-                  chunk: int | None = None, slopes: torch.Tensor | None = None, out_scale: float = 1.0) -> None:
+                  chunk: int | None = None, slopes: torch.Tensor | None = None, out_scale: float = 1.0, pool: int | None = None,
+                  pooled: tuple | None = None) -> None:
     """Attention of the portions listed in ``items`` (device only): ``q [T, Hq, D]``, pages ``k [pages, tokens, Hkv, D]`` and ``v``,
-    block table ``[sequences, pages of one]``."""
+    block table ``[sequences, pages of one]``; ``pooled``: the pages' pooled keys and values (:meth:`PagedKVCache.keep_pooled`)."""
     T, Hq, D = q.shape
     pages, bs, Hkv, Dv = v.shape
     rc = _native.kernels().ft_paged_prefill(
         q.data_ptr(), k.data_ptr(), v.data_ptr(), table.data_ptr(), items.data_ptr(), _ptr(gate), _ptr(sink), out.data_ptr(), items.shape[0], T, Hq, Hkv, D,
-        Dv, q.stride(0), *_gate_args(gate), out.stride(0), bs, table.shape[1], pages, float(scale), int(window or 0), int(chunk or 0), _ptr(slopes),
-        float(out_scale), F._dev(q), F._stream())
+        Dv, q.stride(0), *_gate_args(gate), out.stride(0), bs, table.shape[1], pages, float(scale), int(window or 0), int(chunk or 0), *_pool_args(pool, pooled),
+        _ptr(slopes), float(out_scale), F._dev(q), F._stream())
     _native.check(rc, "ft_paged_prefill")
 
 
@@ -254,6 +261,9 @@ class PagedKVCache:
     K/V pages of every layer.  ``block_size`` tokens per page (16 in the benchmark configs).
     ``n_kv_heads``, ``head_dim`` and ``v_head_dim`` (default: ``head_dim``) are numbers, or one number per layer.
 
+    :meth:`keep_pooled` adds, for a layer, the means of the keys and values of every block of so many consecutive positions.  They lie
+    with the page that holds the block's last position, so they move, are shared and are given back with it.
+
     ``values_in_keys`` (per layer, default none): a layer without values of its own; its values are the leading ``v_head_dim``
     elements of its keys (latent attention).
 
@@ -280,6 +290,7 @@ class PagedKVCache:
         self.v = [k[..., :dv] if shared else torch.zeros((num_blocks, block_size, h, dv), device=self.device, dtype=dtype)
                   for (h, _, dv), k, shared in zip(self.shapes, self.k, self.values_in_keys)]
         self.token_pages: torch.Tensor | None = None
+        self.pooled: dict = {}                            # (layer, tokens of a block): pooled keys, pooled values
         # one row more than there are sequences: the padding rows of a captured decode step own no page
         self.pad_slot = max_seqs
         self._table_host = torch.full((max_seqs + 1, self.max_blocks), -1, dtype=torch.int32)
@@ -300,6 +311,49 @@ class PagedKVCache:
     def keep_tokens(self) -> None:
         """Also keep the token of every position in the pages (for embeddings that look back)."""
         self.token_pages = torch.zeros((self.num_blocks, self.block_size), device=self.device, dtype=torch.int32)
+
+    def keep_pooled(self, layer: int, pool: int) -> None:
+        """Also keep the means of every block of ``pool`` positions (counted from 0) of a layer: ``[pages, blocks that can end in a
+        page, heads, size]``.  Block b is number ``b - first position of its page // pool`` of the page that holds its last position."""
+        if self.values_in_keys[layer]:
+            raise ValueError("PagedKVCache.keep_pooled: layer %d has no values of its own" % layer)
+        if (layer, pool) not in self.pooled:
+            h, d, dv = self.shapes[layer]
+            per = (self.block_size - 1) // pool + 1
+            self.pooled[layer, pool] = tuple(torch.zeros((self.num_blocks, per, h, n), device=self.device, dtype=self.dtype) for n in (d, dv))
+
+    def _pooled_places(self, slots: torch.Tensor, blocks: torch.Tensor, pool: int) -> tuple:
+        """Page and place in it of pooled blocks of sequences (host path)."""
+        page = (blocks * pool + pool - 1) // self.block_size
+        return self._table_host[slots, page].long().clamp(min=0), blocks - page * self.block_size // pool
+
+    def pool_blocks(self, layer: int, batch: RaggedBatch) -> None:
+        """The means of the blocks that end among the rows of a batch, whose keys and values the layer's pages already hold."""
+        for (at, pool), (kp, vp) in self.pooled.items():
+            if at != layer:
+                continue
+            if self.device.type != "cuda":
+                pos, slots = batch.positions.long(), batch.slots.long()
+                ends = ((pos + 1) % pool == 0) & (batch.visible > 0)
+                pos, slots = pos[ends], slots[ends]
+                known = pos[:, None] + torch.arange(1 - pool, 1)
+                pages = self._table_host[slots[:, None], known // self.block_size].long()
+                place = self._pooled_places(slots, pos // pool, pool)
+                for src, dst in ((self.k[layer], kp), (self.v[layer], vp)):
+                    dst[place] = src[pages, known % self.block_size].float().mean(1).to(dst.dtype)
+                continue
+            h, d, dv = self.shapes[layer]
+            rc = _native.kernels().ft_pool_blocks(
+                self.k[layer].data_ptr(), self.v[layer].data_ptr(), kp.data_ptr(), vp.data_ptr(), self.sync_table().data_ptr(), batch.positions.data_ptr(),
+                batch.slots.data_ptr(), batch.n_rows, h, d, dv, pool, int(self.dtype == torch.float32), self.block_size, self.max_blocks, self.num_blocks,
+                F._dev(kp), F._stream())
+            _native.check(rc, "ft_pool_blocks")
+
+    def gather_pooled(self, layer: int, pool: int, seq: int, blocks: int):
+        """Contiguous ``[blocks, Hkv, D]`` pooled keys and ``[blocks, Hkv, Dv]`` values of one sequence (reference path)."""
+        b = torch.arange(blocks)
+        place = self._pooled_places(torch.full_like(b, seq), b, pool)
+        return tuple(t[place] for t in self.pooled[layer, pool])
 
     @property
     def rewindable(self) -> bool:
@@ -385,12 +439,16 @@ class PagedKVCache:
             self.num_blocks, F._dev(k_new), F._stream())
         _native.check(rc, "ft_kv_append")
 
+    def _check_pool(self, layer: int, pool, window, chunk, slopes) -> None:
+        if pool and (not window or chunk or slopes is not None or (layer, pool) not in self.pooled):
+            raise ValueError("PagedKVCache: blocks of %d positions of layer %d are not kept, or come without a window" % (pool, layer))
+
     def _tensor_core_ok(self, layer: int, q: torch.Tensor, max_group: int) -> bool:
         Hkv, D, Dv = self.shapes[layer]
         return (q.dtype == torch.bfloat16 and not self.values_in_keys[layer] and D % 16 == 0 and Dv % 16 == 0 and D <= 128 and Dv <= 128
                 and q.shape[1] // Hkv <= max_group and q.data_ptr() % 16 == 0 and q.stride(0) % 8 == 0)
 
-    def _rows(self, layer: int, q, visible, slots, scale, gate, out, window, sink, chunk=None, slopes=None, out_scale=1.0) -> None:
+    def _rows(self, layer: int, q, visible, slots, scale, gate, out, window, sink, chunk=None, slopes=None, out_scale=1.0, pool=None) -> None:
         """Attention of arbitrary rows, any head sizes, bf16 or fp32 (the simple kernel)."""
         T, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
@@ -398,25 +456,28 @@ class PagedKVCache:
             q.data_ptr(), self.k[layer].data_ptr(), self.v[layer].data_ptr(), self.block_table.data_ptr(), slots.data_ptr(),
             visible.data_ptr(), _ptr(gate), _ptr(sink), out.data_ptr(), T, Hq, Hkv, D, Dv, q.stride(0),
             *_gate_args(gate), out.stride(0), self.v[layer].stride(2), self.block_size, self.max_blocks, self.num_blocks, float(scale),
-            int(window or 0), int(chunk or 0), _ptr(slopes), float(out_scale), int(q.dtype == torch.float32), F._dev(q), F._stream())
+            int(window or 0), int(chunk or 0), *_pool_args(pool, self.pooled.get((layer, pool))), _ptr(slopes), float(out_scale),
+            int(q.dtype == torch.float32), F._dev(q), F._stream())
         _native.check(rc, "ft_paged_rows")
 
     def decode(self, layer: int, q: torch.Tensor, ctx_len: torch.Tensor, scale: float | None = None,
                n_splits: int = 0, seq_ids: torch.Tensor | None = None, gate: torch.Tensor | None = None,
                out: torch.Tensor | None = None, window: int | None = None, sink: torch.Tensor | None = None,
-               chunk: int | None = None, slopes: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
+               chunk: int | None = None, slopes: torch.Tensor | None = None, out_scale: float = 1.0, pool: int | None = None) -> torch.Tensor:
         """One query token per sequence: ``q [B, Hq, D]``, ``ctx_len [B]`` int32 -> ``[B, Hq, Dv]``.  Row b
         reads sequence b, or sequence ``seq_ids[b]`` (int32; a batch of any subset of the live sequences).
         ``gate [B, Hq]`` or ``[B, Hq, Dv]``: output heads or elements are multiplied by its sigmoid.  ``window``: only the
         last so many keys are visible; ``chunk``: those of the query's own chunk of so many positions, counted from 0.  ``sink
         [Hq]`` (fp32): its exponential joins a head's denominator.  ``slopes [Hq]`` (fp32): times the distance of a key, taken off
-        its score.  ``out_scale``: factor of the result.  ``out``: where the result goes (the heads of a row packed, any row stride)."""
+        its score.  ``out_scale``: factor of the result.  ``pool`` (with a window): the means of the blocks of so many positions that lie
+        wholly ahead of the window are visible too (:meth:`keep_pooled`).  ``out``: where the result goes (the heads of a row packed, any row stride)."""
         B, Hq, D = q.shape
         Hkv, _, Dv = self.shapes[layer]
         scale = scale if scale is not None else D ** -0.5
         table = self.sync_table()
+        self._check_pool(layer, pool, window, chunk, slopes)
         if not q.is_cuda:
-            o = self._decode_reference(layer, q, ctx_len, scale, seq_ids, window, sink, chunk, slopes)
+            o = self._decode_reference(layer, q, ctx_len, scale, seq_ids, window, sink, chunk, slopes, pool)
             o = self._finish_reference(o, gate, out_scale)
             return o if out is None else out.copy_(o)
         if out is None:
@@ -426,15 +487,15 @@ class PagedKVCache:
         if plain and self._latent_ok(layer, q):
             return self._latent_rows(layer, q, ctx_len, seq_ids, scale, out, n_splits)
         if not self._tensor_core_ok(layer, q, 16) and (q.dtype != torch.bfloat16 or self.values_in_keys[layer] or D != Dv or D not in (64, 128)
-                                                       or Hq // Hkv not in (1, 2, 4, 8)):
+                                                       or Hq // Hkv not in (1, 2, 4, 8) or pool):
             rows = seq_ids if seq_ids is not None else torch.arange(B, device=q.device, dtype=torch.int32)
-            self._rows(layer, q, ctx_len, rows, scale, gate, out, window, sink, chunk, slopes, out_scale)
+            self._rows(layer, q, ctx_len, rows, scale, gate, out, window, sink, chunk, slopes, out_scale, pool)
             return out
         lib = _native.kernels()
         if n_splits <= 0:
             ctas = B * Hkv
             n_splits = 1 if ctas >= 256 else max(1, min(8, 296 // max(ctas, 1)))
-            if window:
+            if window and not pool:
                 n_splits = min(n_splits, (window + 126) // 128 + 1)          # tiles of 128 keys that a window can touch
             if chunk:
                 n_splits = min(n_splits, (chunk + 126) // 128 + 1)
@@ -445,14 +506,15 @@ class PagedKVCache:
                                  _ptr(gate), _ptr(sink), out.data_ptr(),
                                  scratch.data_ptr() if scratch is not None else None, B, Hq, Hkv, D, Dv, q.stride(0),
                                  *_gate_args(gate), out.stride(0), self.block_size, self.max_blocks, self.num_blocks,
-                                 float(scale), int(window or 0), int(chunk or 0), _ptr(slopes), float(out_scale), n_splits, F._dev(q), F._stream())
+                                 float(scale), int(window or 0), int(chunk or 0), *_pool_args(pool, self.pooled.get((layer, pool))),
+                                 _ptr(slopes), float(out_scale), n_splits, F._dev(q), F._stream())
         _native.check(rc, "ft_paged_decode")
         return out
 
     def attend(self, layer: int, q: torch.Tensor, batch: RaggedBatch, scale: float | None = None,
                gate: torch.Tensor | None = None, out: torch.Tensor | None = None, window: int | None = None,
                sink: torch.Tensor | None = None, chunk: int | None = None, slopes: torch.Tensor | None = None,
-               out_scale: float = 1.0) -> torch.Tensor:
+               out_scale: float = 1.0, pool: int | None = None) -> torch.Tensor:
         """Causal attention of a whole :class:`RaggedBatch` (its keys and values already appended): ``q [T, Hq, D]`` ->
         ``[T, Hq, Dv]``.  Single tokens run on the decode kernel, longer portions on the prefill kernel; head sizes or
         types that those do not cover run on the simple kernel.  The other arguments as in :meth:`decode`."""
@@ -462,17 +524,19 @@ class PagedKVCache:
         if out is None:
             out = torch.empty((T, Hq, Dv), device=q.device, dtype=q.dtype)
         table = self.sync_table()
+        self._check_pool(layer, pool, window, chunk, slopes)
         n1 = batch.n_single
         if n1:
             self.decode(layer, q[:n1], batch.visible[:n1], scale, seq_ids=batch.slots[:n1],
                         gate=gate[:n1] if gate is not None else None, out=out[:n1], window=window, sink=sink, chunk=chunk, slopes=slopes,
-                        out_scale=out_scale)
+                        out_scale=out_scale, pool=pool)
         if not batch.spans:
             return out
         if not q.is_cuda:
             for slot, row, start, n in batch.spans:
                 k, v = self.gather(layer, slot, start + n)
-                o = ref.attention(q[None, row:row + n], k[None], v[None], True, scale, start, window, sink, chunk, slopes)[0][0]
+                kp, vp = self.gather_pooled(layer, pool, slot, max(0, start + n - window) // pool) if pool else (k[:0], v[:0])
+                o = ref.attention(q[None, row:row + n], k[None], v[None], True, scale, start, window, sink, chunk, slopes, pool, (kp[None], vp[None]))[0][0]
                 out[row:row + n] = self._finish_reference(o, gate[row:row + n] if gate is not None else None, out_scale)
             return out
         bs = self.block_size
@@ -482,11 +546,11 @@ class PagedKVCache:
             return out
         if not (self._tensor_core_ok(layer, q, 128) and scale > 0 and bs >= 8 and (128 % bs == 0 or bs % 128 == 0)):
             self._rows(layer, q[n1:], batch.visible[n1:], batch.slots[n1:], scale, gate[n1:] if gate is not None else None, out[n1:],
-                       window, sink, chunk, slopes, out_scale)
+                       window, sink, chunk, slopes, out_scale, pool)
             return out
         items = batch.work_items(int(_native.kernels().ft_paged_prefill_tile(Hq // Hkv)))
         prefill_pages(q, self.k[layer], self.v[layer], table, items, scale, out=out, gate=gate, window=window, sink=sink, chunk=chunk, slopes=slopes,
-                      out_scale=out_scale)
+                      out_scale=out_scale, pool=pool, pooled=self.pooled.get((layer, pool)))
         return out
 
     def _latent_ok(self, layer: int, q: torch.Tensor) -> bool:
@@ -557,7 +621,7 @@ class PagedKVCache:
         o = o if gate is None else ref.head_gate(o, gate)
         return o if out_scale == 1.0 else (o.float() * out_scale).to(o.dtype)
 
-    def _decode_reference(self, layer, q, ctx_len, scale, seq_ids=None, window=None, sink=None, chunk=None, slopes=None):
+    def _decode_reference(self, layer, q, ctx_len, scale, seq_ids=None, window=None, sink=None, chunk=None, slopes=None, pool=None):
         """Host form of the paged-decode kernel, all rows at once: the pages of every row are gathered through
         the block table into a padded ``[B, L, Hkv, D]`` view and positions past a row's length are masked."""
         B, Hq, D = q.shape
@@ -579,6 +643,13 @@ class PagedKVCache:
         if slopes is not None:
             s = s - slopes.float().view(1, Hkv, Hq // Hkv, 1) * (ctx[:, None] - 1 - at).float()[:, None, None, :]
         s = s.masked_fill(dead[:, None, None, :], float("-inf"))
+        seen = (ctx - window).clamp(min=0) // pool if pool else torch.zeros(1, dtype=torch.long)
+        if int(seen.max()):
+            b = torch.arange(int(seen.max()))[None]
+            kp, vp = (t[self._pooled_places(rows[:, None], b, pool)].float() for t in self.pooled[layer, pool])
+            sp = torch.einsum("bhgd,blhd->bhgl", qf, kp) * scale
+            s = torch.cat([s, sp.masked_fill((b >= seen[:, None])[:, None, None, :], float("-inf"))], -1)
+            v = torch.cat([v, vp], 1)
         if sink is not None:                              # one more column of the softmax, without a value
             s = torch.cat([s, sink.float().view(1, Hkv, Hq // Hkv, 1).expand(B, -1, -1, 1)], -1)
         o = torch.einsum("bhgl,blhd->bhgd", torch.softmax(s, -1)[..., :v.shape[1]], v)

@@ -1,7 +1,7 @@
-"""Front ends of the kernels that pre-norm decoders over paged caches use beside the projections and the attention: RMS
-norm of fp32 residual rows, the per-head pass between projection and attention (``csrc/decoder_rows.cu``), residuals of
-several streams and n-gram embeddings (``csrc/streams.cu``), short convolution and gated linear recurrence
-(``csrc/recurrent.cu``), matrix memories (``csrc/matrix_memory.cu``), the pass ahead of latent attention
+"""Front ends of the kernels that decoders over paged caches use beside the projections and the attention: RMS
+norm of fp32 residual rows, norm after a residual sum, norms of parts and powers of a row, the per-head pass between projection and
+attention (``csrc/decoder_rows.cu``), residuals of several streams and n-gram embeddings (``csrc/streams.cu``), short convolution and gated linear recurrence
+(``csrc/recurrent.cu``), matrix memories and state-space heads (``csrc/matrix_memory.cu``), the pass ahead of latent attention
 (``csrc/latent_attn.cu``), routing and grouped products of expert layers and products by blocks (``csrc/grouped_gemm.cu``).
 
 CUDA tensors run the kernels (bf16 on the tensor cores where there is a product, fp32 in true 32-bit); CPU tensors run
@@ -21,11 +21,15 @@ _i, _ll, _f, _vp = _native._i, _native._ll, _native._f, _native._vp
 _native.register_protos({
     "ft_rms_rows": (_i, [_vp, _vp, _i, _i] + [_vp] * 3 + [_i, _i, _vp, _vp] + [_i] * 4 + [_ll] * 4 + [_f, _f, _i, _vp]),
     "ft_qkv_head_finish": (_i, [_vp, _ll] + [_vp] * 8 + [_i] * 11 + [_f] + [_i] * 5 + [_vp]),
-    "ft_causal_conv": (_i, [_vp, _ll] + [_vp] * 4 + [_ll] + [_vp] * 3 + [_i] * 6 + [_vp]),
+    "ft_sum_norm_rows": (_i, [_vp, _ll, _vp, _i, _i, _vp, _vp, _ll, _vp, _vp, _ll, _i, _vp, _vp, _i, _vp, _ll, _f] + [_vp] * 3 + [_ll, _vp, _ll] + [_i] * 5 + [_f, _i, _vp]),
+    "ft_part_norm": (_i, [_vp, _ll, _vp] + [_i] * 5 + [_f, _i, _i, _vp]),
+    "ft_poly_norm": (_i, [_vp, _ll, _vp, _ll, _vp] + [_i] * 3 + [_f, _i, _i, _vp]),
+    "ft_causal_conv": (_i, [_vp, _ll] + [_vp] * 4 + [_ll] + [_vp] * 3 + [_i] * 7 + [_vp]),
+    "ft_conv_tail": (_i, [_vp, _ll, _vp, _vp] + [_i] * 5 + [_vp]),
     "ft_rglru_gates": (_i, [_vp, _ll] + [_vp] * 4 + [_i] * 3 + [_vp, _vp, _i] + [_vp] * 4 + [_ll, _vp, _ll] + [_i] * 3 + [_vp]),
     "ft_rglru_scan": (_i, [_vp] * 3 + [_ll, _vp, _ll, _vp, _vp, _i, _vp, _ll, _vp] + [_i] * 4 + [_vp]),
     "ft_moe_max_items": (_i, [_i, _i]),
-    "ft_moe_route": (_i, [_vp, _ll, _vp, _vp, _ll] + [_i] * 6 + [_vp, _i, _i] + [_vp] * 5 + [_i, _vp, _vp, _i, _vp]),
+    "ft_moe_route": (_i, [_vp, _ll, _vp, _vp, _ll] + [_i] * 6 + [_vp, _vp, _i, _vp, _i] + [_vp] * 5 + [_i, _vp, _vp, _i, _vp]),
     "ft_block_linear": (_i, [_vp, _ll, _i, _vp] + [_i] * 6 + [_vp, _ll, _i, _vp, _ll] + [_i] * 3 + [_vp]),
     "ft_few_outputs": (_i, [_vp, _ll, _vp, _vp] + [_i] * 5 + [_vp]),
     "ft_stream_step": (_i, [_vp, _ll, _ll, _vp, _i] + [_vp] * 4 + [_i, _vp, _ll, _vp, _ll, _i, _vp, _vp, _i, _vp, _ll, _vp, _vp, _ll] + [_i] * 3 + [_f, _i, _i, _vp]),
@@ -35,6 +39,9 @@ _native.register_protos({
     "ft_memory_scratch": (_ll, [_i] * 5),
     "ft_memory_chunks": (_i, [_vp] * 4 + [_ll, _vp, _ll, _i] + [_vp] * 7 + [_ll] + [_i] * 4 + [_f] * 4 + [_i, _vp, _i, _vp, _vp, _i, _vp, _i, _vp]),
     "ft_memory_steps": (_i, [_vp] * 4 + [_ll, _vp, _ll, _i] + [_vp] * 7 + [_ll] + [_i] * 4 + [_f] * 4 + [_vp] * 3 + [_i] * 3 + [_vp]),
+    "ft_state_scratch": (_ll, [_i] * 5),
+    "ft_state_chunks": (_i, [_vp] * 3 + [_ll, _vp, _ll, _vp, _ll] + [_vp] * 5 + [_ll] + [_i] * 5 + [_vp, _i, _vp, _vp, _i, _vp, _i, _vp]),
+    "ft_state_steps": (_i, [_vp] * 3 + [_ll, _vp, _ll, _vp, _ll] + [_vp] * 5 + [_ll] + [_i] * 4 + [_vp] * 3 + [_i] * 3 + [_vp]),
     "ft_grouped_gemm": (_i, [_vp, _ll, _i] + [_vp] * 3 + [_i] * 5 + [_vp, _i, _vp, _ll] + [_i] * 4 + [_vp]),
 })
 
@@ -88,25 +95,63 @@ def embedding_rms(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, 
     return x, h
 
 
-# --------------------------------------------------------------------------- residuals of several streams
+# --------------------------------------------------------------------------- residuals of one or several streams
 class SublayerTerms(NamedTuple):
     """What a sublayer adds to the residual, not yet summed: rows ``terms[where[i, j]]`` for all j (times ``weight[i, j]``), a dense
-    row ``dense[i]``; where ``where[i, j]`` is negative, ``weight[i, j]`` times the sublayer's own input ``own[i]``."""
+    row ``dense[i]`` (times ``dense_weight[i]``); where ``where[i, j]`` is negative, ``weight[i, j]`` times the sublayer's own input
+    ``own[i]``."""
     terms: torch.Tensor | None = None
     where: torch.Tensor | None = None
     weight: torch.Tensor | None = None
     dense: torch.Tensor | None = None
     own: torch.Tensor | None = None
+    dense_weight: torch.Tensor | None = None
 
     def total(self) -> torch.Tensor:
         """The sum, fp32."""
         y = self.dense.float() if self.dense is not None else 0.0
+        if self.dense_weight is not None:
+            y = y * self.dense_weight[:, None]
         if self.terms is None:
             return y
         t, w = self.terms[self.where.clamp(min=0).long()].float(), self.weight if self.weight is not None else torch.ones_like(self.where, dtype=torch.float32)
         if self.own is not None:
             t = torch.where(self.where[..., None] < 0, self.own.float()[:, None], t)
         return y + (t * w[..., None]).sum(1)
+
+
+def sum_norm(x: torch.Tensor, y: SublayerTerms, gate: torch.Tensor | None, alpha: float, weight: torch.Tensor, eps: float, *, count: int,
+             out_dtype: torch.dtype, ids: torch.Tensor | None = None, rows: torch.Tensor | None = None, last: torch.Tensor | None = None):
+    """Norm after the sum: ``x' = norm(alpha x + sigmoid(gate) y) * weight`` (RMS over ``count`` elements), fp32 and as the next input.
+
+    ``x [T, H]`` fp32 rows, or with ``ids`` rows ``x[ids]`` of an embedding table; ``gate [T, H]``: pre-activations, a view of a
+    projection (``None``: no gate).  Returns ``(x', h)``; fp32 ``x`` is updated in place, and with an fp32 ``out_dtype`` both are one
+    tensor.  ``rows``: only these rows, and no ``x'``; ``last``: weight of a second norm, of ``x'``, that ``h`` goes through."""
+    H = x.shape[1]
+    if not x.is_cuda:
+        s = x[ids].float() if ids is not None else x
+        t = y.total()
+        s = alpha * s + (t if gate is None else t * torch.sigmoid(gate.float()))
+        s = ref.rms_rows(s if rows is None else s[rows], weight, eps, count)
+        h = s if last is None else ref.rms_rows(s, last, eps, count)
+        return s, h.to(out_dtype)
+    if y.own is not None:
+        raise ValueError("sum_norm: terms of a sublayer's own input")
+    T = x.shape[0] if ids is None else ids.numel()
+    n = T if rows is None else rows.numel()
+    new = None
+    if rows is None:
+        new = x if ids is None else torch.empty((T, H), device=x.device, dtype=torch.float32)
+    same = new is not None and last is None and out_dtype == torch.float32
+    h = None if same else torch.empty((n, H), device=x.device, dtype=out_dtype)
+    t, dense = y.terms, y.dense
+    rc = _native.kernels().ft_sum_norm_rows(
+        x.data_ptr(), x.stride(0), _ptr(ids), x.shape[0], int(x.dtype == torch.bfloat16), _ptr(rows), _ptr(dense), dense.stride(0) if dense is not None else 0,
+        _ptr(y.dense_weight), _ptr(t), t.stride(0) if t is not None else 0, t.shape[0] if t is not None else 0, _ptr(y.where), _ptr(y.weight),
+        y.where.shape[1] if t is not None else 0, _ptr(gate), gate.stride(0) if gate is not None else 0, float(alpha), weight.data_ptr(), _ptr(last),
+        _ptr(new), H, _ptr(h), H, int(out_dtype == torch.float32), n, T, H, count, float(eps), F._dev(x), F._stream())
+    _native.check(rc, "ft_sum_norm_rows")
+    return new, (new if same else h)
 
 
 def stream_step(x: torch.Tensor, y: SublayerTerms, mix: torch.Tensor, out: torch.Tensor, into: torch.Tensor, weight: torch.Tensor, eps: float,
@@ -117,6 +162,8 @@ def stream_step(x: torch.Tensor, y: SublayerTerms, mix: torch.Tensor, out: torch
     where ``x`` is dense; ``h`` the RMS norm of ``sum_t into[t] x'_t`` times ``weight``.  ``rows``: only these rows; without
     ``update`` (always with ``rows``) the streams are not written."""
     T, S, H = x.shape
+    if y.dense_weight is not None:
+        raise ValueError("stream_step: dense rows have no weights of their own")
     if not x.is_cuda:
         new = torch.einsum("nsh,st->nth", x, mix) + out[:, None] * y.total()[:, None, :]
         u = torch.einsum("nth,t->nh", new if rows is None else new[rows], into)
@@ -173,6 +220,33 @@ def softcap_(z: torch.Tensor, cap: float) -> torch.Tensor:
     rc = _native.kernels().ft_softcap(z.data_ptr(), z.numel(), float(cap), F._dev(z), F._stream())
     _native.check(rc, "ft_softcap")
     return z
+
+
+# --------------------------------------------------------------------------- norms inside sublayers
+def part_norm_(y: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, *, heads: int, vdim: int) -> torch.Tensor:
+    """RMS norm of ``parts`` equal runs of every row on their own, times ``weight``, in place.  Rows ``[T, heads * vp]`` are heads of
+    ``vdim`` elements padded to ``vp``, and runs count the true elements."""
+    T, vp = y.shape[0], y.shape[1] // heads
+    if not y.is_cuda:
+        true = y.unflatten(1, (heads, vp))[:, :, :vdim]
+        true.copy_(ref.part_rms(true.flatten(1), weight.view(heads, vp)[:, :vdim].flatten(), parts, eps).view(T, heads, vdim))
+        return y
+    rc = _native.kernels().ft_part_norm(y.data_ptr(), y.stride(0), weight.data_ptr(), T, heads, vdim, vp, parts, float(eps), int(y.dtype == torch.float32),
+                                        F._dev(y), F._stream())
+    _native.check(rc, "ft_part_norm")
+    return y
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, *, count: int) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e``, ``coef [4] = (a, b, c, e)`` fp32, N dividing a row (zero beyond ``count`` elements) by its
+    root mean square."""
+    if not z.is_cuda:
+        return ref.poly_norm(z, coef, count, eps).to(z.dtype)
+    out = torch.empty(z.shape, device=z.device, dtype=z.dtype)
+    rc = _native.kernels().ft_poly_norm(z.data_ptr(), z.stride(0), out.data_ptr(), out.stride(0), coef.data_ptr(), z.shape[0], z.shape[1], count, float(eps),
+                                        int(z.dtype == torch.float32), F._dev(z), F._stream())
+    _native.check(rc, "ft_poly_norm")
+    return out
 
 
 # --------------------------------------------------------------------------- projection -> attention, per head
@@ -285,10 +359,11 @@ def _span_list(batch) -> list:
     return [(s, i, p, 1) for i, (s, p) in enumerate(zip(slots, pos))] + [tuple(s) for s in batch.spans]
 
 
-def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, batch) -> torch.Tensor:
+def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, batch, silu: bool = False) -> torch.Tensor:
     """Causal convolution per channel over the rows ``x [T, C]`` of a ragged batch: ``weight [taps, C]`` (the last one weighs
-    the row itself), ``bias [C]``, fp32.  ``state [slots, taps - 1, C]`` holds the inputs ahead of a sequence's next row.
-    Rows that are a sequence's only token store theirs here, portions in :func:`rglru_scan`."""
+    the row itself), ``bias [C]``, fp32; ``silu``: of the result.  ``state [slots, taps - 1, C]`` holds the inputs ahead of a
+    sequence's next row.  Rows that are a sequence's only token store theirs here, portions in :func:`conv_tail` or
+    :func:`rglru_scan`."""
     taps, C = weight.shape
     u = torch.empty((x.shape[0], C), device=x.device, dtype=x.dtype)
     if not x.is_cuda:
@@ -296,16 +371,31 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, state
             known = min(start, taps - 1)
             ahead = torch.cat([x.new_zeros(taps - 1 - known, C), state[slot, taps - 1 - known:]])
             z = torch.cat([ahead, x[row:row + n]]).float()
-            u[row:row + n] = sum(weight[j] * z[j:j + n] for j in range(taps)) + bias
+            out = sum(weight[j] * z[j:j + n] for j in range(taps)) + bias
+            u[row:row + n] = ref.activation(out, "silu") if silu else out
             if row < batch.n_single:
                 state[slot] = z[n:].to(state.dtype)
         return u
     rc = _native.kernels().ft_causal_conv(
         x.data_ptr(), x.stride(0), weight.data_ptr(), bias.data_ptr(), state.data_ptr(), u.data_ptr(), u.stride(0),
         batch.positions.data_ptr(), batch.slots.data_ptr(), batch.starts.data_ptr(), x.shape[0], batch.n_single, C, taps,
-        int(x.dtype == torch.float32), F._dev(x), F._stream())
+        int(silu), int(x.dtype == torch.float32), F._dev(x), F._stream())
     _native.check(rc, "ft_causal_conv")
     return u
+
+
+def conv_tail(x: torch.Tensor, state: torch.Tensor, batch) -> None:
+    """The last inputs of the portions of a batch, ``x [T, C]``, into the slots of a convolution's ``state [slots, taps - 1, C]``."""
+    keep = state.shape[1]
+    if not batch.spans or not keep:
+        return
+    if not x.is_cuda:
+        for slot, row, _, n in batch.spans:
+            state[slot] = torch.cat([state[slot], x[row:row + n].to(state.dtype)])[n:n + keep]
+        return
+    rc = _native.kernels().ft_conv_tail(x.data_ptr(), x.stride(0), state.data_ptr(), batch.span_table.data_ptr(), len(batch.spans), x.shape[1], keep,
+                                        int(x.dtype == torch.float32), F._dev(x), F._stream())
+    _native.check(rc, "ft_conv_tail")
 
 
 def gated_recurrence(u: torch.Tensor, y: torch.Tensor, gates: torch.Tensor, r_bias: torch.Tensor, i_bias: torch.Tensor,
@@ -409,11 +499,56 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch
     return out
 
 
+def state_space(u: torch.Tensor, gate: torch.Tensor, step: torch.Tensor, step_bias: torch.Tensor, rate: torch.Tensor, skip: torch.Tensor, state: torch.Tensor,
+                batch, out: torch.Tensor, *, heads: int, groups: int, chunks: bool = False) -> torch.Tensor:
+    """State-space heads over the rows of a ragged batch (see ``csrc/matrix_memory.cu``): ``S <- exp(-rate dt) S + dt B x^T`` with ``dt =
+    softplus(step + step_bias)``, ``out = (S^T C + skip x) silu(gate)``.
+
+    ``u [T, heads * vp + 2 * groups * np]``: x of the heads, B and C of the groups (head h uses group ``h // (heads / groups)``), padded
+    sizes; ``gate, out [T, heads * vp]``; ``step [T, >= heads]`` fp32; ``step_bias, rate, skip [heads]``; ``state [slots, heads, np, vp]``
+    fp32.  Portions in bf16 run in chunks (short ones only with ``chunks``), everything else token by token."""
+    np_, vp = state.shape[2:]
+    hx, gn = heads * vp, groups * np_
+    x, B, C = u[:, :hx], u[:, hx:hx + gn], u[:, hx + gn:]
+    if not u.is_cuda:
+        dt = torch.nn.functional.softplus(step[:, :heads] + step_bias, threshold=1e9)
+        Bs, Cs = (t.float().unflatten(1, (groups, np_)).repeat_interleave(heads // groups, 1) for t in (B, C))
+        xs = x.float().unflatten(1, (heads, vp))
+        for slot, row, start, n in _span_list(batch):
+            if start == 0:
+                state[slot].zero_()
+            r = slice(row, row + n)
+            y = ref.state_space(Cs[r], Bs[r], xs[r], dt[r], rate, state[slot]) + skip[:, None] * xs[r]
+            out[r] = (y.flatten(1) * ref.activation(gate[r].float(), "silu")).to(out.dtype)
+        return out
+    lib, f32, group, T = _native.kernels(), u.dtype == torch.float32, heads // groups, u.shape[0]
+    args = (C.data_ptr(), B.data_ptr(), x.data_ptr(), u.stride(0), gate.data_ptr(), gate.stride(0), step.data_ptr(), step.stride(0), step_bias.data_ptr(),
+            rate.data_ptr(), skip.data_ptr(), state.data_ptr(), out.data_ptr(), out.stride(0), heads, group, np_, vp)
+
+    def steps(spans, items):
+        rc = lib.ft_state_steps(*args, _ptr(spans), batch.positions.data_ptr(), batch.slots.data_ptr(), items, int(f32), F._dev(u), F._stream())
+        _native.check(rc, "ft_state_steps")
+
+    if batch.n_single:
+        steps(None, batch.n_single)
+    if not batch.spans:
+        return out
+    if f32 or np_ > 128 or vp > 256 or (batch.longest <= MEMORY_STEP_ROWS and not chunks):
+        steps(batch.span_table, len(batch.spans))
+        return out
+    first, table = batch.chunk_table(MEMORY_CHUNK)
+    scratch = F._get_scratch("matrix_memory", (int(lib.ft_state_scratch(T, heads, np_, vp, table.shape[0])) + 3) // 4, u.device)
+    rc = lib.ft_state_chunks(*args, T, batch.span_table.data_ptr(), len(batch.spans), first.data_ptr(), table.data_ptr(), table.shape[0], scratch.data_ptr(),
+                             F._dev(u), F._stream())
+    _native.check(rc, "ft_state_chunks")
+    return out
+
+
 # --------------------------------------------------------------------------- expert layers
 @dataclass
 class Routing:
     """Rows sorted by expert: ``sorted [T * top, H]``, ``place [T, top]`` (where a row's copies lie; -1: a choice without
-    matrices), ``scale [T * top]`` (their weights), ``items`` / ``n_items`` (segments, on the device)."""
+    matrices), ``scale [T * top]`` (their weights), ``items`` / ``n_items`` (segments, on the device); ``gate [T]``: the sigmoid of one more output of the router."""
     index: torch.Tensor
     weight: torch.Tensor
     place: torch.Tensor
@@ -421,6 +556,7 @@ class Routing:
     items: torch.Tensor
     n_items: torch.Tensor
     sorted: torch.Tensor
+    gate: torch.Tensor | None = None
 
 
 _SCORES = {"sigmoid": 0, "softmax": 1}
@@ -428,24 +564,27 @@ ROUTE_ROWS = 512      # up to so many rows the routing kernel computes the logit
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, top: int, *, identity: int = 0, score: str = "sigmoid",
-              correction: torch.Tensor | None = None, normalize: bool = False) -> Routing:
+              correction: torch.Tensor | None = None, normalize: bool = False, bias: torch.Tensor | None = None, gate: bool = False) -> Routing:
     """The ``top`` choices of every row of ``h [T, H]`` by its logits ``router h`` (fp32), and the rows sorted by expert.
 
     ``score``: ``sigmoid`` (the largest logits, weighted by their sigmoid) or ``softmax`` over all logits (the largest scores after
     adding ``correction``, weighted by the score itself; ``normalize``: over the sum of the chosen ones).  The router's first
-    ``experts`` outputs are experts, ``identity`` more have no matrices.  ``router [>= experts + identity, H]`` (padded rows are
+    ``experts`` outputs are experts, ``identity`` more have no matrices.  ``bias`` (fp32, one per output) joins the logits; with ``gate``
+    the output behind these is no choice: its sigmoid is returned.  ``router [>= experts + identity + gate, H]`` (padded rows are
     ignored)."""
     T, H = h.shape
     outputs = experts + identity
     if not h.is_cuda:
-        index, weight = ref.top_experts(h.float() @ router[:outputs].float().t(), top, score, correction, normalize)
+        z = h.float() @ router[:outputs].float().t()
+        index, weight = ref.top_experts(z if bias is None else z + bias, top, score, correction, normalize)
+        own = torch.sigmoid(h.float() @ router[outputs].float()) if gate else None
         order = index.flatten().argsort(stable=True)
         place = torch.empty_like(order)
         place[order] = torch.arange(order.numel())
         place[index.flatten() >= experts] = -1
         real = int((index < experts).sum())
         return Routing(index, weight, place.view(T, top).int(), weight.flatten()[order], index.flatten()[order][:real], torch.tensor(real),
-                       h[order // top])
+                       h[order // top], own)
     lib, dev = _native.kernels(), h.device
     cap = int(lib.ft_moe_max_items(T * top, experts))
     ints = torch.empty(2 * T * top + 3 * cap + 1, device=dev, dtype=torch.int32)
@@ -453,23 +592,24 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, experts: int, top: int, *, 
     items, n_items = rest[:3 * cap].view(cap, 3), rest[3 * cap:]
     weight, scale = torch.empty((2, T * top), device=dev, dtype=torch.float32)
     rows = torch.empty((T * top, H), device=dev, dtype=h.dtype)
+    own = torch.empty(T, device=dev, dtype=torch.float32) if gate else None
     logits = F.linear_f32_out(h, router) if T > ROUTE_ROWS else None
     rc = lib.ft_moe_route(h.data_ptr(), h.stride(0), router.data_ptr(), _ptr(logits), logits.stride(0) if logits is not None else 0, T, H,
-                          experts, outputs, top, _SCORES[score], _ptr(correction), int(normalize), int(h.dtype == torch.float32), index.data_ptr(), weight.data_ptr(), place.data_ptr(),
+                          experts, outputs, top, _SCORES[score], _ptr(correction), _ptr(bias), int(normalize), _ptr(own), int(h.dtype == torch.float32), index.data_ptr(), weight.data_ptr(), place.data_ptr(),
                           scale.data_ptr(), items.data_ptr(), cap, n_items.data_ptr(), rows.data_ptr(), F._dev(h), F._stream())
     _native.check(rc, "ft_moe_route")
-    return Routing(index, weight.view(T, top), place, scale, items, n_items, rows)
+    return Routing(index, weight.view(T, top), place, scale, items, n_items, rows, own)
 
 
 def grouped_linear(a: torch.Tensor, w: torch.Tensor, routing: Routing, *, glu: str | None = None, seg_rows: int = 0,
-                   bn: int = 0, scaled: bool = True) -> torch.Tensor:
+                   bn: int = 0, scaled: bool = True, activation: str | None = None) -> torch.Tensor:
     """Rows sorted by expert through their expert's matrix: ``a [R, K]``, ``w [experts, parts, N, K]`` -> ``[R, N]``.  One part: the
-    product.  Two parts (gate, up) with ``glu`` naming the activation: ``act(gate r a) * (up r a)`` with r the row's routing
+    product, of which ``activation`` (relu2) is taken when named.  Two parts (gate, up) with ``glu`` naming the activation: ``act(gate r a) * (up r a)`` with r the row's routing
     weight (``scaled`` false: 1).  ``seg_rows``: an upper bound of the rows of one expert."""
     E, parts, N, K = w.shape
     R = a.shape[0]
-    if parts != (2 if glu else 1):
-        raise ValueError("grouped_linear: %d parts with activation %r" % (parts, glu))
+    if parts != (2 if glu else 1) or activation not in (None, "relu2") or (glu and activation):
+        raise ValueError("grouped_linear: %d parts with activation %r" % (parts, glu or activation))
     out = torch.empty((R, N), device=a.device, dtype=a.dtype)
     if not a.is_cuda:
         for e in routing.items.unique().tolist():
@@ -479,11 +619,11 @@ def grouped_linear(a: torch.Tensor, w: torch.Tensor, routing: Routing, *, glu: s
                 s = routing.scale[rows][:, None] if scaled else 1.0
                 out[rows] = (ref._ACTS[F._ACT_ID[glu]](s * z[0]) * (s * z[1])).to(out.dtype)
             else:
-                out[rows] = z[0].to(out.dtype)
+                out[rows] = (ref.activation(z[0], activation) if activation else z[0]).to(out.dtype)
         return out
     rc = _native.kernels().ft_grouped_gemm(
         a.data_ptr(), a.stride(0), R, w.data_ptr(), routing.items.data_ptr(), routing.n_items.data_ptr(), routing.items.shape[0], E, N, K,
-        int(glu is not None), routing.scale.data_ptr() if glu and scaled else None, F._ACT_ID[glu] if glu else 0, out.data_ptr(), out.stride(0),
+        int(glu is not None), routing.scale.data_ptr() if glu and scaled else None, F._ACT_ID[glu] if glu else (3 if activation else 0), out.data_ptr(), out.stride(0),
         seg_rows, int(a.dtype == torch.float32), bn, F._dev(a), F._stream())
     _native.check(rc, "ft_grouped_gemm")
     return out

@@ -213,6 +213,32 @@ def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Te
     return out
 
 
+def state_space(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, step: torch.Tensor, rate: torch.Tensor, S: torch.Tensor) -> torch.Tensor:
+    """``S <- exp(-rate step) S + step k v^T``, output ``S^T q``, over rows ``q, k [T, H, N]``, ``v [T, H, V]`` with step sizes ``step
+    [T, H]`` and rates ``[H]``, from (and into) ``S [H, N, V]``: outputs ``[T, H, V]``, fp32."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        S.mul_(torch.exp(-rate * step[t])[:, None, None]).add_((step[t][:, None] * k[t])[:, :, None] * v[t][:, None, :])
+        out[t] = torch.einsum("hnv,hn->hv", S, q[t])
+    return out
+
+
+def part_rms(x: torch.Tensor, weight: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
+    """RMS norm of ``parts`` equal runs of every row of ``x [T, C]`` on their own, times ``weight [C]``, fp32."""
+    xp = x.float().unflatten(1, (parts, -1))
+    return (xp / torch.sqrt(xp.pow(2).mean(-1, keepdim=True) + eps)).flatten(1) * weight.float()
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, count: int, eps: float) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` with ``coef = (a, b, c, e)``, N dividing a row (zero beyond ``count`` elements) by its root
+    mean square, fp32."""
+    z, out = z.float(), coef[3].float()
+    for power in (1, 2, 3):
+        w = z ** power
+        out = out + coef[power - 1].float() * (w / torch.sqrt(w.pow(2).sum(-1, keepdim=True) / count + eps))
+    return out
+
+
 def swiglu(gu: torch.Tensor, act: int = 0) -> torch.Tensor:
     """``act(gate) * up`` for ``gu = [gate | up]`` on the last dim (ferrotorch-llama/src/gpu.rs:696-703;
     relu / gelu variants: ferrotorch-nn/src/transformer.rs:693-764)."""
@@ -238,14 +264,17 @@ def repeat_kv(x: torch.Tensor, n_rep: int) -> torch.Tensor:
 
 def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = True,
               scale: float | None = None, q_offset: int | None = None, window: int | None = None,
-              sink: torch.Tensor | None = None, chunk: int | None = None, slopes: torch.Tensor | None = None):
+              sink: torch.Tensor | None = None, chunk: int | None = None, slopes: torch.Tensor | None = None,
+              pool: int | None = None, pooled: tuple | None = None):
     """GQA attention on ``[B, S, H, D]`` tensors, returns ``(out [B,Sq,Hq,D], lse [B,Hq,Sq])``.
 
     Scores scaled by ``1/sqrt(D)``, causal mask hides ``j > i + q_offset`` where the default
     offset aligns the last query with the last key (for Sq == Sk this is the reference's
     top-left mask, ferrotorch-nn/src/flash_attention.rs:647-746), max-subtracted softmax.  With ``window`` a query
     sees only its last so many keys, with ``chunk`` those of its own chunk of so many positions; ``slopes [Hq]`` times the
-    distance of a key is taken off its score; with ``sink [Hq]`` a head's denominator gains ``exp(sink)``."""
+    distance of a key is taken off its score; with ``sink [Hq]`` a head's denominator gains ``exp(sink)``.  With ``pool`` and a
+    window a query also sees ``pooled = (keys, values)`` ``[B, blocks, H, D]``, one per block of ``pool`` positions, of the blocks
+    that lie wholly ahead of its window."""
     B, Sq, Hq, D = q.shape
     Sk, Hkv = k.shape[1], k.shape[2]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -264,6 +293,12 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, causal: bool = 
             s = s.masked_fill(j < i // chunk * chunk, float("-inf"))
         if window:
             s = s.masked_fill(i - j >= window, float("-inf"))
+        if pool and pooled[0].shape[1]:
+            kp, vp = (repeat_kv(t.float().permute(0, 2, 1, 3), Hq // Hkv) for t in pooled)
+            sp = torch.matmul(qf, kp.transpose(-1, -2)) * scale
+            seen = (i + 1 - window).clamp(min=0) // pool
+            s = torch.cat([s, sp.masked_fill(torch.arange(kp.shape[2], device=q.device)[None, :] >= seen, float("-inf"))], -1)
+            vf = torch.cat([vf, vp], 2)
     lse = torch.logsumexp(s, dim=-1)
     if sink is not None:
         lse = torch.logaddexp(lse, sink.float().view(1, Hq, 1))

@@ -75,6 +75,8 @@ _MODELS = [
               "ferrotorch_b200.models.zolorax:ZoloraxConfig.preset_3b", 5_734_027_968),
     ModelInfo("tenalorn-3b", "Tenalorn decoder at 3B layer sizes, eight experts of which two are used (a shape: no trained weights)",
               "ferrotorch_b200.models.tenalorn:TenalornConfig.preset_3b", 7_840_391_128),
+    ModelInfo("mogelix-3b", "Mogelix decoder at 3B layer sizes, eight experts of which two are used (a shape: no trained weights)",
+              "ferrotorch_b200.models.mogelix:MogelixConfig.preset_3b", 5_810_345_808),
     ModelInfo("all-MiniLM-L6-v2", "Sentence embeddings, 6-layer MiniLM", "ferrotorch_b200.models.pretrained:SentenceTransformer", 22_713_216),
     ModelInfo("whisper-tiny-encoder", "Whisper tiny audio encoder", "ferrotorch_b200.models.pretrained:WhisperEncoder", 8_208_384),
     ModelInfo("sd-v1-5-unet", "Stable Diffusion 1.5 UNet", "ferrotorch_b200.models.diffusion:UNet2DConditionModel", 859_520_964),

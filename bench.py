@@ -68,7 +68,7 @@ def parse_args():
                     help="decoder-serving: prefill / decode throughput of the decoder families side by side on one GPU "
                     "(benchmarks/decoder_serving.py) instead of the training step")
     ap.add_argument("--serving-sizes", default="1b,3b,8b")
-    ap.add_argument("--serving-families", default="llama,bopudra,zolorax,tenalorn")
+    ap.add_argument("--serving-families", default="llama,bopudra,zolorax,tenalorn,mogelix")
     ap.add_argument("--serving-kernels", action="store_true", help="also time every kernel of a layer against its roofline")
     return ap.parse_args()
 

@@ -21,13 +21,16 @@ import torch
 # two-matrix MLP is 1.5 x as wide, so both have the same number of parameters and matrix-product FLOPs.  Zolorax has the
 # same dense MLP in every other layer and eight experts of half the SwiGLU width, two of them used, in the others: equal
 # FLOPs per token, but more weights to read in a decode step.  Tenalorn has in every layer eight experts of a third of the
-# SwiGLU width, two of them used, and a shared one: again equal FLOPs; memories of 128 x 128 with half the width in all.
+# SwiGLU width, two of them used, and a shared one: again equal FLOPs; memories of 128 x 128 with half the width in all.  Mogelix
+# has the dense MLP in every sixth layer, in the others eight two-matrix experts of half the SwiGLU width, two of them used, and a
+# shared one: equal FLOPs; state-space heads of 64 with twice the width in all and states of 128, and a gate of the width of the
+# model for every sublayer.
 SIZES = {"1b": (2048, 16, 32, 8, 64, 8192, 128256, 2048, 64),
          "3b": (3072, 28, 24, 8, 128, 8192, 128256, 2048, 64),
          "8b": (4096, 32, 32, 8, 128, 14336, 128256, 2048, 64)}
-FAMILIES = ("llama", "bopudra", "zolorax", "tenalorn")
+FAMILIES = ("llama", "bopudra", "zolorax", "tenalorn", "mogelix")
 PAGE = 16
-EXPERTS, TOP, WINDOW = 8, 2, 1024
+EXPERTS, TOP, WINDOW, POOL = 8, 2, 1024, 16
 
 
 def zolorax_config(size: str, n: int):
@@ -48,6 +51,14 @@ def tenalorn_config(size: str, n: int):
                                   memory_vdim=128, rank=512, experts=EXPERTS, top=TOP, identity=0, streams=2, bigram=BigramSpec(131071, 1031, 17))
 
 
+def mogelix_config(size: str, n: int):
+    from ferrotorch_b200.models.mogelix import MogelixConfig
+
+    hidden, _, heads, kv, dim, ff, vocab, _, _ = SIZES[size]
+    return MogelixConfig.pattern(vocab, hidden, n, heads, kv, dim, ff * 3 // 2, window=WINDOW, pool=POOL, state_dim=64, state=128, experts=EXPERTS, top=TOP,
+                                 expert_ff=ff // 2, shared_ff=ff // 2, alpha=3.0)
+
+
 def build(family: str, size: str, layers: int | None = None):
     hidden, n, heads, kv, dim, ff, vocab, _, _ = SIZES[size]
     n = layers or n
@@ -63,6 +74,10 @@ def build(family: str, size: str, layers: int | None = None):
         from ferrotorch_b200.models.tenalorn import TenalornForCausalLM
 
         return TenalornForCausalLM(tenalorn_config(size, n), device="cuda").random_()
+    if family == "mogelix":
+        from ferrotorch_b200.models.mogelix import MogelixForCausalLM
+
+        return MogelixForCausalLM(mogelix_config(size, n), device="cuda").random_()
     from ferrotorch_b200.models.llama import LlamaConfig, LlamaForCausalLM
 
     cfg = LlamaConfig(vocab_size=vocab, hidden_size=hidden, intermediate_size=ff, num_hidden_layers=n, num_attention_heads=heads,
@@ -152,7 +167,7 @@ def kernel_table(size: str, peaks: dict, steps: int, families=FAMILIES) -> list:
 
     lib = _native.kernels()
     for family in families:
-        model = build(family, size, layers={"zolorax": 6, "tenalorn": 3}.get(family, 2))
+        model = build(family, size, layers={"zolorax": 6, "tenalorn": 3, "mogelix": 6}.get(family, 2))
         cache = model.make_paged_cache(batch * ((prompt + 16) // PAGE + 1), PAGE, batch, prompt + 16)
         for s in range(batch):
             cache.reserve(s, prompt + 1)
@@ -174,6 +189,8 @@ def kernel_table(size: str, peaks: dict, steps: int, families=FAMILIES) -> list:
                 _zolorax_kernels(lambda *a: add(family, phase, *a), gemm, model, cache, b, phase == "prefill", (hidden, heads, kv, dim, prompt, per, batch))
             elif family == "tenalorn":
                 _tenalorn_kernels(lambda *a: add(family, phase, *a), gemm, model, cache, b, phase == "prefill", (hidden, heads, kv, dim, prompt, per, batch))
+            elif family == "mogelix":
+                _mogelix_kernels(lambda *a: add(family, phase, *a), gemm, model, cache, b, phase == "prefill", (hidden, heads, kv, dim, prompt, per, batch))
             elif family == "bopudra":
                 blk, nrm = model.blocks[0], model.norms[0]
                 x, h = F.embedding_dynamic_tanh(b.tokens, model.embed, nrm.alpha, nrm.weight, nrm.bias, out_dtype=torch.bfloat16)
@@ -401,6 +418,80 @@ def _tenalorn_kernels(add, gemm, model, cache, b, prefill: bool, sizes: tuple) -
         gemm("head", h, model.head, lambda: F.linear_f32_out(h, model.head))
         logits = F.linear_f32_out(h, model.head)
         add("soft cap", lambda: D.softcap_(logits, 30.0), 0, 8 * logits.numel())
+
+
+def _mogelix_kernels(add, gemm, model, cache, b, prefill: bool, sizes: tuple) -> None:
+    """The kernels of a state-space and an attention mixer, a dense and a routed feed-forward and the sums with their norms."""
+    from ferrotorch_b200.ops import decoder as D
+    from ferrotorch_b200.ops import functional as F
+
+    hidden, heads, kv, dim, prompt, per, batch = sizes
+    T, dt, c = b.n_rows, torch.bfloat16, model.config
+    first, att, routed = model.layers[0], model.layers[1], model.layers[1].mlp
+    add("embedding", lambda: F.embedding(b.tokens, model.embed), 0, T * hidden * 4)
+    h = F.embedding(b.tokens, model.embed)
+    # state-space mixer
+    m, w, st = first.mixer, first.mixer.spec, cache.states[0]
+    C, inner = w.channels, w.padded_inner
+    packed, step = F.linear_rows(h, m.in_proj, m.in_bias), D.few_outputs(h, m.step_proj)
+    gemm("state-space in_proj (x|B|C|z|gate) + bias", h, m.in_proj, lambda: F.linear_rows(h, m.in_proj, m.in_bias))
+    add("step sizes' product (fp32 out)", lambda: D.few_outputs(h, m.step_proj), 0, 2 * T * hidden)
+    xbc, z = packed[:, :C], packed[:, C:m.gate_at]
+    add("causal conv + silu", lambda: D.causal_conv(xbc, m.conv_weight, m.conv_bias, st.conv, b, silu=True), 0, 4 * T * C)
+    u = D.causal_conv(xbc, m.conv_weight, m.conv_bias, st.conv, b, silu=True)
+    y = torch.empty((T, inner), device="cuda", dtype=dt)
+    args = (u, z, step, m.step_bias, m.rate, m.skip, st.S, b, y)
+    flops = T * w.heads * (2 * 64 * (w.state + w.vdim) + 4 * w.state * w.vdim)
+    add("state-space heads" + (" (four passes)" if prefill else " (step)"), lambda: D.state_space(*args, heads=w.heads, groups=w.groups), flops if prefill else 0,
+        2 * T * (3 * inner + 2 * w.groups * w.state) + 4 * T * w.heads + (0 if prefill else 8 * T * w.heads * w.state * w.vdim))
+    add("part norm", lambda: D.part_norm_(y, m.norm, w.norm_groups, m.eps, heads=w.heads, vdim=w.vdim), 0, 4 * T * inner)
+    gemm("state-space out_proj", y, m.out_proj, lambda: F.linear_rows(y, m.out_proj))
+    dense, gate = F.linear_rows(y, m.out_proj), packed[:, m.gate_at:]
+    x = torch.randn((T, hidden), device="cuda")
+    add("sum + gate + norm (mixer)", lambda: D.sum_norm(x, D.SublayerTerms(dense=dense), gate, 3.0, first.norm1.weight, 1e-6, count=hidden, out_dtype=dt), 0, T * hidden * 14)
+    # attention mixer
+    m, s = att.mixer, att.mixer.attn
+    (qo, qn), (ko, kn), (vo, vn), _ = m.segments
+    packed = F.linear_rows(h, m.in_proj, m.in_bias)
+    gemm("attention in_proj (q|k|v|gate) + bias", h, m.in_proj, lambda: F.linear_rows(h, m.in_proj, m.in_bias))
+    add("head norms, rotation, append", lambda: D.qkv_head_finish(
+        packed, cache, 0, b, heads=heads, dim=dim, q_off=qo, k_off=ko, v_off=vo, q_weight=m.q_norm, k_weight=m.k_norm, eps=m.eps,
+        table=cache.rotary_table(s.rotary)), 0, 4 * T * (qn + kn + vn))
+    add("means of blocks", lambda: cache.pool_blocks(0, b), 0, 2 * (T if prefill else batch) * 2 * kv * dim * (1 + 1 / s.pool))
+    q, o = packed[:, qo:qo + qn].unflatten(1, (heads, dim)), torch.empty((T, heads, dim), device="cuda", dtype=dt)
+    seen = sum(min(i + 1, s.window) + max(0, i + 1 - s.window) // s.pool for i in range(prompt))
+    now = min(prompt, s.window) + max(0, prompt - s.window) // s.pool
+    add("attention (window %d, blocks of %d, sink)" % (s.window, s.pool), lambda: cache.attend(0, q, b, s.scale, out=o, window=s.window, sink=m.sink, pool=s.pool),
+        4 * heads * dim * per * seen if prefill else 0, 2 * T * (2 * heads + 2 * kv) * dim if prefill else batch * now * kv * 2 * dim * 2)
+    gemm("attention out_proj", o.flatten(1), m.out_proj, lambda: F.linear_rows(o.flatten(1), m.out_proj))
+    # feed-forwards
+    m = first.mlp
+    n = m.down.shape[1]
+    packed = F.linear_rows(h, m.up, m.bias)
+    gemm("dense up|gate + bias", h, m.up, lambda: F.linear_rows(h, m.up, m.bias))
+    add("poly norm", lambda: D.poly_norm(packed[:, :n], m.act, m.eps, count=n), 0, 4 * T * n)
+    act = D.poly_norm(packed[:, :n], m.act, m.eps, count=n)
+    gemm("dense down", act, m.down, lambda: F.linear_rows(act, m.down))
+    m, e = routed, routed.spec
+    kw = dict(score=e.score, normalize=e.normalize, bias=m.router_bias, gate=True)
+    r = D.moe_route(h, m.router, e.experts, e.top, **kw)
+    add("routing (logits, choice, sort, gather)", lambda: D.moe_route(h, m.router, e.experts, e.top, **kw), 2 * T * hidden * e.experts, 2 * T * hidden * (1 + e.top))
+    act = D.grouped_linear(r.sorted, m.gate_up, r, seg_rows=T, activation="relu2")
+    yt = D.grouped_linear(act, m.down, r, seg_rows=T)
+    n_act = T * e.top
+    add("experts up + squared relu", lambda: D.grouped_linear(r.sorted, m.gate_up, r, seg_rows=T, activation="relu2"), 2 * n_act * hidden * e.ff,
+        2 * (m.gate_up.numel() + n_act * (hidden + e.ff)))
+    add("experts down", lambda: D.grouped_linear(act, m.down, r, seg_rows=T), 2 * n_act * hidden * e.ff, 2 * (m.down.numel() + n_act * (hidden + e.ff)))
+    up = m.shared_gate_up[0, 0]
+    sact = F.linear_rows(h, up, activation="relu2")
+    gemm("shared expert up + squared relu", h, up, lambda: F.linear_rows(h, up, activation="relu2"))
+    gemm("shared expert down", sact, m.shared_down, lambda: F.linear_rows(sact, m.shared_down))
+    gemm("residual gate + bias", h, m.residual_proj, lambda: F.linear_rows(h, m.residual_proj, m.residual_bias))
+    terms = D.SublayerTerms(yt, r.place, r.weight, F.linear_rows(sact, m.shared_down), dense_weight=r.gate)
+    gate = F.linear_rows(h, m.residual_proj, m.residual_bias)
+    add("sum + gate + norm (experts' terms)", lambda: D.sum_norm(x, terms, gate, 3.0, att.norm2.weight, 1e-6, count=hidden, out_dtype=dt), 0, T * hidden * (14 + 2 * e.top))
+    if not prefill:
+        gemm("head", h, model.head, lambda: F.linear_f32_out(h, model.head))
 
 
 def run(args, sampler_cls) -> dict:

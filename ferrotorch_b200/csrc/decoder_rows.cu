@@ -115,8 +115,6 @@ rms_rows_kernel(const RmsRowsParams p) {
 }
 
 // ---------------------------------------------------------------- norm after the sum
-constexpr int SN_TERMS = 4;   // terms whose places and weights a thread keeps in registers
-
 struct SumNormParams {
   const void* x;            // [n_src, ldx]
   const long long* ids;     // token i has x[ids[i]] (null: x[i])
@@ -150,7 +148,7 @@ __device__ __forceinline__ float block_total(float v, float* red) {
 
 // One block per row.
 template <typename TI, typename TO>
-__global__ void __launch_bounds__(ROW_THREADS)
+__global__ void __launch_bounds__(ROW_THREADS, 4)
 sum_norm_rows_kernel(const SumNormParams p) {
   __shared__ float red[ROW_WARPS];
   for (int row = blockIdx.x; row < p.n_rows; row += gridDim.x) {
@@ -170,22 +168,8 @@ sum_norm_rows_kernel(const SumNormParams p) {
     const float dw = p.dense_weight ? p.dense_weight[token] : 1.f;
     const int* where = p.where + token * p.n_terms;
     const float* weight = p.weight ? p.weight + token * p.n_terms : nullptr;
-    int at[SN_TERMS];
-    float tw[SN_TERMS];
-#pragma unroll
-    for (int j = 0; j < SN_TERMS; ++j) {
-      at[j] = j < p.n_terms ? where[j] : -1;
-      tw[j] = weight && j < p.n_terms ? weight[j] : 1.f;
-    }
     float* xo = p.x_out ? p.x_out + static_cast<long long>(row) * p.ldo : nullptr;
     TO* hr = p.h ? static_cast<TO*>(p.h) + static_cast<long long>(row) * p.ldh : nullptr;
-    auto add_term = [&](int t, float wt, int i, float (&y)[8]) {
-      if (t < 0 || t >= p.term_rows) return;
-      float g[8];
-      load8(static_cast<const TO*>(p.terms) + static_cast<long long>(t) * p.ldt + i, g);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) y[e] += wt * g[e];
-    };
     auto fetch = [&](int i, float (&f)[8]) {
       float y[8], g[8];
       load8(xr + i, f);
@@ -197,9 +181,15 @@ sum_norm_rows_kernel(const SumNormParams p) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) y[e] *= dw;
       }
+      for (int j = 0; j < p.n_terms; ++j) {
+        const int t = where[j];
+        const float wt = weight ? weight[j] : 1.f;
+        if (t < 0 || t >= p.term_rows) continue;
+        float z[8];
+        load8(static_cast<const TO*>(p.terms) + static_cast<long long>(t) * p.ldt + i, z);
 #pragma unroll
-      for (int j = 0; j < SN_TERMS; ++j) add_term(at[j], tw[j], i, y);
-      for (int j = SN_TERMS; j < p.n_terms; ++j) add_term(where[j], weight ? weight[j] : 1.f, i, y);
+        for (int e = 0; e < 8; ++e) y[e] += wt * z[e];
+      }
       if (gr) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) y[e] *= sigmoid_row(g[e], static_cast<const TO*>(nullptr));
@@ -364,17 +354,6 @@ part_norm_any_kernel(T* __restrict__ y, long long ld, const float* __restrict__ 
       yr[c] = static_cast<T>(static_cast<float>(yr[c]) * r * w[c]);
     }
   }
-}
-
-__device__ __forceinline__ void raw_load(const __nv_bfloat16* p, uint4 (&v)[1]) { v[0] = *reinterpret_cast<const uint4*>(p); }
-__device__ __forceinline__ void raw_load(const float* p, uint4 (&v)[2]) {
-  v[0] = reinterpret_cast<const uint4*>(p)[0];
-  v[1] = reinterpret_cast<const uint4*>(p)[1];
-}
-__device__ __forceinline__ void raw_unpack(const uint4 (&v)[1], float (&f)[8]) { unpack8(v[0], f); }
-__device__ __forceinline__ void raw_unpack(const uint4 (&v)[2], float (&f)[8]) {
-  f[0] = __uint_as_float(v[0].x); f[1] = __uint_as_float(v[0].y); f[2] = __uint_as_float(v[0].z); f[3] = __uint_as_float(v[0].w);
-  f[4] = __uint_as_float(v[1].x); f[5] = __uint_as_float(v[1].y); f[6] = __uint_as_float(v[1].z); f[7] = __uint_as_float(v[1].w);
 }
 
 // out = a z / rms(z) + b z^2 / rms(z^2) + c z^3 / rms(z^3) + e over rows of N elements of which `count` exist (the others are

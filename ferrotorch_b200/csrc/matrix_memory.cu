@@ -85,7 +85,8 @@ __device__ __forceinline__ float state_decay(float rate, float dt) { return 1.f 
 // ---------------------------------------------------------------- token by token
 // One block per (item, head).  Thread (r, c): rows r, r + groups, .. of the state and columns 4 c .. 4 c + 3 of each run of
 // 4 * lanes columns.  Items are portions (spans) or, with spans null, single rows.  The state of a longer portion is kept
-// in shared memory when it fits.
+// in shared memory when it fits; with KEEP > 0 a single row's state is asked for ahead of everything else and stays in
+// registers, KEEP rows a thread.
 constexpr int MS_THREADS = 256;
 
 struct MemoryItems {
@@ -95,8 +96,8 @@ struct MemoryItems {
   int in_smem;
 };
 
-template <typename T, int RULE>
-__global__ void __launch_bounds__(MS_THREADS)
+template <typename T, int RULE, int KEEP>
+__global__ void __launch_bounds__(MS_THREADS, KEEP == 8 ? 3 : KEEP == 16 ? 2 : 1)
 memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
   extern __shared__ float ms_sm[];
   const int lanes = min(p.vp / 4, MS_THREADS), groups = MS_THREADS / lanes;
@@ -121,6 +122,15 @@ memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
   float* S = it.in_smem ? s_state : S_mem;
   const long long qk = static_cast<long long>(h / p.group) * p.dp;
   bool fresh = pos0 == 0;
+  float4 kept[KEEP > 0 ? KEEP : 1];
+  if constexpr (KEEP > 0) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int d = r + i * groups;
+      kept[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < groups && d < p.dp && !fresh) kept[i] = *reinterpret_cast<const float4*>(S_mem + static_cast<long long>(d) * p.vp + c * 4);
+    }
+  }
   float m = 0.f;
   if constexpr (RULE == MEMORY) {
     m = fresh ? 0.f : p.m[sh];
@@ -162,7 +172,24 @@ memory_steps_kernel(const MemoryParams p, const MemoryItems it) {
       dot = warp_sum(dot);
       if (lane == 0) s_red[warp] = dot;
     }
-    if (r < groups)
+    if constexpr (KEEP > 0) {
+      if (r < groups) {
+        const float4 v4 = *reinterpret_cast<const float4*>(s_v + c * 4);
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i) {
+          const int d = r + i * groups;
+          if (d >= p.dp) continue;
+          const float kd = add * s_k[d], qd = s_q[d];
+          float4 s = kept[i];
+          s.x = keep * s.x + kd * v4.x; s.y = keep * s.y + kd * v4.y;
+          s.z = keep * s.z + kd * v4.z; s.w = keep * s.w + kd * v4.w;
+          *reinterpret_cast<float4*>(S_mem + static_cast<long long>(d) * p.vp + c * 4) = s;
+          acc.x += s.x * qd; acc.y += s.y * qd; acc.z += s.z * qd; acc.w += s.w * qd;
+        }
+        *reinterpret_cast<float4*>(s_part + r * p.vp + c * 4) = acc;
+      }
+    } else if (r < groups)
       for (int j = c * 4; j < p.vp; j += lanes * 4) {
         const float4 v4 = *reinterpret_cast<const float4*>(s_v + j);
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -381,12 +408,20 @@ __device__ __forceinline__ uint32_t mc_unit(int row, int unit) {
   return static_cast<uint32_t>(unit >> 3) * MC_CHUNK + static_cast<uint32_t>(row) * 128u + (static_cast<uint32_t>((unit & 7) ^ (row & 7)) << 4);
 }
 
-// U of one (chunk, head).  The keys' tile [128 tokens, 128] is weighted in place (its low halves go to a second tile) and
-// multiplied as the transposed A operand with V.
+// U of one (chunk, head).  MEMORY: the keys' tile [128 tokens, 128] is weighted in place (its low halves go to a second tile) and
+// multiplied as the transposed A operand with V; their weighted sum is the normaliser's contribution.  STATE_SPACE: V, which is
+// narrower, is weighted instead.
+template <int VC, int RULE>
+struct MemUpdate {       // shared memory: K | low halves of what is weighted | V
+  static constexpr int LO = RULE == MEMORY ? 2 : VC, OFF_LO = 2 * MC_CHUNK, OFF_V = OFF_LO + LO * MC_CHUNK, OFF_N = OFF_V + VC * MC_CHUNK,
+                       OFF_W = OFF_N + (RULE == MEMORY ? 16 * 128 * 4 : 0), OFF_BAR = OFF_W + MC_ROWS * 4, SMEM = OFF_BAR + 64 + 1024;
+};
+
 template <int VC, int RULE>
 __global__ void __launch_bounds__(MC_UPDATE_THREADS)
 memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const MemoryParams p, const MemoryChunks c) {
-  constexpr int OFF_LO = 2 * MC_CHUNK, OFF_V = 4 * MC_CHUNK, OFF_N = OFF_V + VC * MC_CHUNK, OFF_W = OFF_N + 16 * 128 * 4, OFF_BAR = OFF_W + MC_ROWS * 4;
+  using Cfg = MemUpdate<VC, RULE>;
+  constexpr int OFF_LO = Cfg::OFF_LO, OFF_V = Cfg::OFF_V, OFF_N = Cfg::OFF_N, OFF_W = Cfg::OFF_W, OFF_BAR = Cfg::OFF_BAR;
   constexpr uint32_t COLS = VC == 1 ? 64 : (VC == 2 ? 128 : 256);
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -424,16 +459,18 @@ memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
     mbar_expect_tx(bar_v, VC * MC_CHUNK);
     for (int i = 0; i < VC; ++i) tma_load_2d(sbase + OFF_V + i * MC_CHUNK, &tmV, bar_v, h * p.vp + i * 64, row0);
   }
-  bool ok = mbar_wait(bar_k, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE);
+  bool ok = mbar_wait(RULE == MEMORY ? bar_k : bar_v, 0, abort_word, FT_ERR_TIMEOUT_EPILOGUE);
   if (ok) {
-    const int unit = tid & 15, r0 = tid >> 4;
+    constexpr int UNITS = RULE == MEMORY ? 16 : 8 * VC, STEP = MC_UPDATE_THREADS / UNITS, OFF_IN = RULE == MEMORY ? 0 : OFF_V;
+    const int unit = tid % UNITS, r0 = tid / UNITS;
     float acc[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) acc[e] = 0.f;
 #pragma unroll
-    for (int i = 0; i < MC_ROWS / 16; ++i) {
-      const int row = r0 + 16 * i;
-      uint4* at = reinterpret_cast<uint4*>(smem + mc_unit(row, unit));
+    for (int i = 0; i < (MC_ROWS + STEP - 1) / STEP; ++i) {
+      const int row = r0 + STEP * i;
+      if (r0 >= STEP || row >= MC_ROWS) continue;
+      uint4* at = reinterpret_cast<uint4*>(smem + OFF_IN + mc_unit(row, unit));
       const float w = s_w[row];
       float f[8], hi[8];
       unpack8(*at, f);
@@ -456,14 +493,16 @@ memory_update_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
   }
   fence_proxy_async_smem();
   __syncthreads();
-  if (tid == 0 && ok && mbar_wait(bar_v, 0, abort_word, FT_ERR_TIMEOUT_MMA)) {
+  if (tid == 0 && ok && mbar_wait(RULE == MEMORY ? bar_v : bar_k, 0, abort_word, FT_ERR_TIMEOUT_MMA)) {
+    constexpr int OFF_A = RULE == MEMORY ? OFF_LO : 0, OFF_B = RULE == MEMORY ? 0 : OFF_LO - OFF_V;      // from the high to the low halves
+    if (RULE == STATE_SPACE) tc_fence_after();
     constexpr uint32_t idesc = make_idesc_f16(128, VC * 64, 1, 1, 1);
 #pragma unroll
     for (int half = 0; half < 2; ++half)
 #pragma unroll
       for (int kk = 0; kk < MC_ROWS / 16; ++kk)
-        umma_f16_ss(tmem, make_smem_desc_sw128(sbase + half * OFF_LO + kk * 2048, MC_CHUNK, 1024),
-                    make_smem_desc_sw128(sbase + OFF_V + kk * 2048, MC_CHUNK, 1024), idesc, (half > 0 || kk > 0) ? 1u : 0u);
+        umma_f16_ss(tmem, make_smem_desc_sw128(sbase + half * OFF_A + kk * 2048, MC_CHUNK, 1024),
+                    make_smem_desc_sw128(sbase + OFF_V + half * OFF_B + kk * 2048, MC_CHUNK, 1024), idesc, (half > 0 || kk > 0) ? 1u : 0u);
     umma_commit(bar_m);
   }
   if (RULE == MEMORY && tid < p.dp && ok) {
@@ -563,10 +602,14 @@ memory_carry_kernel(const MemoryParams p, const MemoryChunks c) {
 
 // Outputs of one (chunk, head).  Warps 0-3: thread = token.  Warp 4: copies and products.  Shared memory: Q | K, then the low half
 // of the state | the high half of the state, then V; at the end the gate lies over Q (and what follows), and the results over it.
-template <int DC, int VC>
+// With APART the state's high half has a place of its own, so that V is loaded at once, and the gate as soon as that half has been
+// read, to whose place it and then the results go.
+template <int DC, int VC, int RULE>
 struct MemOut {
   static constexpr int MID = DC > VC ? DC : VC;
-  static constexpr int OFF_K = DC * MC_CHUNK, OFF_V = OFF_K + MID * MC_CHUNK, OFF_A = OFF_V + VC * MC_CHUNK, OFF_NB = OFF_A + MC_ROWS * 4,
+  static constexpr bool APART = RULE == STATE_SPACE && VC <= 2;
+  static constexpr int OFF_K = DC * MC_CHUNK, OFF_V = OFF_K + MID * MC_CHUNK, OFF_H = APART ? OFF_V + VC * MC_CHUNK : OFF_V,
+                       OFF_G = APART ? OFF_H : 0, OFF_A = OFF_H + VC * MC_CHUNK, OFF_NB = OFF_A + MC_ROWS * 4,
                        OFF_W = OFF_NB + 128 * 4, OFF_BAR = OFF_W + VC * 64 * 4, SMEM = OFF_BAR + 128 + 1024;
   static constexpr uint32_t COLS = VC <= 2 ? 256 : 512, COL_LOW = 64, COL_O = 128;      // scores (then P high | low), outputs
 };
@@ -576,10 +619,11 @@ __global__ void __launch_bounds__(MC_OUT_THREADS)
 memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                      const __grid_constant__ CUtensorMap tmS, const __grid_constant__ CUtensorMap tmG, const MemoryParams p,
                      const MemoryChunks c) {
-  using Cfg = MemOut<DC, VC>;
+  using Cfg = MemOut<DC, VC, RULE>;
+  constexpr bool APART = Cfg::APART;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-  const uint32_t sQ = smem_u32(smem), sK = sQ + Cfg::OFF_K, sV = sQ + Cfg::OFF_V;
+  const uint32_t sQ = smem_u32(smem), sK = sQ + Cfg::OFF_K, sV = sQ + Cfg::OFF_V, sH = sQ + Cfg::OFF_H;
   float* s_a = reinterpret_cast<float*>(smem + Cfg::OFF_A);
   float* s_nb = reinterpret_cast<float*>(smem + Cfg::OFF_NB);
   float* s_w = reinterpret_cast<float*>(smem + Cfg::OFF_W);
@@ -632,8 +676,13 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         tma_load_2d(sQ + i * MC_CHUNK, &tmQ, bar(QK), h / p.group * p.dp + i * 64, row0);
         tma_load_2d(sK + i * MC_CHUNK, &tmK, bar(QK), h / p.group * p.dp + i * 64, row0);
       }
-      if (fresh) load_v();
-      else load_state(HIGH, sV, ph * p.dp);
+      auto load_gate = [&]() {
+        mbar_expect_tx(bar(GATE), VC * MC_CHUNK);
+        for (int i = 0; i < VC; ++i) tma_load_2d(sQ + Cfg::OFF_G + i * MC_CHUNK, &tmG, bar(GATE), h * p.vp + i * 64, row0);
+      };
+      if (!fresh) load_state(HIGH, sH, ph * p.dp);
+      if (fresh || APART) load_v();
+      if (fresh && APART && p.gate) load_gate();
       bool ok = wait(QK);
       if (ok) {
         tc_fence_after();
@@ -646,11 +695,14 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       if (!fresh) {
         if (ok && (ok = wait(HIGH))) {
           tc_fence_after();
-          q_state(sV, true);
+          q_state(sH, true);
           umma_commit(bar(HIGH_DONE));
         }
         if (ok && (ok = wait(SCORE))) load_state(LOW, sK, (static_cast<long long>(c.n_chunks) * p.H + ph) * p.dp);    // K has been read
-        if (ok && (ok = wait(HIGH_DONE))) load_v();
+        if (ok && (ok = wait(HIGH_DONE))) {
+          if (!APART) load_v();
+          else if (p.gate) load_gate();
+        }
         if (ok && (ok = wait(LOW))) {
           tc_fence_after();
           q_state(sK, false);
@@ -658,10 +710,7 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         }
       }
       // the last product with Q has finished and every token has read its own: the gate takes the place
-      if (ok && p.gate && (ok = wait(fresh ? SCORE : INTER)) && (ok = wait(Q_READ))) {
-        mbar_expect_tx(bar(GATE), VC * MC_CHUNK);
-        for (int i = 0; i < VC; ++i) tma_load_2d(sQ + i * MC_CHUNK, &tmG, bar(GATE), h * p.vp + i * 64, row0);
-      }
+      if (!APART && ok && p.gate && (ok = wait(fresh ? SCORE : INTER)) && (ok = wait(Q_READ))) load_gate();
       if (ok && (ok = wait(V)) && (ok = wait(P_FULL))) {
         tc_fence_after();
 #pragma unroll
@@ -789,7 +838,7 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         tmem_ld_wait();
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
-          uint4* at = reinterpret_cast<uint4*>(smem + mc_unit(tid, col / 8 + g));
+          uint4* at = reinterpret_cast<uint4*>(smem + Cfg::OFF_G + mc_unit(tid, col / 8 + g));
           float f[8], z[8];
 #pragma unroll
           for (int e = 0; e < 8; ++e) f[e] = RULE == MEMORY ? __uint_as_float(t[g * 8 + e]) * r * s_w[col + g * 8 + e] : __uint_as_float(t[g * 8 + e]);
@@ -812,7 +861,7 @@ memory_output_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (static_cast<long long>(row0) + warp * 32) * p.ldo + static_cast<long long>(h) * p.vp;
       for (int i = lane; ok && i < live; i += 32) {
         const int rr = i / units, u = i - rr * units;
-        *reinterpret_cast<uint4*>(out + rr * p.ldo + u * 8) = *reinterpret_cast<const uint4*>(smem + mc_unit(warp * 32 + rr, u));
+        *reinterpret_cast<uint4*>(out + rr * p.ldo + u * 8) = *reinterpret_cast<const uint4*>(smem + Cfg::OFF_G + mc_unit(warp * 32 + rr, u));
       }
     }
   }
@@ -875,7 +924,10 @@ static int run_steps(const MemoryParams& p, const int* spans, const int* pos, co
   }
   FT_REQUIRE(smem <= 200 * 1024, "matrix memory: heads of %d x %d are too large", p.dp, p.vp);
   const dim3 grid(n_items, p.H);
-  auto kern = f32 ? memory_steps_kernel<float, RULE> : memory_steps_kernel<__nv_bfloat16, RULE>;
+  const int per_thread = !spans && p.vp <= 4 * MS_THREADS ? (p.dp + groups - 1) / groups : 1 << 30;     // rows of the state
+  auto kern = f32 ? memory_steps_kernel<float, RULE, 0> : memory_steps_kernel<__nv_bfloat16, RULE, 0>;
+  if (!f32 && per_thread <= 8) kern = memory_steps_kernel<__nv_bfloat16, RULE, 8>;
+  else if (!f32 && per_thread <= 16) kern = memory_steps_kernel<__nv_bfloat16, RULE, 16>;
   FT_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   kern<<<grid, MS_THREADS, smem, stream>>>(p, it);
   FT_CUDA_CHECK(cudaGetLastError());
@@ -934,8 +986,8 @@ FT_API long long ft_memory_scratch(int rows, int H, int dp, int vp, int n_chunks
 template <int DC, int VC, int RULE>
 static int launch_memory(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const CUtensorMap& tg,
                          const MemoryParams& p, const MemoryChunks& c, int device, cudaStream_t stream) {
-  constexpr int UPDATE_SMEM = (4 + VC) * MC_CHUNK + 16 * 128 * 4 + MC_ROWS * 4 + 64 + 1024;
-  constexpr int OUT_SMEM = MemOut<DC, VC>::SMEM;
+  constexpr int UPDATE_SMEM = MemUpdate<VC, RULE>::SMEM;
+  constexpr int OUT_SMEM = MemOut<DC, VC, RULE>::SMEM;
   auto update = memory_update_kernel<VC, RULE>;
   auto output = memory_output_kernel<DC, VC, RULE>;
   static bool attr_set[64] = {false};

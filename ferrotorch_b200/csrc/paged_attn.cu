@@ -55,18 +55,22 @@ __global__ void kv_append_kernel(const uint4* __restrict__ k_new, const uint4* _
 }
 
 // Row i ends a block when (pos[i] + 1) % pool == 0: the means of its pool keys and values (their rows are in the cache) go to the
-// block's place.  A thread owns eight elements of a token's keys or values.
+// block's place.  A thread owns eight elements of a token's keys or values; a CTA takes `walk` (up to 32) consecutive rows, of
+// which a portion has few that end a block.
 constexpr int PB_THREADS = 128;
+constexpr int PB_BATCH = 8;       // rows loaded together
 template <typename T>
 __global__ void __launch_bounds__(PB_THREADS)
 pool_blocks_kernel(const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ k_pool, T* __restrict__ v_pool,
-                   const int* __restrict__ block_table, const int* __restrict__ pos, const int* __restrict__ slots, int rows, int kw, int vw,
+                   const int* __restrict__ block_table, const int* __restrict__ pos, const int* __restrict__ slots, int rows, int walk, int kw, int vw,
                    int pool, int per_page, int block_size, int max_blocks, int num_blocks) {
   const float inv = 1.f / static_cast<float>(pool);
-  for (int row = blockIdx.x; row < rows; row += gridDim.x) {
-    const int last = pos[row];
-    if ((last + 1) % pool != 0) continue;
-    const int* bt = block_table + static_cast<long long>(slots[row]) * max_blocks;
+  const int lane = threadIdx.x & 31, mine = blockIdx.x * walk + lane;
+  const bool there = lane < walk && mine < rows;
+  const int my_pos = there ? pos[mine] : 0, my_slot = there ? slots[mine] : 0;
+  for (unsigned ends = __ballot_sync(0xffffffffu, there && (my_pos + 1) % pool == 0); ends; ends &= ends - 1) {
+    const int at = __ffs(ends) - 1, last = __shfl_sync(0xffffffffu, my_pos, at);
+    const int* bt = block_table + static_cast<long long>(__shfl_sync(0xffffffffu, my_slot, at)) * max_blocks;
     const int page = last / block_size, first = last + 1 - pool;
     if (page >= max_blocks || bt[page] < 0 || bt[page] >= num_blocks) continue;   // a row of no sequence
     const long long dst = static_cast<long long>(bt[page]) * per_page + (last / pool - page * block_size / pool);
@@ -77,14 +81,22 @@ pool_blocks_kernel(const T* __restrict__ k_cache, const T* __restrict__ v_cache,
       float sum[8];
 #pragma unroll
       for (int e = 0; e < 8; ++e) sum[e] = 0.f;
-#pragma unroll 8
-      for (int j = 0; j < pool; ++j) {
-        const int p = first + j;
-        const int blk = min(max(__ldg(bt + p / block_size), 0), num_blocks - 1);
-        float f[8];
-        load8(src + (static_cast<long long>(blk) * block_size + p % block_size) * width + c, f);
+      for (int j0 = 0; j0 < pool; j0 += PB_BATCH) {
+        uint4 raw[PB_BATCH][sizeof(T) / 2];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) sum[e] += f[e];
+        for (int j = 0; j < PB_BATCH; ++j) {            // past the end: the last row again
+          const int p = first + min(j0 + j, pool - 1);
+          const int blk = min(max(__ldg(bt + p / block_size), 0), num_blocks - 1);
+          raw_load(src + (static_cast<long long>(blk) * block_size + p % block_size) * width + c, raw[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < PB_BATCH; ++j) {
+          if (j0 + j >= pool) continue;
+          float f[8];
+          raw_unpack(raw[j], f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) sum[e] += f[e];
+        }
       }
 #pragma unroll
       for (int e = 0; e < 8; ++e) sum[e] *= inv;
@@ -822,12 +834,15 @@ FT_API int ft_pool_blocks(const void* k_cache, const void* v_cache, void* k_pool
   FT_REQUIRE(((reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(k_pool) |
                reinterpret_cast<uintptr_t>(v_pool)) & 15) == 0, "ft_pool_blocks: pointers must be 16-byte aligned");
   if (rows <= 0) return FT_E_OK;
-  const int kw = Hkv * D, vw = Hkv * Dv, per_page = (block_size - 1) / pool + 1, cap = sm_count(device) * 16;
+  const int kw = Hkv * D, vw = Hkv * Dv, per_page = (block_size - 1) / pool + 1;
   const int parts = (kw + vw + PB_THREADS * 8 - 1) / (PB_THREADS * 8);
-  const dim3 grid(rows < cap ? rows : cap, parts);
+  // enough CTAs for the GPU at once, up to a warp's worth of rows each
+  int walk = rows / (sm_count(device) * 3);
+  walk = walk < 1 ? 1 : (walk > 32 ? 32 : walk);
+  const dim3 grid((rows + walk - 1) / walk, parts);
 #define FT_PB(T) \
   pool_blocks_kernel<T><<<grid, PB_THREADS, 0, stream>>>(static_cast<const T*>(k_cache), static_cast<const T*>(v_cache), static_cast<T*>(k_pool), \
-      static_cast<T*>(v_pool), block_table, pos, slots, rows, kw, vw, pool, per_page, block_size, max_blocks, num_blocks)
+      static_cast<T*>(v_pool), block_table, pos, slots, rows, walk, kw, vw, pool, per_page, block_size, max_blocks, num_blocks)
   if (f32) FT_PB(float); else FT_PB(__nv_bfloat16);
 #undef FT_PB
   FT_CUDA_CHECK(cudaGetLastError());

@@ -29,6 +29,18 @@ __device__ __forceinline__ void store8(float* p, const float* f) {
   reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
 }
 
+// Eight elements as they lie in memory, for loads that are to be in flight together.
+__device__ __forceinline__ void raw_load(const __nv_bfloat16* p, uint4 (&v)[1]) { v[0] = *reinterpret_cast<const uint4*>(p); }
+__device__ __forceinline__ void raw_load(const float* p, uint4 (&v)[2]) {
+  v[0] = reinterpret_cast<const uint4*>(p)[0];
+  v[1] = reinterpret_cast<const uint4*>(p)[1];
+}
+__device__ __forceinline__ void raw_unpack(const uint4 (&v)[1], float (&f)[8]) { unpack8(v[0], f); }
+__device__ __forceinline__ void raw_unpack(const uint4 (&v)[2], float (&f)[8]) {
+  f[0] = __uint_as_float(v[0].x); f[1] = __uint_as_float(v[0].y); f[2] = __uint_as_float(v[0].z); f[3] = __uint_as_float(v[0].w);
+  f[4] = __uint_as_float(v[1].x); f[5] = __uint_as_float(v[1].y); f[6] = __uint_as_float(v[1].z); f[7] = __uint_as_float(v[1].w);
+}
+
 // Eight fp32 as one 32-byte store (a whole sector): for lanes that each hold a row.  p 32-byte aligned.
 __device__ __forceinline__ void store8_sector(float* p, const float* f) {
   asm volatile("st.global.v8.f32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "f"(f[0]), "f"(f[1]), "f"(f[2]), "f"(f[3]), "f"(f[4]),

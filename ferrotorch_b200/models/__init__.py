@@ -1,5 +1,5 @@
-"""Model families: Llama (single-GPU, tensor-parallel training, inference engine), Bopudra, Zolorax, ResNet, and the
-small zoo (BERT, Whisper encoder, GCN, PPO policy) and the latent-diffusion stack (``diffusion``)."""
+"""Model families: Llama (single-GPU, tensor-parallel training, inference engine), Bopudra, Zolorax, Tenalorn, Mogelix,
+ResNet, and the small zoo (BERT, Whisper encoder, GCN, PPO policy) and the latent-diffusion stack (``diffusion``)."""
 from .llama import LlamaConfig, LlamaForCausalLM, LlamaModel  # noqa: F401
 from .llama_compat import (AwqQ4, GptqQ4, HqqQ4Axis1, LlamaActivation, LlamaAttention, LlamaGpuLayer, LlamaMLP,  # noqa: F401
                            LayerKvCache, LlamaKvCache, apply_grammar_mask_gpu, gguf_key_to_hf, gguf_to_hf_state_dict,
@@ -32,6 +32,14 @@ def __getattr__(name):
         from . import zolorax
 
         return getattr(zolorax, name)
+    if name in ("TenalornConfig", "TenalornForCausalLM"):
+        from . import tenalorn
+
+        return getattr(tenalorn, name)
+    if name in ("MogelixConfig", "MogelixForCausalLM"):
+        from . import mogelix
+
+        return getattr(mogelix, name)
     if name in ("load_causal_lm", "register_causal_lm", "list_causal_lms"):
         from . import registry
 

@@ -15,9 +15,9 @@ from .extra import (HookedModule, HookHandle, LoRALinear, SqueezeExcitation, fla
                     standard_attention)
 from ..core import BlockMask, flex_attention  # noqa: F401,E402
 from .paged import OutOfPages, PagedAttentionManager, PagedKVCache, PagedSession, RaggedBatch  # noqa: F401,E402
-from .packed_block import AttentionSpec, DynamicTanh, PackedParallelBlock, RotarySpec, YarnScaling  # noqa: F401,E402
+from .packed_block import AttentionSpec, DynamicTanh, PackedParallelBlock, RotarySpec, WavelengthScaling, YarnScaling  # noqa: F401,E402
 from .gated_attention import GatedAttention, ResidualRMSNorm  # noqa: F401,E402
-from .recurrent import RGLRUBlock, RGLRUSpec, RGLRUState  # noqa: F401,E402
+from .recurrent import RGLRUBlock, RGLRUSpec, RGLRUState, StateSpaceBlock, StateSpaceSpec, StateSpaceState  # noqa: F401,E402
 from .feed_forward import ExpertSpec, PackedMLP, RoutedExperts  # noqa: F401,E402
 from ..ops.conv import IgemmConv2d, convert_convs  # noqa: F401,E402  (implicit-GEMM convolution; opt-in, see ops.conv)
 from ..ops.pool import MaxPool2d as NhwcMaxPool2d  # noqa: F401,E402

@@ -141,7 +141,7 @@ def test_rotation_by_wavelength():
     assert O.frequencies({"dims": 4, "base": 9.0}).tolist() == pytest.approx([1.0, 1 / 3])
 
 
-@pytest.mark.parametrize("window,pool", [(40, 12), (1, 1), (5, 16), (16, 4), (17, 3), (64, 7), (3, 50), (200, 8), (128, 16)])
+@pytest.mark.parametrize("window,pool", [(41, 11), (1, 1), (5, 16), (16, 4), (17, 3), (64, 7), (3, 50), (200, 8), (128, 16)])
 @pytest.mark.parametrize("Hq,Hkv,D_,Dv", [(4, 2, 32, 16), (3, 1, 48, 40)])
 def test_attention_sees_its_window_and_pooled_blocks(window, pool, Hq, Hkv, D_, Dv):
     check_planted_blocks(Hq, Hkv, D_, Dv, 16 if pool != 3 else 4, torch.float32, "cpu", 130, window, pool)
